@@ -67,6 +67,7 @@ def get_model(
     max_input_tokens: Optional[int] = None,
     device: Optional[torch.device] = None,
     max_prefill_tokens: Optional[int] = None,
+    max_positions: Optional[int] = None,
 ):
     """Load the shard of ``model_id`` (a local directory) that belongs to this process."""
     from .flash_causal_lm import FlashCausalLM
@@ -115,8 +116,10 @@ def get_model(
 
         return load_padded(path, cfg, process_group, rank, world, tdtype, device, tokenizer)
     text_cfg = cfg.text_config()
+    if ARCHS[model_type].mix:
+        _check_mixed(model_type, tdtype, device, quantize, kv_cache_dtype)
     weights = Weights(weight_files(path), device, tdtype, process_group=process_group, loader=loader,
-                      aliases=_aliases(model_type))
+                      aliases=_aliases(model_type), bare_names=ARCHS[model_type].bare_names)
     prefix = ""
     if model_type in ("gpt2",) and weights.has_tensor("transformer.wte.weight"):
         prefix = "transformer"
@@ -127,7 +130,7 @@ def get_model(
     hidden = int(text_cfg.get("hidden_size", text_cfg.get("n_embd", text_cfg.get("d_model", 0))) or 0)
     comm = make_comm(process_group, rank, world, device, hidden, int(max_prefill_tokens or 4096)) if hidden else None
     model = CausalDecoder(text_cfg, weights, comm=comm, prefix=prefix,
-                          max_positions=_max_positions(text_cfg, max_input_tokens))
+                          max_positions=max_positions or _max_positions(text_cfg, max_input_tokens))
     from .speculative import find_speculator, load_speculator
 
     spec_path = find_speculator(path)
@@ -141,6 +144,18 @@ def get_model(
                            eos_token_ids(path, cfg))
     weights.close()
     return runner
+
+
+def _check_mixed(model_type: str, dtype: torch.dtype, device: torch.device, quantize, kv_cache_dtype) -> None:
+    """Decoders with per-layer mixers: the options their kernels have no build for are refused at load."""
+    if quantize is not None:
+        raise NotImplementedError(f"{model_type}: quantisation is not available")
+    if resolve_kv_dtype(kv_cache_dtype, dtype) != dtype:
+        raise NotImplementedError(f"{model_type}: the KV cache is kept in the serving dtype")
+    if dtype not in (torch.bfloat16, torch.float32):
+        raise NotImplementedError(f"{model_type}: serving dtypes are bfloat16 and float32")
+    if dtype == torch.float32:
+        torch.backends.cuda.matmul.allow_tf32 = False        # fp32 products are true fp32
 
 
 def _max_positions(cfg: ModelConfig, max_input_tokens: Optional[int]) -> int:

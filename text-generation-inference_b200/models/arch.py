@@ -16,14 +16,55 @@ import json
 import math
 from dataclasses import dataclass, field, replace
 from pathlib import Path
-from typing import Any, Dict, List, Optional
+from typing import Any, Dict, List, Optional, Tuple
+
+
+def _fuzuvik_config(d: Dict[str, Any]) -> Dict[str, Any]:
+    """Fuzuvik checkpoints describe every layer on its own (``layers``: mixer type, its sizes, its feed-forward) and use
+    their own key names; brought here to the names the rest of the package reads, with the layers as ``MixerSpec``s."""
+    out = dict(d)
+    layers = d["layers"]
+    specs = []
+    for i, layer in enumerate(layers):
+        m, mlp = layer["mixer"], layer.get("mlp")
+        if mlp is not None and mlp["kind"] != "dense":
+            raise NotImplementedError(f"layer {i}: feed-forward kind {mlp['kind']!r}")
+        ff = 0 if mlp is None else int(mlp["ff"])
+        sizes = dict(heads=int(m["heads"]), kv_heads=int(m.get("kv_heads") or m["heads"]), dim=int(m["dim"]),
+                     vdim=int(m["vdim"]), ff=ff)
+        if layer["type"] == "attention":
+            rot = m.get("rot") or {}
+            sc = rot.get("scaling")
+            specs.append(MixerSpec(
+                "attention", **sizes, scale=float(m["scale"]), chunk=int((m.get("mask") or {}).get("size") or 0), sink=True,
+                qk_unit_rms=True, v_mix=bool(m.get("v_mix")), rot_dims=int(rot.get("dims") or 0),
+                rot_base=float(rot.get("base") or 10000.0),
+                rot_scaling=None if not sc else (float(sc["factor"]), float(sc["low"]), float(sc["high"]), float(sc["original"]))))
+        elif layer["type"] == "channel_delta":
+            specs.append(MixerSpec("delta", **sizes))
+        elif layer["type"] == "lightning":
+            specs.append(MixerSpec("decay", **sizes, decay=tuple(float(x) for x in m["decay"])))
+        else:
+            raise NotImplementedError(f"layer {i}: mixer {layer['type']!r}")
+    attn = [s for s in specs if s.kind == "attention"]
+    out.update(model_type="fuzuvik", hidden_size=int(d["width"]), vocab_size=int(d["vocab"]), num_hidden_layers=len(layers),
+               num_attention_heads=max(s.heads for s in (attn or specs)), rms_norm_eps=float(d["norm"]["eps"]),
+               embedding_multiplier=float((d.get("embedding") or {}).get("scale", 1.0)), mixers=specs,
+               # rotary positions are unbounded by design: the table length is a deployment choice
+               max_position_embeddings=int(d.get("max_position_embeddings") or 131072))
+    return out
+
+
+# ``architecture`` of a config.json without ``model_type`` -> function that brings it to the common names
+CONFIG_READERS = {"Fuzuvik": _fuzuvik_config}
 
 
 class ModelConfig:
     """Attribute access to ``config.json`` with ``get``-style defaults; unknown attributes are ``None``."""
 
     def __init__(self, data: Dict[str, Any]):
-        object.__setattr__(self, "_d", dict(data))
+        reader = CONFIG_READERS.get(data.get("architecture")) if "model_type" not in data else None
+        object.__setattr__(self, "_d", reader(data) if reader else dict(data))
 
     @classmethod
     def from_path(cls, path) -> "ModelConfig":
@@ -55,6 +96,33 @@ class ModelConfig:
             merged.setdefault("quantization_config", self._d.get("quantization_config"))
             return ModelConfig(merged)
         return self
+
+
+@dataclass(frozen=True)
+class MixerSpec:
+    """Token mixer and feed-forward width of one layer of a decoder whose layers differ (``models/mixers.py``)."""
+
+    kind: str                                # "attention" | "delta" (gated delta rule) | "decay" (fixed decay per head)
+    heads: int
+    kv_heads: int                            # attention: key/value heads; delta: query/key heads
+    dim: int                                 # query / key size of a head
+    vdim: int                                # value size of a head
+    ff: int = 0                              # feed-forward width, 0: the layer has none
+    # attention
+    scale: float = 1.0
+    chunk: int = 0                           # > 0: keys of the query's own chunk of this many positions
+    sink: bool = False                       # one more key of score 0, without a value, in the softmax
+    qk_unit_rms: bool = False                # q and k over their root mean square, after the rotation
+    v_mix: bool = False                      # values mixed with those of the first such layer
+    rot_dims: int = 0
+    rot_base: float = 10000.0
+    rot_scaling: Optional[Tuple[float, float, float, float]] = None    # (factor, low, high, original length)
+    # decay
+    decay: Tuple[float, ...] = ()
+
+    @property
+    def recurrent(self) -> bool:
+        return self.kind != "attention"
 
 
 @dataclass(frozen=True)
@@ -112,6 +180,10 @@ class Arch:
     mla: bool = False                        # DeepSeek multi-head latent attention (models/deepseek.py)
     moe_shared_gate: Optional[str] = None
     moe_renormalize: bool = True
+    # ---- layers that differ (config "mixers") ---------------------------------------------------
+    mix: Optional[str] = None                # tensor prefix of a layer's mixer
+    residual_fp32: bool = False              # the residual stream is kept in 32 bits
+    bare_names: bool = False                 # tensors are named without the ".weight" suffix
 
 
 _LLAMA = Arch()
@@ -193,6 +265,10 @@ ARCHS["RefinedWeb"] = ARCHS["RefinedWebModel"] = ARCHS["falcon"]
 ARCHS["deepseek_v2"] = ARCHS["deepseek_v3"] = replace(
     _LLAMA, rope_neox=False, mla=True, moe=True, moe_router="mlp.gate", moe_expert="mlp.experts.{e}",
     moe_gate="gate_proj", moe_up="up_proj", moe_down="down_proj", moe_shared="mlp.shared_experts")
+# decoder whose layers mix tokens in different ways; names inside a mixer are in models/mixers.py
+ARCHS["fuzuvik"] = Arch(embed="embed", layer="l{i}", norm1="norm1", norm2="norm2", final_norm="final.norm", lm_head="head",
+                        mix="mix", gate=None, up="mlp.up", down="mlp.down", gated_mlp=False, act="gelu", rope=False,
+                        residual_fp32=True, bare_names=True)
 ARCHS["gemma3"] = ARCHS["gemma3_text"]
 ARCHS["phi-msft"] = ARCHS["phi"]
 ARCHS["qwen2_vl_text"] = ARCHS["qwen2_5_vl_text"] = ARCHS["qwen2"]   # language models of Qwen2-VL / Qwen2.5-VL
@@ -231,6 +307,7 @@ class ModelDims:
     top_k: int = 0
     total_heads: int = 0
     total_kv_heads: int = 0
+    mixers: Optional[List[MixerSpec]] = None    # per layer, for decoders whose layers differ
     attn_head_dim: int = 0      # head dimension seen by the attention kernels and the KV cache: head_dim padded to 64/128/256
 
 
@@ -305,6 +382,12 @@ def derive_dims(cfg: ModelConfig, arch: Arch, world: int) -> ModelDims:
             windows = [window if i >= cfg.max_window_layers else -1 for i in range(layers)]
         else:
             windows = [window] * layers
+    mixers = cfg.get("mixers")
+    if mixers:
+        # sizes are per layer; the scalars below describe the widest attention layer and are informative only
+        if world != 1:
+            raise NotImplementedError(f"{cfg.model_type} is served on one GPU: its mixers are not sharded")
+        head_dim = 64
     ne = cfg.get("num_local_experts", cfg.get("num_experts", cfg.get("n_routed_experts", 0))) or 0
     tk = cfg.get("num_experts_per_tok", cfg.get("moe_top_k", 0)) or 0
     if isinstance(cfg.get("ffn_config"), dict):
@@ -325,5 +408,5 @@ def derive_dims(cfg: ModelConfig, arch: Arch, world: int) -> ModelDims:
         logit_scale=float(cfg.get("logit_scale", 1.0) or 1.0) / float(cfg.get("logits_scaling", 1.0) or 1.0),
         embed_scale=(math.sqrt(hidden) if arch.embed_scale_sqrt_hidden else float(cfg.get("embedding_multiplier", 1.0) or 1.0)),
         residual_scale=float(cfg.get("residual_multiplier", 1.0) or 1.0),
-        num_experts=ne, top_k=tk, total_heads=heads, total_kv_heads=kv,
+        num_experts=ne, top_k=tk, total_heads=heads, total_kv_heads=kv, mixers=mixers,
     )

@@ -52,12 +52,15 @@ class ForwardMeta:
     rope_cos_sin: Optional[torch.Tensor] = None      # [T, rot_dim] rotary rows of this step (multi-axis positions)
     rope_rows: Optional[torch.Tensor] = None         # [T] = arange(T): row of `rope_cos_sin` per token
     attn_horizon: Optional[torch.Tensor] = None      # [T] last KV position a row may see (image rows: end of their image)
+    state_slots: Optional[torch.Tensor] = None       # [B] slot of every sequence in the recurrent state pools, -1: none
+    v_first: Optional[torch.Tensor] = None           # [T, *] values later layers mix in (set by the first layer that mixes)
     cross: Optional[object] = None                   # rows and image states for cross-attention layers (models/mllama.py)
 
 
 class Norm:
-    def __init__(self, kind: str, weight, bias, eps: float, unit_offset: bool):
+    def __init__(self, kind: str, weight, bias, eps: float, unit_offset: bool, residual_fp32: bool = False):
         self.kind, self.weight, self.bias, self.eps, self.unit_offset = kind, weight, bias, eps, unit_offset
+        self.residual_fp32 = residual_fp32
 
     @classmethod
     def load(cls, arch: Arch, prefix: str, weights, eps: float):
@@ -65,9 +68,12 @@ class Norm:
         b = None
         if arch.norm == "layer" and arch.norm_bias and weights.has_tensor(f"{prefix}.bias"):
             b = weights.get_tensor(f"{prefix}.bias")
-        return cls(arch.norm, w, b, eps, arch.norm_unit_offset)
+        return cls(arch.norm, w, b, eps, arch.norm_unit_offset, arch.residual_fp32)
 
-    def __call__(self, x, residual=None):
+    def __call__(self, x, residual=None, rows=None):
+        if self.residual_fp32:
+            # `x` is the last block's output (None: nothing to add), `rows` ends the stream: only these rows are normed
+            return ops.residual_norm(x, residual, self.weight, self.eps, rows, keep=rows is None)
         if self.kind == "rms":
             return ops.rms_norm(x, residual, self.weight, self.eps, self.unit_offset)
         return ops.layer_norm(x, residual, self.weight, self.bias, self.eps)
@@ -78,7 +84,7 @@ class Norm:
 
     @property
     def can_quant(self):
-        return self.kind == "rms" and self.weight.shape[0] % 128 == 0
+        return self.kind == "rms" and not self.residual_fp32 and self.weight.shape[0] % 128 == 0
 
 
 def _maybe_T(w: torch.Tensor, arch: Arch) -> torch.Tensor:
@@ -436,9 +442,13 @@ def _all_reduce(t, pg):
 
 
 class DecoderLayer:
-    def __init__(self, arch: Arch, cfg, dims: ModelDims, prefix: str, weights, idx: int, comm):
+    def __init__(self, arch: Arch, cfg, dims: ModelDims, prefix: str, weights, idx: int, comm, rotary_tables=None):
         self.arch, self.dims = arch, dims
-        if cfg.model_type in ("falcon", "RefinedWeb", "RefinedWebModel"):
+        spec = dims.mixers[idx] if dims.mixers else None
+        if spec is not None:
+            self.norm1 = Norm.load(arch, f"{prefix}.{arch.norm1}", weights, dims.eps)
+            self.norm2 = Norm.load(arch, f"{prefix}.{arch.norm2}", weights, dims.eps) if spec.ff else None
+        elif cfg.model_type in ("falcon", "RefinedWeb", "RefinedWebModel"):
             # the new decoder architecture names its norms ln_attn / ln_mlp and has no input_layernorm
             self.norm1, self.norm2 = self._falcon_norms(arch, cfg, prefix, weights, dims)
         else:
@@ -446,7 +456,12 @@ class DecoderLayer:
             self.norm2 = Norm.load(arch, f"{prefix}.{arch.norm2}", weights, dims.eps) if arch.norm2 else None
         self.post_attn = Norm.load(arch, f"{prefix}.{arch.post_attn_norm}", weights, dims.eps) if arch.post_attn_norm else None
         self.post_mlp = Norm.load(arch, f"{prefix}.{arch.post_mlp_norm}", weights, dims.eps) if arch.post_mlp_norm else None
-        if arch.mla:
+        if spec is not None:
+            from .mixers import load_mixer
+
+            self.attn = load_mixer(spec, f"{prefix}.{arch.mix}", weights, idx, dims.eps, comm, rotary_tables)
+            is_moe = False
+        elif arch.mla:
             from .deepseek import MLAAttention, is_moe_layer
 
             self.attn = MLAAttention(arch, cfg, dims, prefix, weights, idx, comm)
@@ -456,8 +471,11 @@ class DecoderLayer:
             is_moe = arch.moe
         if is_moe and cfg.get("mlp_only_layers") and idx in cfg.mlp_only_layers:
             is_moe = False
-        self.mlp = (SparseMoE(arch, cfg, dims, prefix, weights, comm) if is_moe
-                    else DenseMLP(arch, cfg, dims, prefix, weights, comm, idx))
+        if spec is not None and not spec.ff:
+            self.mlp = None          # a mixer without a feed-forward
+        else:
+            self.mlp = (SparseMoE(arch, cfg, dims, prefix, weights, comm) if is_moe
+                        else DenseMLP(arch, cfg, dims, prefix, weights, comm, idx))
         self.pg, self.comm = weights.process_group, comm
         qlin = getattr(getattr(self.attn, "qkv", None), "linear", None)
         self.attn_in_quant = isinstance(qlin, Fp8Linear) and qlin.wants_quantized_input and self.norm1.can_quant
@@ -499,6 +517,8 @@ class DecoderLayer:
             attn, _ = self.post_attn(attn, None)
         if rs != 1.0:
             attn = attn * rs
+        if self.mlp is None:
+            return attn, residual
         if self.mlp_in_quant and meta.adapter_data is None:
             xq, xs, residual = self.norm2.quant(attn, residual)
             mlp = self.mlp(xq, xs, meta=meta)
@@ -516,7 +536,7 @@ class DecoderLayer:
         """True when the layer is a plain pre-norm block whose two reductions can each be fused with
         the residual add and the following RMSNorm."""
         a = self.arch
-        return (not a.parallel_residual and a.norm == "rms" and self.norm2 is not None and self.post_attn is None
+        return (not a.parallel_residual and not a.residual_fp32 and a.norm == "rms" and self.norm2 is not None and self.post_attn is None
                 and self.post_mlp is None and self.dims.residual_scale == 1.0)
 
     def fused_tp(self, x, meta: ForwardMeta, rotary, kv, next_norm: Norm, next_quant: bool, comm):
@@ -567,6 +587,12 @@ class CausalDecoder:
         self.embed_norm = Norm.load(a, px + a.embed_norm, weights, dims.eps) if a.embed_norm else None
         from ..utils.quantization import DefaultWeightsLoader, Fp8Loader
 
+        self.max_positions = int(max_positions or dims.max_positions)
+        rotary_tables = None
+        if dims.mixers:
+            from .mixers import RotaryTables
+
+            rotary_tables = RotaryTables(self.max_positions, self.device)
         self.layers: List[DecoderLayer] = []
         cross_layers = set(cfg.get("cross_attention_layers") or [])
         for i in range(dims.num_layers):
@@ -582,7 +608,7 @@ class CausalDecoder:
                 with weights.use_loader(DefaultWeightsLoader()):
                     self.layers.append(DecoderLayer(a, cfg, dims, px + a.layer.format(i=i), weights, i, comm))
             else:
-                self.layers.append(DecoderLayer(a, cfg, dims, px + a.layer.format(i=i), weights, i, comm))
+                self.layers.append(DecoderLayer(a, cfg, dims, px + a.layer.format(i=i), weights, i, comm, rotary_tables))
         self.final_norm = Norm.load(a, px + a.final_norm, weights, dims.eps)
         head_name = px + a.lm_head if not a.lm_head.startswith("lm_head") or not prefix else a.lm_head
         candidates = [head_name, px + a.lm_head, a.lm_head, px + a.embed]
@@ -595,7 +621,6 @@ class CausalDecoder:
                     break
             else:
                 raise KeyError("no lm_head / tied embedding weight found")
-        self.max_positions = int(max_positions or dims.max_positions)
         self.rotary = RotaryTable.from_config(cfg, dims.rot_dim, dims.rope_theta, self.max_positions,
                                               a.rope_neox).to(self.device)
         # Gemma-3: sliding-window layers rotate with their own (unscaled) base frequency
@@ -614,6 +639,11 @@ class CausalDecoder:
             raise NotImplementedError("ALiBi attention bias is served by the padded fallback runner")
 
     # ---------------------------------------------------------------------------------------
+    @property
+    def recurrent(self) -> bool:
+        """True when a sequence carries state that a step advances (and that a step must therefore run exactly once)."""
+        return any(s.recurrent for s in self.dims.mixers or [])
+
     def embed_tokens(self, input_ids: torch.Tensor, positions: Optional[torch.Tensor] = None) -> torch.Tensor:
         h = self.embed(input_ids)
         if self.dims.embed_scale != 1.0:
@@ -656,7 +686,20 @@ class CausalDecoder:
                                nxt.attn_in_quant if nxt else False, comm)
         return x
 
+    def _forward_hidden_fp32_stream(self, meta: ForwardMeta, kv_cache) -> torch.Tensor:
+        """Layers around an fp32 residual stream; the final norm runs on the rows that need logits only."""
+        meta.v_first = None
+        residual = ops.embed_residual(meta.input_ids, self.embed.weight, self.dims.embed_scale)
+        h = None
+        for i, layer in enumerate(self.layers):
+            h, residual = layer(h, residual, meta, None, kv_cache[i])
+        meta.v_first = None
+        return self.final_norm(h, residual, rows=meta.lm_head_indices)[0]
+
     def forward_hidden(self, meta: ForwardMeta, kv_cache) -> torch.Tensor:
+        """Normalised hidden rows: of every token, or with an fp32 residual stream of ``meta.lm_head_indices`` only."""
+        if self.arch.residual_fp32:
+            return self._forward_hidden_fp32_stream(meta, kv_cache)
         if self._fused_tp_ok(meta):
             return self._forward_hidden_fused_tp(meta, kv_cache)
         h = meta.inputs_embeds if meta.inputs_embeds is not None else self.embed_tokens(meta.input_ids, meta.positions)
@@ -699,7 +742,7 @@ class CausalDecoder:
     def forward(self, meta: ForwardMeta, kv_cache) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
         """Returns ``(logits[rows, V], speculative_logits or None)``."""
         h = self.forward_hidden(meta, kv_cache)
-        if meta.lm_head_indices is not None:
+        if meta.lm_head_indices is not None and not self.arch.residual_fp32:
             h = h[meta.lm_head_indices.long()]
         logits = self.logits(h)
         spec = self.speculator(h, logits) if self.speculator is not None else None

@@ -31,10 +31,13 @@ from ..proto import generate_v3 as pb
 from ..utils.tokens import NextTokenChooser, StoppingCriteria, batch_top_tokens
 from .decoder import CausalDecoder, ForwardMeta
 from .model import Model
+from .state import Lease, Pool
 from .types import Batch, GeneratedText, Generation, Tokens
 
 BLOCK_SIZE = int(os.environ.get("TGI_B200_BLOCK_SIZE", "16"))
 WIGGLE_ROOM = float(os.environ.get("TGI_WIGGLE_ROOM", "0.90"))
+# slots of the recurrent state pools = live requests a shard can hold (models with recurrent layers only)
+STATE_SLOTS = int(os.environ.get("TGI_B200_STATE_SLOTS", "256"))
 # set by the launcher (reference: models/globals.py:8-20): whether the router may re-use cached prompt prefixes
 # and split long prompts into chunks
 PREFIX_CACHING = os.environ.get("PREFIX_CACHING", "1").lower() in ("1", "true")
@@ -62,6 +65,12 @@ class Seq:
     prefill_logprobs: List[float] = field(default_factory=list)
     adapter_index: int = 0
     finished: bool = False
+    state: Optional[Lease] = None        # slot of the recurrent state pools, taken by the first step with tokens
+
+    def release_state(self):
+        if self.state is not None:
+            self.state.release()
+            self.state = None
 
     @property
     def want_prefill_logprobs(self) -> bool:
@@ -209,6 +218,8 @@ class FlashCausalLMBatch(Batch):
         ):
             return self
         indices = [self.requests_idx_mapping[rid] for rid in request_ids]
+        for i in set(range(len(self.seqs))) - set(indices):
+            self.seqs[i].release_state()
         self.seqs = [self.seqs[i] for i in indices]
         self.next_token_chooser = self.next_token_chooser.filter(indices)
         self._reindex()
@@ -278,10 +289,16 @@ class FlashCausalLM(Model):
                  speculate: int = 0, kv_cache_dtype: Optional[torch.dtype] = None,
                  max_prefill_tokens: Optional[int] = None, eos_token_ids=None):
         windows = [w for w in model.dims.windows if w > 0]
+        # recurrent layers: the state of a prompt prefix is not kept (no prefix re-use), cannot be rolled back (no
+        # speculation), and a step must not run twice (no replay ahead of a batch change)
+        self.recurrent = bool(getattr(model, "recurrent", False))
+        if self.recurrent and speculate:
+            raise ValueError("speculative decoding needs a cache that can be rolled back; this model has recurrent layers")
         super().__init__(model, tokenizer, requires_padding=False, dtype=dtype, device=device, rank=rank,
                          world_size=world_size, sliding_window=(windows[0] if windows else None),
-                         speculate=speculate, support_chunking=PREFILL_CHUNKING, use_prefix_caching=PREFIX_CACHING,
-                         block_size=BLOCK_SIZE)
+                         speculate=speculate, support_chunking=PREFILL_CHUNKING,
+                         use_prefix_caching=PREFIX_CACHING and not self.recurrent, block_size=BLOCK_SIZE,
+                         max_batch_size=STATE_SLOTS if self.recurrent else None)
         self.dims = model.dims
         self.kv_cache_dtype = kv_cache_dtype or dtype
         self.kv_cache: List[Tuple[torch.Tensor, torch.Tensor]] = []
@@ -293,7 +310,8 @@ class FlashCausalLM(Model):
         # of the previous step, before its text post-processing (see `_prelaunch_next_decode`)
         self._prelaunched = None
         self.overlap_hits = 0          # steps that found their replay already on the stream
-        self.overlap_decode = os.environ.get("TGI_B200_OVERLAP_DECODE", "1") == "1"
+        self.overlap_decode = os.environ.get("TGI_B200_OVERLAP_DECODE", "1") == "1" and not self.recurrent
+        self.state_slots: Optional[Pool] = None      # made with the cache
         self.eos_token_ids = eos_token_ids
         if eos_token_ids is not None and tokenizer is not None:
             try:
@@ -308,6 +326,8 @@ class FlashCausalLM(Model):
     # -- KV cache --------------------------------------------------------------------------------
     def kv_bytes_per_block(self) -> int:
         d = self.dims
+        if getattr(d, "mixers", None):
+            return max(1, sum(l.attn.page_bytes(BLOCK_SIZE) for l in self.model.layers))
         item = torch.empty((), dtype=self.kv_cache_dtype).element_size()
         return 2 * d.num_layers * BLOCK_SIZE * d.num_kv_heads * (d.attn_head_dim or d.head_dim) * item
 
@@ -346,12 +366,19 @@ class FlashCausalLM(Model):
                            chooser.top_k if chooser.any_top_k else None, chooser.top_p if chooser.any_top_p else None,
                            do_sample, seeds, steps)
 
-    def init_kv_cache(self, num_blocks: int):
+    def init_kv_cache(self, num_blocks: int, state_slots: Optional[int] = None):
         d = self.dims
         self.kv_cache = []
         if self.device.type == "cuda":
             torch.cuda.empty_cache()
         self.num_blocks = int(num_blocks)
+        if getattr(d, "mixers", None):
+            # every layer has its own kind of cache: pages, or slots of recurrent state
+            slots = int(state_slots or self.max_batch_size or 1)
+            self.state_slots = Pool(0, slots, "recurrent state slots") if self.recurrent else None
+            for layer in self.model.layers:
+                self.kv_cache.append(layer.attn.cache_tensors(self.num_blocks, BLOCK_SIZE, slots, self.device))
+            return
         for _ in range(d.num_layers):
             k = torch.zeros(num_blocks, BLOCK_SIZE, d.num_kv_heads, d.attn_head_dim or d.head_dim,
                             dtype=self.kv_cache_dtype, device=self.device)
@@ -364,7 +391,7 @@ class FlashCausalLM(Model):
         Returns ``(max_supported_total_tokens, max_input_tokens, max_total_tokens)``.
         """
         batch_blocks = batch.num_blocks
-        self.init_kv_cache(max(batch_blocks, 1))
+        self.init_kv_cache(max(batch_blocks, 1))        # with all slots of recurrent state: what is left goes to pages
         if self.device.type == "cuda":
             torch.cuda.synchronize(self.device)
         self.generate_token(batch)
@@ -393,9 +420,20 @@ class FlashCausalLM(Model):
             self.graphs.capture_all()
         return cap, max_input_tokens, max_total_tokens
 
+    def state_slot(self, seq: Seq, start: int) -> int:
+        """Slot of the recurrent state of ``seq``, whose step starts at position ``start``."""
+        if seq.state is not None and seq.state.pool is not self.state_slots:
+            seq.state = None             # a lease on a cache that has been replaced
+        if seq.state is None:
+            if start > 0:
+                raise RuntimeError(f"request {seq.request.id} continues at position {start} without its recurrent state")
+            seq.state = Lease(self.state_slots)
+        return seq.state.unit
+
     # -- forward ---------------------------------------------------------------------------------
-    def build_meta(self, batch: FlashCausalLMBatch, counts: List[int]):
-        """Pack the step's metadata; returns ``(ForwardMeta, row bookkeeping)``."""
+    def build_meta(self, batch: FlashCausalLMBatch, counts: List[int], head_rows_of: Optional[List[List[int]]] = None):
+        """Pack the step's metadata; returns ``(ForwardMeta, row bookkeeping)``.  ``head_rows_of`` (per sequence, offsets
+        inside its tokens of this step) replaces the rule of which rows get logits."""
         seqs = batch.seqs
         B = len(seqs)
         T = sum(counts)
@@ -406,6 +444,7 @@ class FlashCausalLM(Model):
         kv_lens = np.empty(B, dtype=np.int32)
         max_blocks = max(1, max(len(s.blocks) for s in seqs))
         tables = np.zeros((B, max_blocks), dtype=np.int32)
+        state = np.full(B, -1, dtype=np.int32)
         head_rows: List[int] = []       # rows of the hidden state that need logits
         row_owner: List[Tuple[int, int]] = []  # (seq index, offset inside the chunk) per logits row
         t = 0
@@ -424,7 +463,12 @@ class FlashCausalLM(Model):
             cu[i + 1] = t + n
             kv_lens[i] = start + n
             tables[i, :len(s.blocks)] = s.blocks
-            if n > 0:
+            if n > 0 and self.recurrent:
+                state[i] = self.state_slot(s, start)
+            if head_rows_of is not None:
+                head_rows.extend(t + j for j in head_rows_of[i])
+                row_owner.extend((i, j) for j in head_rows_of[i])
+            elif n > 0:
                 finishing = s.prefilling and (start + n == s.prompt_len)
                 if s.prefilling and s.want_prefill_logprobs:
                     head_rows.extend(range(t, t + n))
@@ -437,11 +481,15 @@ class FlashCausalLM(Model):
                     row_owner.extend((i, j) for j in range(n))
             t += n
         head = np.asarray(head_rows, dtype=np.int32)
-        dev = self.staging.upload([input_ids, positions, slots, cu, kv_lens, tables, head])
+        arrays = [input_ids, positions, slots, cu, kv_lens, tables, head]
+        if self.recurrent:
+            arrays.append(state)
+        dev = self.staging.upload(arrays)
         meta = ForwardMeta(
             input_ids=dev[0], positions=dev[1], slots=dev[2], cu_seqlens_q=dev[3], kv_lens=dev[4],
             block_tables=dev[5], max_q=max(counts) if counts else 0, max_kv=int(kv_lens.max()) if B else 0,
-            lm_head_indices=dev[6] if len(head_rows) != T else None,
+            lm_head_indices=dev[6] if head_rows_of is not None or len(head_rows) != T else None,
+            state_slots=dev[7] if self.recurrent else None,
         )
         lora = getattr(self, "lora", None)
         if lora is not None and any(s.adapter_index > 0 for s in seqs):
@@ -479,6 +527,25 @@ class FlashCausalLM(Model):
     def forward(self, meta: ForwardMeta) -> torch.Tensor:
         logits, spec = self.model.forward(meta, self.kv_cache)
         self.last_speculative_logits = spec     # [rows, n_heads, V] when a speculator head is attached
+        return logits
+
+    @torch.no_grad()
+    def step_logits(self, batch: FlashCausalLMBatch, counts: List[int], want: List[List[int]]) -> Optional[torch.Tensor]:
+        """One forward over the next ``counts[i]`` tokens of every sequence, without sampling: the logits of the rows
+        ``want[i]`` (offsets inside those tokens), in order, or ``None``.  Steps of single tokens replay the decode graphs
+        as ``generate_token`` does."""
+        seqs = batch.seqs
+        decode = self.graphs is not None and all(c == 1 and s.cache_len > 0 for c, s in zip(counts, seqs))
+        if decode and self.graphs.supports(batch) and self.graph_eligible(batch):
+            logits, _ = self.graphs.run(batch, counts)
+            rows = [i for i, w in enumerate(want) for _ in w]
+            logits = logits[rows] if rows else None
+        else:
+            meta, owners = self.build_meta(batch, counts, want)
+            logits = self.forward(meta)
+            logits = logits if owners else None
+        for s, n in zip(seqs, counts):
+            s.cache_len += n
         return logits
 
     # -- one engine step -------------------------------------------------------------------------
@@ -713,5 +780,7 @@ class FlashCausalLM(Model):
                 s.first_chunk = None
         decode_ns = time.time_ns() - decode_start
         if all(s.finished for s in seqs):
+            for s in seqs:
+                s.release_state()
             return generations, None, (forward_ns, decode_ns)
         return generations, batch, (forward_ns, decode_ns)

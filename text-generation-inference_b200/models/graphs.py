@@ -8,7 +8,8 @@ is where B200 loses most, and all static inputs of a bucket live in ONE int32 bu
 by a single host-to-device copy per step.
 
 Padding rows use slot ``-1`` (the RoPE+KV-store kernel skips the write) and a KV length of 0 (the
-attention kernel produces zeros), so they never touch real cache pages.
+attention kernel produces zeros), so they never touch real cache pages; their slot of recurrent state is ``-1``, which
+the state kernels neither read nor write.
 """
 from __future__ import annotations
 
@@ -45,12 +46,14 @@ class _Bucket:
         self.off_kv = self.off_cu + seg(bs + 1)
         self.off_bt = self.off_kv + seg(bs)
         self.off_ad = self.off_bt + seg(bs * max_blocks)     # LoRA adapter index per row (0 = none)
-        self.total = self.off_ad + seg(bs)
+        self.off_st = self.off_ad + seg(bs)                  # slot of the recurrent state pools per row (-1 = none)
+        self.total = self.off_st + seg(bs)
         self.host = torch.zeros(self.total, dtype=torch.int32, pin_memory=True)
         self.host_np = self.host.numpy()
         self.dev = torch.zeros(self.total, dtype=torch.int32, device=dev)
         self.host_np[self.off_cu:self.off_cu + bs + 1] = np.arange(bs + 1, dtype=np.int32)
         self.host_np[self.off_slots:self.off_slots + bs] = -1
+        self.host_np[self.off_st:self.off_st + bs] = -1
         self.dev.copy_(self.host)
         d = self.dev
         self.meta = ForwardMeta(
@@ -63,6 +66,7 @@ class _Bucket:
             max_q=1,
             max_kv=runner_max_kv(runner),
             lm_head_indices=None,
+            state_slots=d[self.off_st:self.off_st + bs] if getattr(runner, "recurrent", False) else None,
         )
         self.token_adapter = d[self.off_ad:self.off_ad + bs]
         self.row_owner: List[Optional[tuple]] = [None] * bs   # (block list, its length) whose table sits in row i
@@ -168,6 +172,10 @@ class DecodeGraphs:
                 # the list, so "same list object" cannot be a recycled identity
                 bt[i, :nb] = s.blocks
                 b.row_owner[i] = (s.blocks, nb)
+        if getattr(self.runner, "recurrent", False):
+            st = h[b.off_st:b.off_st + bs]
+            st[:n] = [self.runner.state_slot(s, len(s.ids) - 1) for s in seqs]
+            st[n:] = -1
         if lora:
             ad = h[b.off_ad:b.off_ad + bs]
             ad[:n] = [s.adapter_index for s in seqs]

@@ -25,6 +25,9 @@ class FastLinear:
     """``y = x @ W^T + b`` with ``W[N,K]`` in the serving dtype."""
 
     def __init__(self, weight: torch.Tensor, bias: Optional[torch.Tensor] = None):
+        if weight.is_cuda and weight.dtype == torch.bfloat16 and weight.shape[1] % 8 != 0:
+            # the GEMM fetches rows in 16-byte pieces; `ops.linear` pads the activations to match
+            weight = torch.nn.functional.pad(weight, (0, -weight.shape[1] % 8))
         self.weight = weight
         self.bias = bias
 

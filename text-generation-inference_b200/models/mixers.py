@@ -1,0 +1,209 @@
+"""Token mixers of decoders whose layers differ, configured per layer by an ``arch.MixerSpec``.
+
+Every mixer is called like ``decoder.Attention`` (``x, x_scale, meta, rotary, kv, reduce``), owns the tensors of its
+cache (``cache_tensors``) and runs as a short sequence of fused ops:
+
+    attention   qkv GEMM -> rotate + unit RMS + value mixing + page store -> paged attention -> o GEMM
+    delta       one GEMM for q, k, v, write strengths and both low-rank inputs -> decay / gate GEMMs
+                -> short convolutions + unit norms + decays -> state scan -> norm x gate -> o GEMM
+    decay       one GEMM for q, k, v, gate -> state scan (SiLU applied on the way in) -> norm x gate -> o GEMM
+
+Recurrent layers keep, per slot of the state pool, the matrix state of every head (fp32, ``[H, vdim, pitch]``) and,
+for short convolutions, the last ``taps - 1`` inputs of every channel.  Which tokens a sequence brings and from which
+slot it continues is in the step's metadata, so prompts, portions of prompts and decoded tokens are one code path.
+"""
+from __future__ import annotations
+
+from typing import Dict, List, Optional, Sequence, Tuple
+
+import torch
+
+from .. import ops
+from ..utils.rotary import RotaryTable, scaled_frequencies
+from .arch import MixerSpec
+from .layers import FastLinear, TensorParallelColumnLinear, TensorParallelRowLinear
+
+ALIGN = 8       # elements: 16-byte rows and column offsets of bf16 operands
+
+
+def _up(n: int) -> int:
+    return (n + ALIGN - 1) // ALIGN * ALIGN
+
+
+def pad_columns(w: torch.Tensor) -> torch.Tensor:
+    """Weight ``[N, K]`` with K brought to a multiple of ``ALIGN`` (GEMM operands are fetched in 16-byte pieces)."""
+    return torch.nn.functional.pad(w, (0, _up(w.shape[1]) - w.shape[1])).contiguous()
+
+
+def _column_input(w: torch.Tensor) -> torch.Tensor:
+    return pad_columns(w) if w.dtype == torch.bfloat16 else w.contiguous()
+
+
+def stack_rows(parts: Sequence[torch.Tensor]) -> Tuple[torch.Tensor, List[int]]:
+    """One matrix whose products are those of ``parts`` side by side; every part starts at a multiple of ``ALIGN``
+    columns of the output (zero rows in between).  Returns ``(matrix, column offsets)``."""
+    offs, rows = [], 0
+    for p in parts:
+        offs.append(rows)
+        rows += _up(p.shape[0])
+    w = parts[0].new_zeros(rows, parts[0].shape[1])
+    for p, o in zip(parts, offs):
+        w[o:o + p.shape[0]] = p
+    return _column_input(w), offs
+
+
+def spread_columns(w: torch.Tensor, heads: int, width: int, pitch: int) -> torch.Tensor:
+    """Output projection ``[N, heads * width]`` for inputs whose heads are ``pitch`` columns apart."""
+    if pitch == width:
+        return _column_input(w)
+    out = w.new_zeros(w.shape[0], heads, pitch)
+    out[:, :, :width] = w.view(w.shape[0], heads, width)
+    return out.view(w.shape[0], heads * pitch)
+
+
+class RotaryTables:
+    """Tables shared by the layers of a model that rotate alike."""
+
+    def __init__(self, max_positions: int, device):
+        self.max_positions, self.device = max_positions, device
+        self._tables: Dict[tuple, RotaryTable] = {}
+
+    def get(self, s: MixerSpec) -> RotaryTable:
+        key = (s.rot_dims, s.rot_base, s.rot_scaling)
+        if key not in self._tables:
+            self._tables[key] = RotaryTable.from_frequencies(
+                scaled_frequencies(s.rot_base, s.rot_dims, s.rot_scaling), self.max_positions).to(self.device)
+        return self._tables[key]
+
+
+class Mixer:
+    def __init__(self, spec: MixerSpec, prefix: str, weights, idx: int, eps: float, comm=None):
+        self.spec, self.prefix, self.weights, self.layer_idx, self.eps, self.comm = spec, prefix, weights, idx, eps, comm
+        self.dtype, self.device, self.pg = weights.dtype, weights.device, weights.process_group
+
+    def tensor(self, name: str) -> torch.Tensor:
+        return self.weights.get_tensor(f"{self.prefix}.{name}")
+
+    def f32(self, name: str) -> torch.Tensor:
+        return self.weights.get_tensor(f"{self.prefix}.{name}", to_dtype=False).float().contiguous()
+
+    def fused(self, names: Sequence[str]) -> Tuple[TensorParallelColumnLinear, List[int]]:
+        w, offs = stack_rows([self.tensor(n) for n in names])
+        return TensorParallelColumnLinear(FastLinear(w)), offs
+
+    def row(self, w: torch.Tensor) -> TensorParallelRowLinear:
+        return TensorParallelRowLinear(FastLinear(w), self.pg, self.comm)
+
+    def state_bytes(self) -> int:
+        """Bytes of one slot of the state pool."""
+        return sum(t.numel() * t.element_size() for t in self.cache_tensors(1, 1, 1, "meta")) if self.spec.recurrent else 0
+
+    def page_bytes(self, block_size: int) -> int:
+        return 0 if self.spec.recurrent else sum(
+            t.numel() * t.element_size() for t in self.cache_tensors(1, block_size, 1, "meta"))
+
+
+class MixedAttention(Mixer):
+    """Paged attention with its own head sizes: rotation of the first dimensions, weightless RMS of q and k after it,
+    values mixed with an earlier layer's, keys limited to the query's chunk, a sink in the softmax."""
+
+    def __init__(self, spec, prefix, weights, idx, eps, comm=None, rotary: Optional[RotaryTables] = None):
+        super().__init__(spec, prefix, weights, idx, eps, comm)
+        s = spec
+        self.qkv, self.offs = self.fused(["q", "k", "v"])
+        self.v_lambda = float(self.f32("vmix").reshape(-1)[0]) if s.v_mix and weights.has_tensor(f"{prefix}.vmix") else 0.0
+        self.kd, self.vd = ops.attention_pitch(s.dim, s.vdim, self.dtype, self.device)
+        self.o = self.row(spread_columns(self.tensor("o"), s.heads, s.vdim, self.vd))
+        self.rotary = rotary.get(s)
+
+    def cache_tensors(self, num_blocks: int, block_size: int, slots: int, device):
+        # zeros: the kernels never write the padding columns of a page, and padded queries must meet zeros there
+        return tuple(torch.zeros(num_blocks, block_size, self.spec.kv_heads, d, dtype=self.dtype, device=device)
+                     for d in (self.kd, self.vd))
+
+    def __call__(self, x, x_scale, meta, rotary, kv, reduce: bool = True, out=None):
+        s = self.spec
+        k_cache, v_cache = kv
+        proj = self.qkv(x)
+        v_first = None
+        if s.v_mix:
+            v_first = meta.v_first
+            if v_first is None:      # the first such layer: its values are what the later ones mix in
+                meta.v_first = proj[:, self.offs[2]:self.offs[2] + s.kv_heads * s.vdim]
+        q = ops.rotate_norm_store(proj, self.offs, meta.positions, self.rotary.cos_sin, meta.slots, k_cache, v_cache, s.heads,
+                                  s.kv_heads, s.dim, s.vdim, s.rot_dims, s.qk_unit_rms, self.eps, v_first, self.v_lambda)
+        a = ops.paged_attention(q, k_cache, v_cache, meta.block_tables, meta.cu_seqlens_q, meta.kv_lens, s.scale,
+                                max_q=meta.max_q, max_kv=meta.max_kv, chunk=s.chunk, sink=s.sink)
+        return self.o(a.view(a.shape[0], -1), reduce=reduce, out=out)
+
+
+class GatedDelta(Mixer):
+    """Gated delta rule whose decay acts per head and key channel."""
+
+    def __init__(self, spec, prefix, weights, idx, eps, comm=None, rotary=None):
+        super().__init__(spec, prefix, weights, idx, eps, comm)
+        s = spec
+        self.proj, self.offs = self.fused(["q", "k", "v", "b", "a1", "g1"])
+        self.conv = tuple(self.f32(f"{n}.conv") for n in ("q", "k", "v"))
+        self.taps = self.conv[0].shape[1]
+        self.a_rank, self.g_rank = (_up(self.weights.get_shape(f"{prefix}.{n}")[0]) for n in ("a1", "g1"))
+        # K padded like the rows of a1 / g1: their outputs are read where the fused product left them
+        self.a2, self.g2 = (FastLinear(pad_columns(self.tensor(n))) for n in ("a2", "g2"))
+        self.a_log, self.dt_bias, self.norm = self.f32("A_log"), self.f32("dt_bias"), self.f32("norm")
+        self.pitch = ops.recurrent_pitch(s.dim, self.device)
+        self.o = self.row(_column_input(self.tensor("o")))
+        self.out_cols = self.o.linear.weight.shape[1]
+
+    def cache_tensors(self, num_blocks: int, block_size: int, slots: int, device):
+        s = self.spec
+        channels = 2 * s.kv_heads * s.dim + s.heads * s.vdim
+        return (torch.zeros(slots, self.taps - 1, channels, dtype=self.dtype, device=device),
+                torch.zeros(slots, s.heads, s.vdim, self.pitch, dtype=torch.float32, device=device))
+
+    def __call__(self, x, x_scale, meta, rotary, kv, reduce: bool = True, out=None):
+        s = self.spec
+        conv_state, state = kv
+        p = self.proj(x)
+        a = self.a2(p[:, self.offs[4]:self.offs[4] + self.a_rank])
+        g = self.g2(p[:, self.offs[5]:self.offs[5] + self.g_rank])
+        q, k, v, decay, beta, qk = ops.delta_inputs(
+            p, self.offs, a, *self.conv, self.a_log, self.dt_bias, meta.cu_seqlens_q, meta.kv_lens, meta.state_slots,
+            conv_state, s.kv_heads, s.heads, s.dim, self.pitch, s.vdim, meta.max_q == 1)
+        o = ops.delta_scan(q, k, v, decay, beta, qk, meta.cu_seqlens_q, meta.kv_lens, meta.state_slots, state, s.dim, meta.max_q)
+        y = ops.gated_norm(o, g, self.norm, self.eps, s.heads, self.out_cols)
+        return self.o(y, reduce=reduce, out=out)
+
+
+class DecayAttention(Mixer):
+    """Linear attention whose state shrinks by a fixed factor per head and token."""
+
+    def __init__(self, spec, prefix, weights, idx, eps, comm=None, rotary=None):
+        super().__init__(spec, prefix, weights, idx, eps, comm)
+        s = spec
+        if len(s.decay) != s.heads:
+            raise ValueError(f"{prefix}: {len(s.decay)} decays for {s.heads} heads")
+        self.proj, self.offs = self.fused(["q", "k", "v", "g"])
+        self.decay = torch.tensor(s.decay, dtype=torch.float32, device=self.device)
+        self.norm = self.f32("norm")
+        self.pitch = ops.recurrent_pitch(s.dim, self.device)
+        self.o = self.row(_column_input(self.tensor("o")))
+        self.out_cols = self.o.linear.weight.shape[1]
+
+    def cache_tensors(self, num_blocks: int, block_size: int, slots: int, device):
+        s = self.spec
+        return (torch.zeros(slots, s.heads, s.vdim, self.pitch, dtype=torch.float32, device=device),)
+
+    def __call__(self, x, x_scale, meta, rotary, kv, reduce: bool = True, out=None):
+        s = self.spec
+        p = self.proj(x)
+        o = ops.decay_scan(p, self.offs, self.decay, meta.cu_seqlens_q, meta.kv_lens, meta.state_slots, kv[0], s.heads, s.dim,
+                           s.vdim, meta.max_q)
+        y = ops.gated_norm(o, p[:, self.offs[3]:], self.norm, self.eps, 1, self.out_cols)
+        return self.o(y, reduce=reduce, out=out)
+
+
+MIXERS = {"attention": MixedAttention, "delta": GatedDelta, "decay": DecayAttention}
+
+
+def load_mixer(spec: MixerSpec, prefix: str, weights, idx: int, eps: float, comm, rotary: RotaryTables) -> Mixer:
+    return MIXERS[spec.kind](spec, prefix, weights, idx, eps, comm, rotary)

@@ -17,7 +17,7 @@ class Model(ABC):
     def __init__(self, model, tokenizer, requires_padding: bool, dtype: torch.dtype, device: torch.device,
                  rank: int = 0, world_size: int = 1, sliding_window: Optional[int] = None, speculate: int = 0,
                  support_chunking: bool = True, use_prefix_caching: bool = True, block_size: int = 16,
-                 attention_impl: str = "paged-sm100"):
+                 attention_impl: str = "paged-sm100", max_batch_size: Optional[int] = None):
         self.model = model
         self.tokenizer = tokenizer
         self.all_special_ids = set(getattr(tokenizer, "all_special_ids", []) or [])
@@ -33,6 +33,8 @@ class Model(ABC):
         self.use_prefix_caching = use_prefix_caching
         self.block_size = block_size
         self.attention_impl = attention_impl
+        # live requests the shard can hold state for; the router keeps its batches within it
+        self.max_batch_size = max_batch_size
 
     @property
     def info(self):
@@ -44,6 +46,8 @@ class Model(ABC):
         )
         if self.sliding_window is not None:
             m.window_size = self.sliding_window
+        if self.max_batch_size is not None:
+            m.max_batch_size = self.max_batch_size
         return m
 
     @property

@@ -70,14 +70,15 @@ def rope_and_cache(qkv, positions, cos_sin, slots, k_cache, v_cache, num_heads, 
 
 
 def paged_attention(q, k_cache, v_cache, block_tables, cu_seqlens_q, kv_lens, scale, window=-1, softcap=0.0,
-                    k_scale=None, v_scale=None, max_q=None, max_kv=None, horizon=None):
+                    k_scale=None, v_scale=None, max_q=None, max_kv=None, horizon=None, chunk=0, sink=False):
     """``horizon`` (optional int32 ``[T]``): last KV position each query row may see when that is past its own
-    position (image rows that attend to their whole image); ``None`` is plain causal attention."""
+    position (image rows that attend to their whole image); ``None`` is plain causal attention.  ``chunk`` > 0: rows see
+    only keys of their own chunk of ``chunk`` positions.  ``sink``: one more key of score 0 and no value in the softmax."""
     if use_native(q):
         return native().paged_attention(q, k_cache, v_cache, block_tables, cu_seqlens_q, kv_lens, scale,
-                                        window, softcap, k_scale, v_scale, max_q, max_kv, horizon=horizon)
+                                        window, softcap, k_scale, v_scale, max_q, max_kv, horizon=horizon, chunk=chunk, sink=sink)
     return ref.paged_attention(q, k_cache, v_cache, block_tables, cu_seqlens_q, kv_lens, scale, window,
-                               softcap, k_scale, v_scale, horizon=horizon)
+                               softcap, k_scale, v_scale, horizon=horizon, chunk=chunk, sink=sink)
 
 
 def act_and_mul(gate_up, act="silu"):
@@ -94,7 +95,69 @@ def act_and_mul_quant(gate_up, act="silu"):
 
 
 def activation(x, act):
+    if use_native(x) and x.dtype in (torch.bfloat16, torch.float32) and x.is_contiguous():
+        return native().activation(x, act)
     return ref.activation(x, act)
+
+
+# ---- token mixers of hybrid decoders -------------------------------------------------------------
+def _mixer_backend(t):
+    return native() if use_native(t) else ref
+
+
+def embed_residual(ids, table, scale=1.0):
+    """``table[ids] * scale`` as the fp32 residual stream."""
+    return _mixer_backend(table).embed_residual(ids, table, scale)
+
+
+def residual_norm(delta, residual, weight, eps, rows=None, keep=True):
+    """``r = residual + delta`` in fp32 and ``RMSNorm(r) * weight`` in the weight's dtype: ``(normed, r)``.  ``rows`` picks
+    the rows to compute; ``keep=False`` drops ``r``."""
+    return _mixer_backend(residual).residual_norm(delta, residual, weight, eps, rows, keep)
+
+
+def attention_pitch(dim, vdim, dtype, device):
+    """Page widths of a head's keys and values on ``device`` (see ``ops.cuda.attention_pitch``)."""
+    if torch.device(device).type == "cuda" and not _FORCE_TORCH:
+        return native().attention_pitch(dim, vdim, dtype)
+    return dim, vdim
+
+
+def rotate_norm_store(proj, offs, positions, cos_sin, slots, k_cache, v_cache, num_heads, num_kv_heads, dim, vdim, rot_dim,
+                      qk_norm, eps, v_first=None, v_lambda=0.0):
+    """``proj[T, *]`` with q, k, v from columns ``offs``: rotate q and k, divide them by their root mean square per head
+    (``qk_norm``), mix v with ``v_first`` (``(1 - lambda) v + lambda v_first``), store k and v; returns q ``[T, Hq, Dk]``."""
+    return _mixer_backend(proj).rotate_norm_store(proj, offs, positions, cos_sin, slots, k_cache, v_cache, num_heads,
+                                                  num_kv_heads, dim, vdim, rot_dim, qk_norm, eps, v_first, v_lambda)
+
+
+def recurrent_pitch(dim, device):
+    """Row pitch of a head's recurrent state (``dim`` key channels)."""
+    if torch.device(device).type == "cuda" and not _FORCE_TORCH:
+        return native().recurrent_pitch(dim)
+    return dim
+
+
+def delta_inputs(proj, offs, a_pre, conv_q, conv_k, conv_v, a_log, dt_bias, cu, kv_lens, state_slots, conv_state, kv_heads,
+                 heads, dim, pitch, vdim, single):
+    """Short convolutions, unit norms, decays and write strengths of a gated delta rule; advances ``conv_state``."""
+    return _mixer_backend(proj).delta_inputs(proj, offs, a_pre, conv_q, conv_k, conv_v, a_log, dt_bias, cu, kv_lens,
+                                             state_slots, conv_state, kv_heads, heads, dim, pitch, vdim, single)
+
+
+def delta_scan(q, k, v, g, beta, qk, cu, kv_lens, state_slots, state, dim, max_q):
+    """Gated delta rule over the step's tokens; advances ``state`` and returns the read-outs, fp32 ``[T, H, vdim]``."""
+    return _mixer_backend(v).delta_scan(q, k, v, g, beta, qk, cu, kv_lens, state_slots, state, dim, max_q)
+
+
+def decay_scan(proj, offs, decay, cu, kv_lens, state_slots, state, heads, dim, vdim, max_q):
+    """Linear attention with one decay per head on ``silu`` of q, k, v; advances ``state``, fp32 ``[T, H, vdim]``."""
+    return _mixer_backend(proj).decay_scan(proj, offs, decay, cu, kv_lens, state_slots, state, heads, dim, vdim, max_q)
+
+
+def gated_norm(o, gate, weight, eps, groups, out_cols):
+    """RMSNorm of ``o`` over each of ``groups`` equal parts, times ``weight``, times ``sigmoid(gate)``; ``[T, out_cols]``."""
+    return _mixer_backend(o).gated_norm(o, gate, weight, eps, groups, out_cols)
 
 
 def _into(out, y):
@@ -107,7 +170,10 @@ def _into(out, y):
 
 
 def linear(x, weight, bias=None, out=None):
-    """``x @ weight^T + bias``; ``out`` (bf16, contiguous) receives the result when given."""
+    """``x @ weight^T + bias``; ``out`` (bf16, contiguous) receives the result when given.  A weight with up to 7 more
+    columns than ``x`` was padded at load to the 16-byte rows the GEMM fetches."""
+    if 0 < weight.shape[1] - x.shape[-1] < 8:
+        x = torch.nn.functional.pad(x, (0, weight.shape[1] - x.shape[-1]))
     if use_native(x) and x.dtype == torch.bfloat16 and weight.dtype == torch.bfloat16:
         return native().gemm_bf16(x, weight, bias, out=out)
     return _into(out, ref.linear(x, weight, bias))

@@ -1,9 +1,12 @@
 """Builds the sm_100a kernel library in-tree with nvcc (no GPU needed: nvcc cross-compiles).
 
-``python -m tgi_b200.ops.build`` compiles every ``csrc/*.cu`` with
+``python -m tgi_b200.ops.build [SET]`` compiles every ``csrc/*.cu`` with
 ``-gencode arch=compute_100a,code=sm_100a -lineinfo`` and links ``ops/libtgi_b200_kernels.so``.
 The library exposes plain ``extern "C"`` launchers that take raw device pointers and a stream, so it
 has no dependency on the PyTorch C++ headers and rebuilds in seconds.
+
+``KERNEL_SETS`` names parts of the library that are enough for some models; such a part becomes a library of its
+own, for tools that run one model from a checkout where nothing is built yet.
 """
 from __future__ import annotations
 
@@ -13,12 +16,17 @@ import subprocess
 import sys
 from concurrent.futures import ThreadPoolExecutor
 from pathlib import Path
-from typing import List
+from typing import List, Optional
 
 HERE = Path(__file__).resolve().parent
 CSRC = HERE / "csrc"
 BUILD_DIR = HERE / "_build"
 LIB_PATH = HERE / "libtgi_b200_kernels.so"
+KERNEL_SETS = {
+    # decoders in bf16 / fp32 on one GPU, with attention and recurrent layers
+    "decoder": ["attention_prefill_sm100", "attention_sm100", "fused_ops", "gemm_sm100", "gemm_static_scratch", "mixer_ops",
+                "recurrent_sm100"],
+}
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",
@@ -36,8 +44,14 @@ def nvcc_path() -> str:
     raise RuntimeError("nvcc not found; set NVCC or install the CUDA toolkit")
 
 
-def sources() -> List[Path]:
-    return sorted(CSRC.glob("*.cu"))
+def lib_path(kernel_set: Optional[str] = None) -> Path:
+    return LIB_PATH if kernel_set is None else HERE / f"libtgi_b200_{kernel_set}.so"
+
+
+def sources(kernel_set: Optional[str] = None) -> List[Path]:
+    if kernel_set is None:
+        return sorted(CSRC.glob("*.cu"))
+    return [CSRC / f"{name}.cu" for name in KERNEL_SETS[kernel_set]]
 
 
 def _stale(target: Path, deps: List[Path]) -> bool:
@@ -47,13 +61,14 @@ def _stale(target: Path, deps: List[Path]) -> bool:
     return any(d.stat().st_mtime > t for d in deps)
 
 
-def build(force: bool = False, verbose: bool = False, ptxas_info: bool = False) -> Path:
+def build(force: bool = False, verbose: bool = False, ptxas_info: bool = False, kernel_set: Optional[str] = None) -> Path:
+    target = lib_path(kernel_set)
     nvcc = nvcc_path()
     BUILD_DIR.mkdir(exist_ok=True)
     headers = sorted(CSRC.glob("*.cuh")) + sorted(CSRC.glob("*.h"))
     jobs = []
     objs = []
-    for src in sources():
+    for src in sources(kernel_set):
         obj = BUILD_DIR / (src.stem + ".o")
         objs.append(obj)
         if force or _stale(obj, [src] + headers):
@@ -74,11 +89,13 @@ def build(force: bool = False, verbose: bool = False, ptxas_info: bool = False) 
     if jobs:
         with ThreadPoolExecutor(max_workers=min(len(jobs), os.cpu_count() or 4)) as ex:
             list(ex.map(run, jobs))
-    if force or jobs or _stale(LIB_PATH, objs):
-        run([nvcc, "-shared", "-o", str(LIB_PATH), *map(str, objs), "-lcudart_static", "-ldl", "-lrt", "-lpthread"])
-    return LIB_PATH
+    if force or jobs or _stale(target, objs):
+        run([nvcc, "-shared", "-o", str(target), *map(str, objs), "-lcudart_static", "-ldl", "-lrt", "-lpthread"])
+    return target
 
 
 if __name__ == "__main__":
-    path = build(force="--force" in sys.argv, verbose=True, ptxas_info="--ptxas" in sys.argv)
+    named = [a for a in sys.argv[1:] if a in KERNEL_SETS]
+    path = build(force="--force" in sys.argv, verbose=True, ptxas_info="--ptxas" in sys.argv,
+                 kernel_set=named[0] if named else None)
     print(path)

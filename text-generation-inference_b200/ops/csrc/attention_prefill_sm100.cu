@@ -59,8 +59,17 @@ struct PrefillParams {
   int max_blocks, Hq, Hkv, num_blocks;
   float scale, softcap;
   int window;
+  int chunk;                    // > 0: a row sees only keys of its own chunk of `chunk` positions
+  int sink;                     // 1: the denominator counts one more key of score 0 that has no value
   int* status;
 };
+
+// First KV position that the query at `pos` may see.
+__device__ __forceinline__ int first_visible(const PrefillParams& p, int pos) {
+  int lo = p.window > 0 ? pos - p.window + 1 : 0;
+  if (p.chunk > 0 && pos > 0) lo = max(lo, pos - pos % p.chunk);
+  return max(lo, 0);
+}
 
 __device__ __forceinline__ void report(int* status, int code) {
   if (status != nullptr) atomicCAS(status, 0, code);
@@ -222,8 +231,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
   const int row_base = qt * kRows;
   const int pos_first = Lkv - n + row_base;
   const int pos_last = min(Lkv - 1, pos_first + kRows - 1);
-  int t_lo = 0;
-  if (p.window > 0) t_lo = max(0, pos_first - p.window + 1) / kKeys * kKeys;
+  const int t_lo = first_visible(p, pos_first) / kKeys * kKeys;
   const int t_hi = p.horizon != nullptr ? Lkv : pos_last + 1;
   const int ntiles = (t_hi - t_lo + kKeys - 1) / kKeys;
 
@@ -426,7 +434,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
     sa.cap_out = p.softcap * kLog2e;
     // visible keys of this row: [t_min, t_max]
     const int t_max = min(hz, Lkv - 1);
-    const int t_min = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+    const int t_min = first_visible(p, pos);
     float m = -INFINITY, l = 0.f;
     // The two threads of a row meet at a named barrier once per tile, so they must leave the loop together: a
     // thread whose wait ran out raises the quarter's flag of the NEXT barrier's parity and keeps walking to that
@@ -502,6 +510,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
       fail = true;
     }
     if (!fail) {
+      if (p.sink && hf == 0) l += exp2f(-m);      // both threads of a row hold the same maximum
       reinterpret_cast<float*>(smem + L::kP + (ntiles & 1) * kTileBytes)[hf * 128 + r] = l;
       __syncwarp();
       if (lane == 0) mbar_arrive(l_ready);
@@ -640,7 +649,8 @@ extern "C" {
 int tgi_prefill_attention_tc(const void* q, const void* k_cache, const void* v_cache, const int* block_tables,
                              const int* cu_seqlens_q, const int* kv_lens, const float* k_scale, const float* v_scale,
                              void* out, int B, int max_q, int max_blocks, int num_blocks, int Hq, int Hkv, float scale,
-                             float softcap, int window, int fp8_kv, const int* horizon, int* status, cudaStream_t stream) {
+                             float softcap, int window, int chunk, int sink, int fp8_kv, const int* horizon, int* status,
+                             cudaStream_t stream) {
   if (B <= 0 || max_q <= 0) return 0;
   if (Hq % Hkv != 0 || B > 65535 || Hq > 65535) return -10;
   PrefillParams p;
@@ -659,6 +669,8 @@ int tgi_prefill_attention_tc(const void* q, const void* k_cache, const void* v_c
   p.scale = scale;
   p.softcap = softcap;
   p.window = window;
+  p.chunk = chunk;
+  p.sink = sink;
   p.status = status;
   return fp8_kv ? launch_prefill<true>(p, k_cache, v_cache, B, max_q, stream)
                 : launch_prefill<false>(p, k_cache, v_cache, B, max_q, stream);

@@ -114,8 +114,19 @@ struct Params {
   int max_blocks, block_size, bs_shift, Hq, Hkv, num_blocks;   // block_size == 1 << bs_shift
   float scale, softcap;
   int window;
+  int chunk;                    // > 0: a row sees only keys of its own chunk of `chunk` positions
+  int sink;                     // 1: the softmax denominator counts one more key of score 0 that has no value
   int nsplit;
 };
+
+// First KV position that the query at `pos` may see.
+__device__ __forceinline__ int first_visible(const Params& p, int pos) {
+  int lo = p.window > 0 ? pos - p.window + 1 : 0;
+  if (p.chunk > 0 && pos > 0) lo = max(lo, pos - pos % p.chunk);
+  return max(lo, 0);
+}
+// exp(0 - m) for a running maximum kept in the log2 domain: the share of the sink in the denominator.
+__device__ __forceinline__ float sink_term(int sink, float m_log2) { return sink ? exp2f(-m_log2) : 0.f; }
 
 // Gather one 64-token K or V tile (tokens t0..t0+63 of sequence b, KV head kvh) into shared memory.
 // bf16 pages land directly in the swizzled compute tile; e4m3 pages land in a raw staging tile.
@@ -224,8 +235,10 @@ __device__ __forceinline__ float fast_exp2(float x) {   // ex2.approx: 2 ulp, -i
 
 template <int NT>
 __device__ __forceinline__ void softmax_update(float (&s)[NT][4], float (&m)[2], float (&l)[2], float (&alpha)[2],
-                                               int tbase, int pos0, int pos1, int L, int window, float scale_log2,
-                                               float softcap, float raw_scale, int hz0 = -1, int hz1 = -1) {
+                                               int tbase, int pos0, int pos1, int lo0, int lo1, int lo_max, int L,
+                                               float scale_log2, float softcap, float raw_scale, int hz0 = -1,
+                                               int hz1 = -1) {
+  // lo0 / lo1: first visible KV position of the two rows, lo_max: of the warp's last row
   // hz0 / hz1: last visible KV position of the two rows (defaults: their own positions, i.e. causal)
   if (hz0 < 0) hz0 = pos0;
   if (hz1 < 0) hz1 = pos1;
@@ -233,8 +246,8 @@ __device__ __forceinline__ void softmax_update(float (&s)[NT][4], float (&m)[2],
   float mx[2] = {-INFINITY, -INFINITY};
   // a tile that lies entirely below the diagonal of all 16 rows of the warp, inside the window and inside the
   // sequence needs no per-element mask (warp-uniform test: the warp's first row is pos0 - lane / 4)
-  const int row_lo = hz0 - (lane >> 2), row_hi = pos0 - (lane >> 2) + 15, t_last = tbase + NT * 8 - 1;
-  const bool plain = softcap <= 0.f && t_last <= row_lo && t_last < L && (window <= 0 || tbase > row_hi - window);
+  const int row_lo = hz0 - (lane >> 2), t_last = tbase + NT * 8 - 1;
+  const bool plain = softcap <= 0.f && t_last <= row_lo && t_last < L && tbase >= lo_max;
   if (plain) {
 #pragma unroll
     for (int i = 0; i < NT; ++i) {
@@ -249,12 +262,12 @@ __device__ __forceinline__ void softmax_update(float (&s)[NT][4], float (&m)[2],
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int t = tbase + i * 8 + (lane & 3) * 2 + (e & 1);
-        const int pos = (e < 2) ? pos0 : pos1;
+        const int lo = (e < 2) ? lo0 : lo1;
         const int hz = (e < 2) ? hz0 : hz1;
         float v = s[i][e];
         if (softcap > 0.f) v = softcap * tanhf(v * raw_scale / softcap) * kLog2e;
         else v = v * scale_log2;
-        const bool ok = t <= hz && t < L && (window <= 0 || t > pos - window);
+        const bool ok = t <= hz && t < L && t >= lo;
         v = ok ? v : -INFINITY;
         s[i][e] = v;
         mx[e >> 1] = fmaxf(mx[e >> 1], v);
@@ -324,8 +337,7 @@ prefill_kernel(Params p) {
   const int row_base = qt * kTile;                         // first query row of this CTA inside the chunk
   const int pos_first = L - n + row_base;
   const int pos_last = min(L - 1, pos_first + kTile - 1);
-  int t_lo = 0;
-  if (p.window > 0) t_lo = max(0, pos_first - p.window + 1) / kTile * kTile;
+  const int t_lo = first_visible(p, pos_first) / kTile * kTile;
   const int t_hi = p.horizon != nullptr ? L : pos_last + 1;   // exclusive; with horizons a row may see up to L - 1
   const int ntiles = (t_hi - t_lo + kTile - 1) / kTile;
 
@@ -373,6 +385,7 @@ prefill_kernel(Params p) {
   const float scale_log2 = raw_scale * kLog2e;
   const int pos0 = pos_first + warp * 16 + (lane >> 2);
   const int pos1 = pos0 + 8;
+  const int lo0 = first_visible(p, pos0), lo1 = first_visible(p, pos1), lo_max = first_visible(p, pos0 - (lane >> 2) + 15);
   int hz0 = pos0, hz1 = pos1;
   if (p.horizon != nullptr) {
     const int r0 = row_base + warp * 16 + (lane >> 2), r1 = r0 + 8;
@@ -406,8 +419,8 @@ prefill_kernel(Params p) {
     float s[8][4];
     qk_warp<D, 8, FP8>(qf, cK, 0, s);
     float alpha[2];
-    softmax_update<8>(s, m, l, alpha, t_lo + j * kTile, pos0, pos1, L, p.window, scale_log2, p.softcap, raw_scale,
-                      hz0, hz1);
+    softmax_update<8>(s, m, l, alpha, t_lo + j * kTile, pos0, pos1, lo0, lo1, lo_max, L, scale_log2, p.softcap,
+                      raw_scale, hz0, hz1);
 #pragma unroll
     for (int i = 0; i < D / 8; ++i) {
       o[i][0] *= alpha[0]; o[i][1] *= alpha[0];
@@ -418,8 +431,8 @@ prefill_kernel(Params p) {
   }
   cp_async_wait<0>();
 
-  const float inv0 = l[0] > 0.f ? (FP8 ? vs : 1.f) / l[0] : 0.f;
-  const float inv1 = l[1] > 0.f ? (FP8 ? vs : 1.f) / l[1] : 0.f;
+  const float inv0 = l[0] > 0.f ? (FP8 ? vs : 1.f) / (l[0] + sink_term(p.sink, m[0])) : 0.f;
+  const float inv1 = l[1] > 0.f ? (FP8 ? vs : 1.f) / (l[1] + sink_term(p.sink, m[1])) : 0.f;
   const int r0 = row_base + warp * 16 + (lane >> 2), r1 = r0 + 8;
 #pragma unroll
   for (int i = 0; i < D / 8; ++i) {
@@ -568,8 +581,8 @@ decode_kernel_v2(Params p) {
   const int q_row = p.cu_seqlens_q[b];
   if (p.cu_seqlens_q[b + 1] == q_row) return;   // sequence contributes no query this step
   const int pos = L - 1;
-  int t_lo = 0;
-  if (p.window > 0) t_lo = max(0, pos - p.window + 1) / CT * CT;
+  const int lo = first_visible(p, pos);
+  const int t_lo = lo / CT * CT;
   const int chunks_total = (L - t_lo + CT - 1) / CT;
   const int chunks_per = (chunks_total + p.nsplit - 1) / p.nsplit;
   const int c0 = split * chunks_per;
@@ -644,7 +657,7 @@ decode_kernel_v2(Params p) {
       cV = static_cast<const uint16_t*>(vstage(i % S::kStages));
     }
     float alpha[2];
-    softmax_update<NT>(s, m, l, alpha, t_lo + (c0 + warp + 4 * i) * CT, pos, pos, L, p.window, scale_log2, p.softcap,
+    softmax_update<NT>(s, m, l, alpha, t_lo + (c0 + warp + 4 * i) * CT, pos, pos, lo, lo, lo, L, scale_log2, p.softcap,
                        raw_scale);
 #pragma unroll
     for (int j = 0; j < D / 8; ++j) {
@@ -693,7 +706,7 @@ decode_kernel_v2(Params p) {
     }
     const int h = h0 + row;
     if (p.nsplit == 1) {
-      const float inv = ll > 0.f ? (FP8 ? vsc : 1.f) / ll : 0.f;
+      const float inv = ll > 0.f ? (FP8 ? vsc : 1.f) / (ll + sink_term(p.sink, mm)) : 0.f;
       p.out[(static_cast<size_t>(q_row) * p.Hq + h) * D + col] = __float2bfloat16(acc * inv);
     } else {
       const size_t pi = (static_cast<size_t>(b) * p.Hq + h) * p.nsplit + split;
@@ -788,8 +801,8 @@ decode_kernel_v3(Params p, const __grid_constant__ CUtensorMap tmK, const __grid
   const int q_row = p.cu_seqlens_q[b];
   if (p.cu_seqlens_q[b + 1] == q_row) return;   // sequence contributes no query this step
   const int pos = L - 1;
-  int t_lo = 0;
-  if (p.window > 0) t_lo = max(0, pos - p.window + 1) / CT * CT;
+  const int lo = first_visible(p, pos);
+  const int t_lo = lo / CT * CT;
   const int chunks_total = (L - t_lo + CT - 1) / CT;
   const int chunks_per = (chunks_total + p.nsplit - 1) / p.nsplit;
   const int c0 = split * chunks_per;
@@ -944,7 +957,7 @@ decode_kernel_v3(Params p, const __grid_constant__ CUtensorMap tmK, const __grid
 
     // ---- online softmax over the tokens of the chunk, per head ----
     // m[] is kept in the scaled log2 domain; a chunk that needs no masking takes the short path
-    const bool plain = p.softcap <= 0.f && tbase + CT <= L && (p.window <= 0 || tbase > pos - p.window);
+    const bool plain = p.softcap <= 0.f && tbase + CT <= L && tbase >= lo;
     float mx[2] = {-INFINITY, -INFINITY};
     if (plain) {
 #pragma unroll
@@ -963,7 +976,7 @@ decode_kernel_v3(Params p, const __grid_constant__ CUtensorMap tmK, const __grid
           float v = s[mt][e];
           if (p.softcap > 0.f) v = p.softcap * tanhf(v * raw_scale / p.softcap) * kLog2e;
           else v = v * scale_log2;
-          const bool ok = t < L && (p.window <= 0 || t > pos - p.window);
+          const bool ok = t < L && t >= lo;
           v = ok ? v : -INFINITY;
           s[mt][e] = v;
           mx[e & 1] = fmaxf(mx[e & 1], v);
@@ -1102,7 +1115,7 @@ decode_kernel_v3(Params p, const __grid_constant__ CUtensorMap tmK, const __grid
     }
     const int h = h0 + row;
     if (p.nsplit == 1) {
-      const float inv = ll > 0.f ? (FP8 ? vsc : 1.f) / ll : 0.f;
+      const float inv = ll > 0.f ? (FP8 ? vsc : 1.f) / (ll + sink_term(p.sink, mm)) : 0.f;
       p.out[(static_cast<size_t>(q_row) * p.Hq + h) * D + col] = __float2bfloat16(acc * inv);
     } else {
       const size_t pi = (static_cast<size_t>(b) * p.Hq + h) * p.nsplit + split;
@@ -1118,7 +1131,7 @@ decode_kernel_v3(Params p, const __grid_constant__ CUtensorMap tmK, const __grid
 // merge split partials: grid (B, Hq), block D
 __global__ void decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                     const int* __restrict__ cu_seqlens_q, __nv_bfloat16* __restrict__ out, int Hq,
-                                    int D, int nsplit) {
+                                    int D, int nsplit, int sink) {
   tgi::pdl_wait();
   tgi::pdl_trigger();
   const int b = blockIdx.x, h = blockIdx.y;
@@ -1139,7 +1152,7 @@ __global__ void decode_merge_kernel(const float* __restrict__ part_o, const floa
         wsum += w;
       }
     }
-    out[(static_cast<size_t>(cu_seqlens_q[b]) * Hq + h) * D + col] = __float2bfloat16(wsum > 0.f ? acc / wsum : 0.f);
+    out[(static_cast<size_t>(cu_seqlens_q[b]) * Hq + h) * D + col] = __float2bfloat16(wsum > 0.f ? acc / (wsum + sink_term(sink, mm)) : 0.f);
   }
 }
 
@@ -1206,7 +1219,7 @@ int launch_v3_cfg(const Params& p, int B, cudaStream_t stream) {
   if (p.nsplit > 1) {
     dim3 g2(B, p.Hq);
     tgi::launch(decode_merge_kernel, dim3(g2), dim3(128), 0, stream, p.part_o, p.part_ml, p.cu_seqlens_q, p.out, p.Hq,
-                128, p.nsplit);
+                128, p.nsplit, p.sink);
   }
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
@@ -1247,8 +1260,8 @@ int launch_v3(const Params& p, int B, cudaStream_t stream) {
 extern "C" int tgi_prefill_attention_tc(const void* q, const void* k_cache, const void* v_cache, const int* block_tables,
                                         const int* cu_seqlens_q, const int* kv_lens, const float* k_scale,
                                         const float* v_scale, void* out, int B, int max_q, int max_blocks, int num_blocks,
-                                        int Hq, int Hkv, float scale, float softcap, int window, int fp8_kv,
-                                        const int* horizon, int* status, cudaStream_t stream);
+                                        int Hq, int Hkv, float scale, float softcap, int window, int chunk, int sink,
+                                        int fp8_kv, const int* horizon, int* status, cudaStream_t stream);
 
 bool prefill_tc_enabled() {
   static const bool on = [] {
@@ -1267,7 +1280,7 @@ int launch(const Params& p, int B, int max_q, cudaStream_t stream) {
     if (cudaGetSymbolAddress(reinterpret_cast<void**>(&status), g_attn_status) != cudaSuccess) return -2;
     return tgi_prefill_attention_tc(p.q, p.k_cache, p.v_cache, p.block_tables, p.cu_seqlens_q, p.kv_lens, p.k_scale,
                                     p.v_scale, p.out, B, max_q, p.max_blocks, p.num_blocks, p.Hq, p.Hkv, p.scale, p.softcap,
-                                    p.window, FP8 ? 1 : 0, p.horizon, status, stream);
+                                    p.window, p.chunk, p.sink, FP8 ? 1 : 0, p.horizon, status, stream);
   }
   if (max_q > 1) {
     auto k = prefill_kernel<D, FP8>;
@@ -1296,7 +1309,7 @@ int launch(const Params& p, int B, int max_q, cudaStream_t stream) {
     if (p.nsplit > 1) {
       dim3 g2(B, p.Hq);
       tgi::launch(decode_merge_kernel, dim3(g2), dim3(D < 128 ? D : 128), 0, stream, p.part_o, p.part_ml, p.cu_seqlens_q, p.out, p.Hq, D,
-                                                                p.nsplit);
+                                                                p.nsplit, p.sink);
     }
   }
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
@@ -1338,12 +1351,14 @@ int tgi_attn_status(int reset) {
   return v;
 }
 
-// `horizon` (optional, prefill only): per query row the last KV position it may attend to; null = causal
+// `horizon` (optional, prefill only): per query row the last KV position it may attend to; null = causal.
+// `chunk` > 0: rows see only keys of their own chunk of `chunk` positions, counted from position 0.
+// `sink` != 0: exp(0) is added to every softmax denominator.
 int tgi_paged_attention_ex(const void* q, const void* k_cache, const void* v_cache, const int* block_tables,
                            const int* cu_seqlens_q, const int* kv_lens, const float* k_scale, const float* v_scale,
                            void* out, float* part_o, float* part_ml, int B, int max_q, int max_blocks, int block_size,
-                           int num_blocks, int Hq, int Hkv, int D, float scale, float softcap, int window, int nsplit,
-                           int fp8_kv, const int* horizon, cudaStream_t stream);
+                           int num_blocks, int Hq, int Hkv, int D, float scale, float softcap, int window, int chunk,
+                           int sink, int nsplit, int fp8_kv, const int* horizon, cudaStream_t stream);
 
 int tgi_paged_attention(const void* q, const void* k_cache, const void* v_cache, const int* block_tables,
                         const int* cu_seqlens_q, const int* kv_lens, const float* k_scale, const float* v_scale,
@@ -1352,14 +1367,14 @@ int tgi_paged_attention(const void* q, const void* k_cache, const void* v_cache,
                         int fp8_kv, cudaStream_t stream) {
   return tgi_paged_attention_ex(q, k_cache, v_cache, block_tables, cu_seqlens_q, kv_lens, k_scale, v_scale, out, part_o,
                                 part_ml, B, max_q, max_blocks, block_size, num_blocks, Hq, Hkv, D, scale, softcap, window,
-                                nsplit, fp8_kv, nullptr, stream);
+                                0, 0, nsplit, fp8_kv, nullptr, stream);
 }
 
 int tgi_paged_attention_ex(const void* q, const void* k_cache, const void* v_cache, const int* block_tables,
                            const int* cu_seqlens_q, const int* kv_lens, const float* k_scale, const float* v_scale,
                            void* out, float* part_o, float* part_ml, int B, int max_q, int max_blocks, int block_size,
-                           int num_blocks, int Hq, int Hkv, int D, float scale, float softcap, int window, int nsplit,
-                           int fp8_kv, const int* horizon, cudaStream_t stream) {
+                           int num_blocks, int Hq, int Hkv, int D, float scale, float softcap, int window, int chunk,
+                           int sink, int nsplit, int fp8_kv, const int* horizon, cudaStream_t stream) {
   if (B <= 0 || max_q <= 0) return 0;
   if (Hq % Hkv != 0) return -10;
   Params p;
@@ -1386,6 +1401,8 @@ int tgi_paged_attention_ex(const void* q, const void* k_cache, const void* v_cac
   p.scale = scale;
   p.softcap = softcap;
   p.window = window;
+  p.chunk = chunk;
+  p.sink = sink;
   p.nsplit = (max_q > 1 || nsplit < 1) ? 1 : nsplit;
   if (p.nsplit > 1 && (part_o == nullptr || part_ml == nullptr)) return -11;
   switch (D) {

@@ -723,7 +723,7 @@ int g_streamk_small = 0;   // 1: problems with fewer tiles than workers may also
 
 template <int MH, int TN, int STAGES, bool FP8, bool PAIR, bool MX = false>
 int launch(const void* X, const float* xs_t, int xs_pitch, const void* W, const float* wscale, void* C,
-           const void* bias, int M, int N, int K, int max_ctas, float* ws, int* counters, int* status,
+           const void* bias, int M, int N, int K, int ldx, int max_ctas, float* ws, int* counters, int* status,
            cudaStream_t stream, const PushArgs* push_args = nullptr) {
   using Cfg = TileCfg<MH, TN, PAIR, FP8, MX>;
   PushArgs push;
@@ -739,7 +739,8 @@ int launch(const void* X, const float* xs_t, int xs_pitch, const void* W, const 
   // both operands are fetched in boxes of 128 rows x 128 bytes (one swizzle atom wide)
   int rc = make_map_2d(&tmW, dt, W, N, K, pitch, 128, BK, CU_TENSOR_MAP_SWIZZLE_128B);
   if (rc) return rc;
-  rc = make_map_2d(&tmX, dt, X, M, K, pitch, 128, BK, CU_TENSOR_MAP_SWIZZLE_128B);
+  const uint64_t pitch_x = static_cast<uint64_t>(ldx) * (FP8 ? 1 : 2);     // X may be a column slice of a wider matrix
+  rc = make_map_2d(&tmX, dt, X, M, K, pitch_x, 128, BK, CU_TENSOR_MAP_SWIZZLE_128B);
   if (rc) return rc;
   if (FP8) {
     rc = make_map_2d(&tmS, CU_TENSOR_MAP_DATA_TYPE_FLOAT32, xs_t, K / 128, M, static_cast<uint64_t>(xs_pitch) * 4, 1,
@@ -854,11 +855,11 @@ static int g_mx_pairs = 1;        // CTA pairs in the block-scaled mode
 namespace {
 template <bool FP8>
 int dispatch(const void* X, const float* xs_t, int xs_pitch, const void* W, const float* wscale, void* C, const void* bias,
-             int M, int N, int K, int max_ctas, float* ws, int* counters, int* status, cudaStream_t stream,
+             int M, int N, int K, int ldx, int max_ctas, float* ws, int* counters, int* status, cudaStream_t stream,
              const PushArgs* push) {
   if (FP8 && g_fp8_mx) {
     if (M <= g_wide_m)
-      return launch<1, 256, 4, FP8, false, FP8>(X, xs_t, xs_pitch, W, wscale, C, bias, M, N, K, max_ctas, ws, counters,
+      return launch<1, 256, 4, FP8, false, FP8>(X, xs_t, xs_pitch, W, wscale, C, bias, M, N, K, ldx, max_ctas, ws, counters,
                                                  status, stream, push);
     const long long mx_pair_tiles = static_cast<long long>((N + 255) / 256) * ((M + 255) / 256);
     // pairs need enough work to repay their fixed cost: 256 x 8192 x 4096 (32 tiles of 32 K blocks) takes 30.7 us in
@@ -867,26 +868,26 @@ int dispatch(const void* X, const float* xs_t, int xs_pitch, const void* W, cons
     const long long mx_pair_units = mx_pair_tiles * ((K + 127) / 128);
     if (g_pairs && g_mx_pairs && max_ctas >= 2 && mx_pair_tiles >= g_pair_min_tiles &&
         (mx_pair_units >= 2048 || g_pair_min_tiles < 32)) {
-      const int rc = launch<1, 256, 6, FP8, FP8, FP8>(X, xs_t, xs_pitch, W, wscale, C, bias, M, N, K, max_ctas, ws, counters,
+      const int rc = launch<1, 256, 6, FP8, FP8, FP8>(X, xs_t, xs_pitch, W, wscale, C, bias, M, N, K, ldx, max_ctas, ws, counters,
                                                        status, stream, push);
       if (rc != -4) return rc;
     }
-    return launch<2, 128, 4, FP8, false, FP8>(X, xs_t, xs_pitch, W, wscale, C, bias, M, N, K, max_ctas, ws, counters, status,
+    return launch<2, 128, 4, FP8, false, FP8>(X, xs_t, xs_pitch, W, wscale, C, bias, M, N, K, ldx, max_ctas, ws, counters, status,
                                                stream, push);
   }
   if (M <= g_wide_m)
-    return launch<1, 256, 4, FP8, false>(X, xs_t, xs_pitch, W, wscale, C, bias, M, N, K, max_ctas, ws, counters, status,
+    return launch<1, 256, 4, FP8, false>(X, xs_t, xs_pitch, W, wscale, C, bias, M, N, K, ldx, max_ctas, ws, counters, status,
                                          stream, push);
   // Pairs pay off when there are enough 256 x 256 tiles to go round: with few tiles (tensor-parallel shards, narrow
   // projections) the 74 pairs split K deeper than 148 single CTAs on 256 x 128 tiles do, and the fix-up of split
   // tiles costs more than the saved operand traffic (measured: 256 x 7168 x 8192 51 us in pairs, 48 us without).
   const long long pair_tiles = static_cast<long long>((N + 255) / 256) * ((M + 255) / 256);
   if (g_pairs && max_ctas >= 2 && pair_tiles >= g_pair_min_tiles) {
-    const int rc = launch<1, 256, 6, FP8, true>(X, xs_t, xs_pitch, W, wscale, C, bias, M, N, K, max_ctas, ws, counters,
+    const int rc = launch<1, 256, 6, FP8, true>(X, xs_t, xs_pitch, W, wscale, C, bias, M, N, K, ldx, max_ctas, ws, counters,
                                                 status, stream, push);
     if (rc != -4) return rc;   // -4: this device cannot place a pair; fall back to single CTAs
   }
-  return launch<2, 128, 4, FP8, false>(X, xs_t, xs_pitch, W, wscale, C, bias, M, N, K, max_ctas, ws, counters, status,
+  return launch<2, 128, 4, FP8, false>(X, xs_t, xs_pitch, W, wscale, C, bias, M, N, K, ldx, max_ctas, ws, counters, status,
                                        stream, push);
 }
 }  // namespace
@@ -924,7 +925,15 @@ int tgi_gemm_bf16(const void* X, const void* W, void* C, const void* bias, int M
                   float* ws, int* counters, int* status, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (K % 8 != 0) return -10;  // TMA row pitch must be a multiple of 16 bytes
-  return dispatch<false>(X, nullptr, 0, W, nullptr, C, bias, M, N, K, max_ctas, ws, counters, status, stream, nullptr);
+  return dispatch<false>(X, nullptr, 0, W, nullptr, C, bias, M, N, K, K, max_ctas, ws, counters, status, stream, nullptr);
+}
+
+// The same with rows of X `ldx` elements apart (X is a column slice of a wider matrix, 16-byte aligned).
+int tgi_gemm_bf16_ld(const void* X, int ldx, const void* W, void* C, const void* bias, int M, int N, int K, int max_ctas,
+                     float* ws, int* counters, int* status, cudaStream_t stream) {
+  if (M <= 0 || N <= 0) return 0;
+  if (K % 8 != 0 || ldx % 8 != 0 || ldx < K) return -10;
+  return dispatch<false>(X, nullptr, 0, W, nullptr, C, bias, M, N, K, ldx, max_ctas, ws, counters, status, stream, nullptr);
 }
 
 int tgi_gemm_fp8_block(const void* X, const float* xs_t, int xs_pitch, const void* W, const float* wscale, void* C,
@@ -932,7 +941,7 @@ int tgi_gemm_fp8_block(const void* X, const float* xs_t, int xs_pitch, const voi
                        cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (K % 128 != 0 || xs_pitch % 4 != 0) return -10;
-  return dispatch<true>(X, xs_t, xs_pitch, W, wscale, C, bias, M, N, K, max_ctas, ws, counters, status, stream, nullptr);
+  return dispatch<true>(X, xs_t, xs_pitch, W, wscale, C, bias, M, N, K, K, max_ctas, ws, counters, status, stream, nullptr);
 }
 
 // Row-parallel GEMMs of a tensor-parallel group: same products, but every output row is stored into the
@@ -949,10 +958,10 @@ int tgi_gemm_push(int fp8, const void* X, const float* xs_t, int xs_pitch, const
   if (rc) return rc;
   if (fp8) {
     if (K % 128 != 0 || xs_pitch % 4 != 0) return -10;
-    return dispatch<true>(X, xs_t, xs_pitch, W, wscale, nullptr, bias, M, N, K, max_ctas, ws, counters, status, stream, &p);
+    return dispatch<true>(X, xs_t, xs_pitch, W, wscale, nullptr, bias, M, N, K, K, max_ctas, ws, counters, status, stream, &p);
   }
   if (K % 8 != 0) return -10;
-  return dispatch<false>(X, nullptr, 0, W, nullptr, nullptr, bias, M, N, K, max_ctas, ws, counters, status, stream, &p);
+  return dispatch<false>(X, nullptr, 0, W, nullptr, nullptr, bias, M, N, K, K, max_ctas, ws, counters, status, stream, &p);
 }
 
 }  // extern "C"

@@ -1,0 +1,681 @@
+// Kernels around the token mixers of hybrid decoders (attention layers between recurrent ones), each in a bf16 and
+// an fp32 build of the activations:
+//   residual add (fp32 stream) + RMSNorm, optional row gather
+//   embedding gather into the fp32 residual stream
+//   element-wise activation of a non-gated feed-forward
+//   RoPE -> per-head RMS of q and k -> value mixing -> paged K / V store
+//   paged attention for any head size and for fp32 pages (the tensor-core kernels serve bf16 at 64 / 128 / 256)
+//   causal short convolution + SiLU, unit norms, decays and write strengths of a gated delta rule
+//   per-group RMSNorm x weight x sigmoid(gate) on the output of a recurrent mixer
+//
+// Norms, angles, scores, decays and the residual stream are fp32 in both builds; only matrix operands and what the
+// matrix products return are bf16.
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+#include <stdint.h>
+
+#include "launch.cuh"
+
+namespace {
+
+using bf16 = __nv_bfloat16;
+
+__device__ __forceinline__ float to_f(float x) { return x; }
+__device__ __forceinline__ float to_f(bf16 x) { return __bfloat162float(x); }
+__device__ __forceinline__ void put(float* p, float v) { *p = v; }
+__device__ __forceinline__ void put(bf16* p, float v) { *p = __float2bfloat16(v); }
+// four consecutive elements (16-byte aligned fp32, 8-byte aligned bf16)
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4(const bf16* p) {
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(bf16* p, float4 v) {
+  __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+  uint2 u;
+  u.x = *reinterpret_cast<uint32_t*>(&a);
+  u.y = *reinterpret_cast<uint32_t*>(&b);
+  *reinterpret_cast<uint2*>(p) = u;
+}
+
+__device__ __forceinline__ float warp_sum(float v) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  return v;
+}
+// sum over the block, returned to every thread; `red` holds one float per warp plus the total
+__device__ __forceinline__ float block_sum(float v, float* red) {
+  v = warp_sum(v);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float t = 0.f;
+  for (int w = 0; w < static_cast<int>(blockDim.x >> 5); ++w) t += red[w];
+  __syncthreads();
+  return t;
+}
+__device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
+__device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
+
+// sequence that owns token t (cu[0] = 0 .. cu[B] = T)
+__device__ __forceinline__ int sequence_of(const int* __restrict__ cu, int B, int t) {
+  int lo = 0, hi = B - 1;
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) >> 1;
+    if (cu[mid] <= t) lo = mid;
+    else hi = mid - 1;
+  }
+  return lo;
+}
+
+// ------------------------------------------------------------------------------------------------
+// residual (fp32) + delta -> RMSNorm.  One CTA per output row; `rows` (optional) picks the input row.
+// VPT float4 per thread stay in registers; VPT == 0: any width, the row is read twice.
+// ------------------------------------------------------------------------------------------------
+template <typename T, int VPT>
+__global__ void __launch_bounds__(1024)
+residual_norm_kernel(const T* __restrict__ delta, const float* __restrict__ residual, const int* __restrict__ rows,
+                     const T* __restrict__ weight, T* __restrict__ out, float* __restrict__ res_out, int H, float eps) {
+  tgi::pdl_wait();
+  tgi::pdl_trigger();
+  __shared__ float red[33];
+  const int row = rows != nullptr ? rows[blockIdx.x] : blockIdx.x;
+  const size_t in = static_cast<size_t>(row) * H, ob = static_cast<size_t>(blockIdx.x) * H;
+  float sumsq = 0.f;
+  if (VPT > 0) {
+    float4 x[VPT > 0 ? VPT : 1];
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = (threadIdx.x + i * blockDim.x) * 4;
+      if (c < H) {
+        float4 a = *reinterpret_cast<const float4*>(residual + in + c);
+        if (delta != nullptr) {
+          const float4 d = load4(delta + in + c);
+          a.x += d.x; a.y += d.y; a.z += d.z; a.w += d.w;
+        }
+        if (res_out != nullptr) store4(res_out + ob + c, a);
+        x[i] = a;
+        sumsq += a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;
+      }
+    }
+    const float inv = 1.f / sqrtf(block_sum(sumsq, red) / H + eps);
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = (threadIdx.x + i * blockDim.x) * 4;
+      if (c < H) {
+        const float4 w = load4(weight + c);
+        store4(out + ob + c, make_float4(x[i].x * inv * w.x, x[i].y * inv * w.y, x[i].z * inv * w.z, x[i].w * inv * w.w));
+      }
+    }
+  } else {
+    for (int c = threadIdx.x; c < H; c += blockDim.x) {
+      float a = residual[in + c];
+      if (delta != nullptr) a += to_f(delta[in + c]);
+      if (res_out != nullptr) res_out[ob + c] = a;
+      sumsq += a * a;
+    }
+    const float inv = 1.f / sqrtf(block_sum(sumsq, red) / H + eps);
+    for (int c = threadIdx.x; c < H; c += blockDim.x) {
+      float a = residual[in + c];
+      if (delta != nullptr) a += to_f(delta[in + c]);
+      put(out + ob + c, a * inv * to_f(weight[c]));
+    }
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+embed_residual_kernel(const int* __restrict__ ids, const T* __restrict__ table, float* __restrict__ out, int H, int vocab,
+                      float scale) {
+  tgi::pdl_wait();
+  tgi::pdl_trigger();
+  const int id = min(max(ids[blockIdx.x], 0), vocab - 1);
+  const T* src = table + static_cast<size_t>(id) * H;
+  float* dst = out + static_cast<size_t>(blockIdx.x) * H;
+  if (H % 4 == 0) {
+    for (int c = threadIdx.x * 4; c < H; c += blockDim.x * 4) {
+      float4 v = load4(src + c);
+      store4(dst + c, make_float4(v.x * scale, v.y * scale, v.z * scale, v.w * scale));
+    }
+  } else {
+    for (int c = threadIdx.x; c < H; c += blockDim.x) dst[c] = to_f(src[c]) * scale;
+  }
+}
+
+// ------------------------------------------------------------------------------------------------
+// element-wise activation (codes as in the gated kernel: 0 silu, 1 gelu erf, 2 gelu tanh, 3 relu, 4 quick gelu)
+// ------------------------------------------------------------------------------------------------
+__device__ __forceinline__ float act_value(float x, int act) {
+  switch (act) {
+    case 0: return silu_f(x);
+    case 1: return 0.5f * x * (1.f + erff(x * 0.70710678118654752f));
+    case 2: return 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
+    case 3: return fmaxf(x, 0.f);
+    default: return x / (1.f + expf(-1.702f * x));
+  }
+}
+template <typename T>
+__global__ void __launch_bounds__(256)
+activation_kernel(const T* __restrict__ in, T* __restrict__ out, long long n, int act) {
+  tgi::pdl_wait();
+  tgi::pdl_trigger();
+  const long long stride = static_cast<long long>(gridDim.x) * blockDim.x;
+  const long long first = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x;
+  const long long n4 = n / 4;
+  for (long long i = first; i < n4; i += stride) {
+    const float4 v = load4(in + i * 4);
+    store4(out + i * 4, make_float4(act_value(v.x, act), act_value(v.y, act), act_value(v.z, act), act_value(v.w, act)));
+  }
+  for (long long i = n4 * 4 + first; i < n; i += stride) put(out + i, act_value(to_f(in[i]), act));
+}
+
+// ------------------------------------------------------------------------------------------------
+// Attention inputs.  proj[T, ld] holds q (Hq heads of `dim`), k (Hkv of `dim`) and v (Hkv of `vdim`) at columns
+// 0, off_k, off_v.  One warp per (token, head): rotate the first `rot` dimensions (pairs i, i + rot / 2), divide q
+// and k by their root mean square over the head, mix v with the values of an earlier layer, and store k / v at the
+// token's slot.  q_out rows are Dk wide; columns past `dim` are zeroed.  The page pools are zero there already.
+// ------------------------------------------------------------------------------------------------
+template <typename T>
+__global__ void __launch_bounds__(256)
+attn_prep_kernel(const T* __restrict__ proj, long long ld, int off_k, int off_v, const int* __restrict__ positions,
+                 const float* __restrict__ cos_sin, const int* __restrict__ slots, const T* __restrict__ v_first,
+                 long long ld_first, float lambda, T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache,
+                 T* __restrict__ v_mixed, int T_, int Hq, int Hkv, int dim, int vdim, int Dk, int Dv, int rot, int max_pos,
+                 long long num_slots, int qk_norm, float eps) {
+  tgi::pdl_wait();
+  tgi::pdl_trigger();
+  const int lane = threadIdx.x & 31;
+  const int heads = Hq + 2 * Hkv;
+  const long long job = static_cast<long long>(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (job >= static_cast<long long>(T_) * heads) return;
+  const int t = static_cast<int>(job / heads), h = static_cast<int>(job % heads);
+  const long long slot = slots[t];
+  const bool slot_ok = slot >= 0 && slot < num_slots;      // padding rows have slot -1
+  const T* row = proj + static_cast<size_t>(t) * ld;
+  if (h >= Hq + Hkv) {
+    const int g = h - Hq - Hkv;
+    if (!slot_ok && v_mixed == nullptr) return;
+    const T* v = row + off_v + static_cast<size_t>(g) * vdim;
+    const T* f = v_first != nullptr ? v_first + static_cast<size_t>(t) * ld_first + static_cast<size_t>(g) * vdim : nullptr;
+    for (int i = lane; i < vdim; i += 32) {
+      float x = to_f(v[i]);
+      if (f != nullptr) x = (1.f - lambda) * x + lambda * to_f(f[i]);
+      if (slot_ok) put(v_cache + (static_cast<size_t>(slot) * Hkv + g) * Dv + i, x);
+      if (v_mixed != nullptr) put(v_mixed + (static_cast<size_t>(t) * Hkv + g) * vdim + i, x);
+    }
+    return;
+  }
+  const bool is_q = h < Hq;
+  const int g = is_q ? h : h - Hq;
+  const T* x = row + (is_q ? 0 : off_k) + static_cast<size_t>(g) * dim;
+  const int pos = min(max(positions[t], 0), max_pos - 1);
+  const float* cs = cos_sin + static_cast<size_t>(pos) * rot;
+  const int rh = rot / 2;
+  float ss = 0.f;
+  for (int i = lane; i < rh; i += 32) {
+    const float u = to_f(x[i]), w = to_f(x[i + rh]), c = cs[i], s = cs[rh + i];
+    const float a = u * c - w * s, b = w * c + u * s;
+    ss += a * a + b * b;
+  }
+  for (int i = rot + lane; i < dim; i += 32) {
+    const float a = to_f(x[i]);
+    ss += a * a;
+  }
+  const float inv = qk_norm ? 1.f / sqrtf(warp_sum(ss) / dim + eps) : 1.f;
+  if (!is_q && !slot_ok) return;
+  T* dst = is_q ? q_out + (static_cast<size_t>(t) * Hq + g) * Dk : k_cache + (static_cast<size_t>(slot) * Hkv + g) * Dk;
+  for (int i = lane; i < rh; i += 32) {
+    const float u = to_f(x[i]), w = to_f(x[i + rh]), c = cs[i], s = cs[rh + i];
+    put(dst + i, (u * c - w * s) * inv);
+    put(dst + i + rh, (w * c + u * s) * inv);
+  }
+  for (int i = rot + lane; i < dim; i += 32) put(dst + i, to_f(x[i]) * inv);
+  if (is_q)
+    for (int i = dim + lane; i < Dk; i += 32) put(dst + i, 0.f);
+}
+
+// ------------------------------------------------------------------------------------------------
+// Paged attention for any head size, fp32 arithmetic.  One warp per (token, query head): each lane scores one key
+// of a group of 32, the group's softmax is exchanged by shuffles, and the lanes then split the value dimensions.
+// ------------------------------------------------------------------------------------------------
+constexpr int kAttnWarps = 4;
+constexpr int kMaxOut = 16;        // value dimensions per lane: vdim <= 512
+template <typename T, int NV>
+__global__ void __launch_bounds__(kAttnWarps * 32)
+attn_any_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
+                const int* __restrict__ block_tables, const int* __restrict__ cu, const int* __restrict__ kv_lens,
+                T* __restrict__ out, int T_, int B, int max_blocks, int bs_shift, int Hq, int Hkv, int Dk, int Dv, float scale,
+                int window, int chunk, int sink) {
+  tgi::pdl_wait();
+  tgi::pdl_trigger();
+  extern __shared__ float sq[];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  float* qs = sq + warp * Dk;
+  const long long job = static_cast<long long>(blockIdx.x) * kAttnWarps + warp;
+  if (job >= static_cast<long long>(T_) * Hq) return;
+  const int t = static_cast<int>(job / Hq), h = static_cast<int>(job % Hq);
+  const int b = sequence_of(cu, B, t);
+  const int L = kv_lens[b], n = cu[b + 1] - cu[b];
+  const int pos = L - n + (t - cu[b]);
+  const int kvh = h / (Hq / Hkv);
+  for (int i = lane; i < Dk; i += 32) qs[i] = to_f(q[(static_cast<size_t>(t) * Hq + h) * Dk + i]);
+  __syncwarp();
+  int lo = window > 0 ? pos - window + 1 : 0;
+  if (chunk > 0 && pos > 0) lo = max(lo, pos - pos % chunk);
+  lo = max(lo, 0);
+  float m = sink ? 0.f : -INFINITY, l = sink ? 1.f : 0.f;
+  float o[NV];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) o[i] = 0.f;
+  const int* table = block_tables + static_cast<size_t>(b) * max_blocks;
+  for (int t0 = lo; t0 <= pos; t0 += 32) {
+    const int key = t0 + lane;
+    long long row = 0;
+    float s = -INFINITY;
+    if (key <= pos) {
+      row = (static_cast<long long>(table[key >> bs_shift]) << bs_shift) + (key & ((1 << bs_shift) - 1));
+      const T* kp = k_cache + (static_cast<size_t>(row) * Hkv + kvh) * Dk;
+      float acc = 0.f;
+      int i = 0;
+      if (Dk % 4 == 0) {
+        float a0 = 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f;
+        for (; i < Dk; i += 4) {
+          const float4 kv = load4(kp + i);
+          a0 = fmaf(kv.x, qs[i], a0);
+          a1 = fmaf(kv.y, qs[i + 1], a1);
+          a2 = fmaf(kv.z, qs[i + 2], a2);
+          a3 = fmaf(kv.w, qs[i + 3], a3);
+        }
+        acc = (a0 + a1) + (a2 + a3);
+      }
+      for (; i < Dk; ++i) acc = fmaf(to_f(kp[i]), qs[i], acc);
+      s = acc * scale;
+    }
+    float mx = s;
+#pragma unroll
+    for (int d = 16; d > 0; d >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
+    const float mn = fmaxf(m, mx);
+    const float alpha = expf(m - mn);                 // m = -inf only before the first group: exp(-inf) = 0
+    const float pr = expf(s - mn);
+    l = l * alpha + warp_sum(pr);
+    m = mn;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) o[i] *= alpha;
+    const int cnt = min(32, pos - t0 + 1);
+    for (int j = 0; j < cnt; ++j) {
+      const float pj = __shfl_sync(0xffffffffu, pr, j);
+      const long long rj = __shfl_sync(0xffffffffu, row, j);
+      const T* vp = v_cache + (static_cast<size_t>(rj) * Hkv + kvh) * Dv;
+#pragma unroll
+      for (int i = 0; i < NV; ++i)
+        if (lane + 32 * i < Dv) o[i] = fmaf(pj, to_f(vp[lane + 32 * i]), o[i]);
+    }
+  }
+  const float inv = l > 0.f ? 1.f / l : 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i)
+    if (lane + 32 * i < Dv) put(out + (static_cast<size_t>(t) * Hq + h) * Dv + lane + 32 * i, o[i] * inv);
+}
+
+// ------------------------------------------------------------------------------------------------
+// Inputs of a gated delta rule.  proj[T, ld]: q and k (G heads of dim), v (H of vdim), b (H) at off_q .. off_b;
+// decay[T, ld_a]: pre-activations of the decays (H x dim).  One warp per (token, unit):
+//   units 0 .. G-1            q and k of a head: convolution, SiLU, unit norm (q also times dim^-1/2), and q . k
+//   units G .. G+H-1          v of a head: convolution, SiLU; write strength sigmoid(b)
+//   units G+H .. G+2H-1       decay exp(-exp(A_log) softplus(a + dt_bias)) of every key channel
+// q, k and the decays are written with `dimP` columns per head, zero padded.  The convolution reads the previous
+// taps - 1 inputs from the step's rows or, before them, from the sequence's state [taps - 1][C] (C = (2 G dim + H vdim)
+// channels, oldest first); a sequence that starts at position 0 has zeros there.  With `update` (every sequence
+// contributes at most one token) the state is shifted here, otherwise conv_state_kernel does it afterwards.
+// ------------------------------------------------------------------------------------------------
+struct DeltaPrep {
+  long long ld, ld_a;
+  int off_q, off_k, off_v, off_b;
+  int B, G, H, dim, dimP, vdim, taps, update;
+};
+
+// convolved value of channel `c` (column `col` of proj) for the token at row t, local index i of its sequence
+template <typename T>
+__device__ __forceinline__ float conv_value(const T* __restrict__ proj, long long ld, int col, int t, int i,
+                                            const float* __restrict__ w, const T* __restrict__ st, int C, int c,
+                                            int taps) {
+  float acc = 0.f;
+  for (int j = 0; j < taps - 1; ++j) {             // tap j multiplies the input taps - 1 - j tokens back
+    const int back = taps - 1 - j;
+    float v = 0.f;
+    if (i >= back) {
+      v = to_f(proj[static_cast<size_t>(t - back) * ld + col]);
+    } else if (st != nullptr) {
+      v = to_f(st[static_cast<size_t>(taps - 1 + i - back) * C + c]);
+    }
+    acc = fmaf(w[j], v, acc);
+  }
+  return fmaf(w[taps - 1], to_f(proj[static_cast<size_t>(t) * ld + col]), acc);
+}
+
+template <typename T, int NV>
+__global__ void __launch_bounds__(256)
+delta_prep_kernel(const T* __restrict__ proj, const T* __restrict__ a_pre, const float* __restrict__ conv_q,
+                  const float* __restrict__ conv_k, const float* __restrict__ conv_v, const float* __restrict__ A_log,
+                  const float* __restrict__ dt_bias, const int* __restrict__ cu, const int* __restrict__ kv_lens,
+                  const int* __restrict__ state_slots, T* __restrict__ conv_state, float* __restrict__ q_out,
+                  float* __restrict__ k_out, float* __restrict__ v_out, float* __restrict__ g_out,
+                  float* __restrict__ beta_out, float* __restrict__ qk_out, int T_, int num_slots, DeltaPrep p) {
+  tgi::pdl_wait();
+  tgi::pdl_trigger();
+  const int lane = threadIdx.x & 31;
+  const int units = p.G + 2 * p.H;
+  const long long job = static_cast<long long>(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (job >= static_cast<long long>(T_) * units) return;
+  const int t = static_cast<int>(job / units), u = static_cast<int>(job % units);
+  if (u >= p.G + p.H) {
+    const int h = u - p.G - p.H;
+    const float rate = expf(A_log[h]);
+    const T* a = a_pre + static_cast<size_t>(t) * p.ld_a + static_cast<size_t>(h) * p.dim;
+    float* g = g_out + (static_cast<size_t>(t) * p.H + h) * p.dimP;
+    for (int i = lane; i < p.dimP; i += 32) {
+      float v = 0.f;
+      if (i < p.dim) {
+        const float z = to_f(a[i]) + dt_bias[h * p.dim + i];
+        const float sp = z > 20.f ? z : log1pf(expf(z));
+        v = expf(-rate * sp);
+      }
+      g[i] = v;
+    }
+    return;
+  }
+  const int b = sequence_of(cu, p.B, t);
+  const int n = cu[b + 1] - cu[b], i0 = t - cu[b];
+  const int start = kv_lens[b] - n, slot = state_slots[b];
+  const int C = 2 * p.G * p.dim + p.H * p.vdim;
+  const bool has = slot >= 0 && slot < num_slots;
+  T* st = has ? conv_state + static_cast<size_t>(slot) * (p.taps - 1) * C : nullptr;
+  T* old = start > 0 ? st : nullptr;                    // null: the sequence starts here, zeros before it
+  const bool shift = p.update && has;
+  // the lane that convolved channel c (column col) also moves its state by one token
+  auto shift_state = [&](int c, int col) {
+    for (int j = 0; j + 1 < p.taps - 1; ++j)
+      st[static_cast<size_t>(j) * C + c] = old != nullptr ? st[static_cast<size_t>(j + 1) * C + c] : T(0.f);
+    if (p.taps > 1) st[static_cast<size_t>(p.taps - 2) * C + c] = proj[static_cast<size_t>(t) * p.ld + col];
+  };
+  if (u < p.G) {
+    float q[NV], k[NV];
+    float sq = 0.f, sk = 0.f, dot = 0.f;
+#pragma unroll
+    for (int e = 0; e < NV; ++e) {
+      const int i = lane + 32 * e;
+      q[e] = k[e] = 0.f;
+      if (i < p.dim) {
+        const int c = u * p.dim + i, ck = p.G * p.dim + c;
+        q[e] = silu_f(conv_value(proj, p.ld, p.off_q + c, t, i0, conv_q + static_cast<size_t>(c) * p.taps, old, C, c,
+                                 p.taps));
+        k[e] = silu_f(conv_value(proj, p.ld, p.off_k + c, t, i0, conv_k + static_cast<size_t>(c) * p.taps, old, C, ck,
+                                 p.taps));
+        if (shift) {
+          shift_state(c, p.off_q + c);
+          shift_state(ck, p.off_k + c);
+        }
+        sq += q[e] * q[e];
+        sk += k[e] * k[e];
+        dot += q[e] * k[e];
+      }
+    }
+    const float iq = 1.f / (sqrtf(warp_sum(sq) + 1e-6f) * sqrtf(static_cast<float>(p.dim)));
+    const float ik = 1.f / sqrtf(warp_sum(sk) + 1e-6f);
+    dot = warp_sum(dot);
+    const size_t o = (static_cast<size_t>(t) * p.G + u) * p.dimP;
+#pragma unroll
+    for (int e = 0; e < NV; ++e) {
+      const int i = lane + 32 * e;
+      if (i < p.dimP) {
+        q_out[o + i] = q[e] * iq;
+        k_out[o + i] = k[e] * ik;
+      }
+    }
+    if (lane == 0) qk_out[static_cast<size_t>(t) * p.G + u] = dot * iq * ik;
+    return;
+  }
+  const int h = u - p.G;
+  for (int i = lane; i < p.vdim; i += 32) {
+    const int cv = h * p.vdim + i, c = 2 * p.G * p.dim + cv;
+    v_out[(static_cast<size_t>(t) * p.H + h) * p.vdim + i] = silu_f(
+        conv_value(proj, p.ld, p.off_v + cv, t, i0, conv_v + static_cast<size_t>(cv) * p.taps, old, C, c, p.taps));
+    if (shift) shift_state(c, p.off_v + cv);
+  }
+  if (lane == 0)
+    beta_out[static_cast<size_t>(t) * p.H + h] = sigmoid_f(to_f(proj[static_cast<size_t>(t) * p.ld + p.off_b + h]));
+}
+
+// last taps - 1 inputs of every sequence that contributed tokens -> its convolution state.  Grid (channels / 256, B).
+template <typename T>
+__global__ void __launch_bounds__(256)
+conv_state_kernel(const T* __restrict__ proj, const int* __restrict__ cu, const int* __restrict__ kv_lens,
+                  const int* __restrict__ state_slots, T* __restrict__ conv_state, int num_slots, DeltaPrep p) {
+  tgi::pdl_wait();
+  tgi::pdl_trigger();
+  const int b = blockIdx.y, c = blockIdx.x * blockDim.x + threadIdx.x;
+  const int nq = p.G * p.dim, C = 2 * nq + p.H * p.vdim;
+  const int n = cu[b + 1] - cu[b], slot = state_slots[b];
+  if (c >= C || n <= 0 || slot < 0 || slot >= num_slots) return;
+  const int col = c < nq ? p.off_q + c : (c < 2 * nq ? p.off_k + c - nq : p.off_v + c - 2 * nq);
+  const bool fresh = kv_lens[b] - n <= 0;
+  T* st = conv_state + static_cast<size_t>(slot) * (p.taps - 1) * C + c;
+  for (int j = 0; j < p.taps - 1; ++j) {            // ascending: entry j is only read by entries before it
+    const int i = n - (p.taps - 1) + j;             // local index of the input that belongs at entry j
+    T v = T(0.f);
+    if (i >= 0) v = proj[static_cast<size_t>(cu[b] + i) * p.ld + col];
+    else if (!fresh) v = st[static_cast<size_t>(p.taps - 1 + i) * C];
+    st[static_cast<size_t>(j) * C] = v;
+  }
+}
+
+// ------------------------------------------------------------------------------------------------
+// out = RMSNorm(o over `width`) * weight * sigmoid(gate).  o fp32 [T, groups, width]; gate at column `off` of a
+// [T, ld] matrix; out rows are `ld_out` wide, columns past groups * width are zeroed by group 0.
+// One warp (width <= 1024) or one block per (token, group).
+// ------------------------------------------------------------------------------------------------
+template <typename T, bool WARP>
+__global__ void __launch_bounds__(256)
+gated_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, long long ld, int off,
+                  const float* __restrict__ weight, T* __restrict__ out, long long ld_out, int T_, int groups, int width,
+                  float eps) {
+  tgi::pdl_wait();
+  tgi::pdl_trigger();
+  __shared__ float red[33];
+  const long long job = WARP ? static_cast<long long>(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5)
+                             : static_cast<long long>(blockIdx.x);
+  if (job >= static_cast<long long>(T_) * groups) return;      // warp- or block-uniform
+  const int t = static_cast<int>(job / groups), g = static_cast<int>(job % groups);
+  const int first = WARP ? (threadIdx.x & 31) : threadIdx.x, step = WARP ? 32 : blockDim.x;
+  const float* x = o + (static_cast<size_t>(t) * groups + g) * width;
+  const T* gt = gate + static_cast<size_t>(t) * ld + off + static_cast<size_t>(g) * width;
+  T* dst = out + static_cast<size_t>(t) * ld_out + static_cast<size_t>(g) * width;
+  float ss = 0.f;
+  const bool vec = width % 4 == 0 && ld % 4 == 0 && off % 4 == 0 && ld_out % 4 == 0;
+  if (vec) {
+    for (int i = first * 4; i < width; i += step * 4) {
+      const float4 v = load4(x + i);
+      ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    }
+  } else {
+    for (int i = first; i < width; i += step) ss += x[i] * x[i];
+  }
+  ss = WARP ? warp_sum(ss) : block_sum(ss, red);
+  const float inv = 1.f / sqrtf(ss / width + eps);
+  if (vec) {
+    for (int i = first * 4; i < width; i += step * 4) {
+      const float4 v = load4(x + i), w = load4(weight + i), s = load4(gt + i);
+      store4(dst + i, make_float4(v.x * inv * w.x * sigmoid_f(s.x), v.y * inv * w.y * sigmoid_f(s.y),
+                                  v.z * inv * w.z * sigmoid_f(s.z), v.w * inv * w.w * sigmoid_f(s.w)));
+    }
+  } else {
+    for (int i = first; i < width; i += step) put(dst + i, x[i] * inv * weight[i] * sigmoid_f(to_f(gt[i])));
+  }
+  if (g == 0)
+    for (int i = groups * width + first; i < ld_out; i += step) put(out + static_cast<size_t>(t) * ld_out + i, 0.f);
+}
+
+int done() { return cudaGetLastError() == cudaSuccess ? 0 : -3; }
+
+template <typename T>
+int residual_norm(const void* delta, const float* residual, const int* rows, const void* weight, void* out, float* res_out,
+                  int n, int H, float eps, cudaStream_t stream) {
+  const T* d = static_cast<const T*>(delta);
+  const T* w = static_cast<const T*>(weight);
+  T* o = static_cast<T*>(out);
+  if (H % 4 == 0 && H / 4 <= 4 * 1024) {
+    const int vecs = H / 4;
+    int threads = vecs >= 1024 ? 512 : ((vecs + 31) / 32) * 32;
+    if (threads > 256 && vecs <= 1024) threads = 256;
+    const int vpt = (vecs + threads - 1) / threads;
+    if (vpt <= 1) tgi::launch(residual_norm_kernel<T, 1>, dim3(n), dim3(threads), 0, stream, d, residual, rows, w, o, res_out, H, eps);
+    else if (vpt <= 2) tgi::launch(residual_norm_kernel<T, 2>, dim3(n), dim3(threads), 0, stream, d, residual, rows, w, o, res_out, H, eps);
+    else if (vpt <= 4) tgi::launch(residual_norm_kernel<T, 4>, dim3(n), dim3(threads), 0, stream, d, residual, rows, w, o, res_out, H, eps);
+    else tgi::launch(residual_norm_kernel<T, 8>, dim3(n), dim3(threads), 0, stream, d, residual, rows, w, o, res_out, H, eps);
+  } else {
+    tgi::launch(residual_norm_kernel<T, 0>, dim3(n), dim3(256), 0, stream, d, residual, rows, w, o, res_out, H, eps);
+  }
+  return done();
+}
+
+template <typename T>
+int attn_any(const void* q, const void* k, const void* v, const int* bt, const int* cu, const int* kv, void* out, int T_,
+             int B, int max_blocks, int bs_shift, int Hq, int Hkv, int Dk, int Dv, float scale, int window, int chunk,
+             int sink, cudaStream_t stream) {
+  const long long jobs = static_cast<long long>(T_) * Hq;
+  const dim3 grid(static_cast<unsigned>((jobs + kAttnWarps - 1) / kAttnWarps)), block(kAttnWarps * 32);
+  const size_t smem = static_cast<size_t>(kAttnWarps) * Dk * sizeof(float);
+  if (smem > 48 * 1024 || Dv > 32 * kMaxOut) return -12;
+  auto go = [&](auto kern) {
+    tgi::launch(kern, grid, block, smem, stream, static_cast<const T*>(q), static_cast<const T*>(k), static_cast<const T*>(v),
+                bt, cu, kv, static_cast<T*>(out), T_, B, max_blocks, bs_shift, Hq, Hkv, Dk, Dv, scale, window, chunk, sink);
+    return done();
+  };
+  if (Dv <= 64) return go(attn_any_kernel<T, 2>);
+  if (Dv <= 128) return go(attn_any_kernel<T, 4>);
+  if (Dv <= 256) return go(attn_any_kernel<T, 8>);
+  return go(attn_any_kernel<T, kMaxOut>);
+}
+
+template <typename T>
+int delta_prep(const void* proj, const void* a_pre, const float* cq, const float* ck, const float* cv, const float* A_log,
+               const float* dt_bias, const int* cu, const int* kv, const int* slots, void* conv_state, float* q, float* k,
+               float* v, float* g, float* beta, float* qk, int T_, int num_slots, const DeltaPrep& p, cudaStream_t stream) {
+  const T* x = static_cast<const T*>(proj);
+  T* st = static_cast<T*>(conv_state);
+  const long long jobs = static_cast<long long>(T_) * (p.G + 2 * p.H);
+  const dim3 grid(static_cast<unsigned>((jobs + 7) / 8));
+  auto go = [&](auto kern) {
+    tgi::launch(kern, grid, dim3(256), 0, stream, x, static_cast<const T*>(a_pre), cq, ck, cv, A_log, dt_bias, cu, kv, slots,
+                st, q, k, v, g, beta, qk, T_, num_slots, p);
+  };
+  if (p.dimP <= 64) go(delta_prep_kernel<T, 2>);
+  else if (p.dimP <= 128) go(delta_prep_kernel<T, 4>);
+  else go(delta_prep_kernel<T, 8>);
+  if (!p.update && p.taps > 1) {
+    const int C = 2 * p.G * p.dim + p.H * p.vdim;
+    tgi::launch(conv_state_kernel<T>, dim3((C + 255) / 256, p.B), dim3(256), 0, stream, x, cu, kv, slots, st, num_slots, p);
+  }
+  return done();
+}
+
+template <typename T>
+int gated_norm(const float* o, const void* gate, long long ld, int off, const float* w, void* out, long long ld_out, int T_,
+               int groups, int width, float eps, cudaStream_t stream) {
+  const long long jobs = static_cast<long long>(T_) * groups;
+  if (width <= 1024)
+    tgi::launch(gated_norm_kernel<T, true>, dim3(static_cast<unsigned>((jobs + 7) / 8)), dim3(256), 0, stream, o,
+                static_cast<const T*>(gate), ld, off, w, static_cast<T*>(out), ld_out, T_, groups, width, eps);
+  else
+    tgi::launch(gated_norm_kernel<T, false>, dim3(static_cast<unsigned>(jobs)), dim3(256), 0, stream, o,
+                static_cast<const T*>(gate), ld, off, w, static_cast<T*>(out), ld_out, T_, groups, width, eps);
+  return done();
+}
+
+}  // namespace
+
+// `f32` selects the build: 1 = fp32 activations, weights and pages, 0 = bf16.
+extern "C" {
+
+int tgi_residual_norm(int f32, const void* delta, const float* residual, const int* rows, const void* weight, void* out,
+                      float* res_out, int n, int H, float eps, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  return f32 ? residual_norm<float>(delta, residual, rows, weight, out, res_out, n, H, eps, stream)
+             : residual_norm<bf16>(delta, residual, rows, weight, out, res_out, n, H, eps, stream);
+}
+
+int tgi_embed_residual(int f32, const int* ids, const void* table, float* out, int T, int H, int vocab, float scale,
+                       cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (f32) tgi::launch(embed_residual_kernel<float>, dim3(T), dim3(256), 0, stream, ids, static_cast<const float*>(table), out, H, vocab, scale);
+  else tgi::launch(embed_residual_kernel<bf16>, dim3(T), dim3(256), 0, stream, ids, static_cast<const bf16*>(table), out, H, vocab, scale);
+  return done();
+}
+
+int tgi_activation(int f32, const void* in, void* out, long long n, int act, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  long long blocks = (n / 4 + 255) / 256;
+  if (blocks > 148 * 16) blocks = 148 * 16;
+  if (blocks < 1) blocks = 1;
+  const dim3 grid(static_cast<unsigned>(blocks));
+  if (f32) tgi::launch(activation_kernel<float>, grid, dim3(256), 0, stream, static_cast<const float*>(in), static_cast<float*>(out), n, act);
+  else tgi::launch(activation_kernel<bf16>, grid, dim3(256), 0, stream, static_cast<const bf16*>(in), static_cast<bf16*>(out), n, act);
+  return done();
+}
+
+int tgi_attn_prep(int f32, const void* proj, long long ld, int off_k, int off_v, const int* positions, const float* cos_sin,
+                  const int* slots, const void* v_first, long long ld_first, float lambda, void* q_out, void* k_cache,
+                  void* v_cache, void* v_mixed, int T, int Hq, int Hkv, int dim, int vdim, int Dk, int Dv, int rot, int max_pos,
+                  long long num_slots, int qk_norm, float eps, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (rot % 2 != 0 || rot > dim || Dk < dim || Dv < vdim) return -10;
+  const long long jobs = static_cast<long long>(T) * (Hq + 2 * Hkv);
+  const dim3 grid(static_cast<unsigned>((jobs + 7) / 8));
+  auto go = [&](auto kern, auto tag) {
+    using E = decltype(tag);
+    tgi::launch(kern, grid, dim3(256), 0, stream, static_cast<const E*>(proj), ld, off_k, off_v, positions, cos_sin, slots,
+                static_cast<const E*>(v_first), ld_first, lambda, static_cast<E*>(q_out), static_cast<E*>(k_cache),
+                static_cast<E*>(v_cache), static_cast<E*>(v_mixed), T, Hq, Hkv, dim, vdim, Dk, Dv, rot, max_pos, num_slots,
+                qk_norm, eps);
+    return done();
+  };
+  return f32 ? go(attn_prep_kernel<float>, float()) : go(attn_prep_kernel<bf16>, bf16());
+}
+
+int tgi_attn_any(int f32, const void* q, const void* k_cache, const void* v_cache, const int* block_tables, const int* cu,
+                 const int* kv_lens, void* out, int T, int B, int max_blocks, int block_size, int Hq, int Hkv, int Dk, int Dv,
+                 float scale, int window, int chunk, int sink, cudaStream_t stream) {
+  if (T <= 0 || B <= 0) return 0;
+  if (Hq % Hkv != 0 || block_size <= 0 || (block_size & (block_size - 1)) != 0) return -10;
+  int shift = 0;
+  while ((1 << shift) < block_size) ++shift;
+  return f32 ? attn_any<float>(q, k_cache, v_cache, block_tables, cu, kv_lens, out, T, B, max_blocks, shift, Hq, Hkv, Dk, Dv,
+                               scale, window, chunk, sink, stream)
+             : attn_any<bf16>(q, k_cache, v_cache, block_tables, cu, kv_lens, out, T, B, max_blocks, shift, Hq, Hkv, Dk, Dv,
+                              scale, window, chunk, sink, stream);
+}
+
+int tgi_delta_prep(int f32, const void* proj, long long ld, int off_q, int off_k, int off_v, int off_b, const void* a_pre,
+                   long long ld_a, const float* conv_q, const float* conv_k, const float* conv_v, const float* A_log,
+                   const float* dt_bias, const int* cu, const int* kv_lens, const int* state_slots, void* conv_state, float* q,
+                   float* k, float* v, float* g, float* beta, float* qk, int T, int B, int num_slots, int G, int H, int dim,
+                   int dimP, int vdim, int taps, int update, cudaStream_t stream) {
+  if (T <= 0 || B <= 0) return 0;
+  if (H % G != 0 || dimP < dim || dimP > 256 || taps < 1 || B > 65535) return -10;
+  const DeltaPrep p{ld, ld_a, off_q, off_k, off_v, off_b, B, G, H, dim, dimP, vdim, taps, update};
+  return f32 ? delta_prep<float>(proj, a_pre, conv_q, conv_k, conv_v, A_log, dt_bias, cu, kv_lens, state_slots, conv_state, q,
+                                 k, v, g, beta, qk, T, num_slots, p, stream)
+             : delta_prep<bf16>(proj, a_pre, conv_q, conv_k, conv_v, A_log, dt_bias, cu, kv_lens, state_slots, conv_state, q,
+                                k, v, g, beta, qk, T, num_slots, p, stream);
+}
+
+int tgi_gated_norm(int f32, const float* o, const void* gate, long long ld, int off, const float* weight, void* out,
+                   long long ld_out, int T, int groups, int width, float eps, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  return f32 ? gated_norm<float>(o, gate, ld, off, weight, out, ld_out, T, groups, width, eps, stream)
+             : gated_norm<bf16>(o, gate, ld, off, weight, out, ld_out, T, groups, width, eps, stream);
+}
+
+}  // extern "C"

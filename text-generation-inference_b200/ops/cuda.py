@@ -33,6 +33,16 @@ def lib_path() -> Path:
     return _LIB_PATH
 
 
+def use_kernel_set(name: str) -> None:
+    """Before the first kernel call: load the part ``name`` of the library (``build.KERNEL_SETS``), compiled now if need
+    be, unless the whole library is there already."""
+    global _LIB_PATH
+    if _LIB is None and not _LIB_PATH.exists():
+        from .build import build
+
+        _LIB_PATH = build(kernel_set=name)
+
+
 def load():
     """Load the kernel library; a missing library on a CUDA machine is an error, never a silent fallback."""
     global _LIB
@@ -53,8 +63,11 @@ def load():
                  "tgi_gemm_num_tiles", "tgi_attn_decode_splits", "tgi_attn_status", "tgi_lora_shrink",
                  "tgi_lora_expand", "tgi_moe_topk_softmax", "tgi_moe_sort", "tgi_moe_gather", "tgi_moe_grouped_gemm",
                  "tgi_moe_combine", "tgi_gemm_last_grid", "tgi_penalties", "tgi_gemm_wq", "tgi_wq_dequant", "tgi_qk_norm",
-                 "tgi_quant_set_pow2", "tgi_peer_set_quant_pow2"):
-        getattr(_LIB, name).restype = c_int
+                 "tgi_quant_set_pow2", "tgi_peer_set_quant_pow2", "tgi_gemm_bf16_ld", "tgi_residual_norm", "tgi_embed_residual",
+                 "tgi_activation", "tgi_attn_prep", "tgi_attn_any", "tgi_delta_prep", "tgi_delta_scan", "tgi_decay_scan",
+                 "tgi_gated_norm", "tgi_recurrent_pitch"):
+        if hasattr(_LIB, name):        # a library built for one family of models lacks the other families' kernels
+            getattr(_LIB, name).restype = c_int
     _LIB.tgi_gemm_workspace_floats.restype = c_ll
     wide = os.environ.get("TGI_B200_GEMM_WIDE_M")
     if wide:
@@ -66,7 +79,7 @@ def load():
     if os.environ.get("TGI_B200_GEMM_STREAMK_SMALL", "0") == "1":   # stream-K also below one tile per worker
         _LIB.tgi_gemm_set_streamk_small(c_int(1))
     # fp8 GEMMs run on the block-scaled MMA unless TGI_B200_FP8_MX=0 (then: per-K-block promotion, arbitrary scales)
-    if os.environ.get("TGI_B200_FP8_MX", "1") == "1" and torch.cuda.is_available():
+    if os.environ.get("TGI_B200_FP8_MX", "1") == "1" and torch.cuda.is_available() and hasattr(_LIB, "tgi_peer_set_quant_pow2"):
         set_fp8_mx(True)
     return _LIB
 
@@ -208,8 +221,11 @@ def gemm_bf16(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = N
               out: Optional[torch.Tensor] = None):
     lib = load()
     lead = x.shape[:-1]
-    x2 = x.reshape(-1, x.shape[-1])
-    if not x2.is_contiguous():
+    x2 = x if x.dim() == 2 else x.reshape(-1, x.shape[-1])
+    # a column slice of a wider matrix is read in place when its rows start on 16-byte boundaries
+    sliced = (x2.stride(1) == 1 and x2.stride(0) > x2.shape[1] and x2.stride(0) % 8 == 0 and x2.data_ptr() % 16 == 0
+              and not getattr(out, "is_peer_push", False))
+    if not sliced and not x2.is_contiguous():
         x2 = x2.contiguous()
     M, K = x2.shape
     N = w.shape[0]
@@ -233,6 +249,11 @@ def gemm_bf16(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = N
         return out.reshape(*lead, N)
     st = state(x.device)
     ctas = _gemm_ctas(lib, st, M, N, max_ctas)
+    if sliced:
+        _check(lib.tgi_gemm_bf16_ld(_ptr(x2), c_int(x2.stride(0)), _ptr(w), _ptr(out), _ptr(bias), c_int(M), c_int(N),
+                                    c_int(K), c_int(ctas), _ptr(st.ws), _ptr(st.counters), _ptr(st.status), _stream()),
+               "gemm_bf16_ld")
+        return out.reshape(*lead, N)
     _check(lib.tgi_gemm_bf16(_ptr(x2), _ptr(w), _ptr(out), _ptr(bias), c_int(M), c_int(N), c_int(K), c_int(ctas),
                              _ptr(st.ws), _ptr(st.counters), _ptr(st.status), _stream()), "gemm_bf16")
     return out.reshape(*lead, N)
@@ -380,19 +401,44 @@ def rope_and_cache(qkv, positions, cos_sin, slots, k_cache, v_cache, num_heads, 
 
 
 # ---- attention ---------------------------------------------------------------------------------
+ATTN_HEAD_DIMS = (64, 128, 256)      # head sizes of the tensor-core kernels (bf16 queries)
+
+
+def attention_pitch(dim: int, vdim: int, dtype: torch.dtype) -> Tuple[int, int]:
+    """Page widths ``(K, V)`` of a head with ``dim`` query/key and ``vdim`` value dimensions: both padded to one size of
+    the tensor-core kernels where there is one, otherwise as they are (``tgi_attn_any``)."""
+    if dtype == torch.bfloat16:
+        for w in ATTN_HEAD_DIMS:
+            if max(dim, vdim) <= w:
+                return w, w
+    return dim, vdim
+
+
 def paged_attention(q, k_cache, v_cache, block_tables, cu_seqlens_q, kv_lens, scale, window=-1, softcap=0.0,
-                    k_scale=None, v_scale=None, max_q=None, max_kv=None, nsplit: Optional[int] = None, horizon=None):
+                    k_scale=None, v_scale=None, max_q=None, max_kv=None, nsplit: Optional[int] = None, horizon=None,
+                    chunk: int = 0, sink: bool = False):
     lib = load()
     T, Hq, D = q.shape
     nblk, bs, Hkv, _ = k_cache.shape
+    Dv = v_cache.shape[3]
     B = kv_lens.shape[0]
-    out = torch.empty_like(q)
+    out = q.new_empty(T, Hq, Dv)
     if T == 0 or B == 0:
+        return out
+    if q.dtype == torch.float32 or D != Dv or D not in ATTN_HEAD_DIMS:
+        assert softcap <= 0 and horizon is None and k_cache.dtype == q.dtype and v_cache.dtype == q.dtype
+        _check(lib.tgi_attn_any(
+            c_int(1 if q.dtype == torch.float32 else 0), _ptr(q.contiguous()), _ptr(k_cache), _ptr(v_cache),
+            _ptr(block_tables), _ptr(cu_seqlens_q), _ptr(kv_lens), _ptr(out), c_int(T), c_int(B),
+            c_int(block_tables.shape[1]), c_int(bs), c_int(Hq), c_int(Hkv), c_int(D), c_int(Dv), c_float(scale),
+            c_int(window if window and window > 0 else -1), c_int(chunk), c_int(1 if sink else 0), _stream()), "attn_any")
         return out
     if max_q is None:
         max_q = int((cu_seqlens_q[1:] - cu_seqlens_q[:-1]).max().item())
     if max_kv is None:
         max_kv = int(kv_lens.max().item())
+    if chunk > 0:
+        max_kv = min(max_kv, chunk)      # keys a row can see: decides how far a decode step is split
     fp8 = k_cache.dtype == FP8
     st = state(q.device)
     part_o = part_ml = None
@@ -411,8 +457,116 @@ def paged_attention(q, k_cache, v_cache, block_tables, cu_seqlens_q, kv_lens, sc
         _ptr(q.contiguous()), _ptr(k_cache), _ptr(v_cache), _ptr(block_tables), _ptr(cu_seqlens_q), _ptr(kv_lens),
         _ptr(k_scale if fp8 else None), _ptr(v_scale if fp8 else None), _ptr(out), _ptr(part_o), _ptr(part_ml),
         c_int(B), c_int(max_q), c_int(block_tables.shape[1]), c_int(bs), c_int(nblk), c_int(Hq), c_int(Hkv), c_int(D),
-        c_float(scale), c_float(softcap), c_int(window if window and window > 0 else -1), c_int(nsplit),
-        c_int(1 if fp8 else 0), _ptr(horizon), _stream()), "paged_attention")
+        c_float(scale), c_float(softcap), c_int(window if window and window > 0 else -1), c_int(chunk),
+        c_int(1 if sink else 0), c_int(nsplit), c_int(1 if fp8 else 0), _ptr(horizon), _stream()), "paged_attention")
+    return out
+
+
+# ---- token mixers of hybrid decoders -------------------------------------------------------------
+def _f32(t: torch.Tensor):
+    if t.dtype not in (torch.float32, torch.bfloat16):
+        raise KernelError(f"hybrid decoders run in bfloat16 or float32, not {t.dtype}")
+    return c_int(1 if t.dtype == torch.float32 else 0)
+
+
+def embed_residual(ids, table, scale: float):
+    T, H = ids.numel(), table.shape[1]
+    out = torch.empty(T, H, dtype=torch.float32, device=table.device)
+    _check(load().tgi_embed_residual(_f32(table), _ptr(ids), _ptr(table), _ptr(out), c_int(T), c_int(H),
+                                     c_int(table.shape[0]), c_float(scale), _stream()), "embed_residual")
+    return out
+
+
+def residual_norm(delta, residual, weight, eps, rows=None, keep: bool = True):
+    H = residual.shape[1]
+    n = residual.shape[0] if rows is None else rows.shape[0]
+    out = torch.empty(n, H, dtype=weight.dtype, device=residual.device)
+    if delta is None and rows is None:
+        res = None if not keep else residual
+        dst = None
+    else:
+        res = dst = torch.empty(n, H, dtype=torch.float32, device=residual.device) if keep else None
+    assert residual.dtype == torch.float32 and residual.is_contiguous()
+    assert delta is None or (delta.dtype == weight.dtype and delta.is_contiguous())
+    _check(load().tgi_residual_norm(_f32(weight), _ptr(delta), _ptr(residual), _ptr(rows), _ptr(weight), _ptr(out), _ptr(dst),
+                                    c_int(n), c_int(H), c_float(eps), _stream()), "residual_norm")
+    return out, res
+
+
+def activation(x, act: str):
+    out = torch.empty_like(x)
+    _check(load().tgi_activation(_f32(x), _ptr(x), _ptr(out), c_ll(x.numel()), c_int(_ACT_CODES[act]), _stream()),
+           "activation")
+    return out
+
+
+def rotate_norm_store(proj, offs, positions, cos_sin, slots, k_cache, v_cache, num_heads, num_kv_heads, dim, vdim, rot_dim,
+                      qk_norm, eps, v_first=None, v_lambda: float = 0.0):
+    T = proj.shape[0]
+    Dk, Dv = k_cache.shape[3], v_cache.shape[3]
+    q = torch.empty(T, num_heads, Dk, dtype=proj.dtype, device=proj.device)
+    assert proj.stride(1) == 1 and k_cache.dtype == proj.dtype and v_cache.dtype == proj.dtype
+    assert v_first is None or (v_first.stride(1) == 1 and v_first.shape[1] == num_kv_heads * vdim and v_first.dtype == proj.dtype)
+    _check(load().tgi_attn_prep(
+        _f32(proj), _ptr(proj), c_ll(proj.stride(0)), c_int(offs[1]), c_int(offs[2]), _ptr(positions), _ptr(cos_sin),
+        _ptr(slots), _ptr(v_first), c_ll(0 if v_first is None else v_first.stride(0)), c_float(v_lambda), _ptr(q),
+        _ptr(k_cache), _ptr(v_cache), c_void_p(0), c_int(T), c_int(num_heads), c_int(num_kv_heads), c_int(dim), c_int(vdim),
+        c_int(Dk), c_int(Dv), c_int(rot_dim), c_int(cos_sin.shape[0]), c_ll(k_cache.shape[0] * k_cache.shape[1]),
+        c_int(1 if qk_norm else 0), c_float(eps), _stream()), "attn_prep")
+    return q
+
+
+def recurrent_pitch(dim: int) -> int:
+    w = int(load().tgi_recurrent_pitch(c_int(dim)))
+    if w == 0:
+        raise KernelError(f"recurrent heads of {dim} key channels are wider than the kernels support (256)")
+    return w
+
+
+def delta_inputs(proj, offs, a_pre, conv_q, conv_k, conv_v, a_log, dt_bias, cu, kv_lens, state_slots, conv_state, kv_heads,
+                 heads, dim, pitch, vdim, single: bool):
+    T, dev = proj.shape[0], proj.device
+    new = lambda *shape: torch.empty(*shape, dtype=torch.float32, device=dev)
+    q, k, g = new(T, kv_heads, pitch), new(T, kv_heads, pitch), new(T, heads, pitch)
+    v, beta, qk = new(T, heads, vdim), new(T, heads), new(T, kv_heads)
+    taps = conv_q.shape[1]
+    assert proj.stride(1) == 1 and a_pre.stride(1) == 1 and conv_state.dtype == proj.dtype
+    _check(load().tgi_delta_prep(
+        _f32(proj), _ptr(proj), c_ll(proj.stride(0)), c_int(offs[0]), c_int(offs[1]), c_int(offs[2]), c_int(offs[3]),
+        _ptr(a_pre), c_ll(a_pre.stride(0)), _ptr(conv_q), _ptr(conv_k), _ptr(conv_v), _ptr(a_log), _ptr(dt_bias), _ptr(cu),
+        _ptr(kv_lens), _ptr(state_slots), _ptr(conv_state), _ptr(q), _ptr(k), _ptr(v), _ptr(g), _ptr(beta), _ptr(qk),
+        c_int(T), c_int(kv_lens.shape[0]), c_int(conv_state.shape[0]), c_int(kv_heads), c_int(heads), c_int(dim),
+        c_int(pitch), c_int(vdim), c_int(taps), c_int(1 if single else 0), _stream()), "delta_prep")
+    return q, k, v, g, beta, qk
+
+
+def delta_scan(q, k, v, g, beta, qk, cu, kv_lens, state_slots, state, dim: int, max_q: int):
+    T, heads, vdim = v.shape
+    out = torch.empty(T, heads, vdim, dtype=torch.float32, device=v.device)
+    _check(load().tgi_delta_scan(
+        _ptr(q), _ptr(k), _ptr(g), _ptr(v), _ptr(beta), _ptr(qk), _ptr(cu), _ptr(kv_lens), _ptr(state_slots), _ptr(state),
+        _ptr(out), c_int(kv_lens.shape[0]), c_int(max_q), c_int(state.shape[0]), c_int(k.shape[1]), c_int(heads), c_int(dim),
+        c_int(state.shape[3]), c_int(vdim), _stream()), "delta_scan")
+    return out
+
+
+def decay_scan(proj, offs, decay, cu, kv_lens, state_slots, state, heads: int, dim: int, vdim: int, max_q: int):
+    T = proj.shape[0]
+    out = torch.empty(T, heads, vdim, dtype=torch.float32, device=proj.device)
+    _check(load().tgi_decay_scan(
+        _f32(proj), _ptr(proj), c_ll(proj.stride(0)), c_int(offs[0]), c_int(offs[1]), c_int(offs[2]), _ptr(decay), _ptr(cu),
+        _ptr(kv_lens), _ptr(state_slots), _ptr(state), _ptr(out), c_int(kv_lens.shape[0]), c_int(max_q),
+        c_int(state.shape[0]), c_int(heads), c_int(dim), c_int(state.shape[3]), c_int(vdim), _stream()), "decay_scan")
+    return out
+
+
+def gated_norm(o, gate, weight, eps, groups: int, out_cols: int):
+    T = o.shape[0]
+    width = o.numel() // max(T * groups, 1)
+    out = torch.empty(T, out_cols, dtype=gate.dtype, device=o.device)
+    assert gate.stride(1) == 1 and weight.dtype == torch.float32
+    _check(load().tgi_gated_norm(_f32(gate), _ptr(o), _ptr(gate), c_ll(gate.stride(0)), c_int(0), _ptr(weight), _ptr(out),
+                                 c_ll(out_cols), c_int(T), c_int(groups), c_int(width), c_float(eps), _stream()), "gated_norm")
     return out
 
 

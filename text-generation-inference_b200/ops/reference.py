@@ -128,9 +128,12 @@ def paged_attention(
     max_q: Optional[int] = None,
     max_kv: Optional[int] = None,
     horizon: Optional[torch.Tensor] = None,
+    chunk: int = 0,
+    sink: bool = False,
 ) -> torch.Tensor:
     """Causal attention of ragged queries over paged KV (covers prefill, chunked prefill and decode).
-    ``horizon[t]`` (optional) replaces the causal limit of query row ``t`` by a later position.
+    ``horizon[t]`` (optional) replaces the causal limit of query row ``t`` by a later position.  With ``chunk`` a row
+    sees only keys ``t`` with ``t // chunk == pos // chunk``; ``sink`` adds ``exp(0)`` to the softmax denominator.
 
     Query ``i`` (0-based inside its sequence's chunk of ``n`` queries) of a sequence with ``L`` KV
     tokens sits at absolute position ``L - n + i`` and attends to KV positions ``<=`` its own
@@ -139,11 +142,12 @@ def paged_attention(
     T, Hq, D = q.shape
     nblk, bs, Hkv, _ = k_cache.shape
     group = Hq // Hkv
-    out = torch.empty_like(q)
+    Dv = v_cache.shape[3]
+    out = q.new_empty(T, Hq, Dv)
     cu = cu_seqlens_q.tolist()
     lens = kv_lens.tolist()
     kc = k_cache.view(-1, Hkv, D)
-    vc = v_cache.view(-1, Hkv, D)
+    vc = v_cache.view(-1, Hkv, Dv)
     for b in range(len(lens)):
         s, e = cu[b], cu[b + 1]
         n, L = e - s, lens[b]
@@ -174,8 +178,13 @@ def paged_attention(
         mask = kpos <= limit
         if window > 0:
             mask &= kpos > qpos - window
+        if chunk > 0:
+            mask &= torch.div(kpos, chunk, rounding_mode="floor") == torch.div(qpos, chunk, rounding_mode="floor")
         scores = scores.masked_fill(~mask.unsqueeze(0), float("-inf"))
-        p = torch.softmax(scores, dim=-1)
+        if sink:
+            p = torch.softmax(torch.cat([scores, scores.new_zeros(Hq, n, 1)], dim=-1), dim=-1)[..., :-1]
+        else:
+            p = torch.softmax(scores, dim=-1)
         out[s:e] = torch.einsum("hnl,lhd->nhd", p, v).to(q.dtype)
     return out
 
@@ -332,3 +341,118 @@ def moe_experts(
         y = F.linear(h, w_down[e]).float()
         out.index_add_(0, tok, y * topk_weights[tok, slot].unsqueeze(1).float())
     return out.to(x.dtype)
+
+
+# ---- token mixers of hybrid decoders -------------------------------------------------------------
+def embed_residual(ids, table, scale: float = 1.0):
+    return F.embedding(ids.long(), table).float() * scale
+
+
+def residual_norm(delta, residual, weight, eps: float, rows=None, keep: bool = True):
+    r = residual if delta is None else residual + delta.float()
+    if rows is not None:
+        r = r[rows.long()]
+    y = r * torch.rsqrt(r.pow(2).mean(-1, keepdim=True) + eps) * weight.float()
+    return y.to(weight.dtype), (r if keep else None)
+
+
+def rotate_norm_store(proj, offs, positions, cos_sin, slots, k_cache, v_cache, num_heads, num_kv_heads, dim, vdim, rot_dim,
+                      qk_norm, eps, v_first=None, v_lambda: float = 0.0):
+    T = proj.shape[0]
+    cs = cos_sin[positions.long()]
+    cos, sin = cs[:, : rot_dim // 2], cs[:, rot_dim // 2:]
+
+    def head(off, n):
+        x = proj[:, off:off + n * dim].reshape(T, n, dim).float()
+        if rot_dim > 0:
+            x = rotate(x, cos, sin, rot_dim, True)
+        return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) if qk_norm else x
+
+    q, k = head(offs[0], num_heads), head(offs[1], num_kv_heads)
+    v = proj[:, offs[2]:offs[2] + num_kv_heads * vdim].float()
+    if v_first is not None:
+        v = (1.0 - v_lambda) * v + v_lambda * v_first.float()
+    ok = (slots >= 0).nonzero(as_tuple=True)[0]
+    idx = slots[ok].long()
+    k_cache.view(-1, num_kv_heads, k_cache.shape[3])[idx, :, :dim] = k[ok].to(k_cache.dtype)
+    v_cache.view(-1, num_kv_heads, v_cache.shape[3])[idx, :, :vdim] = v.view(T, num_kv_heads, vdim)[ok].to(v_cache.dtype)
+    return F.pad(q, (0, k_cache.shape[3] - dim)).to(proj.dtype)
+
+
+def _sequences(cu, kv_lens, state_slots):
+    """``(sequence, first row, rows, position of the first row, slot)`` of every sequence that brings tokens."""
+    cu, lens, slots = cu.tolist(), kv_lens.tolist(), state_slots.tolist()
+    for b, (s, e) in enumerate(zip(cu[:-1], cu[1:])):
+        if e > s:
+            yield b, s, e - s, lens[b] - (e - s), slots[b]
+
+
+def _short_conv(x, w, past):
+    """``x[n, C]`` after ``past[taps - 1, C]``; returns the convolved, SiLU-ed rows and the new past."""
+    taps = w.shape[1]
+    full = torch.cat([past.float(), x.float()], dim=0)
+    y = sum(full[j:j + x.shape[0]] * w[:, j].float() for j in range(taps))
+    return F.silu(y), full[full.shape[0] - (taps - 1):]
+
+
+def delta_inputs(proj, offs, a_pre, conv_q, conv_k, conv_v, a_log, dt_bias, cu, kv_lens, state_slots, conv_state, kv_heads,
+                 heads, dim, pitch, vdim, single: bool):
+    T, taps = proj.shape[0], conv_q.shape[1]
+    nq, nv = kv_heads * dim, heads * vdim
+    x = torch.cat([proj[:, offs[0]:offs[0] + nq], proj[:, offs[1]:offs[1] + nq], proj[:, offs[2]:offs[2] + nv]], dim=1)
+    w = torch.cat([conv_q, conv_k, conv_v], dim=0)
+    y = torch.zeros(T, 2 * nq + nv)
+    for _, s, n, start, slot in _sequences(cu, kv_lens, state_slots):
+        past = conv_state[slot] if slot >= 0 and start > 0 else torch.zeros(taps - 1, x.shape[1])
+        y[s:s + n], new = _short_conv(x[s:s + n], w, past)
+        if slot >= 0:
+            conv_state[slot] = new.to(conv_state.dtype)
+    q, k = (y[:, i * nq:(i + 1) * nq].view(T, kv_heads, dim) for i in range(2))
+    q = q * torch.rsqrt(q.pow(2).sum(-1, keepdim=True) + 1e-6) * dim ** -0.5
+    k = k * torch.rsqrt(k.pow(2).sum(-1, keepdim=True) + 1e-6)
+    g = torch.exp(-torch.exp(a_log).view(1, heads, 1) * F.softplus(a_pre.float() + dt_bias).view(T, heads, dim))
+    beta = torch.sigmoid(proj[:, offs[3]:offs[3] + heads].float())
+    pad = (0, pitch - dim)
+    return F.pad(q, pad), F.pad(k, pad), y[:, 2 * nq:].view(T, heads, vdim), F.pad(g, pad), beta, (q * k).sum(-1)
+
+
+def delta_scan(q, k, v, g, beta, qk, cu, kv_lens, state_slots, state, dim: int, max_q: int):
+    T, heads, vdim = v.shape
+    rep = heads // k.shape[1]
+    q, k = q.repeat_interleave(rep, 1), k.repeat_interleave(rep, 1)
+    out = torch.zeros(T, heads, vdim)
+    for _, s, n, start, slot in _sequences(cu, kv_lens, state_slots):
+        S = state[slot].clone() if slot >= 0 and start > 0 else torch.zeros(state.shape[1:])      # [H, vdim, pitch]
+        for t in range(s, s + n):
+            S = S * g[t].unsqueeze(1)
+            u = beta[t].unsqueeze(1) * (v[t] - torch.einsum("hvd,hd->hv", S, k[t]))
+            S = S + u.unsqueeze(2) * k[t].unsqueeze(1)
+            out[t] = torch.einsum("hvd,hd->hv", S, q[t])
+        if slot >= 0:
+            state[slot] = S
+    return out
+
+
+def decay_scan(proj, offs, decay, cu, kv_lens, state_slots, state, heads: int, dim: int, vdim: int, max_q: int):
+    T = proj.shape[0]
+    q, k = (F.silu(proj[:, o:o + heads * dim].float()).view(T, heads, dim) for o in offs[:2])
+    v = F.silu(proj[:, offs[2]:offs[2] + heads * vdim].float()).view(T, heads, vdim)
+    pad = (0, state.shape[3] - dim)
+    q, k = F.pad(q, pad), F.pad(k, pad)
+    out = torch.zeros(T, heads, vdim)
+    for _, s, n, start, slot in _sequences(cu, kv_lens, state_slots):
+        S = state[slot].clone() if slot >= 0 and start > 0 else torch.zeros(state.shape[1:])
+        for t in range(s, s + n):
+            S = S * decay.view(-1, 1, 1) + v[t].unsqueeze(2) * k[t].unsqueeze(1)
+            out[t] = torch.einsum("hvd,hd->hv", S, q[t])
+        if slot >= 0:
+            state[slot] = S
+    return out
+
+
+def gated_norm(o, gate, weight, eps: float, groups: int, out_cols: int):
+    T = o.shape[0]
+    x = o.reshape(T, groups, -1)
+    y = x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * weight
+    y = y.reshape(T, -1) * torch.sigmoid(gate[:, :y.numel() // T].float())
+    return F.pad(y, (0, out_cols - y.shape[1])).to(gate.dtype)

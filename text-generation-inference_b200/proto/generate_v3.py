@@ -56,6 +56,8 @@ _MESSAGES = {
         ("use_prefix_caching", 7, "bool", ""),
         ("attention_impl", 8, "string", ""),
         ("block_size", 9, "uint32", ""),
+        # not in the reference's message: live requests the shard can hold state for (models with recurrent layers)
+        ("max_batch_size", 32, "uint32", "optional"),
     ],
     "ServiceDiscoveryRequest": [],
     "ServiceDiscoveryResponse": [("urls", 1, "string", "repeated")],

@@ -222,6 +222,10 @@ int main(int argc, char** argv) {
     bc.max_waiting_tokens = static_cast<uint32_t>(args.num("max-waiting-tokens", 20));
     bc.waiting_served_ratio_x100 = static_cast<uint32_t>(std::atof(args.get("waiting-served-ratio", "0.3").c_str()) * 100);
     if (args.has("max-batch-size")) bc.max_batch_size = static_cast<size_t>(args.num("max-batch-size", 0));
+    if (info.max_batch_size && (!bc.max_batch_size || *bc.max_batch_size > *info.max_batch_size)) {
+      bc.max_batch_size = *info.max_batch_size;    // one slot of recurrent state per live request
+      std::cerr << "[router] batches are limited to " << *info.max_batch_size << " requests by the shards" << std::endl;
+    }
     auto backend = std::make_shared<sched::Backend>(client, qc, bc, &metrics);
     backend->start_thread();
 

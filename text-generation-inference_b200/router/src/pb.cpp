@@ -38,6 +38,7 @@ InfoResponse InfoResponse::decode(const std::string& s) {
       case 7: m.use_prefix_caching = r.varint(); return true;
       case 8: m.attention_impl = r.bytes(); return true;
       case 9: m.block_size = static_cast<uint32_t>(r.varint()); return true;
+      case 32: m.max_batch_size = static_cast<uint32_t>(r.varint()); return true;
     }
     (void)wt;
     return false;

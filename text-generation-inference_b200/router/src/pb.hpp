@@ -102,6 +102,7 @@ struct InfoResponse {
   bool requires_padding = false;
   std::string dtype, device_type, attention_impl;
   std::optional<uint32_t> window_size;
+  std::optional<uint32_t> max_batch_size;   // live requests the shard can hold state for
   uint32_t speculate = 0, block_size = 0;
   bool support_chunking = false, use_prefix_caching = false;
   static InfoResponse decode(const std::string& s);

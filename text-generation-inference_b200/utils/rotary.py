@@ -55,6 +55,19 @@ def llama3_inv_freq(inv_freq: torch.Tensor, factor: float, low: float, high: flo
     return torch.tensor(out, dtype=torch.float32)
 
 
+def scaled_frequencies(base: float, dim: int, scaling: Optional[Tuple[float, float, float, float]] = None) -> torch.Tensor:
+    """fp64 frequencies ``base^(-2i/dim)``; ``scaling = (factor, low, high, original length)`` divides those of long
+    wavelengths by ``factor`` as ``llama3_inv_freq`` does."""
+    f = float(base) ** (-torch.arange(0, dim, 2, dtype=torch.float64) / max(dim, 1))
+    if scaling is None:
+        return f
+    factor, low, high, original = scaling
+    wave = 2 * math.pi / f
+    s = (original / wave - low) / (high - low)
+    mid = (1 - s) * f / factor + s * f
+    return torch.where(wave < original / high, f, torch.where(wave > original / low, f / factor, mid))
+
+
 class RotaryTable:
     """cos/sin table for one model.
 
@@ -81,6 +94,13 @@ class RotaryTable:
         t = torch.arange(max_positions, dtype=torch.float32) / position_scale
         freqs = torch.outer(t, inv_freq)
         return torch.cat([freqs.cos() * mscale, freqs.sin() * mscale], dim=-1).contiguous()
+
+    @classmethod
+    def from_frequencies(cls, freq: torch.Tensor, max_positions: int, neox: bool = True) -> "RotaryTable":
+        """Table of the given fp64 frequencies, with the angles formed in fp64 (an fp32 product of a position in the
+        thousands and a frequency near 1 is off by 1e-4)."""
+        ang = torch.outer(torch.arange(max_positions, dtype=torch.float64), freq.double())
+        return cls(torch.cat([ang.cos(), ang.sin()], dim=-1).float().contiguous(), 2 * freq.numel(), neox)
 
     @classmethod
     def from_config(cls, config, dim: int, base: float, max_positions: int, neox: bool = True) -> "RotaryTable":

@@ -200,6 +200,7 @@ class Weights:
         prefix: Optional[str] = None,
         loader=None,
         renames: Optional[List[Tuple[str, str]]] = None,
+        bare_names: bool = False,
     ):
         self._handles: List[SafetensorsFile] = []
         self.routing: Dict[str, int] = {}
@@ -218,6 +219,8 @@ class Weights:
         # (old prefix, new prefix) pairs: a name that starts with the old prefix is also looked up under the
         # new one (checkpoints of one architecture published under different module layouts)
         self.renames = list(renames or [])
+        # the checkpoint names its tensors without the ".weight" suffix the layers ask for
+        self.bare_names = bare_names
         self.device = torch.device(device)
         self.dtype = dtype
         self.process_group = process_group or ProcessGroupView()
@@ -239,6 +242,8 @@ class Weights:
         for old, new in self.renames:
             if name.startswith(old):
                 names.append(new + name[len(old):])
+        if self.bare_names and name.endswith(".weight"):
+            names.append(name[:-len(".weight")])
         return names
 
     def resolve(self, name: str) -> Tuple[SafetensorsFile, str]:
