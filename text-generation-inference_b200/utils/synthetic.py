@@ -263,3 +263,114 @@ def mixtral_8x7b_config(**kw) -> dict:
     return llama_config(hidden=4096, layers=32, heads=32, kv_heads=8, intermediate=14336, vocab=32000,
                         theta=1000000.0, max_pos=32768, model_type="mixtral", num_local_experts=8,
                         num_experts_per_tok=2, **kw)
+
+
+# ---------------------------------------------------------------------------------------------
+# decoders whose layers differ
+# ---------------------------------------------------------------------------------------------
+class DictWeights:
+    """``Weights`` over tensors that are in memory already."""
+
+    def __new__(cls, tensors: Dict[str, torch.Tensor], device, dtype, bare_names: bool = False):
+        from .weights import Weights
+
+        self = Weights([], device, dtype, bare_names=bare_names)
+
+        class _Slice:
+            def __init__(self, t):
+                self.t = t
+
+            def get_shape(self):
+                return tuple(self.t.shape)
+
+            def tensor(self):
+                return self.t
+
+            def slice_dim(self, dim, start, stop):
+                return self.t.narrow(dim, start, max(0, stop - start)) if self.t.dim() else self.t
+
+        def resolve(name):
+            for cand in self._candidates(name):
+                if cand in tensors:
+                    return None, cand
+            raise KeyError(f"weight {name} does not exist")
+
+        self.resolve = resolve
+        self._slice = lambda name: _Slice(tensors[resolve(name)[1]])
+        return self
+
+
+def fuzuvik_attention(heads=4, kv_heads=2, dim=32, vdim=16, chunk=48, rot_dims=None, base=10000.0, scaling=None, scale=None,
+                      v_mix=True, ff=96) -> dict:
+    rot = {"base": base, "dims": dim if rot_dims is None else rot_dims}
+    if scaling is not None:
+        rot["scaling"] = dict(zip(("factor", "low", "high", "original"), scaling))
+    return {"type": "attention", "mlp": {"ff": ff, "kind": "dense"} if ff else None,
+            "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "mask": {"size": chunk}, "rot": rot,
+                      "scale": dim ** -0.5 if scale is None else scale, "v_mix": v_mix}}
+
+
+def fuzuvik_delta(heads=4, kv_heads=2, dim=24, vdim=40, conv=4, ff=96) -> dict:
+    return {"type": "channel_delta", "mlp": {"ff": ff, "kind": "dense"} if ff else None,
+            "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv}}
+
+
+def fuzuvik_lightning(heads=3, dim=16, vdim=24, decay=None, ff=96) -> dict:
+    decay = decay or [1.0 - 2.0 ** -(1 + 7 * (h + 1) / heads) for h in range(heads)]
+    return {"type": "lightning", "mlp": {"ff": ff, "kind": "dense"} if ff else None,
+            "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "decay": list(decay)}}
+
+
+def fuzuvik_config(layers, width=80, vocab=203, eps=1e-5, embed_scale=3.0) -> dict:
+    return {"architecture": "Fuzuvik", "width": width, "vocab": vocab, "norm": {"eps": eps},
+            "embedding": {"scale": embed_scale}, "layers": list(layers)}
+
+
+def fuzuvik_state_dict(cfg: dict, seed: int = 0, dtype=torch.float32, device: str = "cpu",
+                       rank: Optional[int] = None) -> Dict[str, torch.Tensor]:
+    """Random weights of a Fuzuvik shape.  ``rank``: width of the low-rank decay and gate projections."""
+    g = torch.Generator(device=device).manual_seed(seed)
+    W, sd = cfg["width"], {}
+
+    def rnd(*shape, std=None, mean=0.0):
+        std = shape[-1] ** -0.5 if std is None else std
+        return (mean + torch.randn(*shape, generator=g, device=device) * std).to(dtype)
+
+    def uniform(lo, hi, *shape):
+        return (lo + (hi - lo) * torch.rand(shape, generator=g, device=device)).to(dtype)
+
+    sd["embed"], sd["head"] = rnd(cfg["vocab"], W, std=0.4), rnd(cfg["vocab"], W)
+    sd["final.norm"] = rnd(W, std=0.1, mean=1.0)
+    for i, layer in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", layer["mixer"]
+        H, d, dv = m["heads"], m["dim"], m["vdim"]
+        G = m.get("kv_heads", H)
+        mix = p + "mix."
+        sd[p + "norm1"] = rnd(W, std=0.1, mean=1.0)
+        sd[mix + "o"] = rnd(W, H * dv)
+        if layer["type"] == "attention":
+            sd.update({mix + "q": rnd(H * d, W), mix + "k": rnd(G * d, W), mix + "v": rnd(G * dv, W),
+                       mix + "vmix": uniform(0.2, 0.8)})
+        elif layer["type"] == "channel_delta":
+            r = rank or max(8, W // 8)
+            taps = m["conv"]
+            sd.update({mix + "q": rnd(G * d, W), mix + "k": rnd(G * d, W), mix + "v": rnd(H * dv, W), mix + "b": rnd(H, W),
+                       mix + "q.conv": rnd(G * d, taps), mix + "k.conv": rnd(G * d, taps), mix + "v.conv": rnd(H * dv, taps),
+                       mix + "A_log": uniform(-3.0, 1.0, H), mix + "dt_bias": uniform(-4.0, 0.5, H * d),
+                       mix + "norm": rnd(dv, std=0.1, mean=1.0), mix + "a1": rnd(r, W), mix + "a2": rnd(H * d, r),
+                       mix + "g1": rnd(r, W), mix + "g2": rnd(H * dv, r)})
+        else:
+            sd.update({mix + "q": rnd(H * d, W), mix + "k": rnd(H * d, W), mix + "v": rnd(H * dv, W), mix + "g": rnd(H * dv, W),
+                       mix + "norm": rnd(H * dv, std=0.1, mean=1.0)})
+        if layer.get("mlp"):
+            ff = layer["mlp"]["ff"]
+            sd.update({p + "norm2": rnd(W, std=0.1, mean=1.0), p + "mlp.up": rnd(ff, W), p + "mlp.down": rnd(W, ff)})
+    return sd
+
+
+def write_fuzuvik_checkpoint(path, cfg: dict, sd: Dict[str, torch.Tensor]) -> Path:
+    out = Path(path)
+    out.mkdir(parents=True, exist_ok=True)
+    (out / "config.json").write_text(json.dumps(cfg))
+    save_safetensors(sd, out / "model.safetensors")
+    return out
