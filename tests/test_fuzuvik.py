@@ -405,3 +405,59 @@ def test_router_reads_the_batch_limit():
     raw = pb.InfoResponse(max_batch_size=300).SerializeToString()
     assert pb.InfoResponse.FromString(raw).max_batch_size == 300
     assert not pb.InfoResponse().HasField("max_batch_size")
+
+
+def test_served_by_router_and_shard(tmp_path):
+    """Router and shard processes: concurrent requests, more than there are state slots, prompts longer than a prefill
+    step; every answer is the greedy continuation of its prompt alone."""
+    import os
+    import signal
+    import subprocess
+    import time
+    from concurrent.futures import ThreadPoolExecutor
+
+    from test_router_e2e import ROOT, _free_port, _get, _post
+    from tgi_b200.router.build import build
+
+    router_bin = build()
+    cfg = syn.fuzuvik_config([syn.fuzuvik_attention(chunk=24), syn.fuzuvik_delta(), syn.fuzuvik_lightning(),
+                              syn.fuzuvik_attention(chunk=24, ff=0)], width=64, vocab=300)
+    sd = syn.fuzuvik_state_dict(cfg, seed=3)
+    path = syn.write_fuzuvik_checkpoint(tmp_path / "m", cfg, sd)
+    prompts = ["hello world", "a", "the quick brown fox jumps over the lazy dog, twice", "recurrent", "0123456789" * 4]
+    n = 4
+    want = [O.greedy(cfg, sd, [b + 3 for b in p.encode()], n) for p in prompts]
+    uds, port = str(tmp_path / "s"), _free_port()
+    env = dict(os.environ, PYTHONPATH=ROOT, TGI_B200_CPU_KV_BLOCKS="64", TGI_B200_STATE_SLOTS="2", CUDA_VISIBLE_DEVICES="",
+               VIRTUAL_ENV=os.environ.get("VIRTUAL_ENV", sys.prefix))
+    shard = subprocess.Popen([sys.executable, "-m", "tgi_b200.server.cli", "serve", str(path), "--uds-path", uds,
+                              "--dtype", "float32"], env=env, cwd=ROOT)
+    router = subprocess.Popen([str(router_bin), "--master-shard-uds-path", uds, "--tokenizer-name", str(path), "--port",
+                               str(port), "--hostname", "127.0.0.1", "--max-input-tokens", "64", "--max-total-tokens", "96",
+                               "--max-batch-prefill-tokens", "64", "--repo-root", ROOT], env=env, cwd=ROOT,
+                              stderr=subprocess.PIPE, text=True)
+    try:
+        deadline = time.time() + 120
+        while time.time() < deadline:
+            assert shard.poll() is None and router.poll() is None
+            try:
+                if _get(port, "/health")[0] == 200:
+                    break
+            except Exception:
+                time.sleep(0.3)
+        ask = lambda p: _post(port, "/generate", {"inputs": p, "parameters": {"max_new_tokens": n, "details": True}})
+        with ThreadPoolExecutor(5) as ex:
+            answers = list(ex.map(ask, prompts))
+        for (st, _, body), w in zip(answers, want):
+            assert st == 200, body
+            got = [t["id"] for t in json.loads(body)["details"]["tokens"]]
+            assert got == w[:len(got)] and (len(got) == n or got[-1] == 2)
+    finally:
+        for p in (router, shard):
+            p.send_signal(signal.SIGTERM)
+        for p in (router, shard):
+            try:
+                p.wait(timeout=20)
+            except subprocess.TimeoutExpired:
+                p.kill()
+    assert "limited to 2 requests" in router.stderr.read()
