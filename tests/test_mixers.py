@@ -227,7 +227,7 @@ def delta_case(dt, G, H, d, dv, taps, rank=16):
 
 
 DELTA = [(2, 4, 24, 40, 4), (3, 3, 64, 64, 2), (1, 2, 100, 33, 3), (2, 2, 128, 128, 4), (1, 1, 150, 8, 5), (1, 3, 256, 20, 4),
-         (2, 2, 16, 130, 1)]
+         (2, 2, 16, 132, 1), (2, 4, 64, 260, 9), (2, 4, 128, 64, 7), (1, 2, 30, 50, 3)]
 
 
 @pytest.mark.parametrize("shape", DELTA, ids=str)
@@ -239,8 +239,7 @@ def test_delta_rule(be, shape):
     G, H, d, dv, taps = shape
     case, want = delta_case(dt, *shape)
     pitch = ops.recurrent_pitch(d, dev)
-    dv_ = lambda ts: [t.to(dev).contiguous() for t in ts]
-    conv, a_log, bias = dv_(case["conv"]), case["a_log"].to(dev), case["dt_bias"].to(dev)
+    conv, a_log, bias = ops.conv_weights(case["conv"], dev), case["a_log"].to(dev), case["dt_bias"].to(dev)
     for whole in (True, False):
         conv_state = torch.full((4, taps - 1, 2 * G * d + H * dv), 3.0, dtype=dt, device=dev)
         state = torch.full((4, H, dv, pitch), 5.0, device=dev)
@@ -250,7 +249,7 @@ def test_delta_rule(be, shape):
             st = Step(parts, dev)
             x = torch.cat([case["proj"][i][a:b] for i, a, b in rows]).to(dev)
             a_pre = torch.cat([case["a"][i][a:b] for i, a, b in rows]).to(dev)
-            q, k, v, g, beta, qk = ops.delta_inputs(x, case["offs"], a_pre, *conv, a_log, bias, st.cu, st.kv, st.slots,
+            q, k, v, g, beta, qk = ops.delta_inputs(x, case["offs"], a_pre, conv, a_log, bias, st.cu, st.kv, st.slots,
                                                     conv_state, G, H, d, pitch, dv, st.max_q == 1)
             for j, (i, a, b) in enumerate(rows):
                 lo, hi = int(st.cu[j]), int(st.cu[j + 1])
@@ -333,7 +332,7 @@ def test_padding_rows(be):
     conv_state = torch.full((2, 3, 2 * 48 + 160), 3.0, dtype=dt, device=dev)
     state = torch.full((2, 4, 40, 32), 5.0, device=dev)
     r = ops.delta_inputs(case["proj"][0][:3].to(dev), case["offs"], case["a"][0][:3].to(dev),
-                         *[c.to(dev) for c in case["conv"]], case["a_log"].to(dev), case["dt_bias"].to(dev), cu, kv, slots,
+                         ops.conv_weights(case["conv"], dev), case["a_log"].to(dev), case["dt_bias"].to(dev), cu, kv, slots,
                          conv_state, 2, 4, 24, 32, 40, True)
     ops.delta_scan(*r, cu, kv, slots, state, 24, 1)
     assert (state[0] == 5.0).all() and (conv_state[0] == 3.0).all() and not (state[1] == 5.0).any()

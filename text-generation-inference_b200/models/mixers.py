@@ -144,8 +144,9 @@ class GatedDelta(Mixer):
         super().__init__(spec, prefix, weights, idx, eps, comm)
         s = spec
         self.proj, self.offs = self.fused(["q", "k", "v", "b", "a1", "g1"])
-        self.conv = tuple(self.f32(f"{n}.conv") for n in ("q", "k", "v"))
-        self.taps = self.conv[0].shape[1]
+        parts = [self.f32(f"{n}.conv") for n in ("q", "k", "v")]
+        self.taps = parts[0].shape[1]
+        self.conv = ops.conv_weights(parts, self.device)
         self.a_rank, self.g_rank = (_up(self.weights.get_shape(f"{prefix}.{n}")[0]) for n in ("a1", "g1"))
         # K padded like the rows of a1 / g1: their outputs are read where the fused product left them
         self.a2, self.g2 = (FastLinear(pad_columns(self.tensor(n))) for n in ("a2", "g2"))
@@ -167,7 +168,7 @@ class GatedDelta(Mixer):
         a = self.a2(p[:, self.offs[4]:self.offs[4] + self.a_rank])
         g = self.g2(p[:, self.offs[5]:self.offs[5] + self.g_rank])
         q, k, v, decay, beta, qk = ops.delta_inputs(
-            p, self.offs, a, *self.conv, self.a_log, self.dt_bias, meta.cu_seqlens_q, meta.kv_lens, meta.state_slots,
+            p, self.offs, a, self.conv, self.a_log, self.dt_bias, meta.cu_seqlens_q, meta.kv_lens, meta.state_slots,
             conv_state, s.kv_heads, s.heads, s.dim, self.pitch, s.vdim, meta.max_q == 1)
         o = ops.delta_scan(q, k, v, decay, beta, qk, meta.cu_seqlens_q, meta.kv_lens, meta.state_slots, state, s.dim, meta.max_q)
         y = ops.gated_norm(o, g, self.norm, self.eps, s.heads, self.out_cols)

@@ -138,11 +138,20 @@ def recurrent_pitch(dim, device):
     return dim
 
 
-def delta_inputs(proj, offs, a_pre, conv_q, conv_k, conv_v, a_log, dt_bias, cu, kv_lens, state_slots, conv_state, kv_heads,
-                 heads, dim, pitch, vdim, single):
-    """Short convolutions, unit norms, decays and write strengths of a gated delta rule; advances ``conv_state``."""
-    return _mixer_backend(proj).delta_inputs(proj, offs, a_pre, conv_q, conv_k, conv_v, a_log, dt_bias, cu, kv_lens,
-                                             state_slots, conv_state, kv_heads, heads, dim, pitch, vdim, single)
+def conv_weights(parts, device):
+    """Short convolutions ``[channels, taps]`` side by side as fp32 ``[rows, channels]``, oldest tap first; the kernels want
+    a certain number of rows (absent taps are zero rows in front)."""
+    w = torch.cat([p.float() for p in parts], dim=0).t()
+    rows = native().conv_rows(w.shape[0]) if torch.device(device).type == "cuda" and not _FORCE_TORCH else w.shape[0]
+    return torch.nn.functional.pad(w, (0, 0, rows - w.shape[0], 0)).contiguous().to(device)
+
+
+def delta_inputs(proj, offs, a_pre, conv_t, a_log, dt_bias, cu, kv_lens, state_slots, conv_state, kv_heads, heads, dim, pitch,
+                 vdim, single):
+    """Short convolutions (``conv_weights`` of q, k, v), unit norms, decays and write strengths of a gated delta rule;
+    advances ``conv_state``."""
+    return _mixer_backend(proj).delta_inputs(proj, offs, a_pre, conv_t, a_log, dt_bias, cu, kv_lens, state_slots, conv_state,
+                                             kv_heads, heads, dim, pitch, vdim, single)
 
 
 def delta_scan(q, k, v, g, beta, qk, cu, kv_lens, state_slots, state, dim, max_q):

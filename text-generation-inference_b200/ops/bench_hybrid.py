@@ -1,0 +1,280 @@
+"""Prefill and decode throughput of a Fuzuvik-shaped decoder beside a Llama-shaped one of the same width, depth, heads
+and parameter count, and the kernels of both against their rooflines.
+
+``python bench.py --model fuzuvik-bf16`` prints one JSON line.  Weights are random; token rates are timed with CUDA
+events around the model's forward (prefill) and around replays of its decode graph.  Kernels are timed one by one
+with the L2 flushed in front of every launch; a roofline is the larger of bytes over the measured copy bandwidth and
+FLOPs over the measured rate of the unit that does them (bf16 tensor cores, or fp32 FMA for the state recurrences).
+"""
+from __future__ import annotations
+
+import json
+import math
+import os
+from pathlib import Path
+
+import numpy as np
+import torch
+
+FP32_TFLOPS = 148 * 128 * 2 * 1.965e9 / 1e12      # nominal: 128 fp32 FMA per SM and cycle
+
+
+def peaks():
+    f = Path(__file__).resolve().parents[2] / "MEASURED_PEAKS.json"
+    if f.exists():
+        d = json.loads(f.read_text())
+        return d["hbm_gbs"] * 1e9, d["bf16_tflops"] * 1e12, "measured"
+    return 6.65e12, 1.59e15, "fallback"
+
+
+def fuzuvik_like(width: int, layers: int, vocab: int, chunk: int) -> dict:
+    from ..utils import synthetic as syn
+
+    h, ff = width // 128, 4 * width
+    kinds = [syn.fuzuvik_attention(h, h // 4, 128, 128, chunk, ff=ff, scaling=(8.0, 1.0, 4.0, 8192), base=500000.0),
+             syn.fuzuvik_delta(h, h, 128, 128, 4, ff=ff),
+             syn.fuzuvik_attention(h, h // 4, 128, 128, chunk, ff=ff, scaling=(8.0, 1.0, 4.0, 8192), base=500000.0),
+             syn.fuzuvik_lightning(h, 128, 128, ff=ff)]
+    return syn.fuzuvik_config([kinds[i % 4] for i in range(layers)], width=width, vocab=vocab, eps=1e-6)
+
+
+def llama_like(width: int, layers: int, vocab: int) -> dict:
+    from ..utils import synthetic as syn
+
+    # a gated feed-forward of 8/3 width has the parameters of a plain one of 4 width
+    return syn.llama_config(hidden=width, layers=layers, heads=width // 128, kv_heads=width // 512,
+                            intermediate=(8 * width // 3 + 127) // 128 * 128, vocab=vocab, theta=500000.0, max_pos=16384)
+
+
+def make_runner(cfg: dict, dev):
+    from ..models.arch import ModelConfig
+    from ..models.decoder import CausalDecoder
+    from ..models.flash_causal_lm import FlashCausalLM
+    from ..utils import synthetic as syn
+    from ..utils.tokenizer import ByteTokenizer
+
+    mc = ModelConfig(cfg)
+    if cfg.get("architecture"):
+        w = syn.DictWeights(syn.fuzuvik_state_dict(cfg, dtype=torch.bfloat16, device=str(dev), rank=128), dev, torch.bfloat16,
+                            bare_names=True)
+    else:
+        w = syn.SyntheticWeights(cfg, dev, torch.bfloat16)
+    model = CausalDecoder(mc, w, max_positions=16384)
+    return FlashCausalLM(model, ByteTokenizer(mc.vocab_size), torch.bfloat16, dev)
+
+
+def timed(fn, steps: int, warmup: int) -> float:
+    """Milliseconds per call."""
+    for _ in range(warmup):
+        fn()
+    torch.cuda.synchronize()
+    a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    a.record()
+    for _ in range(steps):
+        fn()
+    b.record()
+    torch.cuda.synchronize()
+    return a.elapsed_time(b) / steps
+
+
+class Sequences:
+    """Batch of sequences with pages and (for recurrent layers) slots, driven through the runner's metadata builder."""
+
+    def __init__(self, runner, batch: int, ctx: int, vocab: int):
+        from ..models.flash_causal_lm import BLOCK_SIZE, FlashCausalLMBatch, Seq
+        from ..proto import generate_v3 as pb
+
+        per = math.ceil((ctx + 16) / BLOCK_SIZE)
+        runner.init_kv_cache(1 + batch * per, state_slots=batch)
+        rng = np.random.default_rng(0)
+        seqs = []
+        for i in range(batch):
+            blocks = list(range(1 + i * per, 1 + (i + 1) * per))
+            slots = (np.asarray(blocks, dtype=np.int32)[:, None] * BLOCK_SIZE
+                     + np.arange(BLOCK_SIZE, dtype=np.int32)[None]).reshape(-1)
+            ids = rng.integers(3, vocab, size=ctx).tolist()
+            seqs.append(Seq(request=pb.Request(id=i), ids=ids, prompt_len=ctx, cache_len=0, blocks=blocks, slots=slots,
+                            stopping=None, top_n=0, prefix_offset=0, read_offset=0))
+        self.runner, self.batch, self.ctx = runner, FlashCausalLMBatch(0, seqs, None, runner.device), ctx
+
+    def prefill(self):
+        meta, _ = self.runner.build_meta(self.batch, [self.ctx] * len(self.batch))
+        return meta
+
+
+def model_rates(cfg: dict, dev, vocab: int, prefills, decodes, steps: int, warmup: int) -> dict:
+    from ..models.graphs import DecodeGraphs
+    from . import cuda as K
+
+    runner = make_runner(cfg, dev)
+    out = {"prefill_tok_s": {}, "decode_tok_s": {}}
+    for b, t in prefills:
+        s = Sequences(runner, b, t, vocab)
+        meta = s.prefill()
+        ms = timed(lambda: runner.model.forward(meta, runner.kv_cache), max(3, steps // 4), warmup)
+        out["prefill_tok_s"][f"{b}x{t}"] = round(b * t / ms * 1e3)
+    for b, ctx in decodes:
+        s = Sequences(runner, b, ctx, vocab)
+        for q in s.batch.seqs:
+            if runner.recurrent:
+                runner.state_slot(q, 0)
+            q.cache_len, q.prefilling = ctx - 1, False
+        g = DecodeGraphs(runner, ctx + 16, buckets=[b])
+        g.capture_all()
+        g.run(s.batch, [1] * b)
+        graph = g.buckets[b].graph
+        ms = timed(graph.replay, steps, warmup)
+        out["decode_tok_s"][f"{b}@{ctx}"] = round(b / ms * 1e3)
+        del g, graph
+    assert K.check_status(dev) == 0, "a kernel wait timed out"
+    del runner
+    torch.cuda.empty_cache()
+    return out
+
+
+class KernelTimer:
+    def __init__(self, dev, iters: int = 12):
+        self.flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+        self.iters = iters
+        self.hbm, self.tensor, self.source = peaks()
+        self.rows = []
+
+    def __call__(self, name: str, fn, bytes_: float, flops: float = 0.0, unit: str = "tensor"):
+        for _ in range(3):
+            fn()
+        us = []
+        for _ in range(self.iters):
+            self.flush.zero_()
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            a.record()
+            fn()
+            b.record()
+            torch.cuda.synchronize()
+            us.append(a.elapsed_time(b) * 1e3)
+        t = sorted(us)[len(us) // 2]
+        rate = self.tensor if unit == "tensor" else FP32_TFLOPS * 1e12
+        roof = max(bytes_ / self.hbm, flops / rate) * 1e6
+        self.rows.append({"kernel": name, "us": round(t, 1), "roofline_us": round(roof, 1), "frac": round(roof / t, 3),
+                          "bound": "bytes" if bytes_ / self.hbm >= flops / rate else unit})
+
+
+def kernel_rows(dev, width: int, chunk: int, prefill, decode) -> list:
+    """Every kernel of the design at layer size, and the like kernels of the Llama-shaped model."""
+    from .. import ops
+    from . import cuda as K
+    from ..models.arch import MixerSpec
+    from ..models.mixers import RotaryTables
+    from ..utils.rotary import RotaryTable
+
+    H, G, d = width // 128, width // 512, 128
+    kt = KernelTimer(dev)
+    bf = torch.bfloat16
+    spec = MixerSpec("attention", H, G, d, d, rot_dims=d, rot_base=500000.0)
+    tab = RotaryTables(16384, dev).get(spec).cos_sin
+    taps = 4
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+    rn = lambda *s, dt=bf: torch.randn(*s, device=dev, dtype=torch.float32).to(dt)
+    for label, B, n, ctx in [("prefill", *prefill, prefill[1]), ("decode", decode[0], 1, decode[1])]:
+        T = B * n
+        tag = f"{label} {B}x{n}" + (f" @{ctx}" if n == 1 else "")
+        cu, kv, slots = i32([i * n for i in range(B + 1)]), i32([ctx] * B), i32(list(range(B)))
+        per = math.ceil(ctx / 16)
+        bt = torch.arange(B * per, dtype=torch.int32, device=dev).view(B, per)
+        pos = i32([ctx - n + i for _ in range(B) for i in range(n)])
+        page = i32([b * per * 16 + ctx - n + i for b in range(B) for i in range(n)])
+        kc, vc = rn(B * per, 16, G, d), rn(B * per, 16, G, d)
+        # ---- attention layer
+        qw = (H + 2 * G) * d
+        proj, first = rn(T, qw), rn(T, G * d)
+        offs = [0, H * d, H * d + G * d]
+        io = T * qw * 2 * 2
+        kt(f"{tag}: rotate + unit rms + value mix + store", lambda: ops.rotate_norm_store(
+            proj, offs, pos, tab, page, kc, vc, H, G, d, d, d, True, 1e-6, first, 0.3), io + T * G * d * 2)
+        kt(f"{tag}: [llama] rope + store", lambda: ops.rope_and_cache(proj, pos, tab, page, kc, vc, H, G, d, d), io)
+        q = rn(T, H, d)
+        for c, nm in ((chunk, "attention, chunk + sink"), (0, "[llama] attention")):
+            span = min(ctx, c) if c else ctx
+            if n > 1:
+                pairs = B * (sum(min(i % c + 1, i + 1) if c else i + 1 for i in range(n)))
+                by, fl = T * H * d * 4 + 2 * T * G * d * 2, 4.0 * pairs * H * d
+            else:
+                span = (ctx - 1) % c + 1 if c else ctx
+                by, fl = 2 * B * span * G * d * 2 + T * H * d * 4, 0.0
+            kt(f"{tag}: {nm}", lambda: ops.paged_attention(q, kc, vc, bt, cu, kv, d ** -0.5, max_q=n, max_kv=ctx, chunk=c,
+                                                           sink=bool(c)), by, fl)
+        # ---- delta layer
+        C = 3 * H * d
+        cols = C + (H + 7) // 8 * 8 + 256
+        x, a = rn(T, cols), rn(T, H * d)
+        conv = ops.conv_weights([torch.randn(H * d, taps, device=dev) for _ in range(3)], dev)
+        a_log, bias = torch.zeros(H, device=dev), torch.randn(H * d, device=dev) - 2
+        cs, S = torch.zeros(B, taps - 1, C, dtype=bf, device=dev), torch.zeros(B, H, d, d, device=dev)
+        do = [0, H * d, 2 * H * d, 3 * H * d]
+        prep = lambda: ops.delta_inputs(x, do, a, conv, a_log, bias, cu, kv, slots, cs, H, H, d, d, d, n == 1)
+        cbytes = B * (taps - 1) * C * 2 * (2 if n == 1 else 1)
+        kt(f"{tag}: delta inputs (conv, norms, decays)", prep, T * H * d * (4 * 2 + 4 * 4) + cbytes)
+        r = prep()
+        st = B * H * d * d * 4 * (2 if n == 1 else 1)
+        kt(f"{tag}: delta scan", lambda: ops.delta_scan(*r, cu, kv, slots, S, d, n), T * H * d * 4 * 5 + st,
+           7.0 * T * H * d * d, "fp32")
+        o = rn(T, H, d, dt=torch.float32)
+        w1 = torch.ones(d, device=dev)
+        kt(f"{tag}: norm x gate, per head", lambda: ops.gated_norm(o, a, w1, 1e-6, H, H * d), T * H * d * 8)
+        # ---- fixed-decay layer
+        dec = torch.full((H,), 0.99, device=dev)
+        y = rn(T, 4 * H * d)
+        kt(f"{tag}: decay scan", lambda: ops.decay_scan(y, [0, H * d, 2 * H * d], dec, cu, kv, slots, S, H, d, d, n),
+           T * H * d * (3 * 2 + 4) + st, 5.0 * T * H * d * d, "fp32")
+        w2 = torch.ones(H * d, device=dev)
+        kt(f"{tag}: norm x gate, whole row", lambda: ops.gated_norm(o, y[:, 3 * H * d:], w2, 1e-6, 1, H * d), T * H * d * 8)
+        # ---- common
+        res, dl, w = rn(T, width, dt=torch.float32), rn(T, width), rn(width)
+        kt(f"{tag}: residual (fp32) + norm", lambda: ops.residual_norm(dl, res, w, 1e-6), T * width * 12)
+        rb = rn(T, width)
+        kt(f"{tag}: [llama] residual (bf16) + norm", lambda: ops.rms_norm(dl, rb, w, 1e-6), T * width * 8)
+        u = rn(T, 4 * width)
+        kt(f"{tag}: gelu", lambda: ops.activation(u, "gelu"), T * 4 * width * 4)
+        gu = rn(T, 2 * (8 * width // 3 // 128 * 128))
+        kt(f"{tag}: [llama] silu x up", lambda: ops.act_and_mul(gu, "silu"), gu.numel() * 3)
+        ids, table = i32([i % 1000 for i in range(T)]), rn(1000, width)
+        kt(f"{tag}: embedding to fp32", lambda: ops.embed_residual(ids, table, 2.0), T * width * 6)
+        wq = rn(cols, width)
+        xw = rn(T, width)
+        kt(f"{tag}: GEMM q k v b a1 g1", lambda: ops.linear(xw, wq), (T + cols) * width * 2 + T * cols * 2, 2.0 * T * cols * width)
+        wl = rn(qw, width)
+        kt(f"{tag}: [llama] GEMM q k v", lambda: ops.linear(xw, wl), (T + qw) * width * 2 + T * qw * 2, 2.0 * T * qw * width)
+        w3 = rn(H * d, 128)
+        kt(f"{tag}: GEMM a2 (rank 128)", lambda: ops.linear(x[:, C + (H + 7) // 8 * 8:][:, :128], w3),
+           (T + H * d) * 256 + T * H * d * 2, 2.0 * T * H * d * 128)
+        assert K.check_status(dev) == 0
+        torch.cuda.empty_cache()
+    return kt.rows
+
+
+def run(args, clock_sampler) -> int:
+    from . import cuda as K
+
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    K.load()
+    vocab, layers, chunk = 32000, args.layers or 8, 8192
+    sampler = clock_sampler(0)
+    sampler.start()
+    sizes = {}
+    prefills, decodes = [(4, 2048), (1, 8192)], [(16, 2048), (256, 2048)]
+    for width in (2048, 4096):
+        K.LAUNCHES = 0
+        sizes[str(width)] = {
+            "fuzuvik": model_rates(fuzuvik_like(width, layers, vocab, chunk), dev, vocab, prefills, decodes, args.steps, args.warmup),
+            "llama": model_rates(llama_like(width, layers, vocab), dev, vocab, prefills, decodes, args.steps, args.warmup)}
+    rows = kernel_rows(dev, 4096, chunk, (4, 2048), (256, 2048))
+    clocks = sampler.stop()
+    value = sizes["4096"]["fuzuvik"]["decode_tok_s"]["256@2048"]
+    print(json.dumps({
+        "metric": "output tok/s (decode, fuzuvik-bf16)", "value": value, "unit": "tok/s", "n_gpus": 1, "steps": args.steps,
+        "warmup": args.warmup, "ms_per_step": round(256e3 / value, 4), "higher_is_better": True, "scaling": "strong",
+        "vs_baseline": None, "dtype": "bf16", "data": "synthetic: random tokens, random weights", "impl": "b200",
+        "config": {"model": f"fuzuvik-{layers}L", "global_batch": 256, "seq_len": 2048, "chunk": chunk, "parallelism": "tp1",
+                   "l2": "models: inputs larger than L2; kernels: L2 flushed before every launch"},
+        "sizes": sizes, "kernels": rows, "peaks": peaks()[2], "clocks": clocks}), flush=True)
+    return 0

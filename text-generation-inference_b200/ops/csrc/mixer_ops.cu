@@ -182,7 +182,7 @@ __global__ void __launch_bounds__(256)
 attn_prep_kernel(const T* __restrict__ proj, long long ld, int off_k, int off_v, const int* __restrict__ positions,
                  const float* __restrict__ cos_sin, const int* __restrict__ slots, const T* __restrict__ v_first,
                  long long ld_first, float lambda, T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache,
-                 T* __restrict__ v_mixed, int T_, int Hq, int Hkv, int dim, int vdim, int Dk, int Dv, int rot, int max_pos,
+                 int T_, int Hq, int Hkv, int dim, int vdim, int Dk, int Dv, int rot, int max_pos,
                  long long num_slots, int qk_norm, float eps) {
   tgi::pdl_wait();
   tgi::pdl_trigger();
@@ -196,14 +196,13 @@ attn_prep_kernel(const T* __restrict__ proj, long long ld, int off_k, int off_v,
   const T* row = proj + static_cast<size_t>(t) * ld;
   if (h >= Hq + Hkv) {
     const int g = h - Hq - Hkv;
-    if (!slot_ok && v_mixed == nullptr) return;
+    if (!slot_ok) return;
     const T* v = row + off_v + static_cast<size_t>(g) * vdim;
     const T* f = v_first != nullptr ? v_first + static_cast<size_t>(t) * ld_first + static_cast<size_t>(g) * vdim : nullptr;
     for (int i = lane; i < vdim; i += 32) {
       float x = to_f(v[i]);
       if (f != nullptr) x = (1.f - lambda) * x + lambda * to_f(f[i]);
-      if (slot_ok) put(v_cache + (static_cast<size_t>(slot) * Hkv + g) * Dv + i, x);
-      if (v_mixed != nullptr) put(v_mixed + (static_cast<size_t>(t) * Hkv + g) * vdim + i, x);
+      put(v_cache + (static_cast<size_t>(slot) * Hkv + g) * Dv + i, x);
     }
     return;
   }
@@ -234,6 +233,81 @@ attn_prep_kernel(const T* __restrict__ proj, long long ld, int off_k, int off_v,
   for (int i = rot + lane; i < dim; i += 32) put(dst + i, to_f(x[i]) * inv);
   if (is_q)
     for (int i = dim + lane; i < Dk; i += 32) put(dst + i, 0.f);
+}
+
+// The same for rows that can be read four elements at a time (every offset, size and pitch a multiple of 4, `rot` of 8):
+// one CTA per token, sixteen lanes per head, all pieces of a head in registers between the norm and the store.
+template <typename T, int NP>
+__global__ void __launch_bounds__(256)
+attn_prep_vec_kernel(const T* __restrict__ proj, long long ld, int off_k, int off_v, const int* __restrict__ positions,
+                     const float* __restrict__ cos_sin, const int* __restrict__ slots, const T* __restrict__ v_first,
+                     long long ld_first, float lambda, T* __restrict__ q_out, T* __restrict__ k_cache,
+                     T* __restrict__ v_cache, int Hq, int Hkv, int dim, int vdim, int Dk, int Dv, int rot, int max_pos,
+                     long long num_slots, int qk_norm, float eps) {
+  tgi::pdl_wait();
+  tgi::pdl_trigger();
+  const int t = blockIdx.x, l = threadIdx.x & 15;
+  const long long slot = slots[t];
+  const bool slot_ok = slot >= 0 && slot < num_slots;
+  const T* row = proj + static_cast<size_t>(t) * ld;
+  const int pos = min(max(positions[t], 0), max_pos - 1);
+  const float* cs = cos_sin + static_cast<size_t>(pos) * rot;
+  const int rh = rot / 2;
+  const int heads = Hq + 2 * Hkv, groups = blockDim.x >> 4;
+  for (int h0 = 0; h0 < heads; h0 += groups) {          // all lanes of a warp stay in the loop (shuffles below)
+    const int h = h0 + (threadIdx.x >> 4);
+    if (h >= Hq + Hkv) {
+      const int g = h - Hq - Hkv;
+      if (g < Hkv && slot_ok) {
+        const T* v = row + off_v + static_cast<size_t>(g) * vdim;
+        const T* f = v_first + static_cast<size_t>(t) * ld_first + static_cast<size_t>(g) * vdim;
+        for (int i = 4 * l; i < vdim; i += 64) {
+          float4 x = load4(v + i);
+          if (v_first != nullptr) {
+            const float4 y = load4(f + i);
+            const float m = 1.f - lambda;
+            x = make_float4(m * x.x + lambda * y.x, m * x.y + lambda * y.y, m * x.z + lambda * y.z, m * x.w + lambda * y.w);
+          }
+          store4(v_cache + (static_cast<size_t>(slot) * Hkv + g) * Dv + i, x);
+        }
+      }
+    }
+    const bool qk = h < Hq + Hkv, is_q = h < Hq;
+    const int g = is_q ? h : h - Hq;
+    const T* x = row + (is_q ? 0 : off_k) + static_cast<size_t>(g) * dim;
+    float4 u[NP], w[NP], r[NP];                           // rotated pairs, dimensions past the rotated ones
+    float ss = 0.f;
+#pragma unroll
+    for (int e = 0; e < NP; ++e) {
+      const int i = 4 * (l + 16 * e);
+      u[e] = w[e] = r[e] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (qk && i < rh) {
+        const float4 a = load4(x + i), b = load4(x + rh + i);
+        const float4 c = *reinterpret_cast<const float4*>(cs + i), s = *reinterpret_cast<const float4*>(cs + rh + i);
+        u[e] = make_float4(a.x * c.x - b.x * s.x, a.y * c.y - b.y * s.y, a.z * c.z - b.z * s.z, a.w * c.w - b.w * s.w);
+        w[e] = make_float4(b.x * c.x + a.x * s.x, b.y * c.y + a.y * s.y, b.z * c.z + a.z * s.z, b.w * c.w + a.w * s.w);
+      }
+      if (qk && rot + i < dim) r[e] = load4(x + rot + i);
+      ss += u[e].x * u[e].x + u[e].y * u[e].y + u[e].z * u[e].z + u[e].w * u[e].w + w[e].x * w[e].x + w[e].y * w[e].y +
+            w[e].z * w[e].z + w[e].w * w[e].w + r[e].x * r[e].x + r[e].y * r[e].y + r[e].z * r[e].z + r[e].w * r[e].w;
+    }
+#pragma unroll
+    for (int o = 8; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (!qk || (!is_q && !slot_ok)) continue;
+    const float inv = qk_norm ? 1.f / sqrtf(ss / dim + eps) : 1.f;
+    T* dst = is_q ? q_out + (static_cast<size_t>(t) * Hq + g) * Dk : k_cache + (static_cast<size_t>(slot) * Hkv + g) * Dk;
+#pragma unroll
+    for (int e = 0; e < NP; ++e) {
+      const int i = 4 * (l + 16 * e);
+      if (i < rh) {
+        store4(dst + i, make_float4(u[e].x * inv, u[e].y * inv, u[e].z * inv, u[e].w * inv));
+        store4(dst + rh + i, make_float4(w[e].x * inv, w[e].y * inv, w[e].z * inv, w[e].w * inv));
+      }
+      if (rot + i < dim) store4(dst + rot + i, make_float4(r[e].x * inv, r[e].y * inv, r[e].z * inv, r[e].w * inv));
+    }
+    if (is_q)
+      for (int i = dim + 4 * l; i < Dk; i += 64) store4(dst + i, make_float4(0.f, 0.f, 0.f, 0.f));
+  }
 }
 
 // ------------------------------------------------------------------------------------------------
@@ -340,7 +414,7 @@ struct DeltaPrep {
 template <typename T>
 __device__ __forceinline__ float conv_value(const T* __restrict__ proj, long long ld, int col, int t, int i,
                                             const float* __restrict__ w, const T* __restrict__ st, int C, int c,
-                                            int taps) {
+                                            int taps) {   // w: the channel's first tap, taps C floats apart
   float acc = 0.f;
   for (int j = 0; j < taps - 1; ++j) {             // tap j multiplies the input taps - 1 - j tokens back
     const int back = taps - 1 - j;
@@ -350,16 +424,15 @@ __device__ __forceinline__ float conv_value(const T* __restrict__ proj, long lon
     } else if (st != nullptr) {
       v = to_f(st[static_cast<size_t>(taps - 1 + i - back) * C + c]);
     }
-    acc = fmaf(w[j], v, acc);
+    acc = fmaf(w[static_cast<size_t>(j) * C], v, acc);
   }
-  return fmaf(w[taps - 1], to_f(proj[static_cast<size_t>(t) * ld + col]), acc);
+  return fmaf(w[static_cast<size_t>(taps - 1) * C], to_f(proj[static_cast<size_t>(t) * ld + col]), acc);
 }
 
 template <typename T, int NV>
 __global__ void __launch_bounds__(256)
-delta_prep_kernel(const T* __restrict__ proj, const T* __restrict__ a_pre, const float* __restrict__ conv_q,
-                  const float* __restrict__ conv_k, const float* __restrict__ conv_v, const float* __restrict__ A_log,
-                  const float* __restrict__ dt_bias, const int* __restrict__ cu, const int* __restrict__ kv_lens,
+delta_prep_kernel(const T* __restrict__ proj, const T* __restrict__ a_pre, const float* __restrict__ conv_t,
+                  const float* __restrict__ A_log, const float* __restrict__ dt_bias, const int* __restrict__ cu, const int* __restrict__ kv_lens,
                   const int* __restrict__ state_slots, T* __restrict__ conv_state, float* __restrict__ q_out,
                   float* __restrict__ k_out, float* __restrict__ v_out, float* __restrict__ g_out,
                   float* __restrict__ beta_out, float* __restrict__ qk_out, int T_, int num_slots, DeltaPrep p) {
@@ -409,10 +482,8 @@ delta_prep_kernel(const T* __restrict__ proj, const T* __restrict__ a_pre, const
       q[e] = k[e] = 0.f;
       if (i < p.dim) {
         const int c = u * p.dim + i, ck = p.G * p.dim + c;
-        q[e] = silu_f(conv_value(proj, p.ld, p.off_q + c, t, i0, conv_q + static_cast<size_t>(c) * p.taps, old, C, c,
-                                 p.taps));
-        k[e] = silu_f(conv_value(proj, p.ld, p.off_k + c, t, i0, conv_k + static_cast<size_t>(c) * p.taps, old, C, ck,
-                                 p.taps));
+        q[e] = silu_f(conv_value(proj, p.ld, p.off_q + c, t, i0, conv_t + c, old, C, c, p.taps));
+        k[e] = silu_f(conv_value(proj, p.ld, p.off_k + c, t, i0, conv_t + ck, old, C, ck, p.taps));
         if (shift) {
           shift_state(c, p.off_q + c);
           shift_state(ck, p.off_k + c);
@@ -441,11 +512,174 @@ delta_prep_kernel(const T* __restrict__ proj, const T* __restrict__ a_pre, const
   for (int i = lane; i < p.vdim; i += 32) {
     const int cv = h * p.vdim + i, c = 2 * p.G * p.dim + cv;
     v_out[(static_cast<size_t>(t) * p.H + h) * p.vdim + i] = silu_f(
-        conv_value(proj, p.ld, p.off_v + cv, t, i0, conv_v + static_cast<size_t>(cv) * p.taps, old, C, c, p.taps));
+        conv_value(proj, p.ld, p.off_v + cv, t, i0, conv_t + c, old, C, c, p.taps));
     if (shift) shift_state(c, p.off_v + cv);
   }
   if (lane == 0)
     beta_out[static_cast<size_t>(t) * p.H + h] = sigmoid_f(to_f(proj[static_cast<size_t>(t) * p.ld + p.off_b + h]));
+}
+
+// The same for up to TAPS <= 8 taps, with one warp per (run of `run` consecutive rows, unit): convolution weights and
+// the window of previous inputs stay in registers while the warp walks the rows, four channels per lane and piece
+// (E pieces of 128 channels).  Weights come as [TAPS][C] with absent taps zero, so the window is always TAPS - 1 long.
+// Units as above; the convolved values of q and k go through one window each.
+template <typename T, int TAPS>
+struct ConvWindow {
+  float4 w[TAPS], x[TAPS - 1];       // weights; previous inputs, oldest first
+  __device__ __forceinline__ void weights(const float* __restrict__ wt, int C, int c, int lim) {
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j)
+      w[j] = c < lim ? *reinterpret_cast<const float4*>(wt + static_cast<size_t>(j) * C + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  // inputs before the row t (local index i of its sequence): rows of this step, then the state, then zeros
+  __device__ __forceinline__ void start(const T* __restrict__ col, long long ld, int t, int i, const T* __restrict__ st, int C,
+                                        int taps, bool ok) {
+#pragma unroll
+    for (int j = 0; j < TAPS - 1; ++j) {
+      const int back = TAPS - 1 - j;
+      x[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (!ok) continue;
+      if (i >= back) x[j] = load4(col + static_cast<long long>(t - back) * ld);
+      else if (st != nullptr && taps - 1 + i - back >= 0) x[j] = load4(st + static_cast<size_t>(taps - 1 + i - back) * C);
+    }
+  }
+  __device__ __forceinline__ float4 push(float4 v) {
+    float4 a = make_float4(w[TAPS - 1].x * v.x, w[TAPS - 1].y * v.y, w[TAPS - 1].z * v.z, w[TAPS - 1].w * v.w);
+#pragma unroll
+    for (int j = 0; j < TAPS - 1; ++j) {
+      a.x = fmaf(w[j].x, x[j].x, a.x);
+      a.y = fmaf(w[j].y, x[j].y, a.y);
+      a.z = fmaf(w[j].z, x[j].z, a.z);
+      a.w = fmaf(w[j].w, x[j].w, a.w);
+    }
+#pragma unroll
+    for (int j = 0; j + 1 < TAPS - 1; ++j) x[j] = x[j + 1];
+    x[TAPS - 2] = v;
+    return make_float4(silu_f(a.x), silu_f(a.y), silu_f(a.z), silu_f(a.w));
+  }
+  // after the last push the window holds the new state (single-token steps)
+  __device__ __forceinline__ void save(T* __restrict__ st, int C, int taps, bool ok) const {
+#pragma unroll
+    for (int j = 0; j < TAPS - 1; ++j) {
+      const int e = j - (TAPS - taps);
+      if (ok && e >= 0) store4(st + static_cast<size_t>(e) * C, x[j]);
+    }
+  }
+};
+__device__ __forceinline__ float dot4(float4 a, float4 b) { return a.x * b.x + a.y * b.y + a.z * b.z + a.w * b.w; }
+__device__ __forceinline__ float decay_value(float z, float rate) {
+  return expf(-rate * (z > 20.f ? z : log1pf(expf(z))));
+}
+
+template <typename T, int E, int TAPS>
+__global__ void __launch_bounds__(128)
+delta_prep_run_kernel(const T* __restrict__ proj, const T* __restrict__ a_pre, const float* __restrict__ conv_t,
+                      const float* __restrict__ A_log, const float* __restrict__ dt_bias, const int* __restrict__ cu,
+                      const int* __restrict__ kv_lens, const int* __restrict__ state_slots, T* __restrict__ conv_state,
+                      float* __restrict__ q_out, float* __restrict__ k_out, float* __restrict__ v_out,
+                      float* __restrict__ g_out, float* __restrict__ beta_out, float* __restrict__ qk_out, int T_,
+                      int num_slots, int run, DeltaPrep p) {
+  tgi::pdl_wait();
+  tgi::pdl_trigger();
+  const int lane = threadIdx.x & 31;
+  const int u = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (u >= p.G + 2 * p.H) return;
+  const int t0 = blockIdx.x * run, t1 = min(T_, t0 + run);
+  if (u >= p.G + p.H) {
+    const int h = u - p.G - p.H;
+    const float rate = expf(A_log[h]);
+#pragma unroll
+    for (int e = 0; e < E; ++e) {
+      const int i = 4 * lane + 128 * e;
+      if (i >= p.dimP) continue;
+      const bool in = i < p.dim;
+      const float4 bias = in ? *reinterpret_cast<const float4*>(dt_bias + h * p.dim + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      for (int t = t0; t < t1; ++t) {
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (in) {
+          const float4 a = load4(a_pre + static_cast<size_t>(t) * p.ld_a + h * p.dim + i);
+          v = make_float4(decay_value(a.x + bias.x, rate), decay_value(a.y + bias.y, rate), decay_value(a.z + bias.z, rate),
+                          decay_value(a.w + bias.w, rate));
+        }
+        store4(g_out + (static_cast<size_t>(t) * p.H + h) * p.dimP + i, v);
+      }
+    }
+    return;
+  }
+  const int C = 2 * p.G * p.dim + p.H * p.vdim;
+  const bool is_v = u >= p.G;
+  const int h = is_v ? u - p.G : u, width = is_v ? p.vdim : p.dim;
+  // channel and column of the head's first element: q (or v), and k
+  const int ca = is_v ? 2 * p.G * p.dim + h * p.vdim : h * p.dim, ck = p.G * p.dim + h * p.dim;
+  const int cola = (is_v ? p.off_v + h * p.vdim : p.off_q + h * p.dim), colk = p.off_k + h * p.dim;
+  ConvWindow<T, TAPS> wa[E], wk[E];
+#pragma unroll
+  for (int e = 0; e < E; ++e) {
+    const int i = 4 * lane + 128 * e;
+    wa[e].weights(conv_t, C, ca + i, ca + width);
+    if (!is_v) wk[e].weights(conv_t, C, ck + i, ck + width);
+  }
+  int b = sequence_of(cu, p.B, t0), next = t0;     // `next`: the row where a window has to be set up
+  T* st = nullptr;
+  for (int t = t0; t < t1; ++t) {
+    if (t == next) {
+      while (cu[b + 1] <= t) ++b;                  // sequences without tokens in this step are skipped
+      next = cu[b + 1];
+      const int n = next - cu[b], slot = state_slots[b];
+      st = slot >= 0 && slot < num_slots ? conv_state + static_cast<size_t>(slot) * (p.taps - 1) * C : nullptr;
+      const T* old = kv_lens[b] - n > 0 ? st : nullptr;
+#pragma unroll
+      for (int e = 0; e < E; ++e) {
+        const int i = 4 * lane + 128 * e;
+        wa[e].start(proj + cola + i, p.ld, t, t - cu[b], old != nullptr ? old + ca + i : nullptr, C, p.taps, i < width);
+        if (!is_v) wk[e].start(proj + colk + i, p.ld, t, t - cu[b], old != nullptr ? old + ck + i : nullptr, C, p.taps, i < width);
+      }
+    }
+    const T* row = proj + static_cast<size_t>(t) * p.ld;
+    float4 a[E], k[E];
+    float sq = 0.f, sk = 0.f, dq = 0.f;
+#pragma unroll
+    for (int e = 0; e < E; ++e) {
+      const int i = 4 * lane + 128 * e;
+      const float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
+      a[e] = wa[e].push(i < width ? load4(row + cola + i) : z);
+      if (!is_v) {
+        k[e] = wk[e].push(i < width ? load4(row + colk + i) : z);
+        sq += dot4(a[e], a[e]);
+        sk += dot4(k[e], k[e]);
+        dq += dot4(a[e], k[e]);
+      }
+    }
+    if (is_v) {
+#pragma unroll
+      for (int e = 0; e < E; ++e) {
+        const int i = 4 * lane + 128 * e;
+        if (i < width) store4(v_out + (static_cast<size_t>(t) * p.H + h) * p.vdim + i, a[e]);
+      }
+      if (lane == 0) beta_out[static_cast<size_t>(t) * p.H + h] = sigmoid_f(to_f(row[p.off_b + h]));
+    } else {
+      const float iq = 1.f / (sqrtf(warp_sum(sq) + 1e-6f) * sqrtf(static_cast<float>(p.dim)));
+      const float ik = 1.f / sqrtf(warp_sum(sk) + 1e-6f);
+      dq = warp_sum(dq);
+#pragma unroll
+      for (int e = 0; e < E; ++e) {
+        const int i = 4 * lane + 128 * e;
+        if (i >= p.dimP) continue;
+        const size_t o = (static_cast<size_t>(t) * p.G + h) * p.dimP + i;
+        store4(q_out + o, make_float4(a[e].x * iq, a[e].y * iq, a[e].z * iq, a[e].w * iq));
+        store4(k_out + o, make_float4(k[e].x * ik, k[e].y * ik, k[e].z * ik, k[e].w * ik));
+      }
+      if (lane == 0) qk_out[static_cast<size_t>(t) * p.G + h] = dq * iq * ik;
+    }
+  }
+  if (p.update && st != nullptr) {                 // run == 1: this warp alone reads and writes these channels' state
+#pragma unroll
+    for (int e = 0; e < E; ++e) {
+      const int i = 4 * lane + 128 * e;
+      wa[e].save(st + ca + i, C, p.taps, i < width);
+      if (!is_v) wk[e].save(st + ck + i, C, p.taps, i < width);
+    }
+  }
 }
 
 // last taps - 1 inputs of every sequence that contributed tokens -> its convolution state.  Grid (channels / 256, B).
@@ -474,7 +708,7 @@ conv_state_kernel(const T* __restrict__ proj, const int* __restrict__ cu, const 
 // ------------------------------------------------------------------------------------------------
 // out = RMSNorm(o over `width`) * weight * sigmoid(gate).  o fp32 [T, groups, width]; gate at column `off` of a
 // [T, ld] matrix; out rows are `ld_out` wide, columns past groups * width are zeroed by group 0.
-// One warp (width <= 1024) or one block per (token, group).
+// One warp (width <= 1024) or one block per (token, group); grid (tokens, groups / warps of a block).
 // ------------------------------------------------------------------------------------------------
 template <typename T, bool WARP>
 __global__ void __launch_bounds__(256)
@@ -484,16 +718,39 @@ gated_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, long 
   tgi::pdl_wait();
   tgi::pdl_trigger();
   __shared__ float red[33];
-  const long long job = WARP ? static_cast<long long>(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5)
-                             : static_cast<long long>(blockIdx.x);
-  if (job >= static_cast<long long>(T_) * groups) return;      // warp- or block-uniform
-  const int t = static_cast<int>(job / groups), g = static_cast<int>(job % groups);
+  const int t = blockIdx.x;
+  const int g = WARP ? blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5) : blockIdx.y;
+  if (g >= groups) return;                                      // warp- or block-uniform
   const int first = WARP ? (threadIdx.x & 31) : threadIdx.x, step = WARP ? 32 : blockDim.x;
   const float* x = o + (static_cast<size_t>(t) * groups + g) * width;
   const T* gt = gate + static_cast<size_t>(t) * ld + off + static_cast<size_t>(g) * width;
   T* dst = out + static_cast<size_t>(t) * ld_out + static_cast<size_t>(g) * width;
   float ss = 0.f;
   const bool vec = width % 4 == 0 && ld % 4 == 0 && off % 4 == 0 && ld_out % 4 == 0;
+  constexpr int NV = WARP ? 2 : 8;                              // pieces per thread kept in registers
+  if (vec && width <= NV * 4 * step) {
+    float4 v[NV];
+#pragma unroll
+    for (int e = 0; e < NV; ++e) {
+      const int i = (first + e * step) * 4;
+      v[e] = i < width ? load4(x + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      ss += dot4(v[e], v[e]);
+    }
+    ss = WARP ? warp_sum(ss) : block_sum(ss, red);
+    const float inv = 1.f / sqrtf(ss / width + eps);
+#pragma unroll
+    for (int e = 0; e < NV; ++e) {
+      const int i = (first + e * step) * 4;
+      if (i < width) {
+        const float4 w = load4(weight + i), s = load4(gt + i);
+        store4(dst + i, make_float4(v[e].x * inv * w.x * sigmoid_f(s.x), v[e].y * inv * w.y * sigmoid_f(s.y),
+                                    v[e].z * inv * w.z * sigmoid_f(s.z), v[e].w * inv * w.w * sigmoid_f(s.w)));
+      }
+    }
+    if (g == 0)
+      for (int i = groups * width + first; i < ld_out; i += step) put(out + static_cast<size_t>(t) * ld_out + i, 0.f);
+    return;
+  }
   if (vec) {
     for (int i = first * 4; i < width; i += step * 4) {
       const float4 v = load4(x + i);
@@ -516,6 +773,9 @@ gated_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, long 
   if (g == 0)
     for (int i = groups * width + first; i < ld_out; i += step) put(out + static_cast<size_t>(t) * ld_out + i, 0.f);
 }
+
+// rows of the transposed convolution weights: absent taps in front are zero rows
+int delta_tap_rows(int taps) { return taps <= 4 ? 4 : (taps <= 8 ? 8 : taps); }
 
 int done() { return cudaGetLastError() == cudaSuccess ? 0 : -3; }
 
@@ -560,37 +820,55 @@ int attn_any(const void* q, const void* k, const void* v, const int* bt, const i
 }
 
 template <typename T>
-int delta_prep(const void* proj, const void* a_pre, const float* cq, const float* ck, const float* cv, const float* A_log,
-               const float* dt_bias, const int* cu, const int* kv, const int* slots, void* conv_state, float* q, float* k,
-               float* v, float* g, float* beta, float* qk, int T_, int num_slots, const DeltaPrep& p, cudaStream_t stream) {
+int delta_prep(const void* proj, const void* a_pre, const float* conv_t, const float* A_log, const float* dt_bias,
+               const int* cu, const int* kv, const int* slots, void* conv_state, float* q, float* k, float* v, float* g,
+               float* beta, float* qk, int T_, int num_slots, const DeltaPrep& p, cudaStream_t stream) {
   const T* x = static_cast<const T*>(proj);
+  const T* a = static_cast<const T*>(a_pre);
   T* st = static_cast<T*>(conv_state);
-  const long long jobs = static_cast<long long>(T_) * (p.G + 2 * p.H);
-  const dim3 grid(static_cast<unsigned>((jobs + 7) / 8));
-  auto go = [&](auto kern) {
-    tgi::launch(kern, grid, dim3(256), 0, stream, x, static_cast<const T*>(a_pre), cq, ck, cv, A_log, dt_bias, cu, kv, slots,
-                st, q, k, v, g, beta, qk, T_, num_slots, p);
-  };
-  if (p.dimP <= 64) go(delta_prep_kernel<T, 2>);
-  else if (p.dimP <= 128) go(delta_prep_kernel<T, 4>);
-  else go(delta_prep_kernel<T, 8>);
-  if (!p.update && p.taps > 1) {
-    const int C = 2 * p.G * p.dim + p.H * p.vdim;
-    tgi::launch(conv_state_kernel<T>, dim3((C + 255) / 256, p.B), dim3(256), 0, stream, x, cu, kv, slots, st, num_slots, p);
+  const int units = p.G + 2 * p.H, C = 2 * p.G * p.dim + p.H * p.vdim;
+  const bool vec = p.taps <= 8 && p.dim % 4 == 0 && p.vdim % 4 == 0 && p.vdim <= 256 && p.ld % 4 == 0 && p.ld_a % 4 == 0 &&
+                   p.off_q % 4 == 0 && p.off_k % 4 == 0 && p.off_v % 4 == 0 &&
+                   reinterpret_cast<uintptr_t>(proj) % (4 * sizeof(T)) == 0 &&
+                   reinterpret_cast<uintptr_t>(a_pre) % (4 * sizeof(T)) == 0;
+  if (vec) {
+    const int run = p.update ? 1 : 16;
+    const dim3 grid((T_ + run - 1) / run, (units + 3) / 4);
+    auto go = [&](auto kern) {
+      tgi::launch(kern, grid, dim3(128), 0, stream, x, a, conv_t, A_log, dt_bias, cu, kv, slots, st, q, k, v, g, beta, qk, T_,
+                  num_slots, run, p);
+    };
+    const bool one = p.dimP <= 128 && p.vdim <= 128;
+    if (p.taps <= 4) one ? go(delta_prep_run_kernel<T, 1, 4>) : go(delta_prep_run_kernel<T, 2, 4>);
+    else one ? go(delta_prep_run_kernel<T, 1, 8>) : go(delta_prep_run_kernel<T, 2, 8>);
+  } else {
+    const float* first = conv_t + static_cast<size_t>(delta_tap_rows(p.taps) - p.taps) * C;
+    const long long jobs = static_cast<long long>(T_) * units;
+    const dim3 grid(static_cast<unsigned>((jobs + 7) / 8));
+    auto go = [&](auto kern) {
+      tgi::launch(kern, grid, dim3(256), 0, stream, x, a, first, A_log, dt_bias, cu, kv, slots, st, q, k, v, g, beta, qk, T_,
+                  num_slots, p);
+    };
+    if (p.dimP <= 64) go(delta_prep_kernel<T, 2>);
+    else if (p.dimP <= 128) go(delta_prep_kernel<T, 4>);
+    else go(delta_prep_kernel<T, 8>);
   }
+  if (!p.update && p.taps > 1)
+    tgi::launch(conv_state_kernel<T>, dim3((C + 255) / 256, p.B), dim3(256), 0, stream, x, cu, kv, slots, st, num_slots, p);
   return done();
 }
 
 template <typename T>
 int gated_norm(const float* o, const void* gate, long long ld, int off, const float* w, void* out, long long ld_out, int T_,
                int groups, int width, float eps, cudaStream_t stream) {
-  const long long jobs = static_cast<long long>(T_) * groups;
-  if (width <= 1024)
-    tgi::launch(gated_norm_kernel<T, true>, dim3(static_cast<unsigned>((jobs + 7) / 8)), dim3(256), 0, stream, o,
+  if (width <= 1024) {
+    const int warps = groups < 8 ? groups : 8;
+    tgi::launch(gated_norm_kernel<T, true>, dim3(T_, (groups + warps - 1) / warps), dim3(32 * warps), 0, stream, o,
                 static_cast<const T*>(gate), ld, off, w, static_cast<T*>(out), ld_out, T_, groups, width, eps);
-  else
-    tgi::launch(gated_norm_kernel<T, false>, dim3(static_cast<unsigned>(jobs)), dim3(256), 0, stream, o,
-                static_cast<const T*>(gate), ld, off, w, static_cast<T*>(out), ld_out, T_, groups, width, eps);
+  } else {
+    tgi::launch(gated_norm_kernel<T, false>, dim3(T_, groups), dim3(256), 0, stream, o, static_cast<const T*>(gate), ld, off, w,
+                static_cast<T*>(out), ld_out, T_, groups, width, eps);
+  }
   return done();
 }
 
@@ -627,17 +905,35 @@ int tgi_activation(int f32, const void* in, void* out, long long n, int act, cud
 
 int tgi_attn_prep(int f32, const void* proj, long long ld, int off_k, int off_v, const int* positions, const float* cos_sin,
                   const int* slots, const void* v_first, long long ld_first, float lambda, void* q_out, void* k_cache,
-                  void* v_cache, void* v_mixed, int T, int Hq, int Hkv, int dim, int vdim, int Dk, int Dv, int rot, int max_pos,
+                  void* v_cache, int T, int Hq, int Hkv, int dim, int vdim, int Dk, int Dv, int rot, int max_pos,
                   long long num_slots, int qk_norm, float eps, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (rot % 2 != 0 || rot > dim || Dk < dim || Dv < vdim) return -10;
+  const bool vec = rot % 8 == 0 && ld % 4 == 0 && off_k % 4 == 0 && off_v % 4 == 0 && ld_first % 4 == 0 && dim % 4 == 0 &&
+                   vdim % 4 == 0 && Dk % 4 == 0 && Dv % 4 == 0 && dim <= 256 &&
+                   reinterpret_cast<uintptr_t>(proj) % (f32 ? 16 : 8) == 0 &&
+                   reinterpret_cast<uintptr_t>(v_first) % (f32 ? 16 : 8) == 0;
+  if (vec) {
+    auto go = [&](auto kern, auto tag) {
+      using E = decltype(tag);
+      tgi::launch(kern, dim3(T), dim3(256), 0, stream, static_cast<const E*>(proj), ld, off_k, off_v, positions, cos_sin,
+                  slots, static_cast<const E*>(v_first), ld_first, lambda, static_cast<E*>(q_out), static_cast<E*>(k_cache),
+                  static_cast<E*>(v_cache), Hq, Hkv, dim, vdim, Dk, Dv, rot, max_pos, num_slots, qk_norm, eps);
+      return done();
+    };
+    // pieces per lane: rotated halves and the rest are each at most NP x 64 elements
+    const int np = (max(rot / 2, dim - rot) + 63) / 64;
+    if (np <= 1) return f32 ? go(attn_prep_vec_kernel<float, 1>, float()) : go(attn_prep_vec_kernel<bf16, 1>, bf16());
+    if (np <= 2) return f32 ? go(attn_prep_vec_kernel<float, 2>, float()) : go(attn_prep_vec_kernel<bf16, 2>, bf16());
+    return f32 ? go(attn_prep_vec_kernel<float, 4>, float()) : go(attn_prep_vec_kernel<bf16, 4>, bf16());
+  }
   const long long jobs = static_cast<long long>(T) * (Hq + 2 * Hkv);
   const dim3 grid(static_cast<unsigned>((jobs + 7) / 8));
   auto go = [&](auto kern, auto tag) {
     using E = decltype(tag);
     tgi::launch(kern, grid, dim3(256), 0, stream, static_cast<const E*>(proj), ld, off_k, off_v, positions, cos_sin, slots,
                 static_cast<const E*>(v_first), ld_first, lambda, static_cast<E*>(q_out), static_cast<E*>(k_cache),
-                static_cast<E*>(v_cache), static_cast<E*>(v_mixed), T, Hq, Hkv, dim, vdim, Dk, Dv, rot, max_pos, num_slots,
+                static_cast<E*>(v_cache), T, Hq, Hkv, dim, vdim, Dk, Dv, rot, max_pos, num_slots,
                 qk_norm, eps);
     return done();
   };
@@ -657,18 +953,21 @@ int tgi_attn_any(int f32, const void* q, const void* k_cache, const void* v_cach
                               scale, window, chunk, sink, stream);
 }
 
+// Rows of the [rows][channels] convolution weights tgi_delta_prep wants for `taps` taps (the first rows are zero).
+int tgi_delta_tap_rows(int taps) { return delta_tap_rows(taps); }
+
 int tgi_delta_prep(int f32, const void* proj, long long ld, int off_q, int off_k, int off_v, int off_b, const void* a_pre,
-                   long long ld_a, const float* conv_q, const float* conv_k, const float* conv_v, const float* A_log,
-                   const float* dt_bias, const int* cu, const int* kv_lens, const int* state_slots, void* conv_state, float* q,
-                   float* k, float* v, float* g, float* beta, float* qk, int T, int B, int num_slots, int G, int H, int dim,
-                   int dimP, int vdim, int taps, int update, cudaStream_t stream) {
+                   long long ld_a, const float* conv_t, const float* A_log, const float* dt_bias, const int* cu,
+                   const int* kv_lens, const int* state_slots, void* conv_state, float* q, float* k, float* v, float* g,
+                   float* beta, float* qk, int T, int B, int num_slots, int G, int H, int dim, int dimP, int vdim, int taps,
+                   int update, cudaStream_t stream) {
   if (T <= 0 || B <= 0) return 0;
   if (H % G != 0 || dimP < dim || dimP > 256 || taps < 1 || B > 65535) return -10;
   const DeltaPrep p{ld, ld_a, off_q, off_k, off_v, off_b, B, G, H, dim, dimP, vdim, taps, update};
-  return f32 ? delta_prep<float>(proj, a_pre, conv_q, conv_k, conv_v, A_log, dt_bias, cu, kv_lens, state_slots, conv_state, q,
-                                 k, v, g, beta, qk, T, num_slots, p, stream)
-             : delta_prep<bf16>(proj, a_pre, conv_q, conv_k, conv_v, A_log, dt_bias, cu, kv_lens, state_slots, conv_state, q,
-                                k, v, g, beta, qk, T, num_slots, p, stream);
+  return f32 ? delta_prep<float>(proj, a_pre, conv_t, A_log, dt_bias, cu, kv_lens, state_slots, conv_state, q, k, v, g, beta,
+                                 qk, T, num_slots, p, stream)
+             : delta_prep<bf16>(proj, a_pre, conv_t, A_log, dt_bias, cu, kv_lens, state_slots, conv_state, q, k, v, g, beta, qk,
+                                T, num_slots, p, stream);
 }
 
 int tgi_gated_norm(int f32, const float* o, const void* gate, long long ld, int off, const float* weight, void* out,

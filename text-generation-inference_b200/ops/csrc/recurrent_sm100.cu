@@ -3,16 +3,18 @@
 //   gated delta rule, one decay per key channel      S <- g * S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
 //   linear attention with a fixed decay per head     S <- d S + k v^T;                                    o = S^T q
 //
-// The columns of S never meet: column j of a head needs k, q, g of the head and only v_j of its own.  A column is
-// spread over eight lanes, lane l holding the rows 4 l + 32 j + (0..3), so that state, k, q and g are read as 16-byte
-// pieces and a dot product over the rows is a short register sum followed by three shuffles.
+// The columns of S never meet: column j of a head needs k, q, g of the head and only v_j of its own.
 //
 // scan_kernel walks the tokens a sequence brings in this step with the state in registers (one load and one store of
-// the state per step, whatever the number of tokens).  Tiles of kTile tokens are staged in shared memory one tile
+// the state per step, whatever the number of tokens).  Sixteen lanes share CN columns, lane l holding rows
+// 4 l + 64 j + (0..3) of each: a 16-byte shared-memory read of k (q, g) then feeds 4 CN multiply-adds, done in pairs
+// (fma.rn.f32x2).  The sums of the CN columns are reduced by halving exchanges, after which every lane owns one
+// column; the lane of a column forms its u and read-out.  Tiles of kTile tokens are staged in shared memory one tile
 // ahead.  For the delta rule the tile also holds g * k and g * q, because
 //   S_new^T q = (g S)^T q + (k . q) u = S^T (g q) + (k . q) u
 // lets both dot products run on the old state: one reduction per token sits on the critical path, not two.
-// step_kernel is the single-token form of decode: no staging, bound by reading and writing the state once.
+// step_kernel is the single-token form of decode: eight lanes per column, no staging, bound by reading and writing the
+// state once.
 //
 // Pools are [slots, H, vdim, dimP] with dimP = dim rounded up to 32; rows dim .. dimP - 1 stay zero.  A sequence whose
 // step starts at position 0 starts from a zero state without reading its slot; slot -1 (padding rows of a captured
@@ -47,6 +49,7 @@ struct ScanArgs {
   float* state;                   // [num_slots, H, vdim, dimP]
   float* out;                     // [T, H, vdim]
   int num_slots, G, H, dim, dimP, vdim;
+  int vec;                        // proj: heads may be read four elements at a time
 };
 
 // sum over the eight lanes of a column group
@@ -56,18 +59,62 @@ __device__ __forceinline__ float sum8(float v) {
   v += __shfl_xor_sync(0xffffffffu, v, 4);
   return v;
 }
-// sums of two values over the eight lanes: even lanes end with the first, odd lanes with the second
-__device__ __forceinline__ float sum8_pair(float a, float b, int lane) {
-  const bool odd = lane & 1;
-  const float keep = odd ? b : a, give = odd ? a : b;
-  float v = keep + __shfl_xor_sync(0xffffffffu, give, 1);
-  v += __shfl_xor_sync(0xffffffffu, v, 2);
-  v += __shfl_xor_sync(0xffffffffu, v, 4);
-  return v;
+
+// two fp32 in a 64-bit register
+using pair = unsigned long long;
+__device__ __forceinline__ pair pk(float x, float y) {
+  pair r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(x), "f"(y));
+  return r;
+}
+__device__ __forceinline__ float pair_sum(pair p) {
+  float x, y;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(p));
+  return x + y;
+}
+__device__ __forceinline__ pair fma2(pair a, pair b, pair c) {
+  pair r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ pair mul2(pair a, pair b) {
+  pair r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
 }
 
+// Sums of CN values over sixteen lanes; lane l ends with the total of value l / (16 / CN).
+template <int CN>
+__device__ __forceinline__ float scatter_sum(float (&v)[CN], int l) {
+  int m = 8;
+#pragma unroll
+  for (int half = CN / 2; half >= 1; half /= 2, m >>= 1) {
+    const bool up = l & m;
+#pragma unroll
+    for (int i = 0; i < half; ++i) {
+      const float give = up ? v[i] : v[i + half], keep = up ? v[i + half] : v[i];
+      v[i] = keep + __shfl_xor_sync(0xffffffffu, give, m);
+    }
+  }
+#pragma unroll
+  for (; m >= 1; m >>= 1) v[0] += __shfl_xor_sync(0xffffffffu, v[0], m);
+  return v[0];
+}
+
+__device__ __forceinline__ float4 raw4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 raw4(const bf16* p) {
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+// columns c .. c + 3 of a head after SiLU, zero past `dim`; `vec`: the four may be read at once
 template <typename T>
-__device__ __forceinline__ float4 load4_silu(const T* p, int c, int dim) {   // columns c .. c + 3 of a head, SiLU, zero past dim
+__device__ __forceinline__ float4 load4_silu(const T* p, int c, int dim, bool vec) {
+  if (vec && c < dim) {
+    const float4 x = raw4(p + c);
+    return make_float4(silu_f(x.x), silu_f(x.y), silu_f(x.z), silu_f(x.w));
+  }
   float v[4];
 #pragma unroll
   for (int i = 0; i < 4; ++i) v[i] = c + i < dim ? silu_f(to_f(p[c + i])) : 0.f;
@@ -75,69 +122,75 @@ __device__ __forceinline__ float4 load4_silu(const T* p, int c, int dim) {   // 
 }
 __device__ __forceinline__ float4 mul4(float4 a, float4 b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); }
 
-template <bool DELTA, int J>
+template <bool DELTA, int J, int CN>
 struct ScanSmem {
-  static constexpr int kRow = 32 * J;
+  static constexpr int kRow = 64 * J;
+  static constexpr int kCols = 8 * CN;                          // columns of a CTA
   static constexpr int kArrays = DELTA ? 4 : 2;                 // k, g, g k, g q   |   k, q
   static constexpr int kVec = kTile * kRow;                     // floats of one array
-  static constexpr int kStage = kArrays * kVec + kTile * 32 + 2 * kTile;   // + v tile, beta, q . k
+  static constexpr int kStage = kArrays * kVec + kTile * kCols + 2 * kTile;   // + v tile, beta, q . k
   static constexpr int kBytes = 2 * kStage * 4;
 };
 
-// grid (ceil(vdim / 32), H, B), 128 threads: 32 columns, two per thread
-template <typename T, bool DELTA, int J>
+// grid (ceil(vdim / (8 CN)), H, B), 128 threads: eight groups of sixteen lanes, CN columns per group
+template <typename T, bool DELTA, int J, int CN>
 __global__ void __launch_bounds__(kThreads)
 scan_kernel(ScanArgs p) {
   tgi::pdl_wait();
   tgi::pdl_trigger();
   extern __shared__ __align__(16) float smem[];
-  using S = ScanSmem<DELTA, J>;
-  constexpr int kQuads = kTile * 8 * J;                         // float4 pieces of one array
-  constexpr int NI = (kQuads + kThreads - 1) / kThreads;
-  const int b = blockIdx.z, h = blockIdx.y, c0 = blockIdx.x * 32;
+  using S = ScanSmem<DELTA, J, CN>;
+  constexpr int NI = J;                                         // float4 pieces per thread of one array: kTile 16 J / 128
+  constexpr int NV = kTile * S::kCols / kThreads;
+  static_assert(kTile * 16 == kThreads, "a tile row is 16 J pieces");
+  const int b = blockIdx.z, h = blockIdx.y, c0 = blockIdx.x * S::kCols;
   const int begin = p.cu[b], n = p.cu[b + 1] - begin;
   if (n <= 0) return;
   const int start = p.kv_lens[b] - n, slot = p.state_slots[b];
   const bool has = slot >= 0 && slot < p.num_slots;
-  const int tid = threadIdx.x, lane = tid & 31, l = lane & 7;
-  const int col = (tid >> 3) * 2;                               // first of this thread's two columns, inside the tile
+  const int tid = threadIdx.x, l = tid & 15;
+  const int col = (tid >> 4) * CN;                              // first column of this group, inside the tile
+  const int mine = l / (16 / CN);                               // the column whose sums this lane ends up with
   const int hg = h / (p.H / p.G);
   float* st0 = p.state + ((static_cast<size_t>(has ? slot : 0) * p.H + h) * p.vdim + c0 + col) * p.dimP + 4 * l;
-  const bool own[2] = {c0 + col < p.vdim, c0 + col + 1 < p.vdim};
+  const bool store_out = l % (16 / CN) == 0 && c0 + col + mine < p.vdim;
 
-  float s[2][J][4];
+  pair s[CN][J][2];
 #pragma unroll
-  for (int c = 0; c < 2; ++c) {
+  for (int c = 0; c < CN; ++c) {
 #pragma unroll
     for (int j = 0; j < J; ++j) {
-      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (has && start > 0 && own[c]) v = *reinterpret_cast<const float4*>(st0 + c * p.dimP + 32 * j);
-      s[c][j][0] = v.x; s[c][j][1] = v.y; s[c][j][2] = v.z; s[c][j][3] = v.w;
+      s[c][j][0] = s[c][j][1] = 0ull;
+      if (has && start > 0 && c0 + col + c < p.vdim && 4 * l + 64 * j < p.dimP) {
+        const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(st0 + c * p.dimP + 64 * j);
+        s[c][j][0] = v.x;
+        s[c][j][1] = v.y;
+      }
     }
   }
 
   float4 rk[NI], rq[NI], rg[DELTA ? NI : 1];
-  float rv[2], rb = 0.f, rd = 0.f;
+  float rv[NV], rb = 0.f, rd = 0.f;
   auto fetch = [&](int t0) {                                    // tokens t0 .. of the sequence into registers
 #pragma unroll
     for (int i = 0; i < NI; ++i) {
-      const int it = tid + i * kThreads, tk = it / (8 * J), c4 = (it % (8 * J)) * 4;
-      const bool ok = it < kQuads && t0 + tk < n;
+      const int it = tid + i * kThreads, tk = it / (16 * J), c4 = (it % (16 * J)) * 4;
+      const bool ok = t0 + tk < n && c4 < p.dimP;
       const size_t t = begin + t0 + tk;
       const float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
       if (DELTA) {
-        rk[i] = ok ? *reinterpret_cast<const float4*>(p.k + (t * p.G + hg) * p.dimP + c4) : z;
-        rq[i] = ok ? *reinterpret_cast<const float4*>(p.q + (t * p.G + hg) * p.dimP + c4) : z;
-        rg[DELTA ? i : 0] = ok ? *reinterpret_cast<const float4*>(p.g + (t * p.H + h) * p.dimP + c4) : z;
+        rk[i] = ok ? raw4(p.k + (t * p.G + hg) * p.dimP + c4) : z;
+        rq[i] = ok ? raw4(p.q + (t * p.G + hg) * p.dimP + c4) : z;
+        rg[DELTA ? i : 0] = ok ? raw4(p.g + (t * p.H + h) * p.dimP + c4) : z;
       } else {
         const T* row = static_cast<const T*>(p.proj) + t * p.ld + h * p.dim;
-        rk[i] = ok ? load4_silu(row + p.off_k, c4, p.dim) : z;
-        rq[i] = ok ? load4_silu(row + p.off_q, c4, p.dim) : z;
+        rk[i] = ok ? load4_silu(row + p.off_k, c4, p.dim, p.vec) : z;
+        rq[i] = ok ? load4_silu(row + p.off_q, c4, p.dim, p.vec) : z;
       }
     }
 #pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      const int it = tid + i * kThreads, tk = it >> 5, c = c0 + (it & 31);
+    for (int i = 0; i < NV; ++i) {
+      const int it = tid + i * kThreads, tk = it / S::kCols, c = c0 + it % S::kCols;
       const bool ok = t0 + tk < n && c < p.vdim;
       const size_t t = begin + t0 + tk;
       if (DELTA) rv[i] = ok ? p.v[(t * p.H + h) * p.vdim + c] : 0.f;
@@ -153,32 +206,31 @@ scan_kernel(ScanArgs p) {
   auto stage = [&](float* d) {
 #pragma unroll
     for (int i = 0; i < NI; ++i) {
-      const int it = tid + i * kThreads;
-      if (it < kQuads) {
-        float4* k4 = reinterpret_cast<float4*>(d) + it;
-        k4[0] = rk[i];
-        if (DELTA) {
-          k4[S::kVec / 4] = rg[DELTA ? i : 0];
-          k4[2 * (S::kVec / 4)] = mul4(rg[DELTA ? i : 0], rk[i]);
-          k4[3 * (S::kVec / 4)] = mul4(rg[DELTA ? i : 0], rq[i]);
-        } else {
-          k4[S::kVec / 4] = rq[i];
-        }
+      float4* k4 = reinterpret_cast<float4*>(d) + tid + i * kThreads;
+      k4[0] = rk[i];
+      if (DELTA) {
+        k4[S::kVec / 4] = rg[DELTA ? i : 0];
+        k4[2 * (S::kVec / 4)] = mul4(rg[DELTA ? i : 0], rk[i]);
+        k4[3 * (S::kVec / 4)] = mul4(rg[DELTA ? i : 0], rq[i]);
+      } else {
+        k4[S::kVec / 4] = rq[i];
       }
     }
     float* v = d + S::kArrays * S::kVec;
-    v[tid] = rv[0];
-    v[tid + kThreads] = rv[1];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) v[tid + i * kThreads] = rv[i];
     if (DELTA && tid < kTile) {
-      v[kTile * 32 + tid] = rb;
-      v[kTile * 33 + tid] = rd;
+      v[kTile * S::kCols + tid] = rb;
+      v[kTile * S::kCols + kTile + tid] = rd;
     }
   };
   const float dec = DELTA ? 0.f : p.decay[h];
+  const pair dec2 = pk(dec, dec);
   fetch(0);
   stage(smem);
   __syncthreads();
-  float* const out0 = p.out + (static_cast<size_t>(begin) * p.H + h) * p.vdim + c0 + col;
+  float* const out0 = p.out + (static_cast<size_t>(begin) * p.H + h) * p.vdim + c0 + col + mine;
+  const size_t out_step = static_cast<size_t>(p.H) * p.vdim;
   for (int t0 = 0, cur = 0; t0 < n; t0 += kTile, cur ^= 1) {
     const bool more = t0 + kTile < n;
     if (more) fetch(t0 + kTile);
@@ -188,65 +240,87 @@ scan_kernel(ScanArgs p) {
 #pragma unroll 1
     for (int i = 0; i < cnt; ++i) {
       const float* kr = d + i * S::kRow + 4 * l;
-      const float2 v = *reinterpret_cast<const float2*>(vt + i * 32 + col);
       float o;
       if (DELTA) {
-        float a[2] = {0.f, 0.f}, w[2] = {0.f, 0.f};
+        pair a2[CN], w2[CN];
+#pragma unroll
+        for (int c = 0; c < CN; ++c) a2[c] = w2[c] = 0ull;
 #pragma unroll
         for (int j = 0; j < J; ++j) {
-          const float4 gk = *reinterpret_cast<const float4*>(kr + 2 * S::kVec + 32 * j);
-          const float4 gq = *reinterpret_cast<const float4*>(kr + 3 * S::kVec + 32 * j);
+          const ulonglong2 gk = *reinterpret_cast<const ulonglong2*>(kr + 2 * S::kVec + 64 * j);
+          const ulonglong2 gq = *reinterpret_cast<const ulonglong2*>(kr + 3 * S::kVec + 64 * j);
 #pragma unroll
-          for (int c = 0; c < 2; ++c) {
-            a[c] = fmaf(s[c][j][0], gk.x, a[c]); w[c] = fmaf(s[c][j][0], gq.x, w[c]);
-            a[c] = fmaf(s[c][j][1], gk.y, a[c]); w[c] = fmaf(s[c][j][1], gq.y, w[c]);
-            a[c] = fmaf(s[c][j][2], gk.z, a[c]); w[c] = fmaf(s[c][j][2], gq.z, w[c]);
-            a[c] = fmaf(s[c][j][3], gk.w, a[c]); w[c] = fmaf(s[c][j][3], gq.w, w[c]);
+          for (int c = 0; c < CN; ++c) a2[c] = fma2(s[c][j][1], gk.y, fma2(s[c][j][0], gk.x, a2[c]));
+#pragma unroll
+          for (int c = 0; c < CN; ++c) w2[c] = fma2(s[c][j][1], gq.y, fma2(s[c][j][0], gq.x, w2[c]));
+        }
+        float a[CN], w[CN];
+#pragma unroll
+        for (int c = 0; c < CN; ++c) {
+          a[c] = pair_sum(a2[c]);
+          w[c] = pair_sum(w2[c]);
+        }
+        const float beta = vt[kTile * S::kCols + i], kq = vt[kTile * S::kCols + kTile + i];
+        const float u = beta * (vt[i * S::kCols + col + mine] - scatter_sum<CN>(a, l));
+        pair u2[CN];
+#pragma unroll
+        for (int c = 0; c < CN; ++c) {
+          const float x = __shfl_sync(0xffffffffu, u, c * (16 / CN), 16);
+          u2[c] = pk(x, x);
+        }
+#pragma unroll
+        for (int j = 0; j < J; ++j) {
+          const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(kr + 64 * j);
+          const ulonglong2 g = *reinterpret_cast<const ulonglong2*>(kr + S::kVec + 64 * j);
+#pragma unroll
+          for (int c = 0; c < CN; ++c) {
+            s[c][j][0] = fma2(k.x, u2[c], mul2(g.x, s[c][j][0]));
+            s[c][j][1] = fma2(k.y, u2[c], mul2(g.y, s[c][j][1]));
           }
         }
-        const float beta = vt[kTile * 32 + i], kq = vt[kTile * 33 + i];
-        a[0] = sum8(a[0]);
-        a[1] = sum8(a[1]);
-        const float u0 = beta * (v.x - a[0]), u1 = beta * (v.y - a[1]);
-#pragma unroll
-        for (int j = 0; j < J; ++j) {
-          const float4 k = *reinterpret_cast<const float4*>(kr + 32 * j);
-          const float4 g = *reinterpret_cast<const float4*>(kr + S::kVec + 32 * j);
-          s[0][j][0] = fmaf(k.x, u0, g.x * s[0][j][0]); s[1][j][0] = fmaf(k.x, u1, g.x * s[1][j][0]);
-          s[0][j][1] = fmaf(k.y, u0, g.y * s[0][j][1]); s[1][j][1] = fmaf(k.y, u1, g.y * s[1][j][1]);
-          s[0][j][2] = fmaf(k.z, u0, g.z * s[0][j][2]); s[1][j][2] = fmaf(k.z, u1, g.z * s[1][j][2]);
-          s[0][j][3] = fmaf(k.w, u0, g.w * s[0][j][3]); s[1][j][3] = fmaf(k.w, u1, g.w * s[1][j][3]);
-        }
-        o = fmaf(kq, (l & 1) ? u1 : u0, sum8_pair(w[0], w[1], lane));
+        o = fmaf(kq, u, scatter_sum<CN>(w, l));
       } else {
-        float w[2] = {0.f, 0.f};
+        pair w2[CN], v2[CN];
+#pragma unroll
+        for (int c = 0; c < CN; c += 4) {
+          const float4 v = *reinterpret_cast<const float4*>(vt + i * S::kCols + col + c);
+          v2[c] = pk(v.x, v.x); v2[c + 1] = pk(v.y, v.y); v2[c + 2] = pk(v.z, v.z); v2[c + 3] = pk(v.w, v.w);
+        }
+#pragma unroll
+        for (int c = 0; c < CN; ++c) w2[c] = 0ull;
 #pragma unroll
         for (int j = 0; j < J; ++j) {
-          const float4 k = *reinterpret_cast<const float4*>(kr + 32 * j);
-          const float4 q = *reinterpret_cast<const float4*>(kr + S::kVec + 32 * j);
+          const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(kr + 64 * j);
+          const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(kr + S::kVec + 64 * j);
 #pragma unroll
-          for (int c = 0; c < 2; ++c) {
-            const float vc = c ? v.y : v.x;
-            s[c][j][0] = fmaf(k.x, vc, dec * s[c][j][0]); w[c] = fmaf(s[c][j][0], q.x, w[c]);
-            s[c][j][1] = fmaf(k.y, vc, dec * s[c][j][1]); w[c] = fmaf(s[c][j][1], q.y, w[c]);
-            s[c][j][2] = fmaf(k.z, vc, dec * s[c][j][2]); w[c] = fmaf(s[c][j][2], q.z, w[c]);
-            s[c][j][3] = fmaf(k.w, vc, dec * s[c][j][3]); w[c] = fmaf(s[c][j][3], q.w, w[c]);
+          for (int c = 0; c < CN; ++c) {
+            s[c][j][0] = fma2(k.x, v2[c], mul2(dec2, s[c][j][0]));
+            s[c][j][1] = fma2(k.y, v2[c], mul2(dec2, s[c][j][1]));
+            w2[c] = fma2(s[c][j][1], q.y, fma2(s[c][j][0], q.x, w2[c]));
           }
         }
-        o = sum8_pair(w[0], w[1], lane);
+        float w[CN];
+#pragma unroll
+        for (int c = 0; c < CN; ++c) w[c] = pair_sum(w2[c]);
+        o = scatter_sum<CN>(w, l);
       }
-      if (l < 2 && own[l]) out0[static_cast<size_t>(t0 + i) * p.H * p.vdim + l] = o;
+      if (store_out) out0[static_cast<size_t>(t0 + i) * out_step] = o;
     }
     if (more) stage(smem + (cur ^ 1) * S::kStage);
     __syncthreads();
   }
   if (has) {
 #pragma unroll
-    for (int c = 0; c < 2; ++c) {
-      if (!own[c]) continue;
+    for (int c = 0; c < CN; ++c) {
 #pragma unroll
-      for (int j = 0; j < J; ++j)
-        *reinterpret_cast<float4*>(st0 + c * p.dimP + 32 * j) = make_float4(s[c][j][0], s[c][j][1], s[c][j][2], s[c][j][3]);
+      for (int j = 0; j < J; ++j) {
+        if (c0 + col + c < p.vdim && 4 * l + 64 * j < p.dimP) {
+          ulonglong2 v;
+          v.x = s[c][j][0];
+          v.y = s[c][j][1];
+          *reinterpret_cast<ulonglong2*>(st0 + c * p.dimP + 64 * j) = v;
+        }
+      }
     }
   }
 }
@@ -263,6 +337,7 @@ step_kernel(ScanArgs p) {
   const int slot = p.state_slots[b];
   const bool has = slot >= 0 && slot < p.num_slots;
   const bool load = has && p.kv_lens[b] > 1;
+  __shared__ __align__(16) float kq_s[DELTA ? 4 : 2 * 32 * J];
   const int lane = threadIdx.x & 31, l = lane & 7;
   const int col = (blockIdx.x * 16 + (threadIdx.x >> 3)) * CN;
   const int hg = h / (p.H / p.G);
@@ -316,6 +391,12 @@ step_kernel(ScanArgs p) {
   } else {
     const T* row = static_cast<const T*>(p.proj) + static_cast<size_t>(t) * p.ld;
     const float dec = p.decay[h];
+    // SiLU of the head's k and q once per block (the state is on its way meanwhile)
+    for (int i = threadIdx.x; i < 16 * J; i += kThreads) {
+      const int c4 = (i % (8 * J)) * 4;
+      *reinterpret_cast<float4*>(kq_s + i * 4) = load4_silu(row + (i < 8 * J ? p.off_k : p.off_q) + h * p.dim, c4, p.dim, p.vec);
+    }
+    __syncthreads();
 #pragma unroll
     for (int c = 0; c < CN; ++c) {
       v[c] = col + c < p.vdim ? silu_f(to_f(row[p.off_v + h * p.vdim + col + c])) : 0.f;
@@ -323,8 +404,8 @@ step_kernel(ScanArgs p) {
     }
 #pragma unroll
     for (int j = 0; j < J; ++j) {
-      k[j] = load4_silu(row + p.off_k + h * p.dim, 4 * l + 32 * j, p.dim);
-      q[j] = load4_silu(row + p.off_q + h * p.dim, 4 * l + 32 * j, p.dim);
+      k[j] = *reinterpret_cast<const float4*>(kq_s + 4 * l + 32 * j);
+      q[j] = *reinterpret_cast<const float4*>(kq_s + 32 * J + 4 * l + 32 * j);
 #pragma unroll
       for (int c = 0; c < CN; ++c) {
         float4& x = s[c][j];
@@ -349,18 +430,30 @@ step_kernel(ScanArgs p) {
   }
 }
 
+template <typename T, bool DELTA, int J, int CN>
+int launch_scan(const ScanArgs& p, int B, cudaStream_t stream) {
+  using S = ScanSmem<DELTA, J, CN>;
+  auto kern = scan_kernel<T, DELTA, J, CN>;
+  if (S::kBytes > 48 * 1024 &&
+      cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, S::kBytes) != cudaSuccess)
+    return -2;
+  tgi::launch(kern, dim3((p.vdim + S::kCols - 1) / S::kCols, p.H, B), dim3(kThreads), S::kBytes, stream, p);
+  return cudaGetLastError() == cudaSuccess ? 0 : -3;
+}
+
 template <typename T, bool DELTA, int J>
 int run(const ScanArgs& p, int B, int max_q, cudaStream_t stream) {
   if (max_q == 1) {
     constexpr int CN = J <= 4 ? 4 : 2;
     tgi::launch(step_kernel<T, DELTA, J, CN>, dim3((p.vdim + 16 * CN - 1) / (16 * CN), p.H, B), dim3(kThreads), 0, stream, p);
   } else {
-    using S = ScanSmem<DELTA, J>;
-    auto kern = scan_kernel<T, DELTA, J>;
-    if (S::kBytes > 48 * 1024 &&
-        cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, S::kBytes) != cudaSuccess)
-      return -2;
-    tgi::launch(kern, dim3((p.vdim + 31) / 32, p.H, B), dim3(kThreads), S::kBytes, stream, p);
+    // eight columns per sixteen lanes use shared memory best; four keep more schedulers busy when there are few columns
+    constexpr int JS = (J + 1) / 2;
+    const long long wide = static_cast<long long>(B) * p.H * ((p.vdim + 63) / 64);
+    if constexpr (JS <= 2) {
+      if (wide >= 200) return launch_scan<T, DELTA, JS, 8>(p, B, stream);
+    }
+    return launch_scan<T, DELTA, JS, 4>(p, B, stream);
   }
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
@@ -410,6 +503,8 @@ int tgi_decay_scan(int f32, const void* proj, long long ld, int off_q, int off_k
   p.cu = cu; p.kv_lens = kv_lens; p.state_slots = state_slots;
   p.state = state; p.out = out;
   p.num_slots = num_slots; p.G = H; p.H = H; p.dim = dim; p.dimP = dimP; p.vdim = vdim;
+  p.vec = dim % 4 == 0 && ld % 4 == 0 && off_q % 4 == 0 && off_k % 4 == 0 &&
+          reinterpret_cast<uintptr_t>(proj) % (f32 ? 16 : 8) == 0;
   return f32 ? dispatch<float, false>(p, B, max_q, stream) : dispatch<bf16, false>(p, B, max_q, stream);
 }
 

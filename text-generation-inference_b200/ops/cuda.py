@@ -65,7 +65,7 @@ def load():
                  "tgi_moe_combine", "tgi_gemm_last_grid", "tgi_penalties", "tgi_gemm_wq", "tgi_wq_dequant", "tgi_qk_norm",
                  "tgi_quant_set_pow2", "tgi_peer_set_quant_pow2", "tgi_gemm_bf16_ld", "tgi_residual_norm", "tgi_embed_residual",
                  "tgi_activation", "tgi_attn_prep", "tgi_attn_any", "tgi_delta_prep", "tgi_delta_scan", "tgi_decay_scan",
-                 "tgi_gated_norm", "tgi_recurrent_pitch"):
+                 "tgi_gated_norm", "tgi_recurrent_pitch", "tgi_delta_tap_rows"):
         if hasattr(_LIB, name):        # a library built for one family of models lacks the other families' kernels
             getattr(_LIB, name).restype = c_int
     _LIB.tgi_gemm_workspace_floats.restype = c_ll
@@ -510,7 +510,7 @@ def rotate_norm_store(proj, offs, positions, cos_sin, slots, k_cache, v_cache, n
     _check(load().tgi_attn_prep(
         _f32(proj), _ptr(proj), c_ll(proj.stride(0)), c_int(offs[1]), c_int(offs[2]), _ptr(positions), _ptr(cos_sin),
         _ptr(slots), _ptr(v_first), c_ll(0 if v_first is None else v_first.stride(0)), c_float(v_lambda), _ptr(q),
-        _ptr(k_cache), _ptr(v_cache), c_void_p(0), c_int(T), c_int(num_heads), c_int(num_kv_heads), c_int(dim), c_int(vdim),
+        _ptr(k_cache), _ptr(v_cache), c_int(T), c_int(num_heads), c_int(num_kv_heads), c_int(dim), c_int(vdim),
         c_int(Dk), c_int(Dv), c_int(rot_dim), c_int(cos_sin.shape[0]), c_ll(k_cache.shape[0] * k_cache.shape[1]),
         c_int(1 if qk_norm else 0), c_float(eps), _stream()), "attn_prep")
     return q
@@ -523,17 +523,22 @@ def recurrent_pitch(dim: int) -> int:
     return w
 
 
-def delta_inputs(proj, offs, a_pre, conv_q, conv_k, conv_v, a_log, dt_bias, cu, kv_lens, state_slots, conv_state, kv_heads,
-                 heads, dim, pitch, vdim, single: bool):
+def conv_rows(taps: int) -> int:
+    return int(load().tgi_delta_tap_rows(c_int(taps)))
+
+
+def delta_inputs(proj, offs, a_pre, conv_t, a_log, dt_bias, cu, kv_lens, state_slots, conv_state, kv_heads, heads, dim,
+                 pitch, vdim, single: bool):
     T, dev = proj.shape[0], proj.device
     new = lambda *shape: torch.empty(*shape, dtype=torch.float32, device=dev)
     q, k, g = new(T, kv_heads, pitch), new(T, kv_heads, pitch), new(T, heads, pitch)
     v, beta, qk = new(T, heads, vdim), new(T, heads), new(T, kv_heads)
-    taps = conv_q.shape[1]
+    taps = conv_state.shape[1] + 1
     assert proj.stride(1) == 1 and a_pre.stride(1) == 1 and conv_state.dtype == proj.dtype
+    assert conv_t.is_contiguous() and tuple(conv_t.shape) == (conv_rows(taps), conv_state.shape[2])
     _check(load().tgi_delta_prep(
         _f32(proj), _ptr(proj), c_ll(proj.stride(0)), c_int(offs[0]), c_int(offs[1]), c_int(offs[2]), c_int(offs[3]),
-        _ptr(a_pre), c_ll(a_pre.stride(0)), _ptr(conv_q), _ptr(conv_k), _ptr(conv_v), _ptr(a_log), _ptr(dt_bias), _ptr(cu),
+        _ptr(a_pre), c_ll(a_pre.stride(0)), _ptr(conv_t), _ptr(a_log), _ptr(dt_bias), _ptr(cu),
         _ptr(kv_lens), _ptr(state_slots), _ptr(conv_state), _ptr(q), _ptr(k), _ptr(v), _ptr(g), _ptr(beta), _ptr(qk),
         c_int(T), c_int(kv_lens.shape[0]), c_int(conv_state.shape[0]), c_int(kv_heads), c_int(heads), c_int(dim),
         c_int(pitch), c_int(vdim), c_int(taps), c_int(1 if single else 0), _stream()), "delta_prep")

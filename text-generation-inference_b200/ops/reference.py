@@ -389,18 +389,18 @@ def _sequences(cu, kv_lens, state_slots):
 
 def _short_conv(x, w, past):
     """``x[n, C]`` after ``past[taps - 1, C]``; returns the convolved, SiLU-ed rows and the new past."""
-    taps = w.shape[1]
+    taps = w.shape[0]
     full = torch.cat([past.float(), x.float()], dim=0)
-    y = sum(full[j:j + x.shape[0]] * w[:, j].float() for j in range(taps))
+    y = sum(full[j:j + x.shape[0]] * w[j].float() for j in range(taps))
     return F.silu(y), full[full.shape[0] - (taps - 1):]
 
 
-def delta_inputs(proj, offs, a_pre, conv_q, conv_k, conv_v, a_log, dt_bias, cu, kv_lens, state_slots, conv_state, kv_heads,
-                 heads, dim, pitch, vdim, single: bool):
-    T, taps = proj.shape[0], conv_q.shape[1]
+def delta_inputs(proj, offs, a_pre, conv_t, a_log, dt_bias, cu, kv_lens, state_slots, conv_state, kv_heads, heads, dim,
+                 pitch, vdim, single: bool):
+    T, taps = proj.shape[0], conv_state.shape[1] + 1
     nq, nv = kv_heads * dim, heads * vdim
     x = torch.cat([proj[:, offs[0]:offs[0] + nq], proj[:, offs[1]:offs[1] + nq], proj[:, offs[2]:offs[2] + nv]], dim=1)
-    w = torch.cat([conv_q, conv_k, conv_v], dim=0)
+    w = conv_t[conv_t.shape[0] - taps:]
     y = torch.zeros(T, 2 * nq + nv)
     for _, s, n, start, slot in _sequences(cu, kv_lens, state_slots):
         past = conv_state[slot] if slot >= 0 and start > 0 else torch.zeros(taps - 1, x.shape[1])
