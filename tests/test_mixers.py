@@ -318,6 +318,41 @@ def test_decay_attention(be, shape):
         assert (state[1] == -2.0).all()
 
 
+@pytest.mark.parametrize("batch", [1, 40, 130])
+@pytest.mark.parametrize("dims", [(64, 64), (128, 96)], ids=str)
+def test_scan_layouts(be, batch, dims):
+    """Few and many sequences in a step take different layouts of the state over lanes: prompts, then more tokens."""
+    from tgi_b200 import ops
+
+    dev, dt = be
+    if dev.type == "cpu" and batch > 1:
+        pytest.skip("one layout on the CPU")
+    d, dv, H, lens = dims[0], dims[1], 2, (13, 6)
+    pitch = ops.recurrent_pitch(d, dev)
+    n = sum(lens)
+    k, q, v = (rnd(i, batch, n, H, w) for i, w in enumerate((d, d, dv)))
+    k, q = O.unit(k), O.unit(q)
+    g, beta = torch.sigmoid(rnd(4, batch, n, H, d) + 2), torch.sigmoid(rnd(5, batch, n, H))
+    decay = torch.tensor([0.7, 0.98])
+    y = torch.cat([x.reshape(batch, n, -1) for x in (q, k, v)], -1).to(dt)
+    s1, s2 = (torch.zeros(batch, H, dv, pitch, device=dev) for _ in range(2))
+    pad = lambda x, value=0.0: torch.nn.functional.pad(x, (0, pitch - d), value=value)
+    a = 0
+    outs = [[], []]
+    for m in lens:
+        st = Step([(a, m, batch - 1 - i) for i in range(batch)], dev)
+        row = lambda x: x[:, a:a + m].reshape(batch * m, *x.shape[2:]).to(dev).contiguous()
+        outs[0].append(ops.delta_scan(row(pad(q)), row(pad(k)), row(v), row(pad(g)), row(beta), row((q * k).sum(-1)), st.cu,
+                                      st.kv, st.slots, s1, d, m).cpu().view(batch, m, H, dv))
+        outs[1].append(ops.decay_scan(row(y), [0, H * d, 2 * H * d], decay.to(dev), st.cu, st.kv, st.slots, s2, H, d, dv,
+                                      m).cpu().view(batch, m, H, dv))
+        a += m
+    for i in {0, batch // 2, batch - 1}:
+        close(torch.cat(outs[0], 1)[i], O.delta_scan(*(x[i].double() for x in (q, k, v, g, beta))), torch.float32)
+        c = [O.silu(t.double()).view(n, H, -1) for t in y[i].split([H * d, H * d, H * dv], -1)]
+        close(torch.cat(outs[1], 1)[i], O.lightning_scan(*c, decay.tolist()), torch.float32)
+
+
 def test_padding_rows(be):
     """Rows of a captured batch without a sequence (length 0, slot -1) leave every pool as it is."""
     from tgi_b200 import ops

@@ -6,13 +6,18 @@
 // The columns of S never meet: column j of a head needs k, q, g of the head and only v_j of its own.
 //
 // scan_kernel walks the tokens a sequence brings in this step with the state in registers (one load and one store of
-// the state per step, whatever the number of tokens).  Sixteen lanes share CN columns, lane l holding rows
-// 4 l + 64 j + (0..3) of each: a 16-byte shared-memory read of k (q, g) then feeds 4 CN multiply-adds, done in pairs
-// (fma.rn.f32x2).  The sums of the CN columns are reduced by halving exchanges, after which every lane owns one
-// column; the lane of a column forms its u and read-out.  Tiles of kTile tokens are staged in shared memory one tile
-// ahead.  For the delta rule the tile also holds g * k and g * q, because
-//   S_new^T q = (g S)^T q + (k . q) u = S^T (g q) + (k . q) u
-// lets both dot products run on the old state: one reduction per token sits on the critical path, not two.
+// the state per step, whatever the number of tokens), four tokens at a time.  With G_i the product of the decays since
+// the start of a block (elementwise over key channels), S the state before it and D_ji the decays after token j up to i:
+//   u_i = beta_i (v_i - S^T (G_i k_i) - sum_{j<i} (k_j . D_ji k_i) u_j)
+//   o_i = S^T (G_i q_i) + sum_{j<=i} (k_j . D_ji q_i) u_j
+//   S  <- G_3 S + sum_j (D_j3 k_j) u_j^T
+// which is the token-by-token rule with all products on the old state: they are independent, one reduction latency is
+// paid per block, and the scalars are shared by all columns.  Only products of decays appear, never quotients, so a
+// channel that forgets within a token loses nothing.  (Fixed decay: u = v, D and G are powers of d.)
+// L lanes share CN columns, lane l holding rows 4 (l + L j) + (0..3) of each: a 16-byte shared-memory read feeds 4 CN
+// multiply-adds, done in pairs (fma.rn.f32x2).  The sums of the CN columns are reduced by halving exchanges, after which
+// every lane owns one column.  The vectors and scalars of the next tile of kTile tokens are prepared from registers
+// while the current one runs.
 // step_kernel is the single-token form of decode: eight lanes per column, no staging, bound by reading and writing the
 // state once.
 //
@@ -83,10 +88,10 @@ __device__ __forceinline__ pair mul2(pair a, pair b) {
   return r;
 }
 
-// Sums of CN values over sixteen lanes; lane l ends with the total of value l / (16 / CN).
-template <int CN>
+// Sums of CN values over L lanes; lane l ends with the total of value l / (L / CN).
+template <int CN, int L>
 __device__ __forceinline__ float scatter_sum(float (&v)[CN], int l) {
-  int m = 8;
+  int m = L / 2;
 #pragma unroll
   for (int half = CN / 2; half >= 1; half /= 2, m >>= 1) {
     const bool up = l & m;
@@ -108,6 +113,24 @@ __device__ __forceinline__ float4 raw4(const bf16* p) {
   const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
   return make_float4(a.x, a.y, b.x, b.y);
 }
+// Two neighbouring elements as they are loaded, kept in the registers of a float2 until they are converted.
+template <typename T>
+struct PairOf;
+template <>
+struct PairOf<float> {
+  using type = float2;
+  static __device__ __forceinline__ float2 hold(float2 v) { return v; }
+  static __device__ __forceinline__ float2 value(float2 v) { return v; }
+};
+template <>
+struct PairOf<bf16> {
+  using type = uint32_t;
+  static __device__ __forceinline__ float2 hold(uint32_t v) { return make_float2(__uint_as_float(v), 0.f); }
+  static __device__ __forceinline__ float2 value(float2 v) {
+    const uint32_t w = __float_as_uint(v.x);
+    return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w));
+  }
+};
 // columns c .. c + 3 of a head after SiLU, zero past `dim`; `vec`: the four may be read at once
 template <typename T>
 __device__ __forceinline__ float4 load4_silu(const T* p, int c, int dim, bool vec) {
@@ -122,203 +145,332 @@ __device__ __forceinline__ float4 load4_silu(const T* p, int c, int dim, bool ve
 }
 __device__ __forceinline__ float4 mul4(float4 a, float4 b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); }
 
-template <bool DELTA, int J, int CN>
-struct ScanSmem {
+constexpr int kBlock = 4;         // tokens whose products with the state are formed together
+
+// L lanes share CN columns of a head whose vectors are 64 J wide
+template <bool DELTA, int J, int L, int CN>
+struct ScanCfg {
   static constexpr int kRow = 64 * J;
-  static constexpr int kCols = 8 * CN;                          // columns of a CTA
-  static constexpr int kArrays = DELTA ? 4 : 2;                 // k, g, g k, g q   |   k, q
-  static constexpr int kVec = kTile * kRow;                     // floats of one array
-  static constexpr int kStage = kArrays * kVec + kTile * kCols + 2 * kTile;   // + v tile, beta, q . k
+  static constexpr int kQuads = 16 * J / L;                     // 16-byte pieces of a column per lane
+  static constexpr int kCols = kThreads / L * CN;               // columns of a CTA
+  static constexpr int kRows = DELTA ? 13 : 8;                  // vectors of a block: q', k^ (x 4 each) | + k' (x 4), decay
+  static constexpr int kQ = 0, kEnd = 4, kK = DELTA ? 8 : 0, kG = DELTA ? 12 : 0;      // first row of each kind
+  static constexpr int kVecs = 2 * kRows * kRow;                // floats: two blocks per tile
+  static constexpr int kOffV = kVecs, kOffBeta = kOffV + kTile * kCols, kOffScal = kOffBeta + kTile,
+                       kOffPart = kOffScal + 32, kStage = kOffPart + 2 * J * 16;
   static constexpr int kBytes = 2 * kStage * 4;
 };
 
-// grid (ceil(vdim / (8 CN)), H, B), 128 threads: eight groups of sixteen lanes, CN columns per group
-template <typename T, bool DELTA, int J, int CN>
+// grid (ceil(vdim / kCols), H, B), 128 threads.  VEC: the heads of proj may be read in aligned pairs.
+template <typename T, bool DELTA, bool VEC, int J, int L, int CN>
 __global__ void __launch_bounds__(kThreads)
 scan_kernel(ScanArgs p) {
   tgi::pdl_wait();
   tgi::pdl_trigger();
   extern __shared__ __align__(16) float smem[];
-  using S = ScanSmem<DELTA, J, CN>;
-  constexpr int NI = J;                                         // float4 pieces per thread of one array: kTile 16 J / 128
+  using S = ScanCfg<DELTA, J, L, CN>;
+  constexpr int kItems = 64 * J;                                // (block, channel pair) items of a tile
+  constexpr int NI = (kItems + kThreads - 1) / kThreads;
   constexpr int NV = kTile * S::kCols / kThreads;
-  static_assert(kTile * 16 == kThreads, "a tile row is 16 J pieces");
+  constexpr int NQ = S::kQuads;
   const int b = blockIdx.z, h = blockIdx.y, c0 = blockIdx.x * S::kCols;
   const int begin = p.cu[b], n = p.cu[b + 1] - begin;
   if (n <= 0) return;
   const int start = p.kv_lens[b] - n, slot = p.state_slots[b];
   const bool has = slot >= 0 && slot < p.num_slots;
-  const int tid = threadIdx.x, l = tid & 15;
-  const int col = (tid >> 4) * CN;                              // first column of this group, inside the tile
-  const int mine = l / (16 / CN);                               // the column whose sums this lane ends up with
+  const int tid = threadIdx.x, l = tid % L;
+  const int col = (tid / L) * CN;                               // first column of this group, inside the tile
+  const int mine = l / (L / CN);                                // the column whose sums this lane ends up with
   const int hg = h / (p.H / p.G);
   float* st0 = p.state + ((static_cast<size_t>(has ? slot : 0) * p.H + h) * p.vdim + c0 + col) * p.dimP + 4 * l;
-  const bool store_out = l % (16 / CN) == 0 && c0 + col + mine < p.vdim;
+  const bool store_out = l % (L / CN) == 0 && c0 + col + mine < p.vdim;
+  const float dec = DELTA ? 1.f : p.decay[h];
 
-  pair s[CN][J][2];
+  pair s[CN][NQ][2];
 #pragma unroll
   for (int c = 0; c < CN; ++c) {
 #pragma unroll
-    for (int j = 0; j < J; ++j) {
+    for (int j = 0; j < NQ; ++j) {
       s[c][j][0] = s[c][j][1] = 0ull;
-      if (has && start > 0 && c0 + col + c < p.vdim && 4 * l + 64 * j < p.dimP) {
-        const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(st0 + c * p.dimP + 64 * j);
+      if (has && start > 0 && c0 + col + c < p.vdim && 4 * (l + L * j) < p.dimP) {
+        const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(st0 + c * p.dimP + 4 * L * j);
         s[c][j][0] = v.x;
         s[c][j][1] = v.y;
       }
     }
   }
 
-  float4 rk[NI], rq[NI], rg[DELTA ? NI : 1];
-  float rv[NV], rb = 0.f, rd = 0.f;
-  auto fetch = [&](int t0) {                                    // tokens t0 .. of the sequence into registers
+  // two channels of the four tokens of a block, as they come from memory; pointers advance by a tile
+  using E2 = typename PairOf<T>::type;
+  float2 rk[NI][kBlock], rq[NI][kBlock], rg[DELTA ? NI : 1][kBlock];
+  T rv[DELTA ? 1 : NV];
+  float rvf[DELTA ? NV : 1], rb = 0.f;
+  const size_t sk = DELTA ? static_cast<size_t>(p.G) * p.dimP : static_cast<size_t>(p.ld);   // token pitch of q and k
+  const size_t sg = static_cast<size_t>(p.H) * p.dimP, sv = static_cast<size_t>(p.H) * p.vdim;
+  const T* const proj = static_cast<const T*>(p.proj);
+  auto fetch = [&](int t0) {
 #pragma unroll
     for (int i = 0; i < NI; ++i) {
-      const int it = tid + i * kThreads, tk = it / (16 * J), c4 = (it % (16 * J)) * 4;
-      const bool ok = t0 + tk < n && c4 < p.dimP;
-      const size_t t = begin + t0 + tk;
-      const float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (DELTA) {
-        rk[i] = ok ? raw4(p.k + (t * p.G + hg) * p.dimP + c4) : z;
-        rq[i] = ok ? raw4(p.q + (t * p.G + hg) * p.dimP + c4) : z;
-        rg[DELTA ? i : 0] = ok ? raw4(p.g + (t * p.H + h) * p.dimP + c4) : z;
-      } else {
-        const T* row = static_cast<const T*>(p.proj) + t * p.ld + h * p.dim;
-        rk[i] = ok ? load4_silu(row + p.off_k, c4, p.dim, p.vec) : z;
-        rq[i] = ok ? load4_silu(row + p.off_q, c4, p.dim, p.vec) : z;
+      const int it = tid + i * kThreads, tb = t0 + it / (32 * J) * kBlock, c2 = (it % (32 * J)) * 2;
+      const bool in = it < kItems && c2 < (DELTA ? p.dimP : p.dim);
+      const size_t tok = begin + tb;
+      const float* fk = p.k + tok * sk + hg * p.dimP + c2;
+      const float* fq = p.q + tok * sk + hg * p.dimP + c2;
+      const float* fg = p.g + tok * sg + h * p.dimP + c2;
+      const T* xk = proj + tok * sk + p.off_k + h * p.dim + c2;
+      const T* xq = proj + tok * sk + p.off_q + h * p.dim + c2;
+#pragma unroll
+      for (int e = 0; e < kBlock; ++e) {
+        const bool ok = in && tb + e < n;
+        if (DELTA) {
+          rk[i][e] = rq[i][e] = make_float2(0.f, 0.f);
+          rg[DELTA ? i : 0][e] = make_float2(1.f, 1.f);
+          if (ok) {
+            rk[i][e] = *reinterpret_cast<const float2*>(fk + e * sk);
+            rq[i][e] = *reinterpret_cast<const float2*>(fq + e * sk);
+            rg[DELTA ? i : 0][e] = *reinterpret_cast<const float2*>(fg + e * sg);
+          }
+        } else if (VEC) {
+          E2 a = E2(), c = E2();
+          if (ok) {
+            a = *reinterpret_cast<const E2*>(xk + e * sk);
+            c = *reinterpret_cast<const E2*>(xq + e * sk);
+          }
+          // kept as loaded: the conversion waits for the data, and belongs to `stage`
+          rk[i][e] = PairOf<T>::hold(a);
+          rq[i][e] = PairOf<T>::hold(c);
+        } else {
+          const bool two = c2 + 1 < p.dim;
+          rk[i][e] = make_float2(ok ? to_f(xk[e * sk]) : 0.f, ok && two ? to_f(xk[e * sk + 1]) : 0.f);
+          rq[i][e] = make_float2(ok ? to_f(xq[e * sk]) : 0.f, ok && two ? to_f(xq[e * sk + 1]) : 0.f);
+        }
       }
     }
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
-      const int it = tid + i * kThreads, tk = it / S::kCols, c = c0 + it % S::kCols;
-      const bool ok = t0 + tk < n && c < p.vdim;
-      const size_t t = begin + t0 + tk;
-      if (DELTA) rv[i] = ok ? p.v[(t * p.H + h) * p.vdim + c] : 0.f;
-      else rv[i] = ok ? silu_f(to_f(static_cast<const T*>(p.proj)[t * p.ld + p.off_v + h * p.vdim + c])) : 0.f;
-    }
-    if (DELTA && tid < kTile) {
-      const bool ok = t0 + tid < n;
-      const size_t t = begin + t0 + tid;
-      rb = ok ? p.beta[t * p.H + h] : 0.f;
-      rd = ok ? p.qk[t * p.G + hg] : 0.f;
-    }
-  };
-  auto stage = [&](float* d) {
-#pragma unroll
-    for (int i = 0; i < NI; ++i) {
-      float4* k4 = reinterpret_cast<float4*>(d) + tid + i * kThreads;
-      k4[0] = rk[i];
+      const int it = tid + i * kThreads, tk = t0 + it / S::kCols, c = c0 + it % S::kCols;
+      const bool ok = tk < n && c < p.vdim;
+      const size_t tok = begin + tk;
       if (DELTA) {
-        k4[S::kVec / 4] = rg[DELTA ? i : 0];
-        k4[2 * (S::kVec / 4)] = mul4(rg[DELTA ? i : 0], rk[i]);
-        k4[3 * (S::kVec / 4)] = mul4(rg[DELTA ? i : 0], rq[i]);
+        rvf[DELTA ? i : 0] = 0.f;
+        if (ok) rvf[DELTA ? i : 0] = p.v[tok * sv + h * p.vdim + c];
       } else {
-        k4[S::kVec / 4] = rq[i];
+        rv[DELTA ? 0 : i] = T(0.f);
+        if (ok) rv[DELTA ? 0 : i] = proj[tok * p.ld + p.off_v + h * p.vdim + c];
       }
     }
-    float* v = d + S::kArrays * S::kVec;
+    if (DELTA && tid < kTile) rb = t0 + tid < n ? p.beta[static_cast<size_t>(begin + t0 + tid) * p.H + h] : 0.f;
+  };
+  // vectors and partial scalar products of the fetched tile (tokens t0 ..) -> shared memory
+  auto stage = [&](float* d, int t0) {
 #pragma unroll
-    for (int i = 0; i < NV; ++i) v[tid + i * kThreads] = rv[i];
-    if (DELTA && tid < kTile) {
-      v[kTile * S::kCols + tid] = rb;
-      v[kTile * S::kCols + kTile + tid] = rd;
+    for (int i = 0; i < NI; ++i) {
+      const int it = tid + i * kThreads, blk = it / (32 * J), c2 = (it % (32 * J)) * 2;
+      if (it >= kItems) continue;                               // warp-uniform
+      float2 k[kBlock], q[kBlock], g[kBlock];
+      const int cnt = min(kBlock, n - t0 - blk * kBlock);       // <= 0: a block past the end, nothing reads it
+#pragma unroll
+      for (int e = 0; e < kBlock; ++e) {
+        k[e] = rk[i][e];
+        q[e] = rq[i][e];
+        if (DELTA) {
+          g[e] = rg[DELTA ? i : 0][e];
+        } else {
+          if (VEC) {
+            k[e] = PairOf<T>::value(k[e]);
+            q[e] = PairOf<T>::value(q[e]);
+          }
+          k[e] = make_float2(silu_f(k[e].x), silu_f(k[e].y));   // SiLU(0) = 0: absent tokens and channels stay 0
+          q[e] = make_float2(silu_f(q[e].x), silu_f(q[e].y));
+          g[e].x = g[e].y = e < cnt ? dec : 1.f;
+        }
+      }
+      float* r = d + blk * S::kRows * S::kRow + c2;
+      auto row = [&](int x, float2 v) { *reinterpret_cast<float2*>(r + x * S::kRow) = v; };
+      auto mul = [](float2 a, float2 b) { return make_float2(a.x * b.x, a.y * b.y); };
+      auto dot = [](float2 a, float2 b) { return a.x * b.x + a.y * b.y; };
+      // decays since the start of the block, and from a token to its end
+      float2 to[kBlock], from[kBlock];
+      to[0] = g[0];
+#pragma unroll
+      for (int e = 1; e < kBlock; ++e) to[e] = mul(to[e - 1], g[e]);
+      from[kBlock - 1] = make_float2(1.f, 1.f);
+#pragma unroll
+      for (int e = kBlock - 2; e >= 0; --e) from[e] = mul(from[e + 1], g[e + 1]);
+#pragma unroll
+      for (int e = 0; e < kBlock; ++e) {
+        row(S::kQ + e, mul(to[e], q[e]));
+        row(S::kEnd + e, mul(from[e], k[e]));
+        if (DELTA) row(S::kK + e, mul(to[e], k[e]));
+      }
+      if (DELTA) row(S::kG, to[kBlock - 1]);
+      // token a's key, decayed to token e, times e's query (10 sums over channels) and e's key (6 sums)
+      float sc[16];
+      int at = 0;
+#pragma unroll
+      for (int a = 0; a < kBlock; ++a) {
+        float2 kd = k[a];
+        sc[at++] = dot(kd, q[a]);
+#pragma unroll
+        for (int e = a + 1; e < kBlock; ++e) {
+          kd = mul(kd, g[e]);
+          sc[at++] = dot(kd, q[e]);
+          sc[10 + a * (7 - a) / 2 + (e - a - 1)] = DELTA ? dot(kd, k[e]) : 0.f;
+        }
+      }
+      // over the warp: lanes 2 x and 2 x + 1 end with sum x
+#pragma unroll
+      for (int half = 8, m = 16; half >= 1; half /= 2, m >>= 1) {
+        const bool up = tid & m;
+#pragma unroll
+        for (int a = 0; a < half; ++a) {
+          const float give = up ? sc[a] : sc[a + half], keep = up ? sc[a + half] : sc[a];
+          sc[a] = keep + __shfl_xor_sync(0xffffffffu, give, m);
+        }
+      }
+      sc[0] += __shfl_xor_sync(0xffffffffu, sc[0], 1);
+      if ((tid & 1) == 0) d[S::kOffPart + (blk * J + c2 / 64) * 16 + (tid & 31) / 2] = sc[0];
+    }
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+      d[S::kOffV + tid + i * kThreads] = DELTA ? rvf[DELTA ? i : 0] : silu_f(to_f(rv[DELTA ? 0 : i]));
+    if (DELTA && tid < kTile) d[S::kOffBeta + tid] = rb;
+  };
+  // the sums of the warps that shared a block
+  auto finish = [&](float* d) {
+    if (tid < 32) {
+      float x = 0.f;
+#pragma unroll
+      for (int j = 0; j < J; ++j) x += d[S::kOffPart + ((tid >> 4) * J + j) * 16 + (tid & 15)];
+      d[S::kOffScal + tid] = x;
     }
   };
-  const float dec = DELTA ? 0.f : p.decay[h];
-  const pair dec2 = pk(dec, dec);
   fetch(0);
-  stage(smem);
+  stage(smem, 0);
+  __syncthreads();
+  finish(smem);
   __syncthreads();
   float* const out0 = p.out + (static_cast<size_t>(begin) * p.H + h) * p.vdim + c0 + col + mine;
-  const size_t out_step = static_cast<size_t>(p.H) * p.vdim;
   for (int t0 = 0, cur = 0; t0 < n; t0 += kTile, cur ^= 1) {
     const bool more = t0 + kTile < n;
     if (more) fetch(t0 + kTile);
     const float* d = smem + cur * S::kStage;
-    const float* vt = d + S::kArrays * S::kVec;
-    const int cnt = min(kTile, n - t0);
 #pragma unroll 1
-    for (int i = 0; i < cnt; ++i) {
-      const float* kr = d + i * S::kRow + 4 * l;
-      float o;
+    for (int blk = 0; blk < 2 && t0 + blk * kBlock < n; ++blk) {
+      const float* r = d + blk * S::kRows * S::kRow + 4 * l;
+      const float* vt = d + S::kOffV + blk * kBlock * S::kCols + col;
+      float w[kBlock], u[kBlock];
+      // products of every token of the block with the state before it
+#pragma unroll
+      for (int e = 0; e < kBlock; ++e) {
+        float a[CN];
+        pair x2[CN];
+        u[e] = vt[e * S::kCols + mine];
+        if (DELTA) {
+#pragma unroll
+          for (int j = 0; j < NQ; ++j) {
+            const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(r + (S::kK + e) * S::kRow + 4 * L * j);
+#pragma unroll
+            for (int c = 0; c < CN; ++c)
+              x2[c] = fma2(s[c][j][1], k.y, j == 0 ? mul2(s[c][j][0], k.x) : fma2(s[c][j][0], k.x, x2[c]));
+          }
+#pragma unroll
+          for (int c = 0; c < CN; ++c) a[c] = pair_sum(x2[c]);
+          u[e] -= scatter_sum<CN, L>(a, l);
+        }
+#pragma unroll
+        for (int j = 0; j < NQ; ++j) {
+          const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(r + (S::kQ + e) * S::kRow + 4 * L * j);
+#pragma unroll
+          for (int c = 0; c < CN; ++c)
+            x2[c] = fma2(s[c][j][1], q.y, j == 0 ? mul2(s[c][j][0], q.x) : fma2(s[c][j][0], q.x, x2[c]));
+        }
+#pragma unroll
+        for (int c = 0; c < CN; ++c) a[c] = pair_sum(x2[c]);
+        w[e] = scatter_sum<CN, L>(a, l);
+      }
+      // what the tokens write, first to last, and what they read of each other
+      const float4* sc = reinterpret_cast<const float4*>(d + S::kOffScal + blk * 16);
+      const float4 s0 = sc[0], s1 = sc[1], s2 = sc[2];          // q: 00 01 02 03 | 11 12 13 22 | 23 33, k: 01 02
       if (DELTA) {
-        pair a2[CN], w2[CN];
+        const float4 s3 = sc[3];                                // k: 03 12 13 23
+        const float4 beta = *reinterpret_cast<const float4*>(d + S::kOffBeta + blk * kBlock);
+        u[0] *= beta.x;
+        u[1] = beta.y * fmaf(-s2.z, u[0], u[1]);
+        u[2] = beta.z * fmaf(-s3.y, u[1], fmaf(-s2.w, u[0], u[2]));
+        u[3] = beta.w * fmaf(-s3.w, u[2], fmaf(-s3.z, u[1], fmaf(-s3.x, u[0], u[3])));
+      }
+      w[0] = fmaf(s0.x, u[0], w[0]);
+      w[1] = fmaf(s0.y, u[0], fmaf(s1.x, u[1], w[1]));
+      w[2] = fmaf(s0.z, u[0], fmaf(s1.y, u[1], fmaf(s1.w, u[2], w[2])));
+      w[3] = fmaf(s0.w, u[0], fmaf(s1.z, u[1], fmaf(s2.x, u[2], fmaf(s2.y, u[3], w[3]))));
+      // the state after the block
+      const int cnt = min(kBlock, n - t0 - blk * kBlock);
+      if (DELTA) {
 #pragma unroll
-        for (int c = 0; c < CN; ++c) a2[c] = w2[c] = 0ull;
+        for (int j = 0; j < NQ; ++j) {
+          const ulonglong2 g = *reinterpret_cast<const ulonglong2*>(r + S::kG * S::kRow + 4 * L * j);
 #pragma unroll
-        for (int j = 0; j < J; ++j) {
-          const ulonglong2 gk = *reinterpret_cast<const ulonglong2*>(kr + 2 * S::kVec + 64 * j);
-          const ulonglong2 gq = *reinterpret_cast<const ulonglong2*>(kr + 3 * S::kVec + 64 * j);
-#pragma unroll
-          for (int c = 0; c < CN; ++c) a2[c] = fma2(s[c][j][1], gk.y, fma2(s[c][j][0], gk.x, a2[c]));
-#pragma unroll
-          for (int c = 0; c < CN; ++c) w2[c] = fma2(s[c][j][1], gq.y, fma2(s[c][j][0], gq.x, w2[c]));
+          for (int c = 0; c < CN; ++c) {
+            s[c][j][0] = mul2(g.x, s[c][j][0]);
+            s[c][j][1] = mul2(g.y, s[c][j][1]);
+          }
         }
-        float a[CN], w[CN];
+      } else {
+        const float d2 = dec * dec;
+        const float f = cnt == 4 ? d2 * d2 : (cnt == 3 ? d2 * dec : (cnt == 2 ? d2 : dec));
+        const pair f2 = pk(f, f);
 #pragma unroll
-        for (int c = 0; c < CN; ++c) {
-          a[c] = pair_sum(a2[c]);
-          w[c] = pair_sum(w2[c]);
+        for (int j = 0; j < NQ; ++j) {
+#pragma unroll
+          for (int c = 0; c < CN; ++c) {
+            s[c][j][0] = mul2(f2, s[c][j][0]);
+            s[c][j][1] = mul2(f2, s[c][j][1]);
+          }
         }
-        const float beta = vt[kTile * S::kCols + i], kq = vt[kTile * S::kCols + kTile + i];
-        const float u = beta * (vt[i * S::kCols + col + mine] - scatter_sum<CN>(a, l));
+      }
+#pragma unroll
+      for (int e = 0; e < kBlock; ++e) {
         pair u2[CN];
 #pragma unroll
         for (int c = 0; c < CN; ++c) {
-          const float x = __shfl_sync(0xffffffffu, u, c * (16 / CN), 16);
+          const float x = DELTA ? __shfl_sync(0xffffffffu, u[e], c * (L / CN), L) : vt[e * S::kCols + c];
           u2[c] = pk(x, x);
         }
 #pragma unroll
-        for (int j = 0; j < J; ++j) {
-          const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(kr + 64 * j);
-          const ulonglong2 g = *reinterpret_cast<const ulonglong2*>(kr + S::kVec + 64 * j);
+        for (int j = 0; j < NQ; ++j) {
+          const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(r + (S::kEnd + e) * S::kRow + 4 * L * j);
 #pragma unroll
           for (int c = 0; c < CN; ++c) {
-            s[c][j][0] = fma2(k.x, u2[c], mul2(g.x, s[c][j][0]));
-            s[c][j][1] = fma2(k.y, u2[c], mul2(g.y, s[c][j][1]));
+            s[c][j][0] = fma2(k.x, u2[c], s[c][j][0]);
+            s[c][j][1] = fma2(k.y, u2[c], s[c][j][1]);
           }
         }
-        o = fmaf(kq, u, scatter_sum<CN>(w, l));
-      } else {
-        pair w2[CN], v2[CN];
-#pragma unroll
-        for (int c = 0; c < CN; c += 4) {
-          const float4 v = *reinterpret_cast<const float4*>(vt + i * S::kCols + col + c);
-          v2[c] = pk(v.x, v.x); v2[c + 1] = pk(v.y, v.y); v2[c + 2] = pk(v.z, v.z); v2[c + 3] = pk(v.w, v.w);
-        }
-#pragma unroll
-        for (int c = 0; c < CN; ++c) w2[c] = 0ull;
-#pragma unroll
-        for (int j = 0; j < J; ++j) {
-          const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(kr + 64 * j);
-          const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(kr + S::kVec + 64 * j);
-#pragma unroll
-          for (int c = 0; c < CN; ++c) {
-            s[c][j][0] = fma2(k.x, v2[c], mul2(dec2, s[c][j][0]));
-            s[c][j][1] = fma2(k.y, v2[c], mul2(dec2, s[c][j][1]));
-            w2[c] = fma2(s[c][j][1], q.y, fma2(s[c][j][0], q.x, w2[c]));
-          }
-        }
-        float w[CN];
-#pragma unroll
-        for (int c = 0; c < CN; ++c) w[c] = pair_sum(w2[c]);
-        o = scatter_sum<CN>(w, l);
       }
-      if (store_out) out0[static_cast<size_t>(t0 + i) * out_step] = o;
+      if (store_out) {
+        float* o = out0 + (t0 + blk * kBlock) * sv;
+#pragma unroll
+        for (int e = 0; e < kBlock; ++e)
+          if (e < cnt) o[e * sv] = w[e];
+      }
     }
-    if (more) stage(smem + (cur ^ 1) * S::kStage);
+    if (more) {
+      stage(smem + (cur ^ 1) * S::kStage, t0 + kTile);
+      __syncthreads();
+      finish(smem + (cur ^ 1) * S::kStage);
+    }
     __syncthreads();
   }
   if (has) {
 #pragma unroll
     for (int c = 0; c < CN; ++c) {
 #pragma unroll
-      for (int j = 0; j < J; ++j) {
-        if (c0 + col + c < p.vdim && 4 * l + 64 * j < p.dimP) {
+      for (int j = 0; j < NQ; ++j) {
+        if (c0 + col + c < p.vdim && 4 * (l + L * j) < p.dimP) {
           ulonglong2 v;
           v.x = s[c][j][0];
           v.y = s[c][j][1];
-          *reinterpret_cast<ulonglong2*>(st0 + c * p.dimP + 64 * j) = v;
+          *reinterpret_cast<ulonglong2*>(st0 + c * p.dimP + 4 * L * j) = v;
         }
       }
     }
@@ -430,10 +582,10 @@ step_kernel(ScanArgs p) {
   }
 }
 
-template <typename T, bool DELTA, int J, int CN>
+template <typename T, bool DELTA, bool VEC, int J, int L, int CN>
 int launch_scan(const ScanArgs& p, int B, cudaStream_t stream) {
-  using S = ScanSmem<DELTA, J, CN>;
-  auto kern = scan_kernel<T, DELTA, J, CN>;
+  using S = ScanCfg<DELTA, J, L, CN>;
+  auto kern = scan_kernel<T, DELTA, VEC, J, L, CN>;
   if (S::kBytes > 48 * 1024 &&
       cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, S::kBytes) != cudaSuccess)
     return -2;
@@ -447,13 +599,20 @@ int run(const ScanArgs& p, int B, int max_q, cudaStream_t stream) {
     constexpr int CN = J <= 4 ? 4 : 2;
     tgi::launch(step_kernel<T, DELTA, J, CN>, dim3((p.vdim + 16 * CN - 1) / (16 * CN), p.H, B), dim3(kThreads), 0, stream, p);
   } else {
-    // eight columns per sixteen lanes use shared memory best; four keep more schedulers busy when there are few columns
+    // Wide lanes and few columns keep every scheduler busy when there are few sequences; many columns per lane need
+    // fewer shared-memory reads and shuffles per column.  Measured, 32 heads of 128 x 128, delta rule, us (16 lanes x 4
+    // columns, 16 x 8, 4 x 4): 1 sequence of 8192 tokens 1973, 2593, 3816; 2 x 4096 1399, 1300, 1913; 4 x 2048 1235,
+    // 1045, 962; 16 x 512 1041, 845, 813.  Fixed decay: 2418, 3006, 4141; 1498, 1508, 2076; 1146, 990, 1043; 984, 771, 752.
     constexpr int JS = (J + 1) / 2;
-    const long long wide = static_cast<long long>(B) * p.H * ((p.vdim + 63) / 64);
-    if constexpr (JS <= 2) {
-      if (wide >= 200) return launch_scan<T, DELTA, JS, 8>(p, B, stream);
+    if (DELTA || p.vec) {
+      if constexpr (JS <= 2) {
+        const long long heads = static_cast<long long>(B) * p.H;
+        if (heads * ((p.vdim + 127) / 128) >= (DELTA ? 128 : 192)) return launch_scan<T, DELTA, true, JS, 4, 4>(p, B, stream);
+        if (heads * ((p.vdim + 63) / 64) >= 128) return launch_scan<T, DELTA, true, JS, 16, 8>(p, B, stream);
+      }
+      return launch_scan<T, DELTA, true, JS, 16, 4>(p, B, stream);
     }
-    return launch_scan<T, DELTA, JS, 4>(p, B, stream);
+    if constexpr (!DELTA) return launch_scan<T, DELTA, false, JS, 16, 4>(p, B, stream);
   }
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
