@@ -149,7 +149,7 @@ class GatedDelta(Mixer):
         self.conv = ops.conv_weights(parts, self.device)
         self.a_rank, self.g_rank = (_up(self.weights.get_shape(f"{prefix}.{n}")[0]) for n in ("a1", "g1"))
         # K padded like the rows of a1 / g1: their outputs are read where the fused product left them
-        self.a2, self.g2 = (FastLinear(pad_columns(self.tensor(n))) for n in ("a2", "g2"))
+        self.a2, self.g2 = (pad_columns(self.tensor(n)) for n in ("a2", "g2"))
         self.a_log, self.dt_bias, self.norm = self.f32("A_log"), self.f32("dt_bias"), self.f32("norm")
         self.pitch = ops.recurrent_pitch(s.dim, self.device)
         self.o = self.row(_column_input(self.tensor("o")))
@@ -165,8 +165,8 @@ class GatedDelta(Mixer):
         s = self.spec
         conv_state, state = kv
         p = self.proj(x)
-        a = self.a2(p[:, self.offs[4]:self.offs[4] + self.a_rank])
-        g = self.g2(p[:, self.offs[5]:self.offs[5] + self.g_rank])
+        a = ops.linear_shallow(p[:, self.offs[4]:self.offs[4] + self.a_rank], self.a2)
+        g = ops.linear_shallow(p[:, self.offs[5]:self.offs[5] + self.g_rank], self.g2)
         q, k, v, decay, beta, qk = ops.delta_inputs(
             p, self.offs, a, self.conv, self.a_log, self.dt_bias, meta.cu_seqlens_q, meta.kv_lens, meta.state_slots,
             conv_state, s.kv_heads, s.heads, s.dim, self.pitch, s.vdim, meta.max_q == 1)

@@ -188,6 +188,14 @@ def linear(x, weight, bias=None, out=None):
     return _into(out, ref.linear(x, weight, bias))
 
 
+def linear_shallow(x, weight):
+    """Product over a short inner dimension (low-rank projections).  The persistent GEMM is built for deep K and its
+    epilogue dominates here: 8192 x 4096 x 128 takes 77 us, the library's 19 us; few rows stay on the persistent one."""
+    if use_native(x) and x.dtype == torch.bfloat16 and x.shape[0] >= 512 and weight.shape[1] <= 512:
+        return torch.nn.functional.linear(x, weight)
+    return linear(x, weight)
+
+
 def fp8_quant_act(x, group=128):
     if use_native(x):
         return native().fp8_quant_act(x, group)

@@ -244,7 +244,7 @@ def kernel_rows(dev, width: int, chunk: int, prefill, decode) -> list:
         wl = rn(qw, width)
         kt(f"{tag}: [llama] GEMM q k v", lambda: ops.linear(xw, wl), (T + qw) * width * 2 + T * qw * 2, 2.0 * T * qw * width)
         w3 = rn(H * d, 128)
-        kt(f"{tag}: GEMM a2 (rank 128)", lambda: ops.linear(x[:, C + (H + 7) // 8 * 8:][:, :128], w3),
+        kt(f"{tag}: GEMM a2 (rank 128)", lambda: ops.linear_shallow(x[:, C + (H + 7) // 8 * 8:][:, :128], w3),
            (T + H * d) * 256 + T * H * d * 2, 2.0 * T * H * d * 128)
         assert K.check_status(dev) == 0
         torch.cuda.empty_cache()

@@ -58,6 +58,15 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
 }
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
+// the same for values that came from, or end in, bf16: the hardware exponential and reciprocal (a few ulp of fp32)
+template <typename T>
+__device__ __forceinline__ float sigmoid_t(float x) { return sigmoid_f(x); }
+template <>
+__device__ __forceinline__ float sigmoid_t<bf16>(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
+template <typename T>
+__device__ __forceinline__ float silu_t(float x) { return x * sigmoid_t<T>(x); }
+template <>
+__device__ __forceinline__ float silu_t<float>(float x) { return silu_f(x); }
 
 // sequence that owns token t (cu[0] = 0 .. cu[B] = T)
 __device__ __forceinline__ int sequence_of(const int* __restrict__ cu, int B, int t) {
@@ -519,49 +528,53 @@ delta_prep_kernel(const T* __restrict__ proj, const T* __restrict__ a_pre, const
     beta_out[static_cast<size_t>(t) * p.H + h] = sigmoid_f(to_f(proj[static_cast<size_t>(t) * p.ld + p.off_b + h]));
 }
 
-// The same for up to TAPS <= 8 taps, with one warp per (run of `run` consecutive rows, unit): convolution weights and
-// the window of previous inputs stay in registers while the warp walks the rows, four channels per lane and piece
-// (E pieces of 128 channels).  Weights come as [TAPS][C] with absent taps zero, so the window is always TAPS - 1 long.
-// Units as above; the convolved values of q and k go through one window each.
+// The same for up to TAPS <= 8 taps, with one warp per (run of `run` consecutive rows, unit): the convolution weights
+// stay in registers while the warp walks the rows, four channels per lane and piece (E pieces of 128 channels).  A row
+// reads its TAPS - 1 predecessors again (they are in L1), so that the rows of a run are independent loads.  Weights come
+// as [TAPS][C] with absent taps zero.  Units as above.
 template <typename T, int TAPS>
-struct ConvWindow {
-  float4 w[TAPS], x[TAPS - 1];       // weights; previous inputs, oldest first
-  __device__ __forceinline__ void weights(const float* __restrict__ wt, int C, int c, int lim) {
+struct ShortConv {
+  float4 w[TAPS];
+  __device__ __forceinline__ void weights(const float* __restrict__ wt, int C, int c, bool ok) {
 #pragma unroll
     for (int j = 0; j < TAPS; ++j)
-      w[j] = c < lim ? *reinterpret_cast<const float4*>(wt + static_cast<size_t>(j) * C + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      w[j] = ok ? *reinterpret_cast<const float4*>(wt + static_cast<size_t>(j) * C + c) : make_float4(0.f, 0.f, 0.f, 0.f);
   }
-  // inputs before the row t (local index i of its sequence): rows of this step, then the state, then zeros
-  __device__ __forceinline__ void start(const T* __restrict__ col, long long ld, int t, int i, const T* __restrict__ st, int C,
-                                        int taps, bool ok) {
+  // inputs of the token at `row` (local index i of its sequence), oldest first: rows of this step, before them the
+  // state (`st`, null: zeros)
+  __device__ __forceinline__ void inputs(float4 (&x)[TAPS], const T* __restrict__ row, long long ld, int i,
+                                         const T* __restrict__ st, int C, int taps, bool ok) const {
+    const float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i >= TAPS - 1) {               // warp-uniform
 #pragma unroll
-    for (int j = 0; j < TAPS - 1; ++j) {
-      const int back = TAPS - 1 - j;
-      x[j] = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (!ok) continue;
-      if (i >= back) x[j] = load4(col + static_cast<long long>(t - back) * ld);
-      else if (st != nullptr && taps - 1 + i - back >= 0) x[j] = load4(st + static_cast<size_t>(taps - 1 + i - back) * C);
+      for (int j = 0; j < TAPS; ++j) x[j] = ok ? load4(row - (TAPS - 1 - j) * ld) : z;
+    } else {
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) {
+        const int back = TAPS - 1 - j;
+        x[j] = z;
+        if (!ok) continue;
+        if (i >= back) x[j] = load4(row - back * ld);
+        else if (st != nullptr && taps - 1 + i - back >= 0) x[j] = load4(st + static_cast<size_t>(taps - 1 + i - back) * C);
+      }
     }
   }
-  __device__ __forceinline__ float4 push(float4 v) {
-    float4 a = make_float4(w[TAPS - 1].x * v.x, w[TAPS - 1].y * v.y, w[TAPS - 1].z * v.z, w[TAPS - 1].w * v.w);
+  __device__ __forceinline__ float4 apply(const float4 (&x)[TAPS]) const {
+    float4 a = make_float4(w[0].x * x[0].x, w[0].y * x[0].y, w[0].z * x[0].z, w[0].w * x[0].w);
 #pragma unroll
-    for (int j = 0; j < TAPS - 1; ++j) {
+    for (int j = 1; j < TAPS; ++j) {
       a.x = fmaf(w[j].x, x[j].x, a.x);
       a.y = fmaf(w[j].y, x[j].y, a.y);
       a.z = fmaf(w[j].z, x[j].z, a.z);
       a.w = fmaf(w[j].w, x[j].w, a.w);
     }
-#pragma unroll
-    for (int j = 0; j + 1 < TAPS - 1; ++j) x[j] = x[j + 1];
-    x[TAPS - 2] = v;
-    return make_float4(silu_f(a.x), silu_f(a.y), silu_f(a.z), silu_f(a.w));
+    return make_float4(silu_t<T>(a.x), silu_t<T>(a.y), silu_t<T>(a.z), silu_t<T>(a.w));
   }
-  // after the last push the window holds the new state (single-token steps)
-  __device__ __forceinline__ void save(T* __restrict__ st, int C, int taps, bool ok) const {
+  // the state after this token (single-token steps)
+  static __device__ __forceinline__ void save(const float4 (&x)[TAPS], T* __restrict__ st, int C, int taps, bool ok) {
 #pragma unroll
-    for (int j = 0; j < TAPS - 1; ++j) {
-      const int e = j - (TAPS - taps);
+    for (int j = 1; j < TAPS; ++j) {
+      const int e = j - 1 - (TAPS - taps);
       if (ok && e >= 0) store4(st + static_cast<size_t>(e) * C, x[j]);
     }
   }
@@ -594,6 +607,7 @@ delta_prep_run_kernel(const T* __restrict__ proj, const T* __restrict__ a_pre, c
       if (i >= p.dimP) continue;
       const bool in = i < p.dim;
       const float4 bias = in ? *reinterpret_cast<const float4*>(dt_bias + h * p.dim + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
       for (int t = t0; t < t1; ++t) {
         float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
         if (in) {
@@ -612,42 +626,49 @@ delta_prep_run_kernel(const T* __restrict__ proj, const T* __restrict__ a_pre, c
   // channel and column of the head's first element: q (or v), and k
   const int ca = is_v ? 2 * p.G * p.dim + h * p.vdim : h * p.dim, ck = p.G * p.dim + h * p.dim;
   const int cola = (is_v ? p.off_v + h * p.vdim : p.off_q + h * p.dim), colk = p.off_k + h * p.dim;
-  ConvWindow<T, TAPS> wa[E], wk[E];
+  ShortConv<T, TAPS> wa[E], wk[E];
 #pragma unroll
   for (int e = 0; e < E; ++e) {
     const int i = 4 * lane + 128 * e;
-    wa[e].weights(conv_t, C, ca + i, ca + width);
-    if (!is_v) wk[e].weights(conv_t, C, ck + i, ck + width);
+    wa[e].weights(conv_t, C, ca + i, i < width);
+    if (!is_v) wk[e].weights(conv_t, C, ck + i, i < width);
   }
-  int b = sequence_of(cu, p.B, t0), next = t0;     // `next`: the row where a window has to be set up
+  int b = sequence_of(cu, p.B, t0), end = cu[b + 1];
   T* st = nullptr;
+  const T* old = nullptr;
+  auto enter = [&]() {                             // sequence b: its state, and whether it has a past
+    const int n = end - cu[b], slot = state_slots[b];
+    st = slot >= 0 && slot < num_slots ? conv_state + static_cast<size_t>(slot) * (p.taps - 1) * C : nullptr;
+    old = kv_lens[b] - n > 0 ? st : nullptr;
+  };
+  enter();
   for (int t = t0; t < t1; ++t) {
-    if (t == next) {
+    if (t >= end) {
       while (cu[b + 1] <= t) ++b;                  // sequences without tokens in this step are skipped
-      next = cu[b + 1];
-      const int n = next - cu[b], slot = state_slots[b];
-      st = slot >= 0 && slot < num_slots ? conv_state + static_cast<size_t>(slot) * (p.taps - 1) * C : nullptr;
-      const T* old = kv_lens[b] - n > 0 ? st : nullptr;
-#pragma unroll
-      for (int e = 0; e < E; ++e) {
-        const int i = 4 * lane + 128 * e;
-        wa[e].start(proj + cola + i, p.ld, t, t - cu[b], old != nullptr ? old + ca + i : nullptr, C, p.taps, i < width);
-        if (!is_v) wk[e].start(proj + colk + i, p.ld, t, t - cu[b], old != nullptr ? old + ck + i : nullptr, C, p.taps, i < width);
-      }
+      end = cu[b + 1];
+      enter();
     }
+    const int local = t - cu[b];
     const T* row = proj + static_cast<size_t>(t) * p.ld;
     float4 a[E], k[E];
     float sq = 0.f, sk = 0.f, dq = 0.f;
 #pragma unroll
     for (int e = 0; e < E; ++e) {
       const int i = 4 * lane + 128 * e;
-      const float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
-      a[e] = wa[e].push(i < width ? load4(row + cola + i) : z);
+      const bool ok = i < width;
+      float4 x[TAPS], y[TAPS];
+      wa[e].inputs(x, row + cola + i, p.ld, local, old != nullptr ? old + ca + i : nullptr, C, p.taps, ok);
+      if (!is_v) wk[e].inputs(y, row + colk + i, p.ld, local, old != nullptr ? old + ck + i : nullptr, C, p.taps, ok);
+      a[e] = wa[e].apply(x);
       if (!is_v) {
-        k[e] = wk[e].push(i < width ? load4(row + colk + i) : z);
+        k[e] = wk[e].apply(y);
         sq += dot4(a[e], a[e]);
         sk += dot4(k[e], k[e]);
         dq += dot4(a[e], k[e]);
+      }
+      if (p.update && st != nullptr) {             // run == 1: this warp alone reads and writes these channels' state
+        wa[e].save(x, st + ca + i, C, p.taps, ok);
+        if (!is_v) wk[e].save(y, st + ck + i, C, p.taps, ok);
       }
     }
     if (is_v) {
@@ -660,7 +681,6 @@ delta_prep_run_kernel(const T* __restrict__ proj, const T* __restrict__ a_pre, c
     } else {
       const float iq = 1.f / (sqrtf(warp_sum(sq) + 1e-6f) * sqrtf(static_cast<float>(p.dim)));
       const float ik = 1.f / sqrtf(warp_sum(sk) + 1e-6f);
-      dq = warp_sum(dq);
 #pragma unroll
       for (int e = 0; e < E; ++e) {
         const int i = 4 * lane + 128 * e;
@@ -669,15 +689,10 @@ delta_prep_run_kernel(const T* __restrict__ proj, const T* __restrict__ a_pre, c
         store4(q_out + o, make_float4(a[e].x * iq, a[e].y * iq, a[e].z * iq, a[e].w * iq));
         store4(k_out + o, make_float4(k[e].x * ik, k[e].y * ik, k[e].z * ik, k[e].w * ik));
       }
-      if (lane == 0) qk_out[static_cast<size_t>(t) * p.G + h] = dq * iq * ik;
-    }
-  }
-  if (p.update && st != nullptr) {                 // run == 1: this warp alone reads and writes these channels' state
-#pragma unroll
-    for (int e = 0; e < E; ++e) {
-      const int i = 4 * lane + 128 * e;
-      wa[e].save(st + ca + i, C, p.taps, i < width);
-      if (!is_v) wk[e].save(st + ck + i, C, p.taps, i < width);
+      if (p.update) {                              // only the single-token scan reads q . k
+        dq = warp_sum(dq);
+        if (lane == 0) qk_out[static_cast<size_t>(t) * p.G + h] = dq * iq * ik;
+      }
     }
   }
 }
@@ -743,8 +758,8 @@ gated_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, long 
       const int i = (first + e * step) * 4;
       if (i < width) {
         const float4 w = load4(weight + i), s = load4(gt + i);
-        store4(dst + i, make_float4(v[e].x * inv * w.x * sigmoid_f(s.x), v[e].y * inv * w.y * sigmoid_f(s.y),
-                                    v[e].z * inv * w.z * sigmoid_f(s.z), v[e].w * inv * w.w * sigmoid_f(s.w)));
+        store4(dst + i, make_float4(v[e].x * inv * w.x * sigmoid_t<T>(s.x), v[e].y * inv * w.y * sigmoid_t<T>(s.y),
+                                    v[e].z * inv * w.z * sigmoid_t<T>(s.z), v[e].w * inv * w.w * sigmoid_t<T>(s.w)));
       }
     }
     if (g == 0)
@@ -764,8 +779,8 @@ gated_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, long 
   if (vec) {
     for (int i = first * 4; i < width; i += step * 4) {
       const float4 v = load4(x + i), w = load4(weight + i), s = load4(gt + i);
-      store4(dst + i, make_float4(v.x * inv * w.x * sigmoid_f(s.x), v.y * inv * w.y * sigmoid_f(s.y),
-                                  v.z * inv * w.z * sigmoid_f(s.z), v.w * inv * w.w * sigmoid_f(s.w)));
+      store4(dst + i, make_float4(v.x * inv * w.x * sigmoid_t<T>(s.x), v.y * inv * w.y * sigmoid_t<T>(s.y),
+                                  v.z * inv * w.z * sigmoid_t<T>(s.z), v.w * inv * w.w * sigmoid_t<T>(s.w)));
     }
   } else {
     for (int i = first; i < width; i += step) put(dst + i, x[i] * inv * weight[i] * sigmoid_f(to_f(gt[i])));

@@ -38,7 +38,11 @@ constexpr int kThreads = 128;
 
 __device__ __forceinline__ float to_f(float x) { return x; }
 __device__ __forceinline__ float to_f(bf16 x) { return __bfloat162float(x); }
-__device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
+// bf16 inputs: the hardware exponential and reciprocal (a few ulp of fp32)
+template <typename T>
+__device__ __forceinline__ float silu_t(float x) { return x / (1.f + expf(-x)); }
+template <>
+__device__ __forceinline__ float silu_t<bf16>(float x) { return __fdividef(x, 1.f + __expf(-x)); }
 
 struct ScanArgs {
   // delta rule: fp32 q, k [T, G, dimP], g [T, H, dimP], v [T, H, vdim], beta [T, H], qk = q . k [T, G]
@@ -136,11 +140,11 @@ template <typename T>
 __device__ __forceinline__ float4 load4_silu(const T* p, int c, int dim, bool vec) {
   if (vec && c < dim) {
     const float4 x = raw4(p + c);
-    return make_float4(silu_f(x.x), silu_f(x.y), silu_f(x.z), silu_f(x.w));
+    return make_float4(silu_t<T>(x.x), silu_t<T>(x.y), silu_t<T>(x.z), silu_t<T>(x.w));
   }
   float v[4];
 #pragma unroll
-  for (int i = 0; i < 4; ++i) v[i] = c + i < dim ? silu_f(to_f(p[c + i])) : 0.f;
+  for (int i = 0; i < 4; ++i) v[i] = c + i < dim ? silu_t<T>(to_f(p[c + i])) : 0.f;
   return make_float4(v[0], v[1], v[2], v[3]);
 }
 __device__ __forceinline__ float4 mul4(float4 a, float4 b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); }
@@ -280,8 +284,8 @@ scan_kernel(ScanArgs p) {
             k[e] = PairOf<T>::value(k[e]);
             q[e] = PairOf<T>::value(q[e]);
           }
-          k[e] = make_float2(silu_f(k[e].x), silu_f(k[e].y));   // SiLU(0) = 0: absent tokens and channels stay 0
-          q[e] = make_float2(silu_f(q[e].x), silu_f(q[e].y));
+          k[e] = make_float2(silu_t<T>(k[e].x), silu_t<T>(k[e].y));   // SiLU(0) = 0: absent tokens and channels stay 0
+          q[e] = make_float2(silu_t<T>(q[e].x), silu_t<T>(q[e].y));
           g[e].x = g[e].y = e < cnt ? dec : 1.f;
         }
       }
@@ -333,7 +337,7 @@ scan_kernel(ScanArgs p) {
     }
 #pragma unroll
     for (int i = 0; i < NV; ++i)
-      d[S::kOffV + tid + i * kThreads] = DELTA ? rvf[DELTA ? i : 0] : silu_f(to_f(rv[DELTA ? 0 : i]));
+      d[S::kOffV + tid + i * kThreads] = DELTA ? rvf[DELTA ? i : 0] : silu_t<T>(to_f(rv[DELTA ? 0 : i]));
     if (DELTA && tid < kTile) d[S::kOffBeta + tid] = rb;
   };
   // the sums of the warps that shared a block
@@ -551,7 +555,7 @@ step_kernel(ScanArgs p) {
     __syncthreads();
 #pragma unroll
     for (int c = 0; c < CN; ++c) {
-      v[c] = col + c < p.vdim ? silu_f(to_f(row[p.off_v + h * p.vdim + col + c])) : 0.f;
+      v[c] = col + c < p.vdim ? silu_t<T>(to_f(row[p.off_v + h * p.vdim + col + c])) : 0.f;
       o[c] = 0.f;
     }
 #pragma unroll
