@@ -529,9 +529,10 @@ delta_prep_kernel(const T* __restrict__ proj, const T* __restrict__ a_pre, const
 }
 
 // The same for up to TAPS <= 8 taps, with one warp per (run of `run` consecutive rows, unit): the convolution weights
-// stay in registers while the warp walks the rows, four channels per lane and piece (E pieces of 128 channels).  A row
-// reads its TAPS - 1 predecessors again (they are in L1), so that the rows of a run are independent loads.  Weights come
-// as [TAPS][C] with absent taps zero.  Units as above.
+// stay in registers while the warp walks the rows, four channels per lane and piece (E pieces of 128 channels).  RB rows
+// inside one sequence are loaded together with their TAPS - 1 predecessors (in L1 from the rows before), the first rows
+// of a sequence one by one.  Weights come as [TAPS][C] with absent taps zero.  UNITS: 0 = all units as above, 1 = q and
+// k, 2 = v, 3 = decays (prompts: a kernel each, with the registers it needs).
 template <typename T, int TAPS>
 struct ShortConv {
   float4 w[TAPS];
@@ -559,7 +560,7 @@ struct ShortConv {
       }
     }
   }
-  __device__ __forceinline__ float4 apply(const float4 (&x)[TAPS]) const {
+  __device__ __forceinline__ float4 apply(const float4* x) const {       // x: TAPS inputs, oldest first
     float4 a = make_float4(w[0].x * x[0].x, w[0].y * x[0].y, w[0].z * x[0].z, w[0].w * x[0].w);
 #pragma unroll
     for (int j = 1; j < TAPS; ++j) {
@@ -584,7 +585,7 @@ __device__ __forceinline__ float decay_value(float z, float rate) {
   return expf(-rate * (z > 20.f ? z : log1pf(expf(z))));
 }
 
-template <typename T, int E, int TAPS>
+template <typename T, int E, int TAPS, int UNITS, int RB>
 __global__ void __launch_bounds__(128)
 delta_prep_run_kernel(const T* __restrict__ proj, const T* __restrict__ a_pre, const float* __restrict__ conv_t,
                       const float* __restrict__ A_log, const float* __restrict__ dt_bias, const int* __restrict__ cu,
@@ -595,10 +596,11 @@ delta_prep_run_kernel(const T* __restrict__ proj, const T* __restrict__ a_pre, c
   tgi::pdl_wait();
   tgi::pdl_trigger();
   const int lane = threadIdx.x & 31;
-  const int u = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
-  if (u >= p.G + 2 * p.H) return;
+  const int first = UNITS == 2 ? p.G : (UNITS == 3 ? p.G + p.H : 0);
+  const int u = first + blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (u >= (UNITS == 1 ? p.G : (UNITS == 2 ? p.G + p.H : p.G + 2 * p.H))) return;
   const int t0 = blockIdx.x * run, t1 = min(T_, t0 + run);
-  if (u >= p.G + p.H) {
+  if (UNITS == 3 || (UNITS == 0 && u >= p.G + p.H)) {
     const int h = u - p.G - p.H;
     const float rate = expf(A_log[h]);
 #pragma unroll
@@ -621,7 +623,8 @@ delta_prep_run_kernel(const T* __restrict__ proj, const T* __restrict__ a_pre, c
     return;
   }
   const int C = 2 * p.G * p.dim + p.H * p.vdim;
-  const bool is_v = u >= p.G;
+  if (UNITS == 3) return;
+  const bool is_v = UNITS == 2 || (UNITS == 0 && u >= p.G);
   const int h = is_v ? u - p.G : u, width = is_v ? p.vdim : p.dim;
   // channel and column of the head's first element: q (or v), and k
   const int ca = is_v ? 2 * p.G * p.dim + h * p.vdim : h * p.dim, ck = p.G * p.dim + h * p.dim;
@@ -642,7 +645,40 @@ delta_prep_run_kernel(const T* __restrict__ proj, const T* __restrict__ a_pre, c
     old = kv_lens[b] - n > 0 ? st : nullptr;
   };
   enter();
-  for (int t = t0; t < t1; ++t) {
+  auto emit = [&](int t, const float4 (&a)[E], const float4 (&k)[E]) {
+    if (is_v) {
+#pragma unroll
+      for (int e = 0; e < E; ++e) {
+        const int i = 4 * lane + 128 * e;
+        if (i < width) store4(v_out + (static_cast<size_t>(t) * p.H + h) * p.vdim + i, a[e]);
+      }
+      if (lane == 0)
+        beta_out[static_cast<size_t>(t) * p.H + h] = sigmoid_f(to_f(proj[static_cast<size_t>(t) * p.ld + p.off_b + h]));
+      return;
+    }
+    float sq = 0.f, sk = 0.f, dq = 0.f;
+#pragma unroll
+    for (int e = 0; e < E; ++e) {
+      sq += dot4(a[e], a[e]);
+      sk += dot4(k[e], k[e]);
+      dq += dot4(a[e], k[e]);
+    }
+    const float iq = 1.f / (sqrtf(warp_sum(sq) + 1e-6f) * sqrtf(static_cast<float>(p.dim)));
+    const float ik = 1.f / sqrtf(warp_sum(sk) + 1e-6f);
+#pragma unroll
+    for (int e = 0; e < E; ++e) {
+      const int i = 4 * lane + 128 * e;
+      if (i >= p.dimP) continue;
+      const size_t o = (static_cast<size_t>(t) * p.G + h) * p.dimP + i;
+      store4(q_out + o, make_float4(a[e].x * iq, a[e].y * iq, a[e].z * iq, a[e].w * iq));
+      store4(k_out + o, make_float4(k[e].x * ik, k[e].y * ik, k[e].z * ik, k[e].w * ik));
+    }
+    if (p.update) {                                // only the single-token scan reads q . k
+      dq = warp_sum(dq);
+      if (lane == 0) qk_out[static_cast<size_t>(t) * p.G + h] = dq * iq * ik;
+    }
+  };
+  for (int t = t0; t < t1;) {
     if (t >= end) {
       while (cu[b + 1] <= t) ++b;                  // sequences without tokens in this step are skipped
       end = cu[b + 1];
@@ -650,8 +686,32 @@ delta_prep_run_kernel(const T* __restrict__ proj, const T* __restrict__ a_pre, c
     }
     const int local = t - cu[b];
     const T* row = proj + static_cast<size_t>(t) * p.ld;
+    if (RB > 1 && local >= TAPS - 1 && t + RB <= min(t1, end)) {
+      float4 x[E][TAPS - 1 + RB], y[E][TAPS - 1 + RB];
+#pragma unroll
+      for (int e = 0; e < E; ++e) {
+        const int i = 4 * lane + 128 * e;
+        const float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int j = 0; j < TAPS - 1 + RB; ++j) {
+          x[e][j] = i < width ? load4(row + (j - (TAPS - 1)) * p.ld + cola + i) : z;
+          y[e][j] = !is_v && i < width ? load4(row + (j - (TAPS - 1)) * p.ld + colk + i) : z;
+        }
+      }
+#pragma unroll
+      for (int r = 0; r < RB; ++r) {
+        float4 a[E], k[E];
+#pragma unroll
+        for (int e = 0; e < E; ++e) {
+          a[e] = wa[e].apply(&x[e][r]);
+          if (!is_v) k[e] = wk[e].apply(&y[e][r]);
+        }
+        emit(t + r, a, k);
+      }
+      t += RB;
+      continue;
+    }
     float4 a[E], k[E];
-    float sq = 0.f, sk = 0.f, dq = 0.f;
 #pragma unroll
     for (int e = 0; e < E; ++e) {
       const int i = 4 * lane + 128 * e;
@@ -660,40 +720,14 @@ delta_prep_run_kernel(const T* __restrict__ proj, const T* __restrict__ a_pre, c
       wa[e].inputs(x, row + cola + i, p.ld, local, old != nullptr ? old + ca + i : nullptr, C, p.taps, ok);
       if (!is_v) wk[e].inputs(y, row + colk + i, p.ld, local, old != nullptr ? old + ck + i : nullptr, C, p.taps, ok);
       a[e] = wa[e].apply(x);
-      if (!is_v) {
-        k[e] = wk[e].apply(y);
-        sq += dot4(a[e], a[e]);
-        sk += dot4(k[e], k[e]);
-        dq += dot4(a[e], k[e]);
-      }
+      if (!is_v) k[e] = wk[e].apply(y);
       if (p.update && st != nullptr) {             // run == 1: this warp alone reads and writes these channels' state
         wa[e].save(x, st + ca + i, C, p.taps, ok);
         if (!is_v) wk[e].save(y, st + ck + i, C, p.taps, ok);
       }
     }
-    if (is_v) {
-#pragma unroll
-      for (int e = 0; e < E; ++e) {
-        const int i = 4 * lane + 128 * e;
-        if (i < width) store4(v_out + (static_cast<size_t>(t) * p.H + h) * p.vdim + i, a[e]);
-      }
-      if (lane == 0) beta_out[static_cast<size_t>(t) * p.H + h] = sigmoid_f(to_f(row[p.off_b + h]));
-    } else {
-      const float iq = 1.f / (sqrtf(warp_sum(sq) + 1e-6f) * sqrtf(static_cast<float>(p.dim)));
-      const float ik = 1.f / sqrtf(warp_sum(sk) + 1e-6f);
-#pragma unroll
-      for (int e = 0; e < E; ++e) {
-        const int i = 4 * lane + 128 * e;
-        if (i >= p.dimP) continue;
-        const size_t o = (static_cast<size_t>(t) * p.G + h) * p.dimP + i;
-        store4(q_out + o, make_float4(a[e].x * iq, a[e].y * iq, a[e].z * iq, a[e].w * iq));
-        store4(k_out + o, make_float4(k[e].x * ik, k[e].y * ik, k[e].z * ik, k[e].w * ik));
-      }
-      if (p.update) {                              // only the single-token scan reads q . k
-        dq = warp_sum(dq);
-        if (lane == 0) qk_out[static_cast<size_t>(t) * p.G + h] = dq * iq * ik;
-      }
-    }
+    emit(t, a, k);
+    ++t;
   }
 }
 
@@ -847,15 +881,23 @@ int delta_prep(const void* proj, const void* a_pre, const float* conv_t, const f
                    reinterpret_cast<uintptr_t>(proj) % (4 * sizeof(T)) == 0 &&
                    reinterpret_cast<uintptr_t>(a_pre) % (4 * sizeof(T)) == 0;
   if (vec) {
-    const int run = p.update ? 1 : 16;
-    const dim3 grid((T_ + run - 1) / run, (units + 3) / 4);
-    auto go = [&](auto kern) {
-      tgi::launch(kern, grid, dim3(128), 0, stream, x, a, conv_t, A_log, dt_bias, cu, kv, slots, st, q, k, v, g, beta, qk, T_,
-                  num_slots, run, p);
-    };
     const bool one = p.dimP <= 128 && p.vdim <= 128;
-    if (p.taps <= 4) one ? go(delta_prep_run_kernel<T, 1, 4>) : go(delta_prep_run_kernel<T, 2, 4>);
-    else one ? go(delta_prep_run_kernel<T, 1, 8>) : go(delta_prep_run_kernel<T, 2, 8>);
+    auto go = [&](auto kern, int count, int run) {
+      tgi::launch(kern, dim3((T_ + run - 1) / run, (count + 3) / 4), dim3(128), 0, stream, x, a, conv_t, A_log, dt_bias, cu, kv,
+                  slots, st, q, k, v, g, beta, qk, T_, num_slots, run, p);
+    };
+    if (p.update) {
+      if (p.taps <= 4) one ? go(delta_prep_run_kernel<T, 1, 4, 0, 1>, units, 1) : go(delta_prep_run_kernel<T, 2, 4, 0, 1>, units, 1);
+      else one ? go(delta_prep_run_kernel<T, 1, 8, 0, 1>, units, 1) : go(delta_prep_run_kernel<T, 2, 8, 0, 1>, units, 1);
+    } else if (p.taps <= 4 && one) {
+      go(delta_prep_run_kernel<T, 1, 4, 1, 2>, p.G, 16);
+      go(delta_prep_run_kernel<T, 1, 4, 2, 4>, p.H, 32);
+      go(delta_prep_run_kernel<T, 1, 4, 3, 1>, p.H, 16);
+    } else if (p.taps <= 4) {
+      go(delta_prep_run_kernel<T, 2, 4, 0, 1>, units, 16);
+    } else {
+      one ? go(delta_prep_run_kernel<T, 1, 8, 0, 1>, units, 16) : go(delta_prep_run_kernel<T, 2, 8, 0, 1>, units, 16);
+    }
   } else {
     const float* first = conv_t + static_cast<size_t>(delta_tap_rows(p.taps) - p.taps) * C;
     const long long jobs = static_cast<long long>(T_) * units;
