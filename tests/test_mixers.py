@@ -432,6 +432,8 @@ def test_sliced_product(be):
     x = rnd(1, 37, 200).to(dt)
     w = rnd(2, 50, 24).to(dt)
     close(ops.linear(x.to(dev)[:, 104:128], w.to(dev)), x[:, 104:128].double() @ w.double().t(), dt)
+    long = rnd(7, 700, 64).to(dt)        # many rows over a short inner dimension
+    close(ops.linear_shallow(long.to(dev)[:, 32:56], w.to(dev)), long[:, 32:56].double() @ w.double().t(), dt)
     w = rnd(3, 50, 21).to(dt)
     close(ops.linear(x[:, :21].contiguous().to(dev), pad_columns(w.to(dev))), x[:, :21].double() @ w.double().t(), dt)
     m, offs = stack_rows([rnd(4, 5, 200).to(dt).to(dev), rnd(5, 16, 200).to(dt).to(dev), rnd(6, 3, 200).to(dt).to(dev)])

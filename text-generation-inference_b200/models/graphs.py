@@ -13,6 +13,7 @@ the state kernels neither read nor write.
 """
 from __future__ import annotations
 
+import gc
 import math
 import os
 from typing import Dict, List, Optional, Tuple
@@ -100,6 +101,16 @@ class DecodeGraphs:
             self.capture(bs)
 
     def capture(self, bs: int, lora: bool = False):
+        # a collection that destroys another runner's graphs in the middle of a capture would invalidate it
+        collecting = gc.isenabled()
+        gc.disable()
+        try:
+            self._capture(bs, lora)
+        finally:
+            if collecting:
+                gc.enable()
+
+    def _capture(self, bs: int, lora: bool):
         r = self.runner
         b = _Bucket(r, bs, self.max_blocks, self.pool)
         if lora:
