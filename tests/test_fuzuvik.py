@@ -49,7 +49,7 @@ def checkpoints(tmp_path_factory):
         if name not in _CKPT:
             cfg = CONFIGS[name]
             sd = {k: v.to(torch.bfloat16) for k, v in syn.fuzuvik_state_dict(cfg, seed=len(name)).items()}
-            _CKPT[name] = (cfg, sd, syn.write_fuzuvik_checkpoint(tmp_path_factory.mktemp(name), cfg, sd), {})
+            _CKPT[name] = (cfg, sd, syn.write_checkpoint(tmp_path_factory.mktemp(name), cfg, sd), {})
         return _CKPT[name]
 
     return get
@@ -423,7 +423,7 @@ def test_served_by_router_and_shard(tmp_path):
     cfg = syn.fuzuvik_config([syn.fuzuvik_attention(chunk=24), syn.fuzuvik_delta(), syn.fuzuvik_lightning(),
                               syn.fuzuvik_attention(chunk=24, ff=0)], width=64, vocab=300)
     sd = syn.fuzuvik_state_dict(cfg, seed=3)
-    path = syn.write_fuzuvik_checkpoint(tmp_path / "m", cfg, sd)
+    path = syn.write_checkpoint(tmp_path / "m", cfg, sd)
     prompts = ["hello world", "a", "the quick brown fox jumps over the lazy dog, twice", "recurrent", "0123456789" * 4]
     n = 4
     want = [O.greedy(cfg, sd, [b + 3 for b in p.encode()], n) for p in prompts]

@@ -41,7 +41,7 @@ def _fuzuvik_config(d: Dict[str, Any]) -> Dict[str, Any]:
                 rot_base=float(rot.get("base") or 10000.0),
                 rot_scaling=None if not sc else (float(sc["factor"]), float(sc["low"]), float(sc["high"]), float(sc["original"]))))
         elif layer["type"] == "channel_delta":
-            specs.append(MixerSpec("delta", **sizes))
+            specs.append(MixerSpec("delta", **sizes, short_conv=True))
         elif layer["type"] == "lightning":
             specs.append(MixerSpec("decay", **sizes, decay=tuple(float(x) for x in m["decay"])))
         else:
@@ -55,8 +55,57 @@ def _fuzuvik_config(d: Dict[str, Any]) -> Dict[str, Any]:
     return out
 
 
+def _layer_order(count: int, loop: Optional[Dict[str, Any]]) -> List[int]:
+    """Layers in the order they run: ``loop`` repeats layers ``start .. stop - 1`` ``times`` times in a row."""
+    if not loop:
+        return list(range(count))
+    lo, hi, times = int(loop["start"]), int(loop["stop"]), int(loop["times"])
+    if not 0 <= lo <= hi <= count or times < 1:
+        raise ValueError(f"a loop over layers {lo} .. {hi - 1}, {times} times, does not fit {count} layers")
+    return list(range(lo)) + list(range(lo, hi)) * times + list(range(hi, count))
+
+
+def _kipedra_config(d: Dict[str, Any]) -> Dict[str, Any]:
+    """Kipedra checkpoints: layers described one by one as in Fuzuvik's, mixer and feed-forward side by side, layers that
+    may run several times."""
+    out = dict(d)
+    layers = d["layers"]
+    specs = []
+    for i, layer in enumerate(layers):
+        m, mlp = layer["mixer"], layer.get("mlp")
+        ff, moe = 0, None
+        if mlp is not None and mlp["kind"] == "dense":
+            ff = int(mlp["ff"])
+        elif mlp is not None and mlp["kind"] == "moe":
+            r = mlp["router"]
+            moe = ExpertSpec(experts=int(r["experts"]), top=int(r["top"]), ff=int(mlp["expert"]["ff"]), scale=float(r["scale"]),
+                             act="relu2")
+        elif mlp is not None:
+            raise NotImplementedError(f"layer {i}: feed-forward kind {mlp['kind']!r}")
+        sizes = dict(heads=int(m["heads"]), kv_heads=int(m.get("kv_heads") or m["heads"]), dim=int(m["dim"]),
+                     vdim=int(m["vdim"]), ff=ff, moe=moe)
+        if layer["type"] == "attention":
+            rot = m.get("rot") or {}
+            specs.append(MixerSpec(
+                "attention", **sizes, scale=float(m["scale"]), window=int((m.get("mask") or {}).get("size") or 0),
+                short_conv=bool(m.get("conv")), qkv_bias=True, rot_dims=int(rot.get("dims") or 0), rot_base=float(rot.get("base") or 10000.0),
+                rot_interleaved=True))
+        elif layer["type"] == "delta":
+            specs.append(MixerSpec("delta", **sizes, short_conv=True, head_decay=True, gate_act="silu"))
+        else:
+            raise NotImplementedError(f"layer {i}: mixer {layer['type']!r}")
+    attn = [s for s in specs if s.kind == "attention"]
+    out.update(model_type="kipedra", hidden_size=int(d["width"]), vocab_size=int(d["vocab"]), num_hidden_layers=len(layers),
+               num_attention_heads=max(s.heads for s in (attn or specs)), rms_norm_eps=float(d["norm"]["eps"]),
+               residual_multiplier=float(d.get("residual_mult", 1.0)), mixers=specs,
+               layer_order=_layer_order(len(layers), d.get("loop")), tie_word_embeddings=True,
+               # rotary positions are unbounded by design: the table length is a deployment choice
+               max_position_embeddings=int(d.get("max_position_embeddings") or 131072))
+    return out
+
+
 # ``architecture`` of a config.json without ``model_type`` -> function that brings it to the common names
-CONFIG_READERS = {"Fuzuvik": _fuzuvik_config}
+CONFIG_READERS = {"Fuzuvik": _fuzuvik_config, "Kipedra": _kipedra_config}
 
 
 class ModelConfig:
@@ -99,17 +148,32 @@ class ModelConfig:
 
 
 @dataclass(frozen=True)
+class ExpertSpec:
+    """Routed feed-forward of one layer: ungated experts (``down(act(up(h)))``) chosen by the sigmoid of their router
+    logits plus a stored correction, weighted by the sigmoids alone, which are brought to the sum ``scale``."""
+
+    experts: int
+    top: int                                 # experts per token
+    ff: int                                  # width of an expert
+    scale: float = 1.0
+    act: str = "relu2"
+
+
+@dataclass(frozen=True)
 class MixerSpec:
-    """Token mixer and feed-forward width of one layer of a decoder whose layers differ (``models/mixers.py``)."""
+    """Token mixer and feed-forward of one layer of a decoder whose layers differ (``models/mixers.py``)."""
 
     kind: str                                # "attention" | "delta" (gated delta rule) | "decay" (fixed decay per head)
     heads: int
     kv_heads: int                            # attention: key/value heads; delta: query/key heads
     dim: int                                 # query / key size of a head
     vdim: int                                # value size of a head
-    ff: int = 0                              # feed-forward width, 0: the layer has none
+    ff: int = 0                              # width of a dense feed-forward, 0: the layer has none
+    moe: Optional[ExpertSpec] = None         # routed experts in its place
+    short_conv: bool = False                 # causal convolution over time on every channel of q, k and v
     # attention
     scale: float = 1.0
+    window: int = 0                          # > 0: the token itself and the window - 1 tokens before it
     chunk: int = 0                           # > 0: keys of the query's own chunk of this many positions
     sink: bool = False                       # one more key of score 0, without a value, in the softmax
     qk_unit_rms: bool = False                # q and k over their root mean square, after the rotation
@@ -117,12 +181,28 @@ class MixerSpec:
     rot_dims: int = 0
     rot_base: float = 10000.0
     rot_scaling: Optional[Tuple[float, float, float, float]] = None    # (factor, low, high, original length)
+    rot_interleaved: bool = False            # pairs 2i, 2i + 1 (False: i, i + rot_dims / 2)
+    qkv_bias: bool = False
+    # delta
+    head_decay: bool = False                 # one decay per head, full-rank decay and gate projections (False: one per
+                                             # head and key channel, low-rank projections)
+    gate_act: str = "sigmoid"                # of the output gate
     # decay
     decay: Tuple[float, ...] = ()
 
     @property
+    def paged(self) -> bool:
+        """Keeps keys and values of every token."""
+        return self.kind == "attention"
+
+    @property
     def recurrent(self) -> bool:
-        return self.kind != "attention"
+        """Keeps a state per sequence that every token advances."""
+        return self.kind != "attention" or self.short_conv
+
+    @property
+    def feed_forward(self) -> bool:
+        return self.ff > 0 or self.moe is not None
 
 
 @dataclass(frozen=True)
@@ -180,6 +260,7 @@ class Arch:
     mla: bool = False                        # DeepSeek multi-head latent attention (models/deepseek.py)
     moe_shared_gate: Optional[str] = None
     moe_renormalize: bool = True
+    moe_correction: Optional[str] = None     # correction of the choice scores (layers with an `ExpertSpec`)
     # ---- layers that differ (config "mixers") ---------------------------------------------------
     mix: Optional[str] = None                # tensor prefix of a layer's mixer
     residual_fp32: bool = False              # the residual stream is kept in 32 bits
@@ -269,6 +350,11 @@ ARCHS["deepseek_v2"] = ARCHS["deepseek_v3"] = replace(
 ARCHS["fuzuvik"] = Arch(embed="embed", layer="l{i}", norm1="norm1", norm2="norm2", final_norm="final.norm", lm_head="head",
                         mix="mix", gate=None, up="mlp.up", down="mlp.down", gated_mlp=False, act="gelu", rope=False,
                         residual_fp32=True, bare_names=True)
+ARCHS["kipedra"] = Arch(embed="embed", layer="l{i}", norm1="norm1", norm2="norm2", final_norm="final.norm", lm_head="head",
+                        mix="mix", gate="mlp.gate", up="mlp.up", down="mlp.down", act="gelu_tanh", rope=False,
+                        norm_unit_offset=True, parallel_residual=True, parallel_shared_norm=False, residual_fp32=True,
+                        bare_names=True, moe_router="mlp.router", moe_expert="mlp.e{e}", moe_up="up", moe_down="down",
+                        moe_correction="mlp.correction")
 ARCHS["gemma3"] = ARCHS["gemma3_text"]
 ARCHS["phi-msft"] = ARCHS["phi"]
 ARCHS["qwen2_vl_text"] = ARCHS["qwen2_5_vl_text"] = ARCHS["qwen2"]   # language models of Qwen2-VL / Qwen2.5-VL
@@ -308,6 +394,7 @@ class ModelDims:
     total_heads: int = 0
     total_kv_heads: int = 0
     mixers: Optional[List[MixerSpec]] = None    # per layer, for decoders whose layers differ
+    layer_order: Optional[List[int]] = None     # layers in the order they run (None: each once)
     attn_head_dim: int = 0      # head dimension seen by the attention kernels and the KV cache: head_dim padded to 64/128/256
 
 
@@ -409,4 +496,5 @@ def derive_dims(cfg: ModelConfig, arch: Arch, world: int) -> ModelDims:
         embed_scale=(math.sqrt(hidden) if arch.embed_scale_sqrt_hidden else float(cfg.get("embedding_multiplier", 1.0) or 1.0)),
         residual_scale=float(cfg.get("residual_multiplier", 1.0) or 1.0),
         num_experts=ne, top_k=tk, total_heads=heads, total_kv_heads=kv, mixers=mixers,
+        layer_order=cfg.get("layer_order"),
     )

@@ -22,7 +22,7 @@ import torch
 
 from .. import ops
 from ..utils.rotary import RotaryTable
-from .arch import Arch, ModelConfig, ModelDims, arch_for, derive_dims
+from .arch import Arch, ExpertSpec, ModelConfig, ModelDims, arch_for, derive_dims
 from .layers import (
     FastLinear,
     Fp8Linear,
@@ -58,25 +58,34 @@ class ForwardMeta:
 
 
 class Norm:
-    def __init__(self, kind: str, weight, bias, eps: float, unit_offset: bool, residual_fp32: bool = False):
+    def __init__(self, kind: str, weight, bias, eps: float, unit_offset: bool, residual_fp32: bool = False,
+                 residual_scale: float = 1.0):
         self.kind, self.weight, self.bias, self.eps, self.unit_offset = kind, weight, bias, eps, unit_offset
         self.residual_fp32 = residual_fp32
+        self.residual_scale = residual_scale     # fp32 streams: what a block's output is multiplied by when it is added
 
     @classmethod
-    def load(cls, arch: Arch, prefix: str, weights, eps: float):
+    def load(cls, arch: Arch, prefix: str, weights, eps: float, residual_scale: float = 1.0):
         w = weights.get_tensor(f"{prefix}.weight")
         b = None
         if arch.norm == "layer" and arch.norm_bias and weights.has_tensor(f"{prefix}.bias"):
             b = weights.get_tensor(f"{prefix}.bias")
-        return cls(arch.norm, w, b, eps, arch.norm_unit_offset, arch.residual_fp32)
+        return cls(arch.norm, w, b, eps, arch.norm_unit_offset, arch.residual_fp32, residual_scale)
 
     def __call__(self, x, residual=None, rows=None):
         if self.residual_fp32:
-            # `x` is the last block's output (None: nothing to add), `rows` ends the stream: only these rows are normed
-            return ops.residual_norm(x, residual, self.weight, self.eps, rows, keep=rows is None)
+            # `x` is the last block's output, a pair of outputs or None (nothing to add); `rows` ends the stream: only
+            # these rows are normed
+            return ops.residual_norm(x, residual, self.weight, self.eps, rows, keep=rows is None, scale=self.residual_scale,
+                                     unit_offset=self.unit_offset)
         if self.kind == "rms":
             return ops.rms_norm(x, residual, self.weight, self.eps, self.unit_offset)
         return ops.layer_norm(x, residual, self.weight, self.bias, self.eps)
+
+    def with_second(self, second: "Norm", x, residual):
+        """fp32 streams: one addition, two norms of its result -> ``(normed, normed by second, residual)``."""
+        return ops.residual_norm(x, residual, self.weight, self.eps, scale=self.residual_scale, unit_offset=self.unit_offset,
+                                 weight2=second.weight)
 
     def quant(self, x, residual=None):
         """Fused add + RMSNorm + 1x128 fp8 quantisation -> ``(xq, scales, residual)``."""
@@ -352,14 +361,18 @@ class SparseMoE:
     """Top-k routed experts.  Tensor-parallel mode slices every expert's intermediate dimension
     (what the reference does, ``layers/moe/unquantized.py:107-163``); expert-parallel mode
     (``parallel/expert.py``) places whole experts on ranks.  Either way a rank ends up with a partial
-    ``[T, H]`` output that is summed over ranks by the layer's reduction."""
+    ``[T, H]`` output that is summed over ranks by the layer's reduction.  With an ``ExpertSpec`` the layer has its own
+    expert count and sizes, ungated experts and a router in 32 bits (sigmoid scores, corrected choice)."""
 
-    def __init__(self, arch: Arch, cfg, dims: ModelDims, prefix: str, weights, comm):
+    def __init__(self, arch: Arch, cfg, dims: ModelDims, prefix: str, weights, comm, spec: Optional[ExpertSpec] = None):
         pg = weights.process_group
-        self.pg, self.comm = pg, comm
+        self.pg, self.comm, self.spec = pg, comm, spec
         self.top_k, self.num_experts, self.act = dims.top_k, dims.num_experts, dims.act
         self.renorm = arch.moe_renormalize if cfg.get("norm_topk_prob") is None else bool(cfg.norm_topk_prob)
         self.router = FastLinear(weights.get_tensor(f"{prefix}.{arch.moe_router}.weight"))
+        if spec is not None:
+            self._load_plain_experts(arch, cfg, prefix, weights, spec)
+            return
         self.sparsemixer_eps = float(cfg.get("router_jitter_noise", 0.01)) if cfg.model_type == "phimoe" else None
         self.deepseek_router = None
         if arch.mla:
@@ -409,10 +422,24 @@ class SparseMoE:
             if arch.moe_shared_gate and weights.has_tensor(f"{prefix}.{arch.moe_shared_gate}.weight"):
                 self.shared_gate = FastLinear(weights.get_tensor(f"{prefix}.{arch.moe_shared_gate}.weight"))
 
+    def _load_plain_experts(self, arch: Arch, cfg, prefix: str, weights, spec: ExpertSpec) -> None:
+        if weights.process_group.size() > 1:
+            raise NotImplementedError("layers with an expert count of their own are served on one GPU")
+        self.top_k, self.num_experts, self.act = spec.top, spec.experts, spec.act
+        self.deepseek_router = self.sparsemixer_eps = self.expert_parallel = self.shared = self.shared_gate = None
+        self.correction = weights.get_tensor(f"{prefix}.{arch.moe_correction}", to_dtype=False).float()
+        ep = [f"{prefix}.{arch.moe_expert.format(e=e)}" for e in range(spec.experts)]
+        self.w_up, self.w_down = ops.plain_expert_weights(
+            torch.stack([_expert_weight(weights, cfg, f"{p}.{arch.moe_up}") for p in ep]),        # [E, I, H]
+            torch.stack([_expert_weight(weights, cfg, f"{p}.{arch.moe_down}") for p in ep]))      # [E, H, I]
+
     def __call__(self, x, x_scale=None, reduce: bool = True, meta=None, out=None):
         if out is not None:
             out.copy_(self(x, x_scale, reduce=False, meta=meta))
             return out
+        if self.spec is not None:
+            w, idx = ops.moe_route_sigmoid(x, self.router.weight, self.correction, self.top_k, self.spec.scale)
+            return ops.moe_plain_experts(x, self.w_up, self.w_down, w, idx, self.act)
         logits = self.router(x)
         if self.deepseek_router is not None:
             w, idx = self.deepseek_router(logits)
@@ -446,8 +473,9 @@ class DecoderLayer:
         self.arch, self.dims = arch, dims
         spec = dims.mixers[idx] if dims.mixers else None
         if spec is not None:
-            self.norm1 = Norm.load(arch, f"{prefix}.{arch.norm1}", weights, dims.eps)
-            self.norm2 = Norm.load(arch, f"{prefix}.{arch.norm2}", weights, dims.eps) if spec.ff else None
+            rs = dims.residual_scale
+            self.norm1 = Norm.load(arch, f"{prefix}.{arch.norm1}", weights, dims.eps, rs)
+            self.norm2 = Norm.load(arch, f"{prefix}.{arch.norm2}", weights, dims.eps, rs) if spec.feed_forward else None
         elif cfg.model_type in ("falcon", "RefinedWeb", "RefinedWebModel"):
             # the new decoder architecture names its norms ln_attn / ln_mlp and has no input_layernorm
             self.norm1, self.norm2 = self._falcon_norms(arch, cfg, prefix, weights, dims)
@@ -460,7 +488,7 @@ class DecoderLayer:
             from .mixers import load_mixer
 
             self.attn = load_mixer(spec, f"{prefix}.{arch.mix}", weights, idx, dims.eps, comm, rotary_tables)
-            is_moe = False
+            is_moe = spec.moe is not None
         elif arch.mla:
             from .deepseek import MLAAttention, is_moe_layer
 
@@ -471,10 +499,10 @@ class DecoderLayer:
             is_moe = arch.moe
         if is_moe and cfg.get("mlp_only_layers") and idx in cfg.mlp_only_layers:
             is_moe = False
-        if spec is not None and not spec.ff:
+        if spec is not None and not spec.feed_forward:
             self.mlp = None          # a mixer without a feed-forward
         else:
-            self.mlp = (SparseMoE(arch, cfg, dims, prefix, weights, comm) if is_moe
+            self.mlp = (SparseMoE(arch, cfg, dims, prefix, weights, comm, spec.moe if spec is not None else None) if is_moe
                         else DenseMLP(arch, cfg, dims, prefix, weights, comm, idx))
         self.pg, self.comm = weights.process_group, comm
         qlin = getattr(getattr(self.attn, "qkv", None), "linear", None)
@@ -493,7 +521,10 @@ class DecoderLayer:
 
     def __call__(self, h, residual, meta: ForwardMeta, rotary, kv):
         a = self.arch
-        rs = self.dims.residual_scale
+        # an fp32 stream scales a block's output where it adds it
+        rs = 1.0 if a.residual_fp32 else self.dims.residual_scale
+        if a.parallel_residual and a.residual_fp32:
+            return self._side_by_side(h, residual, meta, rotary, kv)
         if a.parallel_residual:
             normed, residual = self.norm1(h, residual)
             # attention and MLP partial sums of a parallel block share one reduction
@@ -530,6 +561,15 @@ class DecoderLayer:
         if rs != 1.0:
             mlp = mlp * rs
         return mlp, residual
+
+    def _side_by_side(self, h, residual, meta: ForwardMeta, rotary, kv):
+        """Mixer and feed-forward of the same fp32 stream, each through its own norm; what they return is added to the
+        stream by the next norm."""
+        if self.mlp is None:
+            normed, residual = self.norm1(h, residual)
+            return self.attn(normed, None, meta, rotary, kv), residual
+        normed, mlp_in, residual = self.norm1.with_second(self.norm2, h, residual)
+        return (self.attn(normed, None, meta, rotary, kv), self.mlp(mlp_in, meta=meta)), residual
 
     @property
     def fusable_tp(self) -> bool:
@@ -609,7 +649,9 @@ class CausalDecoder:
                     self.layers.append(DecoderLayer(a, cfg, dims, px + a.layer.format(i=i), weights, i, comm))
             else:
                 self.layers.append(DecoderLayer(a, cfg, dims, px + a.layer.format(i=i), weights, i, comm, rotary_tables))
-        self.final_norm = Norm.load(a, px + a.final_norm, weights, dims.eps)
+        # layers in the order a step runs them, with a cache each: a layer may run several times
+        self.layer_runs = self.layers if dims.layer_order is None else [self.layers[i] for i in dims.layer_order]
+        self.final_norm = Norm.load(a, px + a.final_norm, weights, dims.eps, dims.residual_scale if dims.mixers else 1.0)
         head_name = px + a.lm_head if not a.lm_head.startswith("lm_head") or not prefix else a.lm_head
         candidates = [head_name, px + a.lm_head, a.lm_head, px + a.embed]
         if cfg.get("tie_word_embeddings") and not any(weights.has_tensor(f"{c}.weight") for c in candidates[:3]):
@@ -617,7 +659,10 @@ class CausalDecoder:
         with weights.use_loader(DefaultWeightsLoader()):
             for cand in candidates:
                 if weights.has_tensor(f"{cand}.weight"):
-                    self.head = TensorParallelHead.load(cfg, cand, weights)
+                    if dims.mixers and cand == px + a.embed:      # one copy of a shared table (one GPU)
+                        self.head = TensorParallelHead(FastLinear(self.embed.weight), pg, False)
+                    else:
+                        self.head = TensorParallelHead.load(cfg, cand, weights)
                     break
             else:
                 raise KeyError("no lm_head / tied embedding weight found")
@@ -691,8 +736,8 @@ class CausalDecoder:
         meta.v_first = None
         residual = ops.embed_residual(meta.input_ids, self.embed.weight, self.dims.embed_scale)
         h = None
-        for i, layer in enumerate(self.layers):
-            h, residual = layer(h, residual, meta, None, kv_cache[i])
+        for layer, cache in zip(self.layer_runs, kv_cache):
+            h, residual = layer(h, residual, meta, None, cache)
         meta.v_first = None
         return self.final_norm(h, residual, rows=meta.lm_head_indices)[0]
 

@@ -289,7 +289,7 @@ class FlashCausalLM(Model):
                  speculate: int = 0, kv_cache_dtype: Optional[torch.dtype] = None,
                  max_prefill_tokens: Optional[int] = None, eos_token_ids=None):
         windows = [w for w in model.dims.windows if w > 0]
-        # recurrent layers: the state of a prompt prefix is not kept (no prefix re-use), cannot be rolled back (no
+        # recurrent layers (short convolutions count): the state of a prompt prefix is not kept (no prefix re-use), cannot be rolled back (no
         # speculation), and a step must not run twice (no replay ahead of a batch change)
         self.recurrent = bool(getattr(model, "recurrent", False))
         if self.recurrent and speculate:
@@ -327,7 +327,7 @@ class FlashCausalLM(Model):
     def kv_bytes_per_block(self) -> int:
         d = self.dims
         if getattr(d, "mixers", None):
-            return max(1, sum(l.attn.page_bytes(BLOCK_SIZE) for l in self.model.layers))
+            return max(1, sum(l.attn.page_bytes(BLOCK_SIZE) for l in self.model.layer_runs))
         item = torch.empty((), dtype=self.kv_cache_dtype).element_size()
         return 2 * d.num_layers * BLOCK_SIZE * d.num_kv_heads * (d.attn_head_dim or d.head_dim) * item
 
@@ -373,10 +373,10 @@ class FlashCausalLM(Model):
             torch.cuda.empty_cache()
         self.num_blocks = int(num_blocks)
         if getattr(d, "mixers", None):
-            # every layer has its own kind of cache: pages, or slots of recurrent state
+            # every layer (every run of a layer) has its own kind of cache: pages, slots of recurrent state, or both
             slots = int(state_slots or self.max_batch_size or 1)
             self.state_slots = Pool(0, slots, "recurrent state slots") if self.recurrent else None
-            for layer in self.model.layers:
+            for layer in self.model.layer_runs:
                 self.kv_cache.append(layer.attn.cache_tensors(self.num_blocks, BLOCK_SIZE, slots, self.device))
             return
         for _ in range(d.num_layers):

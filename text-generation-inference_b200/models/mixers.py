@@ -3,14 +3,16 @@
 Every mixer is called like ``decoder.Attention`` (``x, x_scale, meta, rotary, kv, reduce``), owns the tensors of its
 cache (``cache_tensors``) and runs as a short sequence of fused ops:
 
-    attention   qkv GEMM -> rotate + unit RMS + value mixing + page store -> paged attention -> o GEMM
-    delta       one GEMM for q, k, v, write strengths and both low-rank inputs -> decay / gate GEMMs
+    attention   qkv GEMM -> [short convolutions +] rotate + unit RMS + value mixing + page store -> paged attention
+                -> o GEMM
+    delta       one GEMM for q, k, v, write strengths and decay / gate inputs (-> low-rank decay / gate GEMMs)
                 -> short convolutions + unit norms + decays -> state scan -> norm x gate -> o GEMM
     decay       one GEMM for q, k, v, gate -> state scan (SiLU applied on the way in) -> norm x gate -> o GEMM
 
-Recurrent layers keep, per slot of the state pool, the matrix state of every head (fp32, ``[H, vdim, pitch]``) and,
-for short convolutions, the last ``taps - 1`` inputs of every channel.  Which tokens a sequence brings and from which
-slot it continues is in the step's metadata, so prompts, portions of prompts and decoded tokens are one code path.
+Recurrent layers keep, per slot of the state pool, the matrix state of every head (fp32, ``[H, vdim, pitch]``); layers
+with short convolutions, attention layers included, the last ``taps - 1`` inputs of every channel.  Which tokens a
+sequence brings and from which slot it continues is in the step's metadata, so prompts, portions of prompts and decoded
+tokens are one code path.
 """
 from __future__ import annotations
 
@@ -87,91 +89,129 @@ class Mixer:
     def f32(self, name: str) -> torch.Tensor:
         return self.weights.get_tensor(f"{self.prefix}.{name}", to_dtype=False).float().contiguous()
 
-    def fused(self, names: Sequence[str]) -> Tuple[TensorParallelColumnLinear, List[int]]:
+    def fused(self, names: Sequence[str], bias: bool = False) -> Tuple[TensorParallelColumnLinear, List[int]]:
         w, offs = stack_rows([self.tensor(n) for n in names])
-        return TensorParallelColumnLinear(FastLinear(w)), offs
+        b = None
+        if bias:
+            b = w.new_zeros(w.shape[0])
+            for n, o in zip(names, offs):
+                part = self.tensor(f"{n}.b")
+                b[o:o + part.shape[0]] = part
+        return TensorParallelColumnLinear(FastLinear(w, b)), offs
+
+    def load_conv(self) -> None:
+        """Convolution weights of q, k and v side by side (channels of q first)."""
+        parts = [self.f32(f"{n}.conv") for n in ("q", "k", "v")]
+        self.channels, self.taps = sum(p.shape[0] for p in parts), parts[0].shape[1]
+        self.conv = ops.conv_weights(parts, self.device)
+
+    def conv_state(self, slots: int, device) -> torch.Tensor:
+        """Last ``taps - 1`` inputs of every channel, oldest first, per slot."""
+        return torch.zeros(slots, self.taps - 1, self.channels, dtype=self.dtype, device=device)
 
     def row(self, w: torch.Tensor) -> TensorParallelRowLinear:
         return TensorParallelRowLinear(FastLinear(w), self.pg, self.comm)
 
+    def page_tensors(self, num_blocks: int, block_size: int, device) -> Tuple[torch.Tensor, ...]:
+        return ()
+
+    def state_tensors(self, slots: int, device) -> Tuple[torch.Tensor, ...]:
+        return ()
+
+    def cache_tensors(self, num_blocks: int, block_size: int, slots: int, device) -> Tuple[torch.Tensor, ...]:
+        """What the mixer keeps between steps: pages (addressed by token), then states (addressed by request)."""
+        return self.page_tensors(num_blocks, block_size, device) + self.state_tensors(slots, device)
+
     def state_bytes(self) -> int:
         """Bytes of one slot of the state pool."""
-        return sum(t.numel() * t.element_size() for t in self.cache_tensors(1, 1, 1, "meta")) if self.spec.recurrent else 0
+        return sum(t.numel() * t.element_size() for t in self.state_tensors(1, "meta"))
 
     def page_bytes(self, block_size: int) -> int:
-        return 0 if self.spec.recurrent else sum(
-            t.numel() * t.element_size() for t in self.cache_tensors(1, block_size, 1, "meta"))
+        return sum(t.numel() * t.element_size() for t in self.page_tensors(1, block_size, "meta"))
 
 
 class MixedAttention(Mixer):
-    """Paged attention with its own head sizes: rotation of the first dimensions, weightless RMS of q and k after it,
-    values mixed with an earlier layer's, keys limited to the query's chunk, a sink in the softmax."""
+    """Paged attention with its own head sizes: short convolutions of q, k and v, rotation of the first dimensions,
+    weightless RMS of q and k after it, values mixed with an earlier layer's, keys limited to the query's chunk or window,
+    a sink in the softmax."""
 
     def __init__(self, spec, prefix, weights, idx, eps, comm=None, rotary: Optional[RotaryTables] = None):
         super().__init__(spec, prefix, weights, idx, eps, comm)
         s = spec
-        self.qkv, self.offs = self.fused(["q", "k", "v"])
+        self.qkv, self.offs = self.fused(["q", "k", "v"], bias=s.qkv_bias)
+        self.conv = None
+        if s.short_conv:
+            self.load_conv()
         self.v_lambda = float(self.f32("vmix").reshape(-1)[0]) if s.v_mix and weights.has_tensor(f"{prefix}.vmix") else 0.0
         self.kd, self.vd = ops.attention_pitch(s.dim, s.vdim, self.dtype, self.device)
         self.o = self.row(spread_columns(self.tensor("o"), s.heads, s.vdim, self.vd))
         self.rotary = rotary.get(s)
 
-    def cache_tensors(self, num_blocks: int, block_size: int, slots: int, device):
+    def page_tensors(self, num_blocks: int, block_size: int, device):
         # zeros: the kernels never write the padding columns of a page, and padded queries must meet zeros there
         return tuple(torch.zeros(num_blocks, block_size, self.spec.kv_heads, d, dtype=self.dtype, device=device)
                      for d in (self.kd, self.vd))
 
+    def state_tensors(self, slots: int, device):
+        return () if self.conv is None else (self.conv_state(slots, device),)
+
     def __call__(self, x, x_scale, meta, rotary, kv, reduce: bool = True, out=None):
         s = self.spec
-        k_cache, v_cache = kv
+        k_cache, v_cache = kv[:2]
         proj = self.qkv(x)
         v_first = None
         if s.v_mix:
             v_first = meta.v_first
             if v_first is None:      # the first such layer: its values are what the later ones mix in
                 meta.v_first = proj[:, self.offs[2]:self.offs[2] + s.kv_heads * s.vdim]
+        conv = None
+        if self.conv is not None:
+            conv = ops.ShortConv(self.conv, kv[2], meta.cu_seqlens_q, meta.kv_lens, meta.state_slots, meta.max_q == 1)
         q = ops.rotate_norm_store(proj, self.offs, meta.positions, self.rotary.cos_sin, meta.slots, k_cache, v_cache, s.heads,
-                                  s.kv_heads, s.dim, s.vdim, s.rot_dims, s.qk_unit_rms, self.eps, v_first, self.v_lambda)
+                                  s.kv_heads, s.dim, s.vdim, s.rot_dims, s.qk_unit_rms, self.eps, v_first, self.v_lambda,
+                                  s.rot_interleaved, conv)
         a = ops.paged_attention(q, k_cache, v_cache, meta.block_tables, meta.cu_seqlens_q, meta.kv_lens, s.scale,
-                                max_q=meta.max_q, max_kv=meta.max_kv, chunk=s.chunk, sink=s.sink)
+                                window=s.window or -1, max_q=meta.max_q, max_kv=meta.max_kv, chunk=s.chunk, sink=s.sink)
         return self.o(a.view(a.shape[0], -1), reduce=reduce, out=out)
 
 
 class GatedDelta(Mixer):
-    """Gated delta rule whose decay acts per head and key channel."""
+    """Gated delta rule whose decay acts per head and key channel (decay and gate of low rank) or per head."""
 
     def __init__(self, spec, prefix, weights, idx, eps, comm=None, rotary=None):
         super().__init__(spec, prefix, weights, idx, eps, comm)
         s = spec
-        self.proj, self.offs = self.fused(["q", "k", "v", "b", "a1", "g1"])
-        parts = [self.f32(f"{n}.conv") for n in ("q", "k", "v")]
-        self.taps = parts[0].shape[1]
-        self.conv = ops.conv_weights(parts, self.device)
-        self.a_rank, self.g_rank = (_up(self.weights.get_shape(f"{prefix}.{n}")[0]) for n in ("a1", "g1"))
-        # K padded like the rows of a1 / g1: their outputs are read where the fused product left them
-        self.a2, self.g2 = (pad_columns(self.tensor(n)) for n in ("a2", "g2"))
+        # decay and gate: read where the fused product leaves them, or low-rank products of what it leaves there
+        self.proj, self.offs = self.fused(["q", "k", "v", "b"] + (["a", "g"] if s.head_decay else ["a1", "g1"]))
+        self.load_conv()
+        if not s.head_decay:
+            self.a_rank, self.g_rank = (_up(self.weights.get_shape(f"{prefix}.{n}")[0]) for n in ("a1", "g1"))
+            # K padded like the rows of a1 / g1: their outputs are read where the fused product left them
+            self.a2, self.g2 = (pad_columns(self.tensor(n)) for n in ("a2", "g2"))
         self.a_log, self.dt_bias, self.norm = self.f32("A_log"), self.f32("dt_bias"), self.f32("norm")
         self.pitch = ops.recurrent_pitch(s.dim, self.device)
         self.o = self.row(_column_input(self.tensor("o")))
         self.out_cols = self.o.linear.weight.shape[1]
 
-    def cache_tensors(self, num_blocks: int, block_size: int, slots: int, device):
+    def state_tensors(self, slots: int, device):
         s = self.spec
-        channels = 2 * s.kv_heads * s.dim + s.heads * s.vdim
-        return (torch.zeros(slots, self.taps - 1, channels, dtype=self.dtype, device=device),
+        return (self.conv_state(slots, device),
                 torch.zeros(slots, s.heads, s.vdim, self.pitch, dtype=torch.float32, device=device))
 
     def __call__(self, x, x_scale, meta, rotary, kv, reduce: bool = True, out=None):
         s = self.spec
         conv_state, state = kv
         p = self.proj(x)
-        a = ops.linear_shallow(p[:, self.offs[4]:self.offs[4] + self.a_rank], self.a2)
-        g = ops.linear_shallow(p[:, self.offs[5]:self.offs[5] + self.g_rank], self.g2)
+        if s.head_decay:
+            a, g = (p[:, o:o + n] for o, n in zip(self.offs[4:], (s.heads, s.heads * s.vdim)))
+        else:
+            a = ops.linear_shallow(p[:, self.offs[4]:self.offs[4] + self.a_rank], self.a2)
+            g = ops.linear_shallow(p[:, self.offs[5]:self.offs[5] + self.g_rank], self.g2)
         q, k, v, decay, beta, qk = ops.delta_inputs(
             p, self.offs, a, self.conv, self.a_log, self.dt_bias, meta.cu_seqlens_q, meta.kv_lens, meta.state_slots,
-            conv_state, s.kv_heads, s.heads, s.dim, self.pitch, s.vdim, meta.max_q == 1)
+            conv_state, s.kv_heads, s.heads, s.dim, self.pitch, s.vdim, meta.max_q == 1, s.head_decay)
         o = ops.delta_scan(q, k, v, decay, beta, qk, meta.cu_seqlens_q, meta.kv_lens, meta.state_slots, state, s.dim, meta.max_q)
-        y = ops.gated_norm(o, g, self.norm, self.eps, s.heads, self.out_cols)
+        y = ops.gated_norm(o, g, self.norm, self.eps, s.heads, self.out_cols, s.gate_act)
         return self.o(y, reduce=reduce, out=out)
 
 
@@ -190,7 +230,7 @@ class DecayAttention(Mixer):
         self.o = self.row(_column_input(self.tensor("o")))
         self.out_cols = self.o.linear.weight.shape[1]
 
-    def cache_tensors(self, num_blocks: int, block_size: int, slots: int, device):
+    def state_tensors(self, slots: int, device):
         s = self.spec
         return (torch.zeros(slots, s.heads, s.vdim, self.pitch, dtype=torch.float32, device=device),)
 

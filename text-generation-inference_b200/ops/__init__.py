@@ -9,6 +9,7 @@ path, never as a default.
 from __future__ import annotations
 
 import os
+from dataclasses import dataclass
 from typing import Optional
 
 import torch
@@ -110,10 +111,24 @@ def embed_residual(ids, table, scale=1.0):
     return _mixer_backend(table).embed_residual(ids, table, scale)
 
 
-def residual_norm(delta, residual, weight, eps, rows=None, keep=True):
-    """``r = residual + delta`` in fp32 and ``RMSNorm(r) * weight`` in the weight's dtype: ``(normed, r)``.  ``rows`` picks
-    the rows to compute; ``keep=False`` drops ``r``."""
-    return _mixer_backend(residual).residual_norm(delta, residual, weight, eps, rows, keep)
+def residual_norm(delta, residual, weight, eps, rows=None, keep=True, scale=1.0, unit_offset=False, weight2=None):
+    """``r = residual + scale * delta`` in fp32 (``delta``: a tensor, a pair whose sum it is, or ``None``) and
+    ``RMSNorm(r) * weight`` (``unit_offset``: times ``1 + weight``) in the weight's dtype: ``(normed, r)``, with
+    ``weight2`` ``(normed, normed by weight2, r)``.  ``rows`` picks the rows to compute; ``keep=False`` drops ``r``."""
+    return _mixer_backend(residual).residual_norm(delta, residual, weight, eps, rows, keep, scale, unit_offset, weight2)
+
+
+@dataclass
+class ShortConv:
+    """Causal convolution over time of a step's q, k and v: weights (``conv_weights``), the pool of past inputs
+    ``[slots, taps - 1, channels]``, and which sequence brings which rows.  ``single``: one token per sequence at most."""
+
+    weights: torch.Tensor
+    state: torch.Tensor
+    cu: torch.Tensor
+    kv_lens: torch.Tensor
+    state_slots: torch.Tensor
+    single: bool
 
 
 def attention_pitch(dim, vdim, dtype, device):
@@ -124,11 +139,14 @@ def attention_pitch(dim, vdim, dtype, device):
 
 
 def rotate_norm_store(proj, offs, positions, cos_sin, slots, k_cache, v_cache, num_heads, num_kv_heads, dim, vdim, rot_dim,
-                      qk_norm, eps, v_first=None, v_lambda=0.0):
-    """``proj[T, *]`` with q, k, v from columns ``offs``: rotate q and k, divide them by their root mean square per head
-    (``qk_norm``), mix v with ``v_first`` (``(1 - lambda) v + lambda v_first``), store k and v; returns q ``[T, Hq, Dk]``."""
+                      qk_norm, eps, v_first=None, v_lambda=0.0, interleaved=False, conv=None):
+    """``proj[T, *]`` with q, k, v from columns ``offs``: convolve all three over time (``conv``, a ``ShortConv``), rotate
+    q and k (pairs ``i, i + rot_dim / 2``, or ``2i, 2i + 1`` when ``interleaved``), divide them by their root mean square
+    per head (``qk_norm``), mix v with ``v_first`` (``(1 - lambda) v + lambda v_first``), store k and v; returns q
+    ``[T, Hq, Dk]``."""
     return _mixer_backend(proj).rotate_norm_store(proj, offs, positions, cos_sin, slots, k_cache, v_cache, num_heads,
-                                                  num_kv_heads, dim, vdim, rot_dim, qk_norm, eps, v_first, v_lambda)
+                                                  num_kv_heads, dim, vdim, rot_dim, qk_norm, eps, v_first, v_lambda,
+                                                  interleaved, conv)
 
 
 def recurrent_pitch(dim, device):
@@ -147,15 +165,17 @@ def conv_weights(parts, device):
 
 
 def delta_inputs(proj, offs, a_pre, conv_t, a_log, dt_bias, cu, kv_lens, state_slots, conv_state, kv_heads, heads, dim, pitch,
-                 vdim, single):
+                 vdim, single, head_decay=False):
     """Short convolutions (``conv_weights`` of q, k, v), unit norms, decays and write strengths of a gated delta rule;
-    advances ``conv_state``."""
+    advances ``conv_state``.  Decays are one per head and key channel, or one per head (``head_decay``: ``a_pre`` and
+    ``dt_bias`` have a value per head)."""
     return _mixer_backend(proj).delta_inputs(proj, offs, a_pre, conv_t, a_log, dt_bias, cu, kv_lens, state_slots, conv_state,
-                                             kv_heads, heads, dim, pitch, vdim, single)
+                                             kv_heads, heads, dim, pitch, vdim, single, head_decay)
 
 
 def delta_scan(q, k, v, g, beta, qk, cu, kv_lens, state_slots, state, dim, max_q):
-    """Gated delta rule over the step's tokens; advances ``state`` and returns the read-outs, fp32 ``[T, H, vdim]``."""
+    """Gated delta rule over the step's tokens (decays ``g[T, H, pitch]`` or ``g[T, H]``); advances ``state`` and returns the
+    read-outs, fp32 ``[T, H, vdim]``."""
     return _mixer_backend(v).delta_scan(q, k, v, g, beta, qk, cu, kv_lens, state_slots, state, dim, max_q)
 
 
@@ -164,9 +184,10 @@ def decay_scan(proj, offs, decay, cu, kv_lens, state_slots, state, heads, dim, v
     return _mixer_backend(proj).decay_scan(proj, offs, decay, cu, kv_lens, state_slots, state, heads, dim, vdim, max_q)
 
 
-def gated_norm(o, gate, weight, eps, groups, out_cols):
-    """RMSNorm of ``o`` over each of ``groups`` equal parts, times ``weight``, times ``sigmoid(gate)``; ``[T, out_cols]``."""
-    return _mixer_backend(o).gated_norm(o, gate, weight, eps, groups, out_cols)
+def gated_norm(o, gate, weight, eps, groups, out_cols, act="sigmoid"):
+    """RMSNorm of ``o`` over each of ``groups`` equal parts, times ``weight``, times ``sigmoid(gate)`` or ``silu(gate)``;
+    ``[T, out_cols]``."""
+    return _mixer_backend(o).gated_norm(o, gate, weight, eps, groups, out_cols, act)
 
 
 def _into(out, y):
@@ -250,3 +271,22 @@ def moe_experts(x, w_gate_up, w_down, topk_weights, topk_ids, act="silu", first:
             and (w_gate_up.shape[1] // 2) % 8 == 0 and w_gate_up.shape[0] <= 256 and topk_ids.shape[1] <= 8:
         return native().moe_experts(x, w_gate_up, w_down, topk_weights, topk_ids, act, first)
     return ref.moe_experts(x, w_gate_up, w_down, topk_weights, topk_ids, act, first)
+
+
+# ---- routed experts of layers with an ``ExpertSpec`` ----------------------------------------------
+def moe_route_sigmoid(x, weight, correction, top_k, scale):
+    """Router product, sigmoid, corrected choice and weights in fp32: ``(weights [T, k], experts [T, k])``."""
+    return _mixer_backend(x).moe_route_sigmoid(x, weight, correction, top_k, scale)
+
+
+def plain_expert_weights(w_up, w_down):
+    """``[E, I, H]`` and ``[E, H, I]`` as the kernels want them: bf16 sizes brought to multiples of 8 with zeros."""
+    if use_native(w_up) and w_up.dtype == torch.bfloat16:
+        pad = lambda w: torch.nn.functional.pad(w, (0, -w.shape[2] % 8, 0, -w.shape[1] % 8))
+        w_up, w_down = pad(w_up), pad(w_down)
+    return w_up.contiguous(), w_down.contiguous()
+
+
+def moe_plain_experts(x, w_up, w_down, topk_weights, topk_ids, act):
+    """``sum over slots of weight * down(act(up x))`` of ungated experts (weights from ``plain_expert_weights``)."""
+    return _mixer_backend(x).moe_plain_experts(x, w_up, w_down, topk_weights, topk_ids, act)

@@ -1,12 +1,12 @@
 // Kernels around the token mixers of hybrid decoders (attention layers between recurrent ones), each in a bf16 and
 // an fp32 build of the activations:
-//   residual add (fp32 stream) + RMSNorm, optional row gather
+//   residual add (fp32 stream) of one or two block outputs + one or two RMSNorms, optional row gather
 //   embedding gather into the fp32 residual stream
-//   element-wise activation of a non-gated feed-forward
-//   RoPE -> per-head RMS of q and k -> value mixing -> paged K / V store
+//   element-wise activation of a non-gated feed-forward, act(gate) * up of a gated one
+//   [causal short convolution ->] RoPE -> per-head RMS of q and k -> value mixing -> paged K / V store
 //   paged attention for any head size and for fp32 pages (the tensor-core kernels serve bf16 at 64 / 128 / 256)
 //   causal short convolution + SiLU, unit norms, decays and write strengths of a gated delta rule
-//   per-group RMSNorm x weight x sigmoid(gate) on the output of a recurrent mixer
+//   per-group RMSNorm x weight x sigmoid(gate) or SiLU(gate) on the output of a recurrent mixer
 //
 // Norms, angles, scores, decays and the residual stream are fp32 in both builds; only matrix operands and what the
 // matrix products return are bf16.
@@ -80,17 +80,27 @@ __device__ __forceinline__ int sequence_of(const int* __restrict__ cu, int B, in
 }
 
 // ------------------------------------------------------------------------------------------------
-// residual (fp32) + delta -> RMSNorm.  One CTA per output row; `rows` (optional) picks the input row.
-// VPT float4 per thread stay in registers; VPT == 0: any width, the row is read twice.
+// r = residual (fp32) + scale * (d1 + d2) -> RMSNorm(r) * (offset + w1), and the same with w2.  One CTA per output row;
+// `rows` (optional) picks the input row.  VPT float4 per thread stay in registers; VPT == 0: any width, read twice.
 // ------------------------------------------------------------------------------------------------
+template <typename T>
+struct ResidualNorm {
+  const T *d1, *d2;               // null: nothing to add
+  const float* residual;
+  const int* rows;
+  const T *w1, *w2;               // w2 null: one norm
+  T *o1, *o2;
+  float* res_out;
+  int H;
+  float eps, scale, offset;
+};
 template <typename T, int VPT>
 __global__ void __launch_bounds__(1024)
-residual_norm_kernel(const T* __restrict__ delta, const float* __restrict__ residual, const int* __restrict__ rows,
-                     const T* __restrict__ weight, T* __restrict__ out, float* __restrict__ res_out, int H, float eps) {
+residual_norm_kernel(ResidualNorm<T> p) {
   tgi::pdl_wait();
   tgi::pdl_trigger();
   __shared__ float red[33];
-  const int row = rows != nullptr ? rows[blockIdx.x] : blockIdx.x;
+  const int row = p.rows != nullptr ? p.rows[blockIdx.x] : blockIdx.x, H = p.H;
   const size_t in = static_cast<size_t>(row) * H, ob = static_cast<size_t>(blockIdx.x) * H;
   float sumsq = 0.f;
   if (VPT > 0) {
@@ -99,37 +109,52 @@ residual_norm_kernel(const T* __restrict__ delta, const float* __restrict__ resi
     for (int i = 0; i < VPT; ++i) {
       const int c = (threadIdx.x + i * blockDim.x) * 4;
       if (c < H) {
-        float4 a = *reinterpret_cast<const float4*>(residual + in + c);
-        if (delta != nullptr) {
-          const float4 d = load4(delta + in + c);
-          a.x += d.x; a.y += d.y; a.z += d.z; a.w += d.w;
+        float4 a = *reinterpret_cast<const float4*>(p.residual + in + c);
+        if (p.d1 != nullptr) {
+          float4 d = load4(p.d1 + in + c);
+          if (p.d2 != nullptr) {
+            const float4 e = load4(p.d2 + in + c);
+            d.x += e.x; d.y += e.y; d.z += e.z; d.w += e.w;
+          }
+          a.x = fmaf(p.scale, d.x, a.x); a.y = fmaf(p.scale, d.y, a.y);
+          a.z = fmaf(p.scale, d.z, a.z); a.w = fmaf(p.scale, d.w, a.w);
         }
-        if (res_out != nullptr) store4(res_out + ob + c, a);
+        if (p.res_out != nullptr) store4(p.res_out + ob + c, a);
         x[i] = a;
         sumsq += a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;
       }
     }
-    const float inv = 1.f / sqrtf(block_sum(sumsq, red) / H + eps);
+    const float inv = 1.f / sqrtf(block_sum(sumsq, red) / H + p.eps);
 #pragma unroll
     for (int i = 0; i < VPT; ++i) {
       const int c = (threadIdx.x + i * blockDim.x) * 4;
       if (c < H) {
-        const float4 w = load4(weight + c);
-        store4(out + ob + c, make_float4(x[i].x * inv * w.x, x[i].y * inv * w.y, x[i].z * inv * w.z, x[i].w * inv * w.w));
+        const float4 y = make_float4(x[i].x * inv, x[i].y * inv, x[i].z * inv, x[i].w * inv);
+        auto put_norm = [&](const T* weight, T* out) {
+          const float4 w = load4(weight + c);
+          store4(out + ob + c, make_float4(y.x * (p.offset + w.x), y.y * (p.offset + w.y), y.z * (p.offset + w.z),
+                                           y.w * (p.offset + w.w)));
+        };
+        put_norm(p.w1, p.o1);
+        if (p.w2 != nullptr) put_norm(p.w2, p.o2);
       }
     }
   } else {
+    auto value = [&](int c) {
+      float a = p.residual[in + c];
+      if (p.d1 != nullptr) a = fmaf(p.scale, to_f(p.d1[in + c]) + (p.d2 != nullptr ? to_f(p.d2[in + c]) : 0.f), a);
+      return a;
+    };
     for (int c = threadIdx.x; c < H; c += blockDim.x) {
-      float a = residual[in + c];
-      if (delta != nullptr) a += to_f(delta[in + c]);
-      if (res_out != nullptr) res_out[ob + c] = a;
+      const float a = value(c);
+      if (p.res_out != nullptr) p.res_out[ob + c] = a;
       sumsq += a * a;
     }
-    const float inv = 1.f / sqrtf(block_sum(sumsq, red) / H + eps);
+    const float inv = 1.f / sqrtf(block_sum(sumsq, red) / H + p.eps);
     for (int c = threadIdx.x; c < H; c += blockDim.x) {
-      float a = residual[in + c];
-      if (delta != nullptr) a += to_f(delta[in + c]);
-      put(out + ob + c, a * inv * to_f(weight[c]));
+      const float y = value(c) * inv;
+      put(p.o1 + ob + c, y * (p.offset + to_f(p.w1[c])));
+      if (p.w2 != nullptr) put(p.o2 + ob + c, y * (p.offset + to_f(p.w2[c])));
     }
   }
 }
@@ -154,7 +179,8 @@ embed_residual_kernel(const int* __restrict__ ids, const T* __restrict__ table, 
 }
 
 // ------------------------------------------------------------------------------------------------
-// element-wise activation (codes as in the gated kernel: 0 silu, 1 gelu erf, 2 gelu tanh, 3 relu, 4 quick gelu)
+// element-wise activation (codes as in the gated kernel: 0 silu, 1 gelu erf, 2 gelu tanh, 3 relu, 4 quick gelu,
+// 5 squared relu), and act(gate) * up for fp32 and for widths the bf16 kernel does not take
 // ------------------------------------------------------------------------------------------------
 __device__ __forceinline__ float act_value(float x, int act) {
   switch (act) {
@@ -162,7 +188,20 @@ __device__ __forceinline__ float act_value(float x, int act) {
     case 1: return 0.5f * x * (1.f + erff(x * 0.70710678118654752f));
     case 2: return 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
     case 3: return fmaxf(x, 0.f);
+    case 5: { const float y = fmaxf(x, 0.f); return y * y; }
     default: return x / (1.f + expf(-1.702f * x));
+  }
+}
+template <typename T>
+__global__ void __launch_bounds__(256)
+act_mul_any_kernel(const T* __restrict__ in, T* __restrict__ out, long long n, int I, int act) {
+  tgi::pdl_wait();
+  tgi::pdl_trigger();
+  const long long stride = static_cast<long long>(gridDim.x) * blockDim.x;
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < n; i += stride) {
+    const long long t = i / I, c = i - t * I;
+    const T* row = in + t * 2 * I;
+    put(out + i, act_value(to_f(row[c]), act) * to_f(row[I + c]));
   }
 }
 template <typename T>
@@ -181,10 +220,126 @@ activation_kernel(const T* __restrict__ in, T* __restrict__ out, long long n, in
 }
 
 // ------------------------------------------------------------------------------------------------
+// Short convolutions over time, one per channel, on three groups of columns of proj[T, ld] (q, k, v).  The previous
+// taps - 1 inputs come from the step's rows or, before them, from the sequence's state [taps - 1][C] (C channels, q first,
+// oldest input first); a sequence that starts at position 0 has zeros there.  In steps of single tokens the kernel that
+// convolves also shifts the state (`update`), otherwise conv_state_kernel does it afterwards.
+// ------------------------------------------------------------------------------------------------
+struct ConvPast {
+  const float* w;                 // [rows][C] taps, oldest first; null: no convolution
+  const int *cu, *kv_lens, *slots;
+  void* state;                    // [num_slots][taps - 1][C]
+  int B, taps, C, num_slots, update;
+};
+
+// convolved value of channel `c` (column `col` of proj) for the token at row t, local index i of its sequence
+template <typename T>
+__device__ __forceinline__ float conv_value(const T* __restrict__ proj, long long ld, int col, int t, int i,
+                                            const float* __restrict__ w, const T* __restrict__ st, int C, int c,
+                                            int taps) {   // w: the channel's first tap, taps C floats apart
+  float acc = 0.f;
+  for (int j = 0; j < taps - 1; ++j) {             // tap j multiplies the input taps - 1 - j tokens back
+    const int back = taps - 1 - j;
+    float v = 0.f;
+    if (i >= back) {
+      v = to_f(proj[static_cast<size_t>(t - back) * ld + col]);
+    } else if (st != nullptr) {
+      v = to_f(st[static_cast<size_t>(taps - 1 + i - back) * C + c]);
+    }
+    acc = fmaf(w[static_cast<size_t>(j) * C], v, acc);
+  }
+  return fmaf(w[static_cast<size_t>(taps - 1) * C], to_f(proj[static_cast<size_t>(t) * ld + col]), acc);
+}
+
+// Weights and inputs of four neighbouring channels, TAPS <= 8; weights come as [TAPS][C] with absent taps zero.
+template <typename T, int TAPS>
+struct ShortConv {
+  float4 w[TAPS];
+  __device__ __forceinline__ void weights(const float* __restrict__ wt, int C, int c, bool ok) {
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j)
+      w[j] = ok ? *reinterpret_cast<const float4*>(wt + static_cast<size_t>(j) * C + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  // inputs of the token at `row` (local index i of its sequence), oldest first: rows of this step, before them the
+  // state (`st`, null: zeros)
+  __device__ __forceinline__ void inputs(float4 (&x)[TAPS], const T* __restrict__ row, long long ld, int i,
+                                         const T* __restrict__ st, int C, int taps, bool ok) const {
+    const float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i >= TAPS - 1) {               // warp-uniform
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) x[j] = ok ? load4(row - (TAPS - 1 - j) * ld) : z;
+    } else {
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) {
+        const int back = TAPS - 1 - j;
+        x[j] = z;
+        if (!ok) continue;
+        if (i >= back) x[j] = load4(row - back * ld);
+        else if (st != nullptr && taps - 1 + i - back >= 0) x[j] = load4(st + static_cast<size_t>(taps - 1 + i - back) * C);
+      }
+    }
+  }
+  __device__ __forceinline__ float4 sum(const float4* x) const {         // x: TAPS inputs, oldest first
+    float4 a = make_float4(w[0].x * x[0].x, w[0].y * x[0].y, w[0].z * x[0].z, w[0].w * x[0].w);
+#pragma unroll
+    for (int j = 1; j < TAPS; ++j) {
+      a.x = fmaf(w[j].x, x[j].x, a.x);
+      a.y = fmaf(w[j].y, x[j].y, a.y);
+      a.z = fmaf(w[j].z, x[j].z, a.z);
+      a.w = fmaf(w[j].w, x[j].w, a.w);
+    }
+    return a;
+  }
+  __device__ __forceinline__ float4 apply(const float4* x) const {       // followed by SiLU
+    const float4 a = sum(x);
+    return make_float4(silu_t<T>(a.x), silu_t<T>(a.y), silu_t<T>(a.z), silu_t<T>(a.w));
+  }
+  // the state after this token (single-token steps)
+  static __device__ __forceinline__ void save(const float4 (&x)[TAPS], T* __restrict__ st, int C, int taps, bool ok) {
+#pragma unroll
+    for (int j = 1; j < TAPS; ++j) {
+      const int e = j - 1 - (TAPS - taps);
+      if (ok && e >= 0) store4(st + static_cast<size_t>(e) * C, x[j]);
+    }
+  }
+};
+__device__ __forceinline__ float dot4(float4 a, float4 b) { return a.x * b.x + a.y * b.y + a.z * b.z + a.w * b.w; }
+__device__ __forceinline__ float decay_value(float z, float rate) {
+  return expf(-rate * (z > 20.f ? z : log1pf(expf(z))));
+}
+
+
+// last taps - 1 inputs of every sequence that contributed tokens -> its convolution state.  Grid (channels / 256, B);
+// channels 0 .. n0 - 1 are at column off0, the next n1 at off1, the rest at off2.
+template <typename T>
+__global__ void __launch_bounds__(256)
+conv_state_kernel(const T* __restrict__ proj, long long ld, int n0, int n1, int off0, int off1, int off2, ConvPast p) {
+  tgi::pdl_wait();
+  tgi::pdl_trigger();
+  const int b = blockIdx.y, c = blockIdx.x * blockDim.x + threadIdx.x;
+  const int n = p.cu[b + 1] - p.cu[b], slot = p.slots[b];
+  if (c >= p.C || n <= 0 || slot < 0 || slot >= p.num_slots) return;
+  const int col = c < n0 ? off0 + c : (c < n0 + n1 ? off1 + c - n0 : off2 + c - n0 - n1);
+  const bool fresh = p.kv_lens[b] - n <= 0;
+  T* st = static_cast<T*>(p.state) + static_cast<size_t>(slot) * (p.taps - 1) * p.C + c;
+  for (int j = 0; j < p.taps - 1; ++j) {            // ascending: entry j is only read by entries before it
+    const int i = n - (p.taps - 1) + j;             // local index of the input that belongs at entry j
+    T v = T(0.f);
+    if (i >= 0) v = proj[static_cast<size_t>(p.cu[b] + i) * ld + col];
+    else if (!fresh) v = st[static_cast<size_t>(p.taps - 1 + i) * p.C];
+    st[static_cast<size_t>(j) * p.C] = v;
+  }
+}
+
+// rows of the transposed convolution weights: absent taps in front are zero rows
+int delta_tap_rows(int taps) { return taps <= 4 ? 4 : (taps <= 8 ? 8 : taps); }
+
+// ------------------------------------------------------------------------------------------------
 // Attention inputs.  proj[T, ld] holds q (Hq heads of `dim`), k (Hkv of `dim`) and v (Hkv of `vdim`) at columns
-// 0, off_k, off_v.  One warp per (token, head): rotate the first `rot` dimensions (pairs i, i + rot / 2), divide q
-// and k by their root mean square over the head, mix v with the values of an earlier layer, and store k / v at the
-// token's slot.  q_out rows are Dk wide; columns past `dim` are zeroed.  The page pools are zero there already.
+// 0, off_k, off_v.  One warp per (token, head): convolve over time (`conv`), rotate the first `rot` dimensions (pairs
+// i, i + rot / 2, or 2i, 2i + 1 when `inter`), divide q and k by their root mean square over the head, mix v with the
+// values of an earlier layer, and store k / v at the token's slot.  q_out rows are Dk wide; columns past `dim` are zeroed.
+// The page pools are zero there already.
 // ------------------------------------------------------------------------------------------------
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -192,7 +347,7 @@ attn_prep_kernel(const T* __restrict__ proj, long long ld, int off_k, int off_v,
                  const float* __restrict__ cos_sin, const int* __restrict__ slots, const T* __restrict__ v_first,
                  long long ld_first, float lambda, T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache,
                  int T_, int Hq, int Hkv, int dim, int vdim, int Dk, int Dv, int rot, int max_pos,
-                 long long num_slots, int qk_norm, float eps) {
+                 long long num_slots, int qk_norm, float eps, int inter, ConvPast cv) {
   tgi::pdl_wait();
   tgi::pdl_trigger();
   const int lane = threadIdx.x & 31;
@@ -202,46 +357,70 @@ attn_prep_kernel(const T* __restrict__ proj, long long ld, int off_k, int off_v,
   const int t = static_cast<int>(job / heads), h = static_cast<int>(job % heads);
   const long long slot = slots[t];
   const bool slot_ok = slot >= 0 && slot < num_slots;      // padding rows have slot -1
-  const T* row = proj + static_cast<size_t>(t) * ld;
-  if (h >= Hq + Hkv) {
-    const int g = h - Hq - Hkv;
-    if (!slot_ok) return;
-    const T* v = row + off_v + static_cast<size_t>(g) * vdim;
-    const T* f = v_first != nullptr ? v_first + static_cast<size_t>(t) * ld_first + static_cast<size_t>(g) * vdim : nullptr;
-    for (int i = lane; i < vdim; i += 32) {
-      float x = to_f(v[i]);
-      if (f != nullptr) x = (1.f - lambda) * x + lambda * to_f(f[i]);
-      put(v_cache + (static_cast<size_t>(slot) * Hkv + g) * Dv + i, x);
+  const bool is_q = h < Hq, is_v = h >= Hq + Hkv;
+  const int g = is_q ? h : (is_v ? h - Hq - Hkv : h - Hq), width = is_v ? vdim : dim;
+  // first column and first channel of the head
+  const int col = (is_q ? 0 : (is_v ? off_v : off_k)) + g * width;
+  const int chan = is_v ? (Hq + Hkv) * dim + g * vdim : h * dim;
+  const T* x = proj + static_cast<size_t>(t) * ld + col;
+  T* st = nullptr;
+  const T* old = nullptr;
+  int local = 0;
+  if (cv.w != nullptr) {
+    const int b = sequence_of(cv.cu, cv.B, t), n = cv.cu[b + 1] - cv.cu[b], own = cv.slots[b];
+    local = t - cv.cu[b];
+    if (own >= 0 && own < cv.num_slots) st = static_cast<T*>(cv.state) + static_cast<size_t>(own) * (cv.taps - 1) * cv.C;
+    old = cv.kv_lens[b] - n > 0 ? st : nullptr;
+  }
+  auto value = [&](int i) {
+    return cv.w != nullptr ? conv_value(proj, ld, col + i, t, local, cv.w + chan + i, old, cv.C, chan + i, cv.taps) : to_f(x[i]);
+  };
+  auto shift_state = [&]() {                               // after every lane has read the state
+    if (cv.w == nullptr || !cv.update || st == nullptr || cv.taps < 2) return;
+    __syncwarp();
+    for (int i = lane; i < width; i += 32) {
+      for (int j = 0; j + 1 < cv.taps - 1; ++j)
+        st[static_cast<size_t>(j) * cv.C + chan + i] = old != nullptr ? st[static_cast<size_t>(j + 1) * cv.C + chan + i] : T(0.f);
+      st[static_cast<size_t>(cv.taps - 2) * cv.C + chan + i] = x[i];
     }
+  };
+  if (is_v) {
+    if (slot_ok) {
+      const T* f = v_first != nullptr ? v_first + static_cast<size_t>(t) * ld_first + static_cast<size_t>(g) * vdim : nullptr;
+      for (int i = lane; i < vdim; i += 32) {
+        float y = value(i);
+        if (f != nullptr) y = (1.f - lambda) * y + lambda * to_f(f[i]);
+        put(v_cache + (static_cast<size_t>(slot) * Hkv + g) * Dv + i, y);
+      }
+    }
+    shift_state();
     return;
   }
-  const bool is_q = h < Hq;
-  const int g = is_q ? h : h - Hq;
-  const T* x = row + (is_q ? 0 : off_k) + static_cast<size_t>(g) * dim;
   const int pos = min(max(positions[t], 0), max_pos - 1);
   const float* cs = cos_sin + static_cast<size_t>(pos) * rot;
-  const int rh = rot / 2;
-  float ss = 0.f;
-  for (int i = lane; i < rh; i += 32) {
-    const float u = to_f(x[i]), w = to_f(x[i + rh]), c = cs[i], s = cs[rh + i];
-    const float a = u * c - w * s, b = w * c + u * s;
-    ss += a * a + b * b;
+  const int rh = rot / 2, step = inter ? 2 : 1, apart = inter ? 1 : rh;
+  float inv = 1.f;
+  if (qk_norm) {
+    float ss = 0.f;
+    for (int i = lane; i < dim; i += 32) {                 // a rotation keeps the sum of squares
+      const float a = value(i);
+      ss += a * a;
+    }
+    inv = 1.f / sqrtf(warp_sum(ss) / dim + eps);
   }
-  for (int i = rot + lane; i < dim; i += 32) {
-    const float a = to_f(x[i]);
-    ss += a * a;
+  if (is_q || slot_ok) {
+    T* dst = is_q ? q_out + (static_cast<size_t>(t) * Hq + g) * Dk : k_cache + (static_cast<size_t>(slot) * Hkv + g) * Dk;
+    for (int i = lane; i < rh; i += 32) {
+      const int a = i * step, b = a + apart;
+      const float u = value(a), w = value(b), c = cs[i], s = cs[rh + i];
+      put(dst + a, (u * c - w * s) * inv);
+      put(dst + b, (w * c + u * s) * inv);
+    }
+    for (int i = rot + lane; i < dim; i += 32) put(dst + i, value(i) * inv);
+    if (is_q)
+      for (int i = dim + lane; i < Dk; i += 32) put(dst + i, 0.f);
   }
-  const float inv = qk_norm ? 1.f / sqrtf(warp_sum(ss) / dim + eps) : 1.f;
-  if (!is_q && !slot_ok) return;
-  T* dst = is_q ? q_out + (static_cast<size_t>(t) * Hq + g) * Dk : k_cache + (static_cast<size_t>(slot) * Hkv + g) * Dk;
-  for (int i = lane; i < rh; i += 32) {
-    const float u = to_f(x[i]), w = to_f(x[i + rh]), c = cs[i], s = cs[rh + i];
-    put(dst + i, (u * c - w * s) * inv);
-    put(dst + i + rh, (w * c + u * s) * inv);
-  }
-  for (int i = rot + lane; i < dim; i += 32) put(dst + i, to_f(x[i]) * inv);
-  if (is_q)
-    for (int i = dim + lane; i < Dk; i += 32) put(dst + i, 0.f);
+  shift_state();
 }
 
 // The same for rows that can be read four elements at a time (every offset, size and pitch a multiple of 4, `rot` of 8):
@@ -316,6 +495,116 @@ attn_prep_vec_kernel(const T* __restrict__ proj, long long ld, int off_k, int of
     }
     if (is_q)
       for (int i = dim + 4 * l; i < Dk; i += 64) store4(dst + i, make_float4(0.f, 0.f, 0.f, 0.f));
+  }
+}
+
+// Convolution, interleaved rotation and store of rows that can be read four elements at a time, TAPS <= 8: L lanes per
+// (run of `run` consecutive rows, head) with the head's convolution weights in registers, E pieces of 4 L channels.  RB rows
+// inside one sequence are loaded together with their TAPS - 1 predecessors (in L1 from the rows before), the first rows of a
+// sequence one by one.
+template <typename T, int L, int E, int TAPS, int RB>
+__global__ void __launch_bounds__(128)
+attn_conv_run_kernel(const T* __restrict__ proj, long long ld, int off_k, int off_v, const int* __restrict__ positions,
+                     const float* __restrict__ cos_sin, const int* __restrict__ slots, T* __restrict__ q_out,
+                     T* __restrict__ k_cache, T* __restrict__ v_cache, int T_, int Hq, int Hkv, int dim, int vdim, int Dk, int Dv,
+                     int rot, int max_pos, long long num_slots, int qk_norm, float eps, int run, ConvPast cv) {
+  tgi::pdl_wait();
+  tgi::pdl_trigger();
+  const int l = threadIdx.x % L;
+  const int h = blockIdx.y * (blockDim.x / L) + threadIdx.x / L;
+  const bool on = h < Hq + 2 * Hkv;                        // lanes past the last head stay for the exchanges
+  const int t0 = blockIdx.x * run, t1 = min(T_, t0 + run);
+  const bool is_q = h < Hq, is_v = h >= Hq + Hkv;
+  const int g = is_q ? h : (is_v ? h - Hq - Hkv : h - Hq), width = is_v ? vdim : dim;
+  const int col = (is_q ? 0 : (is_v ? off_v : off_k)) + g * width;
+  const int chan = is_v ? (Hq + Hkv) * dim + g * vdim : h * dim;
+  const int rh = rot / 2;
+  ShortConv<T, TAPS> wt[E];
+  bool ok[E];
+#pragma unroll
+  for (int e = 0; e < E; ++e) {
+    const int i = 4 * (l + L * e);
+    ok[e] = on && i < width;
+    wt[e].weights(cv.w, cv.C, chan + i, ok[e]);
+  }
+  int b = sequence_of(cv.cu, cv.B, t0), end = cv.cu[b + 1];
+  T* st = nullptr;
+  const T* old = nullptr;
+  auto enter = [&]() {                                     // sequence b: its state, and whether it has a past
+    const int n = end - cv.cu[b], slot = cv.slots[b];
+    st = slot >= 0 && slot < cv.num_slots ? static_cast<T*>(cv.state) + static_cast<size_t>(slot) * (cv.taps - 1) * cv.C : nullptr;
+    old = cv.kv_lens[b] - n > 0 ? st : nullptr;
+  };
+  enter();
+  auto emit = [&](int t, float4 (&a)[E]) {
+    float inv = 1.f;
+    if (qk_norm) {                                         // a rotation keeps the sum of squares
+      float ss = 0.f;
+#pragma unroll
+      for (int e = 0; e < E; ++e) ss += a[e].x * a[e].x + a[e].y * a[e].y + a[e].z * a[e].z + a[e].w * a[e].w;
+#pragma unroll
+      for (int o = L / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      if (!is_v) inv = 1.f / sqrtf(ss / dim + eps);
+    }
+    if (!on) return;
+    const long long slot = slots[t];
+    if (!is_q && (slot < 0 || slot >= num_slots)) return;
+    T* dst = is_q ? q_out + (static_cast<size_t>(t) * Hq + g) * Dk
+                  : (is_v ? v_cache + (static_cast<size_t>(slot) * Hkv + g) * Dv
+                          : k_cache + (static_cast<size_t>(slot) * Hkv + g) * Dk);
+    const float* cs = cos_sin + static_cast<size_t>(min(max(positions[t], 0), max_pos - 1)) * rot;
+#pragma unroll
+    for (int e = 0; e < E; ++e) {
+      const int i = 4 * (l + L * e);
+      if (!ok[e]) {
+        if (is_q && i < Dk) store4(dst + i, make_float4(0.f, 0.f, 0.f, 0.f));
+        continue;
+      }
+      float4 x = a[e];
+      if (!is_v && i < rot) {
+        const float2 c = *reinterpret_cast<const float2*>(cs + i / 2), s = *reinterpret_cast<const float2*>(cs + rh + i / 2);
+        x = make_float4(x.x * c.x - x.y * s.x, x.y * c.x + x.x * s.x, x.z * c.y - x.w * s.y, x.w * c.y + x.z * s.y);
+      }
+      store4(dst + i, make_float4(x.x * inv, x.y * inv, x.z * inv, x.w * inv));
+    }
+  };
+  for (int t = t0; t < t1;) {
+    if (t >= end) {
+      while (cv.cu[b + 1] <= t) ++b;                       // sequences without tokens in this step are skipped
+      end = cv.cu[b + 1];
+      enter();
+    }
+    const int local = t - cv.cu[b];
+    const T* row = proj + static_cast<size_t>(t) * ld + col;
+    if (RB > 1 && local >= TAPS - 1 && t + RB <= min(t1, end)) {
+      float4 x[E][TAPS - 1 + RB];
+#pragma unroll
+      for (int e = 0; e < E; ++e)
+#pragma unroll
+        for (int j = 0; j < TAPS - 1 + RB; ++j)
+          x[e][j] = ok[e] ? load4(row + (j - (TAPS - 1)) * ld + 4 * (l + L * e)) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+      for (int r = 0; r < RB; ++r) {
+        float4 a[E];
+#pragma unroll
+        for (int e = 0; e < E; ++e) a[e] = wt[e].sum(&x[e][r]);
+        emit(t + r, a);
+      }
+      t += RB;
+      continue;
+    }
+    float4 a[E];
+#pragma unroll
+    for (int e = 0; e < E; ++e) {
+      const int i = 4 * (l + L * e);
+      float4 x[TAPS];
+      wt[e].inputs(x, row + i, ld, local, old != nullptr ? old + chan + i : nullptr, cv.C, cv.taps, ok[e]);
+      a[e] = wt[e].sum(x);
+      // run == 1: these lanes alone read and write these channels' state
+      if (cv.update && st != nullptr) wt[e].save(x, st + chan + i, cv.C, cv.taps, ok[e]);
+    }
+    emit(t, a);
+    ++t;
   }
 }
 
@@ -404,10 +693,10 @@ attn_any_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T*
 
 // ------------------------------------------------------------------------------------------------
 // Inputs of a gated delta rule.  proj[T, ld]: q and k (G heads of dim), v (H of vdim), b (H) at off_q .. off_b;
-// decay[T, ld_a]: pre-activations of the decays (H x dim).  One warp per (token, unit):
+// a_pre[T, ld_a]: pre-activations of the decays (H x dim, or H).  One warp per (token, unit):
 //   units 0 .. G-1            q and k of a head: convolution, SiLU, unit norm (q also times dim^-1/2), and q . k
 //   units G .. G+H-1          v of a head: convolution, SiLU; write strength sigmoid(b)
-//   units G+H .. G+2H-1       decay exp(-exp(A_log) softplus(a + dt_bias)) of every key channel
+//   units G+H .. G+2H-1       decay exp(-exp(A_log) softplus(a + dt_bias)) of every key channel (one per head: with v)
 // q, k and the decays are written with `dimP` columns per head, zero padded.  The convolution reads the previous
 // taps - 1 inputs from the step's rows or, before them, from the sequence's state [taps - 1][C] (C = (2 G dim + H vdim)
 // channels, oldest first); a sequence that starts at position 0 has zeros there.  With `update` (every sequence
@@ -417,26 +706,8 @@ struct DeltaPrep {
   long long ld, ld_a;
   int off_q, off_k, off_v, off_b;
   int B, G, H, dim, dimP, vdim, taps, update;
+  int head_decay;                 // one decay per head: a_pre [T, H], dt_bias [H], g_out [T, H], written beside beta
 };
-
-// convolved value of channel `c` (column `col` of proj) for the token at row t, local index i of its sequence
-template <typename T>
-__device__ __forceinline__ float conv_value(const T* __restrict__ proj, long long ld, int col, int t, int i,
-                                            const float* __restrict__ w, const T* __restrict__ st, int C, int c,
-                                            int taps) {   // w: the channel's first tap, taps C floats apart
-  float acc = 0.f;
-  for (int j = 0; j < taps - 1; ++j) {             // tap j multiplies the input taps - 1 - j tokens back
-    const int back = taps - 1 - j;
-    float v = 0.f;
-    if (i >= back) {
-      v = to_f(proj[static_cast<size_t>(t - back) * ld + col]);
-    } else if (st != nullptr) {
-      v = to_f(st[static_cast<size_t>(taps - 1 + i - back) * C + c]);
-    }
-    acc = fmaf(w[static_cast<size_t>(j) * C], v, acc);
-  }
-  return fmaf(w[static_cast<size_t>(taps - 1) * C], to_f(proj[static_cast<size_t>(t) * ld + col]), acc);
-}
 
 template <typename T, int NV>
 __global__ void __launch_bounds__(256)
@@ -448,7 +719,7 @@ delta_prep_kernel(const T* __restrict__ proj, const T* __restrict__ a_pre, const
   tgi::pdl_wait();
   tgi::pdl_trigger();
   const int lane = threadIdx.x & 31;
-  const int units = p.G + 2 * p.H;
+  const int units = p.G + (p.head_decay ? 1 : 2) * p.H;
   const long long job = static_cast<long long>(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (job >= static_cast<long long>(T_) * units) return;
   const int t = static_cast<int>(job / units), u = static_cast<int>(job % units);
@@ -524,8 +795,10 @@ delta_prep_kernel(const T* __restrict__ proj, const T* __restrict__ a_pre, const
         conv_value(proj, p.ld, p.off_v + cv, t, i0, conv_t + c, old, C, c, p.taps));
     if (shift) shift_state(c, p.off_v + cv);
   }
-  if (lane == 0)
-    beta_out[static_cast<size_t>(t) * p.H + h] = sigmoid_f(to_f(proj[static_cast<size_t>(t) * p.ld + p.off_b + h]));
+  const size_t th = static_cast<size_t>(t) * p.H + h;
+  if (lane == 0) beta_out[th] = sigmoid_f(to_f(proj[static_cast<size_t>(t) * p.ld + p.off_b + h]));
+  if (p.head_decay && lane == 0)
+    g_out[th] = decay_value(to_f(a_pre[static_cast<size_t>(t) * p.ld_a + h]) + dt_bias[h], expf(A_log[h]));
 }
 
 // The same for up to TAPS <= 8 taps, with one warp per (run of `run` consecutive rows, unit): the convolution weights
@@ -533,58 +806,6 @@ delta_prep_kernel(const T* __restrict__ proj, const T* __restrict__ a_pre, const
 // inside one sequence are loaded together with their TAPS - 1 predecessors (in L1 from the rows before), the first rows
 // of a sequence one by one.  Weights come as [TAPS][C] with absent taps zero.  UNITS: 0 = all units as above, 1 = q and
 // k, 2 = v, 3 = decays (prompts: a kernel each, with the registers it needs).
-template <typename T, int TAPS>
-struct ShortConv {
-  float4 w[TAPS];
-  __device__ __forceinline__ void weights(const float* __restrict__ wt, int C, int c, bool ok) {
-#pragma unroll
-    for (int j = 0; j < TAPS; ++j)
-      w[j] = ok ? *reinterpret_cast<const float4*>(wt + static_cast<size_t>(j) * C + c) : make_float4(0.f, 0.f, 0.f, 0.f);
-  }
-  // inputs of the token at `row` (local index i of its sequence), oldest first: rows of this step, before them the
-  // state (`st`, null: zeros)
-  __device__ __forceinline__ void inputs(float4 (&x)[TAPS], const T* __restrict__ row, long long ld, int i,
-                                         const T* __restrict__ st, int C, int taps, bool ok) const {
-    const float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (i >= TAPS - 1) {               // warp-uniform
-#pragma unroll
-      for (int j = 0; j < TAPS; ++j) x[j] = ok ? load4(row - (TAPS - 1 - j) * ld) : z;
-    } else {
-#pragma unroll
-      for (int j = 0; j < TAPS; ++j) {
-        const int back = TAPS - 1 - j;
-        x[j] = z;
-        if (!ok) continue;
-        if (i >= back) x[j] = load4(row - back * ld);
-        else if (st != nullptr && taps - 1 + i - back >= 0) x[j] = load4(st + static_cast<size_t>(taps - 1 + i - back) * C);
-      }
-    }
-  }
-  __device__ __forceinline__ float4 apply(const float4* x) const {       // x: TAPS inputs, oldest first
-    float4 a = make_float4(w[0].x * x[0].x, w[0].y * x[0].y, w[0].z * x[0].z, w[0].w * x[0].w);
-#pragma unroll
-    for (int j = 1; j < TAPS; ++j) {
-      a.x = fmaf(w[j].x, x[j].x, a.x);
-      a.y = fmaf(w[j].y, x[j].y, a.y);
-      a.z = fmaf(w[j].z, x[j].z, a.z);
-      a.w = fmaf(w[j].w, x[j].w, a.w);
-    }
-    return make_float4(silu_t<T>(a.x), silu_t<T>(a.y), silu_t<T>(a.z), silu_t<T>(a.w));
-  }
-  // the state after this token (single-token steps)
-  static __device__ __forceinline__ void save(const float4 (&x)[TAPS], T* __restrict__ st, int C, int taps, bool ok) {
-#pragma unroll
-    for (int j = 1; j < TAPS; ++j) {
-      const int e = j - 1 - (TAPS - taps);
-      if (ok && e >= 0) store4(st + static_cast<size_t>(e) * C, x[j]);
-    }
-  }
-};
-__device__ __forceinline__ float dot4(float4 a, float4 b) { return a.x * b.x + a.y * b.y + a.z * b.z + a.w * b.w; }
-__device__ __forceinline__ float decay_value(float z, float rate) {
-  return expf(-rate * (z > 20.f ? z : log1pf(expf(z))));
-}
-
 template <typename T, int E, int TAPS, int UNITS, int RB>
 __global__ void __launch_bounds__(128)
 delta_prep_run_kernel(const T* __restrict__ proj, const T* __restrict__ a_pre, const float* __restrict__ conv_t,
@@ -598,7 +819,7 @@ delta_prep_run_kernel(const T* __restrict__ proj, const T* __restrict__ a_pre, c
   const int lane = threadIdx.x & 31;
   const int first = UNITS == 2 ? p.G : (UNITS == 3 ? p.G + p.H : 0);
   const int u = first + blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
-  if (u >= (UNITS == 1 ? p.G : (UNITS == 2 ? p.G + p.H : p.G + 2 * p.H))) return;
+  if (u >= (UNITS == 1 ? p.G : (UNITS == 2 || p.head_decay ? p.G + p.H : p.G + 2 * p.H))) return;
   const int t0 = blockIdx.x * run, t1 = min(T_, t0 + run);
   if (UNITS == 3 || (UNITS == 0 && u >= p.G + p.H)) {
     const int h = u - p.G - p.H;
@@ -629,6 +850,8 @@ delta_prep_run_kernel(const T* __restrict__ proj, const T* __restrict__ a_pre, c
   // channel and column of the head's first element: q (or v), and k
   const int ca = is_v ? 2 * p.G * p.dim + h * p.vdim : h * p.dim, ck = p.G * p.dim + h * p.dim;
   const int cola = (is_v ? p.off_v + h * p.vdim : p.off_q + h * p.dim), colk = p.off_k + h * p.dim;
+  const bool decays = is_v && p.head_decay;
+  const float rate_h = decays ? expf(A_log[h]) : 0.f, bias_h = decays ? dt_bias[h] : 0.f;
   ShortConv<T, TAPS> wa[E], wk[E];
 #pragma unroll
   for (int e = 0; e < E; ++e) {
@@ -652,8 +875,10 @@ delta_prep_run_kernel(const T* __restrict__ proj, const T* __restrict__ a_pre, c
         const int i = 4 * lane + 128 * e;
         if (i < width) store4(v_out + (static_cast<size_t>(t) * p.H + h) * p.vdim + i, a[e]);
       }
-      if (lane == 0)
-        beta_out[static_cast<size_t>(t) * p.H + h] = sigmoid_f(to_f(proj[static_cast<size_t>(t) * p.ld + p.off_b + h]));
+      const size_t th = static_cast<size_t>(t) * p.H + h;
+      if (lane == 0) beta_out[th] = sigmoid_f(to_f(proj[static_cast<size_t>(t) * p.ld + p.off_b + h]));
+      if (p.head_decay && lane == 1)
+        g_out[th] = decay_value(to_f(a_pre[static_cast<size_t>(t) * p.ld_a + h]) + bias_h, rate_h);
       return;
     }
     float sq = 0.f, sk = 0.f, dq = 0.f;
@@ -731,35 +956,17 @@ delta_prep_run_kernel(const T* __restrict__ proj, const T* __restrict__ a_pre, c
   }
 }
 
-// last taps - 1 inputs of every sequence that contributed tokens -> its convolution state.  Grid (channels / 256, B).
-template <typename T>
-__global__ void __launch_bounds__(256)
-conv_state_kernel(const T* __restrict__ proj, const int* __restrict__ cu, const int* __restrict__ kv_lens,
-                  const int* __restrict__ state_slots, T* __restrict__ conv_state, int num_slots, DeltaPrep p) {
-  tgi::pdl_wait();
-  tgi::pdl_trigger();
-  const int b = blockIdx.y, c = blockIdx.x * blockDim.x + threadIdx.x;
-  const int nq = p.G * p.dim, C = 2 * nq + p.H * p.vdim;
-  const int n = cu[b + 1] - cu[b], slot = state_slots[b];
-  if (c >= C || n <= 0 || slot < 0 || slot >= num_slots) return;
-  const int col = c < nq ? p.off_q + c : (c < 2 * nq ? p.off_k + c - nq : p.off_v + c - 2 * nq);
-  const bool fresh = kv_lens[b] - n <= 0;
-  T* st = conv_state + static_cast<size_t>(slot) * (p.taps - 1) * C + c;
-  for (int j = 0; j < p.taps - 1; ++j) {            // ascending: entry j is only read by entries before it
-    const int i = n - (p.taps - 1) + j;             // local index of the input that belongs at entry j
-    T v = T(0.f);
-    if (i >= 0) v = proj[static_cast<size_t>(cu[b] + i) * p.ld + col];
-    else if (!fresh) v = st[static_cast<size_t>(p.taps - 1 + i) * C];
-    st[static_cast<size_t>(j) * C] = v;
-  }
-}
-
 // ------------------------------------------------------------------------------------------------
-// out = RMSNorm(o over `width`) * weight * sigmoid(gate).  o fp32 [T, groups, width]; gate at column `off` of a
+// out = RMSNorm(o over `width`) * weight * sigmoid(gate) (SILU: silu(gate)).  o fp32 [T, groups, width]; gate at column `off` of a
 // [T, ld] matrix; out rows are `ld_out` wide, columns past groups * width are zeroed by group 0.
 // One warp (width <= 1024) or one block per (token, group); grid (tokens, groups / warps of a block).
 // ------------------------------------------------------------------------------------------------
-template <typename T, bool WARP>
+template <typename T, bool SILU>
+__device__ __forceinline__ float gate_value(float x) {
+  if (SILU) return silu_t<T>(x);
+  return sigmoid_t<T>(x);
+}
+template <typename T, bool WARP, bool SILU>
 __global__ void __launch_bounds__(256)
 gated_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, long long ld, int off,
                   const float* __restrict__ weight, T* __restrict__ out, long long ld_out, int T_, int groups, int width,
@@ -792,8 +999,8 @@ gated_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, long 
       const int i = (first + e * step) * 4;
       if (i < width) {
         const float4 w = load4(weight + i), s = load4(gt + i);
-        store4(dst + i, make_float4(v[e].x * inv * w.x * sigmoid_t<T>(s.x), v[e].y * inv * w.y * sigmoid_t<T>(s.y),
-                                    v[e].z * inv * w.z * sigmoid_t<T>(s.z), v[e].w * inv * w.w * sigmoid_t<T>(s.w)));
+        store4(dst + i, make_float4(v[e].x * inv * w.x * gate_value<T, SILU>(s.x), v[e].y * inv * w.y * gate_value<T, SILU>(s.y),
+                                    v[e].z * inv * w.z * gate_value<T, SILU>(s.z), v[e].w * inv * w.w * gate_value<T, SILU>(s.w)));
       }
     }
     if (g == 0)
@@ -813,38 +1020,35 @@ gated_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, long 
   if (vec) {
     for (int i = first * 4; i < width; i += step * 4) {
       const float4 v = load4(x + i), w = load4(weight + i), s = load4(gt + i);
-      store4(dst + i, make_float4(v.x * inv * w.x * sigmoid_t<T>(s.x), v.y * inv * w.y * sigmoid_t<T>(s.y),
-                                  v.z * inv * w.z * sigmoid_t<T>(s.z), v.w * inv * w.w * sigmoid_t<T>(s.w)));
+      store4(dst + i, make_float4(v.x * inv * w.x * gate_value<T, SILU>(s.x), v.y * inv * w.y * gate_value<T, SILU>(s.y),
+                                  v.z * inv * w.z * gate_value<T, SILU>(s.z), v.w * inv * w.w * gate_value<T, SILU>(s.w)));
     }
   } else {
-    for (int i = first; i < width; i += step) put(dst + i, x[i] * inv * weight[i] * sigmoid_f(to_f(gt[i])));
+    for (int i = first; i < width; i += step) put(dst + i, x[i] * inv * weight[i] * gate_value<float, SILU>(to_f(gt[i])));
   }
   if (g == 0)
     for (int i = groups * width + first; i < ld_out; i += step) put(out + static_cast<size_t>(t) * ld_out + i, 0.f);
 }
 
-// rows of the transposed convolution weights: absent taps in front are zero rows
-int delta_tap_rows(int taps) { return taps <= 4 ? 4 : (taps <= 8 ? 8 : taps); }
-
 int done() { return cudaGetLastError() == cudaSuccess ? 0 : -3; }
 
 template <typename T>
-int residual_norm(const void* delta, const float* residual, const int* rows, const void* weight, void* out, float* res_out,
-                  int n, int H, float eps, cudaStream_t stream) {
-  const T* d = static_cast<const T*>(delta);
-  const T* w = static_cast<const T*>(weight);
-  T* o = static_cast<T*>(out);
+int residual_norm(const void* d1, const void* d2, const float* residual, const int* rows, const void* w1, const void* w2,
+                  void* o1, void* o2, float* res_out, int n, int H, float eps, float scale, float offset, cudaStream_t stream) {
+  const ResidualNorm<T> p{static_cast<const T*>(d1), static_cast<const T*>(d2), residual, rows, static_cast<const T*>(w1),
+                          static_cast<const T*>(w2), static_cast<T*>(o1), static_cast<T*>(o2), res_out, H, eps, scale, offset};
   if (H % 4 == 0 && H / 4 <= 4 * 1024) {
     const int vecs = H / 4;
     int threads = vecs >= 1024 ? 512 : ((vecs + 31) / 32) * 32;
     if (threads > 256 && vecs <= 1024) threads = 256;
     const int vpt = (vecs + threads - 1) / threads;
-    if (vpt <= 1) tgi::launch(residual_norm_kernel<T, 1>, dim3(n), dim3(threads), 0, stream, d, residual, rows, w, o, res_out, H, eps);
-    else if (vpt <= 2) tgi::launch(residual_norm_kernel<T, 2>, dim3(n), dim3(threads), 0, stream, d, residual, rows, w, o, res_out, H, eps);
-    else if (vpt <= 4) tgi::launch(residual_norm_kernel<T, 4>, dim3(n), dim3(threads), 0, stream, d, residual, rows, w, o, res_out, H, eps);
-    else tgi::launch(residual_norm_kernel<T, 8>, dim3(n), dim3(threads), 0, stream, d, residual, rows, w, o, res_out, H, eps);
+    auto go = [&](auto kern) { tgi::launch(kern, dim3(n), dim3(threads), 0, stream, p); };
+    if (vpt <= 1) go(residual_norm_kernel<T, 1>);
+    else if (vpt <= 2) go(residual_norm_kernel<T, 2>);
+    else if (vpt <= 4) go(residual_norm_kernel<T, 4>);
+    else go(residual_norm_kernel<T, 8>);
   } else {
-    tgi::launch(residual_norm_kernel<T, 0>, dim3(n), dim3(256), 0, stream, d, residual, rows, w, o, res_out, H, eps);
+    tgi::launch(residual_norm_kernel<T, 0>, dim3(n), dim3(256), 0, stream, p);
   }
   return done();
 }
@@ -875,11 +1079,11 @@ int delta_prep(const void* proj, const void* a_pre, const float* conv_t, const f
   const T* x = static_cast<const T*>(proj);
   const T* a = static_cast<const T*>(a_pre);
   T* st = static_cast<T*>(conv_state);
-  const int units = p.G + 2 * p.H, C = 2 * p.G * p.dim + p.H * p.vdim;
-  const bool vec = p.taps <= 8 && p.dim % 4 == 0 && p.vdim % 4 == 0 && p.vdim <= 256 && p.ld % 4 == 0 && p.ld_a % 4 == 0 &&
+  const int units = p.G + (p.head_decay ? 1 : 2) * p.H, C = 2 * p.G * p.dim + p.H * p.vdim;
+  const bool vec = p.taps <= 8 && p.dim % 4 == 0 && p.vdim % 4 == 0 && p.vdim <= 256 && p.ld % 4 == 0 &&
                    p.off_q % 4 == 0 && p.off_k % 4 == 0 && p.off_v % 4 == 0 &&
                    reinterpret_cast<uintptr_t>(proj) % (4 * sizeof(T)) == 0 &&
-                   reinterpret_cast<uintptr_t>(a_pre) % (4 * sizeof(T)) == 0;
+                   (p.head_decay || (p.ld_a % 4 == 0 && reinterpret_cast<uintptr_t>(a_pre) % (4 * sizeof(T)) == 0));
   if (vec) {
     const bool one = p.dimP <= 128 && p.vdim <= 128;
     auto go = [&](auto kern, int count, int run) {
@@ -892,7 +1096,7 @@ int delta_prep(const void* proj, const void* a_pre, const float* conv_t, const f
     } else if (p.taps <= 4 && one) {
       go(delta_prep_run_kernel<T, 1, 4, 1, 2>, p.G, 16);
       go(delta_prep_run_kernel<T, 1, 4, 2, 4>, p.H, 32);
-      go(delta_prep_run_kernel<T, 1, 4, 3, 1>, p.H, 16);
+      if (!p.head_decay) go(delta_prep_run_kernel<T, 1, 4, 3, 1>, p.H, 16);
     } else if (p.taps <= 4) {
       go(delta_prep_run_kernel<T, 2, 4, 0, 1>, units, 16);
     } else {
@@ -911,20 +1115,25 @@ int delta_prep(const void* proj, const void* a_pre, const float* conv_t, const f
     else go(delta_prep_kernel<T, 8>);
   }
   if (!p.update && p.taps > 1)
-    tgi::launch(conv_state_kernel<T>, dim3((C + 255) / 256, p.B), dim3(256), 0, stream, x, cu, kv, slots, st, num_slots, p);
+    tgi::launch(conv_state_kernel<T>, dim3((C + 255) / 256, p.B), dim3(256), 0, stream, x, p.ld, p.G * p.dim, p.G * p.dim,
+                p.off_q, p.off_k, p.off_v, ConvPast{nullptr, cu, kv, slots, conv_state, p.B, p.taps, C, num_slots, 0});
   return done();
 }
 
 template <typename T>
 int gated_norm(const float* o, const void* gate, long long ld, int off, const float* w, void* out, long long ld_out, int T_,
-               int groups, int width, float eps, cudaStream_t stream) {
+               int groups, int width, float eps, int silu, cudaStream_t stream) {
+  auto go = [&](auto kern, dim3 grid, int threads) {
+    tgi::launch(kern, grid, dim3(threads), 0, stream, o, static_cast<const T*>(gate), ld, off, w, static_cast<T*>(out), ld_out,
+                T_, groups, width, eps);
+  };
   if (width <= 1024) {
     const int warps = groups < 8 ? groups : 8;
-    tgi::launch(gated_norm_kernel<T, true>, dim3(T_, (groups + warps - 1) / warps), dim3(32 * warps), 0, stream, o,
-                static_cast<const T*>(gate), ld, off, w, static_cast<T*>(out), ld_out, T_, groups, width, eps);
+    const dim3 grid(T_, (groups + warps - 1) / warps);
+    silu ? go(gated_norm_kernel<T, true, true>, grid, 32 * warps) : go(gated_norm_kernel<T, true, false>, grid, 32 * warps);
   } else {
-    tgi::launch(gated_norm_kernel<T, false>, dim3(T_, groups), dim3(256), 0, stream, o, static_cast<const T*>(gate), ld, off, w,
-                static_cast<T*>(out), ld_out, T_, groups, width, eps);
+    const dim3 grid(T_, groups);
+    silu ? go(gated_norm_kernel<T, false, true>, grid, 256) : go(gated_norm_kernel<T, false, false>, grid, 256);
   }
   return done();
 }
@@ -934,11 +1143,13 @@ int gated_norm(const float* o, const void* gate, long long ld, int off, const fl
 // `f32` selects the build: 1 = fp32 activations, weights and pages, 0 = bf16.
 extern "C" {
 
-int tgi_residual_norm(int f32, const void* delta, const float* residual, const int* rows, const void* weight, void* out,
-                      float* res_out, int n, int H, float eps, cudaStream_t stream) {
+// d2, w2 (with o2) and rows may be null; d1 null: the stream as it is
+int tgi_residual_norm(int f32, const void* d1, const void* d2, const float* residual, const int* rows, const void* w1,
+                      const void* w2, void* o1, void* o2, float* res_out, int n, int H, float eps, float scale, float offset,
+                      cudaStream_t stream) {
   if (n <= 0) return 0;
-  return f32 ? residual_norm<float>(delta, residual, rows, weight, out, res_out, n, H, eps, stream)
-             : residual_norm<bf16>(delta, residual, rows, weight, out, res_out, n, H, eps, stream);
+  return f32 ? residual_norm<float>(d1, d2, residual, rows, w1, w2, o1, o2, res_out, n, H, eps, scale, offset, stream)
+             : residual_norm<bf16>(d1, d2, residual, rows, w1, w2, o1, o2, res_out, n, H, eps, scale, offset, stream);
 }
 
 int tgi_embed_residual(int f32, const int* ids, const void* table, float* out, int T, int H, int vocab, float scale,
@@ -960,15 +1171,72 @@ int tgi_activation(int f32, const void* in, void* out, long long n, int act, cud
   return done();
 }
 
+// in [T, 2 I] (gate, up) -> out [T, I] = act(gate) * up
+int tgi_act_mul_any(int f32, const void* in, void* out, int T, int I, int act, cudaStream_t stream) {
+  const long long n = static_cast<long long>(T) * I;
+  if (n <= 0) return 0;
+  const dim3 grid(static_cast<unsigned>((n + 255) / 256 < 148 * 16 ? (n + 255) / 256 : 148 * 16));
+  if (f32) tgi::launch(act_mul_any_kernel<float>, grid, dim3(256), 0, stream, static_cast<const float*>(in), static_cast<float*>(out), n, I, act);
+  else tgi::launch(act_mul_any_kernel<bf16>, grid, dim3(256), 0, stream, static_cast<const bf16*>(in), static_cast<bf16*>(out), n, I, act);
+  return done();
+}
+
+// `conv_t` (optional): weights [tgi_delta_tap_rows(taps)][C] of short convolutions on q, k and v, with the sequences' past
+// inputs in conv_state [conv_slots][taps - 1][C]; `update`: no sequence brings more than one token.  `inter`: rotate pairs
+// 2i, 2i + 1.
 int tgi_attn_prep(int f32, const void* proj, long long ld, int off_k, int off_v, const int* positions, const float* cos_sin,
                   const int* slots, const void* v_first, long long ld_first, float lambda, void* q_out, void* k_cache,
                   void* v_cache, int T, int Hq, int Hkv, int dim, int vdim, int Dk, int Dv, int rot, int max_pos,
-                  long long num_slots, int qk_norm, float eps, cudaStream_t stream) {
+                  long long num_slots, int qk_norm, float eps, int inter, const float* conv_t, const int* cu,
+                  const int* kv_lens, const int* state_slots, void* conv_state, int B, int taps, int conv_slots, int update,
+                  cudaStream_t stream) {
   if (T <= 0) return 0;
   if (rot % 2 != 0 || rot > dim || Dk < dim || Dv < vdim) return -10;
-  const bool vec = rot % 8 == 0 && ld % 4 == 0 && off_k % 4 == 0 && off_v % 4 == 0 && ld_first % 4 == 0 && dim % 4 == 0 &&
-                   vdim % 4 == 0 && Dk % 4 == 0 && Dv % 4 == 0 && dim <= 256 &&
-                   reinterpret_cast<uintptr_t>(proj) % (f32 ? 16 : 8) == 0 &&
+  const bool conv = conv_t != nullptr;
+  if (conv && (taps < 1 || B < 1 || B > 65535)) return -10;
+  ConvPast cv{conv_t, cu, kv_lens, state_slots, conv_state, B, taps, (Hq + Hkv) * dim + Hkv * vdim, conv_slots, update};
+  const bool quads = ld % 4 == 0 && off_k % 4 == 0 && off_v % 4 == 0 && dim % 4 == 0 && vdim % 4 == 0 && Dk % 4 == 0 &&
+                     Dv % 4 == 0 && dim <= 256 && reinterpret_cast<uintptr_t>(proj) % (f32 ? 16 : 8) == 0;
+  auto finish = [&]() {                                    // the state of sequences that brought several tokens
+    if (conv && !update && taps > 1) {
+      const dim3 grid((cv.C + 255) / 256, B);
+      if (f32) tgi::launch(conv_state_kernel<float>, grid, dim3(256), 0, stream, static_cast<const float*>(proj), ld, Hq * dim, Hkv * dim, 0, off_k, off_v, cv);
+      else tgi::launch(conv_state_kernel<bf16>, grid, dim3(256), 0, stream, static_cast<const bf16*>(proj), ld, Hq * dim, Hkv * dim, 0, off_k, off_v, cv);
+    }
+    return done();
+  };
+  if (conv && inter && quads && rot % 4 == 0 && v_first == nullptr && taps <= 8 && vdim <= 256 && Dk <= 256) {
+    auto go = [&](auto kern, auto tag, int lanes, int run) {
+      using E = decltype(tag);
+      const int per = 128 / lanes;
+      tgi::launch(kern, dim3((T + run - 1) / run, (Hq + 2 * Hkv + per - 1) / per), dim3(128), 0, stream,
+                  static_cast<const E*>(proj), ld, off_k, off_v, positions, cos_sin, slots, static_cast<E*>(q_out),
+                  static_cast<E*>(k_cache), static_cast<E*>(v_cache), T, Hq, Hkv, dim, vdim, Dk, Dv, rot, max_pos, num_slots,
+                  qk_norm, eps, run, cv);
+    };
+    auto shape = [&](auto tag) {
+      using E = decltype(tag);
+      const int w = Dk > vdim ? Dk : vdim;                 // the columns past `dim` of q_out are written too
+      if (taps <= 4) {
+        if (update) {
+          if (w <= 64) go(attn_conv_run_kernel<E, 16, 1, 4, 1>, tag, 16, 1);
+          else if (w <= 128) go(attn_conv_run_kernel<E, 32, 1, 4, 1>, tag, 32, 1);
+          else go(attn_conv_run_kernel<E, 32, 2, 4, 1>, tag, 32, 1);
+        } else {
+          if (w <= 64) go(attn_conv_run_kernel<E, 16, 1, 4, 4>, tag, 16, 16);
+          else if (w <= 128) go(attn_conv_run_kernel<E, 32, 1, 4, 4>, tag, 32, 16);
+          else go(attn_conv_run_kernel<E, 32, 2, 4, 2>, tag, 32, 16);
+        }
+      } else {
+        if (w <= 128) go(attn_conv_run_kernel<E, 32, 1, 8, 1>, tag, 32, update ? 1 : 16);
+        else go(attn_conv_run_kernel<E, 32, 2, 8, 1>, tag, 32, update ? 1 : 16);
+      }
+    };
+    if (f32) shape(float());
+    else shape(bf16());
+    return finish();
+  }
+  const bool vec = !conv && !inter && quads && rot % 8 == 0 && ld_first % 4 == 0 &&
                    reinterpret_cast<uintptr_t>(v_first) % (f32 ? 16 : 8) == 0;
   if (vec) {
     auto go = [&](auto kern, auto tag) {
@@ -986,15 +1254,17 @@ int tgi_attn_prep(int f32, const void* proj, long long ld, int off_k, int off_v,
   }
   const long long jobs = static_cast<long long>(T) * (Hq + 2 * Hkv);
   const dim3 grid(static_cast<unsigned>((jobs + 7) / 8));
+  if (conv) cv.w += static_cast<size_t>(delta_tap_rows(taps) - taps) * cv.C;
   auto go = [&](auto kern, auto tag) {
     using E = decltype(tag);
     tgi::launch(kern, grid, dim3(256), 0, stream, static_cast<const E*>(proj), ld, off_k, off_v, positions, cos_sin, slots,
                 static_cast<const E*>(v_first), ld_first, lambda, static_cast<E*>(q_out), static_cast<E*>(k_cache),
                 static_cast<E*>(v_cache), T, Hq, Hkv, dim, vdim, Dk, Dv, rot, max_pos, num_slots,
-                qk_norm, eps);
-    return done();
+                qk_norm, eps, inter, cv);
   };
-  return f32 ? go(attn_prep_kernel<float>, float()) : go(attn_prep_kernel<bf16>, bf16());
+  if (f32) go(attn_prep_kernel<float>, float());
+  else go(attn_prep_kernel<bf16>, bf16());
+  return finish();
 }
 
 int tgi_attn_any(int f32, const void* q, const void* k_cache, const void* v_cache, const int* block_tables, const int* cu,
@@ -1017,10 +1287,10 @@ int tgi_delta_prep(int f32, const void* proj, long long ld, int off_q, int off_k
                    long long ld_a, const float* conv_t, const float* A_log, const float* dt_bias, const int* cu,
                    const int* kv_lens, const int* state_slots, void* conv_state, float* q, float* k, float* v, float* g,
                    float* beta, float* qk, int T, int B, int num_slots, int G, int H, int dim, int dimP, int vdim, int taps,
-                   int update, cudaStream_t stream) {
+                   int update, int head_decay, cudaStream_t stream) {
   if (T <= 0 || B <= 0) return 0;
   if (H % G != 0 || dimP < dim || dimP > 256 || taps < 1 || B > 65535) return -10;
-  const DeltaPrep p{ld, ld_a, off_q, off_k, off_v, off_b, B, G, H, dim, dimP, vdim, taps, update};
+  const DeltaPrep p{ld, ld_a, off_q, off_k, off_v, off_b, B, G, H, dim, dimP, vdim, taps, update, head_decay};
   return f32 ? delta_prep<float>(proj, a_pre, conv_t, A_log, dt_bias, cu, kv_lens, state_slots, conv_state, q, k, v, g, beta,
                                  qk, T, num_slots, p, stream)
              : delta_prep<bf16>(proj, a_pre, conv_t, A_log, dt_bias, cu, kv_lens, state_slots, conv_state, q, k, v, g, beta, qk,
@@ -1028,10 +1298,10 @@ int tgi_delta_prep(int f32, const void* proj, long long ld, int off_q, int off_k
 }
 
 int tgi_gated_norm(int f32, const float* o, const void* gate, long long ld, int off, const float* weight, void* out,
-                   long long ld_out, int T, int groups, int width, float eps, cudaStream_t stream) {
+                   long long ld_out, int T, int groups, int width, float eps, int silu, cudaStream_t stream) {
   if (T <= 0) return 0;
-  return f32 ? gated_norm<float>(o, gate, ld, off, weight, out, ld_out, T, groups, width, eps, stream)
-             : gated_norm<bf16>(o, gate, ld, off, weight, out, ld_out, T, groups, width, eps, stream);
+  return f32 ? gated_norm<float>(o, gate, ld, off, weight, out, ld_out, T, groups, width, eps, silu, stream)
+             : gated_norm<bf16>(o, gate, ld, off, weight, out, ld_out, T, groups, width, eps, silu, stream);
 }
 
 }  // extern "C"

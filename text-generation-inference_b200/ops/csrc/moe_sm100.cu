@@ -1,13 +1,16 @@
 // Sparse mixture-of-experts on sm_100a without a host round trip:
 //
 //   tgi_moe_topk_softmax   softmax over the router logits + top-k (+ renormalisation), one warp per token
+//   tgi_moe_router         router product in fp32 (bf16 operands), split over K into partial sums
+//   tgi_moe_topk_sigmoid   sigmoid scores, top-k of score + correction, weights scaled to a given sum, one warp per token
 //   tgi_moe_sort           groups the (token, slot) pairs of the LOCAL experts by expert: per-expert counts
 //                          and offsets, position of every pair in the grouped order, and the inverse list
 //   tgi_moe_gather         copies the token rows into the grouped activation matrix
 //   tgi_moe_grouped_gemm   one launch over all local experts: tcgen05 / TMEM / TMA GEMM whose tile list is
-//                          derived on the device from the per-expert counts.  Two epilogues: gate_up with
-//                          act(gate) * up fused (writes [rows, I]), down with the routing weight applied
-//                          (writes [rows, H])
+//                          derived on the device from the per-expert counts.  Three epilogues: gate_up with
+//                          act(gate) * up fused (writes [rows, I]), up of an ungated expert with act fused, down with
+//                          the routing weight applied (writes [rows, H])
+//   tgi_moe_grouped_f32    the same two products of ungated experts in fp32 (FMA)
 //   tgi_moe_combine        sums the top-k rows of every token in slot order (fixed order: bit-reproducible)
 //
 // Replaces, in the reference, `fused_topk` / `grouped_topk` + `moe_align_block_size` + the Triton
@@ -35,7 +38,8 @@ using namespace sm100;
 namespace {
 
 constexpr int kMaxExperts = 256;
-constexpr int kMaxTopK = 8;
+constexpr int kMaxTopK = 8;          // slots the kernels keep in registers
+constexpr int kMaxTopKSigmoid = 32;  // one lane per slot
 
 __device__ __forceinline__ void report(int* status, int code) {
   if (status != nullptr) atomicCAS(status, 0, code);
@@ -109,6 +113,135 @@ moe_topk_softmax_kernel(const T* __restrict__ logits, int tokens, int E, int k, 
 }
 
 // ------------------------------------------------------------------------------------------------
+// routing: router product with fp32 sums, sigmoid scores, corrected choice
+//
+// part[split][t][e] = sum over the K range of the split of x[t][k] w[e][k].  m16n8k16 MMAs whose fragments come straight from
+// global memory: inside an MMA the order of k is free, so lane (g, j) owns the 16 bytes k0 + 8 j .. + 7 of its rows, which
+// serve two MMA steps of a 32-wide slice of K.  WM warps of a CTA take 16 tokens each and share the weight rows (L1), WK
+// warps share the tokens and split K.  Grid (token tiles, K splits, tiles of 8 NT experts).
+// ------------------------------------------------------------------------------------------------
+__device__ __forceinline__ void mma_bf16(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+
+template <int NT, int WM, int WK>
+__global__ void __launch_bounds__(32 * WM * WK)
+moe_router_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __restrict__ w, int tokens, int E, int K,
+                  int k_split, float* __restrict__ part) {
+  tgi::pdl_wait();
+  tgi::pdl_trigger();
+  __shared__ float red[WK > 1 ? (WK - 1) * WM : 1][WK > 1 ? NT * 4 : 1][32];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, j = lane & 3;
+  const int wm = warp % WM, wk = warp / WM;
+  const int t0 = (blockIdx.x * WM + wm) * 16, e0 = blockIdx.z * 8 * NT;
+  const int k_end = min(K, (static_cast<int>(blockIdx.y) + 1) * k_split);
+  const uint4 zero = make_uint4(0, 0, 0, 0);
+  float c[NT][4];
+#pragma unroll
+  for (int n = 0; n < NT; ++n) c[n][0] = c[n][1] = c[n][2] = c[n][3] = 0.f;
+  const bool r0 = t0 + g < tokens, r1 = t0 + g + 8 < tokens;
+  const __nv_bfloat16* x0 = x + static_cast<size_t>(r0 ? t0 + g : 0) * K;
+  const __nv_bfloat16* x1 = x + static_cast<size_t>(r1 ? t0 + g + 8 : 0) * K;
+#pragma unroll 2
+  for (int k = blockIdx.y * k_split + wk * 32; k < k_end; k += 32 * WK) {
+    const int at = k + 8 * j;
+    const bool in = at < k_end;                            // K and the splits are multiples of 8
+    const uint4 a = in && r0 ? *reinterpret_cast<const uint4*>(x0 + at) : zero;
+    const uint4 b = in && r1 ? *reinterpret_cast<const uint4*>(x1 + at) : zero;
+#pragma unroll
+    for (int n = 0; n < NT; ++n) {
+      const int e = e0 + 8 * n + g;
+      const uint4 v = in && e < E ? *reinterpret_cast<const uint4*>(w + static_cast<size_t>(e) * K + at) : zero;
+      mma_bf16(c[n], a.x, b.x, a.y, b.y, v.x, v.y);
+      mma_bf16(c[n], a.z, b.z, a.w, b.w, v.z, v.w);
+    }
+  }
+  if (WK > 1) {
+    if (wk > 0) {
+#pragma unroll
+      for (int i = 0; i < NT * 4; ++i) red[(wk - 1) * WM + wm][i][lane] = c[i / 4][i % 4];
+    }
+    __syncthreads();
+    if (wk > 0) return;
+#pragma unroll
+    for (int i = 0; i < NT * 4; ++i)
+#pragma unroll
+      for (int o = 0; o < WK - 1; ++o) c[i / 4][i % 4] += red[o * WM + wm][i][lane];
+  }
+  float* out = part + static_cast<size_t>(blockIdx.y) * tokens * E;
+#pragma unroll
+  for (int n = 0; n < NT; ++n) {
+    const int e = e0 + 8 * n + 2 * j;
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+      if (e + (i & 1) < E && (i < 2 ? r0 : r1)) out[static_cast<size_t>(t0 + g + (i < 2 ? 0 : 8)) * E + e + (i & 1)] = c[n][i];
+  }
+}
+
+// logits = sum of `parts` matrices [tokens, E]; s = sigmoid(logits); the k experts with the largest s + correction (ties go
+// to the lower index), weight scale * s / (sum of their s + 1e-20)
+__global__ void __launch_bounds__(128)
+moe_topk_sigmoid_kernel(const float* __restrict__ part, int parts, const float* __restrict__ correction, int tokens, int E,
+                        int k, float scale, float* __restrict__ out_w, int* __restrict__ out_ids) {
+  tgi::pdl_wait();
+  tgi::pdl_trigger();
+  const int lane = threadIdx.x & 31;
+  const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (t >= tokens) return;
+  float s[kMaxExperts / 32], v[kMaxExperts / 32];
+#pragma unroll
+  for (int i = 0; i < kMaxExperts / 32; ++i) {
+    const int e = i * 32 + lane;
+    s[i] = 0.f;
+    v[i] = -INFINITY;                                      // not a candidate
+    if (e < E) {
+      float z = 0.f;
+      for (int p = 0; p < parts; ++p) z += part[(static_cast<size_t>(p) * tokens + t) * E + e];
+      s[i] = 1.f / (1.f + expf(-z));
+      v[i] = s[i] + (correction != nullptr ? correction[e] : 0.f);
+    }
+  }
+  float sum = 0.f, my_w = 0.f;
+  int my_id = 0;
+  for (int j = 0; j < k; ++j) {
+    float best = -INFINITY, score = 0.f;
+    int best_e = 0x7fffffff;
+#pragma unroll
+    for (int i = 0; i < kMaxExperts / 32; ++i)
+      if (v[i] > best) {
+        best = v[i];
+        best_e = i * 32 + lane;
+        score = s[i];
+      }
+#pragma unroll
+    for (int o = 16; o; o >>= 1) {
+      const float ob = __shfl_xor_sync(0xffffffffu, best, o), os = __shfl_xor_sync(0xffffffffu, score, o);
+      const int oe = __shfl_xor_sync(0xffffffffu, best_e, o);
+      if (ob > best || (ob == best && oe < best_e)) {
+        best = ob;
+        best_e = oe;
+        score = os;
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < kMaxExperts / 32; ++i)
+      if (i * 32 + lane == best_e) v[i] = -INFINITY;
+    sum += score;
+    if (lane == j) {
+      my_w = score;
+      my_id = min(best_e, E - 1);                          // a row of NaN has no largest score
+    }
+  }
+  if (lane < k) {
+    out_w[static_cast<size_t>(t) * k + lane] = my_w / (sum + 1e-20f) * scale;
+    out_ids[static_cast<size_t>(t) * k + lane] = my_id;
+  }
+}
+
+// ------------------------------------------------------------------------------------------------
 // grouping of the (token, slot) pairs by local expert.  One CTA; shared-memory counters.
 //   pos[entry]        position of the pair in the grouped order, -1 when its expert is not local
 //   order[position]   entry (token * k + slot) found at that position
@@ -175,19 +308,25 @@ moe_combine_kernel(const __nv_bfloat16* __restrict__ y, const int* __restrict__ 
     int p[kMaxTopK];
 #pragma unroll
     for (int j = 0; j < kMaxTopK; ++j) p[j] = j < k ? pos[static_cast<size_t>(t) * k + j] : -1;
+    auto add_row = [&](float (&acc)[8], int row, int i) {
+      const uint4 raw = reinterpret_cast<const uint4*>(y + static_cast<size_t>(row) * H)[i];
+      const __nv_bfloat162* h2 = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float2 f = __bfloat1622float2(h2[e]);
+        acc[2 * e] += f.x;
+        acc[2 * e + 1] += f.y;
+      }
+    };
     for (int i = threadIdx.x; i < vec; i += blockDim.x) {
       float acc[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
 #pragma unroll
       for (int j = 0; j < kMaxTopK; ++j) {
-        if (p[j] < 0) continue;
-        const uint4 raw = reinterpret_cast<const uint4*>(y + static_cast<size_t>(p[j]) * H)[i];
-        const __nv_bfloat162* h2 = reinterpret_cast<const __nv_bfloat162*>(&raw);
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const float2 f = __bfloat1622float2(h2[e]);
-          acc[2 * e] += f.x;
-          acc[2 * e + 1] += f.y;
-        }
+        if (p[j] >= 0) add_row(acc, p[j], i);
+      }
+      for (int j = kMaxTopK; j < k; ++j) {
+        const int row = pos[static_cast<size_t>(t) * k + j];
+        if (row >= 0) add_row(acc, row, i);
       }
       __nv_bfloat162 o[4];
 #pragma unroll
@@ -195,6 +334,22 @@ moe_combine_kernel(const __nv_bfloat16* __restrict__ y, const int* __restrict__ 
       reinterpret_cast<uint4*>(out + static_cast<size_t>(t) * H)[i] = *reinterpret_cast<uint4*>(o);
     }
   }
+}
+
+// the same for fp32 rows of any width and any number of slots
+__global__ void __launch_bounds__(256)
+moe_combine_f32_kernel(const float* __restrict__ y, const int* __restrict__ pos, int tokens, int k, int H, float* __restrict__ out) {
+  tgi::pdl_wait();
+  tgi::pdl_trigger();
+  for (int t = blockIdx.x; t < tokens; t += gridDim.x)
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+      float acc = 0.f;
+      for (int j = 0; j < k; ++j) {
+        const int p = pos[static_cast<size_t>(t) * k + j];
+        if (p >= 0) acc += y[static_cast<size_t>(p) * H + i];
+      }
+      out[static_cast<size_t>(t) * H + i] = acc;
+    }
 }
 
 // ------------------------------------------------------------------------------------------------
@@ -214,6 +369,8 @@ __device__ __forceinline__ float act_fn(float x, int act) {
       const float u = 0.7978845608028654f * (x + 0.044715f * x * x * x);
       return 0.5f * x * (1.f + tanhf(u));
     }
+    case 3: return fmaxf(x, 0.f);                                                       // relu
+    case 5: { const float y = fmaxf(x, 0.f); return y * y; }                            // squared relu
     default: return x / (1.f + __expf(-1.702f * x));                                    // quick gelu
   }
 }
@@ -240,6 +397,7 @@ struct TileWalk {
 // MODE 0: gate_up.  Weights [e_local, 2 * I, K]: gate rows then up rows; a tile takes 128 gate rows and the
 //         matching 128 up rows, the epilogue writes act(gate) * up to out[row, nt * 128 + j], out [rows, I].
 // MODE 1: down.  Weights [e_local, Nw, K]; the epilogue writes scale[row] * acc to out[row, nt * 256 + j].
+// MODE 2: up of an ungated expert.  Weights [e_local, Nw, K]; the epilogue writes act(acc) to out[row, nt * 256 + j].
 template <int MODE>
 __global__ void __launch_bounds__(kThreads, 1)
 moe_grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmW,
@@ -403,7 +561,7 @@ moe_grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_co
         }
       } else {
         const int col0 = nt * 256 + g * 128;
-        const float sc = row_ok ? topk_w[order[row]] : 0.f;   // routing weight of this (token, slot) pair
+        const float sc = MODE == 1 && row_ok ? topk_w[order[row]] : 0.f;   // routing weight of this (token, slot) pair
 #pragma unroll
         for (int c = 0; c < 128; c += 32) {
           uint32_t v[32];
@@ -416,8 +574,10 @@ moe_grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_co
               if (col0 + c + j >= out_cols) break;
               __nv_bfloat162 o[4];
 #pragma unroll
-              for (int q = 0; q < 4; ++q)
-                o[q] = __floats2bfloat162_rn(__uint_as_float(v[j + 2 * q]) * sc, __uint_as_float(v[j + 2 * q + 1]) * sc);
+              for (int q = 0; q < 4; ++q) {
+                const float a0 = __uint_as_float(v[j + 2 * q]), a1 = __uint_as_float(v[j + 2 * q + 1]);
+                o[q] = MODE == 2 ? __floats2bfloat162_rn(act_fn(a0, act), act_fn(a1, act)) : __floats2bfloat162_rn(a0 * sc, a1 * sc);
+              }
               *reinterpret_cast<uint4*>(dst + j) = *reinterpret_cast<uint4*>(o);
             }
           }
@@ -460,6 +620,71 @@ int launch_grouped(const void* A, int rows_cap, const void* W, int e_local, int 
   return err == cudaSuccess && cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
 
+// ------------------------------------------------------------------------------------------------
+// fp32 products of ungated experts: 64 x 64 tiles, 256 threads with 4 x 4 sums each.  MODE 2: A rows are the tokens
+// order[row] / k of x, out = act(A W^T); MODE 1: A rows are grouped, out = topk_w[order[row]] * (A W^T).
+// grid (weight tiles, row tiles an expert layout can have)
+// ------------------------------------------------------------------------------------------------
+template <int MODE>
+__global__ void __launch_bounds__(256)
+moe_grouped_f32_kernel(const float* __restrict__ A, const float* __restrict__ W, const int* __restrict__ offsets,
+                       const int* __restrict__ order, int e_local, int k, int Nw, int K, int act,
+                       const float* __restrict__ topk_w, float* __restrict__ out) {
+  tgi::pdl_wait();
+  tgi::pdl_trigger();
+  __shared__ float sa[16][68], sw[16][68];
+  int tile = blockIdx.y, e = 0;
+  while (e < e_local && tile >= (offsets[e + 1] - offsets[e] + 63) / 64) {
+    tile -= (offsets[e + 1] - offsets[e] + 63) / 64;
+    ++e;
+  }
+  if (e == e_local) return;                                // block-uniform
+  const int row0 = offsets[e] + tile * 64, rows = min(64, offsets[e + 1] - row0), n0 = blockIdx.x * 64;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < K; k0 += 16) {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int r = ty + 16 * i, kk = k0 + tx;
+      float a = 0.f, w = 0.f;
+      if (kk < K && r < rows) {
+        const int row = row0 + r;
+        a = A[static_cast<size_t>(MODE == 2 ? order[row] / k : row) * K + kk];
+      }
+      if (kk < K && n0 + r < Nw) w = W[(static_cast<size_t>(e) * Nw + n0 + r) * K + kk];
+      sa[tx][r] = a;
+      sw[tx][r] = w;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int q = 0; q < 16; ++q) {
+      float a[4], w[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        a[i] = sa[q][4 * ty + i];
+        w[i] = sw[q][4 * tx + i];
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(a[i], w[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int r = 4 * ty + i;
+    if (r >= rows) continue;
+    const int row = row0 + r;
+    const float sc = MODE == 1 ? topk_w[order[row]] : 1.f;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int n = n0 + 4 * tx + j;
+      if (n < Nw) out[static_cast<size_t>(row) * Nw + n] = MODE == 2 ? act_fn(acc[i][j], act) : acc[i][j] * sc;
+    }
+  }
+}
+
 }  // namespace
 
 extern "C" {
@@ -477,6 +702,61 @@ int tgi_moe_topk_softmax(const void* logits, int is_f32, int tokens, int E, int 
   else
     err = tgi::launch(moe_topk_softmax_kernel<__nv_bfloat16>, grid, block, 0, stream,
                       static_cast<const __nv_bfloat16*>(logits), tokens, E, k, renorm, out_w, out_ids);
+  return err == cudaSuccess && cudaGetLastError() == cudaSuccess ? 0 : -3;
+}
+
+// K range and number of the splits of the router product.
+int tgi_moe_router_splits(int tokens, int E, int K, int sm_count) {
+  const int tiles = (tokens + (tokens > 512 ? 63 : 15)) / (tokens > 512 ? 64 : 16) * ((E + 63) / 64);
+  int want = (3 * sm_count + tiles - 1) / tiles;           // a few CTAs per SM: the loads are not staged
+  const int most = (K + 255) / 256;
+  if (want > most) want = most;
+  if (want > 16) want = 16;
+  return want < 1 ? 1 : want;
+}
+
+// x [tokens, K], w [E, K] bf16 -> part fp32 [splits, tokens, E]; K % 8 == 0
+int tgi_moe_router(const void* x, const void* w, int tokens, int E, int K, int splits, float* part, cudaStream_t stream) {
+  if (tokens <= 0) return 0;
+  if (E < 1 || K < 8 || K % 8 != 0 || splits < 1) return -30;
+  const int k_split = ((K + splits - 1) / splits + 31) / 32 * 32;
+  const auto* xb = static_cast<const __nv_bfloat16*>(x);
+  const auto* wb = static_cast<const __nv_bfloat16*>(w);
+  auto go = [&](auto kern, int rows, int nt, int threads) {
+    return tgi::launch(kern, dim3((tokens + rows - 1) / rows, splits, (E + 8 * nt - 1) / (8 * nt)), dim3(threads), 0, stream, xb,
+                       wb, tokens, E, K, k_split, part);
+  };
+  cudaError_t err;
+  if (tokens > 512) err = E <= 32 ? go(moe_router_kernel<4, 4, 1>, 64, 4, 128) : go(moe_router_kernel<8, 4, 1>, 64, 8, 128);
+  else err = E <= 32 ? go(moe_router_kernel<4, 1, 4>, 16, 4, 128) : go(moe_router_kernel<8, 1, 4>, 16, 8, 128);
+  return err == cudaSuccess && cudaGetLastError() == cudaSuccess ? 0 : -3;
+}
+
+int tgi_moe_topk_sigmoid(const float* part, int parts, const float* correction, int tokens, int E, int k, float scale,
+                         float* out_w, int* out_ids, cudaStream_t stream) {
+  if (tokens <= 0) return 0;
+  if (E < 1 || E > kMaxExperts || k < 1 || k > kMaxTopKSigmoid || k > E || parts < 1) return -30;
+  const cudaError_t err = tgi::launch(moe_topk_sigmoid_kernel, dim3((tokens + 3) / 4), dim3(128), 0, stream, part, parts,
+                                      correction, tokens, E, k, scale, out_w, out_ids);
+  return err == cudaSuccess && cudaGetLastError() == cudaSuccess ? 0 : -3;
+}
+
+// mode 2: out[entries, Nw] = act(x[order / k] W^T), mode 1: out[entries, Nw] = topk_w[order] * (A W^T); all fp32
+int tgi_moe_grouped_f32(int mode, const float* A, int entries, const float* W, int e_local, int k, int Nw, int K,
+                        const int* offsets, const int* order, int act, const float* topk_w, float* out, cudaStream_t stream) {
+  if (entries <= 0) return 0;
+  if (e_local < 1 || e_local > kMaxExperts || k < 1) return -30;
+  const dim3 grid((Nw + 63) / 64, entries / 64 + e_local);  // every expert may leave one tile partly filled
+  const cudaError_t err =
+      mode == 2 ? tgi::launch(moe_grouped_f32_kernel<2>, grid, dim3(256), 0, stream, A, W, offsets, order, e_local, k, Nw, K, act, topk_w, out)
+                : tgi::launch(moe_grouped_f32_kernel<1>, grid, dim3(256), 0, stream, A, W, offsets, order, e_local, k, Nw, K, act, topk_w, out);
+  return err == cudaSuccess && cudaGetLastError() == cudaSuccess ? 0 : -3;
+}
+
+int tgi_moe_combine_f32(const float* y, const int* pos, int tokens, int k, int H, float* out, cudaStream_t stream) {
+  if (tokens <= 0) return 0;
+  const cudaError_t err = tgi::launch(moe_combine_f32_kernel, dim3(tokens < 4096 ? tokens : 4096), dim3(256), 0, stream, y, pos,
+                                      tokens, k, H, out);
   return err == cudaSuccess && cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
 
@@ -500,7 +780,8 @@ int tgi_moe_gather(const void* x, const int* order, const int* offsets, int e_lo
   return err == cudaSuccess && cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
 
-// mode 0: out[rows_cap, Nw / 2] = act(A Wg^T) * (A Wu^T); mode 1: out[rows_cap, Nw] = w[row] * (A W^T).
+// mode 0: out[rows_cap, Nw / 2] = act(A Wg^T) * (A Wu^T); mode 1: out[rows_cap, Nw] = w[row] * (A W^T); mode 2:
+// out[rows_cap, Nw] = act(A W^T).
 // A [rows_cap, K] bf16 grouped by expert, W [e_local, Nw, K] bf16, offsets [e_local + 1] on the device.
 int tgi_moe_grouped_gemm(int mode, const void* A, int rows_cap, const void* W, int e_local, int Nw, int K,
                          const int* offsets, int act, const float* topk_w, const int* order, void* out, int ctas,
@@ -512,12 +793,14 @@ int tgi_moe_grouped_gemm(int mode, const void* A, int rows_cap, const void* W, i
     return launch_grouped<0>(A, rows_cap, W, e_local, Nw, K, offsets, act, topk_w, order, out, Nw / 2, ctas, status, stream);
   }
   if (Nw % 8 != 0) return -31;
+  if (mode == 2)
+    return launch_grouped<2>(A, rows_cap, W, e_local, Nw, K, offsets, act, topk_w, order, out, Nw, ctas, status, stream);
   return launch_grouped<1>(A, rows_cap, W, e_local, Nw, K, offsets, act, topk_w, order, out, Nw, ctas, status, stream);
 }
 
 int tgi_moe_combine(const void* y, const int* pos, int tokens, int k, int H, void* out, cudaStream_t stream) {
   if (tokens <= 0) return 0;
-  if (H % 8 != 0 || k > kMaxTopK) return -31;
+  if (H % 8 != 0) return -31;
   const int grid = tokens < 4096 ? tokens : 4096;
   const cudaError_t err = tgi::launch(moe_combine_kernel, dim3(grid), dim3(256), 0, stream,
                                       static_cast<const __nv_bfloat16*>(y), pos, tokens, k, H,

@@ -1,6 +1,7 @@
 // Recurrent token mixers with a matrix state per head, S[dim x vdim] in fp32:
 //
 //   gated delta rule, one decay per key channel      S <- g * S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
+//   the same with one decay per head                 (g a scalar)
 //   linear attention with a fixed decay per head     S <- d S + k v^T;                                    o = S^T q
 //
 // The columns of S never meet: column j of a head needs k, q, g of the head and only v_j of its own.
@@ -13,7 +14,8 @@
 //   S  <- G_3 S + sum_j (D_j3 k_j) u_j^T
 // which is the token-by-token rule with all products on the old state: they are independent, one reduction latency is
 // paid per block, and the scalars are shared by all columns.  Only products of decays appear, never quotients, so a
-// channel that forgets within a token loses nothing.  (Fixed decay: u = v, D and G are powers of d.)
+// channel that forgets within a token loses nothing.  (One decay per head: G and D are scalars, taken out of the products,
+// so that k and q are staged as they are.  Fixed decay: u = v, D and G are powers of d.)
 // L lanes share CN columns, lane l holding rows 4 (l + L j) + (0..3) of each: a 16-byte shared-memory read feeds 4 CN
 // multiply-adds, done in pairs (fma.rn.f32x2).  The sums of the CN columns are reduced by halving exchanges, after which
 // every lane owns one column.  The vectors and scalars of the next tile of kTile tokens are prepared from registers
@@ -34,6 +36,7 @@ namespace {
 
 using bf16 = __nv_bfloat16;
 constexpr int kTile = 8;          // tokens per staged tile
+enum { kFixed = 0, kChannel = 1, kHead = 2 };       // fixed decay, delta rule with a decay per channel, per head
 constexpr int kThreads = 128;
 
 __device__ __forceinline__ float to_f(float x) { return x; }
@@ -45,7 +48,7 @@ template <>
 __device__ __forceinline__ float silu_t<bf16>(float x) { return __fdividef(x, 1.f + __expf(-x)); }
 
 struct ScanArgs {
-  // delta rule: fp32 q, k [T, G, dimP], g [T, H, dimP], v [T, H, vdim], beta [T, H], qk = q . k [T, G]
+  // delta rule: fp32 q, k [T, G, dimP], g [T, H, dimP] (one decay per head: [T, H]), v [T, H, vdim], beta [T, H], qk = q . k [T, G]
   const float *q, *k, *g, *v, *beta, *qk;
   // linear attention: proj [T, ld] with q, k (H x dim) and v (H x vdim) at off_q, off_k, off_v (SiLU applied here)
   const void* proj;
@@ -151,28 +154,33 @@ __device__ __forceinline__ float4 mul4(float4 a, float4 b) { return make_float4(
 
 constexpr int kBlock = 4;         // tokens whose products with the state are formed together
 
+// (first, last) token of the 16 scalars of a block, a nibble each: ten with queries, six with keys
+constexpr unsigned long long kPairFirst = 0x2110003221110000ull, kPairLast = 0x3323213323213210ull;
+
 // L lanes share CN columns of a head whose vectors are 64 J wide
-template <bool DELTA, int J, int L, int CN>
+template <int MODE, int J, int L, int CN>
 struct ScanCfg {
   static constexpr int kRow = 64 * J;
   static constexpr int kQuads = 16 * J / L;                     // 16-byte pieces of a column per lane
   static constexpr int kCols = kThreads / L * CN;               // columns of a CTA
-  static constexpr int kRows = DELTA ? 13 : 8;                  // vectors of a block: q', k^ (x 4 each) | + k' (x 4), decay
-  static constexpr int kQ = 0, kEnd = 4, kK = DELTA ? 8 : 0, kG = DELTA ? 12 : 0;      // first row of each kind
+  static constexpr bool kWide = MODE == kChannel;
+  static constexpr int kRows = kWide ? 13 : 8;                  // vectors of a block: q', k^ (x 4 each) | + k' (x 4), decay
+  static constexpr int kQ = 0, kEnd = 4, kK = kWide ? 8 : 4, kG = kWide ? 12 : 0;      // first row of each kind
   static constexpr int kVecs = 2 * kRows * kRow;                // floats: two blocks per tile
-  static constexpr int kOffV = kVecs, kOffBeta = kOffV + kTile * kCols, kOffScal = kOffBeta + kTile,
-                       kOffPart = kOffScal + 32, kStage = kOffPart + 2 * J * 16;
+  static constexpr int kOffV = kVecs, kOffBeta = kOffV + kTile * kCols, kOffGate = kOffBeta + kTile,
+                       kOffScal = kOffGate + kTile, kOffPart = kOffScal + 32, kStage = kOffPart + 2 * J * 16;
   static constexpr int kBytes = 2 * kStage * 4;
 };
 
 // grid (ceil(vdim / kCols), H, B), 128 threads.  VEC: the heads of proj may be read in aligned pairs.
-template <typename T, bool DELTA, bool VEC, int J, int L, int CN>
+template <typename T, int MODE, bool VEC, int J, int L, int CN>
 __global__ void __launch_bounds__(kThreads)
 scan_kernel(ScanArgs p) {
+  constexpr bool DELTA = MODE != kFixed, WIDE = MODE == kChannel, HEAD = MODE == kHead;
   tgi::pdl_wait();
   tgi::pdl_trigger();
   extern __shared__ __align__(16) float smem[];
-  using S = ScanCfg<DELTA, J, L, CN>;
+  using S = ScanCfg<MODE, J, L, CN>;
   constexpr int kItems = 64 * J;                                // (block, channel pair) items of a tile
   constexpr int NI = (kItems + kThreads - 1) / kThreads;
   constexpr int NV = kTile * S::kCols / kThreads;
@@ -206,9 +214,9 @@ scan_kernel(ScanArgs p) {
 
   // two channels of the four tokens of a block, as they come from memory; pointers advance by a tile
   using E2 = typename PairOf<T>::type;
-  float2 rk[NI][kBlock], rq[NI][kBlock], rg[DELTA ? NI : 1][kBlock];
+  float2 rk[NI][kBlock], rq[NI][kBlock], rg[WIDE ? NI : 1][kBlock];
   T rv[DELTA ? 1 : NV];
-  float rvf[DELTA ? NV : 1], rb = 0.f;
+  float rvf[DELTA ? NV : 1], rb = 0.f, rh = 1.f;
   const size_t sk = DELTA ? static_cast<size_t>(p.G) * p.dimP : static_cast<size_t>(p.ld);   // token pitch of q and k
   const size_t sg = static_cast<size_t>(p.H) * p.dimP, sv = static_cast<size_t>(p.H) * p.vdim;
   const T* const proj = static_cast<const T*>(p.proj);
@@ -228,11 +236,11 @@ scan_kernel(ScanArgs p) {
         const bool ok = in && tb + e < n;
         if (DELTA) {
           rk[i][e] = rq[i][e] = make_float2(0.f, 0.f);
-          rg[DELTA ? i : 0][e] = make_float2(1.f, 1.f);
+          if (WIDE) rg[WIDE ? i : 0][e] = make_float2(1.f, 1.f);
           if (ok) {
             rk[i][e] = *reinterpret_cast<const float2*>(fk + e * sk);
             rq[i][e] = *reinterpret_cast<const float2*>(fq + e * sk);
-            rg[DELTA ? i : 0][e] = *reinterpret_cast<const float2*>(fg + e * sg);
+            if (WIDE) rg[WIDE ? i : 0][e] = *reinterpret_cast<const float2*>(fg + e * sg);
           }
         } else if (VEC) {
           E2 a = E2(), c = E2();
@@ -264,6 +272,7 @@ scan_kernel(ScanArgs p) {
       }
     }
     if (DELTA && tid < kTile) rb = t0 + tid < n ? p.beta[static_cast<size_t>(begin + t0 + tid) * p.H + h] : 0.f;
+    if (HEAD && tid < kTile) rh = t0 + tid < n ? p.g[static_cast<size_t>(begin + t0 + tid) * p.H + h] : 1.f;
   };
   // vectors and partial scalar products of the fetched tile (tokens t0 ..) -> shared memory
   auto stage = [&](float* d, int t0) {
@@ -277,8 +286,10 @@ scan_kernel(ScanArgs p) {
       for (int e = 0; e < kBlock; ++e) {
         k[e] = rk[i][e];
         q[e] = rq[i][e];
-        if (DELTA) {
-          g[e] = rg[DELTA ? i : 0][e];
+        if (WIDE) {
+          g[e] = rg[WIDE ? i : 0][e];
+        } else if (HEAD) {
+          g[e] = make_float2(1.f, 1.f);                         // decays are applied to the sums
         } else {
           if (VEC) {
             k[e] = PairOf<T>::value(k[e]);
@@ -305,9 +316,9 @@ scan_kernel(ScanArgs p) {
       for (int e = 0; e < kBlock; ++e) {
         row(S::kQ + e, mul(to[e], q[e]));
         row(S::kEnd + e, mul(from[e], k[e]));
-        if (DELTA) row(S::kK + e, mul(to[e], k[e]));
+        if (WIDE) row(S::kK + e, mul(to[e], k[e]));
       }
-      if (DELTA) row(S::kG, to[kBlock - 1]);
+      if (WIDE) row(S::kG, to[kBlock - 1]);
       // token a's key, decayed to token e, times e's query (10 sums over channels) and e's key (6 sums)
       float sc[16];
       int at = 0;
@@ -339,6 +350,7 @@ scan_kernel(ScanArgs p) {
     for (int i = 0; i < NV; ++i)
       d[S::kOffV + tid + i * kThreads] = DELTA ? rvf[DELTA ? i : 0] : silu_t<T>(to_f(rv[DELTA ? 0 : i]));
     if (DELTA && tid < kTile) d[S::kOffBeta + tid] = rb;
+    if (HEAD && tid < kTile) d[S::kOffGate + tid] = rh;
   };
   // the sums of the warps that shared a block
   auto finish = [&](float* d) {
@@ -346,6 +358,12 @@ scan_kernel(ScanArgs p) {
       float x = 0.f;
 #pragma unroll
       for (int j = 0; j < J; ++j) x += d[S::kOffPart + ((tid >> 4) * J + j) * 16 + (tid & 15)];
+      if (HEAD) {                                               // decay after the first token of the pair up to the last
+        const int first = kPairFirst >> (4 * (tid & 15)) & 15, last = kPairLast >> (4 * (tid & 15)) & 15;
+#pragma unroll
+        for (int e = 1; e < kBlock; ++e)
+          if (e > first && e <= last) x *= d[S::kOffGate + (tid >> 4) * kBlock + e];
+      }
       d[S::kOffScal + tid] = x;
     }
   };
@@ -363,7 +381,15 @@ scan_kernel(ScanArgs p) {
     for (int blk = 0; blk < 2 && t0 + blk * kBlock < n; ++blk) {
       const float* r = d + blk * S::kRows * S::kRow + 4 * l;
       const float* vt = d + S::kOffV + blk * kBlock * S::kCols + col;
-      float w[kBlock], u[kBlock];
+      float w[kBlock], u[kBlock], since[kBlock];                // decay of the head since the start of the block
+      float4 gate = make_float4(1.f, 1.f, 1.f, 1.f);
+      if (HEAD) {
+        gate = *reinterpret_cast<const float4*>(d + S::kOffGate + blk * kBlock);
+        since[0] = gate.x;
+        since[1] = since[0] * gate.y;
+        since[2] = since[1] * gate.z;
+        since[3] = since[2] * gate.w;
+      }
       // products of every token of the block with the state before it
 #pragma unroll
       for (int e = 0; e < kBlock; ++e) {
@@ -380,7 +406,8 @@ scan_kernel(ScanArgs p) {
           }
 #pragma unroll
           for (int c = 0; c < CN; ++c) a[c] = pair_sum(x2[c]);
-          u[e] -= scatter_sum<CN, L>(a, l);
+          const float r0 = scatter_sum<CN, L>(a, l);
+          u[e] = HEAD ? fmaf(-since[e], r0, u[e]) : u[e] - r0;
         }
 #pragma unroll
         for (int j = 0; j < NQ; ++j) {
@@ -392,6 +419,7 @@ scan_kernel(ScanArgs p) {
 #pragma unroll
         for (int c = 0; c < CN; ++c) a[c] = pair_sum(x2[c]);
         w[e] = scatter_sum<CN, L>(a, l);
+        if (HEAD) w[e] *= since[e];
       }
       // what the tokens write, first to last, and what they read of each other
       const float4* sc = reinterpret_cast<const float4*>(d + S::kOffScal + blk * 16);
@@ -410,7 +438,7 @@ scan_kernel(ScanArgs p) {
       w[3] = fmaf(s0.w, u[0], fmaf(s1.z, u[1], fmaf(s2.x, u[2], fmaf(s2.y, u[3], w[3]))));
       // the state after the block
       const int cnt = min(kBlock, n - t0 - blk * kBlock);
-      if (DELTA) {
+      if (WIDE) {
 #pragma unroll
         for (int j = 0; j < NQ; ++j) {
           const ulonglong2 g = *reinterpret_cast<const ulonglong2*>(r + S::kG * S::kRow + 4 * L * j);
@@ -422,7 +450,7 @@ scan_kernel(ScanArgs p) {
         }
       } else {
         const float d2 = dec * dec;
-        const float f = cnt == 4 ? d2 * d2 : (cnt == 3 ? d2 * dec : (cnt == 2 ? d2 : dec));
+        const float f = HEAD ? since[3] : (cnt == 4 ? d2 * d2 : (cnt == 3 ? d2 * dec : (cnt == 2 ? d2 : dec)));
         const pair f2 = pk(f, f);
 #pragma unroll
         for (int j = 0; j < NQ; ++j) {
@@ -432,6 +460,11 @@ scan_kernel(ScanArgs p) {
             s[c][j][1] = mul2(f2, s[c][j][1]);
           }
         }
+      }
+      if (HEAD) {                                               // what is left of each write at the end of the block
+        u[2] *= gate.w;
+        u[1] *= gate.z * gate.w;
+        u[0] *= gate.y * gate.z * gate.w;
       }
 #pragma unroll
       for (int e = 0; e < kBlock; ++e) {
@@ -482,9 +515,10 @@ scan_kernel(ScanArgs p) {
 }
 
 // one token per sequence.  grid (ceil(vdim / (16 CN)), H, B), 128 threads: CN columns per thread
-template <typename T, bool DELTA, int J, int CN>
+template <typename T, int MODE, int J, int CN>
 __global__ void __launch_bounds__(kThreads)
 step_kernel(ScanArgs p) {
+  constexpr bool DELTA = MODE != kFixed, HEAD = MODE == kHead;
   tgi::pdl_wait();
   tgi::pdl_trigger();
   const int b = blockIdx.z, h = blockIdx.y;
@@ -511,6 +545,7 @@ step_kernel(ScanArgs p) {
     const float* kp = p.k + (static_cast<size_t>(t) * p.G + hg) * p.dimP + 4 * l;
     const float* qp = p.q + (static_cast<size_t>(t) * p.G + hg) * p.dimP + 4 * l;
     const float* gp = p.g + (static_cast<size_t>(t) * p.H + h) * p.dimP + 4 * l;
+    const float gh = HEAD ? p.g[static_cast<size_t>(t) * p.H + h] : 1.f;
     const float beta = p.beta[static_cast<size_t>(t) * p.H + h], kq = p.qk[static_cast<size_t>(t) * p.G + hg];
     float a[CN];
 #pragma unroll
@@ -522,7 +557,7 @@ step_kernel(ScanArgs p) {
     for (int j = 0; j < J; ++j) {
       k[j] = *reinterpret_cast<const float4*>(kp + 32 * j);
       q[j] = *reinterpret_cast<const float4*>(qp + 32 * j);
-      const float4 g = *reinterpret_cast<const float4*>(gp + 32 * j);
+      const float4 g = HEAD ? make_float4(gh, gh, gh, gh) : *reinterpret_cast<const float4*>(gp + 32 * j);
 #pragma unroll
       for (int c = 0; c < CN; ++c) {
         const float4 x = s[c][j] = mul4(g, s[c][j]);
@@ -586,10 +621,10 @@ step_kernel(ScanArgs p) {
   }
 }
 
-template <typename T, bool DELTA, bool VEC, int J, int L, int CN>
+template <typename T, int MODE, bool VEC, int J, int L, int CN>
 int launch_scan(const ScanArgs& p, int B, cudaStream_t stream) {
-  using S = ScanCfg<DELTA, J, L, CN>;
-  auto kern = scan_kernel<T, DELTA, VEC, J, L, CN>;
+  using S = ScanCfg<MODE, J, L, CN>;
+  auto kern = scan_kernel<T, MODE, VEC, J, L, CN>;
   if (S::kBytes > 48 * 1024 &&
       cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, S::kBytes) != cudaSuccess)
     return -2;
@@ -597,11 +632,12 @@ int launch_scan(const ScanArgs& p, int B, cudaStream_t stream) {
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
 
-template <typename T, bool DELTA, int J>
+template <typename T, int MODE, int J>
 int run(const ScanArgs& p, int B, int max_q, cudaStream_t stream) {
+  constexpr bool DELTA = MODE != kFixed;
   if (max_q == 1) {
     constexpr int CN = J <= 4 ? 4 : 2;
-    tgi::launch(step_kernel<T, DELTA, J, CN>, dim3((p.vdim + 16 * CN - 1) / (16 * CN), p.H, B), dim3(kThreads), 0, stream, p);
+    tgi::launch(step_kernel<T, MODE, J, CN>, dim3((p.vdim + 16 * CN - 1) / (16 * CN), p.H, B), dim3(kThreads), 0, stream, p);
   } else {
     // Wide lanes and few columns keep every scheduler busy when there are few sequences; many columns per lane need
     // fewer shared-memory reads and shuffles per column.  Measured, 32 heads of 128 x 128, delta rule, us (16 lanes x 4
@@ -611,27 +647,27 @@ int run(const ScanArgs& p, int B, int max_q, cudaStream_t stream) {
     if (DELTA || p.vec) {
       if constexpr (JS <= 2) {
         const long long heads = static_cast<long long>(B) * p.H;
-        if (heads * ((p.vdim + 127) / 128) >= (DELTA ? 128 : 192)) return launch_scan<T, DELTA, true, JS, 4, 4>(p, B, stream);
-        if (heads * ((p.vdim + 63) / 64) >= 128) return launch_scan<T, DELTA, true, JS, 16, 8>(p, B, stream);
+        if (heads * ((p.vdim + 127) / 128) >= (DELTA ? 128 : 192)) return launch_scan<T, MODE, true, JS, 4, 4>(p, B, stream);
+        if (heads * ((p.vdim + 63) / 64) >= 128) return launch_scan<T, MODE, true, JS, 16, 8>(p, B, stream);
       }
-      return launch_scan<T, DELTA, true, JS, 16, 4>(p, B, stream);
+      return launch_scan<T, MODE, true, JS, 16, 4>(p, B, stream);
     }
-    if constexpr (!DELTA) return launch_scan<T, DELTA, false, JS, 16, 4>(p, B, stream);
+    if constexpr (!DELTA) return launch_scan<T, MODE, false, JS, 16, 4>(p, B, stream);
   }
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
 
-template <typename T, bool DELTA>
+template <typename T, int MODE>
 int dispatch(const ScanArgs& p, int B, int max_q, cudaStream_t stream) {
   if (B <= 0 || max_q <= 0) return 0;
   if (B > 65535 || p.H > 65535 || p.H % p.G != 0 || p.dimP % 32 != 0 || p.dimP < p.dim) return -10;
   switch (p.dimP / 32) {
-    case 1: return run<T, DELTA, 1>(p, B, max_q, stream);
-    case 2: return run<T, DELTA, 2>(p, B, max_q, stream);
-    case 3: return run<T, DELTA, 3>(p, B, max_q, stream);
-    case 4: return run<T, DELTA, 4>(p, B, max_q, stream);
-    case 5: case 6: return p.dimP == 192 ? run<T, DELTA, 6>(p, B, max_q, stream) : -12;
-    case 8: return run<T, DELTA, 8>(p, B, max_q, stream);
+    case 1: return run<T, MODE, 1>(p, B, max_q, stream);
+    case 2: return run<T, MODE, 2>(p, B, max_q, stream);
+    case 3: return run<T, MODE, 3>(p, B, max_q, stream);
+    case 4: return run<T, MODE, 4>(p, B, max_q, stream);
+    case 5: case 6: return p.dimP == 192 ? run<T, MODE, 6>(p, B, max_q, stream) : -12;
+    case 8: return run<T, MODE, 8>(p, B, max_q, stream);
     default: return -12;
   }
 }
@@ -647,15 +683,16 @@ int tgi_recurrent_pitch(int dim) {
   return 0;
 }
 
+// `head_decay`: g is [T, H] instead of [T, H, dimP]
 int tgi_delta_scan(const float* q, const float* k, const float* g, const float* v, const float* beta, const float* qk,
                    const int* cu, const int* kv_lens, const int* state_slots, float* state, float* out, int B, int max_q,
-                   int num_slots, int G, int H, int dim, int dimP, int vdim, cudaStream_t stream) {
+                   int num_slots, int G, int H, int dim, int dimP, int vdim, int head_decay, cudaStream_t stream) {
   ScanArgs p{};
   p.q = q; p.k = k; p.g = g; p.v = v; p.beta = beta; p.qk = qk;
   p.cu = cu; p.kv_lens = kv_lens; p.state_slots = state_slots;
   p.state = state; p.out = out;
   p.num_slots = num_slots; p.G = G; p.H = H; p.dim = dim; p.dimP = dimP; p.vdim = vdim;
-  return dispatch<float, true>(p, B, max_q, stream);
+  return head_decay ? dispatch<float, kHead>(p, B, max_q, stream) : dispatch<float, kChannel>(p, B, max_q, stream);
 }
 
 int tgi_decay_scan(int f32, const void* proj, long long ld, int off_q, int off_k, int off_v, const float* decay, const int* cu,
@@ -668,7 +705,7 @@ int tgi_decay_scan(int f32, const void* proj, long long ld, int off_q, int off_k
   p.num_slots = num_slots; p.G = H; p.H = H; p.dim = dim; p.dimP = dimP; p.vdim = vdim;
   p.vec = dim % 4 == 0 && ld % 4 == 0 && off_q % 4 == 0 && off_k % 4 == 0 &&
           reinterpret_cast<uintptr_t>(proj) % (f32 ? 16 : 8) == 0;
-  return f32 ? dispatch<float, false>(p, B, max_q, stream) : dispatch<bf16, false>(p, B, max_q, stream);
+  return f32 ? dispatch<float, kFixed>(p, B, max_q, stream) : dispatch<bf16, kFixed>(p, B, max_q, stream);
 }
 
 }  // extern "C"

@@ -20,7 +20,7 @@ _LIB_PATH = Path(__file__).resolve().parent / "libtgi_b200_kernels.so"
 FP8 = torch.float8_e4m3fn
 
 _ACT_CODES = {"silu": 0, "swish": 0, "gelu": 1, "gelu_python": 1, "gelu_new": 2, "gelu_fast": 2,
-              "gelu_pytorch_tanh": 2, "gelu_tanh": 2, "relu": 3, "quick_gelu": 4}
+              "gelu_pytorch_tanh": 2, "gelu_tanh": 2, "relu": 3, "quick_gelu": 4, "relu2": 5}
 
 c_void_p, c_int, c_float, c_ll = ctypes.c_void_p, ctypes.c_int, ctypes.c_float, ctypes.c_longlong
 
@@ -65,7 +65,8 @@ def load():
                  "tgi_moe_combine", "tgi_gemm_last_grid", "tgi_penalties", "tgi_gemm_wq", "tgi_wq_dequant", "tgi_qk_norm",
                  "tgi_quant_set_pow2", "tgi_peer_set_quant_pow2", "tgi_gemm_bf16_ld", "tgi_residual_norm", "tgi_embed_residual",
                  "tgi_activation", "tgi_attn_prep", "tgi_attn_any", "tgi_delta_prep", "tgi_delta_scan", "tgi_decay_scan",
-                 "tgi_gated_norm", "tgi_recurrent_pitch", "tgi_delta_tap_rows"):
+                 "tgi_gated_norm", "tgi_recurrent_pitch", "tgi_delta_tap_rows", "tgi_act_mul_any", "tgi_moe_router",
+                 "tgi_moe_router_splits", "tgi_moe_topk_sigmoid", "tgi_moe_grouped_f32", "tgi_moe_combine_f32"):
         if hasattr(_LIB, name):        # a library built for one family of models lacks the other families' kernels
             getattr(_LIB, name).restype = c_int
     _LIB.tgi_gemm_workspace_floats.restype = c_ll
@@ -352,6 +353,10 @@ def act_and_mul(gate_up, act="silu"):
     T, I2 = gate_up.shape
     I = I2 // 2
     out = torch.empty(T, I, dtype=gate_up.dtype, device=gate_up.device)
+    if gate_up.dtype == torch.float32 or I % 8 != 0:
+        _check(lib.tgi_act_mul_any(_f32(gate_up), _ptr(gate_up.contiguous()), _ptr(out), c_int(T), c_int(I),
+                                   c_int(_ACT_CODES[act]), _stream()), "act_and_mul")
+        return out
     _check(lib.tgi_act_mul(_ptr(gate_up.contiguous()), _ptr(out), c_void_p(0), c_void_p(0), c_int(0), c_int(T),
                            c_int(I), c_int(_ACT_CODES[act]), _stream()), "act_and_mul")
     return out
@@ -437,8 +442,9 @@ def paged_attention(q, k_cache, v_cache, block_tables, cu_seqlens_q, kv_lens, sc
         max_q = int((cu_seqlens_q[1:] - cu_seqlens_q[:-1]).max().item())
     if max_kv is None:
         max_kv = int(kv_lens.max().item())
-    if chunk > 0:
-        max_kv = min(max_kv, chunk)      # keys a row can see: decides how far a decode step is split
+    for span in (chunk, window or 0):
+        if span > 0:
+            max_kv = min(max_kv, span)   # keys a row can see: decides how far a decode step is split
     fp8 = k_cache.dtype == FP8
     st = state(q.device)
     part_o = part_ml = None
@@ -477,20 +483,24 @@ def embed_residual(ids, table, scale: float):
     return out
 
 
-def residual_norm(delta, residual, weight, eps, rows=None, keep: bool = True):
+def residual_norm(delta, residual, weight, eps, rows=None, keep: bool = True, scale: float = 1.0, unit_offset: bool = False,
+                  weight2=None):
     H = residual.shape[1]
     n = residual.shape[0] if rows is None else rows.shape[0]
-    out = torch.empty(n, H, dtype=weight.dtype, device=residual.device)
-    if delta is None and rows is None:
+    d1, d2 = delta if isinstance(delta, tuple) else (delta, None)
+    new = lambda: torch.empty(n, H, dtype=weight.dtype, device=residual.device)
+    out, out2 = new(), new() if weight2 is not None else None
+    if d1 is None and rows is None:
         res = None if not keep else residual
         dst = None
     else:
         res = dst = torch.empty(n, H, dtype=torch.float32, device=residual.device) if keep else None
     assert residual.dtype == torch.float32 and residual.is_contiguous()
-    assert delta is None or (delta.dtype == weight.dtype and delta.is_contiguous())
-    _check(load().tgi_residual_norm(_f32(weight), _ptr(delta), _ptr(residual), _ptr(rows), _ptr(weight), _ptr(out), _ptr(dst),
-                                    c_int(n), c_int(H), c_float(eps), _stream()), "residual_norm")
-    return out, res
+    assert all(d is None or (d.dtype == weight.dtype and d.is_contiguous() and d.shape == residual.shape) for d in (d1, d2))
+    _check(load().tgi_residual_norm(_f32(weight), _ptr(d1), _ptr(d2), _ptr(residual), _ptr(rows), _ptr(weight), _ptr(weight2),
+                                    _ptr(out), _ptr(out2), _ptr(dst), c_int(n), c_int(H), c_float(eps), c_float(scale),
+                                    c_float(1.0 if unit_offset else 0.0), _stream()), "residual_norm")
+    return (out, res) if weight2 is None else (out, out2, res)
 
 
 def activation(x, act: str):
@@ -501,18 +511,26 @@ def activation(x, act: str):
 
 
 def rotate_norm_store(proj, offs, positions, cos_sin, slots, k_cache, v_cache, num_heads, num_kv_heads, dim, vdim, rot_dim,
-                      qk_norm, eps, v_first=None, v_lambda: float = 0.0):
+                      qk_norm, eps, v_first=None, v_lambda: float = 0.0, interleaved: bool = False, conv=None):
     T = proj.shape[0]
     Dk, Dv = k_cache.shape[3], v_cache.shape[3]
     q = torch.empty(T, num_heads, Dk, dtype=proj.dtype, device=proj.device)
     assert proj.stride(1) == 1 and k_cache.dtype == proj.dtype and v_cache.dtype == proj.dtype
     assert v_first is None or (v_first.stride(1) == 1 and v_first.shape[1] == num_kv_heads * vdim and v_first.dtype == proj.dtype)
+    past = [None] * 5 + [0] * 4
+    if conv is not None:
+        taps, channels = conv.state.shape[1] + 1, (num_heads + num_kv_heads) * dim + num_kv_heads * vdim
+        assert conv.weights.is_contiguous() and tuple(conv.weights.shape) == (conv_rows(taps), channels)
+        assert conv.state.is_contiguous() and conv.state.shape[2] == channels and conv.state.dtype == proj.dtype
+        past = [conv.weights, conv.cu, conv.kv_lens, conv.state_slots, conv.state, conv.kv_lens.shape[0], taps,
+                conv.state.shape[0], int(conv.single)]
     _check(load().tgi_attn_prep(
         _f32(proj), _ptr(proj), c_ll(proj.stride(0)), c_int(offs[1]), c_int(offs[2]), _ptr(positions), _ptr(cos_sin),
         _ptr(slots), _ptr(v_first), c_ll(0 if v_first is None else v_first.stride(0)), c_float(v_lambda), _ptr(q),
         _ptr(k_cache), _ptr(v_cache), c_int(T), c_int(num_heads), c_int(num_kv_heads), c_int(dim), c_int(vdim),
         c_int(Dk), c_int(Dv), c_int(rot_dim), c_int(cos_sin.shape[0]), c_ll(k_cache.shape[0] * k_cache.shape[1]),
-        c_int(1 if qk_norm else 0), c_float(eps), _stream()), "attn_prep")
+        c_int(1 if qk_norm else 0), c_float(eps), c_int(1 if interleaved else 0), *map(_ptr, past[:5]),
+        *map(c_int, past[5:]), _stream()), "attn_prep")
     return q
 
 
@@ -528,10 +546,11 @@ def conv_rows(taps: int) -> int:
 
 
 def delta_inputs(proj, offs, a_pre, conv_t, a_log, dt_bias, cu, kv_lens, state_slots, conv_state, kv_heads, heads, dim,
-                 pitch, vdim, single: bool):
+                 pitch, vdim, single: bool, head_decay: bool = False):
     T, dev = proj.shape[0], proj.device
     new = lambda *shape: torch.empty(*shape, dtype=torch.float32, device=dev)
-    q, k, g = new(T, kv_heads, pitch), new(T, kv_heads, pitch), new(T, heads, pitch)
+    q, k = new(T, kv_heads, pitch), new(T, kv_heads, pitch)
+    g = new(T, heads) if head_decay else new(T, heads, pitch)
     v, beta, qk = new(T, heads, vdim), new(T, heads), new(T, kv_heads)
     taps = conv_state.shape[1] + 1
     assert proj.stride(1) == 1 and a_pre.stride(1) == 1 and conv_state.dtype == proj.dtype
@@ -541,7 +560,8 @@ def delta_inputs(proj, offs, a_pre, conv_t, a_log, dt_bias, cu, kv_lens, state_s
         _ptr(a_pre), c_ll(a_pre.stride(0)), _ptr(conv_t), _ptr(a_log), _ptr(dt_bias), _ptr(cu),
         _ptr(kv_lens), _ptr(state_slots), _ptr(conv_state), _ptr(q), _ptr(k), _ptr(v), _ptr(g), _ptr(beta), _ptr(qk),
         c_int(T), c_int(kv_lens.shape[0]), c_int(conv_state.shape[0]), c_int(kv_heads), c_int(heads), c_int(dim),
-        c_int(pitch), c_int(vdim), c_int(taps), c_int(1 if single else 0), _stream()), "delta_prep")
+        c_int(pitch), c_int(vdim), c_int(taps), c_int(1 if single else 0), c_int(1 if head_decay else 0), _stream()),
+        "delta_prep")
     return q, k, v, g, beta, qk
 
 
@@ -551,7 +571,7 @@ def delta_scan(q, k, v, g, beta, qk, cu, kv_lens, state_slots, state, dim: int, 
     _check(load().tgi_delta_scan(
         _ptr(q), _ptr(k), _ptr(g), _ptr(v), _ptr(beta), _ptr(qk), _ptr(cu), _ptr(kv_lens), _ptr(state_slots), _ptr(state),
         _ptr(out), c_int(kv_lens.shape[0]), c_int(max_q), c_int(state.shape[0]), c_int(k.shape[1]), c_int(heads), c_int(dim),
-        c_int(state.shape[3]), c_int(vdim), _stream()), "delta_scan")
+        c_int(state.shape[3]), c_int(vdim), c_int(1 if g.dim() == 2 else 0), _stream()), "delta_scan")
     return out
 
 
@@ -565,13 +585,14 @@ def decay_scan(proj, offs, decay, cu, kv_lens, state_slots, state, heads: int, d
     return out
 
 
-def gated_norm(o, gate, weight, eps, groups: int, out_cols: int):
+def gated_norm(o, gate, weight, eps, groups: int, out_cols: int, act: str = "sigmoid"):
     T = o.shape[0]
     width = o.numel() // max(T * groups, 1)
     out = torch.empty(T, out_cols, dtype=gate.dtype, device=o.device)
     assert gate.stride(1) == 1 and weight.dtype == torch.float32
     _check(load().tgi_gated_norm(_f32(gate), _ptr(o), _ptr(gate), c_ll(gate.stride(0)), c_int(0), _ptr(weight), _ptr(out),
-                                 c_ll(out_cols), c_int(T), c_int(groups), c_int(width), c_float(eps), _stream()), "gated_norm")
+                                 c_ll(out_cols), c_int(T), c_int(groups), c_int(width), c_float(eps),
+                                 c_int({"sigmoid": 0, "silu": 1}[act]), _stream()), "gated_norm")
     return out
 
 
@@ -756,6 +777,63 @@ def moe_experts(x, w_gate_up, w_down, topk_weights, topk_ids, act="silu", first:
                                     c_int(st.sm_count), _ptr(st.status), s), "moe_grouped_gemm(down)")
     _check(lib.tgi_moe_combine(_ptr(y), _ptr(pos), c_int(T), c_int(k), c_int(H), _ptr(out), s), "moe_combine")
     return out
+
+
+def moe_route_sigmoid(x, weight, correction, top_k: int, scale: float):
+    """Router logits ``x @ weight^T`` in fp32, experts chosen by ``sigmoid + correction``, weights ``scale * s / sum(s)``."""
+    lib = load()
+    T, E = x.shape[0], weight.shape[0]
+    if x.dtype == torch.bfloat16:
+        K = weight.shape[1]                    # rows of 16-byte pieces: padded at load where the width is no multiple of 8
+        x = torch.nn.functional.pad(x, (0, K - x.shape[1])) if K > x.shape[1] else x.contiguous()
+        splits = int(lib.tgi_moe_router_splits(c_int(T), c_int(E), c_int(K), c_int(state(x.device).sm_count)))
+        part = torch.empty(splits, T, E, dtype=torch.float32, device=x.device)
+        assert weight.is_contiguous() and weight.dtype == x.dtype
+        _check(lib.tgi_moe_router(_ptr(x), _ptr(weight), c_int(T), c_int(E), c_int(K), c_int(splits), _ptr(part), _stream()),
+               "moe_router")
+    else:
+        part, splits = torch.nn.functional.linear(x, weight), 1
+    w = torch.empty(T, top_k, dtype=torch.float32, device=x.device)
+    ids = torch.empty(T, top_k, dtype=torch.int32, device=x.device)
+    _check(lib.tgi_moe_topk_sigmoid(_ptr(part), c_int(splits), _ptr(correction), c_int(T), c_int(E), c_int(top_k), c_float(scale),
+                                    _ptr(w), _ptr(ids), _stream()), "moe_topk_sigmoid")
+    return w, ids
+
+
+def moe_plain_experts(x, w_up, w_down, topk_weights, topk_ids, act: str):
+    """Ungated experts ``w_up [E, I, H]``, ``w_down [E, H, I]`` (``ops.plain_expert_weights``) on their routed rows, in bf16
+    (grouped tcgen05 GEMMs) or fp32; no host synchronisation."""
+    lib, st, s = load(), state(x.device), _stream()
+    T, H = x.shape
+    E, I, Hp = w_up.shape
+    k = topk_ids.shape[1]
+    n = T * k
+    new = lambda *shape, dtype=x.dtype: torch.empty(*shape, dtype=dtype, device=x.device)
+    assert w_up.is_contiguous() and w_down.is_contiguous() and tuple(w_down.shape) == (E, Hp, I) and w_up.dtype == x.dtype
+    assert topk_ids.dtype == torch.int32 and topk_weights.dtype == torch.float32
+    pos, order, offsets = new(n, dtype=torch.int32), new(n, dtype=torch.int32), new(E + 1, dtype=torch.int32)
+    hidden, y, out = new(n, I), new(n, Hp), new(T, Hp)
+    if T == 0:
+        return x.new_zeros(0, H)
+    x = torch.nn.functional.pad(x, (0, Hp - H)) if Hp > H else x.contiguous()
+    _check(lib.tgi_moe_sort(_ptr(topk_ids), c_int(n), c_int(0), c_int(E), _ptr(pos), _ptr(order), _ptr(offsets), s), "moe_sort")
+    code = c_int(_ACT_CODES[act])
+    if x.dtype == torch.float32:
+        for mode, src, w, dst in ((2, x, w_up, hidden), (1, hidden, w_down, y)):
+            _check(lib.tgi_moe_grouped_f32(c_int(mode), _ptr(src), c_int(n), _ptr(w), c_int(E), c_int(k), c_int(w.shape[1]),
+                                           c_int(w.shape[2]), _ptr(offsets), _ptr(order), code, _ptr(topk_weights), _ptr(dst), s),
+                   "moe_grouped_f32")
+        _check(lib.tgi_moe_combine_f32(_ptr(y), _ptr(pos), c_int(T), c_int(k), c_int(Hp), _ptr(out), s), "moe_combine_f32")
+        return out
+    grouped = new(n, Hp)
+    _check(lib.tgi_moe_gather(_ptr(x), _ptr(order), _ptr(offsets), c_int(E), c_int(k), c_int(Hp), c_int(n), _ptr(grouped), s),
+           "moe_gather")
+    for mode, src, w, dst in ((2, grouped, w_up, hidden), (1, hidden, w_down, y)):
+        _check(lib.tgi_moe_grouped_gemm(c_int(mode), _ptr(src), c_int(n), _ptr(w), c_int(E), c_int(w.shape[1]), c_int(w.shape[2]),
+                                        _ptr(offsets), code, _ptr(topk_weights), _ptr(order), _ptr(dst), c_int(st.sm_count),
+                                        _ptr(st.status), s), "moe_grouped_gemm")
+    _check(lib.tgi_moe_combine(_ptr(y), _ptr(pos), c_int(T), c_int(k), c_int(Hp), _ptr(out), s), "moe_combine")
+    return out if Hp == H else out[:, :H].contiguous()
 
 
 # ---- multi-adapter LoRA ------------------------------------------------------------------------

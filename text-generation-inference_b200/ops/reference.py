@@ -203,6 +203,8 @@ def activation(x: torch.Tensor, act: str) -> torch.Tensor:
         return F.gelu(x, approximate="tanh")
     if act == "relu":
         return F.relu(x)
+    if act == "relu2":
+        return F.relu(x).square()
     if act == "quick_gelu":
         return x * torch.sigmoid(1.702 * x)
     raise ValueError(f"unknown activation {act}")
@@ -302,6 +304,24 @@ def moe_topk_softmax(router_logits: torch.Tensor, top_k: int, renormalize: bool 
     return w, idx
 
 
+def moe_route_sigmoid(x, weight, correction, top_k: int, scale: float):
+    s = torch.sigmoid(F.linear(x.float(), weight.float()))
+    idx = torch.topk(s + correction, top_k, dim=-1)[1]
+    w = s.gather(1, idx)
+    return w / (w.sum(-1, keepdim=True) + 1e-20) * scale, idx
+
+
+def moe_plain_experts(x, w_up, w_down, topk_weights, topk_ids, act: str):
+    """``w_up[E, I, H]``, ``w_down[E, H, I]``: sum over a token's experts of weight times ``down(act(up x))``."""
+    out = torch.zeros(x.shape, dtype=torch.float32, device=x.device)
+    for e in range(w_up.shape[0]):
+        tok, slot = (topk_ids == e).nonzero(as_tuple=True)
+        if tok.numel():
+            y = F.linear(activation(F.linear(x[tok], w_up[e]), act), w_down[e]).float()
+            out.index_add_(0, tok, y * topk_weights[tok, slot].unsqueeze(1).float())
+    return out.to(x.dtype)
+
+
 def moe_sparsemixer(router_logits: torch.Tensor, jitter_eps: float = 0.01) -> Tuple[torch.Tensor, torch.Tensor]:
     """Top-2 routing of Phi-3.5-MoE ("sparsemixer", inference form): each of the two picks is the arg-max of
     the remaining logits, and its weight is the softmax over the logits that lie within a relative
@@ -348,35 +368,17 @@ def embed_residual(ids, table, scale: float = 1.0):
     return F.embedding(ids.long(), table).float() * scale
 
 
-def residual_norm(delta, residual, weight, eps: float, rows=None, keep: bool = True):
-    r = residual if delta is None else residual + delta.float()
+def residual_norm(delta, residual, weight, eps: float, rows=None, keep: bool = True, scale: float = 1.0,
+                  unit_offset: bool = False, weight2=None):
+    r = residual
+    if delta is not None:
+        parts = delta if isinstance(delta, tuple) else (delta,)
+        r = residual + scale * sum(d.float() for d in parts)
     if rows is not None:
         r = r[rows.long()]
-    y = r * torch.rsqrt(r.pow(2).mean(-1, keepdim=True) + eps) * weight.float()
-    return y.to(weight.dtype), (r if keep else None)
-
-
-def rotate_norm_store(proj, offs, positions, cos_sin, slots, k_cache, v_cache, num_heads, num_kv_heads, dim, vdim, rot_dim,
-                      qk_norm, eps, v_first=None, v_lambda: float = 0.0):
-    T = proj.shape[0]
-    cs = cos_sin[positions.long()]
-    cos, sin = cs[:, : rot_dim // 2], cs[:, rot_dim // 2:]
-
-    def head(off, n):
-        x = proj[:, off:off + n * dim].reshape(T, n, dim).float()
-        if rot_dim > 0:
-            x = rotate(x, cos, sin, rot_dim, True)
-        return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) if qk_norm else x
-
-    q, k = head(offs[0], num_heads), head(offs[1], num_kv_heads)
-    v = proj[:, offs[2]:offs[2] + num_kv_heads * vdim].float()
-    if v_first is not None:
-        v = (1.0 - v_lambda) * v + v_lambda * v_first.float()
-    ok = (slots >= 0).nonzero(as_tuple=True)[0]
-    idx = slots[ok].long()
-    k_cache.view(-1, num_kv_heads, k_cache.shape[3])[idx, :, :dim] = k[ok].to(k_cache.dtype)
-    v_cache.view(-1, num_kv_heads, v_cache.shape[3])[idx, :, :vdim] = v.view(T, num_kv_heads, vdim)[ok].to(v_cache.dtype)
-    return F.pad(q, (0, k_cache.shape[3] - dim)).to(proj.dtype)
+    x = r * torch.rsqrt(r.pow(2).mean(-1, keepdim=True) + eps)
+    ys = tuple((x * (w.float() + (1.0 if unit_offset else 0.0))).to(w.dtype) for w in (weight, weight2) if w is not None)
+    return ys + (r if keep else None,)
 
 
 def _sequences(cu, kv_lens, state_slots):
@@ -388,32 +390,72 @@ def _sequences(cu, kv_lens, state_slots):
 
 
 def _short_conv(x, w, past):
-    """``x[n, C]`` after ``past[taps - 1, C]``; returns the convolved, SiLU-ed rows and the new past."""
+    """``x[n, C]`` after ``past[taps - 1, C]``; returns the convolved rows and the new past."""
     taps = w.shape[0]
     full = torch.cat([past.float(), x.float()], dim=0)
     y = sum(full[j:j + x.shape[0]] * w[j].float() for j in range(taps))
-    return F.silu(y), full[full.shape[0] - (taps - 1):]
+    return y, full[full.shape[0] - (taps - 1):]
 
 
-def delta_inputs(proj, offs, a_pre, conv_t, a_log, dt_bias, cu, kv_lens, state_slots, conv_state, kv_heads, heads, dim,
-                 pitch, vdim, single: bool):
-    T, taps = proj.shape[0], conv_state.shape[1] + 1
-    nq, nv = kv_heads * dim, heads * vdim
-    x = torch.cat([proj[:, offs[0]:offs[0] + nq], proj[:, offs[1]:offs[1] + nq], proj[:, offs[2]:offs[2] + nv]], dim=1)
+def _conv_rows(proj, offs, widths, conv_t, cu, kv_lens, state_slots, conv_state):
+    """Column groups ``offs`` / ``widths`` of ``proj`` side by side after their short convolutions, fp32; advances
+    ``conv_state``."""
+    x = torch.cat([proj[:, o:o + w] for o, w in zip(offs, widths)], dim=1)
+    taps = conv_state.shape[1] + 1
     w = conv_t[conv_t.shape[0] - taps:]
-    y = torch.zeros(T, 2 * nq + nv)
+    y = torch.zeros(x.shape)
     for _, s, n, start, slot in _sequences(cu, kv_lens, state_slots):
         past = conv_state[slot] if slot >= 0 and start > 0 else torch.zeros(taps - 1, x.shape[1])
         y[s:s + n], new = _short_conv(x[s:s + n], w, past)
         if slot >= 0:
             conv_state[slot] = new.to(conv_state.dtype)
+    return y
+
+
+def rotate_norm_store(proj, offs, positions, cos_sin, slots, k_cache, v_cache, num_heads, num_kv_heads, dim, vdim, rot_dim,
+                      qk_norm, eps, v_first=None, v_lambda: float = 0.0, interleaved: bool = False, conv=None):
+    T = proj.shape[0]
+    if conv is not None:
+        widths = (num_heads * dim, num_kv_heads * dim, num_kv_heads * vdim)
+        proj_dtype, proj = proj.dtype, _conv_rows(proj, offs, widths, conv.weights, conv.cu, conv.kv_lens, conv.state_slots,
+                                                  conv.state)
+        offs = (0, widths[0], widths[0] + widths[1])
+    else:
+        proj_dtype = proj.dtype
+    cs = cos_sin[positions.long()]
+    cos, sin = cs[:, : rot_dim // 2], cs[:, rot_dim // 2:]
+
+    def head(off, n):
+        x = proj[:, off:off + n * dim].reshape(T, n, dim).float()
+        if rot_dim > 0:
+            x = rotate(x, cos, sin, rot_dim, not interleaved)
+        return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) if qk_norm else x
+
+    q, k = head(offs[0], num_heads), head(offs[1], num_kv_heads)
+    v = proj[:, offs[2]:offs[2] + num_kv_heads * vdim].float()
+    if v_first is not None:
+        v = (1.0 - v_lambda) * v + v_lambda * v_first.float()
+    ok = (slots >= 0).nonzero(as_tuple=True)[0]
+    idx = slots[ok].long()
+    k_cache.view(-1, num_kv_heads, k_cache.shape[3])[idx, :, :dim] = k[ok].to(k_cache.dtype)
+    v_cache.view(-1, num_kv_heads, v_cache.shape[3])[idx, :, :vdim] = v.view(T, num_kv_heads, vdim)[ok].to(v_cache.dtype)
+    return F.pad(q, (0, k_cache.shape[3] - dim)).to(proj_dtype)
+
+
+def delta_inputs(proj, offs, a_pre, conv_t, a_log, dt_bias, cu, kv_lens, state_slots, conv_state, kv_heads, heads, dim,
+                 pitch, vdim, single: bool, head_decay: bool = False):
+    T = proj.shape[0]
+    nq, nv = kv_heads * dim, heads * vdim
+    y = F.silu(_conv_rows(proj, offs, (nq, nq, nv), conv_t, cu, kv_lens, state_slots, conv_state))
     q, k = (y[:, i * nq:(i + 1) * nq].view(T, kv_heads, dim) for i in range(2))
     q = q * torch.rsqrt(q.pow(2).sum(-1, keepdim=True) + 1e-6) * dim ** -0.5
     k = k * torch.rsqrt(k.pow(2).sum(-1, keepdim=True) + 1e-6)
-    g = torch.exp(-torch.exp(a_log).view(1, heads, 1) * F.softplus(a_pre.float() + dt_bias).view(T, heads, dim))
+    step = F.softplus(a_pre.float() + dt_bias).view(T, heads, 1 if head_decay else dim)
+    g = torch.exp(-torch.exp(a_log).view(1, heads, 1) * step)
     beta = torch.sigmoid(proj[:, offs[3]:offs[3] + heads].float())
     pad = (0, pitch - dim)
-    return F.pad(q, pad), F.pad(k, pad), y[:, 2 * nq:].view(T, heads, vdim), F.pad(g, pad), beta, (q * k).sum(-1)
+    g = g.squeeze(2) if head_decay else F.pad(g, pad)
+    return F.pad(q, pad), F.pad(k, pad), y[:, 2 * nq:].view(T, heads, vdim), g, beta, (q * k).sum(-1)
 
 
 def delta_scan(q, k, v, g, beta, qk, cu, kv_lens, state_slots, state, dim: int, max_q: int):
@@ -424,7 +466,7 @@ def delta_scan(q, k, v, g, beta, qk, cu, kv_lens, state_slots, state, dim: int, 
     for _, s, n, start, slot in _sequences(cu, kv_lens, state_slots):
         S = state[slot].clone() if slot >= 0 and start > 0 else torch.zeros(state.shape[1:])      # [H, vdim, pitch]
         for t in range(s, s + n):
-            S = S * g[t].unsqueeze(1)
+            S = S * g[t].view(heads, 1, -1)
             u = beta[t].unsqueeze(1) * (v[t] - torch.einsum("hvd,hd->hv", S, k[t]))
             S = S + u.unsqueeze(2) * k[t].unsqueeze(1)
             out[t] = torch.einsum("hvd,hd->hv", S, q[t])
@@ -450,9 +492,10 @@ def decay_scan(proj, offs, decay, cu, kv_lens, state_slots, state, heads: int, d
     return out
 
 
-def gated_norm(o, gate, weight, eps: float, groups: int, out_cols: int):
+def gated_norm(o, gate, weight, eps: float, groups: int, out_cols: int, act: str = "sigmoid"):
     T = o.shape[0]
     x = o.reshape(T, groups, -1)
     y = x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * weight
-    y = y.reshape(T, -1) * torch.sigmoid(gate[:, :y.numel() // T].float())
+    fn = torch.sigmoid if act == "sigmoid" else F.silu
+    y = y.reshape(T, -1) * fn(gate[:, :y.shape[1] * y.shape[2]].float())
     return F.pad(y, (0, out_cols - y.shape[1])).to(gate.dtype)

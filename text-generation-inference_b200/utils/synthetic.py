@@ -368,9 +368,78 @@ def fuzuvik_state_dict(cfg: dict, seed: int = 0, dtype=torch.float32, device: st
     return sd
 
 
-def write_fuzuvik_checkpoint(path, cfg: dict, sd: Dict[str, torch.Tensor]) -> Path:
+def write_checkpoint(path, cfg: dict, sd: Dict[str, torch.Tensor]) -> Path:
     out = Path(path)
     out.mkdir(parents=True, exist_ok=True)
     (out / "config.json").write_text(json.dumps(cfg))
     save_safetensors(sd, out / "model.safetensors")
     return out
+
+
+def kipedra_attention(heads=4, kv_heads=2, dim=32, vdim=16, window=24, rot_dims=None, base=10000.0, scale=None, conv=4,
+                      mlp=None) -> dict:
+    return {"type": "attention", "mlp": mlp,
+            "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv, "mask": {"size": window},
+                      "rot": {"base": base, "dims": dim if rot_dims is None else rot_dims},
+                      "scale": dim ** -0.5 if scale is None else scale}}
+
+
+def kipedra_delta(heads=4, kv_heads=2, dim=24, vdim=40, conv=4, mlp=None) -> dict:
+    return {"type": "delta", "mlp": mlp,
+            "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv}}
+
+
+def kipedra_dense(ff=96) -> dict:
+    return {"kind": "dense", "ff": ff}
+
+
+def kipedra_moe(ff=40, experts=10, top=3, scale=2.5) -> dict:
+    return {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top, "scale": scale}}
+
+
+def kipedra_config(layers, width=80, vocab=203, eps=1e-5, residual_mult=0.4, loop=None) -> dict:
+    return {"architecture": "Kipedra", "width": width, "vocab": vocab, "norm": {"eps": eps}, "residual_mult": residual_mult,
+            "loop": dict(zip(("start", "stop", "times"), loop or (0, len(layers), 1))), "layers": list(layers)}
+
+
+def kipedra_state_dict(cfg: dict, seed: int = 0, dtype=torch.float32, device: str = "cpu") -> Dict[str, torch.Tensor]:
+    """Random weights of a Kipedra shape."""
+    g = torch.Generator(device=device).manual_seed(seed)
+    W, sd = cfg["width"], {}
+
+    def rnd(*shape, std=None, mean=0.0):
+        std = shape[-1] ** -0.5 if std is None else std
+        return (mean + torch.randn(*shape, generator=g, device=device) * std).to(dtype)
+
+    def uniform(lo, hi, *shape):
+        return (lo + (hi - lo) * torch.rand(shape, generator=g, device=device)).to(dtype)
+
+    sd["embed"], sd["final.norm"] = rnd(cfg["vocab"], W, std=0.5), rnd(W, std=0.2)
+    for i, layer in enumerate(cfg["layers"]):
+        p, m, mlp = f"l{i}.", layer["mixer"], layer.get("mlp")
+        H, G, d, dv, taps = m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["conv"]
+        mix, attn = p + "mix.", layer["type"] == "attention"
+        sd[p + "norm1"] = rnd(W, std=0.2)
+        for n, rows in (("q", (H if attn else G) * d), ("k", G * d), ("v", (G if attn else H) * dv)):
+            sd.update({mix + n: rnd(rows, W), mix + n + ".conv": rnd(rows, taps)})
+            if attn:
+                sd[mix + n + ".b"] = rnd(rows, std=0.3)
+        sd[mix + "o"] = rnd(W, H * dv)
+        if not attn:
+            sd.update({mix + "b": rnd(H, W), mix + "a": rnd(H, W), mix + "g": rnd(H * dv, W), mix + "norm": rnd(dv, std=0.1, mean=1.0),
+                       mix + "A_log": uniform(-3.0, 1.0, H), mix + "dt_bias": uniform(-4.0, 0.5, H)})
+        if mlp is None:
+            continue
+        sd[p + "norm2"] = rnd(W, std=0.2)
+        if mlp["kind"] == "dense":
+            ff = mlp["ff"]
+            sd.update({p + "mlp.gate": rnd(ff, W), p + "mlp.up": rnd(ff, W), p + "mlp.down": rnd(W, ff)})
+            continue
+        ff, E = mlp["expert"]["ff"], mlp["router"]["experts"]
+        sd.update({p + "mlp.router": rnd(E, W), p + "mlp.correction": rnd(E, std=0.2)})
+        for e in range(E):
+            sd.update({f"{p}mlp.e{e}.up": rnd(ff, W), f"{p}mlp.e{e}.down": rnd(W, ff)})
+    return sd
+
+
+
