@@ -9,9 +9,9 @@ import pytest
 import torch
 
 import fuzuvik_oracle as O
+from decoder_harness import (be, check, expected, feed, generate, replay_for, requests, runner_for, sure_prompts,  # noqa: F401
+                             tokens)
 from tgi_b200.utils import synthetic as syn
-
-BACKENDS = ["cpu-f32", pytest.param("cuda-f32", marks=pytest.mark.gpu), pytest.param("cuda-bf16", marks=pytest.mark.gpu)]
 
 CONFIGS = {
     # every mixer, shared q/k heads, three layers that mix values (one between them that does not), one without ff
@@ -34,12 +34,6 @@ CONFIGS = {
 }
 
 
-@pytest.fixture(params=BACKENDS)
-def be(request):
-    dev, dt = request.param.split("-")
-    return torch.device(dev), torch.float32 if dt == "f32" else torch.bfloat16
-
-
 _CKPT = {}
 
 
@@ -49,54 +43,10 @@ def checkpoints(tmp_path_factory):
         if name not in _CKPT:
             cfg = CONFIGS[name]
             sd = {k: v.to(torch.bfloat16) for k, v in syn.fuzuvik_state_dict(cfg, seed=len(name)).items()}
-            _CKPT[name] = (cfg, sd, syn.write_checkpoint(tmp_path_factory.mktemp(name), cfg, sd), {})
+            _CKPT[name] = (cfg, sd, syn.write_checkpoint(tmp_path_factory.mktemp(name), cfg, sd), {}, O)
         return _CKPT[name]
 
     return get
-
-
-def tokens(cfg, n, seed):
-    return random.Random(seed).choices(range(cfg["vocab"]), k=n)
-
-
-def expected(ck, ids):
-    cfg, sd, _, memo = ck
-    key = tuple(ids)
-    if key not in memo:
-        memo[key] = O.forward(cfg, sd, ids)
-    return memo[key]
-
-
-def runner_for(ck, be):
-    from tgi_b200.models import get_model
-
-    dev, dt = be
-    return get_model(str(ck[2]), dtype="float32" if dt == torch.float32 else "bfloat16", device=dev, max_positions=512)
-
-
-def replay_for(ck, be, max_tokens):
-    from tgi_b200.server.replay import Replay
-
-    return Replay(runner_for(ck, be), max_tokens)
-
-
-def check(got, want, dtype):
-    """Largest per-position error (mean over the vocabulary taken off) against the spread of the expected logits."""
-    d = got.double() - want
-    d = d - d.mean(-1, keepdim=True)
-    err = (d.pow(2).mean(-1).sqrt() / want.std()).max().item()
-    assert err < (2e-5 if dtype == torch.float32 else 0.04), err
-
-
-def feed(rp, name, ids, portions, end=True):
-    """All logits of ``ids`` brought in ``portions``."""
-    out, at = [], 0
-    for i, n in enumerate(portions):
-        last = at + n == len(ids)
-        out.append(rp.step([{"id": name, "tokens": ids[at:at + n], "want": list(range(n))}], [name] if last and end else []))
-        at += n
-    assert at == len(ids)
-    return torch.cat(out)
 
 
 @pytest.mark.parametrize("name", CONFIGS)
@@ -176,7 +126,7 @@ def test_batches_of_unequal_requests(be, checkpoints, name):
 
 def test_first_layer_values_reach_every_later_layer(be, checkpoints):
     """Another first layer value, the same later ones: the change goes through the mixing and nowhere else."""
-    cfg, sd, _, _ = ck = checkpoints("attention")
+    cfg, sd, _, _, _ = ck = checkpoints("attention")
     sd2 = dict(sd)
     sd2["l0.mix.o"] = torch.zeros_like(sd["l0.mix.o"])        # the first layer itself writes nothing
     ids = tokens(cfg, 40, 3)
@@ -188,70 +138,6 @@ def test_first_layer_values_reach_every_later_layer(be, checkpoints):
 
 
 # ---- generation ----------------------------------------------------------------------------------
-def requests(prompts, new_tokens):
-    from tgi_b200.proto import generate_v3 as pb
-
-    out, block = [], 1
-    for i, p in enumerate(prompts):
-        r = pb.Request(id=i, inputs="")
-        r.parameters.temperature = r.parameters.top_p = r.parameters.typical_p = r.parameters.repetition_penalty = 1.0
-        r.stopping_parameters.max_new_tokens = new_tokens[i]
-        r.stopping_parameters.ignore_eos_token = True
-        n = (len(p) + new_tokens[i] + 15) // 16
-        r.blocks.extend(range(block, block + n))
-        block += n
-        out.append(r)
-    return out, block
-
-
-def generate(runner, prompts, new_tokens, max_prefill=None, late=()):
-    """Through ``generate_token``; requests in ``late`` join the running batch after two steps."""
-    from tgi_b200.models.flash_causal_lm import FlashCausalLMBatch as B
-    from tgi_b200.proto import generate_v3 as pb
-
-    reqs, blocks = requests(prompts, new_tokens)
-    runner.init_kv_cache(blocks, state_slots=len(prompts))
-
-    def batch_of(idx):
-        return B.from_tokenized(pb.Batch(id=idx[0], requests=[reqs[i] for i in idx], size=len(idx)), [prompts[i] for i in idx],
-                                runner.tokenizer, runner.dtype, runner.device)
-
-    early = [i for i in range(len(prompts)) if i not in late]
-    batch, toks, step = batch_of(early), {i: [] for i in range(len(prompts))}, 0
-    batch.max_prefill_tokens = max_prefill
-    while batch is not None:
-        if step == 2 and late:
-            joined = batch_of(list(late))
-            joined.max_prefill_tokens = max_prefill
-            batch = B.concatenate([batch, joined])
-        gens, batch, _ = runner.generate_token(batch)
-        step += 1
-        for g in gens:
-            toks[g.request_id].extend(g.tokens.token_ids)
-        if batch is not None:
-            keep = [s.request.id for s in batch.seqs if not s.finished]
-            batch = batch.filter(keep)
-    return toks
-
-
-def sure_prompts(ck, count, n, new):
-    """Prompts whose greedy continuation never hangs on a near tie."""
-    out, seed = [], 100
-    while len(out) < count:
-        ids = tokens(ck[0], n + 7 * len(out), seed)
-        seed += 1
-        logits = []
-        cur = list(ids)
-        for _ in range(new):
-            row = O.forward(ck[0], ck[1], cur)[-1]
-            logits.append(row)
-            cur.append(int(row.argmax()))
-        top = torch.stack(logits).topk(2).values
-        if (top[:, 0] - top[:, 1]).min() > 0.12:
-            out.append((ids, cur[len(ids):]))
-    return out
-
-
 _SURE = {}
 
 

@@ -1,7 +1,8 @@
-"""Prefill and decode throughput of a Fuzuvik-shaped decoder beside a Llama-shaped one of the same width, depth, heads
-and parameter count, and the kernels of both against their rooflines.
+"""Prefill and decode throughput of a hybrid decoder beside its closest relative of the same width, depth, heads and
+active parameters per token, and the kernels of both against their rooflines.
 
-``python bench.py --model fuzuvik-bf16`` prints one JSON line.  Weights are random; token rates are timed with CUDA
+``python bench.py --model fuzuvik-bf16`` (beside a Llama shape) and ``--model kipedra-bf16`` (beside a Fuzuvik shape; expert
+kernels beside those of gated experts) print one JSON line.  Weights are random; token rates are timed with CUDA
 events around the model's forward (prefill) and around replays of its decode graph.  Kernels are timed one by one
 with the L2 flushed in front of every launch; a roofline is the larger of bytes over the measured copy bandwidth and
 FLOPs over the measured rate of the unit that does them (bf16 tensor cores, or fp32 FMA for the state recurrences).
@@ -46,6 +47,27 @@ def llama_like(width: int, layers: int, vocab: int) -> dict:
                             intermediate=(8 * width // 3 + 127) // 128 * 128, vocab=vocab, theta=500000.0, max_pos=16384)
 
 
+def kipedra_like(width: int, layers: int, vocab: int, window: int) -> dict:
+    """Every fourth layer dense, the others with 16 experts of which a token uses four: per token the parameters of a plain
+    feed-forward of 4 x width."""
+    from ..utils import synthetic as syn
+
+    h = width // 128
+    dense, moe = syn.kipedra_dense((8 * width // 3 + 127) // 128 * 128), syn.kipedra_moe(ff=width, experts=16, top=4, scale=1.0)
+    attn = lambda mlp: syn.kipedra_attention(h, h // 4, 128, 128, window, base=500000.0, mlp=mlp)
+    kinds = [attn(dense), syn.kipedra_delta(h, h, 128, 128, 4, mlp=moe), attn(moe), syn.kipedra_delta(h, h, 128, 128, 4, mlp=moe)]
+    return syn.kipedra_config([kinds[i % 4] for i in range(layers)], width=width, vocab=vocab, eps=1e-6, residual_mult=0.3)
+
+
+def fuzuvik_twin(width: int, layers: int, vocab: int, window: int) -> dict:
+    """The Fuzuvik shape that ``kipedra_like`` is measured beside: attention and delta layers in turn, chunks as long as the
+    windows, dense feed-forwards."""
+    cfg = fuzuvik_like(width, layers, vocab, window)
+    for i in range(3, layers, 4):
+        cfg["layers"][i] = cfg["layers"][1]
+    return cfg
+
+
 def make_runner(cfg: dict, dev):
     from ..models.arch import ModelConfig
     from ..models.decoder import CausalDecoder
@@ -55,8 +77,10 @@ def make_runner(cfg: dict, dev):
 
     mc = ModelConfig(cfg)
     if cfg.get("architecture"):
-        w = syn.DictWeights(syn.fuzuvik_state_dict(cfg, dtype=torch.bfloat16, device=str(dev), rank=128), dev, torch.bfloat16,
-                            bare_names=True)
+        tensors = (syn.kipedra_state_dict(cfg, dtype=torch.bfloat16, device=str(dev)) if cfg["architecture"] == "Kipedra" else
+                   syn.fuzuvik_state_dict(cfg, dtype=torch.bfloat16, device=str(dev), rank=128))
+        w = syn.DictWeights(tensors, dev, torch.bfloat16, bare_names=True)
+        del tensors
     else:
         w = syn.SyntheticWeights(cfg, dev, torch.bfloat16)
     model = CausalDecoder(mc, w, max_positions=16384)
@@ -251,30 +275,131 @@ def kernel_rows(dev, width: int, chunk: int, prefill, decode) -> list:
     return kt.rows
 
 
+def kipedra_rows(dev, width: int, window: int, prefill, decode) -> list:
+    """Every kernel of the design at layer size, and the like kernels of the Fuzuvik shape and of gated experts."""
+    from .. import ops
+    from . import cuda as K
+    from ..models.arch import MixerSpec
+    from ..models.mixers import RotaryTables
+
+    H, G, d, taps = width // 128, width // 512, 128, 4
+    kt = KernelTimer(dev)
+    bf, f32 = torch.bfloat16, torch.float32
+    tab = RotaryTables(16384, dev).get(MixerSpec("attention", H, G, d, d, rot_dims=d, rot_base=500000.0)).cos_sin
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+    rn = lambda *s, dt=bf: torch.randn(*s, device=dev, dtype=f32).to(dt)
+    for label, B, n, ctx in [("prefill", *prefill, prefill[1]), ("decode", decode[0], 1, decode[1])]:
+        T, one = B * n, n == 1
+        tag = f"{label} {B}x{n}" + (f" @{ctx}" if one else "")
+        cu, kv, slots = i32([i * n for i in range(B + 1)]), i32([ctx] * B), i32(list(range(B)))
+        per = math.ceil(ctx / 16)
+        bt = torch.arange(B * per, dtype=torch.int32, device=dev).view(B, per)
+        pos = i32([ctx - n + i for _ in range(B) for i in range(n)])
+        page = i32([b * per * 16 + ctx - n + i for b in range(B) for i in range(n)])
+        kc, vc = rn(B * per, 16, G, d), rn(B * per, 16, G, d)
+        # ---- attention layer
+        qw = (H + 2 * G) * d
+        proj, first, offs = rn(T, qw), rn(T, G * d), [0, H * d, H * d + G * d]
+        past = torch.zeros(B, taps - 1, qw, dtype=bf, device=dev)
+        conv = ops.ShortConv(ops.conv_weights([torch.randn(w * d, taps, device=dev) for w in (H, G, G)], dev), past, cu, kv, slots, one)
+        io, pb = T * qw * 4, B * (taps - 1) * qw * 2 * (2 if one else 1)
+        kt(f"{tag}: convolution + rotate + store", lambda: ops.rotate_norm_store(
+            proj, offs, pos, tab, page, kc, vc, H, G, d, d, d, False, 1e-6, interleaved=True, conv=conv), io + pb)
+        kt(f"{tag}: [fuzuvik] rotate + unit rms + value mix + store", lambda: ops.rotate_norm_store(
+            proj, offs, pos, tab, page, kc, vc, H, G, d, d, d, True, 1e-6, first, 0.3), io + T * G * d * 2)
+        q = rn(T, H, d)
+        for name, kw in (("attention, window", dict(window=window)), ("[fuzuvik] attention, chunk + sink", dict(chunk=window, sink=True))):
+            if one:
+                span = min(ctx, window) if "window" in kw else (ctx - 1) % window + 1
+                by, fl = 2 * B * span * G * d * 2 + T * H * d * 4, 0.0
+            else:
+                pairs = B * sum(min(i + 1, window) if "window" in kw else i % window + 1 for i in range(n))
+                by, fl = T * H * d * 4 + 2 * T * G * d * 2, 4.0 * pairs * H * d
+            kt(f"{tag}: {name}", lambda: ops.paged_attention(q, kc, vc, bt, cu, kv, d ** -0.5, max_q=n, max_kv=ctx, **kw), by, fl)
+        wl, xw, bias = rn(qw, width), rn(T, width), rn(qw)
+        kt(f"{tag}: GEMM q k v + bias", lambda: ops.linear(xw, wl, bias), (T + qw) * width * 2 + T * qw * 2, 2.0 * T * qw * width)
+        kt(f"{tag}: [fuzuvik] GEMM q k v", lambda: ops.linear(xw, wl), (T + qw) * width * 2 + T * qw * 2, 2.0 * T * qw * width)
+        # ---- delta layer
+        C, hp = 3 * H * d, (H + 7) // 8 * 8
+        cols = C + 2 * hp + H * d
+        x, a = rn(T, cols), rn(T, H * d)
+        taps_w = ops.conv_weights([torch.randn(H * d, taps, device=dev) for _ in range(3)], dev)
+        a_log, bh, bc = torch.zeros(H, device=dev), torch.randn(H, device=dev) - 2, torch.randn(H * d, device=dev) - 2
+        cs, S = torch.zeros(B, taps - 1, C, dtype=bf, device=dev), torch.zeros(B, H, d, d, device=dev)
+        do = [0, H * d, 2 * H * d, C, C + hp, C + 2 * hp]
+        cb, st = B * (taps - 1) * C * 2 * (2 if one else 1), B * H * d * d * 4 * (2 if one else 1)
+        prep = lambda: ops.delta_inputs(x, do, x[:, do[4]:do[4] + H], taps_w, a_log, bh, cu, kv, slots, cs, H, H, d, d, d, one, True)
+        wide = lambda: ops.delta_inputs(x, do, a, taps_w, a_log, bc, cu, kv, slots, cs, H, H, d, d, d, one)
+        kt(f"{tag}: delta inputs, decay per head", prep, T * H * (d * (3 * 2 + 3 * 4) + 16) + cb)
+        kt(f"{tag}: [fuzuvik] delta inputs", wide, T * H * d * (4 * 2 + 4 * 4) + cb)
+        r = prep()
+        kt(f"{tag}: delta scan, decay per head", lambda: ops.delta_scan(*r, cu, kv, slots, S, d, n), T * H * (d * 16 + 8) + st,
+           7.0 * T * H * d * d, "fp32")
+        r2 = wide()
+        kt(f"{tag}: [fuzuvik] delta scan", lambda: ops.delta_scan(*r2, cu, kv, slots, S, d, n), T * H * d * 20 + st,
+           7.0 * T * H * d * d, "fp32")
+        del r2
+        o, w1 = rn(T, H, d, dt=f32), torch.ones(d, device=dev)
+        kt(f"{tag}: norm x silu gate", lambda: ops.gated_norm(o, x[:, do[5]:], w1, 1e-6, H, H * d, "silu"), T * H * d * 8)
+        kt(f"{tag}: [fuzuvik] norm x gate", lambda: ops.gated_norm(o, a, w1, 1e-6, H, H * d), T * H * d * 8)
+        wq = rn(cols, width)
+        kt(f"{tag}: GEMM q k v b a g", lambda: ops.linear(xw, wq), (T + cols) * width * 2 + T * cols * 2, 2.0 * T * cols * width)
+        # ---- stream
+        res, d1, d2, n1, n2 = rn(T, width, dt=f32), rn(T, width), rn(T, width), rn(width), rn(width)
+        kt(f"{tag}: residual (fp32, two outputs) + two norms", lambda: ops.residual_norm(
+            (d1, d2), res, n1, 1e-6, scale=0.3, unit_offset=True, weight2=n2), T * width * 16)
+        kt(f"{tag}: [fuzuvik] residual (fp32) + norm", lambda: ops.residual_norm(d1, res, n1, 1e-6), T * width * 12)
+        # ---- feed-forwards
+        ff = (8 * width // 3 + 127) // 128 * 128
+        gu, u = rn(T, 2 * ff), rn(T, 4 * width)
+        kt(f"{tag}: gelu x up", lambda: ops.act_and_mul(gu, "gelu_tanh"), gu.numel() * 3)
+        kt(f"{tag}: [llama] silu x up", lambda: ops.act_and_mul(gu, "silu"), gu.numel() * 3)
+        kt(f"{tag}: [fuzuvik] gelu", lambda: ops.activation(u, "gelu"), u.numel() * 4)
+        del gu, u
+        E, top, I = 16, 4, width
+        rw, corr = rn(E, width) * 0.02, torch.zeros(E, device=dev)
+        rb = (T + E) * width * 2 + T * top * 8
+        route = lambda: ops.moe_route_sigmoid(xw, rw, corr, top, 1.0)
+        kt(f"{tag}: router (sigmoid, fp32)", route, rb, 2.0 * T * E * width)
+        kt(f"{tag}: [mixtral] router (softmax)", lambda: ops.moe_topk_softmax(ops.linear(xw, rw), top), rb, 2.0 * T * E * width)
+        tw, ti = route()
+        up, down, used = rn(E, I, width) * 0.02, rn(E, width, I) * 0.02, min(E, T * top)
+        kt(f"{tag}: experts, ungated", lambda: ops.moe_plain_experts(xw, up, down, tw, ti, "relu2"),
+           used * 2 * I * width * 2 + T * width * 4, 4.0 * T * top * I * width)
+        wgu, wd = rn(E, I, width) * 0.02, rn(E, width, I // 2) * 0.02
+        kt(f"{tag}: [mixtral] experts, gated, half as wide", lambda: ops.moe_experts(xw, wgu, wd, tw, ti, "silu"),
+           used * 3 * (I // 2) * width * 2 + T * width * 4, 3.0 * T * top * I * width)
+        assert K.check_status(dev) == 0
+        del up, down, wgu, wd
+        torch.cuda.empty_cache()
+    return kt.rows
+
+
 def run(args, clock_sampler) -> int:
     from . import cuda as K
 
+    kipedra = args.model == "kipedra-bf16"
     dev = torch.device("cuda", 0)
     torch.cuda.set_device(dev)
     K.load()
-    vocab, layers, chunk = 32000, args.layers or 8, 8192
+    vocab, layers, span = 32000, args.layers or 8, 1024 if kipedra else 8192
+    name, other = ("kipedra", "fuzuvik") if kipedra else ("fuzuvik", "llama")
     sampler = clock_sampler(0)
     sampler.start()
     sizes = {}
     prefills, decodes = [(4, 2048), (1, 8192)], [(16, 2048), (256, 2048)]
     for width in (2048, 4096):
-        K.LAUNCHES = 0
-        sizes[str(width)] = {
-            "fuzuvik": model_rates(fuzuvik_like(width, layers, vocab, chunk), dev, vocab, prefills, decodes, args.steps, args.warmup),
-            "llama": model_rates(llama_like(width, layers, vocab), dev, vocab, prefills, decodes, args.steps, args.warmup)}
-    rows = kernel_rows(dev, 4096, chunk, (4, 2048), (256, 2048))
+        cfgs = {name: (kipedra_like if kipedra else fuzuvik_like)(width, layers, vocab, span),
+                other: fuzuvik_twin(width, layers, vocab, span) if kipedra else llama_like(width, layers, vocab)}
+        sizes[str(width)] = {k: model_rates(c, dev, vocab, prefills, decodes, args.steps, args.warmup) for k, c in cfgs.items()}
+    rows = (kipedra_rows if kipedra else kernel_rows)(dev, 4096, span, (4, 2048), (256, 2048))
     clocks = sampler.stop()
-    value = sizes["4096"]["fuzuvik"]["decode_tok_s"]["256@2048"]
+    value = sizes["4096"][name]["decode_tok_s"]["256@2048"]
     print(json.dumps({
-        "metric": "output tok/s (decode, fuzuvik-bf16)", "value": value, "unit": "tok/s", "n_gpus": 1, "steps": args.steps,
+        "metric": f"output tok/s (decode, {args.model})", "value": value, "unit": "tok/s", "n_gpus": 1, "steps": args.steps,
         "warmup": args.warmup, "ms_per_step": round(256e3 / value, 4), "higher_is_better": True, "scaling": "strong",
         "vs_baseline": None, "dtype": "bf16", "data": "synthetic: random tokens, random weights", "impl": "b200",
-        "config": {"model": f"fuzuvik-{layers}L", "global_batch": 256, "seq_len": 2048, "chunk": chunk, "parallelism": "tp1",
-                   "l2": "models: inputs larger than L2; kernels: L2 flushed before every launch"},
+        "config": {"model": f"{name}-{layers}L", "global_batch": 256, "seq_len": 2048, "window" if kipedra else "chunk": span,
+                   "parallelism": "tp1", "l2": "models: inputs larger than L2; kernels: L2 flushed before every launch"},
         "sizes": sizes, "kernels": rows, "peaks": peaks()[2], "clocks": clocks}), flush=True)
     return 0

@@ -70,6 +70,7 @@ __device__ __forceinline__ float silu_t<float>(float x) { return silu_f(x); }
 
 // sequence that owns token t (cu[0] = 0 .. cu[B] = T)
 __device__ __forceinline__ int sequence_of(const int* __restrict__ cu, int B, int t) {
+  if (t < B && cu[t] <= t && cu[t + 1] > t) return t;       // one token per sequence up to here: decode steps
   int lo = 0, hi = B - 1;
   while (lo < hi) {
     const int mid = (lo + hi + 1) >> 1;
@@ -536,7 +537,32 @@ attn_conv_run_kernel(const T* __restrict__ proj, long long ld, int off_k, int of
     old = cv.kv_lens[b] - n > 0 ? st : nullptr;
   };
   enter();
-  auto emit = [&](int t, float4 (&a)[E]) {
+  // where a row goes and its angles: loaded before the row's channels are needed
+  struct Target {
+    T* dst;                                                // null: nowhere
+    float2 c[E], s[E];
+  };
+  auto target = [&](int t) {
+    Target r;
+    const long long slot = slots[t];
+    const bool to = on && (is_q || (slot >= 0 && slot < num_slots));
+    r.dst = !to ? nullptr : is_q ? q_out + (static_cast<size_t>(t) * Hq + g) * Dk
+                          : is_v ? v_cache + (static_cast<size_t>(slot) * Hkv + g) * Dv
+                                 : k_cache + (static_cast<size_t>(slot) * Hkv + g) * Dk;
+    const float* cs = cos_sin + static_cast<size_t>(min(max(positions[t], 0), max_pos - 1)) * rot;
+#pragma unroll
+    for (int e = 0; e < E; ++e) {
+      const int i = 4 * (l + L * e);
+      r.c[e] = make_float2(1.f, 1.f);
+      r.s[e] = make_float2(0.f, 0.f);
+      if (to && !is_v && i < rot) {
+        r.c[e] = *reinterpret_cast<const float2*>(cs + i / 2);
+        r.s[e] = *reinterpret_cast<const float2*>(cs + rh + i / 2);
+      }
+    }
+    return r;
+  };
+  auto emit = [&](const Target& r, const float4 (&a)[E]) {
     float inv = 1.f;
     if (qk_norm) {                                         // a rotation keeps the sum of squares
       float ss = 0.f;
@@ -546,26 +572,17 @@ attn_conv_run_kernel(const T* __restrict__ proj, long long ld, int off_k, int of
       for (int o = L / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
       if (!is_v) inv = 1.f / sqrtf(ss / dim + eps);
     }
-    if (!on) return;
-    const long long slot = slots[t];
-    if (!is_q && (slot < 0 || slot >= num_slots)) return;
-    T* dst = is_q ? q_out + (static_cast<size_t>(t) * Hq + g) * Dk
-                  : (is_v ? v_cache + (static_cast<size_t>(slot) * Hkv + g) * Dv
-                          : k_cache + (static_cast<size_t>(slot) * Hkv + g) * Dk);
-    const float* cs = cos_sin + static_cast<size_t>(min(max(positions[t], 0), max_pos - 1)) * rot;
+    if (r.dst == nullptr) return;
 #pragma unroll
     for (int e = 0; e < E; ++e) {
       const int i = 4 * (l + L * e);
       if (!ok[e]) {
-        if (is_q && i < Dk) store4(dst + i, make_float4(0.f, 0.f, 0.f, 0.f));
+        if (is_q && i < Dk) store4(r.dst + i, make_float4(0.f, 0.f, 0.f, 0.f));
         continue;
       }
-      float4 x = a[e];
-      if (!is_v && i < rot) {
-        const float2 c = *reinterpret_cast<const float2*>(cs + i / 2), s = *reinterpret_cast<const float2*>(cs + rh + i / 2);
-        x = make_float4(x.x * c.x - x.y * s.x, x.y * c.x + x.x * s.x, x.z * c.y - x.w * s.y, x.w * c.y + x.z * s.y);
-      }
-      store4(dst + i, make_float4(x.x * inv, x.y * inv, x.z * inv, x.w * inv));
+      const float4 x = a[e];
+      store4(r.dst + i, make_float4((x.x * r.c[e].x - x.y * r.s[e].x) * inv, (x.y * r.c[e].x + x.x * r.s[e].x) * inv,
+                                    (x.z * r.c[e].y - x.w * r.s[e].y) * inv, (x.w * r.c[e].y + x.z * r.s[e].y) * inv));
     }
   };
   for (int t = t0; t < t1;) {
@@ -578,6 +595,9 @@ attn_conv_run_kernel(const T* __restrict__ proj, long long ld, int off_k, int of
     const T* row = proj + static_cast<size_t>(t) * ld + col;
     if (RB > 1 && local >= TAPS - 1 && t + RB <= min(t1, end)) {
       float4 x[E][TAPS - 1 + RB];
+      Target to[RB];
+#pragma unroll
+      for (int r = 0; r < RB; ++r) to[r] = target(t + r);
 #pragma unroll
       for (int e = 0; e < E; ++e)
 #pragma unroll
@@ -588,11 +608,12 @@ attn_conv_run_kernel(const T* __restrict__ proj, long long ld, int off_k, int of
         float4 a[E];
 #pragma unroll
         for (int e = 0; e < E; ++e) a[e] = wt[e].sum(&x[e][r]);
-        emit(t + r, a);
+        emit(to[r], a);
       }
       t += RB;
       continue;
     }
+    const Target to = target(t);
     float4 a[E];
 #pragma unroll
     for (int e = 0; e < E; ++e) {
@@ -603,7 +624,7 @@ attn_conv_run_kernel(const T* __restrict__ proj, long long ld, int off_k, int of
       // run == 1: these lanes alone read and write these channels' state
       if (cv.update && st != nullptr) wt[e].save(x, st + chan + i, cv.C, cv.taps, ok[e]);
     }
-    emit(t, a);
+    emit(to, a);
     ++t;
   }
 }
@@ -957,6 +978,161 @@ delta_prep_run_kernel(const T* __restrict__ proj, const T* __restrict__ a_pre, c
 }
 
 // ------------------------------------------------------------------------------------------------
+// Prompts with up to four taps and heads of 32, 64 or 128: a CTA convolves 32 rows of 256 neighbouring channels (heads of
+// one kind: q, k or v), brought to shared memory with the three rows before them.  A thread owns four channels of eight
+// consecutive rows.  ATTN: attention inputs as attn_conv_run_kernel writes them, otherwise those of a delta rule.
+// grid (row tiles, channel tiles of q, then k, then v)
+// ------------------------------------------------------------------------------------------------
+constexpr int kTileRows = 32, kTileCols = 256;
+struct ConvTile {
+  long long ld;
+  int T, off[3], heads[3], width[3];       // of q, k, v
+  // attention
+  const int *positions, *page_slots;
+  const float* cos_sin;
+  void *q_out, *k_cache, *v_cache;
+  long long num_pages;                     // token slots of the pools
+  int rot, max_pos, qk_norm, Dk, Dv;
+  float eps;
+  // delta rule
+  float *q, *k, *v, *g, *beta;
+  const void* a_pre;
+  long long ld_a;
+  const float *A_log, *dt_bias;
+  int off_b, head_decay;
+};
+
+template <typename T, bool ATTN>
+__global__ void __launch_bounds__(256, 3)
+conv_tile_kernel(const T* __restrict__ proj, ConvTile p, ConvPast cv) {
+  tgi::pdl_wait();
+  tgi::pdl_trigger();
+  constexpr int TAPS = 4, HALO = TAPS - 1, PER = 16 / sizeof(T);      // elements of a 16-byte piece
+  __shared__ __align__(16) T tile[kTileRows + HALO][kTileCols];
+  __shared__ int s_local[kTileRows], s_old[kTileRows];                // place in its sequence; state slot with a past, or -1
+  __shared__ long long s_page[ATTN ? kTileRows : 1];
+  __shared__ int s_pos[ATTN ? kTileRows : 1];
+  const int t0 = blockIdx.x * kTileRows;
+  // which channels: kind (0 q, 1 k, 2 v) and first column inside it
+  int kind = 0, first = blockIdx.y * kTileCols, chan0 = 0;
+  while (kind < 2 && first >= (p.heads[kind] * p.width[kind] + kTileCols - 1) / kTileCols * kTileCols) {
+    first -= (p.heads[kind] * p.width[kind] + kTileCols - 1) / kTileCols * kTileCols;
+    chan0 += p.heads[kind] * p.width[kind];
+    ++kind;
+  }
+  const int width = p.width[kind], cols = min(kTileCols, p.heads[kind] * width - first);
+  const T* src = proj + p.off[kind] + first;
+  for (int i = threadIdx.x; i < (kTileRows + HALO) * (kTileCols / PER); i += 256) {
+    const int r = i / (kTileCols / PER), c = i % (kTileCols / PER) * PER, t = t0 + r - HALO;
+    const bool in = t >= 0 && t < p.T && c < cols;
+    const uint32_t dst = static_cast<uint32_t>(__cvta_generic_to_shared(&tile[r][c]));
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(in ? src + static_cast<size_t>(t) * p.ld + c : src),
+                 "r"(in ? 16 : 0)
+                 : "memory");
+  }
+  asm volatile("cp.async.commit_group;" ::: "memory");
+  if (threadIdx.x < kTileRows && t0 + threadIdx.x < p.T) {
+    const int t = t0 + threadIdx.x, b = sequence_of(cv.cu, cv.B, t), begin = cv.cu[b], slot = cv.slots[b];
+    s_local[threadIdx.x] = t - begin;
+    s_old[threadIdx.x] = cv.kv_lens[b] - (cv.cu[b + 1] - begin) > 0 && slot >= 0 && slot < cv.num_slots ? slot : -1;
+    if (ATTN) {
+      s_page[threadIdx.x] = p.page_slots[t];
+      s_pos[threadIdx.x] = min(max(p.positions[t], 0), p.max_pos - 1);
+    }
+  }
+  const int c = threadIdx.x % 64 * 4, r0 = threadIdx.x / 64 * 8;
+  const bool on = c < cols;
+  const int chan = chan0 + first + c, h = (first + c) / width, i = (first + c) % width, lanes = width / 4;
+  ShortConv<T, TAPS> wt;
+  wt.weights(cv.w, cv.C, chan, on);
+  float rate = 0.f, bias = 0.f;
+  const bool decays = !ATTN && kind == 2 && p.head_decay && on && i == 0;
+  if (decays) {
+    rate = expf(p.A_log[h]);
+    bias = p.dt_bias[h];
+  }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  __syncthreads();
+#pragma unroll 1
+  for (int r = r0; r < r0 + 8; r += 4) {
+    float4 x[4 + HALO];
+#pragma unroll
+    for (int e = 0; e < 4 + HALO; ++e) x[e] = load4(&tile[r + e][c]);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int t = t0 + r + e;
+      if (t >= p.T) return;                                             // the same for the whole warp
+      const int local = s_local[r + e];
+      float4 y;
+      if (local >= HALO) {
+        y = wt.sum(&x[e]);
+      } else {                                                          // the first rows of a sequence
+        float4 in[TAPS];
+        const int old = s_old[r + e];
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) {
+          const int back = HALO - j, at = cv.taps - 1 + local - back;
+          in[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+          if (local >= back) in[j] = x[e + j];
+          else if (old >= 0 && at >= 0 && on)
+            in[j] = load4(static_cast<const T*>(cv.state) + (static_cast<size_t>(old) * (cv.taps - 1) + at) * cv.C + chan);
+        }
+        y = wt.sum(in);
+      }
+      if (!ATTN) y = make_float4(silu_t<T>(y.x), silu_t<T>(y.y), silu_t<T>(y.z), silu_t<T>(y.w));
+      float inv = 1.f;
+      if (kind < 2 && (!ATTN || p.qk_norm)) {                           // a rotation keeps the sum of squares
+        float ss = y.x * y.x + y.y * y.y + y.z * y.z + y.w * y.w;
+        for (int o = lanes / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        if (ATTN) inv = 1.f / sqrtf(ss / width + p.eps);
+        else inv = 1.f / (sqrtf(ss + 1e-6f) * (kind == 0 ? sqrtf(static_cast<float>(width)) : 1.f));
+      }
+      if (!on) continue;
+      if (ATTN) {
+        if (kind < 2 && i < p.rot) {
+          const float* cs = p.cos_sin + static_cast<size_t>(s_pos[r + e]) * p.rot + i / 2;
+          const float2 co = *reinterpret_cast<const float2*>(cs), si = *reinterpret_cast<const float2*>(cs + p.rot / 2);
+          y = make_float4(y.x * co.x - y.y * si.x, y.y * co.x + y.x * si.x, y.z * co.y - y.w * si.y, y.w * co.y + y.z * si.y);
+        }
+        const long long page = s_page[r + e];
+        T* dst;
+        if (kind == 0) {
+          dst = static_cast<T*>(p.q_out) + (static_cast<size_t>(t) * p.heads[0] + h) * p.Dk + i;
+        } else {
+          if (page < 0 || page >= p.num_pages) continue;
+          dst = (kind == 1 ? static_cast<T*>(p.k_cache) + (static_cast<size_t>(page) * p.heads[1] + h) * p.Dk
+                           : static_cast<T*>(p.v_cache) + (static_cast<size_t>(page) * p.heads[2] + h) * p.Dv) + i;
+        }
+        store4(dst, make_float4(y.x * inv, y.y * inv, y.z * inv, y.w * inv));
+      } else {
+        float* dst = kind == 0 ? p.q : (kind == 1 ? p.k : p.v);
+        store4(dst + (static_cast<size_t>(t) * p.heads[kind] + h) * width + i, make_float4(y.x * inv, y.y * inv, y.z * inv, y.w * inv));
+        if (kind == 2 && i == 0) {
+          const size_t th = static_cast<size_t>(t) * p.heads[2] + h;
+          p.beta[th] = sigmoid_f(to_f(proj[static_cast<size_t>(t) * p.ld + p.off_b + h]));
+          if (decays) p.g[th] = decay_value(to_f(static_cast<const T*>(p.a_pre)[static_cast<size_t>(t) * p.ld_a + h]) + bias, rate);
+        }
+      }
+    }
+  }
+}
+
+// shapes conv_tile_kernel takes
+template <typename T>
+bool conv_tiles(const T* proj, long long ld, const int (&off)[3], int dim, int vdim, int taps) {
+  constexpr int PER = 16 / sizeof(T);
+  auto fits = [](int w) { return w == 32 || w == 64 || w == 128; };
+  return taps <= 4 && fits(dim) && fits(vdim) && ld % PER == 0 && off[0] % PER == 0 && off[1] % PER == 0 && off[2] % PER == 0 &&
+         reinterpret_cast<uintptr_t>(proj) % 16 == 0;
+}
+template <typename T, bool ATTN>
+void launch_conv_tiles(const T* proj, const ConvTile& p, const ConvPast& cv, cudaStream_t stream) {
+  int tiles = 0;
+  for (int i = 0; i < 3; ++i) tiles += (p.heads[i] * p.width[i] + kTileCols - 1) / kTileCols;
+  tgi::launch(conv_tile_kernel<T, ATTN>, dim3((p.T + kTileRows - 1) / kTileRows, tiles), dim3(256), 0, stream, proj, p, cv);
+}
+
+// ------------------------------------------------------------------------------------------------
 // out = RMSNorm(o over `width`) * weight * sigmoid(gate) (SILU: silu(gate)).  o fp32 [T, groups, width]; gate at column `off` of a
 // [T, ld] matrix; out rows are `ld_out` wide, columns past groups * width are zeroed by group 0.
 // One warp (width <= 1024) or one block per (token, group); grid (tokens, groups / warps of a block).
@@ -1093,6 +1269,16 @@ int delta_prep(const void* proj, const void* a_pre, const float* conv_t, const f
     if (p.update) {
       if (p.taps <= 4) one ? go(delta_prep_run_kernel<T, 1, 4, 0, 1>, units, 1) : go(delta_prep_run_kernel<T, 2, 4, 0, 1>, units, 1);
       else one ? go(delta_prep_run_kernel<T, 1, 8, 0, 1>, units, 1) : go(delta_prep_run_kernel<T, 2, 8, 0, 1>, units, 1);
+    } else if (p.dimP == p.dim && conv_tiles<T>(x, p.ld, {p.off_q, p.off_k, p.off_v}, p.dim, p.vdim, p.taps)) {
+      ConvTile c{};
+      c.ld = p.ld; c.T = T_; c.off_b = p.off_b; c.head_decay = p.head_decay;
+      c.off[0] = p.off_q; c.off[1] = p.off_k; c.off[2] = p.off_v;
+      c.heads[0] = c.heads[1] = p.G; c.heads[2] = p.H;
+      c.width[0] = c.width[1] = p.dim; c.width[2] = p.vdim;
+      c.q = q; c.k = k; c.v = v; c.g = g; c.beta = beta;
+      c.a_pre = a_pre; c.ld_a = p.ld_a; c.A_log = A_log; c.dt_bias = dt_bias;
+      launch_conv_tiles<T, false>(x, c, ConvPast{conv_t, cu, kv, slots, conv_state, p.B, p.taps, C, num_slots, 0}, stream);
+      if (!p.head_decay) go(delta_prep_run_kernel<T, 1, 4, 3, 1>, p.H, 16);
     } else if (p.taps <= 4 && one) {
       go(delta_prep_run_kernel<T, 1, 4, 1, 2>, p.G, 16);
       go(delta_prep_run_kernel<T, 1, 4, 2, 4>, p.H, 32);
@@ -1216,6 +1402,19 @@ int tgi_attn_prep(int f32, const void* proj, long long ld, int off_k, int off_v,
     };
     auto shape = [&](auto tag) {
       using E = decltype(tag);
+      const E* x = static_cast<const E*>(proj);
+      if (!update && Dk == dim && conv_tiles<E>(x, ld, {0, off_k, off_v}, dim, vdim, taps)) {
+        ConvTile c{};
+        c.ld = ld; c.T = T;
+        c.off[1] = off_k; c.off[2] = off_v;
+        c.heads[0] = Hq; c.heads[1] = c.heads[2] = Hkv;
+        c.width[0] = c.width[1] = dim; c.width[2] = vdim;
+        c.positions = positions; c.page_slots = slots; c.cos_sin = cos_sin;
+        c.q_out = q_out; c.k_cache = k_cache; c.v_cache = v_cache; c.num_pages = num_slots;
+        c.rot = rot; c.max_pos = max_pos; c.qk_norm = qk_norm; c.Dk = Dk; c.Dv = Dv; c.eps = eps;
+        launch_conv_tiles<E, true>(x, c, cv, stream);
+        return;
+      }
       const int w = Dk > vdim ? Dk : vdim;                 // the columns past `dim` of q_out are written too
       if (taps <= 4) {
         if (update) {

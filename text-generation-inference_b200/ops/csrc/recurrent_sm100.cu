@@ -95,6 +95,15 @@ __device__ __forceinline__ pair mul2(pair a, pair b) {
   return r;
 }
 
+// A second read of shared memory that the compiler must not replace by keeping the first one in registers
+__device__ __forceinline__ ulonglong2 reread(const float* p) {
+  ulonglong2 v;
+  asm volatile("ld.volatile.shared.v2.u64 {%0, %1}, [%2];"
+               : "=l"(v.x), "=l"(v.y)
+               : "r"(static_cast<uint32_t>(__cvta_generic_to_shared(p))));
+  return v;
+}
+
 // Sums of CN values over L lanes; lane l ends with the total of value l / (L / CN).
 template <int CN, int L>
 __device__ __forceinline__ float scatter_sum(float (&v)[CN], int l) {
@@ -476,7 +485,8 @@ scan_kernel(ScanArgs p) {
         }
 #pragma unroll
         for (int j = 0; j < NQ; ++j) {
-          const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(r + (S::kEnd + e) * S::kRow + 4 * L * j);
+          const float* kp = r + (S::kEnd + e) * S::kRow + 4 * L * j;
+          const ulonglong2 k = HEAD ? reread(kp) : *reinterpret_cast<const ulonglong2*>(kp);
 #pragma unroll
           for (int c = 0; c < CN; ++c) {
             s[c][j][0] = fma2(k.x, u2[c], s[c][j][0]);
