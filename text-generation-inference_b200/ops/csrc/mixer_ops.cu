@@ -14,6 +14,8 @@
 #include <cuda_runtime.h>
 #include <stdint.h>
 
+#include <type_traits>
+
 #include "launch.cuh"
 
 namespace {
@@ -979,9 +981,9 @@ delta_prep_run_kernel(const T* __restrict__ proj, const T* __restrict__ a_pre, c
 
 // ------------------------------------------------------------------------------------------------
 // Prompts with up to four taps and heads of 32, 64 or 128: a CTA convolves 32 rows of 256 neighbouring channels (heads of
-// one kind: q, k or v), brought to shared memory with the three rows before them.  A thread owns four channels of eight
-// consecutive rows.  ATTN: attention inputs as attn_conv_run_kernel writes them, otherwise those of a delta rule.
-// grid (row tiles, channel tiles of q, then k, then v)
+// one kind: q, k or v), brought to shared memory with the three rows before them.  A lane owns eight channels of four
+// consecutive rows (bound by instructions: 16-byte accesses, packed fp32 multiply-adds).  ATTN: attention inputs as
+// attn_conv_run_kernel writes them, otherwise those of a delta rule.  grid (row tiles, channel tiles of q, then k, then v)
 // ------------------------------------------------------------------------------------------------
 constexpr int kTileRows = 32, kTileCols = 256;
 struct ConvTile {
@@ -1002,16 +1004,59 @@ struct ConvTile {
   int off_b, head_decay;
 };
 
+// eight neighbouring values as four packed pairs
+using pair = unsigned long long;
+struct Oct {
+  pair v[4];
+};
+__device__ __forceinline__ pair pack_pair(float x, float y) {
+  pair r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(x), "f"(y));
+  return r;
+}
+__device__ __forceinline__ float2 unpack_pair(pair p) {
+  float2 r;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(p));
+  return r;
+}
+__device__ __forceinline__ pair fma_pair(pair a, pair b, pair c) {
+  pair r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ Oct load8(const float* p) {
+  const ulonglong2 a = *reinterpret_cast<const ulonglong2*>(p), b = *reinterpret_cast<const ulonglong2*>(p + 4);
+  return Oct{{a.x, a.y, b.x, b.y}};
+}
+__device__ __forceinline__ Oct load8(const bf16* p) {
+  const uint4 u = *reinterpret_cast<const uint4*>(p);
+  auto two = [](uint32_t w) { return pack_pair(__uint_as_float(w << 16), __uint_as_float(w & 0xffff0000u)); };
+  return Oct{{two(u.x), two(u.y), two(u.z), two(u.w)}};
+}
+__device__ __forceinline__ void store8(float* p, const float (&v)[8]) {
+  store4(p, make_float4(v[0], v[1], v[2], v[3]));
+  store4(p + 4, make_float4(v[4], v[5], v[6], v[7]));
+}
+__device__ __forceinline__ void store8(bf16* p, const float (&v)[8]) {
+  uint32_t u[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+    u[i] = *reinterpret_cast<const uint32_t*>(&h);
+  }
+  *reinterpret_cast<uint4*>(p) = make_uint4(u[0], u[1], u[2], u[3]);
+}
+
 template <typename T, bool ATTN>
-__global__ void __launch_bounds__(256, 3)
+__global__ void __launch_bounds__(256, 2)
 conv_tile_kernel(const T* __restrict__ proj, ConvTile p, ConvPast cv) {
   tgi::pdl_wait();
   tgi::pdl_trigger();
   constexpr int TAPS = 4, HALO = TAPS - 1, PER = 16 / sizeof(T);      // elements of a 16-byte piece
+  using Out = typename std::conditional<ATTN, T, float>::type;
   __shared__ __align__(16) T tile[kTileRows + HALO][kTileCols];
   __shared__ int s_local[kTileRows], s_old[kTileRows];                // place in its sequence; state slot with a past, or -1
-  __shared__ long long s_page[ATTN ? kTileRows : 1];
-  __shared__ int s_pos[ATTN ? kTileRows : 1];
+  __shared__ int s_row[kTileRows], s_pos[kTileRows];                  // row it is written to (-1: none), position
   const int t0 = blockIdx.x * kTileRows;
   // which channels: kind (0 q, 1 k, 2 v) and first column inside it
   int kind = 0, first = blockIdx.y * kTileCols, chan0 = 0;
@@ -1020,7 +1065,7 @@ conv_tile_kernel(const T* __restrict__ proj, ConvTile p, ConvPast cv) {
     chan0 += p.heads[kind] * p.width[kind];
     ++kind;
   }
-  const int width = p.width[kind], cols = min(kTileCols, p.heads[kind] * width - first);
+  const int width = p.width[kind], heads = p.heads[kind], cols = min(kTileCols, heads * width - first);
   const T* src = proj + p.off[kind] + first;
   for (int i = threadIdx.x; i < (kTileRows + HALO) * (kTileCols / PER); i += 256) {
     const int r = i / (kTileCols / PER), c = i % (kTileCols / PER) * PER, t = t0 + r - HALO;
@@ -1035,94 +1080,107 @@ conv_tile_kernel(const T* __restrict__ proj, ConvTile p, ConvPast cv) {
     const int t = t0 + threadIdx.x, b = sequence_of(cv.cu, cv.B, t), begin = cv.cu[b], slot = cv.slots[b];
     s_local[threadIdx.x] = t - begin;
     s_old[threadIdx.x] = cv.kv_lens[b] - (cv.cu[b + 1] - begin) > 0 && slot >= 0 && slot < cv.num_slots ? slot : -1;
+    int row = t;
     if (ATTN) {
-      s_page[threadIdx.x] = p.page_slots[t];
       s_pos[threadIdx.x] = min(max(p.positions[t], 0), p.max_pos - 1);
+      if (kind > 0) {
+        const int page = p.page_slots[t];
+        row = page >= 0 && page < p.num_pages ? page : -1;
+      }
     }
+    s_row[threadIdx.x] = row;
   }
-  const int c = threadIdx.x % 64 * 4, r0 = threadIdx.x / 64 * 8;
+  const int lane = threadIdx.x & 31, c = lane * 8, r0 = (threadIdx.x >> 5) * 4;
   const bool on = c < cols;
-  const int chan = chan0 + first + c, h = (first + c) / width, i = (first + c) % width, lanes = width / 4;
-  ShortConv<T, TAPS> wt;
-  wt.weights(cv.w, cv.C, chan, on);
+  const int chan = chan0 + first + c, h = (first + c) / width, i = (first + c) % width, lanes = width / 8;
+  const bool rotate = ATTN && kind < 2 && i < p.rot, normed = kind < 2 && (!ATTN || p.qk_norm);
+  const bool scalars = !ATTN && kind == 2 && on && i == 0, decays = scalars && p.head_decay;
+  Out* const base = static_cast<Out*>(ATTN ? (kind == 0 ? p.q_out : (kind == 1 ? p.k_cache : p.v_cache))
+                                           : static_cast<void*>(kind == 0 ? p.q : (kind == 1 ? p.k : p.v)));
+  const int head_pitch = !ATTN ? width : (kind == 2 ? p.Dv : p.Dk);
+  Out* const dst0 = base + h * head_pitch + i;
+  const size_t pitch = static_cast<size_t>(heads) * head_pitch;
+  Oct w[TAPS];
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j) w[j] = on ? load8(cv.w + static_cast<size_t>(j) * cv.C + chan) : Oct{};
   float rate = 0.f, bias = 0.f;
-  const bool decays = !ATTN && kind == 2 && p.head_decay && on && i == 0;
   if (decays) {
     rate = expf(p.A_log[h]);
     bias = p.dt_bias[h];
   }
   asm volatile("cp.async.wait_group 0;" ::: "memory");
   __syncthreads();
-#pragma unroll 1
-  for (int r = r0; r < r0 + 8; r += 4) {
-    float4 x[4 + HALO];
+  Oct x[4 + HALO];
 #pragma unroll
-    for (int e = 0; e < 4 + HALO; ++e) x[e] = load4(&tile[r + e][c]);
+  for (int e = 0; e < 4 + HALO; ++e) x[e] = load8(&tile[r0 + e][c]);
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int t = t0 + r + e;
-      if (t >= p.T) return;                                             // the same for the whole warp
-      const int local = s_local[r + e];
-      float4 y;
-      if (local >= HALO) {
-        y = wt.sum(&x[e]);
-      } else {                                                          // the first rows of a sequence
-        float4 in[TAPS];
-        const int old = s_old[r + e];
+  for (int e = 0; e < 4; ++e) {
+    const int t = t0 + r0 + e;
+    if (t >= p.T) break;                                              // the same for the whole warp
+    const int local = s_local[r0 + e];
+    pair acc[4] = {};
+    if (local >= HALO) {
 #pragma unroll
-        for (int j = 0; j < TAPS; ++j) {
-          const int back = HALO - j, at = cv.taps - 1 + local - back;
-          in[j] = make_float4(0.f, 0.f, 0.f, 0.f);
-          if (local >= back) in[j] = x[e + j];
-          else if (old >= 0 && at >= 0 && on)
-            in[j] = load4(static_cast<const T*>(cv.state) + (static_cast<size_t>(old) * (cv.taps - 1) + at) * cv.C + chan);
-        }
-        y = wt.sum(in);
+      for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+        for (int q = 0; q < 4; ++q) acc[q] = fma_pair(w[j].v[q], x[e + j].v[q], acc[q]);
+    } else {                                                          // the first rows of a sequence
+      const int old = s_old[r0 + e];
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) {
+        const int back = HALO - j, at = cv.taps - 1 + local - back;
+        Oct in{};
+        if (local >= back) in = x[e + j];
+        else if (old >= 0 && at >= 0 && on)
+          in = load8(static_cast<const T*>(cv.state) + (static_cast<size_t>(old) * (cv.taps - 1) + at) * cv.C + chan);
+#pragma unroll
+        for (int q = 0; q < 4; ++q) acc[q] = fma_pair(w[j].v[q], in.v[q], acc[q]);
       }
-      if (!ATTN) y = make_float4(silu_t<T>(y.x), silu_t<T>(y.y), silu_t<T>(y.z), silu_t<T>(y.w));
-      float inv = 1.f;
-      if (kind < 2 && (!ATTN || p.qk_norm)) {                           // a rotation keeps the sum of squares
-        float ss = y.x * y.x + y.y * y.y + y.z * y.z + y.w * y.w;
-        for (int o = lanes / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-        if (ATTN) inv = 1.f / sqrtf(ss / width + p.eps);
-        else inv = 1.f / (sqrtf(ss + 1e-6f) * (kind == 0 ? sqrtf(static_cast<float>(width)) : 1.f));
+    }
+    float y[8];
+#pragma unroll
+    for (int q = 0; q < 4; ++q) {
+      const float2 f = unpack_pair(acc[q]);
+      y[2 * q] = ATTN ? f.x : silu_t<T>(f.x);
+      y[2 * q + 1] = ATTN ? f.y : silu_t<T>(f.y);
+    }
+    if (normed) {                                                     // a rotation keeps the sum of squares
+      float ss = 0.f;
+#pragma unroll
+      for (int q = 0; q < 8; ++q) ss = fmaf(y[q], y[q], ss);
+      for (int o = lanes / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      const float inv = ATTN ? rsqrtf(ss / width + p.eps) : rsqrtf(ss + 1e-6f) * (kind == 0 ? rsqrtf(static_cast<float>(width)) : 1.f);
+#pragma unroll
+      for (int q = 0; q < 8; ++q) y[q] *= inv;
+    }
+    const int row = s_row[r0 + e];
+    if (!on || row < 0) continue;
+    if (rotate) {
+      const float* cs = p.cos_sin + static_cast<size_t>(s_pos[r0 + e]) * p.rot + i / 2;
+      const float4 co = *reinterpret_cast<const float4*>(cs), si = *reinterpret_cast<const float4*>(cs + p.rot / 2);
+      const float cf[4] = {co.x, co.y, co.z, co.w}, sf[4] = {si.x, si.y, si.z, si.w};
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        const float u = y[2 * q], v = y[2 * q + 1];
+        y[2 * q] = u * cf[q] - v * sf[q];
+        y[2 * q + 1] = v * cf[q] + u * sf[q];
       }
-      if (!on) continue;
-      if (ATTN) {
-        if (kind < 2 && i < p.rot) {
-          const float* cs = p.cos_sin + static_cast<size_t>(s_pos[r + e]) * p.rot + i / 2;
-          const float2 co = *reinterpret_cast<const float2*>(cs), si = *reinterpret_cast<const float2*>(cs + p.rot / 2);
-          y = make_float4(y.x * co.x - y.y * si.x, y.y * co.x + y.x * si.x, y.z * co.y - y.w * si.y, y.w * co.y + y.z * si.y);
-        }
-        const long long page = s_page[r + e];
-        T* dst;
-        if (kind == 0) {
-          dst = static_cast<T*>(p.q_out) + (static_cast<size_t>(t) * p.heads[0] + h) * p.Dk + i;
-        } else {
-          if (page < 0 || page >= p.num_pages) continue;
-          dst = (kind == 1 ? static_cast<T*>(p.k_cache) + (static_cast<size_t>(page) * p.heads[1] + h) * p.Dk
-                           : static_cast<T*>(p.v_cache) + (static_cast<size_t>(page) * p.heads[2] + h) * p.Dv) + i;
-        }
-        store4(dst, make_float4(y.x * inv, y.y * inv, y.z * inv, y.w * inv));
-      } else {
-        float* dst = kind == 0 ? p.q : (kind == 1 ? p.k : p.v);
-        store4(dst + (static_cast<size_t>(t) * p.heads[kind] + h) * width + i, make_float4(y.x * inv, y.y * inv, y.z * inv, y.w * inv));
-        if (kind == 2 && i == 0) {
-          const size_t th = static_cast<size_t>(t) * p.heads[2] + h;
-          p.beta[th] = sigmoid_f(to_f(proj[static_cast<size_t>(t) * p.ld + p.off_b + h]));
-          if (decays) p.g[th] = decay_value(to_f(static_cast<const T*>(p.a_pre)[static_cast<size_t>(t) * p.ld_a + h]) + bias, rate);
-        }
-      }
+    }
+    store8(dst0 + row * pitch, y);
+    if (scalars) {
+      const size_t th = static_cast<size_t>(t) * heads + h;
+      p.beta[th] = sigmoid_f(to_f(proj[static_cast<size_t>(t) * p.ld + p.off_b + h]));
+      if (decays) p.g[th] = decay_value(to_f(static_cast<const T*>(p.a_pre)[static_cast<size_t>(t) * p.ld_a + h]) + bias, rate);
     }
   }
 }
 
 // shapes conv_tile_kernel takes
 template <typename T>
-bool conv_tiles(const T* proj, long long ld, const int (&off)[3], int dim, int vdim, int taps) {
+bool conv_tiles(const T* proj, long long ld, const int (&off)[3], int dim, int vdim, int taps, int rot) {
   constexpr int PER = 16 / sizeof(T);
   auto fits = [](int w) { return w == 32 || w == 64 || w == 128; };
-  return taps <= 4 && fits(dim) && fits(vdim) && ld % PER == 0 && off[0] % PER == 0 && off[1] % PER == 0 && off[2] % PER == 0 &&
+  return taps <= 4 && fits(dim) && fits(vdim) && rot % 8 == 0 && ld % PER == 0 && off[0] % PER == 0 && off[1] % PER == 0 && off[2] % PER == 0 &&
          reinterpret_cast<uintptr_t>(proj) % 16 == 0;
 }
 template <typename T, bool ATTN>
@@ -1269,7 +1327,7 @@ int delta_prep(const void* proj, const void* a_pre, const float* conv_t, const f
     if (p.update) {
       if (p.taps <= 4) one ? go(delta_prep_run_kernel<T, 1, 4, 0, 1>, units, 1) : go(delta_prep_run_kernel<T, 2, 4, 0, 1>, units, 1);
       else one ? go(delta_prep_run_kernel<T, 1, 8, 0, 1>, units, 1) : go(delta_prep_run_kernel<T, 2, 8, 0, 1>, units, 1);
-    } else if (p.dimP == p.dim && conv_tiles<T>(x, p.ld, {p.off_q, p.off_k, p.off_v}, p.dim, p.vdim, p.taps)) {
+    } else if (p.dimP == p.dim && conv_tiles<T>(x, p.ld, {p.off_q, p.off_k, p.off_v}, p.dim, p.vdim, p.taps, 0)) {
       ConvTile c{};
       c.ld = p.ld; c.T = T_; c.off_b = p.off_b; c.head_decay = p.head_decay;
       c.off[0] = p.off_q; c.off[1] = p.off_k; c.off[2] = p.off_v;
@@ -1403,7 +1461,7 @@ int tgi_attn_prep(int f32, const void* proj, long long ld, int off_k, int off_v,
     auto shape = [&](auto tag) {
       using E = decltype(tag);
       const E* x = static_cast<const E*>(proj);
-      if (!update && Dk == dim && conv_tiles<E>(x, ld, {0, off_k, off_v}, dim, vdim, taps)) {
+      if (!update && Dk == dim && Dv % 8 == 0 && num_slots < (1ll << 31) && conv_tiles<E>(x, ld, {0, off_k, off_v}, dim, vdim, taps, rot)) {
         ConvTile c{};
         c.ld = ld; c.T = T;
         c.off[1] = off_k; c.off[2] = off_v;
