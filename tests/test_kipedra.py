@@ -201,6 +201,29 @@ def test_greedy_generation(be, checkpoints, graphs):
     assert runner.state_slots.available == 3
 
 
+@pytest.mark.gpu
+def test_warmup_then_generation(checkpoints, monkeypatch):
+    """The server's start: a first step sizes pages and slots and captures the decode steps; generation on them."""
+    from tgi_b200.models.flash_causal_lm import FlashCausalLMBatch as B
+    from tgi_b200.proto import generate_v3 as pb
+
+    monkeypatch.setenv("CUDA_MEMORY_FRACTION", "0.1")
+    monkeypatch.setenv("CUDA_GRAPHS", "1,2,4")
+    ck = checkpoints("all")
+    if not _SURE:
+        _SURE["all"] = sure_prompts(ck, 3, 30, 6)
+    r = runner_for(ck, (torch.device("cuda"), torch.bfloat16))
+    reqs, _ = requests([tokens(ck[0], 60, 1)], [4])
+    del reqs[0].blocks[:]
+    cap, _, total = r.warmup(B.from_tokenized(pb.Batch(id=0, requests=reqs, size=1), [tokens(ck[0], 60, 1)], r.tokenizer, r.dtype,
+                                              r.device), 64, 96)
+    assert cap >= total == 96 and r.graphs is not None and r.state_slots.available == r.max_batch_size
+    r.init_kv_cache = lambda *a, **k: None       # generate on the cache that was captured
+    cases = _SURE["all"]
+    assert generate(r, [c[0] for c in cases], [6] * 3, late=(2,)) == {i: c[1] for i, c in enumerate(cases)}
+    assert r.state_slots.available == r.max_batch_size
+
+
 def test_attention_layers_alone_still_hold_slots(tmp_path):
     """Short convolutions make a state: an attention-only model has slots, keeps no prefixes, and is not run ahead."""
     from tgi_b200.models import get_model
