@@ -156,6 +156,7 @@ def _check_mixed(model_type: str, dtype: torch.dtype, device: torch.device, quan
         raise NotImplementedError(f"{model_type}: serving dtypes are bfloat16 and float32")
     if dtype == torch.float32:
         torch.backends.cuda.matmul.allow_tf32 = False        # fp32 products are true fp32
+    torch.backends.cuda.matmul.allow_bf16_reduced_precision_reduction = False      # library products sum in fp32
 
 
 def _max_positions(cfg: ModelConfig, max_input_tokens: Optional[int]) -> int:

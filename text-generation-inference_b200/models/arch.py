@@ -104,8 +104,58 @@ def _kipedra_config(d: Dict[str, Any]) -> Dict[str, Any]:
     return out
 
 
+def _gisilix_config(d: Dict[str, Any]) -> Dict[str, Any]:
+    """Gisilix checkpoints: layers described one by one as in Fuzuvik's; attention over latents, attention with learned sinks
+    whose keys and values other layers may share, softmax-routed gated experts beside a shared one."""
+    out = dict(d)
+    layers = d["layers"]
+    specs = []
+    for i, layer in enumerate(layers):
+        m, mlp = layer["mixer"], layer.get("mlp")
+        ff, moe = 0, None
+        if mlp is not None and mlp["kind"] == "dense":
+            ff = int(mlp["ff"])
+        elif mlp is not None and mlp["kind"] == "moe":
+            r = mlp["router"]
+            moe = ExpertSpec(experts=int(r["experts"]), top=int(r["top"]), ff=int(mlp["expert"]["ff"]), act="silu", gated=True,
+                             router="softmax", shared_ff=int((mlp.get("shared") or {}).get("ff") or 0))
+        elif mlp is not None:
+            raise NotImplementedError(f"layer {i}: feed-forward kind {mlp['kind']!r}")
+        sizes = dict(heads=int(m["heads"]), kv_heads=int(m.get("kv_heads") or m["heads"]), dim=int(m["dim"]),
+                     vdim=int(m["vdim"]), ff=ff, moe=moe, scale=float(m["scale"]),
+                     window=int((m.get("mask") or {}).get("size") or 0))
+        if layer["type"] == "attention":
+            temp, src = m.get("q_temp"), m.get("kv_from")
+            specs.append(MixerSpec(
+                "attention", **sizes, row_norm=True, softcap=float(m.get("softcap") or 0.0), learned_sink=True,
+                q_temp=None if not temp else (float(temp["coef"]), int(temp["every"])), out_gate="element",
+                kv_from=None if src is None else int(src)))
+        elif layer["type"] in ("latent_attention", "latent_attention_2"):
+            rotated = layer["type"] == "latent_attention_2"
+            rot = (m.get("rot") or {}) if rotated else {}
+            sc = rot.get("scaling")
+            specs.append(MixerSpec(
+                "latent", **{**sizes, "kv_heads": 1}, kv_rank=int(m["kv_rank"]), rot_dims=int(m.get("rot_dim") or 0) if rotated else 0,
+                rot_base=float(rot.get("base") or 10000.0), rot_interleaved=True,
+                rot_yarn=None if not sc else tuple(float(sc[k]) for k in ("factor", "fast", "slow", "original")),
+                out_gate="head" if rotated else ""))
+        else:
+            raise NotImplementedError(f"layer {i}: mixer {layer['type']!r}")
+    for i, s in enumerate(specs):
+        if s.kv_from is not None:
+            src = specs[s.kv_from] if 0 <= s.kv_from < i else None
+            if src is None or src.kind != "attention" or src.kv_from is not None or (src.kv_heads, src.dim, src.vdim) != (s.kv_heads, s.dim, s.vdim):
+                raise ValueError(f"layer {i} cannot use the keys and values of layer {s.kv_from}")
+    out.update(model_type="gisilix", hidden_size=int(d["width"]), vocab_size=int(d["vocab"]), num_hidden_layers=len(layers),
+               num_attention_heads=max(s.heads for s in specs), rms_norm_eps=float(d["norm"]["eps"]), mixers=specs,
+               tie_word_embeddings=True,
+               # rotary positions are unbounded by design: the table length is a deployment choice
+               max_position_embeddings=int(d.get("max_position_embeddings") or 131072))
+    return out
+
+
 # ``architecture`` of a config.json without ``model_type`` -> function that brings it to the common names
-CONFIG_READERS = {"Fuzuvik": _fuzuvik_config, "Kipedra": _kipedra_config}
+CONFIG_READERS = {"Fuzuvik": _fuzuvik_config, "Kipedra": _kipedra_config, "Gisilix": _gisilix_config}
 
 
 class ModelConfig:
@@ -149,21 +199,28 @@ class ModelConfig:
 
 @dataclass(frozen=True)
 class ExpertSpec:
-    """Routed feed-forward of one layer: ungated experts (``down(act(up(h)))``) chosen by the sigmoid of their router
-    logits plus a stored correction, weighted by the sigmoids alone, which are brought to the sum ``scale``."""
+    """Routed feed-forward of one layer: experts ``down(act(up(h)))``, or ``down(act(gate(h)) * up(h))`` when ``gated``.
+
+    ``router="sigmoid"``: chosen by the sigmoid of their router logits plus a stored correction, weighted by the sigmoids
+    alone, which are brought to the sum ``scale``.  ``router="softmax"``: chosen by their router logits, stored bias included,
+    weighted by the softmax over the chosen logits."""
 
     experts: int
     top: int                                 # experts per token
     ff: int                                  # width of an expert
     scale: float = 1.0
     act: str = "relu2"
+    gated: bool = False
+    router: str = "sigmoid"
+    shared_ff: int = 0                       # width of a feed-forward that every token runs beside its experts, 0: none
 
 
 @dataclass(frozen=True)
 class MixerSpec:
     """Token mixer and feed-forward of one layer of a decoder whose layers differ (``models/mixers.py``)."""
 
-    kind: str                                # "attention" | "delta" (gated delta rule) | "decay" (fixed decay per head)
+    kind: str                                # "attention" | "latent" (attention over a latent that all heads share) |
+                                             # "delta" (gated delta rule) | "decay" (fixed decay per head)
     heads: int
     kv_heads: int                            # attention: key/value heads; delta: query/key heads
     dim: int                                 # query / key size of a head
@@ -171,16 +228,24 @@ class MixerSpec:
     ff: int = 0                              # width of a dense feed-forward, 0: the layer has none
     moe: Optional[ExpertSpec] = None         # routed experts in its place
     short_conv: bool = False                 # causal convolution over time on every channel of q, k and v
-    # attention
+    # attention, latent
     scale: float = 1.0
     window: int = 0                          # > 0: the token itself and the window - 1 tokens before it
     chunk: int = 0                           # > 0: keys of the query's own chunk of this many positions
     sink: bool = False                       # one more key of score 0, without a value, in the softmax
+    learned_sink: bool = False               # the same with a stored score per head
+    softcap: float = 0.0                     # > 0: scores become softcap * tanh(score / softcap)
     qk_unit_rms: bool = False                # q and k over their root mean square, after the rotation
+    row_norm: bool = False                   # q and k normed over all heads at once, with weights (no rotation)
+    q_temp: Optional[Tuple[float, int]] = None    # (coef, every): q times 1 + coef * ln(floor((p + 1) / every) + 1)
+    out_gate: str = ""                       # output times the sigmoid of a projection: "element" | "head" (one per head)
+    kv_from: Optional[int] = None            # layer whose keys and values this one reads
+    kv_rank: int = 0                         # latent: its size
     v_mix: bool = False                      # values mixed with those of the first such layer
     rot_dims: int = 0
     rot_base: float = 10000.0
     rot_scaling: Optional[Tuple[float, float, float, float]] = None    # (factor, low, high, original length)
+    rot_yarn: Optional[Tuple[float, float, float, float]] = None       # (factor, fast, slow, original length)
     rot_interleaved: bool = False            # pairs 2i, 2i + 1 (False: i, i + rot_dims / 2)
     qkv_bias: bool = False
     # delta
@@ -192,13 +257,13 @@ class MixerSpec:
 
     @property
     def paged(self) -> bool:
-        """Keeps keys and values of every token."""
-        return self.kind == "attention"
+        """Keeps something of every token: keys and values, or what they are made from."""
+        return self.kind in ("attention", "latent")
 
     @property
     def recurrent(self) -> bool:
         """Keeps a state per sequence that every token advances."""
-        return self.kind != "attention" or self.short_conv
+        return not self.paged or self.short_conv
 
     @property
     def feed_forward(self) -> bool:
@@ -260,11 +325,11 @@ class Arch:
     mla: bool = False                        # DeepSeek multi-head latent attention (models/deepseek.py)
     moe_shared_gate: Optional[str] = None
     moe_renormalize: bool = True
-    moe_correction: Optional[str] = None     # correction of the choice scores (layers with an `ExpertSpec`)
+    moe_correction: Optional[str] = None     # correction of the choice scores, or bias of the logits (layers with an `ExpertSpec`)
     # ---- layers that differ (config "mixers") ---------------------------------------------------
     mix: Optional[str] = None                # tensor prefix of a layer's mixer
     residual_fp32: bool = False              # the residual stream is kept in 32 bits
-    bare_names: bool = False                 # tensors are named without the ".weight" suffix
+    bare_names: bool = False                 # tensors are named without the ".weight" suffix, biases end in ".b"
 
 
 _LLAMA = Arch()
@@ -355,6 +420,10 @@ ARCHS["kipedra"] = Arch(embed="embed", layer="l{i}", norm1="norm1", norm2="norm2
                         norm_unit_offset=True, parallel_residual=True, parallel_shared_norm=False, residual_fp32=True,
                         bare_names=True, moe_router="mlp.router", moe_expert="mlp.e{e}", moe_up="up", moe_down="down",
                         moe_correction="mlp.correction")
+ARCHS["gisilix"] = Arch(embed="embed", layer="l{i}", norm1="norm1", norm2="norm2", final_norm="final.norm", lm_head="head",
+                        mix="mix", gate="mlp.gate", up="mlp.up", down="mlp.down", act="silu", rope=False, norm="layer",
+                        residual_fp32=True, bare_names=True, moe_router="mlp.router", moe_expert="mlp.e{e}", moe_gate="gate",
+                        moe_up="up", moe_down="down", moe_correction="mlp.router.b", moe_shared="mlp.shared")
 ARCHS["gemma3"] = ARCHS["gemma3_text"]
 ARCHS["phi-msft"] = ARCHS["phi"]
 ARCHS["qwen2_vl_text"] = ARCHS["qwen2_5_vl_text"] = ARCHS["qwen2"]   # language models of Qwen2-VL / Qwen2.5-VL

@@ -77,7 +77,7 @@ class Norm:
             # `x` is the last block's output, a pair of outputs or None (nothing to add); `rows` ends the stream: only
             # these rows are normed
             return ops.residual_norm(x, residual, self.weight, self.eps, rows, keep=rows is None, scale=self.residual_scale,
-                                     unit_offset=self.unit_offset)
+                                     unit_offset=self.unit_offset, layer=self.kind == "layer", bias=self.bias)
         if self.kind == "rms":
             return ops.rms_norm(x, residual, self.weight, self.eps, self.unit_offset)
         return ops.layer_norm(x, residual, self.weight, self.bias, self.eps)
@@ -362,7 +362,8 @@ class SparseMoE:
     (what the reference does, ``layers/moe/unquantized.py:107-163``); expert-parallel mode
     (``parallel/expert.py``) places whole experts on ranks.  Either way a rank ends up with a partial
     ``[T, H]`` output that is summed over ranks by the layer's reduction.  With an ``ExpertSpec`` the layer has its own
-    expert count and sizes, ungated experts and a router in 32 bits (sigmoid scores, corrected choice)."""
+    expert count and sizes, gated or ungated experts and a router in 32 bits; with a shared feed-forward beside them it
+    returns the pair (routed, shared) for the next norm to add to the fp32 stream."""
 
     def __init__(self, arch: Arch, cfg, dims: ModelDims, prefix: str, weights, comm, spec: Optional[ExpertSpec] = None):
         pg = weights.process_group
@@ -371,7 +372,7 @@ class SparseMoE:
         self.renorm = arch.moe_renormalize if cfg.get("norm_topk_prob") is None else bool(cfg.norm_topk_prob)
         self.router = FastLinear(weights.get_tensor(f"{prefix}.{arch.moe_router}.weight"))
         if spec is not None:
-            self._load_plain_experts(arch, cfg, prefix, weights, spec)
+            self._load_spec(arch, cfg, dims, prefix, weights, comm, spec)
             return
         self.sparsemixer_eps = float(cfg.get("router_jitter_noise", 0.01)) if cfg.model_type == "phimoe" else None
         self.deepseek_router = None
@@ -422,24 +423,33 @@ class SparseMoE:
             if arch.moe_shared_gate and weights.has_tensor(f"{prefix}.{arch.moe_shared_gate}.weight"):
                 self.shared_gate = FastLinear(weights.get_tensor(f"{prefix}.{arch.moe_shared_gate}.weight"))
 
-    def _load_plain_experts(self, arch: Arch, cfg, prefix: str, weights, spec: ExpertSpec) -> None:
+    def _load_spec(self, arch: Arch, cfg, dims: ModelDims, prefix: str, weights, comm, spec: ExpertSpec) -> None:
         if weights.process_group.size() > 1:
             raise NotImplementedError("layers with an expert count of their own are served on one GPU")
         self.top_k, self.num_experts, self.act = spec.top, spec.experts, spec.act
         self.deepseek_router = self.sparsemixer_eps = self.expert_parallel = self.shared = self.shared_gate = None
         self.correction = weights.get_tensor(f"{prefix}.{arch.moe_correction}", to_dtype=False).float()
         ep = [f"{prefix}.{arch.moe_expert.format(e=e)}" for e in range(spec.experts)]
-        self.w_up, self.w_down = ops.plain_expert_weights(
-            torch.stack([_expert_weight(weights, cfg, f"{p}.{arch.moe_up}") for p in ep]),        # [E, I, H]
-            torch.stack([_expert_weight(weights, cfg, f"{p}.{arch.moe_down}") for p in ep]))      # [E, H, I]
+        # [E, I, H] per projection (gate first where there is one) and [E, H, I]
+        gate, up, down = (torch.stack([_expert_weight(weights, cfg, f"{p}.{n}") for p in ep]) if n else None
+                          for n in (arch.moe_gate if spec.gated else None, arch.moe_up, arch.moe_down))
+        self.w_up, self.w_down = ops.plain_expert_weights(up, down, gate)
+        if spec.shared_ff:
+            self.shared = DenseMLP(arch, cfg, dims, f"{prefix}.{arch.moe_shared}", weights, comm,
+                                   names=(arch.moe_gate, arch.moe_up, arch.moe_down))
 
     def __call__(self, x, x_scale=None, reduce: bool = True, meta=None, out=None):
         if out is not None:
             out.copy_(self(x, x_scale, reduce=False, meta=meta))
             return out
         if self.spec is not None:
-            w, idx = ops.moe_route_sigmoid(x, self.router.weight, self.correction, self.top_k, self.spec.scale)
-            return ops.moe_plain_experts(x, self.w_up, self.w_down, w, idx, self.act)
+            s = self.spec
+            if s.router == "softmax":
+                w, idx = ops.moe_route_softmax(x, self.router.weight, self.correction, self.top_k)
+            else:
+                w, idx = ops.moe_route_sigmoid(x, self.router.weight, self.correction, self.top_k, s.scale)
+            y = ops.moe_plain_experts(x, self.w_up, self.w_down, w, idx, self.act, s.gated)
+            return y if self.shared is None else (y, self.shared(x, reduce=False))
         logits = self.router(x)
         if self.deepseek_router is not None:
             w, idx = self.deepseek_router(logits)

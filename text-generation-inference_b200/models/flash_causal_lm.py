@@ -376,8 +376,12 @@ class FlashCausalLM(Model):
             # every layer (every run of a layer) has its own kind of cache: pages, slots of recurrent state, or both
             slots = int(state_slots or self.max_batch_size or 1)
             self.state_slots = Pool(0, slots, "recurrent state slots") if self.recurrent else None
-            for layer in self.model.layer_runs:
-                self.kv_cache.append(layer.attn.cache_tensors(self.num_blocks, BLOCK_SIZE, slots, self.device))
+            for i, layer in enumerate(self.model.layer_runs):
+                src = layer.attn.spec.kv_from
+                if src is not None:              # the cache of the last run of the layer it reads
+                    self.kv_cache.append(self.kv_cache[max(j for j in range(i) if self.model.layer_runs[j] is self.model.layers[src])])
+                else:
+                    self.kv_cache.append(layer.attn.cache_tensors(self.num_blocks, BLOCK_SIZE, slots, self.device))
             return
         for _ in range(d.num_layers):
             k = torch.zeros(num_blocks, BLOCK_SIZE, d.num_kv_heads, d.attn_head_dim or d.head_dim,

@@ -4,7 +4,11 @@ Every mixer is called like ``decoder.Attention`` (``x, x_scale, meta, rotary, kv
 cache (``cache_tensors``) and runs as a short sequence of fused ops:
 
     attention   qkv GEMM -> [short convolutions +] rotate + unit RMS + value mixing + page store -> paged attention
+                -> o GEMM; or qkvg GEMM -> RMS of whole rows + temperature + page store -> paged attention -> output gate
                 -> o GEMM
+    latent      GEMM for q, latent and gate -> RMS of the latent, rotations, page store -> queries times the key
+                up-projection -> attention over the latents (all heads read one row per token), gate -> value
+                up-projection -> o GEMM
     delta       one GEMM for q, k, v, write strengths and decay / gate inputs (-> low-rank decay / gate GEMMs)
                 -> short convolutions + unit norms + decays -> state scan -> norm x gate -> o GEMM
     decay       one GEMM for q, k, v, gate -> state scan (SiLU applied on the way in) -> norm x gate -> o GEMM
@@ -21,7 +25,7 @@ from typing import Dict, List, Optional, Sequence, Tuple
 import torch
 
 from .. import ops
-from ..utils.rotary import RotaryTable, scaled_frequencies
+from ..utils.rotary import RotaryTable, scaled_frequencies, yarn_frequencies
 from .arch import MixerSpec
 from .layers import FastLinear, TensorParallelColumnLinear, TensorParallelRowLinear
 
@@ -71,10 +75,11 @@ class RotaryTables:
         self._tables: Dict[tuple, RotaryTable] = {}
 
     def get(self, s: MixerSpec) -> RotaryTable:
-        key = (s.rot_dims, s.rot_base, s.rot_scaling)
+        key = (s.rot_dims, s.rot_base, s.rot_scaling, s.rot_yarn)
         if key not in self._tables:
-            self._tables[key] = RotaryTable.from_frequencies(
-                scaled_frequencies(s.rot_base, s.rot_dims, s.rot_scaling), self.max_positions).to(self.device)
+            freq, amp = (yarn_frequencies(s.rot_base, s.rot_dims, s.rot_yarn) if s.rot_yarn else
+                         (scaled_frequencies(s.rot_base, s.rot_dims, s.rot_scaling), 1.0))
+            self._tables[key] = RotaryTable.from_frequencies(freq, self.max_positions, amplitude=amp).to(self.device)
         return self._tables[key]
 
 
@@ -133,21 +138,32 @@ class Mixer:
 class MixedAttention(Mixer):
     """Paged attention with its own head sizes: short convolutions of q, k and v, rotation of the first dimensions,
     weightless RMS of q and k after it, values mixed with an earlier layer's, keys limited to the query's chunk or window,
-    a sink in the softmax."""
+    a sink in the softmax.  Or, without any of the first four: weighted RMS of q and k over all heads, queries times a factor
+    of their position, keys and values of an earlier layer.  Capped scores and an output gate go with either."""
 
     def __init__(self, spec, prefix, weights, idx, eps, comm=None, rotary: Optional[RotaryTables] = None):
         super().__init__(spec, prefix, weights, idx, eps, comm)
         s = spec
-        self.qkv, self.offs = self.fused(["q", "k", "v"], bias=s.qkv_bias)
+        if s.row_norm and (s.short_conv or s.rot_dims or s.qk_unit_rms or s.v_mix):
+            raise NotImplementedError(f"{prefix}: a norm over whole rows beside convolutions, rotation, unit norms or value mixing")
+        own = ["q", "k", "v"] if s.kv_from is None else ["q"]
+        self.qkv, offs = self.fused(own + (["g"] if s.out_gate else []), bias=s.qkv_bias)
+        self.offs, self.off_gate = offs[:len(own)], offs[-1]
+        self.q_norm, self.k_norm = (self.f32(f"{n}.norm") if s.row_norm and n in own else None for n in ("q", "k"))
+        self.sink = self.f32("sink") if s.learned_sink else (True if s.sink else None)
         self.conv = None
         if s.short_conv:
             self.load_conv()
         self.v_lambda = float(self.f32("vmix").reshape(-1)[0]) if s.v_mix and weights.has_tensor(f"{prefix}.vmix") else 0.0
         self.kd, self.vd = ops.attention_pitch(s.dim, s.vdim, self.dtype, self.device)
-        self.o = self.row(spread_columns(self.tensor("o"), s.heads, s.vdim, self.vd))
+        # a gate packs the heads again
+        self.o = self.row(_column_input(self.tensor("o")) if s.out_gate else
+                          spread_columns(self.tensor("o"), s.heads, s.vdim, self.vd))
         self.rotary = rotary.get(s)
 
     def page_tensors(self, num_blocks: int, block_size: int, device):
+        if self.spec.kv_from is not None:
+            return ()
         # zeros: the kernels never write the padding columns of a page, and padded queries must meet zeros there
         return tuple(torch.zeros(num_blocks, block_size, self.spec.kv_heads, d, dtype=self.dtype, device=device)
                      for d in (self.kd, self.vd))
@@ -159,6 +175,21 @@ class MixedAttention(Mixer):
         s = self.spec
         k_cache, v_cache = kv[:2]
         proj = self.qkv(x)
+        if s.row_norm:
+            q = ops.row_norm_store(proj, self.offs, meta.positions, meta.slots, k_cache, v_cache, self.q_norm, self.k_norm, self.eps,
+                                   s.heads, s.kv_heads, s.dim, s.vdim, self.kd, s.q_temp)
+        else:
+            q = self._rotated(proj, meta, kv)
+        a = ops.paged_attention(q, k_cache, v_cache, meta.block_tables, meta.cu_seqlens_q, meta.kv_lens, s.scale,
+                                window=s.window or -1, softcap=s.softcap, max_q=meta.max_q, max_kv=meta.max_kv, chunk=s.chunk,
+                                sink=self.sink)
+        if s.out_gate:
+            a = ops.output_gate(a, proj[:, self.off_gate:self.off_gate + s.heads * s.vdim], s.vdim)
+        return self.o(a.view(a.shape[0], -1), reduce=reduce, out=out)
+
+    def _rotated(self, proj, meta, kv):
+        s = self.spec
+        k_cache, v_cache = kv[:2]
         v_first = None
         if s.v_mix:
             v_first = meta.v_first
@@ -167,12 +198,49 @@ class MixedAttention(Mixer):
         conv = None
         if self.conv is not None:
             conv = ops.ShortConv(self.conv, kv[2], meta.cu_seqlens_q, meta.kv_lens, meta.state_slots, meta.max_q == 1)
-        q = ops.rotate_norm_store(proj, self.offs, meta.positions, self.rotary.cos_sin, meta.slots, k_cache, v_cache, s.heads,
-                                  s.kv_heads, s.dim, s.vdim, s.rot_dims, s.qk_unit_rms, self.eps, v_first, self.v_lambda,
-                                  s.rot_interleaved, conv)
-        a = ops.paged_attention(q, k_cache, v_cache, meta.block_tables, meta.cu_seqlens_q, meta.kv_lens, s.scale,
-                                window=s.window or -1, max_q=meta.max_q, max_kv=meta.max_kv, chunk=s.chunk, sink=s.sink)
-        return self.o(a.view(a.shape[0], -1), reduce=reduce, out=out)
+        return ops.rotate_norm_store(proj, self.offs, meta.positions, self.rotary.cos_sin, meta.slots, k_cache, v_cache, s.heads,
+                                     s.kv_heads, s.dim, s.vdim, s.rot_dims, s.qk_unit_rms, self.eps, v_first, self.v_lambda,
+                                     s.rot_interleaved, conv)
+
+
+class LatentAttention(Mixer):
+    """Attention whose keys and values are up-projections of one latent per token, beside which a rotated key part that all
+    heads share may stand.  Only latent and rotated part are cached.  The up-projections are moved to the other side of the
+    attention: ``q . (W_uk c) = (W_uk^T q) . c`` and ``sum p W_uv c = W_uv sum p c``, so every head attends to the same rows."""
+
+    def __init__(self, spec, prefix, weights, idx, eps, comm=None, rotary: Optional[RotaryTables] = None):
+        super().__init__(spec, prefix, weights, idx, eps, comm)
+        s = spec
+        if s.out_gate not in ("", "head"):
+            raise NotImplementedError(f"{prefix}: output gate {s.out_gate!r} on latent attention")
+        self.proj, self.offs = self.fused(["q", "dkv"] + (["g"] if s.out_gate else []))
+        self.norm = self.f32("dkv.norm")
+        self.off_rot, self.width = ops.latent_layout(s.kv_rank, s.rot_dims, self.dtype, self.device)
+        pad = (0, self.off_rot - s.kv_rank)
+        self.uk, self.uv = (torch.nn.functional.pad(self.tensor(n).view(s.heads, d, s.kv_rank), pad).contiguous()
+                            for n, d in (("uk", s.dim), ("uv", s.vdim)))         # [H, d, columns of the latent]
+        self.o = self.row(_column_input(self.tensor("o")))
+        self.rotary = rotary.get(s)
+
+    def page_tensors(self, num_blocks: int, block_size: int, device):
+        # zeros: the kernels never write the padding columns
+        return (torch.zeros(num_blocks, block_size, 1, self.width, dtype=self.dtype, device=device),)
+
+    def __call__(self, x, x_scale, meta, rotary, kv, reduce: bool = True, out=None):
+        s, T = self.spec, x.shape[0]
+        pages, = kv
+        proj = self.proj(x)
+        q = proj.new_empty(T, s.heads, self.width)
+        ops.latent_store(proj, self.offs[1], self.norm, self.eps, meta.positions, self.rotary.cos_sin, meta.slots, pages, q,
+                         self.off_rot, s.kv_rank, s.rot_dims, s.heads, s.dim)
+        plain = proj[:, :s.heads * (s.dim + s.rot_dims)].view(T, s.heads, -1)[..., :s.dim]
+        torch.bmm(plain.transpose(0, 1), self.uk, out=q[..., :self.off_rot].transpose(0, 1))
+        gate = proj[:, self.offs[2]:self.offs[2] + s.heads] if s.out_gate else None
+        a = ops.latent_attention(q, pages, s.kv_rank, meta.block_tables, meta.cu_seqlens_q, meta.kv_lens, s.scale, s.window or -1,
+                                 meta.max_q, meta.max_kv, gate)
+        y = proj.new_empty(T, s.heads, s.vdim)
+        torch.bmm(a.transpose(0, 1), self.uv[..., :a.shape[2]].transpose(1, 2), out=y.transpose(0, 1))
+        return self.o(y.view(T, -1), reduce=reduce, out=out)
 
 
 class GatedDelta(Mixer):
@@ -243,7 +311,7 @@ class DecayAttention(Mixer):
         return self.o(y, reduce=reduce, out=out)
 
 
-MIXERS = {"attention": MixedAttention, "delta": GatedDelta, "decay": DecayAttention}
+MIXERS = {"attention": MixedAttention, "latent": LatentAttention, "delta": GatedDelta, "decay": DecayAttention}
 
 
 def load_mixer(spec: MixerSpec, prefix: str, weights, idx: int, eps: float, comm, rotary: RotaryTables) -> Mixer:

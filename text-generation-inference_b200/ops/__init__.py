@@ -71,10 +71,11 @@ def rope_and_cache(qkv, positions, cos_sin, slots, k_cache, v_cache, num_heads, 
 
 
 def paged_attention(q, k_cache, v_cache, block_tables, cu_seqlens_q, kv_lens, scale, window=-1, softcap=0.0,
-                    k_scale=None, v_scale=None, max_q=None, max_kv=None, horizon=None, chunk=0, sink=False):
+                    k_scale=None, v_scale=None, max_q=None, max_kv=None, horizon=None, chunk=0, sink=None):
     """``horizon`` (optional int32 ``[T]``): last KV position each query row may see when that is past its own
     position (image rows that attend to their whole image); ``None`` is plain causal attention.  ``chunk`` > 0: rows see
-    only keys of their own chunk of ``chunk`` positions.  ``sink``: one more key of score 0 and no value in the softmax."""
+    only keys of their own chunk of ``chunk`` positions.  ``sink``: one more key without a value in the softmax, of the score
+    given per head (fp32 ``[Hq]``; ``True``: 0), which is neither scaled nor capped."""
     if use_native(q):
         return native().paged_attention(q, k_cache, v_cache, block_tables, cu_seqlens_q, kv_lens, scale,
                                         window, softcap, k_scale, v_scale, max_q, max_kv, horizon=horizon, chunk=chunk, sink=sink)
@@ -111,11 +112,14 @@ def embed_residual(ids, table, scale=1.0):
     return _mixer_backend(table).embed_residual(ids, table, scale)
 
 
-def residual_norm(delta, residual, weight, eps, rows=None, keep=True, scale=1.0, unit_offset=False, weight2=None):
+def residual_norm(delta, residual, weight, eps, rows=None, keep=True, scale=1.0, unit_offset=False, weight2=None, layer=False,
+                  bias=None):
     """``r = residual + scale * delta`` in fp32 (``delta``: a tensor, a pair whose sum it is, or ``None``) and
-    ``RMSNorm(r) * weight`` (``unit_offset``: times ``1 + weight``) in the weight's dtype: ``(normed, r)``, with
-    ``weight2`` ``(normed, normed by weight2, r)``.  ``rows`` picks the rows to compute; ``keep=False`` drops ``r``."""
-    return _mixer_backend(residual).residual_norm(delta, residual, weight, eps, rows, keep, scale, unit_offset, weight2)
+    ``RMSNorm(r) * weight`` (``unit_offset``: times ``1 + weight``; ``layer``: of ``r`` minus its mean; plus ``bias``) in the
+    weight's dtype: ``(normed, r)``, with ``weight2`` ``(normed, normed by weight2, r)``.  ``rows`` picks the rows to compute;
+    ``keep=False`` drops ``r``."""
+    return _mixer_backend(residual).residual_norm(delta, residual, weight, eps, rows, keep, scale, unit_offset, weight2, layer,
+                                                  bias)
 
 
 @dataclass
@@ -147,6 +151,43 @@ def rotate_norm_store(proj, offs, positions, cos_sin, slots, k_cache, v_cache, n
     return _mixer_backend(proj).rotate_norm_store(proj, offs, positions, cos_sin, slots, k_cache, v_cache, num_heads,
                                                   num_kv_heads, dim, vdim, rot_dim, qk_norm, eps, v_first, v_lambda,
                                                   interleaved, conv)
+
+
+def row_norm_store(proj, offs, positions, slots, k_cache, v_cache, q_weight, k_weight, eps, num_heads, num_kv_heads, dim, vdim,
+                   width, temperature=None):
+    """``proj[T, *]`` with q, k, v from columns ``offs``: q and k over the root mean square of their whole rows, times their
+    weights; q times ``1 + coef * ln(floor((position + 1) / every) + 1)`` (``temperature = (coef, every)``); k and v stored
+    (``k_weight`` ``None``: the layer has queries only).  Returns q ``[T, Hq, width]``, zeros past ``dim``."""
+    return _mixer_backend(proj).row_norm_store(proj, offs, positions, slots, k_cache, v_cache, q_weight, k_weight, eps, num_heads,
+                                               num_kv_heads, dim, vdim, width, temperature)
+
+
+def output_gate(x, gate, width):
+    """``x[T, H, pitch]``: the first ``width`` columns of every head times ``sigmoid(gate[T, H * width])``, ``[T, H * width]``."""
+    return _mixer_backend(x).output_gate(x, gate, width)
+
+
+def latent_layout(rank, rot, dtype, device):
+    """``(column of the rotated part, width)`` of a cached latent row on ``device`` (see ``ops.cuda.latent_layout``)."""
+    if torch.device(device).type == "cuda" and not _FORCE_TORCH:
+        return native().latent_layout(rank, rot, dtype)
+    return rank, rank + rot
+
+
+def latent_store(proj, off_c, weight, eps, positions, cos_sin, slots, pages, q, off_rot, rank, rot, heads, dim):
+    """Latent attention's inputs from ``proj[T, *]`` (queries, ``dim`` plain and ``rot`` rotated dimensions per head, from
+    column 0; ``rank`` latent columns and the shared key's ``rot`` columns from ``off_c``): the latent over its root mean
+    square times ``weight``, and the shared key rotated (pairs ``2i, 2i + 1``), go to ``pages`` at the tokens' slots; the
+    rotated dimensions of the queries go to ``q[T, H, *]`` from column ``off_rot``, zeros behind them."""
+    _mixer_backend(proj).latent_store(proj, off_c, weight, eps, positions, cos_sin, slots, pages, q, off_rot, rank, rot, heads, dim)
+
+
+def latent_attention(q, pages, rank, block_tables, cu_seqlens_q, kv_lens, scale, window=-1, max_q=None, max_kv=None, gate=None):
+    """Causal attention of ``q[T, H, width]`` over the one key row per token in ``pages[blocks, block_size, 1, width]``, whose
+    first ``rank`` columns are the value too; head outputs times ``sigmoid(gate[T, H])``.  ``[T, H, rank or more]``, zeros
+    past ``rank``."""
+    return _mixer_backend(q).latent_attention(q, pages, rank, block_tables, cu_seqlens_q, kv_lens, scale, window, max_q, max_kv,
+                                              gate)
 
 
 def recurrent_pitch(dim, device):
@@ -279,14 +320,24 @@ def moe_route_sigmoid(x, weight, correction, top_k, scale):
     return _mixer_backend(x).moe_route_sigmoid(x, weight, correction, top_k, scale)
 
 
-def plain_expert_weights(w_up, w_down):
-    """``[E, I, H]`` and ``[E, H, I]`` as the kernels want them: bf16 sizes brought to multiples of 8 with zeros."""
+def moe_route_softmax(x, weight, bias, top_k):
+    """Router product plus bias in fp32, the ``top_k`` largest logits and the softmax over them: ``(weights [T, k], experts
+    [T, k])``."""
+    return _mixer_backend(x).moe_route_softmax(x, weight, bias, top_k)
+
+
+def plain_expert_weights(w_up, w_down, w_gate=None):
+    """``[E, I, H]`` and ``[E, H, I]`` as the kernels want them: bf16 sizes brought to multiples of 8 with zeros.  With
+    ``w_gate`` the first matrix is ``[E, 2 I, H]``, gate rows before up rows."""
     if use_native(w_up) and w_up.dtype == torch.bfloat16:
-        pad = lambda w: torch.nn.functional.pad(w, (0, -w.shape[2] % 8, 0, -w.shape[1] % 8))
-        w_up, w_down = pad(w_up), pad(w_down)
+        pad = lambda w: None if w is None else torch.nn.functional.pad(w, (0, -w.shape[2] % 8, 0, -w.shape[1] % 8))
+        w_up, w_down, w_gate = pad(w_up), pad(w_down), pad(w_gate)
+    if w_gate is not None:
+        w_up = torch.cat([w_gate, w_up], dim=1)
     return w_up.contiguous(), w_down.contiguous()
 
 
-def moe_plain_experts(x, w_up, w_down, topk_weights, topk_ids, act):
-    """``sum over slots of weight * down(act(up x))`` of ungated experts (weights from ``plain_expert_weights``)."""
-    return _mixer_backend(x).moe_plain_experts(x, w_up, w_down, topk_weights, topk_ids, act)
+def moe_plain_experts(x, w_up, w_down, topk_weights, topk_ids, act, gated=False):
+    """``sum over slots of weight * down(act(up x))``, or ``down(act(gate x) * up x)`` when ``gated`` (weights from
+    ``plain_expert_weights``)."""
+    return _mixer_backend(x).moe_plain_experts(x, w_up, w_down, topk_weights, topk_ids, act, gated)

@@ -60,7 +60,7 @@ struct PrefillParams {
   float scale, softcap;
   int window;
   int chunk;                    // > 0: a row sees only keys of its own chunk of `chunk` positions
-  int sink;                     // 1: the denominator counts one more key of score 0 that has no value
+  const float* sink;            // [Hq] or null: score of one more key per head that has no value
   int* status;
 };
 
@@ -510,7 +510,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
       fail = true;
     }
     if (!fail) {
-      if (p.sink && hf == 0) l += exp2f(-m);      // both threads of a row hold the same maximum
+      if (p.sink != nullptr && hf == 0) l += exp2f(fmaf(p.sink[h], kLog2e, -m));      // both threads of a row hold the same maximum
       reinterpret_cast<float*>(smem + L::kP + (ntiles & 1) * kTileBytes)[hf * 128 + r] = l;
       __syncwarp();
       if (lane == 0) mbar_arrive(l_ready);
@@ -649,8 +649,8 @@ extern "C" {
 int tgi_prefill_attention_tc(const void* q, const void* k_cache, const void* v_cache, const int* block_tables,
                              const int* cu_seqlens_q, const int* kv_lens, const float* k_scale, const float* v_scale,
                              void* out, int B, int max_q, int max_blocks, int num_blocks, int Hq, int Hkv, float scale,
-                             float softcap, int window, int chunk, int sink, int fp8_kv, const int* horizon, int* status,
-                             cudaStream_t stream) {
+                             float softcap, int window, int chunk, const float* sink, int fp8_kv, const int* horizon,
+                             int* status, cudaStream_t stream) {
   if (B <= 0 || max_q <= 0) return 0;
   if (Hq % Hkv != 0 || B > 65535 || Hq > 65535) return -10;
   PrefillParams p;

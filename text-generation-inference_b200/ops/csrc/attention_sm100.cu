@@ -115,7 +115,7 @@ struct Params {
   float scale, softcap;
   int window;
   int chunk;                    // > 0: a row sees only keys of its own chunk of `chunk` positions
-  int sink;                     // 1: the softmax denominator counts one more key of score 0 that has no value
+  const float* sink;            // [Hq] or null: score of one more key per head that has no value
   int nsplit;
 };
 
@@ -125,8 +125,10 @@ __device__ __forceinline__ int first_visible(const Params& p, int pos) {
   if (p.chunk > 0 && pos > 0) lo = max(lo, pos - pos % p.chunk);
   return max(lo, 0);
 }
-// exp(0 - m) for a running maximum kept in the log2 domain: the share of the sink in the denominator.
-__device__ __forceinline__ float sink_term(int sink, float m_log2) { return sink ? exp2f(-m_log2) : 0.f; }
+// exp(sink - m) for a running maximum kept in the log2 domain: the share of the sink in the denominator.
+__device__ __forceinline__ float sink_term(const float* sink, int h, float m_log2) {
+  return sink != nullptr ? exp2f(fmaf(sink[h], kLog2e, -m_log2)) : 0.f;
+}
 
 // Gather one 64-token K or V tile (tokens t0..t0+63 of sequence b, KV head kvh) into shared memory.
 // bf16 pages land directly in the swizzled compute tile; e4m3 pages land in a raw staging tile.
@@ -431,8 +433,8 @@ prefill_kernel(Params p) {
   }
   cp_async_wait<0>();
 
-  const float inv0 = l[0] > 0.f ? (FP8 ? vs : 1.f) / (l[0] + sink_term(p.sink, m[0])) : 0.f;
-  const float inv1 = l[1] > 0.f ? (FP8 ? vs : 1.f) / (l[1] + sink_term(p.sink, m[1])) : 0.f;
+  const float inv0 = l[0] > 0.f ? (FP8 ? vs : 1.f) / (l[0] + sink_term(p.sink, h, m[0])) : 0.f;
+  const float inv1 = l[1] > 0.f ? (FP8 ? vs : 1.f) / (l[1] + sink_term(p.sink, h, m[1])) : 0.f;
   const int r0 = row_base + warp * 16 + (lane >> 2), r1 = r0 + 8;
 #pragma unroll
   for (int i = 0; i < D / 8; ++i) {
@@ -706,7 +708,7 @@ decode_kernel_v2(Params p) {
     }
     const int h = h0 + row;
     if (p.nsplit == 1) {
-      const float inv = ll > 0.f ? (FP8 ? vsc : 1.f) / (ll + sink_term(p.sink, mm)) : 0.f;
+      const float inv = ll > 0.f ? (FP8 ? vsc : 1.f) / (ll + sink_term(p.sink, h, mm)) : 0.f;
       p.out[(static_cast<size_t>(q_row) * p.Hq + h) * D + col] = __float2bfloat16(acc * inv);
     } else {
       const size_t pi = (static_cast<size_t>(b) * p.Hq + h) * p.nsplit + split;
@@ -1115,7 +1117,7 @@ decode_kernel_v3(Params p, const __grid_constant__ CUtensorMap tmK, const __grid
     }
     const int h = h0 + row;
     if (p.nsplit == 1) {
-      const float inv = ll > 0.f ? (FP8 ? vsc : 1.f) / (ll + sink_term(p.sink, mm)) : 0.f;
+      const float inv = ll > 0.f ? (FP8 ? vsc : 1.f) / (ll + sink_term(p.sink, h, mm)) : 0.f;
       p.out[(static_cast<size_t>(q_row) * p.Hq + h) * D + col] = __float2bfloat16(acc * inv);
     } else {
       const size_t pi = (static_cast<size_t>(b) * p.Hq + h) * p.nsplit + split;
@@ -1131,7 +1133,7 @@ decode_kernel_v3(Params p, const __grid_constant__ CUtensorMap tmK, const __grid
 // merge split partials: grid (B, Hq), block D
 __global__ void decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                     const int* __restrict__ cu_seqlens_q, __nv_bfloat16* __restrict__ out, int Hq,
-                                    int D, int nsplit, int sink) {
+                                    int D, int nsplit, const float* sink) {
   tgi::pdl_wait();
   tgi::pdl_trigger();
   const int b = blockIdx.x, h = blockIdx.y;
@@ -1152,7 +1154,7 @@ __global__ void decode_merge_kernel(const float* __restrict__ part_o, const floa
         wsum += w;
       }
     }
-    out[(static_cast<size_t>(cu_seqlens_q[b]) * Hq + h) * D + col] = __float2bfloat16(wsum > 0.f ? acc / (wsum + sink_term(sink, mm)) : 0.f);
+    out[(static_cast<size_t>(cu_seqlens_q[b]) * Hq + h) * D + col] = __float2bfloat16(wsum > 0.f ? acc / (wsum + sink_term(sink, h, mm)) : 0.f);
   }
 }
 
@@ -1260,8 +1262,8 @@ int launch_v3(const Params& p, int B, cudaStream_t stream) {
 extern "C" int tgi_prefill_attention_tc(const void* q, const void* k_cache, const void* v_cache, const int* block_tables,
                                         const int* cu_seqlens_q, const int* kv_lens, const float* k_scale,
                                         const float* v_scale, void* out, int B, int max_q, int max_blocks, int num_blocks,
-                                        int Hq, int Hkv, float scale, float softcap, int window, int chunk, int sink,
-                                        int fp8_kv, const int* horizon, int* status, cudaStream_t stream);
+                                        int Hq, int Hkv, float scale, float softcap, int window, int chunk,
+                                        const float* sink, int fp8_kv, const int* horizon, int* status, cudaStream_t stream);
 
 bool prefill_tc_enabled() {
   static const bool on = [] {
@@ -1353,12 +1355,12 @@ int tgi_attn_status(int reset) {
 
 // `horizon` (optional, prefill only): per query row the last KV position it may attend to; null = causal.
 // `chunk` > 0: rows see only keys of their own chunk of `chunk` positions, counted from position 0.
-// `sink` != 0: exp(0) is added to every softmax denominator.
+// `sink` (optional, [Hq]): exp(sink[h]) is added to the softmax denominators of head h.
 int tgi_paged_attention_ex(const void* q, const void* k_cache, const void* v_cache, const int* block_tables,
                            const int* cu_seqlens_q, const int* kv_lens, const float* k_scale, const float* v_scale,
                            void* out, float* part_o, float* part_ml, int B, int max_q, int max_blocks, int block_size,
                            int num_blocks, int Hq, int Hkv, int D, float scale, float softcap, int window, int chunk,
-                           int sink, int nsplit, int fp8_kv, const int* horizon, cudaStream_t stream);
+                           const float* sink, int nsplit, int fp8_kv, const int* horizon, cudaStream_t stream);
 
 int tgi_paged_attention(const void* q, const void* k_cache, const void* v_cache, const int* block_tables,
                         const int* cu_seqlens_q, const int* kv_lens, const float* k_scale, const float* v_scale,
@@ -1367,14 +1369,14 @@ int tgi_paged_attention(const void* q, const void* k_cache, const void* v_cache,
                         int fp8_kv, cudaStream_t stream) {
   return tgi_paged_attention_ex(q, k_cache, v_cache, block_tables, cu_seqlens_q, kv_lens, k_scale, v_scale, out, part_o,
                                 part_ml, B, max_q, max_blocks, block_size, num_blocks, Hq, Hkv, D, scale, softcap, window,
-                                0, 0, nsplit, fp8_kv, nullptr, stream);
+                                0, nullptr, nsplit, fp8_kv, nullptr, stream);
 }
 
 int tgi_paged_attention_ex(const void* q, const void* k_cache, const void* v_cache, const int* block_tables,
                            const int* cu_seqlens_q, const int* kv_lens, const float* k_scale, const float* v_scale,
                            void* out, float* part_o, float* part_ml, int B, int max_q, int max_blocks, int block_size,
                            int num_blocks, int Hq, int Hkv, int D, float scale, float softcap, int window, int chunk,
-                           int sink, int nsplit, int fp8_kv, const int* horizon, cudaStream_t stream) {
+                           const float* sink, int nsplit, int fp8_kv, const int* horizon, cudaStream_t stream) {
   if (B <= 0 || max_q <= 0) return 0;
   if (Hq % Hkv != 0) return -10;
   Params p;

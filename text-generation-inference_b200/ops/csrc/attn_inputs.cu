@@ -1,0 +1,311 @@
+// Kernels between the projections of an attention layer and its attention, in a bf16 and an fp32 build:
+//   row norm + store      RMS of q and of k over all heads at once, times weights; q times a factor of its position; k and v
+//                         to their pages
+//   output gate           attention output times the sigmoid of a projection, heads packed to their true width
+//   latent store          latent attention: RMS of the latent, rotation of the key part that all heads share and of the
+//                         queries' rotated dimensions, page store
+//
+// Norms, temperatures, angles and sigmoids are fp32 in both builds.
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+#include <stdint.h>
+
+#include "launch.cuh"
+#include "mixer_util.cuh"
+
+namespace {
+
+using namespace mixer;
+
+template <typename T>
+struct Vec {                                               // elements of a 16-byte access
+  static constexpr int N = 16 / sizeof(T);
+};
+template <typename T>
+__device__ __forceinline__ void load_vec(const T* p, float (&x)[Vec<T>::N]) {
+#pragma unroll
+  for (int i = 0; i < Vec<T>::N; i += 4) {
+    const float4 v = load4(p + i);
+    x[i] = v.x; x[i + 1] = v.y; x[i + 2] = v.z; x[i + 3] = v.w;
+  }
+}
+template <>
+__device__ __forceinline__ void load_vec<bf16>(const bf16* p, float (&x)[8]) {
+  const uint4 u = *reinterpret_cast<const uint4*>(p);
+  const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&u);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const float2 f = __bfloat1622float2(h[i]);
+    x[2 * i] = f.x;
+    x[2 * i + 1] = f.y;
+  }
+}
+__device__ __forceinline__ void store_vec(float* p, const float (&x)[4]) { store4(p, make_float4(x[0], x[1], x[2], x[3])); }
+__device__ __forceinline__ void store_vec(bf16* p, const float (&x)[8]) {
+  uint4 u;
+  __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&u);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) h[i] = __floats2bfloat162_rn(x[2 * i], x[2 * i + 1]);
+  *reinterpret_cast<uint4*>(p) = u;
+}
+
+// two sums over the block at once; `red` holds 66 floats
+__device__ __forceinline__ float2 block_sum2(float a, float b, float* red) {
+  a = warp_sum(a);
+  b = warp_sum(b);
+  if ((threadIdx.x & 31) == 0) {
+    red[2 * (threadIdx.x >> 5)] = a;
+    red[2 * (threadIdx.x >> 5) + 1] = b;
+  }
+  __syncthreads();
+  float2 s = make_float2(0.f, 0.f);
+  for (int w = 0; w < static_cast<int>(blockDim.x >> 5); ++w) {
+    s.x += red[2 * w];
+    s.y += red[2 * w + 1];
+  }
+  return s;
+}
+
+// ------------------------------------------------------------------------------------------------
+// q, k and v of a token at columns 0, off_k, off_v of proj[T, ld].  One CTA per token.  NP > 0: 16-byte pieces, up to NP per
+// thread, in registers between norm and store (dim, vdim and all pitches multiples of a piece); NP == 0: any size, read twice.
+// ------------------------------------------------------------------------------------------------
+struct RowNorm {
+  long long ld, num_slots;
+  int off_k, off_v, Hq, Hkv, dim, vdim, Dq, Dk, Dv;        // Dq, Dk, Dv: pitches of a head in q_out and in the pages
+  int every;                                               // 0: no temperature
+  float eps, coef;
+};
+template <typename T, int NP>
+__global__ void __launch_bounds__(512)
+row_norm_store_kernel(const T* __restrict__ proj, const int* __restrict__ positions, const int* __restrict__ slots,
+                      const float* __restrict__ wq, const float* __restrict__ wk, T* __restrict__ q_out,
+                      T* __restrict__ k_cache, T* __restrict__ v_cache, RowNorm p) {
+  tgi::pdl_wait();
+  tgi::pdl_trigger();
+  __shared__ float red[66];
+  const int t = blockIdx.x;
+  const T* row = proj + static_cast<size_t>(t) * p.ld;
+  const long long slot = slots[t];
+  const bool keep = wk != nullptr && slot >= 0 && slot < p.num_slots;     // padding rows have slot -1
+  const int nq = p.Hq * p.dim, nk = p.Hkv * p.dim, nv = p.Hkv * p.vdim;
+  float temp = 1.f;
+  if (p.every > 0) temp = 1.f + p.coef * logf(static_cast<float>((positions[t] + 1) / p.every) + 1.f);
+  T* q = q_out + static_cast<size_t>(t) * p.Hq * p.Dq;
+  T* k = k_cache + static_cast<size_t>(keep ? slot : 0) * p.Hkv * p.Dk;
+  T* v = v_cache + static_cast<size_t>(keep ? slot : 0) * p.Hkv * p.Dv;
+  float sq = 0.f, sk = 0.f;
+  if constexpr (NP > 0) {
+    constexpr int N = Vec<T>::N;
+    const int pq = nq / N, pk = keep ? nk / N : 0, pv = keep ? nv / N : 0;
+    float x[NP][N];
+#pragma unroll
+    for (int e = 0; e < NP; ++e) {
+      const int i = threadIdx.x + e * blockDim.x;
+      if (i < pq + pk + pv) {
+        load_vec<T>(i < pq ? row + i * N : i < pq + pk ? row + p.off_k + (i - pq) * N : row + p.off_v + (i - pq - pk) * N, x[e]);
+        float s = 0.f;
+#pragma unroll
+        for (int j = 0; j < N; ++j) s = fmaf(x[e][j], x[e][j], s);
+        if (i < pq) sq += s;
+        else if (i < pq + pk) sk += s;
+      }
+    }
+    const float2 ss = block_sum2(sq, sk, red);
+    const float iq = temp / sqrtf(ss.x / nq + p.eps), ik = 1.f / sqrtf(ss.y / nk + p.eps);
+#pragma unroll
+    for (int e = 0; e < NP; ++e) {
+      const int i = threadIdx.x + e * blockDim.x;
+      if (i >= pq + pk + pv) continue;
+      T* dst;
+      if (i < pq + pk) {
+        const bool is_q = i < pq;
+        const int c = (is_q ? i : i - pq) * N, h = c / p.dim, pitch = is_q ? p.Dq : p.Dk;
+        const float* w = (is_q ? wq : wk) + c;
+        const float inv = is_q ? iq : ik;
+#pragma unroll
+        for (int j = 0; j < N; j += 4) {
+          const float4 f = *reinterpret_cast<const float4*>(w + j);
+          x[e][j] *= inv * f.x; x[e][j + 1] *= inv * f.y; x[e][j + 2] *= inv * f.z; x[e][j + 3] *= inv * f.w;
+        }
+        dst = (is_q ? q : k) + static_cast<size_t>(h) * pitch + (c - h * p.dim);
+      } else {
+        const int c = (i - pq - pk) * N, h = c / p.vdim;
+        dst = v + static_cast<size_t>(h) * p.Dv + (c - h * p.vdim);
+      }
+      store_vec(dst, x[e]);
+    }
+  } else {
+    for (int i = threadIdx.x; i < nq; i += blockDim.x) sq += to_f(row[i]) * to_f(row[i]);
+    if (keep)
+      for (int i = threadIdx.x; i < nk; i += blockDim.x) sk += to_f(row[p.off_k + i]) * to_f(row[p.off_k + i]);
+    const float2 ss = block_sum2(sq, sk, red);
+    const float iq = temp / sqrtf(ss.x / nq + p.eps), ik = 1.f / sqrtf(ss.y / nk + p.eps);
+    for (int i = threadIdx.x; i < nq; i += blockDim.x) put(q + i / p.dim * p.Dq + i % p.dim, to_f(row[i]) * iq * wq[i]);
+    if (keep) {
+      for (int i = threadIdx.x; i < nk; i += blockDim.x) put(k + i / p.dim * p.Dk + i % p.dim, to_f(row[p.off_k + i]) * ik * wk[i]);
+      for (int i = threadIdx.x; i < nv; i += blockDim.x) v[i / p.vdim * p.Dv + i % p.vdim] = row[p.off_v + i];
+    }
+  }
+  const int pad = p.Dq - p.dim;
+  if (pad > 0)
+    for (int i = threadIdx.x; i < p.Hq * pad; i += blockDim.x) put(q + i / pad * p.Dq + p.dim + i % pad, 0.f);
+}
+
+// ------------------------------------------------------------------------------------------------
+// out[t, h * width + i] = x[t, h, i] * sigmoid(gate[t, h * width + i]); x has heads `pitch` elements apart
+// ------------------------------------------------------------------------------------------------
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256)
+output_gate_kernel(const T* __restrict__ x, const T* __restrict__ gate, long long ld, T* __restrict__ out, long long n, int H,
+                   int pitch, int width) {
+  tgi::pdl_wait();
+  tgi::pdl_trigger();
+  constexpr int N = VEC ? Vec<T>::N : 1;
+  const long long stride = static_cast<long long>(gridDim.x) * blockDim.x;
+  const unsigned cols = static_cast<unsigned>(H * width);
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < n / N; i += stride) {
+    const long long e = i * N, t = e / cols;
+    const unsigned c = static_cast<unsigned>(e - t * cols), h = c / width;
+    const T* src = x + (t * H + h) * pitch + (c - h * width);
+    const T* g = gate + t * ld + c;
+    if constexpr (VEC) {
+      float a[N], b[N];
+      load_vec<T>(src, a);
+      load_vec<T>(g, b);
+#pragma unroll
+      for (int j = 0; j < N; ++j) a[j] *= sigmoid_t<T>(b[j]);
+      store_vec(out + e, a);
+    } else {
+      put(out + e, to_f(*src) * sigmoid_t<T>(to_f(*g)));
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------------------------
+// Inputs of latent attention.  proj[T, ld]: queries (H heads of dim plain and rot rotated dimensions) at column 0, latent
+// (rank) and the shared key's rotated part (rot) at off_c.  Grid (T, groups of heads); a warp normalises the latent and
+// rotates the shared part (first group), the others rotate the queries of a head each.  Pairs 2i, 2i + 1.
+// ------------------------------------------------------------------------------------------------
+struct Latent {
+  long long ld, num_slots;
+  int off_c, rank, rot, H, dim, off_rot, width, max_pos;   // width: of a cached row and of a query head
+  float eps;
+};
+template <typename T>
+__global__ void __launch_bounds__(256)
+latent_store_kernel(const T* __restrict__ proj, const float* __restrict__ weight, const int* __restrict__ positions,
+                    const float* __restrict__ cos_sin, const int* __restrict__ slots, T* __restrict__ pages,
+                    T* __restrict__ q_out, Latent p) {
+  tgi::pdl_wait();
+  tgi::pdl_trigger();
+  const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+  const T* row = proj + static_cast<size_t>(t) * p.ld;
+  const int rh = p.rot / 2, pos = min(max(positions[t], 0), p.max_pos - 1);
+  const float* cs = cos_sin + static_cast<size_t>(pos) * p.rot;
+  auto rotate = [&](const T* src, T* dst, int end) {       // rotated pairs, then zeros up to `end`
+    for (int i = lane; i < rh; i += 32) {
+      const float u = to_f(src[2 * i]), v = to_f(src[2 * i + 1]), c = cs[i], s = cs[rh + i];
+      put(dst + 2 * i, u * c - v * s);
+      put(dst + 2 * i + 1, v * c + u * s);
+    }
+    for (int i = p.rot + lane; i < end; i += 32) put(dst + i, 0.f);
+  };
+  for (int u = warp; u <= p.H; u += warps) {
+    if (u == 0) {
+      const long long slot = slots[t];
+      if (slot < 0 || slot >= p.num_slots) continue;       // padding rows have slot -1
+      const T* c = row + p.off_c;
+      T* dst = pages + static_cast<size_t>(slot) * p.width;
+      float ss = 0.f;
+      for (int i = lane; i < p.rank; i += 32) ss = fmaf(to_f(c[i]), to_f(c[i]), ss);
+      const float inv = 1.f / sqrtf(warp_sum(ss) / p.rank + p.eps);
+      for (int i = lane; i < p.rank; i += 32) put(dst + i, to_f(c[i]) * inv * weight[i]);
+      if (p.rot > 0) rotate(c + p.rank, dst + p.off_rot, p.rot);
+    } else if (p.off_rot < p.width) {
+      rotate(row + static_cast<size_t>(u - 1) * (p.dim + p.rot) + p.dim,
+             q_out + (static_cast<size_t>(t) * p.H + u - 1) * p.width + p.off_rot, p.width - p.off_rot);
+    }
+  }
+}
+
+int done() { return cudaGetLastError() == cudaSuccess ? 0 : -3; }
+
+template <typename T>
+int row_norm_store(const void* proj, const int* positions, const int* slots, const float* wq, const float* wk, void* q_out,
+                   void* k_cache, void* v_cache, int T_, const RowNorm& p, cudaStream_t stream) {
+  constexpr int N = Vec<T>::N;
+  auto go = [&](auto kern, int threads) {
+    tgi::launch(kern, dim3(T_), dim3(threads), 0, stream, static_cast<const T*>(proj), positions, slots, wq, wk,
+                static_cast<T*>(q_out), static_cast<T*>(k_cache), static_cast<T*>(v_cache), p);
+    return done();
+  };
+  const int pieces = (p.Hq * p.dim + (wk != nullptr ? p.Hkv * (p.dim + p.vdim) : 0)) / N;
+  const bool vec = p.dim % N == 0 && p.vdim % N == 0 && p.Dq % N == 0 && p.Dk % N == 0 && p.Dv % N == 0 && p.ld % N == 0 &&
+                   p.off_k % N == 0 && p.off_v % N == 0 && reinterpret_cast<uintptr_t>(proj) % 16 == 0;
+  if (vec && pieces <= 4 * 512) {
+    const int threads = pieces >= 1024 ? 512 : pieces >= 256 ? 256 : 128;
+    const int np = (pieces + threads - 1) / threads;
+    return np <= 1 ? go(row_norm_store_kernel<T, 1>, threads) : np <= 2 ? go(row_norm_store_kernel<T, 2>, threads)
+                                                                       : go(row_norm_store_kernel<T, 4>, threads);
+  }
+  return go(row_norm_store_kernel<T, 0>, 256);
+}
+
+template <typename T>
+int output_gate(const void* x, const void* gate, long long ld, void* out, int T_, int H, int pitch, int width, cudaStream_t stream) {
+  constexpr int N = Vec<T>::N;
+  const bool vec = width % N == 0 && pitch % N == 0 && ld % N == 0 && reinterpret_cast<uintptr_t>(gate) % 16 == 0;
+  const long long n = static_cast<long long>(T_) * H * width;
+  long long blocks = (n / (vec ? N : 1) + 255) / 256;
+  if (blocks > 148 * 16) blocks = 148 * 16;
+  auto go = [&](auto kern) {
+    tgi::launch(kern, dim3(static_cast<unsigned>(blocks)), dim3(256), 0, stream, static_cast<const T*>(x),
+                static_cast<const T*>(gate), ld, static_cast<T*>(out), n, H, pitch, width);
+    return done();
+  };
+  return vec ? go(output_gate_kernel<T, true>) : go(output_gate_kernel<T, false>);
+}
+
+}  // namespace
+
+// `f32` selects the build: 1 = fp32 activations and pages, 0 = bf16.
+extern "C" {
+
+// wk null: the layer has queries only and nothing is stored.  every 0: no temperature.
+int tgi_row_norm_store(int f32, const void* proj, long long ld, int off_k, int off_v, const int* positions, const int* slots,
+                       const float* wq, const float* wk, void* q_out, void* k_cache, void* v_cache, int T, int Hq, int Hkv,
+                       int dim, int vdim, int Dq, int Dk, int Dv, long long num_slots, float eps, float coef, int every,
+                       cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (Dq < dim || Dk < dim || Dv < vdim || every < 0) return -10;
+  const RowNorm p{ld, num_slots, off_k, off_v, Hq, Hkv, dim, vdim, Dq, Dk, Dv, every, eps, coef};
+  return f32 ? row_norm_store<float>(proj, positions, slots, wq, wk, q_out, k_cache, v_cache, T, p, stream)
+             : row_norm_store<bf16>(proj, positions, slots, wq, wk, q_out, k_cache, v_cache, T, p, stream);
+}
+
+int tgi_output_gate(int f32, const void* x, const void* gate, long long ld, void* out, int T, int H, int pitch, int width,
+                    cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (pitch < width || width < 1) return -10;
+  return f32 ? output_gate<float>(x, gate, ld, out, T, H, pitch, width, stream)
+             : output_gate<bf16>(x, gate, ld, out, T, H, pitch, width, stream);
+}
+
+int tgi_latent_store(int f32, const void* proj, long long ld, int off_c, const float* weight, float eps, const int* positions,
+                     const float* cos_sin, int max_pos, const int* slots, void* pages, long long num_slots, void* q_out, int T,
+                     int H, int dim, int rank, int rot, int off_rot, int width, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (rot % 2 != 0 || off_rot < rank || width < off_rot + rot || max_pos < 1) return -10;
+  const Latent p{ld, num_slots, off_c, rank, rot, H, dim, off_rot, width, max_pos, eps};
+  const int warps = rot == 0 ? 1 : H + 1 < 8 ? H + 1 : 8;
+  auto go = [&](auto kern, auto tag) {
+    using E = decltype(tag);
+    tgi::launch(kern, dim3(T), dim3(32 * warps), 0, stream, static_cast<const E*>(proj), weight, positions, cos_sin, slots,
+                static_cast<E*>(pages), static_cast<E*>(q_out), p);
+    return done();
+  };
+  return f32 ? go(latent_store_kernel<float>, float()) : go(latent_store_kernel<bf16>, bf16());
+}
+
+}  // extern "C"

@@ -1,6 +1,6 @@
 // Kernels around the token mixers of hybrid decoders (attention layers between recurrent ones), each in a bf16 and
 // an fp32 build of the activations:
-//   residual add (fp32 stream) of one or two block outputs + one or two RMSNorms, optional row gather
+//   residual add (fp32 stream) of one or two block outputs + one or two RMSNorms or a LayerNorm, optional row gather
 //   embedding gather into the fp32 residual stream
 //   element-wise activation of a non-gated feed-forward, act(gate) * up of a gated one
 //   [causal short convolution ->] RoPE -> per-head RMS of q and k -> value mixing -> paged K / V store
@@ -17,73 +17,15 @@
 #include <type_traits>
 
 #include "launch.cuh"
+#include "mixer_util.cuh"
 
 namespace {
 
-using bf16 = __nv_bfloat16;
-
-__device__ __forceinline__ float to_f(float x) { return x; }
-__device__ __forceinline__ float to_f(bf16 x) { return __bfloat162float(x); }
-__device__ __forceinline__ void put(float* p, float v) { *p = v; }
-__device__ __forceinline__ void put(bf16* p, float v) { *p = __float2bfloat16(v); }
-// four consecutive elements (16-byte aligned fp32, 8-byte aligned bf16)
-__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
-__device__ __forceinline__ float4 load4(const bf16* p) {
-  const uint2 u = *reinterpret_cast<const uint2*>(p);
-  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
-  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
-  return make_float4(a.x, a.y, b.x, b.y);
-}
-__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
-__device__ __forceinline__ void store4(bf16* p, float4 v) {
-  __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
-  uint2 u;
-  u.x = *reinterpret_cast<uint32_t*>(&a);
-  u.y = *reinterpret_cast<uint32_t*>(&b);
-  *reinterpret_cast<uint2*>(p) = u;
-}
-
-__device__ __forceinline__ float warp_sum(float v) {
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-  return v;
-}
-// sum over the block, returned to every thread; `red` holds one float per warp plus the total
-__device__ __forceinline__ float block_sum(float v, float* red) {
-  v = warp_sum(v);
-  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
-  __syncthreads();
-  float t = 0.f;
-  for (int w = 0; w < static_cast<int>(blockDim.x >> 5); ++w) t += red[w];
-  __syncthreads();
-  return t;
-}
-__device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
-__device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
-// the same for values that came from, or end in, bf16: the hardware exponential and reciprocal (a few ulp of fp32)
-template <typename T>
-__device__ __forceinline__ float sigmoid_t(float x) { return sigmoid_f(x); }
-template <>
-__device__ __forceinline__ float sigmoid_t<bf16>(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
-template <typename T>
-__device__ __forceinline__ float silu_t(float x) { return x * sigmoid_t<T>(x); }
-template <>
-__device__ __forceinline__ float silu_t<float>(float x) { return silu_f(x); }
-
-// sequence that owns token t (cu[0] = 0 .. cu[B] = T)
-__device__ __forceinline__ int sequence_of(const int* __restrict__ cu, int B, int t) {
-  if (t < B && cu[t] <= t && cu[t + 1] > t) return t;       // one token per sequence up to here: decode steps
-  int lo = 0, hi = B - 1;
-  while (lo < hi) {
-    const int mid = (lo + hi + 1) >> 1;
-    if (cu[mid] <= t) lo = mid;
-    else hi = mid - 1;
-  }
-  return lo;
-}
+using namespace mixer;
 
 // ------------------------------------------------------------------------------------------------
-// r = residual (fp32) + scale * (d1 + d2) -> RMSNorm(r) * (offset + w1), and the same with w2.  One CTA per output row;
+// r = residual (fp32) + scale * (d1 + d2) -> RMSNorm(r) * (offset + w1) + b1 (`layer`: of r minus its mean), and the same with
+// w2 and no bias.  One CTA per output row;
 // `rows` (optional) picks the input row.  VPT float4 per thread stay in registers; VPT == 0: any width, read twice.
 // ------------------------------------------------------------------------------------------------
 template <typename T>
@@ -92,9 +34,10 @@ struct ResidualNorm {
   const float* residual;
   const int* rows;
   const T *w1, *w2;               // w2 null: one norm
+  const T* b1;                    // null: no bias
   T *o1, *o2;
   float* res_out;
-  int H;
+  int H, layer;
   float eps, scale, offset;
 };
 template <typename T, int VPT>
@@ -105,7 +48,7 @@ residual_norm_kernel(ResidualNorm<T> p) {
   __shared__ float red[33];
   const int row = p.rows != nullptr ? p.rows[blockIdx.x] : blockIdx.x, H = p.H;
   const size_t in = static_cast<size_t>(row) * H, ob = static_cast<size_t>(blockIdx.x) * H;
-  float sumsq = 0.f;
+  float sumsq = 0.f, sum = 0.f;
   if (VPT > 0) {
     float4 x[VPT > 0 ? VPT : 1];
 #pragma unroll
@@ -125,6 +68,18 @@ residual_norm_kernel(ResidualNorm<T> p) {
         if (p.res_out != nullptr) store4(p.res_out + ob + c, a);
         x[i] = a;
         sumsq += a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;
+        sum += (a.x + a.y) + (a.z + a.w);
+      }
+    }
+    if (p.layer) {                                         // deviations, then their squares
+      const float mean = block_sum(sum, red) / H;
+      sumsq = 0.f;
+#pragma unroll
+      for (int i = 0; i < VPT; ++i) {
+        if ((threadIdx.x + i * blockDim.x) * 4 < H) {
+          x[i].x -= mean; x[i].y -= mean; x[i].z -= mean; x[i].w -= mean;
+          sumsq += x[i].x * x[i].x + x[i].y * x[i].y + x[i].z * x[i].z + x[i].w * x[i].w;
+        }
       }
     }
     const float inv = 1.f / sqrtf(block_sum(sumsq, red) / H + p.eps);
@@ -133,13 +88,13 @@ residual_norm_kernel(ResidualNorm<T> p) {
       const int c = (threadIdx.x + i * blockDim.x) * 4;
       if (c < H) {
         const float4 y = make_float4(x[i].x * inv, x[i].y * inv, x[i].z * inv, x[i].w * inv);
-        auto put_norm = [&](const T* weight, T* out) {
-          const float4 w = load4(weight + c);
-          store4(out + ob + c, make_float4(y.x * (p.offset + w.x), y.y * (p.offset + w.y), y.z * (p.offset + w.z),
-                                           y.w * (p.offset + w.w)));
+        auto put_norm = [&](const T* weight, const T* bias, T* out) {
+          const float4 w = load4(weight + c), b = bias != nullptr ? load4(bias + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+          store4(out + ob + c, make_float4(fmaf(y.x, p.offset + w.x, b.x), fmaf(y.y, p.offset + w.y, b.y),
+                                           fmaf(y.z, p.offset + w.z, b.z), fmaf(y.w, p.offset + w.w, b.w)));
         };
-        put_norm(p.w1, p.o1);
-        if (p.w2 != nullptr) put_norm(p.w2, p.o2);
+        put_norm(p.w1, p.b1, p.o1);
+        if (p.w2 != nullptr) put_norm(p.w2, nullptr, p.o2);
       }
     }
   } else {
@@ -152,11 +107,21 @@ residual_norm_kernel(ResidualNorm<T> p) {
       const float a = value(c);
       if (p.res_out != nullptr) p.res_out[ob + c] = a;
       sumsq += a * a;
+      sum += a;
+    }
+    float mean = 0.f;
+    if (p.layer) {
+      mean = block_sum(sum, red) / H;
+      sumsq = 0.f;
+      for (int c = threadIdx.x; c < H; c += blockDim.x) {
+        const float a = value(c) - mean;
+        sumsq += a * a;
+      }
     }
     const float inv = 1.f / sqrtf(block_sum(sumsq, red) / H + p.eps);
     for (int c = threadIdx.x; c < H; c += blockDim.x) {
-      const float y = value(c) * inv;
-      put(p.o1 + ob + c, y * (p.offset + to_f(p.w1[c])));
+      const float y = (value(c) - mean) * inv;
+      put(p.o1 + ob + c, fmaf(y, p.offset + to_f(p.w1[c]), p.b1 != nullptr ? to_f(p.b1[c]) : 0.f));
       if (p.w2 != nullptr) put(p.o2 + ob + c, y * (p.offset + to_f(p.w2[c])));
     }
   }
@@ -633,16 +598,26 @@ attn_conv_run_kernel(const T* __restrict__ proj, long long ld, int off_k, int of
 
 // ------------------------------------------------------------------------------------------------
 // Paged attention for any head size, fp32 arithmetic.  One warp per (token, query head): each lane scores one key
-// of a group of 32, the group's softmax is exchanged by shuffles, and the lanes then split the value dimensions.
+// of a group of 32, the group's softmax is exchanged by shuffles, and the lanes then split the value dimensions.  Value
+// rows are `ldv` elements apart (values that are the first columns of the keys), `sink` has a score per head, `gate` a
+// pre-activation per token and head for the output.
 // ------------------------------------------------------------------------------------------------
 constexpr int kAttnWarps = 4;
-constexpr int kMaxOut = 16;        // value dimensions per lane: vdim <= 512
+constexpr int kMaxOut = 32;        // value dimensions per lane: vdim <= 1024
+template <typename T>
+struct AnyAttention {
+  float scale, softcap;             // softcap 0: scores as they are
+  int window, chunk;
+  const float* sink;                // [Hq] or null
+  const T* gate;                    // [T, ld_gate] or null
+  long long ld_gate;
+};
 template <typename T, int NV>
 __global__ void __launch_bounds__(kAttnWarps * 32)
 attn_any_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
                 const int* __restrict__ block_tables, const int* __restrict__ cu, const int* __restrict__ kv_lens,
-                T* __restrict__ out, int T_, int B, int max_blocks, int bs_shift, int Hq, int Hkv, int Dk, int Dv, float scale,
-                int window, int chunk, int sink) {
+                T* __restrict__ out, int T_, int B, int max_blocks, int bs_shift, int Hq, int Hkv, int Dk, int Dv, int ldv,
+                AnyAttention<T> a) {
   tgi::pdl_wait();
   tgi::pdl_trigger();
   extern __shared__ float sq[];
@@ -657,10 +632,10 @@ attn_any_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T*
   const int kvh = h / (Hq / Hkv);
   for (int i = lane; i < Dk; i += 32) qs[i] = to_f(q[(static_cast<size_t>(t) * Hq + h) * Dk + i]);
   __syncwarp();
-  int lo = window > 0 ? pos - window + 1 : 0;
-  if (chunk > 0 && pos > 0) lo = max(lo, pos - pos % chunk);
+  int lo = a.window > 0 ? pos - a.window + 1 : 0;
+  if (a.chunk > 0 && pos > 0) lo = max(lo, pos - pos % a.chunk);
   lo = max(lo, 0);
-  float m = sink ? 0.f : -INFINITY, l = sink ? 1.f : 0.f;
+  float m = a.sink != nullptr ? a.sink[h] : -INFINITY, l = a.sink != nullptr ? 1.f : 0.f;
   float o[NV];
 #pragma unroll
   for (int i = 0; i < NV; ++i) o[i] = 0.f;
@@ -686,7 +661,8 @@ attn_any_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T*
         acc = (a0 + a1) + (a2 + a3);
       }
       for (; i < Dk; ++i) acc = fmaf(to_f(kp[i]), qs[i], acc);
-      s = acc * scale;
+      s = acc * a.scale;
+      if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
     }
     float mx = s;
 #pragma unroll
@@ -702,13 +678,14 @@ attn_any_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T*
     for (int j = 0; j < cnt; ++j) {
       const float pj = __shfl_sync(0xffffffffu, pr, j);
       const long long rj = __shfl_sync(0xffffffffu, row, j);
-      const T* vp = v_cache + (static_cast<size_t>(rj) * Hkv + kvh) * Dv;
+      const T* vp = v_cache + (static_cast<size_t>(rj) * Hkv + kvh) * ldv;
 #pragma unroll
       for (int i = 0; i < NV; ++i)
         if (lane + 32 * i < Dv) o[i] = fmaf(pj, to_f(vp[lane + 32 * i]), o[i]);
     }
   }
-  const float inv = l > 0.f ? 1.f / l : 0.f;
+  float inv = l > 0.f ? 1.f / l : 0.f;
+  if (a.gate != nullptr) inv *= sigmoid_t<T>(to_f(a.gate[static_cast<size_t>(t) * a.ld_gate + h]));
 #pragma unroll
   for (int i = 0; i < NV; ++i)
     if (lane + 32 * i < Dv) put(out + (static_cast<size_t>(t) * Hq + h) * Dv + lane + 32 * i, o[i] * inv);
@@ -1268,9 +1245,11 @@ int done() { return cudaGetLastError() == cudaSuccess ? 0 : -3; }
 
 template <typename T>
 int residual_norm(const void* d1, const void* d2, const float* residual, const int* rows, const void* w1, const void* w2,
-                  void* o1, void* o2, float* res_out, int n, int H, float eps, float scale, float offset, cudaStream_t stream) {
+                  const void* b1, void* o1, void* o2, float* res_out, int n, int H, int layer, float eps, float scale,
+                  float offset, cudaStream_t stream) {
   const ResidualNorm<T> p{static_cast<const T*>(d1), static_cast<const T*>(d2), residual, rows, static_cast<const T*>(w1),
-                          static_cast<const T*>(w2), static_cast<T*>(o1), static_cast<T*>(o2), res_out, H, eps, scale, offset};
+                          static_cast<const T*>(w2), static_cast<const T*>(b1), static_cast<T*>(o1), static_cast<T*>(o2),
+                          res_out, H, layer, eps, scale, offset};
   if (H % 4 == 0 && H / 4 <= 4 * 1024) {
     const int vecs = H / 4;
     int threads = vecs >= 1024 ? 512 : ((vecs + 31) / 32) * 32;
@@ -1289,20 +1268,21 @@ int residual_norm(const void* d1, const void* d2, const float* residual, const i
 
 template <typename T>
 int attn_any(const void* q, const void* k, const void* v, const int* bt, const int* cu, const int* kv, void* out, int T_,
-             int B, int max_blocks, int bs_shift, int Hq, int Hkv, int Dk, int Dv, float scale, int window, int chunk,
-             int sink, cudaStream_t stream) {
+             int B, int max_blocks, int bs_shift, int Hq, int Hkv, int Dk, int Dv, int ldv, const AnyAttention<T>& a,
+             cudaStream_t stream) {
   const long long jobs = static_cast<long long>(T_) * Hq;
   const dim3 grid(static_cast<unsigned>((jobs + kAttnWarps - 1) / kAttnWarps)), block(kAttnWarps * 32);
   const size_t smem = static_cast<size_t>(kAttnWarps) * Dk * sizeof(float);
   if (smem > 48 * 1024 || Dv > 32 * kMaxOut) return -12;
   auto go = [&](auto kern) {
     tgi::launch(kern, grid, block, smem, stream, static_cast<const T*>(q), static_cast<const T*>(k), static_cast<const T*>(v),
-                bt, cu, kv, static_cast<T*>(out), T_, B, max_blocks, bs_shift, Hq, Hkv, Dk, Dv, scale, window, chunk, sink);
+                bt, cu, kv, static_cast<T*>(out), T_, B, max_blocks, bs_shift, Hq, Hkv, Dk, Dv, ldv, a);
     return done();
   };
   if (Dv <= 64) return go(attn_any_kernel<T, 2>);
   if (Dv <= 128) return go(attn_any_kernel<T, 4>);
   if (Dv <= 256) return go(attn_any_kernel<T, 8>);
+  if (Dv <= 512) return go(attn_any_kernel<T, 16>);
   return go(attn_any_kernel<T, kMaxOut>);
 }
 
@@ -1387,13 +1367,13 @@ int gated_norm(const float* o, const void* gate, long long ld, int off, const fl
 // `f32` selects the build: 1 = fp32 activations, weights and pages, 0 = bf16.
 extern "C" {
 
-// d2, w2 (with o2) and rows may be null; d1 null: the stream as it is
+// d2, w2 (with o2), b1 and rows may be null; d1 null: the stream as it is.  layer: LayerNorm instead of RMSNorm
 int tgi_residual_norm(int f32, const void* d1, const void* d2, const float* residual, const int* rows, const void* w1,
-                      const void* w2, void* o1, void* o2, float* res_out, int n, int H, float eps, float scale, float offset,
-                      cudaStream_t stream) {
+                      const void* w2, const void* b1, void* o1, void* o2, float* res_out, int n, int H, int layer, float eps,
+                      float scale, float offset, cudaStream_t stream) {
   if (n <= 0) return 0;
-  return f32 ? residual_norm<float>(d1, d2, residual, rows, w1, w2, o1, o2, res_out, n, H, eps, scale, offset, stream)
-             : residual_norm<bf16>(d1, d2, residual, rows, w1, w2, o1, o2, res_out, n, H, eps, scale, offset, stream);
+  return f32 ? residual_norm<float>(d1, d2, residual, rows, w1, w2, b1, o1, o2, res_out, n, H, layer, eps, scale, offset, stream)
+             : residual_norm<bf16>(d1, d2, residual, rows, w1, w2, b1, o1, o2, res_out, n, H, layer, eps, scale, offset, stream);
 }
 
 int tgi_embed_residual(int f32, const int* ids, const void* table, float* out, int T, int H, int vocab, float scale,
@@ -1524,17 +1504,20 @@ int tgi_attn_prep(int f32, const void* proj, long long ld, int off_k, int off_v,
   return finish();
 }
 
+// Value rows are `ldv` elements apart.  `sink` (optional): a score per head; `gate` (optional, [T, ld_gate]): the output of
+// head h is multiplied by the sigmoid of its column h.
 int tgi_attn_any(int f32, const void* q, const void* k_cache, const void* v_cache, const int* block_tables, const int* cu,
                  const int* kv_lens, void* out, int T, int B, int max_blocks, int block_size, int Hq, int Hkv, int Dk, int Dv,
-                 float scale, int window, int chunk, int sink, cudaStream_t stream) {
+                 int ldv, float scale, float softcap, int window, int chunk, const float* sink, const void* gate,
+                 long long ld_gate, cudaStream_t stream) {
   if (T <= 0 || B <= 0) return 0;
   if (Hq % Hkv != 0 || block_size <= 0 || (block_size & (block_size - 1)) != 0) return -10;
   int shift = 0;
   while ((1 << shift) < block_size) ++shift;
-  return f32 ? attn_any<float>(q, k_cache, v_cache, block_tables, cu, kv_lens, out, T, B, max_blocks, shift, Hq, Hkv, Dk, Dv,
-                               scale, window, chunk, sink, stream)
-             : attn_any<bf16>(q, k_cache, v_cache, block_tables, cu, kv_lens, out, T, B, max_blocks, shift, Hq, Hkv, Dk, Dv,
-                              scale, window, chunk, sink, stream);
+  return f32 ? attn_any<float>(q, k_cache, v_cache, block_tables, cu, kv_lens, out, T, B, max_blocks, shift, Hq, Hkv, Dk, Dv, ldv,
+                               {scale, softcap, window, chunk, sink, static_cast<const float*>(gate), ld_gate}, stream)
+             : attn_any<bf16>(q, k_cache, v_cache, block_tables, cu, kv_lens, out, T, B, max_blocks, shift, Hq, Hkv, Dk, Dv, ldv,
+                              {scale, softcap, window, chunk, sink, static_cast<const bf16*>(gate), ld_gate}, stream);
 }
 
 // Rows of the [rows][channels] convolution weights tgi_delta_prep wants for `taps` taps (the first rows are zero).

@@ -3,6 +3,7 @@
 //   tgi_moe_topk_softmax   softmax over the router logits + top-k (+ renormalisation), one warp per token
 //   tgi_moe_router         router product in fp32 (bf16 operands), split over K into partial sums
 //   tgi_moe_topk_sigmoid   sigmoid scores, top-k of score + correction, weights scaled to a given sum, one warp per token
+//   tgi_moe_topk_logits    top-k of logit + bias, weights the softmax over the chosen, one warp per token
 //   tgi_moe_sort           groups the (token, slot) pairs of the LOCAL experts by expert: per-expert counts
 //                          and offsets, position of every pair in the grouped order, and the inverse list
 //   tgi_moe_gather         copies the token rows into the grouped activation matrix
@@ -10,7 +11,7 @@
 //                          derived on the device from the per-expert counts.  Three epilogues: gate_up with
 //                          act(gate) * up fused (writes [rows, I]), up of an ungated expert with act fused, down with
 //                          the routing weight applied (writes [rows, H])
-//   tgi_moe_grouped_f32    the same two products of ungated experts in fp32 (FMA)
+//   tgi_moe_grouped_f32    the same products in fp32 (FMA)
 //   tgi_moe_combine        sums the top-k rows of every token in slot order (fixed order: bit-reproducible)
 //
 // Replaces, in the reference, `fused_topk` / `grouped_topk` + `moe_align_block_size` + the Triton
@@ -182,9 +183,11 @@ moe_router_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __re
 }
 
 // logits = sum of `parts` matrices [tokens, E]; s = sigmoid(logits); the k experts with the largest s + correction (ties go
-// to the lower index), weight scale * s / (sum of their s + 1e-20)
+// to the lower index), weight scale * s / (sum of their s + 1e-20).  SOFTMAX: the k experts with the largest logit +
+// correction, weight the softmax over those.
+template <bool SOFTMAX>
 __global__ void __launch_bounds__(128)
-moe_topk_sigmoid_kernel(const float* __restrict__ part, int parts, const float* __restrict__ correction, int tokens, int E,
+moe_topk_scores_kernel(const float* __restrict__ part, int parts, const float* __restrict__ correction, int tokens, int E,
                         int k, float scale, float* __restrict__ out_w, int* __restrict__ out_ids) {
   tgi::pdl_wait();
   tgi::pdl_trigger();
@@ -200,11 +203,11 @@ moe_topk_sigmoid_kernel(const float* __restrict__ part, int parts, const float* 
     if (e < E) {
       float z = 0.f;
       for (int p = 0; p < parts; ++p) z += part[(static_cast<size_t>(p) * tokens + t) * E + e];
-      s[i] = 1.f / (1.f + expf(-z));
+      s[i] = SOFTMAX ? z : 1.f / (1.f + expf(-z));
       v[i] = s[i] + (correction != nullptr ? correction[e] : 0.f);
     }
   }
-  float sum = 0.f, my_w = 0.f;
+  float sum = 0.f, my_w = 0.f, top = 0.f;
   int my_id = 0;
   for (int j = 0; j < k; ++j) {
     float best = -INFINITY, score = 0.f;
@@ -229,6 +232,10 @@ moe_topk_sigmoid_kernel(const float* __restrict__ part, int parts, const float* 
 #pragma unroll
     for (int i = 0; i < kMaxExperts / 32; ++i)
       if (i * 32 + lane == best_e) v[i] = -INFINITY;
+    if (SOFTMAX) {
+      if (j == 0) top = best;
+      score = expf(best - top);
+    }
     sum += score;
     if (lane == j) {
       my_w = score;
@@ -236,7 +243,7 @@ moe_topk_sigmoid_kernel(const float* __restrict__ part, int parts, const float* 
     }
   }
   if (lane < k) {
-    out_w[static_cast<size_t>(t) * k + lane] = my_w / (sum + 1e-20f) * scale;
+    out_w[static_cast<size_t>(t) * k + lane] = SOFTMAX ? my_w / sum : my_w / (sum + 1e-20f) * scale;
     out_ids[static_cast<size_t>(t) * k + lane] = my_id;
   }
 }
@@ -374,6 +381,8 @@ __device__ __forceinline__ float act_fn(float x, int act) {
     default: return x / (1.f + __expf(-1.702f * x));                                    // quick gelu
   }
 }
+
+__device__ __forceinline__ float act_fn_f32(float x, int act) { return act == 0 ? x / (1.f + expf(-x)) : act_fn(x, act); }
 
 struct TileWalk {
   // tile -> (expert, first row, rows of the expert left from there, weight tile)
@@ -621,8 +630,9 @@ int launch_grouped(const void* A, int rows_cap, const void* W, int e_local, int 
 }
 
 // ------------------------------------------------------------------------------------------------
-// fp32 products of ungated experts: 64 x 64 tiles, 256 threads with 4 x 4 sums each.  MODE 2: A rows are the tokens
-// order[row] / k of x, out = act(A W^T); MODE 1: A rows are grouped, out = topk_w[order[row]] * (A W^T).
+// fp32 products of experts: 64 x 64 tiles, 256 threads with 4 x 4 sums each.  MODE 2: A rows are the tokens order[row] / k
+// of x, out = act(A W^T); MODE 0: the same rows, W holds Nw gate rows and then Nw up rows, out = act(A Wg^T) * (A Wu^T);
+// MODE 1: A rows are grouped, out = topk_w[order[row]] * (A W^T).
 // grid (weight tiles, row tiles an expert layout can have)
 // ------------------------------------------------------------------------------------------------
 template <int MODE>
@@ -632,7 +642,8 @@ moe_grouped_f32_kernel(const float* __restrict__ A, const float* __restrict__ W,
                        const float* __restrict__ topk_w, float* __restrict__ out) {
   tgi::pdl_wait();
   tgi::pdl_trigger();
-  __shared__ float sa[16][68], sw[16][68];
+  constexpr int P = MODE == 0 ? 2 : 1;                     // products per output
+  __shared__ float sa[16][68], sw[P][16][68];
   int tile = blockIdx.y, e = 0;
   while (e < e_local && tile >= (offsets[e + 1] - offsets[e] + 63) / 64) {
     tile -= (offsets[e + 1] - offsets[e] + 63) / 64;
@@ -641,33 +652,37 @@ moe_grouped_f32_kernel(const float* __restrict__ A, const float* __restrict__ W,
   if (e == e_local) return;                                // block-uniform
   const int row0 = offsets[e] + tile * 64, rows = min(64, offsets[e + 1] - row0), n0 = blockIdx.x * 64;
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
-  float acc[4][4] = {};
+  float acc[P][4][4] = {};
   for (int k0 = 0; k0 < K; k0 += 16) {
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int r = ty + 16 * i, kk = k0 + tx;
-      float a = 0.f, w = 0.f;
+      float a = 0.f;
       if (kk < K && r < rows) {
         const int row = row0 + r;
-        a = A[static_cast<size_t>(MODE == 2 ? order[row] / k : row) * K + kk];
+        a = A[static_cast<size_t>(MODE != 1 ? order[row] / k : row) * K + kk];
       }
-      if (kk < K && n0 + r < Nw) w = W[(static_cast<size_t>(e) * Nw + n0 + r) * K + kk];
       sa[tx][r] = a;
-      sw[tx][r] = w;
+#pragma unroll
+      for (int q = 0; q < P; ++q)
+        sw[q][tx][r] = kk < K && n0 + r < Nw ? W[((static_cast<size_t>(e) * P + q) * Nw + n0 + r) * K + kk] : 0.f;
     }
     __syncthreads();
 #pragma unroll
     for (int q = 0; q < 16; ++q) {
-      float a[4], w[4];
+      float a[4], w[P][4];
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         a[i] = sa[q][4 * ty + i];
-        w[i] = sw[q][4 * tx + i];
+#pragma unroll
+        for (int u = 0; u < P; ++u) w[u][i] = sw[u][q][4 * tx + i];
       }
 #pragma unroll
-      for (int i = 0; i < 4; ++i)
+      for (int u = 0; u < P; ++u)
 #pragma unroll
-        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(a[i], w[j], acc[i][j]);
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) acc[u][i][j] = fmaf(a[i], w[u][j], acc[u][i][j]);
     }
     __syncthreads();
   }
@@ -680,7 +695,9 @@ moe_grouped_f32_kernel(const float* __restrict__ A, const float* __restrict__ W,
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + 4 * tx + j;
-      if (n < Nw) out[static_cast<size_t>(row) * Nw + n] = MODE == 2 ? act_fn(acc[i][j], act) : acc[i][j] * sc;
+      if (n >= Nw) continue;
+      const float y = acc[0][i][j];
+      out[static_cast<size_t>(row) * Nw + n] = MODE == 2 ? act_fn_f32(y, act) : MODE == 0 ? act_fn_f32(y, act) * acc[P - 1][i][j] : y * sc;
     }
   }
 }
@@ -736,20 +753,31 @@ int tgi_moe_topk_sigmoid(const float* part, int parts, const float* correction, 
                          float* out_w, int* out_ids, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (E < 1 || E > kMaxExperts || k < 1 || k > kMaxTopKSigmoid || k > E || parts < 1) return -30;
-  const cudaError_t err = tgi::launch(moe_topk_sigmoid_kernel, dim3((tokens + 3) / 4), dim3(128), 0, stream, part, parts,
+  const cudaError_t err = tgi::launch(moe_topk_scores_kernel<false>, dim3((tokens + 3) / 4), dim3(128), 0, stream, part, parts,
                                       correction, tokens, E, k, scale, out_w, out_ids);
   return err == cudaSuccess && cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
 
-// mode 2: out[entries, Nw] = act(x[order / k] W^T), mode 1: out[entries, Nw] = topk_w[order] * (A W^T); all fp32
+int tgi_moe_topk_logits(const float* part, int parts, const float* bias, int tokens, int E, int k, float* out_w, int* out_ids,
+                        cudaStream_t stream) {
+  if (tokens <= 0) return 0;
+  if (E < 1 || E > kMaxExperts || k < 1 || k > kMaxTopKSigmoid || k > E || parts < 1) return -30;
+  const cudaError_t err = tgi::launch(moe_topk_scores_kernel<true>, dim3((tokens + 3) / 4), dim3(128), 0, stream, part, parts,
+                                      bias, tokens, E, k, 1.f, out_w, out_ids);
+  return err == cudaSuccess && cudaGetLastError() == cudaSuccess ? 0 : -3;
+}
+
+// mode 2: out[entries, Nw] = act(x[order / k] W^T), mode 0: out[entries, Nw] = act(x[order / k] Wg^T) * (x[order / k] Wu^T) with
+// W [e_local, 2 Nw, K], mode 1: out[entries, Nw] = topk_w[order] * (A W^T); all fp32
 int tgi_moe_grouped_f32(int mode, const float* A, int entries, const float* W, int e_local, int k, int Nw, int K,
                         const int* offsets, const int* order, int act, const float* topk_w, float* out, cudaStream_t stream) {
   if (entries <= 0) return 0;
   if (e_local < 1 || e_local > kMaxExperts || k < 1) return -30;
   const dim3 grid((Nw + 63) / 64, entries / 64 + e_local);  // every expert may leave one tile partly filled
-  const cudaError_t err =
-      mode == 2 ? tgi::launch(moe_grouped_f32_kernel<2>, grid, dim3(256), 0, stream, A, W, offsets, order, e_local, k, Nw, K, act, topk_w, out)
-                : tgi::launch(moe_grouped_f32_kernel<1>, grid, dim3(256), 0, stream, A, W, offsets, order, e_local, k, Nw, K, act, topk_w, out);
+  auto go = [&](auto kern) {
+    return tgi::launch(kern, grid, dim3(256), 0, stream, A, W, offsets, order, e_local, k, Nw, K, act, topk_w, out);
+  };
+  const cudaError_t err = mode == 0 ? go(moe_grouped_f32_kernel<0>) : mode == 2 ? go(moe_grouped_f32_kernel<2>) : go(moe_grouped_f32_kernel<1>);
   return err == cudaSuccess && cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
 

@@ -66,7 +66,8 @@ def load():
                  "tgi_quant_set_pow2", "tgi_peer_set_quant_pow2", "tgi_gemm_bf16_ld", "tgi_residual_norm", "tgi_embed_residual",
                  "tgi_activation", "tgi_attn_prep", "tgi_attn_any", "tgi_delta_prep", "tgi_delta_scan", "tgi_decay_scan",
                  "tgi_gated_norm", "tgi_recurrent_pitch", "tgi_delta_tap_rows", "tgi_act_mul_any", "tgi_moe_router",
-                 "tgi_moe_router_splits", "tgi_moe_topk_sigmoid", "tgi_moe_grouped_f32", "tgi_moe_combine_f32"):
+                 "tgi_moe_router_splits", "tgi_moe_topk_sigmoid", "tgi_moe_topk_logits", "tgi_row_norm_store", "tgi_output_gate",
+                 "tgi_latent_store", "tgi_moe_grouped_f32", "tgi_moe_combine_f32"):
         if hasattr(_LIB, name):        # a library built for one family of models lacks the other families' kernels
             getattr(_LIB, name).restype = c_int
     _LIB.tgi_gemm_workspace_floats.restype = c_ll
@@ -421,8 +422,13 @@ def attention_pitch(dim: int, vdim: int, dtype: torch.dtype) -> Tuple[int, int]:
 
 def paged_attention(q, k_cache, v_cache, block_tables, cu_seqlens_q, kv_lens, scale, window=-1, softcap=0.0,
                     k_scale=None, v_scale=None, max_q=None, max_kv=None, nsplit: Optional[int] = None, horizon=None,
-                    chunk: int = 0, sink: bool = False):
+                    chunk: int = 0, sink=None):
     lib = load()
+    if sink is False:
+        sink = None
+    elif sink is True:
+        sink = _zero_sink(q.device, q.shape[1])
+    assert sink is None or (sink.dtype == torch.float32 and sink.shape == (q.shape[1],) and sink.is_contiguous())
     T, Hq, D = q.shape
     nblk, bs, Hkv, _ = k_cache.shape
     Dv = v_cache.shape[3]
@@ -431,13 +437,9 @@ def paged_attention(q, k_cache, v_cache, block_tables, cu_seqlens_q, kv_lens, sc
     if T == 0 or B == 0:
         return out
     if q.dtype == torch.float32 or D != Dv or D not in ATTN_HEAD_DIMS:
-        assert softcap <= 0 and horizon is None and k_cache.dtype == q.dtype and v_cache.dtype == q.dtype
-        _check(lib.tgi_attn_any(
-            c_int(1 if q.dtype == torch.float32 else 0), _ptr(q.contiguous()), _ptr(k_cache), _ptr(v_cache),
-            _ptr(block_tables), _ptr(cu_seqlens_q), _ptr(kv_lens), _ptr(out), c_int(T), c_int(B),
-            c_int(block_tables.shape[1]), c_int(bs), c_int(Hq), c_int(Hkv), c_int(D), c_int(Dv), c_float(scale),
-            c_int(window if window and window > 0 else -1), c_int(chunk), c_int(1 if sink else 0), _stream()), "attn_any")
-        return out
+        assert horizon is None and k_cache.dtype == q.dtype and v_cache.dtype == q.dtype
+        return _attention_any(q.contiguous(), k_cache, v_cache, Dv, block_tables, cu_seqlens_q, kv_lens, out, scale, softcap, window,
+                              chunk, sink, None)
     if max_q is None:
         max_q = int((cu_seqlens_q[1:] - cu_seqlens_q[:-1]).max().item())
     if max_kv is None:
@@ -464,7 +466,77 @@ def paged_attention(q, k_cache, v_cache, block_tables, cu_seqlens_q, kv_lens, sc
         _ptr(k_scale if fp8 else None), _ptr(v_scale if fp8 else None), _ptr(out), _ptr(part_o), _ptr(part_ml),
         c_int(B), c_int(max_q), c_int(block_tables.shape[1]), c_int(bs), c_int(nblk), c_int(Hq), c_int(Hkv), c_int(D),
         c_float(scale), c_float(softcap), c_int(window if window and window > 0 else -1), c_int(chunk),
-        c_int(1 if sink else 0), c_int(nsplit), c_int(1 if fp8 else 0), _ptr(horizon), _stream()), "paged_attention")
+        _ptr(sink), c_int(nsplit), c_int(1 if fp8 else 0), _ptr(horizon), _stream()), "paged_attention")
+    return out
+
+
+_ZERO_SINKS = {}
+
+
+def _zero_sink(device, heads: int) -> torch.Tensor:
+    """Scores of sinks that are 0 for every head (kept: captured decode steps read them)."""
+    key = (device, heads)
+    if key not in _ZERO_SINKS:
+        _ZERO_SINKS[key] = torch.zeros(heads, dtype=torch.float32, device=device)
+    return _ZERO_SINKS[key]
+
+
+def _attention_any(q, k_cache, v_cache, vdim, block_tables, cu_seqlens_q, kv_lens, out, scale, softcap, window, chunk, sink, gate):
+    """The kernel for head sizes without an instance and for fp32; ``vdim`` columns of every value row are read."""
+    T, Hq, D = q.shape
+    _, bs, Hkv, ldv = v_cache.shape
+    _check(load().tgi_attn_any(
+        _f32(q), _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(block_tables), _ptr(cu_seqlens_q), _ptr(kv_lens), _ptr(out), c_int(T),
+        c_int(kv_lens.shape[0]), c_int(block_tables.shape[1]), c_int(bs), c_int(Hq), c_int(Hkv), c_int(D), c_int(vdim), c_int(ldv),
+        c_float(scale), c_float(softcap), c_int(window if window and window > 0 else -1), c_int(chunk), _ptr(sink), _ptr(gate),
+        c_ll(0 if gate is None else gate.stride(0)), _stream()), "attn_any")
+    return out
+
+
+def latent_layout(rank: int, rot: int, dtype: torch.dtype) -> Tuple[int, int]:
+    """``(column of the rotated part, width)`` of a cached latent row."""
+    return rank, rank + rot
+
+
+def latent_store(proj, off_c, weight, eps, positions, cos_sin, slots, pages, q, off_rot, rank: int, rot: int, heads: int, dim: int):
+    assert proj.stride(1) == 1 and pages.is_contiguous() and pages.shape[2] == 1 and pages.dtype == proj.dtype == q.dtype
+    assert q.is_contiguous() and q.shape[2] == pages.shape[3] and weight.dtype == torch.float32 and cos_sin.shape[1] == rot
+    _check(load().tgi_latent_store(
+        _f32(proj), _ptr(proj), c_ll(proj.stride(0)), c_int(off_c), _ptr(weight), c_float(eps), _ptr(positions), _ptr(cos_sin),
+        c_int(cos_sin.shape[0]), _ptr(slots), _ptr(pages), c_ll(pages.shape[0] * pages.shape[1]), _ptr(q), c_int(proj.shape[0]),
+        c_int(heads), c_int(dim), c_int(rank), c_int(rot), c_int(off_rot), c_int(pages.shape[3]), _stream()), "latent_store")
+
+
+def latent_attention(q, pages, rank: int, block_tables, cu_seqlens_q, kv_lens, scale, window=-1, max_q=None, max_kv=None, gate=None):
+    T, H, _ = q.shape
+    out = q.new_empty(T, H, rank)
+    if T == 0:
+        return out
+    assert gate is None or (gate.stride(1) == 1 and gate.dtype == q.dtype)
+    return _attention_any(q, pages, pages, rank, block_tables, cu_seqlens_q, kv_lens, out, scale, 0.0, window, 0, None, gate)
+
+
+def row_norm_store(proj, offs, positions, slots, k_cache, v_cache, q_weight, k_weight, eps, num_heads: int, num_kv_heads: int,
+                   dim: int, vdim: int, width: int, temperature=None):
+    T = proj.shape[0]
+    q = torch.empty(T, num_heads, width, dtype=proj.dtype, device=proj.device)
+    assert proj.stride(1) == 1 and k_cache.dtype == proj.dtype and v_cache.dtype == proj.dtype
+    coef, every = temperature or (0.0, 0)
+    off_k, off_v = (offs[1], offs[2]) if k_weight is not None else (0, 0)
+    _check(load().tgi_row_norm_store(
+        _f32(proj), _ptr(proj), c_ll(proj.stride(0)), c_int(off_k), c_int(off_v), _ptr(positions), _ptr(slots), _ptr(q_weight),
+        _ptr(k_weight), _ptr(q), _ptr(k_cache), _ptr(v_cache), c_int(T), c_int(num_heads), c_int(num_kv_heads), c_int(dim),
+        c_int(vdim), c_int(width), c_int(k_cache.shape[3]), c_int(v_cache.shape[3]), c_ll(k_cache.shape[0] * k_cache.shape[1]),
+        c_float(eps), c_float(coef), c_int(every), _stream()), "row_norm_store")
+    return q
+
+
+def output_gate(x, gate, width: int):
+    T, H, pitch = x.shape
+    out = torch.empty(T, H * width, dtype=x.dtype, device=x.device)
+    assert x.is_contiguous() and gate.stride(1) == 1 and gate.dtype == x.dtype
+    _check(load().tgi_output_gate(_f32(x), _ptr(x), _ptr(gate), c_ll(gate.stride(0)), _ptr(out), c_int(T), c_int(H), c_int(pitch),
+                                  c_int(width), _stream()), "output_gate")
     return out
 
 
@@ -484,7 +556,7 @@ def embed_residual(ids, table, scale: float):
 
 
 def residual_norm(delta, residual, weight, eps, rows=None, keep: bool = True, scale: float = 1.0, unit_offset: bool = False,
-                  weight2=None):
+                  weight2=None, layer: bool = False, bias=None):
     H = residual.shape[1]
     n = residual.shape[0] if rows is None else rows.shape[0]
     d1, d2 = delta if isinstance(delta, tuple) else (delta, None)
@@ -496,9 +568,11 @@ def residual_norm(delta, residual, weight, eps, rows=None, keep: bool = True, sc
     else:
         res = dst = torch.empty(n, H, dtype=torch.float32, device=residual.device) if keep else None
     assert residual.dtype == torch.float32 and residual.is_contiguous()
+    assert bias is None or bias.dtype == weight.dtype
     assert all(d is None or (d.dtype == weight.dtype and d.is_contiguous() and d.shape == residual.shape) for d in (d1, d2))
     _check(load().tgi_residual_norm(_f32(weight), _ptr(d1), _ptr(d2), _ptr(residual), _ptr(rows), _ptr(weight), _ptr(weight2),
-                                    _ptr(out), _ptr(out2), _ptr(dst), c_int(n), c_int(H), c_float(eps), c_float(scale),
+                                    _ptr(bias), _ptr(out), _ptr(out2), _ptr(dst), c_int(n), c_int(H), c_int(1 if layer else 0),
+                                    c_float(eps), c_float(scale),
                                     c_float(1.0 if unit_offset else 0.0), _stream()), "residual_norm")
     return (out, res) if weight2 is None else (out, out2, res)
 
@@ -779,8 +853,8 @@ def moe_experts(x, w_gate_up, w_down, topk_weights, topk_ids, act="silu", first:
     return out
 
 
-def moe_route_sigmoid(x, weight, correction, top_k: int, scale: float):
-    """Router logits ``x @ weight^T`` in fp32, experts chosen by ``sigmoid + correction``, weights ``scale * s / sum(s)``."""
+def _router_logits(x, weight):
+    """``x @ weight^T`` in fp32 as partial sums ``[parts, T, E]`` over ranges of K, and their number."""
     lib = load()
     T, E = x.shape[0], weight.shape[0]
     if x.dtype == torch.bfloat16:
@@ -793,19 +867,40 @@ def moe_route_sigmoid(x, weight, correction, top_k: int, scale: float):
                "moe_router")
     else:
         part, splits = torch.nn.functional.linear(x, weight), 1
+    return part, splits
+
+
+def moe_route_sigmoid(x, weight, correction, top_k: int, scale: float):
+    """Router logits ``x @ weight^T`` in fp32, experts chosen by ``sigmoid + correction``, weights ``scale * s / sum(s)``."""
+    T, E = x.shape[0], weight.shape[0]
+    part, splits = _router_logits(x, weight)
     w = torch.empty(T, top_k, dtype=torch.float32, device=x.device)
     ids = torch.empty(T, top_k, dtype=torch.int32, device=x.device)
-    _check(lib.tgi_moe_topk_sigmoid(_ptr(part), c_int(splits), _ptr(correction), c_int(T), c_int(E), c_int(top_k), c_float(scale),
-                                    _ptr(w), _ptr(ids), _stream()), "moe_topk_sigmoid")
+    _check(load().tgi_moe_topk_sigmoid(_ptr(part), c_int(splits), _ptr(correction), c_int(T), c_int(E), c_int(top_k), c_float(scale),
+                                       _ptr(w), _ptr(ids), _stream()), "moe_topk_sigmoid")
     return w, ids
 
 
-def moe_plain_experts(x, w_up, w_down, topk_weights, topk_ids, act: str):
-    """Ungated experts ``w_up [E, I, H]``, ``w_down [E, H, I]`` (``ops.plain_expert_weights``) on their routed rows, in bf16
-    (grouped tcgen05 GEMMs) or fp32; no host synchronisation."""
+def moe_route_softmax(x, weight, bias, top_k: int):
+    """Experts of the ``top_k`` largest ``x @ weight^T + bias`` (fp32), weights the softmax over those."""
+    T, E = x.shape[0], weight.shape[0]
+    part, splits = _router_logits(x, weight)
+    w = torch.empty(T, top_k, dtype=torch.float32, device=x.device)
+    ids = torch.empty(T, top_k, dtype=torch.int32, device=x.device)
+    _check(load().tgi_moe_topk_logits(_ptr(part), c_int(splits), _ptr(bias), c_int(T), c_int(E), c_int(top_k), _ptr(w), _ptr(ids),
+                                      _stream()), "moe_topk_logits")
+    return w, ids
+
+
+def moe_plain_experts(x, w_up, w_down, topk_weights, topk_ids, act: str, gated: bool = False):
+    """Experts ``w_up [E, I, H]`` (``gated``: ``[E, 2 I, H]``), ``w_down [E, H, I]`` (``ops.plain_expert_weights``) on their
+    routed rows, in bf16 (grouped tcgen05 GEMMs) or fp32; no host synchronisation."""
     lib, st, s = load(), state(x.device), _stream()
     T, H = x.shape
     E, I, Hp = w_up.shape
+    up = 2
+    if gated:
+        I, up = I // 2, 0
     k = topk_ids.shape[1]
     n = T * k
     new = lambda *shape, dtype=x.dtype: torch.empty(*shape, dtype=dtype, device=x.device)
@@ -819,8 +914,8 @@ def moe_plain_experts(x, w_up, w_down, topk_weights, topk_ids, act: str):
     _check(lib.tgi_moe_sort(_ptr(topk_ids), c_int(n), c_int(0), c_int(E), _ptr(pos), _ptr(order), _ptr(offsets), s), "moe_sort")
     code = c_int(_ACT_CODES[act])
     if x.dtype == torch.float32:
-        for mode, src, w, dst in ((2, x, w_up, hidden), (1, hidden, w_down, y)):
-            _check(lib.tgi_moe_grouped_f32(c_int(mode), _ptr(src), c_int(n), _ptr(w), c_int(E), c_int(k), c_int(w.shape[1]),
+        for mode, src, w, dst in ((up, x, w_up, hidden), (1, hidden, w_down, y)):
+            _check(lib.tgi_moe_grouped_f32(c_int(mode), _ptr(src), c_int(n), _ptr(w), c_int(E), c_int(k), c_int(dst.shape[1]),
                                            c_int(w.shape[2]), _ptr(offsets), _ptr(order), code, _ptr(topk_weights), _ptr(dst), s),
                    "moe_grouped_f32")
         _check(lib.tgi_moe_combine_f32(_ptr(y), _ptr(pos), c_int(T), c_int(k), c_int(Hp), _ptr(out), s), "moe_combine_f32")
@@ -828,7 +923,7 @@ def moe_plain_experts(x, w_up, w_down, topk_weights, topk_ids, act: str):
     grouped = new(n, Hp)
     _check(lib.tgi_moe_gather(_ptr(x), _ptr(order), _ptr(offsets), c_int(E), c_int(k), c_int(Hp), c_int(n), _ptr(grouped), s),
            "moe_gather")
-    for mode, src, w, dst in ((2, grouped, w_up, hidden), (1, hidden, w_down, y)):
+    for mode, src, w, dst in ((up, grouped, w_up, hidden), (1, hidden, w_down, y)):
         _check(lib.tgi_moe_grouped_gemm(c_int(mode), _ptr(src), c_int(n), _ptr(w), c_int(E), c_int(w.shape[1]), c_int(w.shape[2]),
                                         _ptr(offsets), code, _ptr(topk_weights), _ptr(order), _ptr(dst), c_int(st.sm_count),
                                         _ptr(st.status), s), "moe_grouped_gemm")

@@ -129,11 +129,11 @@ def paged_attention(
     max_kv: Optional[int] = None,
     horizon: Optional[torch.Tensor] = None,
     chunk: int = 0,
-    sink: bool = False,
+    sink=None,
 ) -> torch.Tensor:
     """Causal attention of ragged queries over paged KV (covers prefill, chunked prefill and decode).
     ``horizon[t]`` (optional) replaces the causal limit of query row ``t`` by a later position.  With ``chunk`` a row
-    sees only keys ``t`` with ``t // chunk == pos // chunk``; ``sink`` adds ``exp(0)`` to the softmax denominator.
+    sees only keys ``t`` with ``t // chunk == pos // chunk``; ``sink`` adds ``exp(sink[h])`` (``True``: ``exp(0)``) to the softmax denominator.
 
     Query ``i`` (0-based inside its sequence's chunk of ``n`` queries) of a sequence with ``L`` KV
     tokens sits at absolute position ``L - n + i`` and attends to KV positions ``<=`` its own
@@ -181,8 +181,9 @@ def paged_attention(
         if chunk > 0:
             mask &= torch.div(kpos, chunk, rounding_mode="floor") == torch.div(qpos, chunk, rounding_mode="floor")
         scores = scores.masked_fill(~mask.unsqueeze(0), float("-inf"))
-        if sink:
-            p = torch.softmax(torch.cat([scores, scores.new_zeros(Hq, n, 1)], dim=-1), dim=-1)[..., :-1]
+        if sink is not None and sink is not False:
+            extra = scores.new_zeros(Hq) if sink is True else sink.float()
+            p = torch.softmax(torch.cat([scores, extra.view(Hq, 1, 1).expand(Hq, n, 1)], dim=-1), dim=-1)[..., :-1]
         else:
             p = torch.softmax(scores, dim=-1)
         out[s:e] = torch.einsum("hnl,lhd->nhd", p, v).to(q.dtype)
@@ -311,8 +312,15 @@ def moe_route_sigmoid(x, weight, correction, top_k: int, scale: float):
     return w / (w.sum(-1, keepdim=True) + 1e-20) * scale, idx
 
 
-def moe_plain_experts(x, w_up, w_down, topk_weights, topk_ids, act: str):
+def moe_route_softmax(x, weight, bias, top_k: int):
+    z, idx = torch.topk(F.linear(x.float(), weight.float(), bias), top_k, dim=-1)
+    return torch.softmax(z, dim=-1), idx
+
+
+def moe_plain_experts(x, w_up, w_down, topk_weights, topk_ids, act: str, gated: bool = False):
     """``w_up[E, I, H]``, ``w_down[E, H, I]``: sum over a token's experts of weight times ``down(act(up x))``."""
+    if gated:
+        return moe_experts(x, w_up, w_down, topk_weights, topk_ids, act)
     out = torch.zeros(x.shape, dtype=torch.float32, device=x.device)
     for e in range(w_up.shape[0]):
         tok, slot = (topk_ids == e).nonzero(as_tuple=True)
@@ -369,15 +377,17 @@ def embed_residual(ids, table, scale: float = 1.0):
 
 
 def residual_norm(delta, residual, weight, eps: float, rows=None, keep: bool = True, scale: float = 1.0,
-                  unit_offset: bool = False, weight2=None):
+                  unit_offset: bool = False, weight2=None, layer: bool = False, bias=None):
     r = residual
     if delta is not None:
         parts = delta if isinstance(delta, tuple) else (delta,)
         r = residual + scale * sum(d.float() for d in parts)
     if rows is not None:
         r = r[rows.long()]
-    x = r * torch.rsqrt(r.pow(2).mean(-1, keepdim=True) + eps)
-    ys = tuple((x * (w.float() + (1.0 if unit_offset else 0.0))).to(w.dtype) for w in (weight, weight2) if w is not None)
+    d = r - r.mean(-1, keepdim=True) if layer else r
+    x = d * torch.rsqrt(d.pow(2).mean(-1, keepdim=True) + eps)
+    b = 0.0 if bias is None else bias.float()
+    ys = tuple((x * (w.float() + (1.0 if unit_offset else 0.0)) + b).to(w.dtype) for w in (weight, weight2) if w is not None)
     return ys + (r if keep else None,)
 
 
@@ -440,6 +450,53 @@ def rotate_norm_store(proj, offs, positions, cos_sin, slots, k_cache, v_cache, n
     k_cache.view(-1, num_kv_heads, k_cache.shape[3])[idx, :, :dim] = k[ok].to(k_cache.dtype)
     v_cache.view(-1, num_kv_heads, v_cache.shape[3])[idx, :, :vdim] = v.view(T, num_kv_heads, vdim)[ok].to(v_cache.dtype)
     return F.pad(q, (0, k_cache.shape[3] - dim)).to(proj_dtype)
+
+
+def _store_rows(pages, slots, rows, col: int = 0):
+    """``rows[T, heads, n]`` to columns ``col ..`` of the tokens' slots."""
+    ok = (slots >= 0).nonzero(as_tuple=True)[0]
+    flat = pages.view(-1, pages.shape[2], pages.shape[3])
+    flat[slots[ok].long(), :, col:col + rows.shape[2]] = rows[ok].to(pages.dtype)
+
+
+def _row_rms(x, weight, eps: float):
+    x = x.float()
+    return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * weight
+
+
+def row_norm_store(proj, offs, positions, slots, k_cache, v_cache, q_weight, k_weight, eps: float, num_heads, num_kv_heads, dim,
+                   vdim, width, temperature=None):
+    T = proj.shape[0]
+    q = _row_rms(proj[:, offs[0]:offs[0] + num_heads * dim], q_weight, eps)
+    if temperature is not None:
+        coef, every = temperature
+        q = q * (1.0 + coef * torch.log(torch.div(positions + 1, every, rounding_mode="floor").float() + 1.0)).unsqueeze(1)
+    if k_weight is not None:
+        k = _row_rms(proj[:, offs[1]:offs[1] + num_kv_heads * dim], k_weight, eps)
+        _store_rows(k_cache, slots, k.view(T, num_kv_heads, dim))
+        _store_rows(v_cache, slots, proj[:, offs[2]:offs[2] + num_kv_heads * vdim].reshape(T, num_kv_heads, vdim))
+    return F.pad(q.view(T, num_heads, dim), (0, width - dim)).to(proj.dtype)
+
+
+def output_gate(x, gate, width: int):
+    T = x.shape[0]
+    return (x[:, :, :width].reshape(T, -1).float() * torch.sigmoid(gate.float())).to(x.dtype)
+
+
+def latent_store(proj, off_c, weight, eps: float, positions, cos_sin, slots, pages, q, off_rot, rank, rot, heads, dim):
+    T = proj.shape[0]
+    _store_rows(pages, slots, _row_rms(proj[:, off_c:off_c + rank], weight, eps).unsqueeze(1))
+    if rot:
+        cs = cos_sin[positions.long()]
+        turn = lambda x: rotate(x.float(), cs[:, :rot // 2], cs[:, rot // 2:], rot, False)
+        _store_rows(pages, slots, turn(proj[:, off_c + rank:off_c + rank + rot].unsqueeze(1)), off_rot)
+        q[:, :, off_rot:off_rot + rot] = turn(proj[:, :heads * (dim + rot)].reshape(T, heads, dim + rot)[..., dim:]).to(q.dtype)
+
+
+def latent_attention(q, pages, rank, block_tables, cu_seqlens_q, kv_lens, scale: float, window: int = -1, max_q=None, max_kv=None,
+                     gate=None):
+    o = paged_attention(q, pages, pages[..., :rank].contiguous(), block_tables, cu_seqlens_q, kv_lens, scale, window)
+    return o if gate is None else (o.float() * torch.sigmoid(gate.float()).unsqueeze(2)).to(o.dtype)
 
 
 def delta_inputs(proj, offs, a_pre, conv_t, a_log, dt_bias, cu, kv_lens, state_slots, conv_state, kv_heads, heads, dim,

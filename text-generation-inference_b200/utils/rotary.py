@@ -68,6 +68,18 @@ def scaled_frequencies(base: float, dim: int, scaling: Optional[Tuple[float, flo
     return torch.where(wave < original / high, f, torch.where(wave > original / low, f / factor, mid))
 
 
+def yarn_frequencies(base: float, dim: int, scaling: Tuple[float, float, float, float]) -> Tuple[torch.Tensor, float]:
+    """fp64 YaRN frequencies for ``scaling = (factor, fast, slow, original length)`` and the factor on cos and sin: pairs that
+    turn more than ``fast`` times over the original length keep their frequency, those that turn less than ``slow`` times
+    have it divided by ``factor``, those between are blended."""
+    factor, fast, slow, original = scaling
+    f = scaled_frequencies(base, dim)
+    lo = max(math.floor(_yarn_find_correction_dim(fast, dim, base, original)), 0)
+    hi = min(math.ceil(_yarn_find_correction_dim(slow, dim, base, original)), dim - 1)
+    ramp = ((torch.arange(dim // 2, dtype=torch.float64) - lo) / max(hi - lo, 0.001)).clamp(0, 1)
+    return f / factor * ramp + f * (1 - ramp), 0.1 * math.log(factor) + 1.0
+
+
 class RotaryTable:
     """cos/sin table for one model.
 
@@ -96,11 +108,11 @@ class RotaryTable:
         return torch.cat([freqs.cos() * mscale, freqs.sin() * mscale], dim=-1).contiguous()
 
     @classmethod
-    def from_frequencies(cls, freq: torch.Tensor, max_positions: int, neox: bool = True) -> "RotaryTable":
-        """Table of the given fp64 frequencies, with the angles formed in fp64 (an fp32 product of a position in the
+    def from_frequencies(cls, freq: torch.Tensor, max_positions: int, neox: bool = True, amplitude: float = 1.0) -> "RotaryTable":
+        """Table of the given fp64 frequencies (cos and sin times ``amplitude``), with the angles formed in fp64 (an fp32 product of a position in the
         thousands and a frequency near 1 is off by 1e-4)."""
         ang = torch.outer(torch.arange(max_positions, dtype=torch.float64), freq.double())
-        return cls(torch.cat([ang.cos(), ang.sin()], dim=-1).float().contiguous(), 2 * freq.numel(), neox)
+        return cls((amplitude * torch.cat([ang.cos(), ang.sin()], dim=-1)).float().contiguous(), 2 * freq.numel(), neox)
 
     @classmethod
     def from_config(cls, config, dim: int, base: float, max_positions: int, neox: bool = True) -> "RotaryTable":

@@ -219,7 +219,7 @@ class Weights:
         # (old prefix, new prefix) pairs: a name that starts with the old prefix is also looked up under the
         # new one (checkpoints of one architecture published under different module layouts)
         self.renames = list(renames or [])
-        # the checkpoint names its tensors without the ".weight" suffix the layers ask for
+        # the checkpoint names its tensors without the ".weight" suffix the layers ask for, its biases "*.b"
         self.bare_names = bare_names
         self.device = torch.device(device)
         self.dtype = dtype
@@ -244,6 +244,8 @@ class Weights:
                 names.append(new + name[len(old):])
         if self.bare_names and name.endswith(".weight"):
             names.append(name[:-len(".weight")])
+        elif self.bare_names and name.endswith(".bias"):
+            names.append(name[:-len(".bias")] + ".b")
         return names
 
     def resolve(self, name: str) -> Tuple[SafetensorsFile, str]:
