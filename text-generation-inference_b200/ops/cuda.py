@@ -67,7 +67,7 @@ def load():
                  "tgi_activation", "tgi_attn_prep", "tgi_attn_any", "tgi_delta_prep", "tgi_delta_scan", "tgi_decay_scan",
                  "tgi_gated_norm", "tgi_recurrent_pitch", "tgi_delta_tap_rows", "tgi_act_mul_any", "tgi_moe_router",
                  "tgi_moe_router_splits", "tgi_moe_topk_sigmoid", "tgi_moe_topk_logits", "tgi_row_norm_store", "tgi_output_gate",
-                 "tgi_latent_store", "tgi_moe_grouped_f32", "tgi_moe_combine_f32"):
+                 "tgi_latent_store", "tgi_latent_rows", "tgi_latent_attention", "tgi_moe_grouped_f32", "tgi_moe_combine_f32"):
         if hasattr(_LIB, name):        # a library built for one family of models lacks the other families' kernels
             getattr(_LIB, name).restype = c_int
     _LIB.tgi_gemm_workspace_floats.restype = c_ll
@@ -164,6 +164,7 @@ class _DeviceState:
                               device=device)
         self.attn_part_o = None
         self.attn_part_ml = None
+        self.kept = {}
 
 
 _STATES = {}
@@ -494,7 +495,12 @@ def _attention_any(q, k_cache, v_cache, vdim, block_tables, cu_seqlens_q, kv_len
 
 
 def latent_layout(rank: int, rot: int, dtype: torch.dtype) -> Tuple[int, int]:
-    """``(column of the rotated part, width)`` of a cached latent row."""
+    """``(column of the rotated part, width)`` of a cached latent row: both parts start at multiples of 64 columns where the
+    tensor-core kernel takes the row."""
+    if dtype == torch.bfloat16:
+        values, rotated = (rank + 63) // 64, (rot + 63) // 64
+        if load().tgi_latent_rows(c_int(values + rotated), c_int(values), c_ll(1)) > 0:
+            return 64 * values, 64 * (values + rotated)
     return rank, rank + rot
 
 
@@ -508,12 +514,42 @@ def latent_store(proj, off_c, weight, eps, positions, cos_sin, slots, pages, q, 
 
 
 def latent_attention(q, pages, rank: int, block_tables, cu_seqlens_q, kv_lens, scale, window=-1, max_q=None, max_kv=None, gate=None):
-    T, H, _ = q.shape
+    """Tensor-core kernel for bf16 rows in 64-column pieces on pages of 16 tokens, ``tgi_attn_any`` otherwise."""
+    lib = load()
+    T, H, width = q.shape
+    B = kv_lens.shape[0]
+    assert gate is None or (gate.stride(1) == 1 and gate.dtype == q.dtype)
+    assert q.is_contiguous() and pages.is_contiguous() and pages.shape[3] == width and pages.dtype == q.dtype
+    values = (rank + 63) // 64
+    if q.dtype == torch.bfloat16 and width % 64 == 0 and pages.shape[1] == 16 and max_q is not None:
+        N = int(lib.tgi_latent_rows(c_int(width // 64), c_int(values), c_ll(max_q * H)))
+        if N > 0:
+            out = q.new_empty(T, H, 64 * values)
+            st = state(q.device)
+            part = _latent_parts(st, N, 64 * values, B * ((H + N - 1) // N)) if max_q == 1 else (None,) * 3
+            _check(lib.tgi_latent_attention(
+                _ptr(q), _ptr(pages), _ptr(block_tables), _ptr(cu_seqlens_q), _ptr(kv_lens), _ptr(gate),
+                c_ll(0 if gate is None else gate.stride(0)), _ptr(out), *map(_ptr, part), c_int(T), c_int(B), c_int(max_q),
+                c_int(block_tables.shape[1]), c_int(pages.shape[0]), c_int(H), c_int(width // 64), c_int(values), c_int(N),
+                c_float(scale), c_int(window if window and window > 0 else -1), c_int(1 << 30), c_int(st.sm_count),
+                _ptr(st.status), _stream()), "latent_attention")
+            return out
     out = q.new_empty(T, H, rank)
     if T == 0:
         return out
-    assert gate is None or (gate.stride(1) == 1 and gate.dtype == q.dtype)
     return _attention_any(q, pages, pages, rank, block_tables, cu_seqlens_q, kv_lens, out, scale, 0.0, window, 0, None, gate)
+
+
+def _latent_parts(st, N: int, cols: int, items: int):
+    """Workspace of a persistent latent attention (kept: captured decode steps use it)."""
+    key = ("latent", N, cols)
+    if key not in st.kept:
+        st.kept[key] = (torch.empty(2 * st.sm_count * N * cols, dtype=torch.float32, device=st.device),
+                        torch.empty(2 * st.sm_count * N * 2, dtype=torch.float32, device=st.device))
+    items = max(1024, 1 << (items - 1).bit_length())
+    if ("range", items) not in st.kept:
+        st.kept["range", items] = torch.zeros(2 * items, dtype=torch.int32, device=st.device)
+    return (*st.kept[key], st.kept["range", items])
 
 
 def row_norm_store(proj, offs, positions, slots, k_cache, v_cache, q_weight, k_weight, eps, num_heads: int, num_kv_heads: int,
