@@ -2,17 +2,20 @@
 // all query heads share: value columns first (the latent), then columns that only the keys have (a rotated part).  A row is
 // read from memory once per tile of query rows; a query row is a (token, head) pair.
 //
-// A CTA owns N query rows (16, 32 or 64) and walks a range of keys in tiles of 128.  Both products are transposed, so that
-// the 128 keys (or 128 value columns) are the rows of the MMA and a tile of few query rows wastes nothing:
-//   S^T = K Q^T     M 128 (keys) x N x K width; the tile's slabs of 64 columns are multiplied as they land
-//   P^T = softmax   four warps, a key per thread: column maxima by a transposing butterfly and shared memory, P^T as bf16
-//                   rows [key][N] in shared memory (MN-major operand B)
-//   O^T = V^T P^T   M 128 (value columns) x N x K 128 (keys), one product per 128 value columns; V^T is the K tile as it
+// A CTA owns N query rows (16, 32 or 64) and walks a range of keys in tiles of 64.  Both products are transposed, so that
+// keys (or value columns) are the rows of the MMA and a tile of few query rows wastes nothing:
+//   S^T = K Q^T     M 64 (keys) x N x K width
+//   P^T = softmax   four warps, half of the query rows of a key per thread: column maxima by a transposing butterfly and
+//                   shared memory, P^T as bf16 rows [key][N] in shared memory (MN-major operand B)
+//   O^T = V^T P^T   M 128 (value columns) x N x K 64 (keys), one product per 128 value columns; V^T is the K tile as it
 //                   lies, taken as the MN-major operand A
 // The output stays in registers of the output warps (a value column per thread, N query rows), which rescale it and add
-// the tile's product.  The K tile is held once: a pair of slabs is loaded again as soon as its O^T product is done, the
-// key-only slabs as soon as S^T is.  Pages (16 tokens) are fetched as TMA boxes of 16 rows x 128 bytes, the query rows as
-// boxes of N rows.
+// the tile's product.  S^T, P^T and O^T are double-buffered and S^T of a tile is issued before O^T of the tile in front of
+// it when the tile has landed by then.
+//
+// A page (16 tokens) is one TMA box: [8 tokens x 128 bytes] atoms of the 128-byte swizzle, first along the row, then the
+// other 8 tokens.  Groups of 8 keys are thus `slabs` KB apart in shared memory, which both operand descriptors take as a
+// stride; a copy of 2 KB boxes (page x 128 bytes) ran at half the rate, a thread's copies issue one after the other.
 //
 // Decode steps (one token per sequence) run persistently: the key tiles of all sequences form one list that the CTAs
 // share out evenly; a CTA's first and last piece may be parts of a sequence and go to a workspace that a second kernel
@@ -32,9 +35,9 @@ using namespace sm100;
 
 namespace {
 
-constexpr int kKeys = 128, kPage = 16;
-constexpr int kSlab = kKeys * 128;              // bytes of 64 columns of a K tile
-constexpr int kMaxSlabs = 12, kMaxSeqs = 1024;
+constexpr int kKeys = 64, kPage = 16;
+constexpr int kMaxSlabs = 12, kMaxSeqs = 1024, kMaxStages = 4;
+constexpr int kPTile = kKeys * 128;             // bytes of a P^T tile
 constexpr float kLog2e = 1.4426950408889634f;
 
 struct LatentParams {
@@ -44,7 +47,7 @@ struct LatentParams {
   __nv_bfloat16* out;             // [T * H, out_cols]
   float *part_o, *part_ml;        // [2 * CTAs][N][out_cols] and [2 * CTAs][N][2]
   int* range;                     // [items][2]: first and last CTA of an item (persistent)
-  int B, max_blocks, num_blocks, H, out_cols, slabs, value_slabs, window, persistent, most;
+  int B, max_blocks, num_blocks, H, out_cols, slabs, value_slabs, stages, window, persistent, most;
   float scale_log2;
   int* status;
 };
@@ -52,11 +55,13 @@ struct LatentParams {
 __device__ __forceinline__ void report(int* status, int code) {
   if (status != nullptr) atomicCAS(status, 0, code);
 }
-__device__ __forceinline__ uint64_t desc_mn(uint32_t addr, uint32_t lbo) {      // MN-major, 128-byte swizzle
+// 128-byte swizzle.  K-major: groups of 8 rows `sbo` bytes apart.  MN-major: groups of 8 K rows `sbo` bytes apart, the next
+// 64 elements of M or N `lbo` bytes further.
+__device__ __forceinline__ uint64_t make_desc(uint32_t addr, uint32_t lbo, uint32_t sbo) {
   uint64_t d = 0;
   d |= static_cast<uint64_t>((addr & 0x3FFFF) >> 4);
   d |= static_cast<uint64_t>(lbo >> 4) << 16;
-  d |= static_cast<uint64_t>(1024 >> 4) << 32;
+  d |= static_cast<uint64_t>(sbo >> 4) << 32;
   d |= static_cast<uint64_t>(1) << 46;
   d |= static_cast<uint64_t>(2) << 61;
   return d;
@@ -84,11 +89,11 @@ __device__ __forceinline__ void tmem_load(uint32_t addr, float (&v)[W]) {
 #pragma unroll
   for (int i = 0; i < W; ++i) v[i] = __uint_as_float(r[i]);
 }
-// W values per lane -> lane l gets the maximum (sum) of value l % W over the warp
-template <int W, bool SUM>
-__device__ __forceinline__ float column_reduce(float (&v)[W], int lane) {
+// C values per lane -> lane l gets the maximum (sum) of value l % C over the 16 lanes of its half warp
+template <int C, bool SUM>
+__device__ __forceinline__ float column_reduce(float (&v)[C], int lane) {
 #pragma unroll
-  for (int o = W / 2; o >= 1; o >>= 1) {
+  for (int o = C / 2; o >= 1; o >>= 1) {
     const bool up = (lane & o) != 0;
 #pragma unroll
     for (int i = 0; i < o; ++i) {
@@ -98,7 +103,7 @@ __device__ __forceinline__ float column_reduce(float (&v)[W], int lane) {
     }
   }
 #pragma unroll
-  for (int o = W; o < 32; o <<= 1) {
+  for (int o = C; o < 16; o <<= 1) {
     const float got = __shfl_xor_sync(0xffffffffu, v[0], o);
     v[0] = SUM ? v[0] + got : fmaxf(v[0], got);
   }
@@ -148,15 +153,17 @@ __device__ __forceinline__ int sequence_at(const int* prefix, int B, int items, 
 template <int N>
 struct Walk {
   long long g, end, total;        // persistent: tiles of the list that are left, and all
-  int items;
+  int items, ctas;                // CTAs that have work: at least two tiles each
   __device__ __forceinline__ void start(const LatentParams& p, const int* prefix) {
     items = (p.H + N - 1) / N;
     g = 0;
     end = 1;
     if (p.persistent) {
       total = static_cast<long long>(prefix[p.B]) * items;
-      g = total * blockIdx.x / gridDim.x;
-      end = total * (blockIdx.x + 1) / gridDim.x;
+      ctas = static_cast<int>(min(static_cast<long long>(gridDim.x), (total + 1) / 2));
+      const int cta = min(static_cast<int>(blockIdx.x), ctas);
+      g = ctas > 0 ? total * cta / ctas : 0;
+      end = cta < ctas ? total * (cta + 1) / ctas : g;
     }
   }
   __device__ __forceinline__ bool next(const LatentParams& p, const int* prefix, Piece& w) {
@@ -171,7 +178,7 @@ struct Walk {
       w.tiles = static_cast<int>(min(static_cast<long long>(nt - w.first), end - g));
       w.part = w.first == 0 && w.tiles == nt ? -1 : (w.first == 0 ? 1 : 0);
       w.item = w.b * items + rt;
-      w.last_cta = static_cast<int>(((g - w.first + nt) * gridDim.x - 1) / total);
+      w.last_cta = static_cast<int>(((g - w.first + nt) * ctas - 1) / total);
       g += w.tiles;
     } else {
       w.b = blockIdx.y;
@@ -207,54 +214,77 @@ struct Waiter {
   }
 };
 
+// one look at a barrier, without suspending
+__device__ __forceinline__ bool mbar_test(uint64_t* bar, uint32_t parity) {
+  uint32_t ok;
+  asm volatile(
+      "{\n\t.reg .pred P;\n\t"
+      "mbarrier.test_wait.parity.shared::cta.b64 P, [%1], %2;\n\t"
+      "selp.b32 %0, 1, 0, P;\n\t}"
+      : "=r"(ok)
+      : "r"(smem_u32(bar)), "r"(parity)
+      : "memory");
+  return ok != 0;
+}
+// box of a page: 64 columns x 8 tokens x slabs x 2
+__device__ __forceinline__ void tma_load_page(void* dst, const CUtensorMap* map, uint64_t* bar, int group) {
+  asm volatile(
+      "cp.async.bulk.tensor.4d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%3, %3, %3, %4}], [%2];"
+      ::"r"(smem_u32(dst)), "l"(reinterpret_cast<uint64_t>(map)), "r"(smem_u32(bar)), "r"(0), "r"(group)
+      : "memory");
+}
+
 template <int N, int OG>
 __global__ void __launch_bounds__(256 + 128 * OG, 1)
 latent_attention_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const LatentParams p) {
   constexpr int W = N < 32 ? N : 32;            // columns per TMEM load
+  constexpr int C = W / 2, NC = N / W;          // columns of a load that a softmax thread works on, loads per tile
   constexpr int NB = N == 64 ? 1 : 2;           // blocks of 128 value columns per output warp group
   extern __shared__ __align__(1024) uint8_t smem[];
   if ((smem_u32(smem) & 1023u) != 0u) {         // uniform over the CTA, before anything is allocated
     if (threadIdx.x == 0) report(p.status, kErrSmemLayout);
     return;
   }
-  const int blocks = (p.value_slabs + 1) / 2, held = max(p.slabs, 2 * blocks);
-  uint8_t* sK = smem;
-  uint8_t* sQ = sK + held * kSlab;              // [slab][N rows of 128 bytes]
-  uint8_t* sP = sQ + p.slabs * N * 128;         // [key][64 columns]
-  float* s_max = reinterpret_cast<float*>(sP + kKeys * 128);      // [4][N] maxima of the softmax warps
+  const int blocks = (p.value_slabs + 1) / 2, tile_bytes = p.slabs * kKeys * 128, group_bytes = p.slabs * 1024;
+  uint8_t* sK = smem;                           // [stage][group of 8 keys][slab][8 x 128 bytes]
+  uint8_t* sQ = sK + p.stages * tile_bytes;     // [slab][N rows of 128 bytes]
+  uint8_t* sP = sQ + p.slabs * N * 128;         // [2][key][64 columns]
+  float* s_max = reinterpret_cast<float*>(sP + 2 * kPTile);       // [4][N] maxima (sums) of the softmax warps
   float* s_m = s_max + 4 * N;                   // [N]
-  float* s_alpha = s_m + N;                     // [N]
-  float* s_l = s_alpha + N;                     // [N] factor of the output
+  float* s_alpha = s_m + N;                     // [2][N]
+  float* s_l = s_alpha + 2 * N;                 // [N] factor of the output
   int* s_lo = reinterpret_cast<int*>(s_l + N);  // [N] first and last visible key of a row
   int* s_hi = s_lo + N;
   uint64_t* bars = reinterpret_cast<uint64_t*>(s_hi + N);
-  uint64_t* k_full = bars;                      // [kMaxSlabs]
-  uint64_t* k_free = bars + kMaxSlabs;          // [kMaxSlabs / 2] by the O^T product of a block
-  uint64_t* kk_free = k_free + kMaxSlabs / 2;   // key-only slabs, by S^T
-  uint64_t* q_full = kk_free + 1;
+  uint64_t* k_full = bars;                      // [kMaxStages]
+  uint64_t* k_free = k_full + kMaxStages;       // [kMaxStages]
+  uint64_t* s_full = k_free + kMaxStages;       // [2]
+  uint64_t* p_ready = s_full + 2;               // [2]
+  uint64_t* o_full = p_ready + 2;               // [2]
+  uint64_t* o_free = o_full + 2;                // [2]
+  uint64_t* q_full = o_free + 2;
   uint64_t* q_free = q_full + 1;
-  uint64_t* s_full = q_full + 2;
-  uint64_t* p_ready = q_full + 3;
-  uint64_t* o_full = q_full + 4;
-  uint64_t* o_free = q_full + 5;
-  uint64_t* l_ready = q_full + 6;
-  uint64_t* l_free = q_full + 7;
-  uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(q_full + 8);
+  uint64_t* l_ready = q_full + 2;
+  uint64_t* l_free = q_full + 3;
+  uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(q_full + 4);
   int* prefix = reinterpret_cast<int*>(tmem_holder + 4);          // [B + 1], persistent only
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   uint32_t cols = 32;
-  while (static_cast<int>(cols) < N * (1 + blocks)) cols <<= 1;
+  while (static_cast<int>(cols) < 2 * N * (1 + blocks)) cols <<= 1;
   if (threadIdx.x == 0) {
-    for (int i = 0; i < kMaxSlabs; ++i) mbar_init(&k_full[i], 1);
-    for (int i = 0; i < kMaxSlabs / 2; ++i) mbar_init(&k_free[i], 1);
-    mbar_init(kk_free, 1);
+    for (int i = 0; i < kMaxStages; ++i) {
+      mbar_init(&k_full[i], 1);
+      mbar_init(&k_free[i], 1);
+    }
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(&s_full[i], 1);
+      mbar_init(&p_ready[i], 4);
+      mbar_init(&o_full[i], 1);
+      mbar_init(&o_free[i], 4 * OG);
+    }
     mbar_init(q_full, 1);
     mbar_init(q_free, 1);
-    mbar_init(s_full, 1);
-    mbar_init(p_ready, 4);
-    mbar_init(o_full, 1);
-    mbar_init(o_free, 4 * OG);
     mbar_init(l_ready, 4);
     mbar_init(l_free, 4 * OG);
     fence_barrier_init();
@@ -271,7 +301,7 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
-  const uint32_t tS = *tmem_holder, tO = tS + N;
+  const uint32_t tS = *tmem_holder, tO = tS + 2 * N;       // S^T: two buffers of N columns, O^T: two of `blocks` x N
   Waiter wait{p.status, false};
   Walk<N> walk;
   walk.start(p, prefix);
@@ -279,195 +309,219 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
   int j = 0, np = 0;                            // tiles and pieces so far
 
   if (warp == 0) {
-    // ---------------- TMA producer: a box of 16 rows x 128 bytes per page and slab, spread over the lanes ----------------
+    // ---------------- TMA producer ----------------
     bool ok = true;
-    auto slab_pair = [&](int s0, int count, int blk, bool go) {     // slabs s0 .. s0 + count - 1 (at most two)
-      if (lane == 0 && go)
-        for (int i = 0; i < count; ++i) mbar_arrive_expect_tx(&k_full[s0 + i], kSlab);
-      __syncwarp();
-      const int s = s0 + (lane >> 3), pg = lane & 7;
-      if (go && (lane >> 3) < count)
-        tma_load_2d(sK + s * kSlab + pg * (kPage * 128), &tmK, &k_full[s], s * 64, blk * kPage);
-    };
+    int stage = 0, round = 0;                   // of tile j
     while (ok && walk.next(p, prefix, w)) {
-      if (np > 0) ok = wait(q_free, (np - 1) & 1, kErrProducerWait);
-      ok = __shfl_sync(0xffffffffu, ok ? 1 : 0, 0) != 0;
-      if (!ok) break;
-      if (lane == 0) mbar_arrive_expect_tx(q_full, p.slabs * N * 128);
-      __syncwarp();
-      if (lane < p.slabs) tma_load_2d(sQ + lane * N * 128, &tmQ, q_full, lane * 64, w.q_row);
       for (int i = 0; i < w.tiles && ok; ++i, ++j) {
-        const int page = (w.t_lo + (w.first + i) * kKeys) / kPage + (lane & 7);
+        const int page = (w.t_lo + (w.first + i) * kKeys) / kPage + (lane & 3);
         int blk = 0;
         if (page < p.max_blocks) blk = p.block_tables[static_cast<size_t>(w.b) * p.max_blocks + page];
         blk = min(max(blk, 0), p.num_blocks - 1);          // pages past the sequence are masked later
-        for (int s = p.value_slabs; s < p.slabs && ok; s += 2) {
-          if (s == p.value_slabs && j > 0) ok = wait(kk_free, (j - 1) & 1, kErrProducerWait);
+        if (i == 0) {
+          if (np > 0) ok = wait(q_free, (np - 1) & 1, kErrProducerWait);
           ok = __shfl_sync(0xffffffffu, ok ? 1 : 0, 0) != 0;
-          slab_pair(s, min(2, p.slabs - s), blk, ok);
+          if (!ok) break;
+          if (lane == 0) mbar_arrive_expect_tx(q_full, p.slabs * N * 128);
+          __syncwarp();
+          if (lane < p.slabs) tma_load_2d(sQ + lane * N * 128, &tmQ, q_full, lane * 64, w.q_row);
         }
-        for (int b = 0; b < blocks && ok; ++b) {
-          if (j > 0) ok = wait(&k_free[b], (j - 1) & 1, kErrProducerWait);
-          ok = __shfl_sync(0xffffffffu, ok ? 1 : 0, 0) != 0;
-          slab_pair(2 * b, min(2, p.value_slabs - 2 * b), blk, ok);
-        }
+        if (round > 0) ok = wait(&k_free[stage], (round - 1) & 1, kErrProducerWait);
+        ok = __shfl_sync(0xffffffffu, ok ? 1 : 0, 0) != 0;
+        if (!ok) break;
+        if (lane == 0) mbar_arrive_expect_tx(&k_full[stage], tile_bytes);
+        __syncwarp();
+        if (lane < 4) tma_load_page(sK + stage * tile_bytes + lane * 2 * group_bytes, &tmK, &k_full[stage], 2 * blk);
+        if (++stage == p.stages) stage = 0, ++round;
       }
       ++np;
     }
-    // copies in flight must land before the CTA's shared memory goes away (after a failed wait: also those of the
-    // tile that was being requested, as far as they were)
+    // copies in flight must land before the CTA's shared memory goes away
     if (lane == 0) {
-      for (int s = 0; s < p.slabs; ++s) {
-        if (j > 0) mbar_wait(&k_full[s], (j - 1) & 1);
-        if (!ok) mbar_wait(&k_full[s], j & 1);
+      for (int s = 0; s < p.stages; ++s) {
+        const int uses = round + (s < stage ? 1 : 0);
+        if (uses > 0) mbar_wait(&k_full[s], (uses - 1) & 1);
       }
+      if (np > 0) mbar_wait(q_full, (np - 1) & 1);
     }
   } else if (warp == 1) {
     // ---------------- MMA issuer ----------------
     if (elect_one()) {
-      constexpr uint32_t id_s = (1u << 4) | (1u << 7) | (1u << 10) | ((static_cast<uint32_t>(N) >> 3) << 17) | ((128u >> 4) << 24);
-      constexpr uint32_t id_o = id_s | (1u << 15) | (1u << 16);          // both operands MN-major
+      constexpr uint32_t id = (1u << 4) | (1u << 7) | (1u << 10) | ((static_cast<uint32_t>(N) >> 3) << 17);
+      constexpr uint32_t id_s = id | ((64u >> 4) << 24), id_o = id | ((128u >> 4) << 24) | (1u << 15) | (1u << 16);    // O^T: both MN-major
       const uint32_t q_addr = smem_u32(sQ), k_addr = smem_u32(sK), p_addr = smem_u32(sP);
-      bool ok = true;
-      while (ok && walk.next(p, prefix, w)) {
-        ok = wait(q_full, np & 1, kErrMmaWaitFull);
-        for (int i = 0; i < w.tiles && ok; ++i, ++j) {
-          // S^T: key-only slabs first, they land first
-          for (int x = 0; x < p.slabs && ok; ++x) {
-            const int s = x < p.slabs - p.value_slabs ? p.value_slabs + x : x - (p.slabs - p.value_slabs);
-            ok = wait(&k_full[s], j & 1, kErrMmaWaitFull);
-            if (!ok) break;
-            tc_fence_after();
-#pragma unroll
-            for (int k = 0; k < 4; ++k)
-              mma_f16(tS, make_desc_sw128(k_addr + s * kSlab) + (k * 32 >> 4), make_desc_sw128(q_addr + s * N * 128) + (k * 32 >> 4), id_s,
-                      x > 0 || k > 0 ? 1u : 0u);
-          }
-          if (!ok) break;
-          tc_commit(s_full);
-          tc_commit(kk_free);
-          if (i + 1 == w.tiles) tc_commit(q_free);
-          ok = wait(p_ready, j & 1, kErrMmaWaitFull);
-          if (!ok) break;
-          tc_fence_after();
-          for (int b = 0; b < blocks; ++b) {
-#pragma unroll
-            for (int k = 0; k < 8; ++k)                    // 16 keys: two groups of eight 128-byte rows
-              mma_f16(tO + b * N, desc_mn(k_addr + 2 * b * kSlab + k * 2048, kSlab), desc_mn(p_addr + k * 2048, kSlab), id_o,
-                      k > 0 ? 1u : 0u);
-            tc_commit(&k_free[b]);
-          }
-          tc_commit(o_full);
+      bool ok = true, more;
+      int i = 0, stage = 0, round = 0, o_stage = 0;        // S^T: tile of the piece w, its stage; O^T: its stage
+      auto next_tile = [&]() {
+        if (j > 0 || np > 0) {
+          ++i;
+          if (++stage == p.stages) stage = 0, ++round;
+          if (i < w.tiles) return true;
         }
-        ++np;
+        i = 0;
+        ++np;                                              // pieces begun
+        return walk.next(p, prefix, w);
+      };
+      auto landed = [&]() { return mbar_test(&k_full[stage], round & 1) && (i > 0 || mbar_test(q_full, (np - 1) & 1)); };
+      auto issue_s = [&](int tile) {
+        if (i == 0 && !wait(q_full, (np - 1) & 1, kErrMmaWaitFull)) return false;
+        if (!wait(&k_full[stage], round & 1, kErrMmaWaitFull)) return false;
+        tc_fence_after();
+        const uint32_t a = k_addr + stage * tile_bytes, d = tS + (tile & 1) * N;
+        for (int x = 0; x < p.slabs; ++x) {
+#pragma unroll
+          for (int k = 0; k < 4; ++k)                      // 16 columns (32 bytes) per MMA
+            mma_f16(d, make_desc(a + x * 1024, 16, group_bytes) + (k * 32 >> 4), make_desc(q_addr + x * N * 128, 16, 1024) + (k * 32 >> 4),
+                    id_s, x > 0 || k > 0 ? 1u : 0u);
+        }
+        tc_commit(&s_full[tile & 1]);
+        if (i + 1 == w.tiles) tc_commit(q_free);
+        return true;
+      };
+      more = next_tile();
+      if (more) ok = issue_s(0);
+      while (more && ok) {
+        uint64_t* ready = &p_ready[j & 1];
+        const uint32_t phase = (j >> 1) & 1;
+        more = next_tile();
+        bool issued = false;
+        if (more) {
+          for (uint32_t polls = 0; polls < (1u << 22) && !issued; ++polls) {
+            if (landed()) {
+              ok = issue_s(j + 1);
+              issued = true;
+            } else if (mbar_test(ready, phase)) {
+              break;
+            }
+          }
+        }
+        if (!ok || !wait(ready, phase, kErrMmaWaitFull)) break;
+        tc_fence_after();
+        const uint32_t a = k_addr + o_stage * tile_bytes, b = p_addr + (j & 1) * kPTile, d = tO + (j & 1) * blocks * N;
+        for (int x = 0; x < blocks; ++x) {
+#pragma unroll
+          for (int k = 0; k < 4; ++k)                      // 16 keys per MMA: two groups of eight rows
+            mma_f16(d + x * N, make_desc(a + 2 * x * 1024 + 2 * k * group_bytes, 1024, group_bytes), make_desc(b + k * 2048, 16, 1024), id_o,
+                    k > 0 ? 1u : 0u);
+        }
+        tc_commit(&o_full[j & 1]);
+        tc_commit(&k_free[o_stage]);
+        if (++o_stage == p.stages) o_stage = 0;
+        if (more && !issued) ok = issue_s(j + 1);
+        ++j;
       }
     }
   } else if (warp >= 4 && warp < 8) {
-    // ---------------- softmax: a key per thread ----------------
-    const int quarter = warp & 3, key = quarter * 32 + lane;
-    const uint32_t addr = tS + (static_cast<uint32_t>(quarter * 32) << 16);
+    // ---------------- softmax: a key and half of the columns of every load per thread ----------------
+    const int quarter = warp & 3, tid = quarter * 32 + lane, half = lane >> 4, key = quarter * 16 + (lane & 15);
+    const uint32_t addr = tS + (static_cast<uint32_t>(quarter * 32) << 16);       // rows 16 q .. 16 q + 15 in the first 16 lanes
     while (walk.next(p, prefix, w)) {
-      const int t_end = w.t_lo + w.first * kKeys;          // first key of the piece
-      float l[N];
+      float l[NC][C];
 #pragma unroll
-      for (int c = 0; c < N; ++c) l[c] = 0.f;
+      for (int x = 0; x < NC; ++x)
+#pragma unroll
+        for (int c = 0; c < C; ++c) l[x][c] = 0.f;
       float m = -INFINITY;                                 // thread c < N: running maximum of row c
-      if (key < N) {
-        const int pos = w.pos0 + (w.row0 % p.H + min(key, w.rows - 1)) / p.H;
-        s_lo[key] = first_visible(pos, p.window);
-        s_hi[key] = pos;
+      if (tid < N) {
+        const int pos = w.pos0 + (w.row0 % p.H + min(tid, w.rows - 1)) / p.H;
+        s_lo[tid] = first_visible(pos, p.window);
+        s_hi[tid] = pos;
       }
       asm volatile("bar.sync 1, 128;" ::: "memory");
       // keys that every row sees
       const int lo_all = first_visible(w.pos1, p.window), hi_all = w.pos0;
       for (int i = 0; i < w.tiles; ++i, ++j) {
-        const int t0 = t_end + i * kKeys, t = t0 + key;
+        const int buf = j & 1;
+        const int t0 = w.t_lo + (w.first + i) * kKeys, t = t0 + key;
         const bool plain = t0 >= lo_all && t0 + kKeys - 1 <= hi_all;
-        auto score = [&](float x, int c) {
-          return plain || (t >= s_lo[c] && t <= s_hi[c]) ? x * p.scale_log2 : -INFINITY;
-        };
-        wait(s_full, j & 1, kErrEpilogueWait);
+        wait(&s_full[buf], (j >> 1) & 1, kErrEpilogueWait);
         tc_fence_after();
+        float x[NC][C];
 #pragma unroll
-        for (int c0 = 0; c0 < N; c0 += W) {
-          float v[W];
-          tmem_load<W>(addr + c0, v);
+        for (int n = 0; n < NC; ++n) {
+          float v[W], y[C];
+          tmem_load<W>(addr + buf * N + n * W, v);
 #pragma unroll
-          for (int c = 0; c < W; ++c) v[c] = score(v[c], c0 + c);
-          const float mx = column_reduce<W, false>(v, lane);
-          if (lane < W) s_max[quarter * N + c0 + lane] = mx;
+          for (int c = 0; c < C; ++c) {                    // the upper lanes take over the second half of the columns
+            const float got = __shfl_xor_sync(0xffffffffu, v[c + C], 16);
+            x[n][c] = (half ? got : v[c]) * p.scale_log2;
+            if (!plain) {
+              const int col = n * W + half * C + c;
+              if (t < s_lo[col] || t > s_hi[col]) x[n][c] = -INFINITY;
+            }
+            y[c] = x[n][c];
+          }
+          const float mx = column_reduce<C, false>(y, lane);
+          if ((lane & 15) < C) s_max[quarter * N + n * W + half * C + (lane & 15)] = mx;
         }
-        // the last tile's output has been taken: its factors and its P^T are free
-        if (j > 0) wait(o_free, (j - 1) & 1, kErrEpilogueWait);
+        // the output of the tile before the last has been taken: its factors and its P^T are free
+        if (j > 1) wait(&o_free[buf], ((j >> 1) - 1) & 1, kErrEpilogueWait);
         asm volatile("bar.sync 1, 128;" ::: "memory");
-        if (key < N) {
-          const float mn = fmaxf(fmaxf(fmaxf(s_max[key], s_max[N + key]), fmaxf(s_max[2 * N + key], s_max[3 * N + key])), m);
-          s_alpha[key] = mn == -INFINITY ? 1.f : ex2(m - mn);
-          s_m[key] = mn == -INFINITY ? 0.f : mn;
+        if (tid < N) {
+          const float mn = fmaxf(fmaxf(fmaxf(s_max[tid], s_max[N + tid]), fmaxf(s_max[2 * N + tid], s_max[3 * N + tid])), m);
+          s_alpha[buf * N + tid] = mn == -INFINITY ? 1.f : ex2(m - mn);
+          s_m[tid] = mn == -INFINITY ? 0.f : mn;
           m = mn;
         }
         asm volatile("bar.sync 1, 128;" ::: "memory");
+        uint8_t* row = sP + buf * kPTile + key * 128;
 #pragma unroll
-        for (int c0 = 0; c0 < N; c0 += W) {
-          float v[W];
-          tmem_load<W>(addr + c0, v);
+        for (int n = 0; n < NC; ++n) {
+          const int col0 = n * W + half * C;
 #pragma unroll
-          for (int c = 0; c < W; c += 8) {
+          for (int c = 0; c < C; c += 8) {
             uint32_t packed[4];
 #pragma unroll
             for (int e = 0; e < 8; e += 4) {
-              const float4 mm = *reinterpret_cast<const float4*>(s_m + c0 + c + e);
-              const float4 al = *reinterpret_cast<const float4*>(s_alpha + c0 + c + e);
-              const float pr[4] = {ex2(score(v[c + e], c0 + c + e) - mm.x), ex2(score(v[c + e + 1], c0 + c + e + 1) - mm.y),
-                                   ex2(score(v[c + e + 2], c0 + c + e + 2) - mm.z), ex2(score(v[c + e + 3], c0 + c + e + 3) - mm.w)};
-              l[c0 + c + e] = fmaf(l[c0 + c + e], al.x, pr[0]);
-              l[c0 + c + e + 1] = fmaf(l[c0 + c + e + 1], al.y, pr[1]);
-              l[c0 + c + e + 2] = fmaf(l[c0 + c + e + 2], al.z, pr[2]);
-              l[c0 + c + e + 3] = fmaf(l[c0 + c + e + 3], al.w, pr[3]);
-              const __nv_bfloat162 a = __floats2bfloat162_rn(pr[0], pr[1]), b = __floats2bfloat162_rn(pr[2], pr[3]);
-              packed[e / 2] = *reinterpret_cast<const uint32_t*>(&a);
-              packed[e / 2 + 1] = *reinterpret_cast<const uint32_t*>(&b);
+              const float4 mm = *reinterpret_cast<const float4*>(s_m + col0 + c + e);
+              const float4 al = *reinterpret_cast<const float4*>(s_alpha + buf * N + col0 + c + e);
+              float* xs = &x[n][c + e];
+              float* ls = &l[n][c + e];
+              const float pr[4] = {ex2(xs[0] - mm.x), ex2(xs[1] - mm.y), ex2(xs[2] - mm.z), ex2(xs[3] - mm.w)};
+              ls[0] = fmaf(ls[0], al.x, pr[0]);
+              ls[1] = fmaf(ls[1], al.y, pr[1]);
+              ls[2] = fmaf(ls[2], al.z, pr[2]);
+              ls[3] = fmaf(ls[3], al.w, pr[3]);
+              const __nv_bfloat162 lo = __floats2bfloat162_rn(pr[0], pr[1]), hi = __floats2bfloat162_rn(pr[2], pr[3]);
+              packed[e / 2] = *reinterpret_cast<const uint32_t*>(&lo);
+              packed[e / 2 + 1] = *reinterpret_cast<const uint32_t*>(&hi);
             }
-            *reinterpret_cast<uint4*>(sP + key * 128 + ((((c0 + c) >> 3) ^ (key & 7)) << 4)) =
-                make_uint4(packed[0], packed[1], packed[2], packed[3]);
+            *reinterpret_cast<uint4*>(row + ((((col0 + c) >> 3) ^ (key & 7)) << 4)) = make_uint4(packed[0], packed[1], packed[2], packed[3]);
           }
         }
         fence_proxy_async();
         tc_fence_before();
         __syncwarp();
-        if (lane == 0) mbar_arrive(p_ready);
+        if (lane == 0) mbar_arrive(&p_ready[buf]);
       }
       // sums over the keys; what the output is multiplied by
 #pragma unroll
-      for (int c0 = 0; c0 < N; c0 += W) {
-        float v[W];
-#pragma unroll
-        for (int c = 0; c < W; ++c) v[c] = l[c0 + c];
-        const float sum = column_reduce<W, true>(v, lane);
-        if (lane < W) s_max[quarter * N + c0 + lane] = sum;
+      for (int n = 0; n < NC; ++n) {
+        const float sum = column_reduce<C, true>(l[n], lane);
+        if ((lane & 15) < C) s_max[quarter * N + n * W + half * C + (lane & 15)] = sum;
       }
       if (np > 0) wait(l_free, (np - 1) & 1, kErrEpilogueWait);
       asm volatile("bar.sync 1, 128;" ::: "memory");
-      if (key < N) {
-        const float sum = (s_max[key] + s_max[N + key]) + (s_max[2 * N + key] + s_max[3 * N + key]);
+      if (tid < N) {
+        const float sum = (s_max[tid] + s_max[N + tid]) + (s_max[2 * N + tid] + s_max[3 * N + tid]);
         float f = 1.f;
         if (w.part < 0) {
-          if (p.persistent && key == 0) p.range[2 * w.item] = p.range[2 * w.item + 1] = 0;
+          if (p.persistent && tid == 0) p.range[2 * w.item] = p.range[2 * w.item + 1] = 0;
           f = sum > 0.f ? 1.f / sum : 0.f;
-          if (p.gate != nullptr && key < w.rows) {
-            const int row = w.q_row + key;
+          if (p.gate != nullptr && tid < w.rows) {
+            const int row = w.q_row + tid;
             f *= __fdividef(1.f, 1.f + __expf(-__bfloat162float(p.gate[static_cast<long long>(row / p.H) * p.ld_gate + row % p.H])));
           }
         } else {
-          if (key == 0 && w.first == 0) {
+          if (tid == 0 && w.first == 0) {
             p.range[2 * w.item] = blockIdx.x;
             p.range[2 * w.item + 1] = w.last_cta;
           }
-          float* ml = p.part_ml + (static_cast<size_t>(2 * blockIdx.x + w.part) * N + key) * 2;
+          float* ml = p.part_ml + (static_cast<size_t>(2 * blockIdx.x + w.part) * N + tid) * 2;
           ml[0] = m;
           ml[1] = sum;
         }
-        s_l[key] = f;
+        s_l[tid] = f;
       }
       __syncwarp();
       if (lane == 0) mbar_arrive(l_ready);
@@ -484,7 +538,8 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
 #pragma unroll
         for (int c = 0; c < N; ++c) o[x][c] = 0.f;
       for (int i = 0; i < w.tiles; ++i, ++j) {
-        wait(o_full, j & 1, kErrEpilogueWait);
+        const int buf = j & 1;
+        wait(&o_full[buf], (j >> 1) & 1, kErrEpilogueWait);
         tc_fence_after();
 #pragma unroll
         for (int x = 0; x < NB; ++x) {
@@ -493,10 +548,10 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
 #pragma unroll
           for (int c0 = 0; c0 < N; c0 += W) {
             float v[W];
-            tmem_load<W>(addr + b * N + c0, v);
+            tmem_load<W>(addr + (buf * blocks + b) * N + c0, v);
 #pragma unroll
             for (int c = 0; c < W; c += 4) {
-              const float4 al = *reinterpret_cast<const float4*>(s_alpha + c0 + c);
+              const float4 al = *reinterpret_cast<const float4*>(s_alpha + buf * N + c0 + c);
               o[x][c0 + c] = fmaf(o[x][c0 + c], al.x, v[c]);
               o[x][c0 + c + 1] = fmaf(o[x][c0 + c + 1], al.y, v[c + 1]);
               o[x][c0 + c + 2] = fmaf(o[x][c0 + c + 2], al.z, v[c + 2]);
@@ -506,7 +561,7 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
         }
         tc_fence_before();
         __syncwarp();
-        if (lane == 0) mbar_arrive(o_free);
+        if (lane == 0) mbar_arrive(&o_free[buf]);
       }
       wait(l_ready, np & 1, kErrEpilogueWait);
       float* part = p.part_o + static_cast<size_t>(2 * blockIdx.x + max(w.part, 0)) * N * p.out_cols;
@@ -531,41 +586,91 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
   if (warp == 1) tmem_dealloc(tS, cols);
 }
 
-// Items of a persistent launch that several CTAs shared.  Grid (items, groups of four query rows).
+// Items of a persistent launch that several CTAs shared.  Grid (items, query rows), a block of 128 threads per row.
 template <int N>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(128)
 latent_merge_kernel(const LatentParams p) {
   tgi::pdl_wait();
   tgi::pdl_trigger();
-  const int items = (p.H + N - 1) / N, b = blockIdx.x / items, rt = blockIdx.x % items;
-  const int begin = p.cu[b], rows = min(N, p.H - rt * N);
-  if (p.cu[b + 1] <= begin) return;
+  constexpr int kBatch = 128;                              // parts whose weights are held at a time
+  __shared__ float s_f[kBatch];
+  __shared__ float red[8];
+  const int items = (p.H + N - 1) / N, b = blockIdx.x / items, row = blockIdx.x % items * N + blockIdx.y, r = blockIdx.y;
+  const int begin = p.cu[b];
+  if (row >= p.H || p.cu[b + 1] <= begin) return;
   const int c0 = p.range[2 * blockIdx.x], c1 = p.range[2 * blockIdx.x + 1];
   if (c0 == c1) return;                                    // one CTA did the whole item
-  for (int i = threadIdx.x; i < 4 * p.out_cols; i += blockDim.x) {
-    const int r = blockIdx.y * 4 + i / p.out_cols, col = i % p.out_cols;
-    if (r >= rows) break;
-    // the first of the CTAs ended with its part (slot 1), the others began with theirs (slot 0)
-    auto slot = [&](int c) { return static_cast<size_t>(2 * c + (c == c0 ? 1 : 0)) * N + r; };
-    float mm = -INFINITY, sum = 0.f, o = 0.f;
-    for (int c = c0; c <= c1; ++c) mm = fmaxf(mm, p.part_ml[slot(c) * 2]);
-    for (int c = c0; c <= c1; ++c) {
-      const float m = p.part_ml[slot(c) * 2];
-      if (m == -INFINITY) continue;
-      const float f = exp2f(m - mm);
-      sum = fmaf(p.part_ml[slot(c) * 2 + 1], f, sum);
-      o = fmaf(p.part_o[slot(c) * p.out_cols + col], f, o);
+  // the first of the CTAs ended with its part (slot 1), the others began with theirs (slot 0)
+  auto slot = [&](int c) { return static_cast<size_t>(2 * c + (c == c0 ? 1 : 0)) * N + r; };
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  float mm = -INFINITY;
+  for (int c = c0 + threadIdx.x; c <= c1; c += blockDim.x) mm = fmaxf(mm, p.part_ml[slot(c) * 2]);
+#pragma unroll
+  for (int o = 16; o; o >>= 1) mm = fmaxf(mm, __shfl_xor_sync(0xffffffffu, mm, o));
+  if (lane == 0) red[warp] = mm;
+  __syncthreads();
+  mm = fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3]));
+  if (mm == -INFINITY) mm = 0.f;
+  float sum = 0.f;
+  constexpr int kCols = 4;                                 // columns per thread: out_cols <= 512
+  float o[kCols] = {};
+  for (int at = c0; at <= c1; at += kBatch) {
+    const int n = min(kBatch, c1 + 1 - at);
+    __syncthreads();
+    if (static_cast<int>(threadIdx.x) < n) {
+      const float* ml = p.part_ml + slot(at + threadIdx.x) * 2;
+      const float f = exp2f(ml[0] - mm);
+      s_f[threadIdx.x] = f;
+      sum = fmaf(ml[1], f, sum);
     }
-    float f = sum > 0.f ? 1.f / sum : 0.f;
-    if (p.gate != nullptr)
-      f *= __fdividef(1.f, 1.f + __expf(-__bfloat162float(p.gate[static_cast<long long>(begin) * p.ld_gate + rt * N + r])));
-    p.out[(static_cast<size_t>(begin) * p.H + rt * N + r) * p.out_cols + col] = __float2bfloat16(o * f);
+    __syncthreads();
+#pragma unroll 8
+    for (int i = 0; i < n; ++i) {
+      const float* src = p.part_o + slot(at + i) * p.out_cols;
+      const float f = s_f[i];
+#pragma unroll
+      for (int e = 0; e < kCols; ++e) {
+        const int col = threadIdx.x + e * 128;
+        if (col < p.out_cols) o[e] = fmaf(src[col], f, o[e]);
+      }
+    }
+  }
+#pragma unroll
+  for (int d = 16; d; d >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, d);
+  if (lane == 0) red[4 + warp] = sum;
+  __syncthreads();
+  sum = (red[4] + red[5]) + (red[6] + red[7]);
+  float f = sum > 0.f ? 1.f / sum : 0.f;
+  if (p.gate != nullptr)
+    f *= __fdividef(1.f, 1.f + __expf(-__bfloat162float(p.gate[static_cast<long long>(begin) * p.ld_gate + row])));
+#pragma unroll
+  for (int e = 0; e < kCols; ++e) {
+    const int col = threadIdx.x + e * 128;
+    if (col < p.out_cols) p.out[(static_cast<size_t>(begin) * p.H + row) * p.out_cols + col] = __float2bfloat16(o[e] * f);
   }
 }
 
-int smem_bytes(int N, int slabs, int value_slabs, int seqs) {
-  const int held = max(slabs, (value_slabs + 1) / 2 * 2);
-  return held * kSlab + slabs * N * 128 + kKeys * 128 + 9 * N * 4 + (kMaxSlabs + kMaxSlabs / 2 + 9) * 8 + 16 + (seqs + 1) * 4;
+int smem_bytes(int N, int slabs, int stages, int seqs) {
+  return stages * slabs * kKeys * 128 + slabs * N * 128 + 2 * kPTile + 10 * N * 4 + (2 * kMaxStages + 12) * 8 + 16 + (seqs + 1) * 4;
+}
+// stages of the K ring that fit (at least two are wanted)
+int stages_for(int N, int slabs) {
+  int n = kMaxStages;
+  while (n > 0 && smem_bytes(N, slabs, n, kMaxSeqs) > 227 * 1024) --n;
+  return n;
+}
+// map over pages [num_blocks, 16, slabs * 64] whose box is one page: 64 columns x 8 tokens x slabs x 2
+int make_page_map(CUtensorMap* map, const void* pages, int num_blocks, int slabs) {
+  tgi::EncodeTiledFn enc = tgi::get_encode();
+  if (enc == nullptr) return -100;
+  const cuuint64_t row = static_cast<cuuint64_t>(slabs) * 128;
+  cuuint64_t dims[4] = {64, 8, static_cast<cuuint64_t>(slabs), 2 * static_cast<cuuint64_t>(num_blocks)};
+  cuuint64_t strides[3] = {row, 128, 8 * row};
+  cuuint32_t box[4] = {64, 8, static_cast<cuuint32_t>(slabs), 2}, step[4] = {1, 1, 1, 1};
+  const CUresult r = enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, const_cast<void*>(pages), dims, strides, box, step,
+                         CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                         CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? 0 : -static_cast<int>(r) - 1000;
 }
 
 template <int N, int OG>
@@ -574,8 +679,7 @@ int launch(const LatentParams& p, const void* q, const void* pages, long long q_
   const uint64_t width = static_cast<uint64_t>(p.slabs) * 64;
   int rc = tgi::make_map_2d(&tmQ, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, q, q_rows, width, width * 2, N, 64, CU_TENSOR_MAP_SWIZZLE_128B);
   if (rc) return rc;
-  rc = tgi::make_map_2d(&tmK, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, pages, static_cast<uint64_t>(p.num_blocks) * kPage, width, width * 2,
-                        kPage, 64, CU_TENSOR_MAP_SWIZZLE_128B);
+  rc = make_page_map(&tmK, pages, p.num_blocks, p.slabs);
   if (rc) return rc;
   auto kern = latent_attention_kernel<N, OG>;
   static std::atomic<unsigned long long> attr_set{0};
@@ -588,9 +692,9 @@ int launch(const LatentParams& p, const void* q, const void* pages, long long q_
   }
   const int items = (max_q * p.H + N - 1) / N;
   const dim3 grid = p.persistent ? dim3(ctas) : dim3(items, p.B);
-  const size_t smem = smem_bytes(N, p.slabs, p.value_slabs, p.persistent ? p.B : 0);
+  const size_t smem = smem_bytes(N, p.slabs, p.stages, p.persistent ? p.B : 0);
   tgi::launch(kern, grid, dim3(256 + 128 * OG), smem, stream, tmQ, tmK, p);
-  if (p.persistent) tgi::launch(latent_merge_kernel<N>, dim3(p.B * items, (min(N, p.H) + 3) / 4), dim3(256), 0, stream, p);
+  if (p.persistent) tgi::launch(latent_merge_kernel<N>, dim3(p.B * items, min(N, p.H)), dim3(128), 0, stream, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
 
@@ -602,7 +706,7 @@ extern "C" {
 int tgi_latent_rows(int slabs, int value_slabs, long long rows) {
   if (value_slabs < 1 || value_slabs > 8 || slabs < value_slabs || slabs > kMaxSlabs) return 0;
   int N = rows <= 16 ? 16 : rows <= 32 || value_slabs > 4 ? 32 : 64;
-  while (N >= 16 && smem_bytes(N, slabs, value_slabs, kMaxSeqs) > 227 * 1024) N /= 2;
+  while (N >= 16 && stages_for(N, slabs) < 2) N /= 2;
   return N >= 16 ? N : 0;
 }
 
@@ -615,7 +719,9 @@ int tgi_latent_attention(const void* q, const void* pages, const int* block_tabl
                          int most, int ctas, int* status, cudaStream_t stream) {
   if (T <= 0 || B <= 0 || max_q <= 0) return 0;
   if (N != 16 && N != 32 && N != 64) return -10;
-  if (B > 65535 || num_blocks < 1 || max_blocks < 1 || ctas < 1 || smem_bytes(N, slabs, value_slabs, kMaxSeqs) > 227 * 1024) return -10;
+  if (B > 65535 || num_blocks < 1 || max_blocks < 1 || ctas < 1 || slabs > kMaxSlabs || value_slabs > 8 ||
+      stages_for(N, slabs) < 2)
+    return -10;
   LatentParams p;
   p.block_tables = block_tables;
   p.cu = cu;
@@ -633,6 +739,7 @@ int tgi_latent_attention(const void* q, const void* pages, const int* block_tabl
   p.out_cols = value_slabs * 64;
   p.slabs = slabs;
   p.value_slabs = value_slabs;
+  p.stages = stages_for(N, slabs);
   p.window = window;
   p.persistent = max_q == 1 && B <= kMaxSeqs && part_o != nullptr && part_ml != nullptr && range != nullptr;
   p.most = most;

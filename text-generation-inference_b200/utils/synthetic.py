@@ -443,3 +443,92 @@ def kipedra_state_dict(cfg: dict, seed: int = 0, dtype=torch.float32, device: st
 
 
 
+
+
+def gisilix_attention(heads=4, kv_heads=2, dim=24, vdim=16, coef=0.25, every=20, softcap=9.0, scale=None, kv_from=None,
+                      mlp=None) -> dict:
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "q_temp": {"coef": coef, "every": every},
+         "softcap": softcap, "scale": dim ** -0.5 if scale is None else scale}
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return {"type": "attention", "mlp": mlp, "mixer": m}
+
+
+def gisilix_latent(heads=4, dim=24, vdim=20, rank=40, scale=None, mlp=None) -> dict:
+    return {"type": "latent_attention", "mlp": mlp,
+            "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "kv_rank": rank, "scale": dim ** -0.5 if scale is None else scale}}
+
+
+def gisilix_rotated_latent(heads=4, dim=24, vdim=20, rank=40, rot_dim=8, window=24, base=1000.0, scaling=(4.0, 8.0, 1.0, 128),
+                           scale=None, mlp=None) -> dict:
+    """``scaling``: (factor, fast, slow, original length)."""
+    rot = {"base": base, "dims": rot_dim}
+    if scaling is not None:
+        rot["scaling"] = dict(zip(("factor", "fast", "slow", "original"), scaling))
+    return {"type": "latent_attention_2", "mlp": mlp,
+            "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "kv_rank": rank, "rot_dim": rot_dim, "mask": {"size": window},
+                      "rot": rot, "scale": (dim + rot_dim) ** -0.5 if scale is None else scale}}
+
+
+def gisilix_moe(ff=24, experts=10, top=3, shared=40) -> dict:
+    mlp = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}}
+    if shared:
+        mlp["shared"] = {"ff": shared}
+    return mlp
+
+
+def gisilix_config(layers, width=80, vocab=203, eps=1e-5) -> dict:
+    return {"architecture": "Gisilix", "width": width, "vocab": vocab, "norm": {"eps": eps}, "layers": list(layers)}
+
+
+def gisilix_state_dict(cfg: dict, seed: int = 0, dtype=torch.float32, device: str = "cpu") -> Dict[str, torch.Tensor]:
+    """Random weights of a Gisilix shape."""
+    g = torch.Generator(device=device).manual_seed(seed)
+    W, sd = cfg["width"], {}
+
+    def rnd(*shape, std=None, mean=0.0):
+        std = shape[-1] ** -0.5 if std is None else std
+        return (mean + torch.randn(*shape, generator=g, device=device) * std).to(dtype)
+
+    def norm(name, n, bias=True):
+        sd[name] = rnd(n, std=0.2, mean=1.0)
+        if bias:
+            sd[name + ".b"] = rnd(n, std=0.1)
+
+    def feed_forward(p, ff):
+        sd.update({p + "gate": rnd(ff, W), p + "up": rnd(ff, W), p + "down": rnd(W, ff)})
+
+    sd["embed"] = rnd(cfg["vocab"], W, std=1.0)
+    norm("final.norm", W)
+    for i, layer in enumerate(cfg["layers"]):
+        p, m, mlp = f"l{i}.", layer["mixer"], layer.get("mlp")
+        H, d, dv = m["heads"], m["dim"], m["vdim"]
+        mix = p + "mix."
+        norm(p + "norm1", W)
+        sd[mix + "o"] = rnd(W, H * dv)
+        if layer["type"] == "attention":
+            G = m["kv_heads"]
+            sd.update({mix + "q": rnd(H * d, W), mix + "g": rnd(H * dv, W), mix + "sink": rnd(H, std=1.5)})
+            norm(mix + "q.norm", H * d, False)
+            if m.get("kv_from") is None:
+                sd.update({mix + "k": rnd(G * d, W), mix + "v": rnd(G * dv, W)})
+                norm(mix + "k.norm", G * d, False)
+        else:
+            r, rot = m["kv_rank"], m.get("rot_dim", 0)
+            sd.update({mix + "q": rnd(H * (d + rot), W), mix + "dkv": rnd(r + rot, W), mix + "uk": rnd(H * d, r), mix + "uv": rnd(H * dv, r)})
+            norm(mix + "dkv.norm", r, False)
+            if layer["type"] == "latent_attention_2":
+                sd[mix + "g"] = rnd(H, W)
+        if mlp is None:
+            continue
+        norm(p + "norm2", W)
+        if mlp["kind"] == "dense":
+            feed_forward(p + "mlp.", mlp["ff"])
+            continue
+        E = mlp["router"]["experts"]
+        sd.update({p + "mlp.router": rnd(E, W), p + "mlp.router.b": rnd(E, std=0.3)})
+        for e in range(E):
+            feed_forward(f"{p}mlp.e{e}.", mlp["expert"]["ff"])
+        if mlp.get("shared"):
+            feed_forward(p + "mlp.shared.", mlp["shared"]["ff"])
+    return sd
