@@ -54,6 +54,7 @@ class ForwardMeta:
     attn_horizon: Optional[torch.Tensor] = None      # [T] last KV position a row may see (image rows: end of their image)
     state_slots: Optional[torch.Tensor] = None       # [B] slot of every sequence in the recurrent state pools, -1: none
     v_first: Optional[torch.Tensor] = None           # [T, *] values later layers mix in (set by the first layer that mixes)
+    expansions: Optional[dict] = None                # window -> mixers.Expansion of layers with latent attention
     cross: Optional[object] = None                   # rows and image states for cross-attention layers (models/mllama.py)
 
 
@@ -698,6 +699,11 @@ class CausalDecoder:
     def recurrent(self) -> bool:
         """True when a sequence carries state that a step advances (and that a step must therefore run exactly once)."""
         return any(s.recurrent for s in self.dims.mixers or [])
+
+    @property
+    def expanded_windows(self) -> List[int]:
+        """Windows (0: none) of the layers that write out keys and values for sequences with many tokens."""
+        return sorted({l.attn.spec.window for l in self.layers if getattr(l.attn, "full", None) is not None})
 
     def embed_tokens(self, input_ids: torch.Tensor, positions: Optional[torch.Tensor] = None) -> torch.Tensor:
         h = self.embed(input_ids)

@@ -312,6 +312,7 @@ class FlashCausalLM(Model):
         self.overlap_hits = 0          # steps that found their replay already on the stream
         self.overlap_decode = os.environ.get("TGI_B200_OVERLAP_DECODE", "1") == "1" and not self.recurrent
         self.state_slots: Optional[Pool] = None      # made with the cache
+        self.expanded_windows = list(getattr(model, "expanded_windows", []))
         self.eos_token_ids = eos_token_ids
         if eos_token_ids is not None and tokenizer is not None:
             try:
@@ -452,6 +453,7 @@ class FlashCausalLM(Model):
         head_rows: List[int] = []       # rows of the hidden state that need logits
         row_owner: List[Tuple[int, int]] = []  # (seq index, offset inside the chunk) per logits row
         t = 0
+        starts = []
         for i, (s, n) in enumerate(zip(seqs, counts)):
             start = s.cache_len
             if s.prefilling:
@@ -460,6 +462,7 @@ class FlashCausalLM(Model):
                 toks = [s.ids[-1]] + s.speculative_ids
                 start = len(s.ids) - 1
             input_ids[t:t + n] = toks
+            starts.append(start)
             # `pos_delta`: offset between rotary position and token index after a prompt with images (Qwen2-VL)
             pos0 = start if s.prefilling else start + getattr(s, "pos_delta", 0)
             positions[t:t + n] = np.arange(pos0, pos0 + n, dtype=np.int32)
@@ -488,12 +491,24 @@ class FlashCausalLM(Model):
         arrays = [input_ids, positions, slots, cu, kv_lens, tables, head]
         if self.recurrent:
             arrays.append(state)
+        plans, at = {}, len(arrays)
+        if self.expanded_windows and max(counts, default=0) > 1:
+            from .mixers import Expansion, plan_expansion
+
+            for window in self.expanded_windows:
+                plan = plan_expansion(window, starts, counts, [s.slots for s in seqs])
+                if plan is not None:
+                    plans[window] = plan
+                    arrays.extend(plan[0])
         dev = self.staging.upload(arrays)
+        for window, (_, scalars) in plans.items():
+            plans[window] = Expansion(*dev[at:at + 4], *scalars)
+            at += 4
         meta = ForwardMeta(
             input_ids=dev[0], positions=dev[1], slots=dev[2], cu_seqlens_q=dev[3], kv_lens=dev[4],
             block_tables=dev[5], max_q=max(counts) if counts else 0, max_kv=int(kv_lens.max()) if B else 0,
             lm_head_indices=dev[6] if head_rows_of is not None or len(head_rows) != T else None,
-            state_slots=dev[7] if self.recurrent else None,
+            state_slots=dev[7] if self.recurrent else None, expansions=plans or None,
         )
         lora = getattr(self, "lora", None)
         if lora is not None and any(s.adapter_index > 0 for s in seqs):

@@ -8,7 +8,8 @@ cache (``cache_tensors``) and runs as a short sequence of fused ops:
                 -> o GEMM
     latent      GEMM for q, latent and gate -> RMS of the latent, rotations, page store -> queries times the key
                 up-projection -> attention over the latents (all heads read one row per token), gate -> value
-                up-projection -> o GEMM
+                up-projection -> o GEMM; for sequences that bring many tokens -> keys and values of the visible tokens
+                written out by one GEMM -> attention per head, gate -> o GEMM
     delta       one GEMM for q, k, v, write strengths and decay / gate inputs (-> low-rank decay / gate GEMMs)
                 -> short convolutions + unit norms + decays -> state scan -> norm x gate -> o GEMM
     decay       one GEMM for q, k, v, gate -> state scan (SiLU applied on the way in) -> norm x gate -> o GEMM
@@ -20,8 +21,11 @@ tokens are one code path.
 """
 from __future__ import annotations
 
+import os
+from dataclasses import dataclass
 from typing import Dict, List, Optional, Sequence, Tuple
 
+import numpy as np
 import torch
 
 from .. import ops
@@ -203,10 +207,63 @@ class MixedAttention(Mixer):
                                      s.rot_interleaved, conv)
 
 
+# tokens of a sequence in one step from which its latents are expanded to keys and values per head, and the most rows
+# that a step expands (their keys and values are held for one layer at a time)
+EXPAND_TOKENS = int(os.environ.get("TGI_B200_LATENT_EXPAND", "64"))
+EXPAND_ROWS = int(os.environ.get("TGI_B200_LATENT_EXPAND_ROWS", "131072"))
+EXPAND_GROUP = 16           # rows of a group that a table entry names
+
+
+@dataclass
+class Expansion:
+    """Tokens whose keys and values a step writes out, for layers with one window: for every expanded sequence those its
+    queries see, from a multiple of ``EXPAND_GROUP`` positions on.  Positions count from there (scores do not depend on it)."""
+
+    rows: torch.Tensor          # [R] page row (slot) of every expanded token; gaps at the sequences' ends repeat one
+    tables: torch.Tensor        # [B, *] groups of rows of a sequence
+    kv_lens: torch.Tensor       # [B] expanded tokens, 0: the sequence is not expanded
+    queries: torch.Tensor       # rows of the step that belong to expanded sequences
+    all: bool                   # every sequence that brings tokens is expanded
+    rest_max_q: int             # most tokens of the others
+
+
+def plan_expansion(window: int, starts: Sequence[int], counts: Sequence[int], slots: Sequence[np.ndarray]):
+    """Host arrays of an ``Expansion`` (``rows, tables, kv_lens, queries``) with its two scalars, or ``None``.  ``starts``:
+    position of a sequence's first token of the step, ``slots``: page rows of its positions."""
+    g, total, at, rest = EXPAND_GROUP, 0, 0, 0
+    rows, groups, queries = [], [], []
+    kv = np.zeros(len(counts), dtype=np.int32)
+    for b, (s, n) in enumerate(zip(starts, counts)):
+        first = max(0, s - window + 1) // g * g if window > 0 else 0
+        length = s + n - first
+        padded = -(-length // g) * g
+        if n >= EXPAND_TOKENS and total + padded <= EXPAND_ROWS:
+            own = np.zeros(padded, dtype=np.int32)
+            own[:length] = slots[b][first:s + n]
+            own[length:] = own[0]
+            rows.append(own)
+            groups.append(np.arange(total // g, (total + padded) // g, dtype=np.int32))
+            queries.append(np.arange(at, at + n, dtype=np.int32))
+            kv[b] = length
+            total += padded
+        else:
+            groups.append(np.zeros(0, dtype=np.int32))
+            rest = max(rest, n)
+        at += n
+    if not rows:
+        return None
+    tables = np.zeros((len(counts), max(len(x) for x in groups)), dtype=np.int32)
+    for b, x in enumerate(groups):
+        tables[b, :len(x)] = x
+    return (np.concatenate(rows), tables, kv, np.concatenate(queries)), (rest == 0, rest)
+
+
 class LatentAttention(Mixer):
     """Attention whose keys and values are up-projections of one latent per token, beside which a rotated key part that all
     heads share may stand.  Only latent and rotated part are cached.  The up-projections are moved to the other side of the
-    attention: ``q . (W_uk c) = (W_uk^T q) . c`` and ``sum p W_uv c = W_uv sum p c``, so every head attends to the same rows."""
+    attention: ``q . (W_uk c) = (W_uk^T q) . c`` and ``sum p W_uv c = W_uv sum p c``, so every head attends to the same rows.
+    That costs more operations per query and key, so sequences that bring many tokens attend to keys and values written out
+    (``Expansion``), one matrix product of the cached rows (the rotated part passes through a block of ones)."""
 
     def __init__(self, spec, prefix, weights, idx, eps, comm=None, rotary: Optional[RotaryTables] = None):
         super().__init__(spec, prefix, weights, idx, eps, comm)
@@ -219,6 +276,14 @@ class LatentAttention(Mixer):
         pad = (0, self.off_rot - s.kv_rank)
         self.uk, self.uv = (torch.nn.functional.pad(self.tensor(n).view(s.heads, d, s.kv_rank), pad).contiguous()
                             for n, d in (("uk", s.dim), ("uv", s.vdim)))         # [H, d, columns of the latent]
+        self.full = ops.expanded_dims(s.dim + s.rot_dims, s.vdim, self.dtype, self.device)
+        if self.full is not None:
+            dk, dv = self.full
+            k, v = self.uk.new_zeros(s.heads, dk, self.width), self.uv.new_zeros(s.heads, dv, self.width)
+            k[:, :s.dim, :self.off_rot], v[:, :s.vdim, :self.off_rot] = self.uk, self.uv
+            turn = torch.arange(s.rot_dims, device=self.device)
+            k[:, s.dim + turn, self.off_rot + turn] = 1
+            self.expand = torch.cat([k.view(-1, self.width), v.view(-1, self.width)])
         self.o = self.row(_column_input(self.tensor("o")))
         self.rotary = rotary.get(s)
 
@@ -230,16 +295,27 @@ class LatentAttention(Mixer):
         s, T = self.spec, x.shape[0]
         pages, = kv
         proj = self.proj(x)
-        q = proj.new_empty(T, s.heads, self.width)
+        plan = meta.expansions.get(s.window) if meta.expansions and self.full is not None else None
+        rest = plan is None or not plan.all
+        q = proj.new_empty(T, s.heads, self.width) if rest else None
+        q_full = None if plan is None else proj.new_empty(T, s.heads, self.full[0])
         ops.latent_store(proj, self.offs[1], self.norm, self.eps, meta.positions, self.rotary.cos_sin, meta.slots, pages, q,
-                         self.off_rot, s.kv_rank, s.rot_dims, s.heads, s.dim)
-        plain = proj[:, :s.heads * (s.dim + s.rot_dims)].view(T, s.heads, -1)[..., :s.dim]
-        torch.bmm(plain.transpose(0, 1), self.uk, out=q[..., :self.off_rot].transpose(0, 1))
+                         self.off_rot, s.kv_rank, s.rot_dims, s.heads, s.dim, q_full)
         gate = proj[:, self.offs[2]:self.offs[2] + s.heads] if s.out_gate else None
-        a = ops.latent_attention(q, pages, s.kv_rank, meta.block_tables, meta.cu_seqlens_q, meta.kv_lens, s.scale, s.window or -1,
-                                 meta.max_q, meta.max_kv, gate)
         y = proj.new_empty(T, s.heads, s.vdim)
-        torch.bmm(a.transpose(0, 1), self.uv[..., :a.shape[2]].transpose(1, 2), out=y.transpose(0, 1))
+        if rest:
+            plain = proj[:, :s.heads * (s.dim + s.rot_dims)].view(T, s.heads, -1)[..., :s.dim]
+            torch.bmm(plain.transpose(0, 1), self.uk, out=q[..., :self.off_rot].transpose(0, 1))
+            a = ops.latent_attention(q, pages, s.kv_rank, meta.block_tables, meta.cu_seqlens_q, meta.kv_lens, s.scale,
+                                     s.window or -1, meta.max_q if plan is None else plan.rest_max_q, meta.max_kv, gate,
+                                     None if plan is None else plan.kv_lens)
+            torch.bmm(a.transpose(0, 1), self.uv[..., :a.shape[2]].transpose(1, 2), out=y.transpose(0, 1))
+        if plan is not None:
+            written = ops.linear_shallow(pages.view(-1, self.width).index_select(0, plan.rows), self.expand)
+            o = y if s.vdim == self.full[1] else proj.new_empty(T, s.heads, self.full[1])
+            ops.expanded_attention(q_full, written, plan, meta.cu_seqlens_q, s.scale, s.window or -1, meta.max_q, gate, o)
+            if o is not y:
+                y.index_copy_(0, plan.queries.long(), o.index_select(0, plan.queries)[..., :s.vdim])
         return self.o(y.view(T, -1), reduce=reduce, out=out)
 
 

@@ -174,20 +174,37 @@ def latent_layout(rank, rot, dtype, device):
     return rank, rank + rot
 
 
-def latent_store(proj, off_c, weight, eps, positions, cos_sin, slots, pages, q, off_rot, rank, rot, heads, dim):
+def latent_store(proj, off_c, weight, eps, positions, cos_sin, slots, pages, q, off_rot, rank, rot, heads, dim, q_full=None):
     """Latent attention's inputs from ``proj[T, *]`` (queries, ``dim`` plain and ``rot`` rotated dimensions per head, from
     column 0; ``rank`` latent columns and the shared key's ``rot`` columns from ``off_c``): the latent over its root mean
     square times ``weight``, and the shared key rotated (pairs ``2i, 2i + 1``), go to ``pages`` at the tokens' slots; the
-    rotated dimensions of the queries go to ``q[T, H, *]`` from column ``off_rot``, zeros behind them."""
-    _mixer_backend(proj).latent_store(proj, off_c, weight, eps, positions, cos_sin, slots, pages, q, off_rot, rank, rot, heads, dim)
+    rotated dimensions of the queries go to ``q[T, H, *]`` from column ``off_rot``, zeros behind them, and whole queries (plain,
+    rotated, zeros) to ``q_full[T, H, *]``; either may be ``None``."""
+    _mixer_backend(proj).latent_store(proj, off_c, weight, eps, positions, cos_sin, slots, pages, q, off_rot, rank, rot, heads, dim,
+                                      q_full)
 
 
-def latent_attention(q, pages, rank, block_tables, cu_seqlens_q, kv_lens, scale, window=-1, max_q=None, max_kv=None, gate=None):
+def latent_attention(q, pages, rank, block_tables, cu_seqlens_q, kv_lens, scale, window=-1, max_q=None, max_kv=None, gate=None,
+                     elsewhere=None):
     """Causal attention of ``q[T, H, width]`` over the one key row per token in ``pages[blocks, block_size, 1, width]``, whose
     first ``rank`` columns are the value too; head outputs times ``sigmoid(gate[T, H])``.  ``[T, H, rank or more]``, zeros
-    past ``rank``."""
+    past ``rank``.  Sequences whose entry in ``elsewhere[B]`` is at least their number of tokens are left out (their rows are
+    not written)."""
     return _mixer_backend(q).latent_attention(q, pages, rank, block_tables, cu_seqlens_q, kv_lens, scale, window, max_q, max_kv,
-                                              gate)
+                                              gate, elsewhere)
+
+
+def expanded_dims(dim, vdim, dtype, device):
+    """Head widths of ``expanded_attention`` for ``dim`` query / key and ``vdim`` value dimensions, ``None``: not available."""
+    if torch.device(device).type == "cuda" and not _FORCE_TORCH:
+        return native().expanded_dims(dim, vdim, dtype)
+    return None
+
+
+def expanded_attention(q, kv, plan, cu_seqlens_q, scale, window, max_q, gate, out):
+    """Causal attention of ``q[T, H, dk]`` over keys and values written out for the step, ``kv[rows, H * dk + H * 128]``, laid out
+    as ``plan`` (``models.mixers.Expansion``) says; rows of the plan's sequences are written to ``out[T, H, 128]``."""
+    native().expanded_attention(q, kv, plan, cu_seqlens_q, scale, window, max_q, gate, out)
 
 
 def recurrent_pitch(dim, device):
@@ -253,7 +270,7 @@ def linear(x, weight, bias=None, out=None):
 def linear_shallow(x, weight):
     """Product over a short inner dimension (low-rank projections).  The persistent GEMM is built for deep K and its
     epilogue dominates here: 8192 x 4096 x 128 takes 77 us, the library's 19 us; few rows stay on the persistent one."""
-    if use_native(x) and x.dtype == torch.bfloat16 and x.shape[0] >= 512 and weight.shape[1] <= 512:
+    if use_native(x) and x.dtype == torch.bfloat16 and x.shape[0] >= 512 and weight.shape[1] <= 768:
         return torch.nn.functional.linear(x, weight)
     return linear(x, weight)
 

@@ -1,6 +1,6 @@
-// Paged causal prefill attention on the 5th-generation tensor cores (sm_100a): head size 128, pages of 16
-// tokens, bf16 or e4m3 KV pages, ragged batches with a cached prefix (chunked prefill), GQA, sliding
-// window, soft-capping and per-row horizons.
+// Paged causal prefill attention on the 5th-generation tensor cores (sm_100a): head size 128 (or, with bf16 pages, 192
+// for queries and keys), pages of 16 tokens, bf16 or e4m3 KV pages, ragged batches with a cached prefix (chunked
+// prefill), GQA, sliding window, soft-capping, per-row horizons and a gate per token and head.
 //
 // Replaces, in the reference, flashinfer `BatchPrefillWithPagedKVCache` / FA2 `varlen_fwd`
 // (layers/attention/cuda.py:244-296, layers/attention/flashinfer.py:58-128).
@@ -19,6 +19,8 @@
 // per-lane address arithmetic.  e4m3 pages are widened to fp16 (exact) on their way into the operand tiles by the
 // eight output warps, which are idle most of a tile (64 bytes per thread), and the MMAs then run in fp16 (Q is
 // converted once); bf16 pages feed bf16 MMAs directly.
+// Queries and keys of 192 take a third 64-element slab each; V and P are then single-buffered (V of the next tile is wanted
+// only after that tile's softmax, P is free again after the PV product, during the softmax's first pass).
 // The S accumulator and the PV accumulator are double-buffered in TMEM (4 x 128 columns), so the tensor core
 // computes S of the next tile while the softmax warps work on the current one.
 // Every wait is bounded; a wait that runs out sets the status word, the CTA drains and frees its TMEM.
@@ -38,7 +40,7 @@ using namespace sm100;
 
 namespace {
 
-constexpr int kD = 128;            // head size
+constexpr int kD = 128;            // value size of a head
 constexpr int kRows = 128;         // query rows per CTA
 constexpr int kKeys = 128;         // KV tokens per tile
 constexpr int kPage = 16;          // tokens per page
@@ -48,7 +50,7 @@ constexpr int kSlab = kRows * 128;             // bytes of one [128 rows x 128 b
 constexpr int kTileBytes = 2 * kSlab;          // a 128 x 128 tile of 16-bit values: two slabs (32 KB)
 
 struct PrefillParams {
-  const __nv_bfloat16* q;       // [T, Hq, 128]
+  const __nv_bfloat16* q;       // [T, Hq, 128 or 192]
   const int* block_tables;      // [B, max_blocks]
   const int* cu_seqlens_q;      // [B + 1]
   const int* kv_lens;           // [B]
@@ -56,6 +58,8 @@ struct PrefillParams {
   const float* v_scale;
   __nv_bfloat16* out;           // [T, Hq, 128]
   const int* horizon;           // optional [T]
+  const __nv_bfloat16* gate;    // optional [T, ld_gate]: the output of head h is multiplied by the sigmoid of column h
+  long long ld_gate;
   int max_blocks, Hq, Hkv, num_blocks;
   float scale, softcap;
   int window;
@@ -121,18 +125,17 @@ __device__ __forceinline__ float fast_tanh(float y) {      // 1 - 2 / (1 + e^(2y
 }
 // How a softmax thread reads its scores.  Key i of a 32-key group is visible when i - lo lies in [0, range]
 // (one unsigned compare); with soft-capping a raw score x becomes cap_out * tanh(x * cap_in), already in log2 units,
-// otherwise it is scaled by scale_log2 (> 0) — after the maximum in the first pass, inside the FMA in the second.
+// otherwise it is scaled by scale_log2 (> 0) — both after the maximum in the first pass, inside the FMA in the second.
 struct ScoreArgs {
   float scale_log2, cap_in, cap_out;
   int lo;
   unsigned range;
 };
-template <bool MASK, bool CAP>
+template <bool MASK>
 __device__ __forceinline__ float group_max(const uint32_t (&v)[32], float mx, const ScoreArgs& a) {
 #pragma unroll
   for (int i = 0; i < 32; ++i) {
     float x = __uint_as_float(v[i]);
-    if (CAP) x = a.cap_out * fast_tanh(x * a.cap_in);
     if (MASK) x = static_cast<unsigned>(i - a.lo) <= a.range ? x : -INFINITY;
     mx = fmaxf(mx, x);
   }
@@ -167,32 +170,39 @@ __device__ __forceinline__ float group_prob(const uint32_t (&v)[32], uint32_t (&
   return rs0 + rs1;
 }
 
-// Shared memory (bytes):  Q 32 K | K: bf16 2 x 32 K, e4m3 raw 2 x 16 K + converted 32 K | V: same | P 32 K | barriers
-template <bool FP8>
+// Shared memory (bytes):  Q 32 K | K: bf16 2 x 32 K, e4m3 raw 2 x 16 K + converted 32 K | V: same | P 2 x 32 K | barriers;
+// with KS = 3 slabs of queries and keys:  Q 48 K | K 2 x 48 K | V 32 K | P 32 K | barriers
+template <bool FP8, int KS>
 struct Layout {
+  static constexpr int kStagesVP = KS == 2 ? 2 : 1;               // of V and of P
   static constexpr int kQ = 0;
-  static constexpr int kK = kTileBytes;
-  static constexpr int kKBytes = 2 * kTileBytes;                  // 64 KB in both modes
-  static constexpr int kV = kK + kKBytes;
-  static constexpr int kP = kV + kKBytes;
+  static constexpr int kK = KS * kSlab;
+  static constexpr int kKTile = KS * kSlab;
+  static constexpr int kV = kK + 2 * kKTile;                      // e4m3: 64 KB as well
+  static constexpr int kP = kV + kStagesVP * kTileBytes;
   // two P tiles: the softmax of tile j + 1 writes one while the PV product of tile j still reads the other.  The
   // final partial row sums (float [2][128]) are written into the P tile that the last product does not read.
-  static constexpr int kBars = kP + 2 * kTileBytes;               // 224 KB
+  static constexpr int kBars = kP + kStagesVP * kTileBytes;
   static constexpr int kAlpha = kBars + 256;                      // float [2][128]
   static constexpr int kRowMax = kAlpha + 2 * 128 * 4;            // float [2][128]: row maxima of the two halves
   static constexpr int kAbort = kRowMax + 2 * 128 * 4;            // int [4][2]: a softmax thread of the lane quarter gave up
+  static constexpr int kSums = kAbort + 64;                       // single-buffered P: the row sums' own place
   // no slack for aligning the base: the kernel checks that the dynamic shared memory starts on a 1024-byte
   // boundary (it does when the kernel has no static shared memory) and reports an error otherwise
-  static constexpr int kTotal = kAbort + 64;
+  static constexpr int kTotal = kSums + (kStagesVP == 1 ? 2 * 128 * 4 : 0);
   static_assert(kTotal <= 227 * 1024, "shared memory of a CTA");
   // e4m3: raw stage s at kK + s * 16 K, converted tile at kK + 32 K
   static constexpr int kRawStage = kKeys * 128;
+  // stage and round of tile j
+  static __device__ __forceinline__ int stage(int j) { return kStagesVP == 2 ? j & 1 : 0; }
+  static __device__ __forceinline__ int round(int j) { return kStagesVP == 2 ? j >> 1 : j; }
 };
 
-template <bool FP8>
+template <bool FP8, int KS>
 __global__ void __launch_bounds__(kThreads, 1)
 prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, const PrefillParams p) {
-  using L = Layout<FP8>;
+  using L = Layout<FP8, KS>;
+  static_assert(KS == 2 || (KS == 3 && !FP8), "queries and keys of two slabs, or three of bf16");
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* smem = smem_raw;
   if ((smem_u32(smem) & 1023u) != 0u) {       // uniform over the CTA, before anything is allocated
@@ -225,8 +235,8 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
   const int b = blockIdx.z, h = blockIdx.y;
   const int qt = gridDim.x - 1 - blockIdx.x;       // long tiles (late rows) first: the grid drains on short ones
   const int q_begin = p.cu_seqlens_q[b], n = p.cu_seqlens_q[b + 1] - q_begin;
-  if (qt * kRows >= n) return;                       // uniform over the CTA, before anything is allocated
   const int Lkv = p.kv_lens[b];
+  if (qt * kRows >= n || Lkv < n) return;            // uniform over the CTA, before anything is allocated; Lkv < n: left out
   const int kvh = h / (p.Hq / p.Hkv);
   const int row_base = qt * kRows;
   const int pos_first = Lkv - n + row_base;
@@ -281,7 +291,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
   auto produce = [&](bool do_k, bool do_v) {
     bool ok = true;
     for (int j = 0; j < ntiles && ok; ++j) {
-      const int s = j & 1;
+      const int s = j & 1, vs = L::stage(j);
       const int t0 = t_lo + j * kKeys;
       int blk = 0;
       if (lane < kKeys / kPage) {
@@ -293,11 +303,11 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
       if (lane == 0) {
         if (do_k) {
           if (j >= 2) ok = mbar_wait(&k_free[s], ((j >> 1) - 1) & 1);
-          if (ok) mbar_arrive_expect_tx(&k_full[s], FP8 ? L::kRawStage : kTileBytes);
+          if (ok) mbar_arrive_expect_tx(&k_full[s], FP8 ? L::kRawStage : L::kKTile);
         }
         if (do_v && ok) {
-          if (j >= 2) ok = mbar_wait(&v_free[s], ((j >> 1) - 1) & 1);
-          if (ok) mbar_arrive_expect_tx(&v_full[s], FP8 ? L::kRawStage : kTileBytes);
+          if (j >= L::kStagesVP) ok = mbar_wait(&v_free[vs], (L::round(j) - 1) & 1);
+          if (ok) mbar_arrive_expect_tx(&v_full[vs], FP8 ? L::kRawStage : kTileBytes);
         }
         if (!ok) report(p.status, kErrProducerWait);
       }
@@ -310,25 +320,25 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
           if (do_k) tma_load_2d(smem + L::kK + s * L::kRawStage + pg * (kPage * 128), &tmK, &k_full[s], kvh * kD, blk * kPage);
           if (do_v) tma_load_2d(smem + L::kV + s * L::kRawStage + pg * (kPage * 128), &tmV, &v_full[s], kvh * kD, blk * kPage);
         }
-      } else if (lane < 16) {
-        const int hf = lane >> 3;
-        if (do_k)
-          tma_load_2d(smem + L::kK + s * kTileBytes + hf * kSlab + pg * (kPage * 128), &tmK, &k_full[s], kvh * kD + hf * 64, blk * kPage);
-        if (do_v)
-          tma_load_2d(smem + L::kV + s * kTileBytes + hf * kSlab + pg * (kPage * 128), &tmV, &v_full[s], kvh * kD + hf * 64, blk * kPage);
+      } else {
+        const int hf = lane >> 3;                              // 64-element slab
+        if (do_k && hf < KS)
+          tma_load_2d(smem + L::kK + s * L::kKTile + hf * kSlab + pg * (kPage * 128), &tmK, &k_full[s], kvh * (64 * KS) + hf * 64, blk * kPage);
+        if (do_v && hf < 2)
+          tma_load_2d(smem + L::kV + vs * kTileBytes + hf * kSlab + pg * (kPage * 128), &tmV, &v_full[vs], kvh * kD + hf * 64, blk * kPage);
       }
       __syncwarp();
     }
   };
   if (warp != 0 && warp != 2) {
-    // ---- Q tile -> shared, swizzled operand layout (two slabs of 64 head elements); fp16 for e4m3 pages.  The
+    // ---- Q tile -> shared, swizzled operand layout (slabs of 64 head elements); fp16 for e4m3 pages.  The
     // two producer warps are already fetching K and V meanwhile; the MMA issuer waits for q_ready. ----
     const int st = (warp == 1 ? 0 : warp - 2) * 32 + lane;       // 0..575
-    for (int c = st; c < kRows * 16; c += 18 * 32) {
-      const int row = c >> 4, ch = c & 15;
+    for (int c = st; c < kRows * 8 * KS; c += 18 * 32) {
+      const int row = c / (8 * KS), ch = c % (8 * KS);
       uint4 v = make_uint4(0, 0, 0, 0);
       if (row_base + row < n)
-        v = *reinterpret_cast<const uint4*>(p.q + (static_cast<size_t>(q_begin + row_base + row) * p.Hq + h) * kD + ch * 8);
+        v = *reinterpret_cast<const uint4*>(p.q + (static_cast<size_t>(q_begin + row_base + row) * p.Hq + h) * (64 * KS) + ch * 8);
       if (FP8) {
         const __nv_bfloat162* bv = reinterpret_cast<const __nv_bfloat162*>(&v);
         uint32_t o[4];
@@ -365,11 +375,11 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
           k_addr = smem_u32(smem + L::kK + 2 * L::kRawStage);
         } else {
           if (!mbar_wait(&k_full[s], (j >> 1) & 1)) { report(p.status, kErrMmaWaitFull); return false; }
-          k_addr = smem_u32(smem + L::kK + s * kTileBytes);
+          k_addr = smem_u32(smem + L::kK + s * L::kKTile);
         }
         tc_fence_after();
 #pragma unroll
-        for (int k = 0; k < 8; ++k) {      // 16 head elements (32 bytes) per MMA; 4 per slab
+        for (int k = 0; k < 4 * KS; ++k) { // 16 head elements (32 bytes) per MMA; 4 per slab
           const uint64_t da = make_desc_sw128(q_addr + (k >> 2) * kSlab) + ((k & 3) * 32 >> 4);
           const uint64_t db = make_desc_sw128(k_addr + (k >> 2) * kSlab) + ((k & 3) * 32 >> 4);
           mma_f16(tS + s * 128, da, db, id_qk, k > 0 ? 1u : 0u);
@@ -379,18 +389,18 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
         return true;
       };
       auto issue_pv = [&](int j) {
-        const int s = j & 1;
+        const int s = j & 1, vs = L::stage(j);
         if (j >= 2 && !mbar_wait(&pv_free[s], ((j >> 1) - 1) & 1)) { report(p.status, kErrMmaWaitAccum); return false; }
         uint32_t v_addr;
         if (FP8) {
           if (!mbar_wait(vc_ready, j & 1)) { report(p.status, kErrMmaWaitFull); return false; }
           v_addr = smem_u32(smem + L::kV + 2 * L::kRawStage);
         } else {
-          if (!mbar_wait(&v_full[s], (j >> 1) & 1)) { report(p.status, kErrMmaWaitFull); return false; }
-          v_addr = smem_u32(smem + L::kV + s * kTileBytes);
+          if (!mbar_wait(&v_full[vs], L::round(j) & 1)) { report(p.status, kErrMmaWaitFull); return false; }
+          v_addr = smem_u32(smem + L::kV + vs * kTileBytes);
         }
-        if (!mbar_wait(&p_ready[s], (j >> 1) & 1)) { report(p.status, kErrMmaWaitFull); return false; }
-        const uint32_t p_addr = p_base + s * kTileBytes;
+        if (!mbar_wait(&p_ready[vs], L::round(j) & 1)) { report(p.status, kErrMmaWaitFull); return false; }
+        const uint32_t p_addr = p_base + vs * kTileBytes;
         tc_fence_after();
 #pragma unroll
         for (int k = 0; k < 8; ++k) {      // 16 keys per MMA: 32 bytes along a P row, two 8-row groups of V
@@ -399,8 +409,8 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
           mma_f16(tPV + s * 128, da, db, id_pv, k > 0 ? 1u : 0u);
         }
         tc_commit(&pv_full[s]);
-        tc_commit(&p_free[s]);
-        tc_commit(FP8 ? vc_free : &v_free[s]);
+        tc_commit(&p_free[vs]);
+        tc_commit(FP8 ? vc_free : &v_free[vs]);
         return true;
       };
       ok = mbar_wait(q_ready, 0);
@@ -441,14 +451,14 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
     // barrier; everyone reads the flag right after the barrier, where all 64 threads see the same value.
     bool fail = false;
     for (int j = 0; j < ntiles; ++j) {
-      const int s = j & 1;
+      const int s = j & 1, ps = L::stage(j);
       const int t0 = t_lo + j * kKeys + hf * 64;    // first key of this thread's half
       if (!fail && !mbar_wait(&s_full[s], (j >> 1) & 1)) { report(p.status, kErrEpilogueWait); fail = true; }
       if (fail) s_abort[quarter * 2 + s] = 1;
       tc_fence_after();
       // a warp whose rows all see their whole half of the tile (below the diagonal / horizon, inside the window and
       // the sequence) takes the code without masks; the choice is per warp so that no path diverges
-      const bool plain = __all_sync(0xffffffffu, !cap && t0 >= t_min && t0 + 63 <= t_max);
+      const bool plain = __all_sync(0xffffffffu, t0 >= t_min && t0 + 63 <= t_max);
       sa.range = t_max >= t_min ? static_cast<unsigned>(t_max - t_min) : 0u;
       // pass 1: maximum of the (masked) scores of this half
       float mx = -INFINITY;
@@ -458,12 +468,13 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
         for (int c = 0; c < 64; c += 32) {
           tmem_ld32(lane_addr + s * 128 + c, v);
           sa.lo = t_max >= t_min ? t_min - (t0 + c) : (1 << 30);
-          if (plain) mx = group_max<false, false>(v, mx, sa);
-          else if (!cap) mx = group_max<true, false>(v, mx, sa);
-          else mx = group_max<true, true>(v, mx, sa);
+          // the cap is monotonic: the maximum of the raw scores is capped below
+          if (plain) mx = group_max<false>(v, mx, sa);
+          else mx = group_max<true>(v, mx, sa);
         }
       }
       if (!cap) mx *= scale_log2;     // scale_log2 > 0
+      else if (mx > -INFINITY) mx = sa.cap_out * fast_tanh(mx * sa.cap_in);
       // the two halves of a row agree on the maximum through shared memory (one named barrier per lane quarter)
       s_rowmax[hf * 128 + r] = mx;
       asm volatile("bar.sync %0, 64;" ::"r"(2 + quarter) : "memory");
@@ -471,7 +482,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
       const float m_new = fmaxf(m, fmaxf(mx, s_rowmax[(hf ^ 1) * 128 + r]));
       const float alpha = m_new == -INFINITY ? 0.f : fast_exp2(m - m_new);
       // the P tile and this parity's alpha slot are free once the PV product two tiles back was consumed
-      if (j >= 2 && !mbar_wait(&p_free[s], ((j >> 1) - 1) & 1)) { report(p.status, kErrEpilogueWait); fail = true; }
+      if (j >= L::kStagesVP && !mbar_wait(&p_free[ps], (L::round(j) - 1) & 1)) { report(p.status, kErrEpilogueWait); fail = true; }
       if (!fail && j >= 2 && !mbar_wait(&pv_free[s], ((j >> 1) - 1) & 1)) { report(p.status, kErrEpilogueWait); fail = true; }
       if (fail) continue;
       // pass 2: probabilities as 16-bit values into the P operand tile, partial row sum.  A row without a visible
@@ -482,13 +493,14 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
         if (c == 0) tmem_ld32(lane_addr + s * 128, v);
         uint32_t packed[16];
         sa.lo = t_max >= t_min ? t_min - (t0 + c) : (1 << 30);
-        if (plain) rs += group_prob<false, false, FP8>(v, packed, m_new, sa);
+        if (plain && !cap) rs += group_prob<false, false, FP8>(v, packed, m_new, sa);
         else if (!cap) rs += group_prob<true, false, FP8>(v, packed, m_new, sa);
+        else if (plain) rs += group_prob<false, true, FP8>(v, packed, m_new, sa);
         else rs += group_prob<true, true, FP8>(v, packed, m_new, sa);
 #pragma unroll
         for (int q4 = 0; q4 < 4; ++q4) {      // four 16-byte chunks (8 keys each) of this 32-key group
           const int ch = hf * 8 + (c >> 3) + q4;   // chunk index among the row's 16
-          *reinterpret_cast<uint4*>(smem + L::kP + s * kTileBytes + (ch >> 3) * kSlab + swz_chunk(r, ch & 7)) =
+          *reinterpret_cast<uint4*>(smem + L::kP + ps * kTileBytes + (ch >> 3) * kSlab + swz_chunk(r, ch & 7)) =
               make_uint4(packed[4 * q4], packed[4 * q4 + 1], packed[4 * q4 + 2], packed[4 * q4 + 3]);
         }
       }
@@ -500,18 +512,18 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
       __syncwarp();
       if (lane == 0) {
         mbar_arrive(&s_free[s]);
-        mbar_arrive(&p_ready[s]);
+        mbar_arrive(&p_ready[ps]);
       }
     }
     // partial row sums into the P tile the last product does not read; that tile was last read by the product of
     // the tile before the last one
-    if (!fail && ntiles >= 2 && !mbar_wait(&p_free[ntiles & 1], ((ntiles - 2) >> 1) & 1)) {
+    if (!fail && L::kStagesVP == 2 && ntiles >= 2 && !mbar_wait(&p_free[ntiles & 1], ((ntiles - 2) >> 1) & 1)) {
       report(p.status, kErrEpilogueWait);
       fail = true;
     }
     if (!fail) {
       if (p.sink != nullptr && hf == 0) l += exp2f(fmaf(p.sink[h], kLog2e, -m));      // both threads of a row hold the same maximum
-      reinterpret_cast<float*>(smem + L::kP + (ntiles & 1) * kTileBytes)[hf * 128 + r] = l;
+      reinterpret_cast<float*>(smem + (L::kStagesVP == 2 ? L::kP + (ntiles & 1) * kTileBytes : L::kSums))[hf * 128 + r] = l;
       __syncwarp();
       if (lane == 0) mbar_arrive(l_ready);
     }
@@ -585,9 +597,11 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
     }
     if (ok && mbar_wait(l_ready, 0)) {
       const float vs = (FP8 && p.v_scale != nullptr) ? p.v_scale[kvh] : 1.f;
-      const float* s_rowsum = reinterpret_cast<const float*>(smem + L::kP + (ntiles & 1) * kTileBytes);
+      const float* s_rowsum = reinterpret_cast<const float*>(smem + (L::kStagesVP == 2 ? L::kP + (ntiles & 1) * kTileBytes : L::kSums));
       const float l = s_rowsum[r] + s_rowsum[128 + r];
-      const float inv = l > 0.f ? vs / l : 0.f;
+      float inv = l > 0.f ? vs / l : 0.f;
+      if (p.gate != nullptr && row_base + r < n)
+        inv *= __fdividef(1.f, 1.f + __expf(-__bfloat162float(p.gate[static_cast<long long>(q_begin + row_base + r) * p.ld_gate + h])));
       if (row_base + r < n) {
         __nv_bfloat16* dst = p.out + (static_cast<size_t>(q_begin + row_base + r) * p.Hq + h) * kD + half * 64;
 #pragma unroll
@@ -607,26 +621,26 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
   if (warp == 1) tmem_dealloc(tmem_base, 512);
 }
 
-template <bool FP8>
-int launch_prefill(const PrefillParams& p, const void* k_cache, const void* v_cache, int B, int max_q, cudaStream_t stream) {
-  using L = Layout<FP8>;
+// `k_pitch`, `v_pitch`: elements from a token's keys (values) to the next token's
+template <bool FP8, int KS>
+int launch_prefill(const PrefillParams& p, const void* k_cache, const void* v_cache, long long k_pitch, long long v_pitch, int B,
+                   int max_q, cudaStream_t stream) {
+  using L = Layout<FP8, KS>;
   CUtensorMap tmK, tmV;
   const uint64_t rows = static_cast<uint64_t>(p.num_blocks) * kPage;
-  const uint64_t cols = static_cast<uint64_t>(p.Hkv) * kD;
+  const uint64_t k_cols = static_cast<uint64_t>(p.Hkv) * 64 * KS, v_cols = static_cast<uint64_t>(p.Hkv) * kD;
   int rc;
   if (FP8) {
-    rc = tgi::make_map_2d(&tmK, CU_TENSOR_MAP_DATA_TYPE_UINT8, k_cache, rows, cols, cols, kPage, 128, CU_TENSOR_MAP_SWIZZLE_NONE);
+    rc = tgi::make_map_2d(&tmK, CU_TENSOR_MAP_DATA_TYPE_UINT8, k_cache, rows, k_cols, k_pitch, kPage, 128, CU_TENSOR_MAP_SWIZZLE_NONE);
     if (rc) return rc;
-    rc = tgi::make_map_2d(&tmV, CU_TENSOR_MAP_DATA_TYPE_UINT8, v_cache, rows, cols, cols, kPage, 128, CU_TENSOR_MAP_SWIZZLE_NONE);
+    rc = tgi::make_map_2d(&tmV, CU_TENSOR_MAP_DATA_TYPE_UINT8, v_cache, rows, v_cols, v_pitch, kPage, 128, CU_TENSOR_MAP_SWIZZLE_NONE);
   } else {
-    rc = tgi::make_map_2d(&tmK, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, k_cache, rows, cols, cols * 2, kPage, 64,
-                          CU_TENSOR_MAP_SWIZZLE_128B);
+    rc = tgi::make_map_2d(&tmK, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, k_cache, rows, k_cols, k_pitch * 2, kPage, 64, CU_TENSOR_MAP_SWIZZLE_128B);
     if (rc) return rc;
-    rc = tgi::make_map_2d(&tmV, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, v_cache, rows, cols, cols * 2, kPage, 64,
-                          CU_TENSOR_MAP_SWIZZLE_128B);
+    rc = tgi::make_map_2d(&tmV, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, v_cache, rows, v_cols, v_pitch * 2, kPage, 64, CU_TENSOR_MAP_SWIZZLE_128B);
   }
   if (rc) return rc;
-  auto kern = prefill_tc_kernel<FP8>;
+  auto kern = prefill_tc_kernel<FP8, KS>;
   static std::atomic<unsigned long long> attr_set{0};
   int dev = 0;
   if (cudaGetDevice(&dev) != cudaSuccess) return -2;
@@ -653,7 +667,7 @@ int tgi_prefill_attention_tc(const void* q, const void* k_cache, const void* v_c
                              int* status, cudaStream_t stream) {
   if (B <= 0 || max_q <= 0) return 0;
   if (Hq % Hkv != 0 || B > 65535 || Hq > 65535) return -10;
-  PrefillParams p;
+  PrefillParams p{};
   p.q = static_cast<const __nv_bfloat16*>(q);
   p.block_tables = block_tables;
   p.cu_seqlens_q = cu_seqlens_q;
@@ -672,8 +686,37 @@ int tgi_prefill_attention_tc(const void* q, const void* k_cache, const void* v_c
   p.chunk = chunk;
   p.sink = sink;
   p.status = status;
-  return fp8_kv ? launch_prefill<true>(p, k_cache, v_cache, B, max_q, stream)
-                : launch_prefill<false>(p, k_cache, v_cache, B, max_q, stream);
+  const long long pitch = static_cast<long long>(Hkv) * kD;
+  return fp8_kv ? launch_prefill<true, 2>(p, k_cache, v_cache, pitch, pitch, B, max_q, stream)
+                : launch_prefill<false, 2>(p, k_cache, v_cache, pitch, pitch, B, max_q, stream);
+}
+
+// The same on keys and values of H heads that were written out for this step: q [T, H, dim] bf16 with dim 128 or 192, a
+// token's keys [H, dim] and values [H, 128] `pitch` elements from the next token's, tokens in groups of 16 that
+// `block_tables` names.  Sequences whose kv_lens entry is smaller than their number of tokens are left out.  gate
+// (optional): [T, ld_gate].
+int tgi_expanded_attention(const void* q, const void* k, const void* v, long long pitch, const int* block_tables,
+                           const int* cu_seqlens_q, const int* kv_lens, const void* gate, long long ld_gate, void* out, int B,
+                           int max_q, int max_blocks, int num_blocks, int H, int dim, float scale, int window, int* status,
+                           cudaStream_t stream) {
+  if (B <= 0 || max_q <= 0) return 0;
+  if (B > 65535 || H > 65535 || num_blocks < 1 || max_blocks < 1 || pitch % 8 != 0 || (dim != 128 && dim != 192)) return -10;
+  PrefillParams p{};
+  p.q = static_cast<const __nv_bfloat16*>(q);
+  p.block_tables = block_tables;
+  p.cu_seqlens_q = cu_seqlens_q;
+  p.kv_lens = kv_lens;
+  p.out = static_cast<__nv_bfloat16*>(out);
+  p.gate = static_cast<const __nv_bfloat16*>(gate);
+  p.ld_gate = ld_gate;
+  p.max_blocks = max_blocks;
+  p.Hq = p.Hkv = H;
+  p.num_blocks = num_blocks;
+  p.scale = scale;
+  p.window = window;
+  p.status = status;
+  return dim == 192 ? launch_prefill<false, 3>(p, k, v, pitch, pitch, B, max_q, stream)
+                    : launch_prefill<false, 2>(p, k, v, pitch, pitch, B, max_q, stream);
 }
 
 }  // extern "C"

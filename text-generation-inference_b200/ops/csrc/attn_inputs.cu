@@ -184,19 +184,21 @@ output_gate_kernel(const T* __restrict__ x, const T* __restrict__ gate, long lon
 
 // ------------------------------------------------------------------------------------------------
 // Inputs of latent attention.  proj[T, ld]: queries (H heads of dim plain and rot rotated dimensions) at column 0, latent
-// (rank) and the shared key's rotated part (rot) at off_c.  Grid (T, groups of heads); a warp normalises the latent and
-// rotates the shared part (first group), the others rotate the queries of a head each.  Pairs 2i, 2i + 1.
+// (rank) and the shared key's rotated part (rot) at off_c.  One CTA per token; a warp normalises the latent and rotates the
+// shared part, the others rotate the queries of a head each.  Pairs 2i, 2i + 1.  Rotated dimensions go to q_out from column
+// off_rot on (null: not wanted), whole queries (plain, rotated, zeros) to q_full, `full` columns per head (null: not wanted).
 // ------------------------------------------------------------------------------------------------
 struct Latent {
   long long ld, num_slots;
-  int off_c, rank, rot, H, dim, off_rot, width, max_pos;   // width: of a cached row and of a query head
+  int off_c, rank, rot, H, dim, off_rot, width, max_pos;   // width: of a cached row and of a head of q_out
+  int full;
   float eps;
 };
 template <typename T>
 __global__ void __launch_bounds__(256)
 latent_store_kernel(const T* __restrict__ proj, const float* __restrict__ weight, const int* __restrict__ positions,
                     const float* __restrict__ cos_sin, const int* __restrict__ slots, T* __restrict__ pages,
-                    T* __restrict__ q_out, Latent p) {
+                    T* __restrict__ q_out, T* __restrict__ q_full, Latent p) {
   tgi::pdl_wait();
   tgi::pdl_trigger();
   const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
@@ -222,9 +224,15 @@ latent_store_kernel(const T* __restrict__ proj, const float* __restrict__ weight
       const float inv = 1.f / sqrtf(warp_sum(ss) / p.rank + p.eps);
       for (int i = lane; i < p.rank; i += 32) put(dst + i, to_f(c[i]) * inv * weight[i]);
       if (p.rot > 0) rotate(c + p.rank, dst + p.off_rot, p.rot);
-    } else if (p.off_rot < p.width) {
-      rotate(row + static_cast<size_t>(u - 1) * (p.dim + p.rot) + p.dim,
-             q_out + (static_cast<size_t>(t) * p.H + u - 1) * p.width + p.off_rot, p.width - p.off_rot);
+    } else {
+      const T* q = row + static_cast<size_t>(u - 1) * (p.dim + p.rot);
+      if (q_out != nullptr && p.off_rot < p.width)
+        rotate(q + p.dim, q_out + (static_cast<size_t>(t) * p.H + u - 1) * p.width + p.off_rot, p.width - p.off_rot);
+      if (q_full != nullptr) {
+        T* dst = q_full + (static_cast<size_t>(t) * p.H + u - 1) * p.full;
+        for (int i = lane; i < p.dim; i += 32) dst[i] = q[i];
+        rotate(q + p.dim, dst + p.dim, p.full - p.dim);
+      }
     }
   }
 }
@@ -293,16 +301,16 @@ int tgi_output_gate(int f32, const void* x, const void* gate, long long ld, void
 }
 
 int tgi_latent_store(int f32, const void* proj, long long ld, int off_c, const float* weight, float eps, const int* positions,
-                     const float* cos_sin, int max_pos, const int* slots, void* pages, long long num_slots, void* q_out, int T,
-                     int H, int dim, int rank, int rot, int off_rot, int width, cudaStream_t stream) {
+                     const float* cos_sin, int max_pos, const int* slots, void* pages, long long num_slots, void* q_out,
+                     void* q_full, int T, int H, int dim, int rank, int rot, int off_rot, int width, int full, cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (rot % 2 != 0 || off_rot < rank || width < off_rot + rot || max_pos < 1) return -10;
-  const Latent p{ld, num_slots, off_c, rank, rot, H, dim, off_rot, width, max_pos, eps};
-  const int warps = rot == 0 ? 1 : H + 1 < 8 ? H + 1 : 8;
+  if (rot % 2 != 0 || off_rot < rank || width < off_rot + rot || max_pos < 1 || (q_full != nullptr && full < dim + rot)) return -10;
+  const Latent p{ld, num_slots, off_c, rank, rot, H, dim, off_rot, width, max_pos, full, eps};
+  const int warps = rot == 0 && q_full == nullptr ? 1 : H + 1 < 8 ? H + 1 : 8;
   auto go = [&](auto kern, auto tag) {
     using E = decltype(tag);
     tgi::launch(kern, dim3(T), dim3(32 * warps), 0, stream, static_cast<const E*>(proj), weight, positions, cos_sin, slots,
-                static_cast<E*>(pages), static_cast<E*>(q_out), p);
+                static_cast<E*>(pages), static_cast<E*>(q_out), static_cast<E*>(q_full), p);
     return done();
   };
   return f32 ? go(latent_store_kernel<float>, float()) : go(latent_store_kernel<bf16>, bf16());

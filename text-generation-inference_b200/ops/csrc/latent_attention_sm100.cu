@@ -42,12 +42,13 @@ constexpr float kLog2e = 1.4426950408889634f;
 
 struct LatentParams {
   const int *block_tables, *cu, *kv_lens;
+  const int* elsewhere;           // null, or [B]: sequences whose entry is at least their number of tokens are left out
   const __nv_bfloat16* gate;      // [T, ld_gate] or null: pre-activation of the factor on a head's output
   long long ld_gate;
   __nv_bfloat16* out;             // [T * H, out_cols]
   float *part_o, *part_ml;        // [2 * CTAs][N][out_cols] and [2 * CTAs][N][2]
   int* range;                     // [items][2]: first and last CTA of an item (persistent)
-  int B, max_blocks, num_blocks, H, out_cols, slabs, value_slabs, stages, window, persistent, most;
+  int B, max_blocks, num_blocks, H, out_cols, slabs, value_slabs, stages, window, persistent;
   float scale_log2;
   int* status;
 };
@@ -124,13 +125,17 @@ struct Piece {
   int part;                       // -1: the whole item, else which of the CTA's workspace slots
   int item, last_cta;             // persistent: number of the item, CTA that ends it
 };
+__device__ __forceinline__ bool taken(const LatentParams& p, int b) {
+  const int n = p.cu[b + 1] - p.cu[b];
+  return n > 0 && (p.elsewhere == nullptr || p.elsewhere[b] < n);
+}
 // tiles before sequence b of a decode step (one warp; every item of a sequence has the same number of tiles)
 __device__ __forceinline__ void decode_prefix(const LatentParams& p, int* prefix, int lane) {
   int sum = 0;
   for (int b0 = 0; b0 < p.B; b0 += 32) {
     const int b = b0 + lane;
     int v = 0, t_lo;
-    if (b < p.B && p.cu[b + 1] > p.cu[b]) v = tiles_of(p.kv_lens[b] - 1, p.kv_lens[b] - 1, p.window, t_lo);
+    if (b < p.B && taken(p, b)) v = tiles_of(p.kv_lens[b] - 1, p.kv_lens[b] - 1, p.window, t_lo);
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
       const int got = __shfl_up_sync(0xffffffffu, v, o);
@@ -190,7 +195,7 @@ struct Walk {
     const int begin = p.cu[w.b], n = p.cu[w.b + 1] - begin;
     w.row0 = rt * N;
     w.rows = min(N, n * p.H - w.row0);
-    if (w.rows <= 0 || n > p.most) return false;           // not persistent: nothing here
+    if (w.rows <= 0 || !taken(p, w.b)) return false;       // not persistent: nothing here
     w.q_row = begin * p.H + w.row0;
     const int base = p.kv_lens[w.b] - n;
     w.pos0 = base + w.row0 / p.H;
@@ -597,7 +602,7 @@ latent_merge_kernel(const LatentParams p) {
   __shared__ float red[8];
   const int items = (p.H + N - 1) / N, b = blockIdx.x / items, row = blockIdx.x % items * N + blockIdx.y, r = blockIdx.y;
   const int begin = p.cu[b];
-  if (row >= p.H || p.cu[b + 1] <= begin) return;
+  if (row >= p.H || !taken(p, b)) return;
   const int c0 = p.range[2 * blockIdx.x], c1 = p.range[2 * blockIdx.x + 1];
   if (c0 == c1) return;                                    // one CTA did the whole item
   // the first of the CTAs ended with its part (slot 1), the others began with theirs (slot 0)
@@ -711,12 +716,13 @@ int tgi_latent_rows(int slabs, int value_slabs, long long rows) {
 }
 
 // q [T, H, slabs * 64] and pages [num_blocks, 16, slabs * 64] bf16 (the first value_slabs * 64 columns of a row are the
-// values), out [T, H, value_slabs * 64].  part_o / part_ml: 2 * ctas slots of N x (value_slabs * 64) and N x 2 floats, range:
-// 2 * B * ceil(H / N) ints; used when max_q == 1.  Sequences with more than `most` tokens are left out.  gate (optional): [T, ld_gate].
+// values), out [T, H, value_slabs * 64]; no sequence brings more than max_q tokens.  part_o / part_ml: 2 * ctas slots of N x (value_slabs * 64) and N x 2 floats, range:
+// 2 * B * ceil(H / N) ints; used when max_q == 1.  Sequences whose entry in `elsewhere` (optional, [B]) is at
+// least their number of tokens are left out (and may bring more than max_q).  gate (optional): [T, ld_gate].
 int tgi_latent_attention(const void* q, const void* pages, const int* block_tables, const int* cu, const int* kv_lens,
                          const void* gate, long long ld_gate, void* out, float* part_o, float* part_ml, int* range, int T, int B, int max_q,
                          int max_blocks, int num_blocks, int H, int slabs, int value_slabs, int N, float scale, int window,
-                         int most, int ctas, int* status, cudaStream_t stream) {
+                         const int* elsewhere, int ctas, int* status, cudaStream_t stream) {
   if (T <= 0 || B <= 0 || max_q <= 0) return 0;
   if (N != 16 && N != 32 && N != 64) return -10;
   if (B > 65535 || num_blocks < 1 || max_blocks < 1 || ctas < 1 || slabs > kMaxSlabs || value_slabs > 8 ||
@@ -742,7 +748,7 @@ int tgi_latent_attention(const void* q, const void* pages, const int* block_tabl
   p.stages = stages_for(N, slabs);
   p.window = window;
   p.persistent = max_q == 1 && B <= kMaxSeqs && part_o != nullptr && part_ml != nullptr && range != nullptr;
-  p.most = most;
+  p.elsewhere = elsewhere;
   p.scale_log2 = scale * kLog2e;
   p.status = status;
   const long long rows = static_cast<long long>(T) * H;

@@ -67,7 +67,7 @@ def load():
                  "tgi_activation", "tgi_attn_prep", "tgi_attn_any", "tgi_delta_prep", "tgi_delta_scan", "tgi_decay_scan",
                  "tgi_gated_norm", "tgi_recurrent_pitch", "tgi_delta_tap_rows", "tgi_act_mul_any", "tgi_moe_router",
                  "tgi_moe_router_splits", "tgi_moe_topk_sigmoid", "tgi_moe_topk_logits", "tgi_row_norm_store", "tgi_output_gate",
-                 "tgi_latent_store", "tgi_latent_rows", "tgi_latent_attention", "tgi_moe_grouped_f32", "tgi_moe_combine_f32"):
+                 "tgi_latent_store", "tgi_latent_rows", "tgi_latent_attention", "tgi_expanded_attention", "tgi_moe_grouped_f32", "tgi_moe_combine_f32"):
         if hasattr(_LIB, name):        # a library built for one family of models lacks the other families' kernels
             getattr(_LIB, name).restype = c_int
     _LIB.tgi_gemm_workspace_floats.restype = c_ll
@@ -504,16 +504,41 @@ def latent_layout(rank: int, rot: int, dtype: torch.dtype) -> Tuple[int, int]:
     return rank, rank + rot
 
 
-def latent_store(proj, off_c, weight, eps, positions, cos_sin, slots, pages, q, off_rot, rank: int, rot: int, heads: int, dim: int):
-    assert proj.stride(1) == 1 and pages.is_contiguous() and pages.shape[2] == 1 and pages.dtype == proj.dtype == q.dtype
-    assert q.is_contiguous() and q.shape[2] == pages.shape[3] and weight.dtype == torch.float32 and cos_sin.shape[1] == rot
+def expanded_dims(dim: int, vdim: int, dtype: torch.dtype):
+    """``(query / key width, value width)`` of a head in ``expanded_attention``, ``None`` where it does not take the sizes."""
+    if dtype != torch.bfloat16 or dim > 192 or vdim > 128:
+        return None
+    return (128 if dim <= 128 else 192), 128
+
+
+def expanded_attention(q, kv, plan, cu_seqlens_q, scale, window, max_q: int, gate, out):
+    T, H, dk = q.shape
+    R = kv.shape[0]
+    assert q.is_contiguous() and out.is_contiguous() and tuple(out.shape) == (T, H, 128) and kv.is_contiguous()
+    assert kv.shape[1] == H * (dk + 128) and R % 16 == 0 and (gate is None or gate.stride(1) == 1)
+    st = state(q.device)
+    _check(load().tgi_expanded_attention(
+        _ptr(q), _ptr(kv), c_void_p(kv.data_ptr() + 2 * H * dk), c_ll(kv.stride(0)), _ptr(plan.tables), _ptr(cu_seqlens_q),
+        _ptr(plan.kv_lens), _ptr(gate), c_ll(0 if gate is None else gate.stride(0)), _ptr(out), c_int(plan.kv_lens.shape[0]),
+        c_int(max_q), c_int(plan.tables.shape[1]), c_int(R // 16), c_int(H), c_int(dk), c_float(scale),
+        c_int(window if window and window > 0 else -1), _ptr(st.status), _stream()), "expanded_attention")
+
+
+def latent_store(proj, off_c, weight, eps, positions, cos_sin, slots, pages, q, off_rot, rank: int, rot: int, heads: int, dim: int,
+                 q_full=None):
+    assert proj.stride(1) == 1 and pages.is_contiguous() and pages.shape[2] == 1 and pages.dtype == proj.dtype
+    assert q is None or (q.is_contiguous() and q.shape[2] == pages.shape[3] and q.dtype == proj.dtype)
+    assert q_full is None or (q_full.is_contiguous() and q_full.dtype == proj.dtype)
+    assert weight.dtype == torch.float32 and cos_sin.shape[1] == rot
     _check(load().tgi_latent_store(
         _f32(proj), _ptr(proj), c_ll(proj.stride(0)), c_int(off_c), _ptr(weight), c_float(eps), _ptr(positions), _ptr(cos_sin),
-        c_int(cos_sin.shape[0]), _ptr(slots), _ptr(pages), c_ll(pages.shape[0] * pages.shape[1]), _ptr(q), c_int(proj.shape[0]),
-        c_int(heads), c_int(dim), c_int(rank), c_int(rot), c_int(off_rot), c_int(pages.shape[3]), _stream()), "latent_store")
+        c_int(cos_sin.shape[0]), _ptr(slots), _ptr(pages), c_ll(pages.shape[0] * pages.shape[1]), _ptr(q), _ptr(q_full),
+        c_int(proj.shape[0]), c_int(heads), c_int(dim), c_int(rank), c_int(rot), c_int(off_rot), c_int(pages.shape[3]),
+        c_int(0 if q_full is None else q_full.shape[2]), _stream()), "latent_store")
 
 
-def latent_attention(q, pages, rank: int, block_tables, cu_seqlens_q, kv_lens, scale, window=-1, max_q=None, max_kv=None, gate=None):
+def latent_attention(q, pages, rank: int, block_tables, cu_seqlens_q, kv_lens, scale, window=-1, max_q=None, max_kv=None, gate=None,
+                     elsewhere=None):
     """Tensor-core kernel for bf16 rows in 64-column pieces on pages of 16 tokens, ``tgi_attn_any`` otherwise."""
     lib = load()
     T, H, width = q.shape
@@ -531,9 +556,10 @@ def latent_attention(q, pages, rank: int, block_tables, cu_seqlens_q, kv_lens, s
                 _ptr(q), _ptr(pages), _ptr(block_tables), _ptr(cu_seqlens_q), _ptr(kv_lens), _ptr(gate),
                 c_ll(0 if gate is None else gate.stride(0)), _ptr(out), *map(_ptr, part), c_int(T), c_int(B), c_int(max_q),
                 c_int(block_tables.shape[1]), c_int(pages.shape[0]), c_int(H), c_int(width // 64), c_int(values), c_int(N),
-                c_float(scale), c_int(window if window and window > 0 else -1), c_int(1 << 30), c_int(st.sm_count),
+                c_float(scale), c_int(window if window and window > 0 else -1), _ptr(elsewhere), c_int(st.sm_count),
                 _ptr(st.status), _stream()), "latent_attention")
             return out
+    assert elsewhere is None
     out = q.new_empty(T, H, rank)
     if T == 0:
         return out

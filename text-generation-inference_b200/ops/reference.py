@@ -483,7 +483,9 @@ def output_gate(x, gate, width: int):
     return (x[:, :, :width].reshape(T, -1).float() * torch.sigmoid(gate.float())).to(x.dtype)
 
 
-def latent_store(proj, off_c, weight, eps: float, positions, cos_sin, slots, pages, q, off_rot, rank, rot, heads, dim):
+def latent_store(proj, off_c, weight, eps: float, positions, cos_sin, slots, pages, q, off_rot, rank, rot, heads, dim,
+                 q_full=None):
+    assert q_full is None
     T = proj.shape[0]
     _store_rows(pages, slots, _row_rms(proj[:, off_c:off_c + rank], weight, eps).unsqueeze(1))
     if rot:
@@ -494,7 +496,8 @@ def latent_store(proj, off_c, weight, eps: float, positions, cos_sin, slots, pag
 
 
 def latent_attention(q, pages, rank, block_tables, cu_seqlens_q, kv_lens, scale: float, window: int = -1, max_q=None, max_kv=None,
-                     gate=None):
+                     gate=None, elsewhere=None):
+    assert elsewhere is None
     o = paged_attention(q, pages, pages[..., :rank].contiguous(), block_tables, cu_seqlens_q, kv_lens, scale, window)
     return o if gate is None else (o.float() * torch.sigmoid(gate.float()).unsqueeze(2)).to(o.dtype)
 
