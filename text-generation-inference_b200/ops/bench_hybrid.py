@@ -1,8 +1,9 @@
 """Prefill and decode throughput of a hybrid decoder beside its closest relative of the same width, depth, heads and
 active parameters per token, and the kernels of both against their rooflines.
 
-``python bench.py --model fuzuvik-bf16`` (beside a Llama shape) and ``--model kipedra-bf16`` (beside a Fuzuvik shape; expert
-kernels beside those of gated experts) print one JSON line.  Weights are random; token rates are timed with CUDA
+``python bench.py --model fuzuvik-bf16`` (beside a Llama shape), ``--model kipedra-bf16`` (beside a Fuzuvik shape; expert
+kernels beside those of gated experts) and ``--model gisilix-bf16`` (beside a DeepSeek shape, ``bench_latent``) print one JSON
+line.  Weights are random; token rates are timed with CUDA
 events around the model's forward (prefill) and around replays of its decode graph.  Kernels are timed one by one
 with the L2 flushed in front of every launch; a roofline is the larger of bytes over the measured copy bandwidth and
 FLOPs over the measured rate of the unit that does them (bf16 tensor cores, or fp32 FMA for the state recurrences).
@@ -76,10 +77,14 @@ def make_runner(cfg: dict, dev):
     from ..utils.tokenizer import ByteTokenizer
 
     mc = ModelConfig(cfg)
-    if cfg.get("architecture"):
-        tensors = (syn.kipedra_state_dict(cfg, dtype=torch.bfloat16, device=str(dev)) if cfg["architecture"] == "Kipedra" else
-                   syn.fuzuvik_state_dict(cfg, dtype=torch.bfloat16, device=str(dev), rank=128))
-        w = syn.DictWeights(tensors, dev, torch.bfloat16, bare_names=True)
+    if cfg.get("architecture") or cfg["model_type"] == "deepseek_v2":
+        from .bench_latent import deepseek_tensors
+
+        kw = dict(dtype=torch.bfloat16, device=str(dev))
+        tensors = {"Kipedra": lambda: syn.kipedra_state_dict(cfg, **kw), "Gisilix": lambda: syn.gisilix_state_dict(cfg, **kw),
+                   "Fuzuvik": lambda: syn.fuzuvik_state_dict(cfg, rank=128, **kw),
+                   None: lambda: deepseek_tensors(cfg, dev)}[cfg.get("architecture")]()
+        w = syn.DictWeights(tensors, dev, torch.bfloat16, bare_names=bool(cfg.get("architecture")))
         del tensors
     else:
         w = syn.SyntheticWeights(cfg, dev, torch.bfloat16)
@@ -377,29 +382,37 @@ def kipedra_rows(dev, width: int, window: int, prefill, decode) -> list:
 
 def run(args, clock_sampler) -> int:
     from . import cuda as K
+    from .bench_latent import deepseek_like, gisilix_like, gisilix_rows
 
-    kipedra = args.model == "kipedra-bf16"
     dev = torch.device("cuda", 0)
     torch.cuda.set_device(dev)
     K.load()
-    vocab, layers, span = 32000, args.layers or 8, 1024 if kipedra else 8192
-    name, other = ("kipedra", "fuzuvik") if kipedra else ("fuzuvik", "llama")
+    vocab, layers = 32000, args.layers or 8
+    # model, its relative, kernels, window or chunk, (batch, context) of the decode steps both run and of those it runs alone
+    name, own, other, twin, rows_of, span, decodes, alone = {
+        "fuzuvik-bf16": ("fuzuvik", fuzuvik_like, "llama", lambda w, n, v, s: llama_like(w, n, v), kernel_rows, 8192, [(16, 2048), (256, 2048)], []),
+        "kipedra-bf16": ("kipedra", kipedra_like, "fuzuvik", fuzuvik_twin, kipedra_rows, 1024, [(16, 2048), (256, 2048)], []),
+        # 256 x 2048 tokens of keys and values per head do not fit beside the weights
+        "gisilix-bf16": ("gisilix", gisilix_like, "deepseek", lambda w, n, v, s: deepseek_like(w, n, v), gisilix_rows, 1024,
+                         [(16, 2048), (64, 2048)], [(256, 2048)]),
+    }[args.model]
     sampler = clock_sampler(0)
     sampler.start()
     sizes = {}
-    prefills, decodes = [(4, 2048), (1, 8192)], [(16, 2048), (256, 2048)]
+    prefills = [(4, 2048), (1, 8192)]
     for width in (2048, 4096):
-        cfgs = {name: (kipedra_like if kipedra else fuzuvik_like)(width, layers, vocab, span),
-                other: fuzuvik_twin(width, layers, vocab, span) if kipedra else llama_like(width, layers, vocab)}
-        sizes[str(width)] = {k: model_rates(c, dev, vocab, prefills, decodes, args.steps, args.warmup) for k, c in cfgs.items()}
-    rows = (kipedra_rows if kipedra else kernel_rows)(dev, 4096, span, (4, 2048), (256, 2048))
+        cfgs = {name: own(width, layers, vocab, span), other: twin(width, layers, vocab, span)}
+        sizes[str(width)] = {k: model_rates(c, dev, vocab, prefills, decodes + (alone if k == name else []), args.steps, args.warmup)
+                             for k, c in cfgs.items()}
+    batch = (decodes + alone)[-1][0]
+    rows = rows_of(dev, 4096, span, (4, 2048), (decodes[-1][0], 2048))
     clocks = sampler.stop()
-    value = sizes["4096"][name]["decode_tok_s"]["256@2048"]
+    value = sizes["4096"][name]["decode_tok_s"][f"{batch}@2048"]
     print(json.dumps({
         "metric": f"output tok/s (decode, {args.model})", "value": value, "unit": "tok/s", "n_gpus": 1, "steps": args.steps,
-        "warmup": args.warmup, "ms_per_step": round(256e3 / value, 4), "higher_is_better": True, "scaling": "strong",
+        "warmup": args.warmup, "ms_per_step": round(batch * 1e3 / value, 4), "higher_is_better": True, "scaling": "strong",
         "vs_baseline": None, "dtype": "bf16", "data": "synthetic: random tokens, random weights", "impl": "b200",
-        "config": {"model": f"{name}-{layers}L", "global_batch": 256, "seq_len": 2048, "window" if kipedra else "chunk": span,
+        "config": {"model": f"{name}-{layers}L", "global_batch": batch, "seq_len": 2048, "chunk" if name == "fuzuvik" else "window": span,
                    "parallelism": "tp1", "l2": "models: inputs larger than L2; kernels: L2 flushed before every launch"},
         "sizes": sizes, "kernels": rows, "peaks": peaks()[2], "clocks": clocks}), flush=True)
     return 0

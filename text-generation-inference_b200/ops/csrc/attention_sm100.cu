@@ -235,6 +235,10 @@ __device__ __forceinline__ float fast_exp2(float x) {   // ex2.approx: 2 ulp, -i
   return y;
 }
 
+__device__ __forceinline__ float fast_tanh(float y) {      // 1 - 2 / (1 + e^(2y)); saturates cleanly at +-1
+  return 1.f - __fdividef(2.f, 1.f + fast_exp2(y * (2.f * kLog2e)));
+}
+
 template <int NT>
 __device__ __forceinline__ void softmax_update(float (&s)[NT][4], float (&m)[2], float (&l)[2], float (&alpha)[2],
                                                int tbase, int pos0, int pos1, int lo0, int lo1, int lo_max, int L,
@@ -250,6 +254,7 @@ __device__ __forceinline__ void softmax_update(float (&s)[NT][4], float (&m)[2],
   // sequence needs no per-element mask (warp-uniform test: the warp's first row is pos0 - lane / 4)
   const int row_lo = hz0 - (lane >> 2), t_last = tbase + NT * 8 - 1;
   const bool plain = softcap <= 0.f && t_last <= row_lo && t_last < L && tbase >= lo_max;
+  const float cap_in = softcap > 0.f ? raw_scale / softcap : 0.f;
   if (plain) {
 #pragma unroll
     for (int i = 0; i < NT; ++i) {
@@ -267,7 +272,7 @@ __device__ __forceinline__ void softmax_update(float (&s)[NT][4], float (&m)[2],
         const int lo = (e < 2) ? lo0 : lo1;
         const int hz = (e < 2) ? hz0 : hz1;
         float v = s[i][e];
-        if (softcap > 0.f) v = softcap * tanhf(v * raw_scale / softcap) * kLog2e;
+        if (softcap > 0.f) v = softcap * kLog2e * fast_tanh(v * cap_in);
         else v = v * scale_log2;
         const bool ok = t <= hz && t < L && t >= lo;
         v = ok ? v : -INFINITY;
@@ -900,6 +905,7 @@ decode_kernel_v3(Params p, const __grid_constant__ CUtensorMap tmK, const __grid
   const float vsc = p.v_scale ? p.v_scale[kvh] : 1.f;
   const float raw_scale = p.scale * (FP8 ? ksc : 1.f);
   const float scale_log2 = raw_scale * kLog2e;
+  const float cap_in = p.softcap > 0.f ? raw_scale / p.softcap : 0.f;
   const int rg = bitrev3(g);                      // token row (mod 8) of this lane's S^T rows
   const int rj0 = bitrev3(j), rj1 = bitrev3(j + 4);   // token rows (mod 8) of this lane's V loads
   bool failed = false;
@@ -976,7 +982,7 @@ decode_kernel_v3(Params p, const __grid_constant__ CUtensorMap tmK, const __grid
         for (int e = 0; e < 4; ++e) {
           const int t = tbase + mt * 16 + rg + (e >> 1) * 8;
           float v = s[mt][e];
-          if (p.softcap > 0.f) v = p.softcap * tanhf(v * raw_scale / p.softcap) * kLog2e;
+          if (p.softcap > 0.f) v = p.softcap * kLog2e * fast_tanh(v * cap_in);
           else v = v * scale_log2;
           const bool ok = t < L && t >= lo;
           v = ok ? v : -INFINITY;

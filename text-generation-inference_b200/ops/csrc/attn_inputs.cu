@@ -184,9 +184,10 @@ output_gate_kernel(const T* __restrict__ x, const T* __restrict__ gate, long lon
 
 // ------------------------------------------------------------------------------------------------
 // Inputs of latent attention.  proj[T, ld]: queries (H heads of dim plain and rot rotated dimensions) at column 0, latent
-// (rank) and the shared key's rotated part (rot) at off_c.  One CTA per token; a warp normalises the latent and rotates the
-// shared part, the others rotate the queries of a head each.  Pairs 2i, 2i + 1.  Rotated dimensions go to q_out from column
-// off_rot on (null: not wanted), whole queries (plain, rotated, zeros) to q_full, `full` columns per head (null: not wanted).
+// (rank) and the shared key's rotated part (rot) at off_c.  Grid (T, groups): a warp of the first group normalises the latent
+// and rotates the shared part, the others rotate the queries of a head each.  Pairs 2i, 2i + 1.  Rotated dimensions go to
+// q_out from column off_rot on (null: not wanted), whole queries (plain, rotated, zeros) to q_full, `full` columns per head
+// (null: not wanted).  VEC: every offset, size and pitch is a multiple of 8 elements; a lane then takes 8 at a time.
 // ------------------------------------------------------------------------------------------------
 struct Latent {
   long long ld, num_slots;
@@ -195,44 +196,128 @@ struct Latent {
   float eps;
 };
 template <typename T>
+__device__ __forceinline__ void load8(const T* p, float (&x)[8]) {
+  if constexpr (sizeof(T) == 2) {
+    load_vec<T>(p, x);
+  } else {
+    const float4 a = load4(p), b = load4(p + 4);
+    x[0] = a.x; x[1] = a.y; x[2] = a.z; x[3] = a.w;
+    x[4] = b.x; x[5] = b.y; x[6] = b.z; x[7] = b.w;
+  }
+}
+template <typename T>
+__device__ __forceinline__ void store8(T* p, const float (&x)[8]) {
+  if constexpr (sizeof(T) == 2) {
+    store_vec(p, x);
+  } else {
+    store4(p, make_float4(x[0], x[1], x[2], x[3]));
+    store4(p + 4, make_float4(x[4], x[5], x[6], x[7]));
+  }
+}
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(256)
 latent_store_kernel(const T* __restrict__ proj, const float* __restrict__ weight, const int* __restrict__ positions,
                     const float* __restrict__ cos_sin, const int* __restrict__ slots, T* __restrict__ pages,
                     T* __restrict__ q_out, T* __restrict__ q_full, Latent p) {
   tgi::pdl_wait();
   tgi::pdl_trigger();
-  const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+  const int t = blockIdx.x, lane = threadIdx.x & 31, warps = (blockDim.x >> 5) * gridDim.y;
+  const int warp = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
   const T* row = proj + static_cast<size_t>(t) * p.ld;
   const int rh = p.rot / 2, pos = min(max(positions[t], 0), p.max_pos - 1);
   const float* cs = cos_sin + static_cast<size_t>(pos) * p.rot;
-  auto rotate = [&](const T* src, T* dst, int end) {       // rotated pairs, then zeros up to `end`
-    for (int i = lane; i < rh; i += 32) {
-      const float u = to_f(src[2 * i]), v = to_f(src[2 * i + 1]), c = cs[i], s = cs[rh + i];
-      put(dst + 2 * i, u * c - v * s);
-      put(dst + 2 * i + 1, v * c + u * s);
+  const float zero[8] = {};
+  auto rotate = [&](const T* src, T* dst, int end, int l, int step) {      // rotated pairs, then zeros up to `end`
+    if constexpr (VEC) {
+      for (int i = 8 * l; i < end; i += 8 * step) {
+        if (i >= p.rot) {
+          store8(dst + i, zero);
+          continue;
+        }
+        float x[8];
+        load8(src + i, x);
+        const float4 c = *reinterpret_cast<const float4*>(cs + i / 2), s = *reinterpret_cast<const float4*>(cs + rh + i / 2);
+        const float y[8] = {x[0] * c.x - x[1] * s.x, x[1] * c.x + x[0] * s.x, x[2] * c.y - x[3] * s.y, x[3] * c.y + x[2] * s.y,
+                            x[4] * c.z - x[5] * s.z, x[5] * c.z + x[4] * s.z, x[6] * c.w - x[7] * s.w, x[7] * c.w + x[6] * s.w};
+        store8(dst + i, y);
+      }
+    } else {
+      for (int i = l; i < rh; i += step) {
+        const float u = to_f(src[2 * i]), v = to_f(src[2 * i + 1]), c = cs[i], s = cs[rh + i];
+        put(dst + 2 * i, u * c - v * s);
+        put(dst + 2 * i + 1, v * c + u * s);
+      }
+      for (int i = p.rot + l; i < end; i += step) put(dst + i, 0.f);
     }
-    for (int i = p.rot + lane; i < end; i += 32) put(dst + i, 0.f);
   };
-  for (int u = warp; u <= p.H; u += warps) {
-    if (u == 0) {
-      const long long slot = slots[t];
-      if (slot < 0 || slot >= p.num_slots) continue;       // padding rows have slot -1
+  if (warp == 0) {
+    const long long slot = slots[t];
+    if (slot >= 0 && slot < p.num_slots) {                 // padding rows have slot -1
       const T* c = row + p.off_c;
       T* dst = pages + static_cast<size_t>(slot) * p.width;
       float ss = 0.f;
-      for (int i = lane; i < p.rank; i += 32) ss = fmaf(to_f(c[i]), to_f(c[i]), ss);
-      const float inv = 1.f / sqrtf(warp_sum(ss) / p.rank + p.eps);
-      for (int i = lane; i < p.rank; i += 32) put(dst + i, to_f(c[i]) * inv * weight[i]);
-      if (p.rot > 0) rotate(c + p.rank, dst + p.off_rot, p.rot);
-    } else {
-      const T* q = row + static_cast<size_t>(u - 1) * (p.dim + p.rot);
-      if (q_out != nullptr && p.off_rot < p.width)
-        rotate(q + p.dim, q_out + (static_cast<size_t>(t) * p.H + u - 1) * p.width + p.off_rot, p.width - p.off_rot);
-      if (q_full != nullptr) {
-        T* dst = q_full + (static_cast<size_t>(t) * p.H + u - 1) * p.full;
-        for (int i = lane; i < p.dim; i += 32) dst[i] = q[i];
-        rotate(q + p.dim, dst + p.dim, p.full - p.dim);
+      if constexpr (VEC) {
+        constexpr int kHeld = 2;                           // pieces per lane that stay in registers
+        float x[kHeld][8];
+#pragma unroll
+        for (int e = 0; e < kHeld; ++e) {
+          const int i = 8 * (lane + 32 * e);
+#pragma unroll
+          for (int k = 0; k < 8; ++k) x[e][k] = 0.f;
+          if (i < p.rank) load8(c + i, x[e]);
+#pragma unroll
+          for (int k = 0; k < 8; ++k) ss = fmaf(x[e][k], x[e][k], ss);
+        }
+        for (int i = 8 * (lane + 32 * kHeld); i < p.rank; i += 256) {
+          float y[8];
+          load8(c + i, y);
+#pragma unroll
+          for (int k = 0; k < 8; ++k) ss = fmaf(y[k], y[k], ss);
+        }
+        const float inv = 1.f / sqrtf(warp_sum(ss) / p.rank + p.eps);
+        auto emit = [&](int i, float (&y)[8]) {
+#pragma unroll
+          for (int k = 0; k < 8; k += 4) {
+            const float4 w = *reinterpret_cast<const float4*>(weight + i + k);
+            y[k] *= inv * w.x; y[k + 1] *= inv * w.y; y[k + 2] *= inv * w.z; y[k + 3] *= inv * w.w;
+          }
+          store8(dst + i, y);
+        };
+#pragma unroll
+        for (int e = 0; e < kHeld; ++e) {
+          const int i = 8 * (lane + 32 * e);
+          if (i < p.rank) emit(i, x[e]);
+        }
+        for (int i = 8 * (lane + 32 * kHeld); i < p.rank; i += 256) {
+          float y[8];
+          load8(c + i, y);
+          emit(i, y);
+        }
+      } else {
+        for (int i = lane; i < p.rank; i += 32) ss = fmaf(to_f(c[i]), to_f(c[i]), ss);
+        const float inv = 1.f / sqrtf(warp_sum(ss) / p.rank + p.eps);
+        for (int i = lane; i < p.rank; i += 32) put(dst + i, to_f(c[i]) * inv * weight[i]);
       }
+      if (p.rot > 0) rotate(c + p.rank, dst + p.off_rot, p.rot, lane, 32);
+    }
+  }
+  // eight lanes per head
+  const int l = lane & 7, tail = p.width - p.off_rot;
+  for (int h = 4 * warp + (lane >> 3); h < p.H; h += 4 * warps) {
+    const T* q = row + static_cast<size_t>(h) * (p.dim + p.rot);
+    if (q_out != nullptr && tail > 0) rotate(q + p.dim, q_out + (static_cast<size_t>(t) * p.H + h) * p.width + p.off_rot, tail, l, 8);
+    if (q_full != nullptr) {
+      T* dst = q_full + (static_cast<size_t>(t) * p.H + h) * p.full;
+      if constexpr (VEC) {
+        for (int i = 8 * l; i < p.dim; i += 64) {
+          float x[8];
+          load8(q + i, x);
+          store8(dst + i, x);
+        }
+      } else {
+        for (int i = l; i < p.dim; i += 8) dst[i] = q[i];
+      }
+      rotate(q + p.dim, dst + p.dim, p.full - p.dim, l, 8);
     }
   }
 }
@@ -306,14 +391,19 @@ int tgi_latent_store(int f32, const void* proj, long long ld, int off_c, const f
   if (T <= 0) return 0;
   if (rot % 2 != 0 || off_rot < rank || width < off_rot + rot || max_pos < 1 || (q_full != nullptr && full < dim + rot)) return -10;
   const Latent p{ld, num_slots, off_c, rank, rot, H, dim, off_rot, width, max_pos, full, eps};
-  const int warps = rot == 0 && q_full == nullptr ? 1 : H + 1 < 8 ? H + 1 : 8;
+  const bool heads = q_full != nullptr || (q_out != nullptr && width > off_rot);
+  const int want = heads ? (H + 3) / 4 : 1, warps = want < 4 ? want : 4;       // four heads per warp at a time
+  const int groups = T >= 1024 ? 1 : (want + warps - 1) / warps;
+  const bool vec = dim % 8 == 0 && rot % 8 == 0 && rank % 8 == 0 && off_c % 8 == 0 && ld % 8 == 0 && off_rot % 8 == 0 && width % 8 == 0 &&
+                   (q_full == nullptr || full % 8 == 0) && reinterpret_cast<uintptr_t>(proj) % 16 == 0;
   auto go = [&](auto kern, auto tag) {
     using E = decltype(tag);
-    tgi::launch(kern, dim3(T), dim3(32 * warps), 0, stream, static_cast<const E*>(proj), weight, positions, cos_sin, slots,
+    tgi::launch(kern, dim3(T, groups), dim3(32 * warps), 0, stream, static_cast<const E*>(proj), weight, positions, cos_sin, slots,
                 static_cast<E*>(pages), static_cast<E*>(q_out), static_cast<E*>(q_full), p);
     return done();
   };
-  return f32 ? go(latent_store_kernel<float>, float()) : go(latent_store_kernel<bf16>, bf16());
+  if (vec) return f32 ? go(latent_store_kernel<float, true>, float()) : go(latent_store_kernel<bf16, true>, bf16());
+  return f32 ? go(latent_store_kernel<float, false>, float()) : go(latent_store_kernel<bf16, false>, bf16());
 }
 
 }  // extern "C"

@@ -5,8 +5,10 @@
 // A CTA owns N query rows (16, 32 or 64) and walks a range of keys in tiles of 64.  Both products are transposed, so that
 // keys (or value columns) are the rows of the MMA and a tile of few query rows wastes nothing:
 //   S^T = K Q^T     M 64 (keys) x N x K width
-//   P^T = softmax   four warps, half of the query rows of a key per thread: column maxima by a transposing butterfly and
-//                   shared memory, P^T as bf16 rows [key][N] in shared memory (MN-major operand B)
+//   P^T = softmax   four warps, half of the query rows of a key per thread, P^T as bf16 rows [key][N] in shared memory
+//                   (MN-major operand B).  The maximum that the exponents refer to is kept while no score passes it by
+//                   more than kSlack (one reducing barrier tells); otherwise column maxima are taken by a transposing
+//                   butterfly and shared memory, and sums and outputs are rescaled
 //   O^T = V^T P^T   M 128 (value columns) x N x K 64 (keys), one product per 128 value columns; V^T is the K tile as it
 //                   lies, taken as the MN-major operand A
 // The output stays in registers of the output warps (a value column per thread, N query rows), which rescale it and add
@@ -38,6 +40,8 @@ namespace {
 constexpr int kKeys = 64, kPage = 16;
 constexpr int kMaxSlabs = 12, kMaxSeqs = 1024, kMaxStages = 4;
 constexpr int kPTile = kKeys * 128;             // bytes of a P^T tile
+constexpr float kSlack = 8.f;                   // log2: probabilities stay below 256 times those of the true maximum
+constexpr float kNoMax = -1e30f;                // maximum of no key
 constexpr float kLog2e = 1.4426950408889634f;
 
 struct LatentParams {
@@ -129,13 +133,20 @@ __device__ __forceinline__ bool taken(const LatentParams& p, int b) {
   const int n = p.cu[b + 1] - p.cu[b];
   return n > 0 && (p.elsewhere == nullptr || p.elsewhere[b] < n);
 }
-// tiles before sequence b of a decode step (one warp; every item of a sequence has the same number of tiles)
+// Tiles before sequence b of a decode step (every item of a sequence has the same number of tiles): the whole CTA looks up
+// the sequences, one warp adds up.
+__device__ __forceinline__ void decode_tiles(const LatentParams& p, int* prefix) {
+  for (int b = threadIdx.x; b < p.B; b += blockDim.x) {
+    int t_lo;
+    prefix[b + 1] = taken(p, b) ? tiles_of(p.kv_lens[b] - 1, p.kv_lens[b] - 1, p.window, t_lo) : 0;
+  }
+  if (threadIdx.x == 0) prefix[0] = 0;
+}
 __device__ __forceinline__ void decode_prefix(const LatentParams& p, int* prefix, int lane) {
   int sum = 0;
   for (int b0 = 0; b0 < p.B; b0 += 32) {
     const int b = b0 + lane;
-    int v = 0, t_lo;
-    if (b < p.B && taken(p, b)) v = tiles_of(p.kv_lens[b] - 1, p.kv_lens[b] - 1, p.window, t_lo);
+    int v = b < p.B ? prefix[b + 1] : 0;
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
       const int got = __shfl_up_sync(0xffffffffu, v, o);
@@ -144,7 +155,6 @@ __device__ __forceinline__ void decode_prefix(const LatentParams& p, int* prefix
     if (b < p.B) prefix[b + 1] = sum + v;
     sum += __shfl_sync(0xffffffffu, v, 31);
   }
-  if (lane == 0) prefix[0] = 0;
 }
 __device__ __forceinline__ int sequence_at(const int* prefix, int B, int items, long long g) {
   int lo = 0, hi = B - 1;         // the last b with prefix[b] * items <= g that has tiles
@@ -231,6 +241,19 @@ __device__ __forceinline__ bool mbar_test(uint64_t* bar, uint32_t parity) {
       : "memory");
   return ok != 0;
 }
+// whether the predicate holds for any thread of the four softmax warps; a barrier for them
+__device__ __forceinline__ bool any_of_128(bool v) {
+  uint32_t r;
+  asm volatile(
+      "{\n\t.reg .pred P, Q;\n\t"
+      "setp.ne.u32 P, %1, 0;\n\t"
+      "bar.red.or.pred Q, 1, 128, P;\n\t"
+      "selp.u32 %0, 1, 0, Q;\n\t}"
+      : "=r"(r)
+      : "r"(static_cast<uint32_t>(v))
+      : "memory");
+  return r != 0;
+}
 // box of a page: 64 columns x 8 tokens x slabs x 2
 __device__ __forceinline__ void tma_load_page(void* dst, const CUtensorMap* map, uint64_t* bar, int group) {
   asm volatile(
@@ -272,6 +295,7 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
   uint64_t* l_ready = q_full + 2;
   uint64_t* l_free = q_full + 3;
   uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(q_full + 4);
+  int* s_rescale = reinterpret_cast<int*>(tmem_holder + 1);       // [2] a tile's s_alpha are not all 1
   int* prefix = reinterpret_cast<int*>(tmem_holder + 4);          // [B + 1], persistent only
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -302,7 +326,11 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
   }
   tgi::pdl_wait();
   tgi::pdl_trigger();
-  if (warp == 2 && p.persistent) decode_prefix(p, prefix, lane);
+  if (p.persistent) {
+    decode_tiles(p, prefix);
+    __syncthreads();
+    if (warp == 2) decode_prefix(p, prefix, lane);
+  }
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
@@ -372,12 +400,12 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
         if (i == 0 && !wait(q_full, (np - 1) & 1, kErrMmaWaitFull)) return false;
         if (!wait(&k_full[stage], round & 1, kErrMmaWaitFull)) return false;
         tc_fence_after();
-        const uint32_t a = k_addr + stage * tile_bytes, d = tS + (tile & 1) * N;
-        for (int x = 0; x < p.slabs; ++x) {
+        const uint32_t d = tS + (tile & 1) * N;
+        uint64_t da = make_desc(k_addr + stage * tile_bytes, 16, group_bytes), db = make_desc(q_addr, 16, 1024);
+        for (int x = 0; x < p.slabs; ++x, da += 1024 >> 4, db += N * 128 >> 4) {
 #pragma unroll
           for (int k = 0; k < 4; ++k)                      // 16 columns (32 bytes) per MMA
-            mma_f16(d, make_desc(a + x * 1024, 16, group_bytes) + (k * 32 >> 4), make_desc(q_addr + x * N * 128, 16, 1024) + (k * 32 >> 4),
-                    id_s, x > 0 || k > 0 ? 1u : 0u);
+            mma_f16(d, da + (k * 32 >> 4), db + (k * 32 >> 4), id_s, x > 0 || k > 0 ? 1u : 0u);
         }
         tc_commit(&s_full[tile & 1]);
         if (i + 1 == w.tiles) tc_commit(q_free);
@@ -402,12 +430,13 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
         }
         if (!ok || !wait(ready, phase, kErrMmaWaitFull)) break;
         tc_fence_after();
-        const uint32_t a = k_addr + o_stage * tile_bytes, b = p_addr + (j & 1) * kPTile, d = tO + (j & 1) * blocks * N;
-        for (int x = 0; x < blocks; ++x) {
+        const uint32_t d = tO + (j & 1) * blocks * N;
+        uint64_t da = make_desc(k_addr + o_stage * tile_bytes, 1024, group_bytes);
+        const uint64_t db = make_desc(p_addr + (j & 1) * kPTile, 16, 1024);
+        for (int x = 0; x < blocks; ++x, da += 2048 >> 4) {
 #pragma unroll
           for (int k = 0; k < 4; ++k)                      // 16 keys per MMA: two groups of eight rows
-            mma_f16(d + x * N, make_desc(a + 2 * x * 1024 + 2 * k * group_bytes, 1024, group_bytes), make_desc(b + k * 2048, 16, 1024), id_o,
-                    k > 0 ? 1u : 0u);
+            mma_f16(d + x * N, da + (2 * k * group_bytes >> 4), db + (k * 2048 >> 4), id_o, k > 0 ? 1u : 0u);
         }
         tc_commit(&o_full[j & 1]);
         tc_commit(&k_free[o_stage]);
@@ -426,8 +455,9 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
       for (int x = 0; x < NC; ++x)
 #pragma unroll
         for (int c = 0; c < C; ++c) l[x][c] = 0.f;
-      float m = -INFINITY;                                 // thread c < N: running maximum of row c
+      float m = kNoMax;                                    // thread c < N: reference maximum of row c
       if (tid < N) {
+        s_m[tid] = kNoMax;
         const int pos = w.pos0 + (w.row0 % p.H + min(tid, w.rows - 1)) / p.H;
         s_lo[tid] = first_visible(pos, p.window);
         s_hi[tid] = pos;
@@ -442,33 +472,53 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
         wait(&s_full[buf], (j >> 1) & 1, kErrEpilogueWait);
         tc_fence_after();
         float x[NC][C];
+        bool over = false;
 #pragma unroll
         for (int n = 0; n < NC; ++n) {
-          float v[W], y[C];
+          float v[W];
           tmem_load<W>(addr + buf * N + n * W, v);
+          const int col0 = n * W + half * C;
 #pragma unroll
           for (int c = 0; c < C; ++c) {                    // the upper lanes take over the second half of the columns
             const float got = __shfl_xor_sync(0xffffffffu, v[c + C], 16);
             x[n][c] = (half ? got : v[c]) * p.scale_log2;
-            if (!plain) {
-              const int col = n * W + half * C + c;
-              if (t < s_lo[col] || t > s_hi[col]) x[n][c] = -INFINITY;
-            }
-            y[c] = x[n][c];
           }
-          const float mx = column_reduce<C, false>(y, lane);
-          if ((lane & 15) < C) s_max[quarter * N + n * W + half * C + (lane & 15)] = mx;
+          if (!plain) {
+#pragma unroll
+            for (int c = 0; c < C; ++c)
+              if (t < s_lo[col0 + c] || t > s_hi[col0 + c]) x[n][c] = -INFINITY;
+          }
+#pragma unroll
+          for (int c = 0; c < C; c += 4) {
+            const float4 mm = *reinterpret_cast<const float4*>(s_m + col0 + c);
+            over |= fmaxf(fmaxf(x[n][c] - mm.x, x[n][c + 1] - mm.y), fmaxf(x[n][c + 2] - mm.z, x[n][c + 3] - mm.w)) > kSlack;
+          }
         }
         // the output of the tile before the last has been taken: its factors and its P^T are free
         if (j > 1) wait(&o_free[buf], ((j >> 1) - 1) & 1, kErrEpilogueWait);
-        asm volatile("bar.sync 1, 128;" ::: "memory");
-        if (tid < N) {
-          const float mn = fmaxf(fmaxf(fmaxf(s_max[tid], s_max[N + tid]), fmaxf(s_max[2 * N + tid], s_max[3 * N + tid])), m);
-          s_alpha[buf * N + tid] = mn == -INFINITY ? 1.f : ex2(m - mn);
-          s_m[tid] = mn == -INFINITY ? 0.f : mn;
-          m = mn;
+        const bool rescale = any_of_128(over);
+        if (tid == 0) s_rescale[buf] = rescale;
+        if (rescale) {                                     // uniform over the four warps
+#pragma unroll
+          for (int n = 0; n < NC; ++n) {
+            float y[C];
+#pragma unroll
+            for (int c = 0; c < C; ++c) y[c] = x[n][c];
+            const float mx = column_reduce<C, false>(y, lane);
+            if ((lane & 15) < C) s_max[quarter * N + n * W + half * C + (lane & 15)] = mx;
+          }
+          asm volatile("bar.sync 1, 128;" ::: "memory");
+          if (tid < N) {
+            const float mn = fmaxf(fmaxf(fmaxf(s_max[tid], s_max[N + tid]), fmaxf(s_max[2 * N + tid], s_max[3 * N + tid])), m);
+            s_alpha[buf * N + tid] = ex2(m - mn);
+            s_m[tid] = m = mn;
+          }
+          asm volatile("bar.sync 1, 128;" ::: "memory");
+#pragma unroll
+          for (int n = 0; n < NC; ++n)
+#pragma unroll
+            for (int c = 0; c < C; ++c) l[n][c] *= s_alpha[buf * N + n * W + half * C + c];
         }
-        asm volatile("bar.sync 1, 128;" ::: "memory");
         uint8_t* row = sP + buf * kPTile + key * 128;
 #pragma unroll
         for (int n = 0; n < NC; ++n) {
@@ -479,14 +529,10 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
 #pragma unroll
             for (int e = 0; e < 8; e += 4) {
               const float4 mm = *reinterpret_cast<const float4*>(s_m + col0 + c + e);
-              const float4 al = *reinterpret_cast<const float4*>(s_alpha + buf * N + col0 + c + e);
               float* xs = &x[n][c + e];
               float* ls = &l[n][c + e];
               const float pr[4] = {ex2(xs[0] - mm.x), ex2(xs[1] - mm.y), ex2(xs[2] - mm.z), ex2(xs[3] - mm.w)};
-              ls[0] = fmaf(ls[0], al.x, pr[0]);
-              ls[1] = fmaf(ls[1], al.y, pr[1]);
-              ls[2] = fmaf(ls[2], al.z, pr[2]);
-              ls[3] = fmaf(ls[3], al.w, pr[3]);
+              ls[0] += pr[0]; ls[1] += pr[1]; ls[2] += pr[2]; ls[3] += pr[3];
               const __nv_bfloat162 lo = __floats2bfloat162_rn(pr[0], pr[1]), hi = __floats2bfloat162_rn(pr[2], pr[3]);
               packed[e / 2] = *reinterpret_cast<const uint32_t*>(&lo);
               packed[e / 2 + 1] = *reinterpret_cast<const uint32_t*>(&hi);
@@ -546,6 +592,7 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
         const int buf = j & 1;
         wait(&o_full[buf], (j >> 1) & 1, kErrEpilogueWait);
         tc_fence_after();
+        const bool rescale = s_rescale[buf] != 0;
 #pragma unroll
         for (int x = 0; x < NB; ++x) {
           const int b = group + OG * x;
@@ -554,14 +601,15 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
           for (int c0 = 0; c0 < N; c0 += W) {
             float v[W];
             tmem_load<W>(addr + (buf * blocks + b) * N + c0, v);
+            if (rescale) {
 #pragma unroll
-            for (int c = 0; c < W; c += 4) {
-              const float4 al = *reinterpret_cast<const float4*>(s_alpha + buf * N + c0 + c);
-              o[x][c0 + c] = fmaf(o[x][c0 + c], al.x, v[c]);
-              o[x][c0 + c + 1] = fmaf(o[x][c0 + c + 1], al.y, v[c + 1]);
-              o[x][c0 + c + 2] = fmaf(o[x][c0 + c + 2], al.z, v[c + 2]);
-              o[x][c0 + c + 3] = fmaf(o[x][c0 + c + 3], al.w, v[c + 3]);
+              for (int c = 0; c < W; c += 4) {
+                const float4 al = *reinterpret_cast<const float4*>(s_alpha + buf * N + c0 + c);
+                o[x][c0 + c] *= al.x; o[x][c0 + c + 1] *= al.y; o[x][c0 + c + 2] *= al.z; o[x][c0 + c + 3] *= al.w;
+              }
             }
+#pragma unroll
+            for (int c = 0; c < W; ++c) o[x][c0 + c] += v[c];
           }
         }
         tc_fence_before();
@@ -572,13 +620,22 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
       float* part = p.part_o + static_cast<size_t>(2 * blockIdx.x + max(w.part, 0)) * N * p.out_cols;
 #pragma unroll
       for (int x = 0; x < NB; ++x) {
-        const int col = (group + OG * x) * 128 + quarter * 32 + lane;
-        if (col >= p.out_cols) continue;
+        const int col0 = (group + OG * x) * 128 + quarter * 32;
+        if (col0 >= p.out_cols) continue;                  // warp-uniform: a multiple of 64 columns
+        if (w.part < 0) {
+          // neighbouring lanes swap columns of two rows: an even lane stores the first row's pair, an odd one the second's
+          __nv_bfloat162* dst = reinterpret_cast<__nv_bfloat162*>(p.out + static_cast<size_t>(w.q_row + (lane & 1)) * p.out_cols + col0 + (lane & ~1));
 #pragma unroll
-        for (int c = 0; c < N; ++c) {
-          if (c >= w.rows) break;
-          if (w.part < 0) p.out[static_cast<size_t>(w.q_row + c) * p.out_cols + col] = __float2bfloat16(o[x][c] * s_l[c]);
-          else part[static_cast<size_t>(c) * p.out_cols + col] = o[x][c];
+          for (int c = 0; c < N; c += 2) {
+            const float a = o[x][c] * s_l[c], b = o[x][c + 1] * s_l[c + 1];
+            const float got = __shfl_xor_sync(0xffffffffu, lane & 1 ? a : b, 1);
+            if (c + (lane & 1) < w.rows) dst[static_cast<size_t>(c) * p.out_cols / 2] = lane & 1 ? __floats2bfloat162_rn(got, b) : __floats2bfloat162_rn(a, got);
+          }
+        } else {
+          float* dst = part + col0 + lane;
+#pragma unroll
+          for (int c = 0; c < N; ++c)
+            if (c < w.rows) dst[static_cast<size_t>(c) * p.out_cols] = o[x][c];
         }
       }
       __syncwarp();
@@ -615,7 +672,6 @@ latent_merge_kernel(const LatentParams p) {
   if (lane == 0) red[warp] = mm;
   __syncthreads();
   mm = fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3]));
-  if (mm == -INFINITY) mm = 0.f;
   float sum = 0.f;
   constexpr int kCols = 4;                                 // columns per thread: out_cols <= 512
   float o[kCols] = {};
