@@ -154,8 +154,52 @@ def _gisilix_config(d: Dict[str, Any]) -> Dict[str, Any]:
     return out
 
 
+def _sobivik_config(d: Dict[str, Any]) -> Dict[str, Any]:
+    """Sobivik checkpoints: layers described one by one as in Fuzuvik's; retention, latent attention with a latent for the
+    queries too, differential attention; norms of one number around both halves of a layer, a convolution on what a mixer
+    reads, and a weighted sum over the results of all layers so far."""
+    out = dict(d)
+    layers = d["layers"]
+    taps = int((d.get("canon") or {}).get("taps") or 0)
+    specs = []
+    for i, layer in enumerate(layers):
+        m, mlp = layer["mixer"], layer.get("mlp")
+        if mlp is not None and mlp["kind"] != "dense":
+            raise NotImplementedError(f"layer {i}: feed-forward kind {mlp['kind']!r}")
+        mask = m.get("mask") or {}
+        sizes = dict(heads=int(m["heads"]), kv_heads=int(m.get("kv_heads") or m["heads"]), dim=int(m["dim"]),
+                     vdim=int(m["vdim"]), ff=0 if mlp is None else int(mlp["ff"]), input_conv=taps)
+        if layer["type"] == "retention":
+            specs.append(MixerSpec("decay", **sizes, decay=tuple(float(x) for x in m["decay"]), qkv_act="",
+                                   k_scale=float(m["dim"]) ** -0.5, head_norm=True, gate_act="silu"))
+        elif layer["type"] == "latent_attention":
+            rot = m["rot"]
+            sc = rot.get("scaling")
+            if int(rot["dims"]) != int(m["rot_dim"]):
+                raise NotImplementedError(f"layer {i}: {rot['dims']} of {m['rot_dim']} key dimensions rotated")
+            specs.append(MixerSpec(
+                "latent", **{**sizes, "kv_heads": 1}, scale=float(m["scale"]), window=int(mask.get("size") or 0),
+                kv_rank=int(m["kv_rank"]), q_rank=int(m["q_rank"]), rot_dims=int(m["rot_dim"]), rot_base=float(rot["base"]),
+                rot_yarn=None if not sc else tuple(float(sc[k]) for k in ("factor", "fast", "slow", "original")),
+                learned_sink=True, out_gate="element"))
+        elif layer["type"] == "attention":
+            specs.append(MixerSpec(
+                "attention", **sizes, scale=float(m["scale"]), window=int(mask.get("size") or 0),
+                keep_first=int(mask.get("keep_first") or 0), diff=float(m["diff"]), out_gate="head"))
+        else:
+            raise NotImplementedError(f"layer {i}: mixer {layer['type']!r}")
+    out.update(model_type="sobivik", hidden_size=int(d["width"]), vocab_size=int(d["vocab"]), num_hidden_layers=len(layers),
+               num_attention_heads=max(s.heads for s in specs), rms_norm_eps=float(d["norm"]["eps"]),
+               embedding_multiplier=float((d.get("embedding") or {}).get("scale", 1.0)),
+               logit_scale=float(d.get("logit_scale", 1.0)), mixers=specs,
+               # rotary positions are unbounded by design: the table length is a deployment choice
+               max_position_embeddings=int(d.get("max_position_embeddings") or 131072))
+    return out
+
+
 # ``architecture`` of a config.json without ``model_type`` -> function that brings it to the common names
-CONFIG_READERS = {"Fuzuvik": _fuzuvik_config, "Kipedra": _kipedra_config, "Gisilix": _gisilix_config}
+CONFIG_READERS = {"Fuzuvik": _fuzuvik_config, "Kipedra": _kipedra_config, "Gisilix": _gisilix_config,
+                  "Sobivik": _sobivik_config}
 
 
 class ModelConfig:
@@ -228,9 +272,11 @@ class MixerSpec:
     ff: int = 0                              # width of a dense feed-forward, 0: the layer has none
     moe: Optional[ExpertSpec] = None         # routed experts in its place
     short_conv: bool = False                 # causal convolution over time on every channel of q, k and v
+    input_conv: int = 0                      # taps of a causal convolution over time added to what the mixer reads
     # attention, latent
     scale: float = 1.0
     window: int = 0                          # > 0: the token itself and the window - 1 tokens before it
+    keep_first: int = 0                      # first tokens of a sequence that stay visible past the window
     chunk: int = 0                           # > 0: keys of the query's own chunk of this many positions
     sink: bool = False                       # one more key of score 0, without a value, in the softmax
     learned_sink: bool = False               # the same with a stored score per head
@@ -240,7 +286,10 @@ class MixerSpec:
     q_temp: Optional[Tuple[float, int]] = None    # (coef, every): q times 1 + coef * ln(floor((p + 1) / every) + 1)
     out_gate: str = ""                       # output times the sigmoid of a projection: "element" | "head" (one per head)
     kv_from: Optional[int] = None            # layer whose keys and values this one reads
+    diff: Optional[float] = None             # two maps per head over the same values: the first minus lambda times the
+                                             # second, normed per head, times 1 - diff (lambda: learned part + diff)
     kv_rank: int = 0                         # latent: its size
+    q_rank: int = 0                          # latent: > 0: queries come from a normed latent of this size
     v_mix: bool = False                      # values mixed with those of the first such layer
     rot_dims: int = 0
     rot_base: float = 10000.0
@@ -254,6 +303,9 @@ class MixerSpec:
     gate_act: str = "sigmoid"                # of the output gate
     # decay
     decay: Tuple[float, ...] = ()
+    qkv_act: str = "silu"                    # of q, k and v, "": none
+    k_scale: float = 1.0                     # factor of k
+    head_norm: bool = False                  # weightless norm per head (False: one weighted norm over all heads)
 
     @property
     def paged(self) -> bool:
@@ -263,7 +315,7 @@ class MixerSpec:
     @property
     def recurrent(self) -> bool:
         """Keeps a state per sequence that every token advances."""
-        return not self.paged or self.short_conv
+        return not self.paged or self.short_conv or self.input_conv > 0
 
     @property
     def feed_forward(self) -> bool:
@@ -328,6 +380,8 @@ class Arch:
     moe_correction: Optional[str] = None     # correction of the choice scores, or bias of the logits (layers with an `ExpertSpec`)
     # ---- layers that differ (config "mixers") ---------------------------------------------------
     mix: Optional[str] = None                # tensor prefix of a layer's mixer
+    input_conv: Optional[str] = None         # layers with `MixerSpec.input_conv`: its tensor
+    depth_average: Optional[str] = None      # weights of the embedding output and of all layers' results so far, whose sum goes on
     residual_fp32: bool = False              # the residual stream is kept in 32 bits
     bare_names: bool = False                 # tensors are named without the ".weight" suffix, biases end in ".b"
 
@@ -424,6 +478,9 @@ ARCHS["gisilix"] = Arch(embed="embed", layer="l{i}", norm1="norm1", norm2="norm2
                         mix="mix", gate="mlp.gate", up="mlp.up", down="mlp.down", act="silu", rope=False, norm="layer",
                         residual_fp32=True, bare_names=True, moe_router="mlp.router", moe_expert="mlp.e{e}", moe_gate="gate",
                         moe_up="up", moe_down="down", moe_correction="mlp.router.b", moe_shared="mlp.shared")
+ARCHS["sobivik"] = Arch(embed="embed", layer="l{i}", norm1="norm1", norm2="norm2", post_attn_norm="norm1b", post_mlp_norm="norm2b",
+                        final_norm="final.norm", lm_head="head", mix="mix", input_conv="canon1", depth_average="dwa",
+                        gate="mlp.gate", up="mlp.up", down="mlp.down", act="silu", rope=False, residual_fp32=True, bare_names=True)
 ARCHS["gemma3"] = ARCHS["gemma3_text"]
 ARCHS["phi-msft"] = ARCHS["phi"]
 ARCHS["qwen2_vl_text"] = ARCHS["qwen2_5_vl_text"] = ARCHS["qwen2"]   # language models of Qwen2-VL / Qwen2.5-VL

@@ -55,7 +55,19 @@ class ForwardMeta:
     state_slots: Optional[torch.Tensor] = None       # [B] slot of every sequence in the recurrent state pools, -1: none
     v_first: Optional[torch.Tensor] = None           # [T, *] values later layers mix in (set by the first layer that mixes)
     expansions: Optional[dict] = None                # window -> mixers.Expansion of layers with latent attention
+    streams: Optional[torch.Tensor] = None           # [layers + 1, T, H] embedding output and results of the layers (fp32)
     cross: Optional[object] = None                   # rows and image states for cross-attention layers (models/mllama.py)
+
+
+@dataclass
+class Pending:
+    """A block's output on its way into an fp32 stream: normed by `post` before it is added.  After a layer's last block
+    the stream may go on as a weighted sum of the embedding output and the results of the layers so far (`average`: weights,
+    fp32, one per result)."""
+
+    out: torch.Tensor
+    post: Optional["Norm"] = None
+    average: Optional[torch.Tensor] = None
 
 
 class Norm:
@@ -64,16 +76,26 @@ class Norm:
         self.kind, self.weight, self.bias, self.eps, self.unit_offset = kind, weight, bias, eps, unit_offset
         self.residual_fp32 = residual_fp32
         self.residual_scale = residual_scale     # fp32 streams: what a block's output is multiplied by when it is added
+        self.gain = 1.0                          # fp32 streams: factor of the normed rows
 
     @classmethod
-    def load(cls, arch: Arch, prefix: str, weights, eps: float, residual_scale: float = 1.0):
+    def load(cls, arch: Arch, prefix: str, weights, eps: float, residual_scale: float = 1.0, width: Optional[int] = None):
         w = weights.get_tensor(f"{prefix}.weight")
+        if w.dim() == 0:                         # one number for all `width` coordinates
+            w = w.expand(width).contiguous()
         b = None
         if arch.norm == "layer" and arch.norm_bias and weights.has_tensor(f"{prefix}.bias"):
             b = weights.get_tensor(f"{prefix}.bias")
         return cls(arch.norm, w, b, eps, arch.norm_unit_offset, arch.residual_fp32, residual_scale)
 
-    def __call__(self, x, residual=None, rows=None):
+    def __call__(self, x, residual=None, rows=None, conv=None, streams=None):
+        if self.residual_fp32 and (isinstance(x, Pending) or conv is not None or self.gain != 1.0):
+            # `conv`: an `ops.ShortConv` that what comes out is convolved by; `streams`: `ForwardMeta.streams`
+            if self.kind != "rms" or self.unit_offset or self.residual_scale != 1.0:
+                raise NotImplementedError("block output norms and input convolutions go with plain RMS norms")
+            p = x if isinstance(x, Pending) else Pending(x)
+            return ops.stream_step(p.out, None if p.post is None else p.post.weight, residual, self.weight, self.eps, rows,
+                                   keep=rows is None, gain=self.gain, average=p.average, streams=streams, conv=conv)
         if self.residual_fp32:
             # `x` is the last block's output, a pair of outputs or None (nothing to add); `rows` ends the stream: only
             # these rows are normed
@@ -485,20 +507,27 @@ class DecoderLayer:
         spec = dims.mixers[idx] if dims.mixers else None
         if spec is not None:
             rs = dims.residual_scale
-            self.norm1 = Norm.load(arch, f"{prefix}.{arch.norm1}", weights, dims.eps, rs)
-            self.norm2 = Norm.load(arch, f"{prefix}.{arch.norm2}", weights, dims.eps, rs) if spec.feed_forward else None
+            self.norm1 = Norm.load(arch, f"{prefix}.{arch.norm1}", weights, dims.eps, rs, dims.hidden)
+            self.norm2 = Norm.load(arch, f"{prefix}.{arch.norm2}", weights, dims.eps, rs, dims.hidden) if spec.feed_forward else None
         elif cfg.model_type in ("falcon", "RefinedWeb", "RefinedWebModel"):
             # the new decoder architecture names its norms ln_attn / ln_mlp and has no input_layernorm
             self.norm1, self.norm2 = self._falcon_norms(arch, cfg, prefix, weights, dims)
         else:
             self.norm1 = Norm.load(arch, f"{prefix}.{arch.norm1}", weights, dims.eps)
             self.norm2 = Norm.load(arch, f"{prefix}.{arch.norm2}", weights, dims.eps) if arch.norm2 else None
-        self.post_attn = Norm.load(arch, f"{prefix}.{arch.post_attn_norm}", weights, dims.eps) if arch.post_attn_norm else None
-        self.post_mlp = Norm.load(arch, f"{prefix}.{arch.post_mlp_norm}", weights, dims.eps) if arch.post_mlp_norm else None
+        post = lambda name: Norm.load(arch, f"{prefix}.{name}", weights, dims.eps, width=dims.hidden)
+        self.post_attn = post(arch.post_attn_norm) if arch.post_attn_norm else None
+        self.post_mlp = post(arch.post_mlp_norm) if arch.post_mlp_norm and (spec is None or spec.feed_forward) else None
+        self.average = None
+        if arch.depth_average:
+            self.average = weights.get_tensor(f"{prefix}.{arch.depth_average}", to_dtype=False).float().contiguous()
+            if self.average.numel() != idx + 2:
+                raise ValueError(f"{prefix}.{arch.depth_average}: {self.average.numel()} weights for {idx + 2} results")
         if spec is not None:
             from .mixers import load_mixer
 
-            self.attn = load_mixer(spec, f"{prefix}.{arch.mix}", weights, idx, dims.eps, comm, rotary_tables)
+            self.attn = load_mixer(spec, f"{prefix}.{arch.mix}", weights, idx, dims.eps, comm, rotary_tables,
+                                   f"{prefix}.{arch.input_conv}" if arch.input_conv else None)
             is_moe = spec.moe is not None
         elif arch.mla:
             from .deepseek import MLAAttention, is_moe_layer
@@ -536,6 +565,8 @@ class DecoderLayer:
         rs = 1.0 if a.residual_fp32 else self.dims.residual_scale
         if a.parallel_residual and a.residual_fp32:
             return self._side_by_side(h, residual, meta, rotary, kv)
+        if a.residual_fp32 and (a.post_attn_norm or a.depth_average):
+            return self._normed_both_ways(h, residual, meta, rotary, kv)
         if a.parallel_residual:
             normed, residual = self.norm1(h, residual)
             # attention and MLP partial sums of a parallel block share one reduction
@@ -581,6 +612,18 @@ class DecoderLayer:
             return self.attn(normed, None, meta, rotary, kv), residual
         normed, mlp_in, residual = self.norm1.with_second(self.norm2, h, residual)
         return (self.attn(normed, None, meta, rotary, kv), self.mlp(mlp_in, meta=meta)), residual
+
+    def _normed_both_ways(self, h, residual, meta: ForwardMeta, rotary, kv):
+        """fp32 stream whose blocks have a norm in front and one behind, which the next norm applies when it adds the output."""
+        conv = self.attn.input_conv
+        if conv is not None:
+            conv, kv = conv.at(meta, kv[-1]), kv[:-1]
+        normed, residual = self.norm1(h, residual, conv=conv, streams=meta.streams)
+        out, post = self.attn(normed, None, meta, rotary, kv), self.post_attn
+        if self.mlp is not None:
+            normed, residual = self.norm2(Pending(out, post), residual)
+            out, post = self.mlp(normed, meta=meta), self.post_mlp
+        return Pending(out, post, self.average), residual
 
     @property
     def fusable_tp(self) -> bool:
@@ -662,7 +705,11 @@ class CausalDecoder:
                 self.layers.append(DecoderLayer(a, cfg, dims, px + a.layer.format(i=i), weights, i, comm, rotary_tables))
         # layers in the order a step runs them, with a cache each: a layer may run several times
         self.layer_runs = self.layers if dims.layer_order is None else [self.layers[i] for i in dims.layer_order]
-        self.final_norm = Norm.load(a, px + a.final_norm, weights, dims.eps, dims.residual_scale if dims.mixers else 1.0)
+        self.final_norm = Norm.load(a, px + a.final_norm, weights, dims.eps, dims.residual_scale if dims.mixers else 1.0, dims.hidden)
+        if a.residual_fp32 and dims.logit_scale != 1.0:       # in front of the head, where rows are fp32
+            self.final_norm.gain, dims.logit_scale = dims.logit_scale, 1.0
+        if a.depth_average and dims.layer_order is not None:
+            raise NotImplementedError("weighted sums over the layers' results where layers run several times")
         head_name = px + a.lm_head if not a.lm_head.startswith("lm_head") or not prefix else a.lm_head
         candidates = [head_name, px + a.lm_head, a.lm_head, px + a.embed]
         if cfg.get("tie_word_embeddings") and not any(weights.has_tensor(f"{c}.weight") for c in candidates[:3]):
@@ -750,12 +797,16 @@ class CausalDecoder:
     def _forward_hidden_fp32_stream(self, meta: ForwardMeta, kv_cache) -> torch.Tensor:
         """Layers around an fp32 residual stream; the final norm runs on the rows that need logits only."""
         meta.v_first = None
-        residual = ops.embed_residual(meta.input_ids, self.embed.weight, self.dims.embed_scale)
+        residual = ops.embed_residual(meta.input_ids, self.embed.weight, self.dims.embed_scale,
+                                      len(self.layers) + 1 if self.arch.depth_average else 1)
+        if self.arch.depth_average:
+            meta.streams, residual = residual, residual[0]
         h = None
         for layer, cache in zip(self.layer_runs, kv_cache):
             h, residual = layer(h, residual, meta, None, cache)
-        meta.v_first = None
-        return self.final_norm(h, residual, rows=meta.lm_head_indices)[0]
+        out = self.final_norm(h, residual, rows=meta.lm_head_indices, streams=meta.streams)[0]
+        meta.v_first = meta.streams = None
+        return out
 
     def forward_hidden(self, meta: ForwardMeta, kv_cache) -> torch.Tensor:
         """Normalised hidden rows: of every token, or with an fp32 residual stream of ``meta.lm_head_indices`` only."""

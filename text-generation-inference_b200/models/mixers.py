@@ -5,15 +5,18 @@ cache (``cache_tensors``) and runs as a short sequence of fused ops:
 
     attention   qkv GEMM -> [short convolutions +] rotate + unit RMS + value mixing + page store -> paged attention
                 -> o GEMM; or qkvg GEMM -> RMS of whole rows + temperature + page store -> paged attention -> output gate
-                -> o GEMM
-    latent      GEMM for q, latent and gate -> RMS of the latent, rotations, page store -> queries times the key
+                -> o GEMM; or, with two maps per head, qkvg GEMM -> page store -> paged attention -> difference of the maps
+                + norm + gate -> o GEMM
+    latent      GEMM for q, latent and gate (or for the queries' latent, then one for q) -> RMS of the latent, rotations,
+                page store -> queries times the key
                 up-projection -> attention over the latents (all heads read one row per token), gate -> value
                 up-projection -> o GEMM; for sequences that bring many tokens -> keys and values of the visible tokens
                 written out by one GEMM -> attention per head, gate -> o GEMM
     delta       one GEMM for q, k, v, write strengths and decay / gate inputs (-> low-rank decay / gate GEMMs)
                 -> short convolutions + unit norms + decays -> state scan -> norm x gate -> o GEMM
-    decay       one GEMM for q, k, v, gate -> state scan (SiLU applied on the way in) -> norm x gate -> o GEMM
+    decay       one GEMM for q, k, v, gate -> state scan (SiLU applied on the way in, if any) -> norm x gate -> o GEMM
 
+What a mixer reads may be convolved over time first (``InputConv``, part of the layer).
 Recurrent layers keep, per slot of the state pool, the matrix state of every head (fp32, ``[H, vdim, pitch]``); layers
 with short convolutions, attention layers included, the last ``taps - 1`` inputs of every channel.  Which tokens a
 sequence brings and from which slot it continues is in the step's metadata, so prompts, portions of prompts and decoded
@@ -21,6 +24,7 @@ tokens are one code path.
 """
 from __future__ import annotations
 
+import math
 import os
 from dataclasses import dataclass
 from typing import Dict, List, Optional, Sequence, Tuple
@@ -121,6 +125,8 @@ class Mixer:
     def row(self, w: torch.Tensor) -> TensorParallelRowLinear:
         return TensorParallelRowLinear(FastLinear(w), self.pg, self.comm)
 
+    input_conv: Optional["InputConv"] = None        # of the layer, which applies it; its state is kept with the mixer's
+
     def page_tensors(self, num_blocks: int, block_size: int, device) -> Tuple[torch.Tensor, ...]:
         return ()
 
@@ -129,27 +135,56 @@ class Mixer:
 
     def cache_tensors(self, num_blocks: int, block_size: int, slots: int, device) -> Tuple[torch.Tensor, ...]:
         """What the mixer keeps between steps: pages (addressed by token), then states (addressed by request)."""
-        return self.page_tensors(num_blocks, block_size, device) + self.state_tensors(slots, device)
+        return self.page_tensors(num_blocks, block_size, device) + self.slot_tensors(slots, device)
+
+    def slot_tensors(self, slots: int, device) -> Tuple[torch.Tensor, ...]:
+        """The mixer's states and, last, that of the input convolution."""
+        conv = () if self.input_conv is None else (self.input_conv.state(slots, device),)
+        return self.state_tensors(slots, device) + conv
 
     def state_bytes(self) -> int:
         """Bytes of one slot of the state pool."""
-        return sum(t.numel() * t.element_size() for t in self.state_tensors(1, "meta"))
+        return sum(t.numel() * t.element_size() for t in self.slot_tensors(1, "meta"))
 
     def page_bytes(self, block_size: int) -> int:
         return sum(t.numel() * t.element_size() for t in self.page_tensors(1, block_size, "meta"))
+
+
+class InputConv:
+    """``h + conv(h)``: a causal convolution over time on every channel of what a mixer reads."""
+
+    def __init__(self, weight: torch.Tensor, dtype, device):
+        self.channels, self.taps = weight.shape
+        w = weight.float().t().contiguous().to(device)        # [taps, channels], oldest input first
+        w[-1] += 1                                             # the input itself
+        self.weight, self.dtype = w, dtype
+
+    def state(self, slots: int, device) -> torch.Tensor:
+        return torch.zeros(slots, self.taps - 1, self.channels, dtype=self.dtype, device=device)
+
+    def at(self, meta, state: torch.Tensor) -> "ops.ShortConv":
+        return ops.ShortConv(self.weight, state, meta.cu_seqlens_q, meta.kv_lens, meta.state_slots, meta.max_q == 1)
 
 
 class MixedAttention(Mixer):
     """Paged attention with its own head sizes: short convolutions of q, k and v, rotation of the first dimensions,
     weightless RMS of q and k after it, values mixed with an earlier layer's, keys limited to the query's chunk or window,
     a sink in the softmax.  Or, without any of the first four: weighted RMS of q and k over all heads, queries times a factor
-    of their position, keys and values of an earlier layer.  Capped scores and an output gate go with either."""
+    of their position, keys and values of an earlier layer.  Capped scores and an output gate go with either.  Or, without
+    any of these but the gate: two maps per head over the same values, and their normed difference.  Both maps of a key lie
+    side by side in one page row, and a query map is a query of its own with zeros at the other map's place."""
 
     def __init__(self, spec, prefix, weights, idx, eps, comm=None, rotary: Optional[RotaryTables] = None):
         super().__init__(spec, prefix, weights, idx, eps, comm)
         s = spec
         if s.row_norm and (s.short_conv or s.rot_dims or s.qk_unit_rms or s.v_mix):
             raise NotImplementedError(f"{prefix}: a norm over whole rows beside convolutions, rotation, unit norms or value mixing")
+        self.maps = 1 if s.diff is None else 2
+        if s.diff is not None and (s.row_norm or s.short_conv or s.rot_dims or s.qk_unit_rms or s.v_mix or s.softcap or s.sink
+                                   or s.learned_sink or s.kv_from is not None or s.out_gate not in ("", "head")):
+            raise NotImplementedError(f"{prefix}: differences of two maps beside norms, rotation, sinks or shared keys")
+        if s.diff is None and s.out_gate not in ("", "element"):
+            raise NotImplementedError(f"{prefix}: output gate {s.out_gate!r} on attention of one map")
         own = ["q", "k", "v"] if s.kv_from is None else ["q"]
         self.qkv, offs = self.fused(own + (["g"] if s.out_gate else []), bias=s.qkv_bias)
         self.offs, self.off_gate = offs[:len(own)], offs[-1]
@@ -159,9 +194,12 @@ class MixedAttention(Mixer):
         if s.short_conv:
             self.load_conv()
         self.v_lambda = float(self.f32("vmix").reshape(-1)[0]) if s.v_mix and weights.has_tensor(f"{prefix}.vmix") else 0.0
-        self.kd, self.vd = ops.attention_pitch(s.dim, s.vdim, self.dtype, self.device)
-        # a gate packs the heads again
-        self.o = self.row(_column_input(self.tensor("o")) if s.out_gate else
+        if s.diff is not None:
+            part = lambda i: math.exp(float((self.f32(f"lq{i}").double() * self.f32(f"lk{i}").double()).sum()))
+            self.map_lambda = part(1) - part(2) + s.diff
+        self.kd, self.vd = ops.attention_pitch(self.maps * s.dim, s.vdim, self.dtype, self.device)
+        # a gate (or the difference of maps) packs the heads again
+        self.o = self.row(_column_input(self.tensor("o")) if s.out_gate or s.diff is not None else
                           spread_columns(self.tensor("o"), s.heads, s.vdim, self.vd))
         self.rotary = rotary.get(s)
 
@@ -182,12 +220,17 @@ class MixedAttention(Mixer):
         if s.row_norm:
             q = ops.row_norm_store(proj, self.offs, meta.positions, meta.slots, k_cache, v_cache, self.q_norm, self.k_norm, self.eps,
                                    s.heads, s.kv_heads, s.dim, s.vdim, self.kd, s.q_temp)
+        elif s.diff is not None:
+            q = ops.map_store(proj, self.offs, meta.slots, k_cache, v_cache, s.heads, s.kv_heads, s.dim, s.vdim)
         else:
             q = self._rotated(proj, meta, kv)
         a = ops.paged_attention(q, k_cache, v_cache, meta.block_tables, meta.cu_seqlens_q, meta.kv_lens, s.scale,
                                 window=s.window or -1, softcap=s.softcap, max_q=meta.max_q, max_kv=meta.max_kv, chunk=s.chunk,
-                                sink=self.sink)
-        if s.out_gate:
+                                sink=self.sink, keep=s.keep_first)
+        if s.diff is not None:
+            gate = proj[:, self.off_gate:self.off_gate + s.heads] if s.out_gate else None
+            a = ops.map_difference(a, gate, self.map_lambda, 1.0 - s.diff, self.eps, s.vdim)
+        elif s.out_gate:
             a = ops.output_gate(a, proj[:, self.off_gate:self.off_gate + s.heads * s.vdim], s.vdim)
         return self.o(a.view(a.shape[0], -1), reduce=reduce, out=out)
 
@@ -268,10 +311,17 @@ class LatentAttention(Mixer):
     def __init__(self, spec, prefix, weights, idx, eps, comm=None, rotary: Optional[RotaryTables] = None):
         super().__init__(spec, prefix, weights, idx, eps, comm)
         s = spec
-        if s.out_gate not in ("", "head"):
-            raise NotImplementedError(f"{prefix}: output gate {s.out_gate!r} on latent attention")
-        self.proj, self.offs = self.fused(["q", "dkv"] + (["g"] if s.out_gate else []))
+        # rotations pair neighbours: with halves for pairs, the rows of the projections are brought to that order
+        self.order = None if s.rot_interleaved or not s.rot_dims else torch.arange(s.rot_dims).view(2, -1).t().reshape(-1)
+        names = ["dq" if s.q_rank else "q", "dkv"] + (["g"] if s.out_gate else [])
+        w, self.offs = stack_rows([self._rows(n) for n in names])
+        self.proj = TensorParallelColumnLinear(FastLinear(w))
         self.norm = self.f32("dkv.norm")
+        if s.q_rank:
+            self.q_norm = self.f32("dq.norm")
+            self.uq = TensorParallelColumnLinear(FastLinear(stack_rows([self._rows("uq")])[0]))
+            self.q_cols = _up(s.q_rank)
+        self.sink = self.f32("sink") if s.learned_sink else None
         self.off_rot, self.width = ops.latent_layout(s.kv_rank, s.rot_dims, self.dtype, self.device)
         pad = (0, self.off_rot - s.kv_rank)
         self.uk, self.uv = (torch.nn.functional.pad(self.tensor(n).view(s.heads, d, s.kv_rank), pad).contiguous()
@@ -287,6 +337,15 @@ class LatentAttention(Mixer):
         self.o = self.row(_column_input(self.tensor("o")))
         self.rotary = rotary.get(s)
 
+    def _rows(self, name: str) -> torch.Tensor:
+        s, w = self.spec, self.tensor(name)
+        if self.order is not None and name == "dkv":
+            w = torch.cat([w[:s.kv_rank], w[s.kv_rank:][self.order.to(w.device)]])
+        elif self.order is not None and name in ("q", "uq"):
+            rows = torch.cat([torch.arange(s.dim), s.dim + self.order]).to(w.device)
+            w = w.view(s.heads, s.dim + s.rot_dims, -1)[:, rows].reshape(w.shape)
+        return w
+
     def page_tensors(self, num_blocks: int, block_size: int, device):
         # zeros: the kernels never write the padding columns
         return (torch.zeros(num_blocks, block_size, 1, self.width, dtype=self.dtype, device=device),)
@@ -299,23 +358,36 @@ class LatentAttention(Mixer):
         rest = plan is None or not plan.all
         q = proj.new_empty(T, s.heads, self.width) if rest else None
         q_full = None if plan is None else proj.new_empty(T, s.heads, self.full[0])
-        ops.latent_store(proj, self.offs[1], self.norm, self.eps, meta.positions, self.rotary.cos_sin, meta.slots, pages, q,
-                         self.off_rot, s.kv_rank, s.rot_dims, s.heads, s.dim, q_full)
-        gate = proj[:, self.offs[2]:self.offs[2] + s.heads] if s.out_gate else None
+        places = (self.off_rot, s.kv_rank, s.rot_dims, s.heads, s.dim)
+        turns = (meta.positions, self.rotary.cos_sin, meta.slots)
+        if s.q_rank:
+            cq = proj.new_empty(T, self.q_cols)
+            ops.latent_store(proj, self.offs[1], self.norm, self.eps, *turns, pages, None, *places, queries=False,
+                             q_latent=(self.offs[0], self.q_norm, cq))
+            queries = self.uq(cq)
+            ops.latent_store(queries, 0, None, self.eps, *turns, None, q, *places, q_full, width=self.width)
+        else:
+            queries = proj
+            ops.latent_store(proj, self.offs[1], self.norm, self.eps, *turns, pages, q, *places, q_full)
+        gate = proj[:, self.offs[2]:self.offs[2] + s.heads] if s.out_gate == "head" else None
         y = proj.new_empty(T, s.heads, s.vdim)
         if rest:
-            plain = proj[:, :s.heads * (s.dim + s.rot_dims)].view(T, s.heads, -1)[..., :s.dim]
+            plain = queries[:, :s.heads * (s.dim + s.rot_dims)].unflatten(1, (s.heads, -1))[..., :s.dim]
             torch.bmm(plain.transpose(0, 1), self.uk, out=q[..., :self.off_rot].transpose(0, 1))
             a = ops.latent_attention(q, pages, s.kv_rank, meta.block_tables, meta.cu_seqlens_q, meta.kv_lens, s.scale,
                                      s.window or -1, meta.max_q if plan is None else plan.rest_max_q, meta.max_kv, gate,
-                                     None if plan is None else plan.kv_lens)
+                                     None if plan is None else plan.kv_lens, self.sink)
             torch.bmm(a.transpose(0, 1), self.uv[..., :a.shape[2]].transpose(1, 2), out=y.transpose(0, 1))
         if plan is not None:
             written = ops.linear_shallow(pages.view(-1, self.width).index_select(0, plan.rows), self.expand)
             o = y if s.vdim == self.full[1] else proj.new_empty(T, s.heads, self.full[1])
-            ops.expanded_attention(q_full, written, plan, meta.cu_seqlens_q, s.scale, s.window or -1, meta.max_q, gate, o)
-            if o is not y:
+            ops.expanded_attention(q_full, written, plan, meta.cu_seqlens_q, s.scale, s.window or -1, meta.max_q, gate, o, self.sink)
+            if o is not y and plan.all and s.out_gate == "element":
+                y = o                    # the gate packs the heads
+            elif o is not y:
                 y.index_copy_(0, plan.queries.long(), o.index_select(0, plan.queries)[..., :s.vdim])
+        if s.out_gate == "element":
+            y = ops.output_gate(y, proj[:, self.offs[2]:self.offs[2] + s.heads * s.vdim], s.vdim)
         return self.o(y.view(T, -1), reduce=reduce, out=out)
 
 
@@ -369,7 +441,8 @@ class DecayAttention(Mixer):
             raise ValueError(f"{prefix}: {len(s.decay)} decays for {s.heads} heads")
         self.proj, self.offs = self.fused(["q", "k", "v", "g"])
         self.decay = torch.tensor(s.decay, dtype=torch.float32, device=self.device)
-        self.norm = self.f32("norm")
+        self.groups = s.heads if s.head_norm else 1
+        self.norm = torch.ones(s.vdim, dtype=torch.float32, device=self.device) if s.head_norm else self.f32("norm")
         self.pitch = ops.recurrent_pitch(s.dim, self.device)
         self.o = self.row(_column_input(self.tensor("o")))
         self.out_cols = self.o.linear.weight.shape[1]
@@ -382,13 +455,21 @@ class DecayAttention(Mixer):
         s = self.spec
         p = self.proj(x)
         o = ops.decay_scan(p, self.offs, self.decay, meta.cu_seqlens_q, meta.kv_lens, meta.state_slots, kv[0], s.heads, s.dim,
-                           s.vdim, meta.max_q)
-        y = ops.gated_norm(o, p[:, self.offs[3]:], self.norm, self.eps, 1, self.out_cols)
+                           s.vdim, meta.max_q, s.qkv_act, s.k_scale)
+        y = ops.gated_norm(o, p[:, self.offs[3]:], self.norm, self.eps, self.groups, self.out_cols, s.gate_act)
         return self.o(y, reduce=reduce, out=out)
 
 
 MIXERS = {"attention": MixedAttention, "latent": LatentAttention, "delta": GatedDelta, "decay": DecayAttention}
 
 
-def load_mixer(spec: MixerSpec, prefix: str, weights, idx: int, eps: float, comm, rotary: RotaryTables) -> Mixer:
-    return MIXERS[spec.kind](spec, prefix, weights, idx, eps, comm, rotary)
+def load_mixer(spec: MixerSpec, prefix: str, weights, idx: int, eps: float, comm, rotary: RotaryTables,
+               input_conv: Optional[str] = None) -> Mixer:
+    """``input_conv``: tensor of the layer's input convolution."""
+    mixer = MIXERS[spec.kind](spec, prefix, weights, idx, eps, comm, rotary)
+    if spec.input_conv:
+        w = weights.get_tensor(input_conv, to_dtype=False)
+        if w.shape[1] != spec.input_conv:
+            raise ValueError(f"{input_conv}: {w.shape[1]} taps instead of {spec.input_conv}")
+        mixer.input_conv = InputConv(w, weights.dtype, weights.device)
+    return mixer

@@ -71,16 +71,17 @@ def rope_and_cache(qkv, positions, cos_sin, slots, k_cache, v_cache, num_heads, 
 
 
 def paged_attention(q, k_cache, v_cache, block_tables, cu_seqlens_q, kv_lens, scale, window=-1, softcap=0.0,
-                    k_scale=None, v_scale=None, max_q=None, max_kv=None, horizon=None, chunk=0, sink=None):
+                    k_scale=None, v_scale=None, max_q=None, max_kv=None, horizon=None, chunk=0, sink=None, keep=0):
     """``horizon`` (optional int32 ``[T]``): last KV position each query row may see when that is past its own
     position (image rows that attend to their whole image); ``None`` is plain causal attention.  ``chunk`` > 0: rows see
     only keys of their own chunk of ``chunk`` positions.  ``sink``: one more key without a value in the softmax, of the score
-    given per head (fp32 ``[Hq]``; ``True``: 0), which is neither scaled nor capped."""
+    given per head (fp32 ``[Hq]``; ``True``: 0), which is neither scaled nor capped.  ``keep``: the first tokens of a sequence,
+    visible whatever the window."""
     if use_native(q):
         return native().paged_attention(q, k_cache, v_cache, block_tables, cu_seqlens_q, kv_lens, scale,
-                                        window, softcap, k_scale, v_scale, max_q, max_kv, horizon=horizon, chunk=chunk, sink=sink)
+                                        window, softcap, k_scale, v_scale, max_q, max_kv, horizon=horizon, chunk=chunk, sink=sink, keep=keep)
     return ref.paged_attention(q, k_cache, v_cache, block_tables, cu_seqlens_q, kv_lens, scale, window,
-                               softcap, k_scale, v_scale, horizon=horizon, chunk=chunk, sink=sink)
+                               softcap, k_scale, v_scale, horizon=horizon, chunk=chunk, sink=sink, keep=keep)
 
 
 def act_and_mul(gate_up, act="silu"):
@@ -107,9 +108,21 @@ def _mixer_backend(t):
     return native() if use_native(t) else ref
 
 
-def embed_residual(ids, table, scale=1.0):
-    """``table[ids] * scale`` as the fp32 residual stream."""
-    return _mixer_backend(table).embed_residual(ids, table, scale)
+def embed_residual(ids, table, scale=1.0, streams=1):
+    """``table[ids] * scale`` as the fp32 residual stream ``[T, H]``; with ``streams`` > 1 as the first of so many,
+    ``[streams, T, H]``, the others not yet written."""
+    return _mixer_backend(table).embed_residual(ids, table, scale, streams)
+
+
+def stream_step(delta, post, residual, weight, eps, rows=None, keep=True, gain=1.0, average=None, streams=None, conv=None):
+    """``r = residual + RMSNorm(delta) * post`` in fp32 (``post`` ``None``: plus ``delta``; ``delta`` ``None``: ``residual``).  With
+    ``average`` (fp32 ``[n]``), ``r`` is kept as ``streams[n - 1]`` and replaced by the sum over ``streams[:n]`` so weighted.
+    Returns ``(RMSNorm(r) * weight * gain, r)`` as ``residual_norm`` does; ``rows`` and ``keep`` as there (chosen rows are not
+    kept in ``streams``).  ``conv`` (a ``ShortConv`` of all columns): what comes out is convolved over time."""
+    backend = _mixer_backend(residual)
+    inside = conv is not None and conv.single
+    out, r = backend.stream_step(delta, post, residual, weight, eps, rows, keep, gain, average, streams, conv if inside else None)
+    return (out if conv is None or inside else backend.input_conv(out, conv)), r
 
 
 def residual_norm(delta, residual, weight, eps, rows=None, keep=True, scale=1.0, unit_offset=False, weight2=None, layer=False,
@@ -162,6 +175,18 @@ def row_norm_store(proj, offs, positions, slots, k_cache, v_cache, q_weight, k_w
                                                num_kv_heads, dim, vdim, width, temperature)
 
 
+def map_store(proj, offs, slots, k_cache, v_cache, num_heads, num_kv_heads, dim, vdim):
+    """``proj[T, *]`` with q and k (two maps of ``dim`` per head) and v from columns ``offs``: k and v stored, the maps of a key
+    head side by side.  Returns ``[T, 2 Hq, Dk]``: every query map alone at its place in such a row, zeros elsewhere."""
+    return _mixer_backend(proj).map_store(proj, offs, slots, k_cache, v_cache, num_heads, num_kv_heads, dim, vdim)
+
+
+def map_difference(a, gate, lam, factor, eps, width):
+    """``a[T, 2 H, pitch]``: even rows minus ``lam`` times odd rows, over their root mean square (first ``width`` columns), times
+    ``factor`` and ``sigmoid(gate[T, H])`` (``None``: no gate); ``[T, H * width]``."""
+    return _mixer_backend(a).map_difference(a, gate, lam, factor, eps, width)
+
+
 def output_gate(x, gate, width):
     """``x[T, H, pitch]``: the first ``width`` columns of every head times ``sigmoid(gate[T, H * width])``, ``[T, H * width]``."""
     return _mixer_backend(x).output_gate(x, gate, width)
@@ -174,24 +199,27 @@ def latent_layout(rank, rot, dtype, device):
     return rank, rank + rot
 
 
-def latent_store(proj, off_c, weight, eps, positions, cos_sin, slots, pages, q, off_rot, rank, rot, heads, dim, q_full=None):
+def latent_store(proj, off_c, weight, eps, positions, cos_sin, slots, pages, q, off_rot, rank, rot, heads, dim, q_full=None,
+                 queries=True, q_latent=None, width=None):
     """Latent attention's inputs from ``proj[T, *]`` (queries, ``dim`` plain and ``rot`` rotated dimensions per head, from
     column 0; ``rank`` latent columns and the shared key's ``rot`` columns from ``off_c``): the latent over its root mean
     square times ``weight``, and the shared key rotated (pairs ``2i, 2i + 1``), go to ``pages`` at the tokens' slots; the
     rotated dimensions of the queries go to ``q[T, H, *]`` from column ``off_rot``, zeros behind them, and whole queries (plain,
-    rotated, zeros) to ``q_full[T, H, *]``; either may be ``None``."""
+    rotated, zeros) to ``q_full[T, H, *]``; either may be ``None``.  ``pages`` ``None``: ``proj`` holds queries only (``width``: that
+    of a page row).  ``queries=False``: it holds none, but with ``q_latent = (column, weight, out)`` another latent, which goes to
+    ``out`` over its root mean square times ``weight``, zeros behind it."""
     _mixer_backend(proj).latent_store(proj, off_c, weight, eps, positions, cos_sin, slots, pages, q, off_rot, rank, rot, heads, dim,
-                                      q_full)
+                                      q_full, queries, q_latent, width)
 
 
 def latent_attention(q, pages, rank, block_tables, cu_seqlens_q, kv_lens, scale, window=-1, max_q=None, max_kv=None, gate=None,
-                     elsewhere=None):
+                     elsewhere=None, sink=None):
     """Causal attention of ``q[T, H, width]`` over the one key row per token in ``pages[blocks, block_size, 1, width]``, whose
     first ``rank`` columns are the value too; head outputs times ``sigmoid(gate[T, H])``.  ``[T, H, rank or more]``, zeros
     past ``rank``.  Sequences whose entry in ``elsewhere[B]`` is at least their number of tokens are left out (their rows are
-    not written)."""
+    not written).  ``sink`` (fp32 ``[H]``): as in ``paged_attention``."""
     return _mixer_backend(q).latent_attention(q, pages, rank, block_tables, cu_seqlens_q, kv_lens, scale, window, max_q, max_kv,
-                                              gate, elsewhere)
+                                              gate, elsewhere, sink)
 
 
 def expanded_dims(dim, vdim, dtype, device):
@@ -201,10 +229,10 @@ def expanded_dims(dim, vdim, dtype, device):
     return None
 
 
-def expanded_attention(q, kv, plan, cu_seqlens_q, scale, window, max_q, gate, out):
+def expanded_attention(q, kv, plan, cu_seqlens_q, scale, window, max_q, gate, out, sink=None):
     """Causal attention of ``q[T, H, dk]`` over keys and values written out for the step, ``kv[rows, H * dk + H * 128]``, laid out
     as ``plan`` (``models.mixers.Expansion``) says; rows of the plan's sequences are written to ``out[T, H, 128]``."""
-    native().expanded_attention(q, kv, plan, cu_seqlens_q, scale, window, max_q, gate, out)
+    native().expanded_attention(q, kv, plan, cu_seqlens_q, scale, window, max_q, gate, out, sink)
 
 
 def recurrent_pitch(dim, device):
@@ -237,9 +265,10 @@ def delta_scan(q, k, v, g, beta, qk, cu, kv_lens, state_slots, state, dim, max_q
     return _mixer_backend(v).delta_scan(q, k, v, g, beta, qk, cu, kv_lens, state_slots, state, dim, max_q)
 
 
-def decay_scan(proj, offs, decay, cu, kv_lens, state_slots, state, heads, dim, vdim, max_q):
-    """Linear attention with one decay per head on ``silu`` of q, k, v; advances ``state``, fp32 ``[T, H, vdim]``."""
-    return _mixer_backend(proj).decay_scan(proj, offs, decay, cu, kv_lens, state_slots, state, heads, dim, vdim, max_q)
+def decay_scan(proj, offs, decay, cu, kv_lens, state_slots, state, heads, dim, vdim, max_q, act="silu", k_scale=1.0):
+    """Linear attention with one decay per head on q, k, v (after ``act``: ``"silu"`` or ``""``), k times ``k_scale``; advances
+    ``state``, fp32 ``[T, H, vdim]``."""
+    return _mixer_backend(proj).decay_scan(proj, offs, decay, cu, kv_lens, state_slots, state, heads, dim, vdim, max_q, act, k_scale)
 
 
 def gated_norm(o, gate, weight, eps, groups, out_cols, act="sigmoid"):

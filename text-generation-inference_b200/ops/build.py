@@ -25,7 +25,7 @@ LIB_PATH = HERE / "libtgi_b200_kernels.so"
 KERNEL_SETS = {
     # decoders in bf16 / fp32 on one GPU, with attention, recurrent layers and routed experts
     "decoder": ["attention_prefill_sm100", "attention_sm100", "attn_inputs", "fused_ops", "gemm_sm100", "gemm_static_scratch",
-                "latent_attention_sm100", "mixer_ops", "moe_sm100", "recurrent_sm100"],
+                "latent_attention_sm100", "mixer_ops", "moe_sm100", "recurrent_sm100", "stream_ops"],
 }
 
 NVCC_FLAGS = [

@@ -1,6 +1,6 @@
 // Paged causal prefill attention on the 5th-generation tensor cores (sm_100a): head size 128 (or, with bf16 pages, 192
 // for queries and keys), pages of 16 tokens, bf16 or e4m3 KV pages, ragged batches with a cached prefix (chunked
-// prefill), GQA, sliding window, soft-capping, per-row horizons and a gate per token and head.
+// prefill), GQA, sliding window with kept first tokens, soft-capping, per-row horizons and a gate per token and head.
 //
 // Replaces, in the reference, flashinfer `BatchPrefillWithPagedKVCache` / FA2 `varlen_fwd`
 // (layers/attention/cuda.py:244-296, layers/attention/flashinfer.py:58-128).
@@ -64,6 +64,7 @@ struct PrefillParams {
   float scale, softcap;
   int window;
   int chunk;                    // > 0: a row sees only keys of its own chunk of `chunk` positions
+  int keep;                     // first tokens that every row sees whatever its window
   const float* sink;            // [Hq] or null: score of one more key per head that has no value
   int* status;
 };
@@ -243,7 +244,11 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
   const int pos_last = min(Lkv - 1, pos_first + kRows - 1);
   const int t_lo = first_visible(p, pos_first) / kKeys * kKeys;
   const int t_hi = p.horizon != nullptr ? Lkv : pos_last + 1;
-  const int ntiles = (t_hi - t_lo + kKeys - 1) / kKeys;
+  // Kept first tokens come in tiles of their own ahead of the window's: a row whose window starts at `lo` reads keys
+  // 0 .. min(keep, lo) - 1 of them and the window's tiles from `lo` on, so a tile has one range of visible keys per row.
+  const int kept = (min(p.keep, first_visible(p, pos_last)) + kKeys - 1) / kKeys;
+  const int ntiles = kept + (t_hi - t_lo + kKeys - 1) / kKeys;
+  auto tile_start = [&](int j) { return j < kept ? j * kKeys : t_lo + (j - kept) * kKeys; };
 
   if (threadIdx.x == 0) {
     for (int i = 0; i < 2; ++i) {
@@ -292,7 +297,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
     bool ok = true;
     for (int j = 0; j < ntiles && ok; ++j) {
       const int s = j & 1, vs = L::stage(j);
-      const int t0 = t_lo + j * kKeys;
+      const int t0 = tile_start(j);
       int blk = 0;
       if (lane < kKeys / kPage) {
         const int blk_i = (t0 >> 4) + lane;
@@ -442,9 +447,8 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
     sa.scale_log2 = scale_log2;
     sa.cap_in = cap ? raw_scale / p.softcap : 0.f;
     sa.cap_out = p.softcap * kLog2e;
-    // visible keys of this row: [t_min, t_max]
-    const int t_max = min(hz, Lkv - 1);
-    const int t_min = first_visible(p, pos);
+    // visible keys of this row in a tile of its window
+    const int win_max = min(hz, Lkv - 1), win_min = first_visible(p, pos);
     float m = -INFINITY, l = 0.f;
     // The two threads of a row meet at a named barrier once per tile, so they must leave the loop together: a
     // thread whose wait ran out raises the quarter's flag of the NEXT barrier's parity and keeps walking to that
@@ -452,7 +456,8 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
     bool fail = false;
     for (int j = 0; j < ntiles; ++j) {
       const int s = j & 1, ps = L::stage(j);
-      const int t0 = t_lo + j * kKeys + hf * 64;    // first key of this thread's half
+      const int t0 = tile_start(j) + hf * 64;       // first key of this thread's half
+      const int t_min = j < kept ? 0 : win_min, t_max = j < kept ? min(p.keep, win_min) - 1 : win_max;
       if (!fail && !mbar_wait(&s_full[s], (j >> 1) & 1)) { report(p.status, kErrEpilogueWait); fail = true; }
       if (fail) s_abort[quarter * 2 + s] = 1;
       tc_fence_after();
@@ -663,7 +668,7 @@ extern "C" {
 int tgi_prefill_attention_tc(const void* q, const void* k_cache, const void* v_cache, const int* block_tables,
                              const int* cu_seqlens_q, const int* kv_lens, const float* k_scale, const float* v_scale,
                              void* out, int B, int max_q, int max_blocks, int num_blocks, int Hq, int Hkv, float scale,
-                             float softcap, int window, int chunk, const float* sink, int fp8_kv, const int* horizon,
+                             float softcap, int window, int chunk, int keep, const float* sink, int fp8_kv, const int* horizon,
                              int* status, cudaStream_t stream) {
   if (B <= 0 || max_q <= 0) return 0;
   if (Hq % Hkv != 0 || B > 65535 || Hq > 65535) return -10;
@@ -684,6 +689,7 @@ int tgi_prefill_attention_tc(const void* q, const void* k_cache, const void* v_c
   p.softcap = softcap;
   p.window = window;
   p.chunk = chunk;
+  p.keep = keep > 0 ? keep : 0;
   p.sink = sink;
   p.status = status;
   const long long pitch = static_cast<long long>(Hkv) * kD;
@@ -694,11 +700,11 @@ int tgi_prefill_attention_tc(const void* q, const void* k_cache, const void* v_c
 // The same on keys and values of H heads that were written out for this step: q [T, H, dim] bf16 with dim 128 or 192, a
 // token's keys [H, dim] and values [H, 128] `pitch` elements from the next token's, tokens in groups of 16 that
 // `block_tables` names.  Sequences whose kv_lens entry is smaller than their number of tokens are left out.  gate
-// (optional): [T, ld_gate].
+// (optional): [T, ld_gate]; sink (optional): [H].
 int tgi_expanded_attention(const void* q, const void* k, const void* v, long long pitch, const int* block_tables,
                            const int* cu_seqlens_q, const int* kv_lens, const void* gate, long long ld_gate, void* out, int B,
-                           int max_q, int max_blocks, int num_blocks, int H, int dim, float scale, int window, int* status,
-                           cudaStream_t stream) {
+                           int max_q, int max_blocks, int num_blocks, int H, int dim, float scale, int window, const float* sink,
+                           int* status, cudaStream_t stream) {
   if (B <= 0 || max_q <= 0) return 0;
   if (B > 65535 || H > 65535 || num_blocks < 1 || max_blocks < 1 || pitch % 8 != 0 || (dim != 128 && dim != 192)) return -10;
   PrefillParams p{};
@@ -714,6 +720,7 @@ int tgi_expanded_attention(const void* q, const void* k, const void* v, long lon
   p.num_blocks = num_blocks;
   p.scale = scale;
   p.window = window;
+  p.sink = sink;
   p.status = status;
   return dim == 192 ? launch_prefill<false, 3>(p, k, v, pitch, pitch, B, max_q, stream)
                     : launch_prefill<false, 2>(p, k, v, pitch, pitch, B, max_q, stream);

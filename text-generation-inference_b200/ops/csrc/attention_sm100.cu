@@ -115,6 +115,7 @@ struct Params {
   float scale, softcap;
   int window;
   int chunk;                    // > 0: a row sees only keys of its own chunk of `chunk` positions
+  int keep;                     // first tokens that every row sees whatever its window
   const float* sink;            // [Hq] or null: score of one more key per head that has no value
   int nsplit;
 };
@@ -125,6 +126,9 @@ __device__ __forceinline__ int first_visible(const Params& p, int pos) {
   if (p.chunk > 0 && pos > 0) lo = max(lo, pos - pos % p.chunk);
   return max(lo, 0);
 }
+// Keys of the kept first tokens come in tiles of their own ahead of the window's: a row whose window starts at `lo` reads
+// keys 0 .. kept_end(lo) - 1 of them, and the window's tiles from `lo` on.  So a tile has one range of visible keys per row.
+__device__ __forceinline__ int kept_end(const Params& p, int lo) { return min(p.keep, lo); }
 // exp(sink - m) for a running maximum kept in the log2 domain: the share of the sink in the denominator.
 __device__ __forceinline__ float sink_term(const float* sink, int h, float m_log2) {
   return sink != nullptr ? exp2f(fmaf(sink[h], kLog2e, -m_log2)) : 0.f;
@@ -239,15 +243,17 @@ __device__ __forceinline__ float fast_tanh(float y) {      // 1 - 2 / (1 + e^(2y
   return 1.f - __fdividef(2.f, 1.f + fast_exp2(y * (2.f * kLog2e)));
 }
 
+constexpr int kCausal = -2;
+
 template <int NT>
 __device__ __forceinline__ void softmax_update(float (&s)[NT][4], float (&m)[2], float (&l)[2], float (&alpha)[2],
                                                int tbase, int pos0, int pos1, int lo0, int lo1, int lo_max, int L,
-                                               float scale_log2, float softcap, float raw_scale, int hz0 = -1,
-                                               int hz1 = -1) {
+                                               float scale_log2, float softcap, float raw_scale, int hz0 = kCausal,
+                                               int hz1 = kCausal) {
   // lo0 / lo1: first visible KV position of the two rows, lo_max: of the warp's last row
-  // hz0 / hz1: last visible KV position of the two rows (defaults: their own positions, i.e. causal)
-  if (hz0 < 0) hz0 = pos0;
-  if (hz1 < 0) hz1 = pos1;
+  // hz0 / hz1: last visible KV position of the two rows, -1: none (defaults: their own positions, i.e. causal)
+  if (hz0 == kCausal) hz0 = pos0;
+  if (hz1 == kCausal) hz1 = pos1;
   const int lane = threadIdx.x & 31;
   float mx[2] = {-INFINITY, -INFINITY};
   // a tile that lies entirely below the diagonal of all 16 rows of the warp, inside the window and inside the
@@ -346,7 +352,9 @@ prefill_kernel(Params p) {
   const int pos_last = min(L - 1, pos_first + kTile - 1);
   const int t_lo = first_visible(p, pos_first) / kTile * kTile;
   const int t_hi = p.horizon != nullptr ? L : pos_last + 1;   // exclusive; with horizons a row may see up to L - 1
-  const int ntiles = (t_hi - t_lo + kTile - 1) / kTile;
+  const int kept = (kept_end(p, first_visible(p, pos_last)) + kTile - 1) / kTile;      // tiles of kept first tokens
+  const int ntiles = kept + (t_hi - t_lo + kTile - 1) / kTile;
+  auto tile_start = [&](int j) { return j < kept ? j * kTile : t_lo + (j - kept) * kTile; };
 
   // ---- Q tile -> shared (bf16, or fp16 for e4m3 pages) ----
   for (int c = threadIdx.x; c < kTile * (D / 8); c += blockDim.x) {
@@ -370,8 +378,8 @@ prefill_kernel(Params p) {
     return FP8 ? static_cast<void*>(region + stg * kTile * D) : static_cast<void*>(region + stg * kTile * D * 2);
   };
   // first tile
-  load_tile<D, FP8>(p, p.k_cache, b, kvh, t_lo, L, stage_ptr(kreg, 0));
-  load_tile<D, FP8>(p, p.v_cache, b, kvh, t_lo, L, stage_ptr(vreg, 0));
+  load_tile<D, FP8>(p, p.k_cache, b, kvh, tile_start(0), L, stage_ptr(kreg, 0));
+  load_tile<D, FP8>(p, p.v_cache, b, kvh, tile_start(0), L, stage_ptr(vreg, 0));
   cp_async_commit();
   __syncthreads();
 
@@ -403,8 +411,8 @@ prefill_kernel(Params p) {
   for (int j = 0; j < ntiles; ++j) {
     const int stg = j & 1;
     if (j + 1 < ntiles) {
-      load_tile<D, FP8>(p, p.k_cache, b, kvh, t_lo + (j + 1) * kTile, L, stage_ptr(kreg, stg ^ 1));
-      load_tile<D, FP8>(p, p.v_cache, b, kvh, t_lo + (j + 1) * kTile, L, stage_ptr(vreg, stg ^ 1));
+      load_tile<D, FP8>(p, p.k_cache, b, kvh, tile_start(j + 1), L, stage_ptr(kreg, stg ^ 1));
+      load_tile<D, FP8>(p, p.v_cache, b, kvh, tile_start(j + 1), L, stage_ptr(vreg, stg ^ 1));
     }
     cp_async_commit();
     cp_async_wait<1>();
@@ -426,8 +434,9 @@ prefill_kernel(Params p) {
     float s[8][4];
     qk_warp<D, 8, FP8>(qf, cK, 0, s);
     float alpha[2];
-    softmax_update<8>(s, m, l, alpha, t_lo + j * kTile, pos0, pos1, lo0, lo1, lo_max, L, scale_log2, p.softcap,
-                      raw_scale, hz0, hz1);
+    const bool first = j < kept;                             // kept first tokens
+    softmax_update<8>(s, m, l, alpha, tile_start(j), pos0, pos1, first ? 0 : lo0, first ? 0 : lo1, first ? 0 : lo_max, L, scale_log2,
+                      p.softcap, raw_scale, first ? kept_end(p, lo0) - 1 : hz0, first ? kept_end(p, lo1) - 1 : hz1);
 #pragma unroll
     for (int i = 0; i < D / 8; ++i) {
       o[i][0] *= alpha[0]; o[i][1] *= alpha[0];
@@ -590,7 +599,9 @@ decode_kernel_v2(Params p) {
   const int pos = L - 1;
   const int lo = first_visible(p, pos);
   const int t_lo = lo / CT * CT;
-  const int chunks_total = (L - t_lo + CT - 1) / CT;
+  const int kept_to = kept_end(p, lo), kept = (kept_to + CT - 1) / CT;       // chunks of kept first tokens
+  const int chunks_total = kept + (L - t_lo + CT - 1) / CT;
+  auto chunk_start = [&](int c) { return c < kept ? c * CT : t_lo + (c - kept) * CT; };
   const int chunks_per = (chunks_total + p.nsplit - 1) / p.nsplit;
   const int c0 = split * chunks_per;
   const int c1 = min(chunks_total, c0 + chunks_per);
@@ -619,7 +630,7 @@ decode_kernel_v2(Params p) {
   auto vstage = [&](int stg) -> void* { return wbase + stg * 2 * S::kChunkBytes + S::kChunkBytes; };
   auto issue = [&](int i) {
     if (i < my_n) {
-      const int t0 = t_lo + (c0 + warp + 4 * i) * CT;
+      const int t0 = chunk_start(c0 + warp + 4 * i);
       warp_load_chunk<D, FP8, CT, true>(p, p.k_cache, b, kvh, t0, L, kstage(i % S::kStages), lane);
       warp_load_chunk<D, FP8, CT, false>(p, p.v_cache, b, kvh, t0, L, vstage(i % S::kStages), lane);
     }
@@ -664,8 +675,9 @@ decode_kernel_v2(Params p) {
       cV = static_cast<const uint16_t*>(vstage(i % S::kStages));
     }
     float alpha[2];
-    softmax_update<NT>(s, m, l, alpha, t_lo + (c0 + warp + 4 * i) * CT, pos, pos, lo, lo, lo, L, scale_log2, p.softcap,
-                       raw_scale);
+    const bool first = c0 + warp + 4 * i < kept;             // kept first tokens: none past kept_to
+    softmax_update<NT>(s, m, l, alpha, chunk_start(c0 + warp + 4 * i), pos, pos, first ? 0 : lo, first ? 0 : lo, first ? 0 : lo,
+                       first ? kept_to : L, scale_log2, p.softcap, raw_scale);
 #pragma unroll
     for (int j = 0; j < D / 8; ++j) {
       o[j][0] *= alpha[0]; o[j][1] *= alpha[0];
@@ -810,7 +822,9 @@ decode_kernel_v3(Params p, const __grid_constant__ CUtensorMap tmK, const __grid
   const int pos = L - 1;
   const int lo = first_visible(p, pos);
   const int t_lo = lo / CT * CT;
-  const int chunks_total = (L - t_lo + CT - 1) / CT;
+  const int kept_to = kept_end(p, lo), kept = (kept_to + CT - 1) / CT;       // chunks of kept first tokens
+  const int chunks_total = kept + (L - t_lo + CT - 1) / CT;
+  auto chunk_start = [&](int c) { return c < kept ? c * CT : t_lo + (c - kept) * CT; };
   const int chunks_per = (chunks_total + p.nsplit - 1) / p.nsplit;
   const int c0 = split * chunks_per;
   const int c1 = min(chunks_total, c0 + chunks_per);
@@ -830,7 +844,7 @@ decode_kernel_v3(Params p, const __grid_constant__ CUtensorMap tmK, const __grid
   // read when chunk i is issued, so that no copy waits for a global load.
   const int isv = lane & 1, box = lane >> 1;
   auto first_token = [&](int i) {
-    int t = t_lo + (c0 + warp + 4 * i) * CT + (box / EB) * 16;
+    int t = chunk_start(c0 + warp + 4 * i) + (box / EB) * 16;
     if (t >= L) t = (L - 1) & ~15;   // past the end: fetch the last group again (masked below)
     return t;
   };
@@ -920,7 +934,9 @@ decode_kernel_v3(Params p, const __grid_constant__ CUtensorMap tmK, const __grid
     done = i + 1;
     const uint8_t* sK = ring + (i % S::kStages) * S::kStageBytes;
     const uint8_t* sV = sK + CT * D * EB;
-    const int tbase = t_lo + (c0 + warp + 4 * i) * CT;
+    const int tbase = chunk_start(c0 + warp + 4 * i);
+    const bool first = c0 + warp + 4 * i < kept;             // kept first tokens
+    const int from = first ? 0 : lo, to = first ? kept_to : L;
 
     // ---- S^T = K Q^T (two accumulators per 16 tokens keep the dependent MMA chains short) ----
     float s[MT][4];
@@ -965,7 +981,7 @@ decode_kernel_v3(Params p, const __grid_constant__ CUtensorMap tmK, const __grid
 
     // ---- online softmax over the tokens of the chunk, per head ----
     // m[] is kept in the scaled log2 domain; a chunk that needs no masking takes the short path
-    const bool plain = p.softcap <= 0.f && tbase + CT <= L && tbase >= lo;
+    const bool plain = p.softcap <= 0.f && tbase + CT <= to && tbase >= from;
     float mx[2] = {-INFINITY, -INFINITY};
     if (plain) {
 #pragma unroll
@@ -984,7 +1000,7 @@ decode_kernel_v3(Params p, const __grid_constant__ CUtensorMap tmK, const __grid
           float v = s[mt][e];
           if (p.softcap > 0.f) v = p.softcap * kLog2e * fast_tanh(v * cap_in);
           else v = v * scale_log2;
-          const bool ok = t < L && t >= lo;
+          const bool ok = t < to && t >= from;
           v = ok ? v : -INFINITY;
           s[mt][e] = v;
           mx[e & 1] = fmaxf(mx[e & 1], v);
@@ -1268,7 +1284,7 @@ int launch_v3(const Params& p, int B, cudaStream_t stream) {
 extern "C" int tgi_prefill_attention_tc(const void* q, const void* k_cache, const void* v_cache, const int* block_tables,
                                         const int* cu_seqlens_q, const int* kv_lens, const float* k_scale,
                                         const float* v_scale, void* out, int B, int max_q, int max_blocks, int num_blocks,
-                                        int Hq, int Hkv, float scale, float softcap, int window, int chunk,
+                                        int Hq, int Hkv, float scale, float softcap, int window, int chunk, int keep,
                                         const float* sink, int fp8_kv, const int* horizon, int* status, cudaStream_t stream);
 
 bool prefill_tc_enabled() {
@@ -1288,7 +1304,7 @@ int launch(const Params& p, int B, int max_q, cudaStream_t stream) {
     if (cudaGetSymbolAddress(reinterpret_cast<void**>(&status), g_attn_status) != cudaSuccess) return -2;
     return tgi_prefill_attention_tc(p.q, p.k_cache, p.v_cache, p.block_tables, p.cu_seqlens_q, p.kv_lens, p.k_scale,
                                     p.v_scale, p.out, B, max_q, p.max_blocks, p.num_blocks, p.Hq, p.Hkv, p.scale, p.softcap,
-                                    p.window, p.chunk, p.sink, FP8 ? 1 : 0, p.horizon, status, stream);
+                                    p.window, p.chunk, p.keep, p.sink, FP8 ? 1 : 0, p.horizon, status, stream);
   }
   if (max_q > 1) {
     auto k = prefill_kernel<D, FP8>;
@@ -1361,12 +1377,13 @@ int tgi_attn_status(int reset) {
 
 // `horizon` (optional, prefill only): per query row the last KV position it may attend to; null = causal.
 // `chunk` > 0: rows see only keys of their own chunk of `chunk` positions, counted from position 0.
+// `keep`: rows see the first `keep` tokens whatever their window or chunk.
 // `sink` (optional, [Hq]): exp(sink[h]) is added to the softmax denominators of head h.
 int tgi_paged_attention_ex(const void* q, const void* k_cache, const void* v_cache, const int* block_tables,
                            const int* cu_seqlens_q, const int* kv_lens, const float* k_scale, const float* v_scale,
                            void* out, float* part_o, float* part_ml, int B, int max_q, int max_blocks, int block_size,
                            int num_blocks, int Hq, int Hkv, int D, float scale, float softcap, int window, int chunk,
-                           const float* sink, int nsplit, int fp8_kv, const int* horizon, cudaStream_t stream);
+                           int keep, const float* sink, int nsplit, int fp8_kv, const int* horizon, cudaStream_t stream);
 
 int tgi_paged_attention(const void* q, const void* k_cache, const void* v_cache, const int* block_tables,
                         const int* cu_seqlens_q, const int* kv_lens, const float* k_scale, const float* v_scale,
@@ -1375,14 +1392,14 @@ int tgi_paged_attention(const void* q, const void* k_cache, const void* v_cache,
                         int fp8_kv, cudaStream_t stream) {
   return tgi_paged_attention_ex(q, k_cache, v_cache, block_tables, cu_seqlens_q, kv_lens, k_scale, v_scale, out, part_o,
                                 part_ml, B, max_q, max_blocks, block_size, num_blocks, Hq, Hkv, D, scale, softcap, window,
-                                0, nullptr, nsplit, fp8_kv, nullptr, stream);
+                                0, 0, nullptr, nsplit, fp8_kv, nullptr, stream);
 }
 
 int tgi_paged_attention_ex(const void* q, const void* k_cache, const void* v_cache, const int* block_tables,
                            const int* cu_seqlens_q, const int* kv_lens, const float* k_scale, const float* v_scale,
                            void* out, float* part_o, float* part_ml, int B, int max_q, int max_blocks, int block_size,
                            int num_blocks, int Hq, int Hkv, int D, float scale, float softcap, int window, int chunk,
-                           const float* sink, int nsplit, int fp8_kv, const int* horizon, cudaStream_t stream) {
+                           int keep, const float* sink, int nsplit, int fp8_kv, const int* horizon, cudaStream_t stream) {
   if (B <= 0 || max_q <= 0) return 0;
   if (Hq % Hkv != 0) return -10;
   Params p;
@@ -1410,6 +1427,7 @@ int tgi_paged_attention_ex(const void* q, const void* k_cache, const void* v_cac
   p.softcap = softcap;
   p.window = window;
   p.chunk = chunk;
+  p.keep = keep > 0 ? keep : 0;
   p.sink = sink;
   p.nsplit = (max_q > 1 || nsplit < 1) ? 1 : nsplit;
   if (p.nsplit > 1 && (part_o == nullptr || part_ml == nullptr)) return -11;

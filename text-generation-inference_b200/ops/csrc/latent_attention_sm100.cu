@@ -49,6 +49,7 @@ struct LatentParams {
   const int* elsewhere;           // null, or [B]: sequences whose entry is at least their number of tokens are left out
   const __nv_bfloat16* gate;      // [T, ld_gate] or null: pre-activation of the factor on a head's output
   long long ld_gate;
+  const float* sink;              // [H] or null: score of one more key per head that has no value
   __nv_bfloat16* out;             // [T * H, out_cols]
   float *part_o, *part_ml;        // [2 * CTAs][N][out_cols] and [2 * CTAs][N][2]
   int* range;                     // [items][2]: first and last CTA of an item (persistent)
@@ -113,6 +114,10 @@ __device__ __forceinline__ float column_reduce(float (&v)[C], int lane) {
     v[0] = SUM ? v[0] + got : fmaxf(v[0], got);
   }
   return v[0];
+}
+// the sink's share of the denominator of head h, for exponents that refer to m
+__device__ __forceinline__ float sink_term(const float* sink, int h, float m) {
+  return sink != nullptr ? exp2f(fmaf(sink[h], kLog2e, -m)) : 0.f;
 }
 __device__ __forceinline__ int first_visible(int pos, int window) { return window > 0 ? max(0, pos - window + 1) : 0; }
 // key tiles of the rows whose first and last token sit at pos0 and pos1 (at least one: its keys are masked), and their start
@@ -558,7 +563,7 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
         float f = 1.f;
         if (w.part < 0) {
           if (p.persistent && tid == 0) p.range[2 * w.item] = p.range[2 * w.item + 1] = 0;
-          f = sum > 0.f ? 1.f / sum : 0.f;
+          f = sum > 0.f ? 1.f / (sum + sink_term(p.sink, (w.q_row + tid) % p.H, m)) : 0.f;
           if (p.gate != nullptr && tid < w.rows) {
             const int row = w.q_row + tid;
             f *= __fdividef(1.f, 1.f + __expf(-__bfloat162float(p.gate[static_cast<long long>(row / p.H) * p.ld_gate + row % p.H])));
@@ -701,7 +706,7 @@ latent_merge_kernel(const LatentParams p) {
   if (lane == 0) red[4 + warp] = sum;
   __syncthreads();
   sum = (red[4] + red[5]) + (red[6] + red[7]);
-  float f = sum > 0.f ? 1.f / sum : 0.f;
+  float f = sum > 0.f ? 1.f / (sum + sink_term(p.sink, row, mm)) : 0.f;
   if (p.gate != nullptr)
     f *= __fdividef(1.f, 1.f + __expf(-__bfloat162float(p.gate[static_cast<long long>(begin) * p.ld_gate + row])));
 #pragma unroll
@@ -774,9 +779,9 @@ int tgi_latent_rows(int slabs, int value_slabs, long long rows) {
 // q [T, H, slabs * 64] and pages [num_blocks, 16, slabs * 64] bf16 (the first value_slabs * 64 columns of a row are the
 // values), out [T, H, value_slabs * 64]; no sequence brings more than max_q tokens.  part_o / part_ml: 2 * ctas slots of N x (value_slabs * 64) and N x 2 floats, range:
 // 2 * B * ceil(H / N) ints; used when max_q == 1.  Sequences whose entry in `elsewhere` (optional, [B]) is at
-// least their number of tokens are left out (and may bring more than max_q).  gate (optional): [T, ld_gate].
+// least their number of tokens are left out (and may bring more than max_q).  gate (optional): [T, ld_gate]; sink (optional): [H].
 int tgi_latent_attention(const void* q, const void* pages, const int* block_tables, const int* cu, const int* kv_lens,
-                         const void* gate, long long ld_gate, void* out, float* part_o, float* part_ml, int* range, int T, int B, int max_q,
+                         const void* gate, long long ld_gate, const float* sink, void* out, float* part_o, float* part_ml, int* range, int T, int B, int max_q,
                          int max_blocks, int num_blocks, int H, int slabs, int value_slabs, int N, float scale, int window,
                          const int* elsewhere, int ctas, int* status, cudaStream_t stream) {
   if (T <= 0 || B <= 0 || max_q <= 0) return 0;
@@ -790,6 +795,7 @@ int tgi_latent_attention(const void* q, const void* pages, const int* block_tabl
   p.kv_lens = kv_lens;
   p.gate = static_cast<const __nv_bfloat16*>(gate);
   p.ld_gate = ld_gate;
+  p.sink = sink;
   p.out = static_cast<__nv_bfloat16*>(out);
   p.part_o = part_o;
   p.part_ml = part_ml;

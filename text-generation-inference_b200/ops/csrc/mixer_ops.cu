@@ -607,7 +607,7 @@ constexpr int kMaxOut = 32;        // value dimensions per lane: vdim <= 1024
 template <typename T>
 struct AnyAttention {
   float scale, softcap;             // softcap 0: scores as they are
-  int window, chunk;
+  int window, chunk, keep;          // keep: first tokens that stay visible past the window
   const float* sink;                // [Hq] or null
   const T* gate;                    // [T, ld_gate] or null
   long long ld_gate;
@@ -640,11 +640,12 @@ attn_any_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T*
 #pragma unroll
   for (int i = 0; i < NV; ++i) o[i] = 0.f;
   const int* table = block_tables + static_cast<size_t>(b) * max_blocks;
-  for (int t0 = lo; t0 <= pos; t0 += 32) {
+  // kept first tokens, then the window
+  for (int t0 = a.keep > 0 && lo > 0 ? 0 : lo, end = t0 < lo ? min(a.keep, lo) : pos + 1; t0 < end;) {
     const int key = t0 + lane;
     long long row = 0;
     float s = -INFINITY;
-    if (key <= pos) {
+    if (key < end) {
       row = (static_cast<long long>(table[key >> bs_shift]) << bs_shift) + (key & ((1 << bs_shift) - 1));
       const T* kp = k_cache + (static_cast<size_t>(row) * Hkv + kvh) * Dk;
       float acc = 0.f;
@@ -674,7 +675,7 @@ attn_any_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T*
     m = mn;
 #pragma unroll
     for (int i = 0; i < NV; ++i) o[i] *= alpha;
-    const int cnt = min(32, pos - t0 + 1);
+    const int cnt = min(32, end - t0);
     for (int j = 0; j < cnt; ++j) {
       const float pj = __shfl_sync(0xffffffffu, pr, j);
       const long long rj = __shfl_sync(0xffffffffu, row, j);
@@ -682,6 +683,11 @@ attn_any_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T*
 #pragma unroll
       for (int i = 0; i < NV; ++i)
         if (lane + 32 * i < Dv) o[i] = fmaf(pj, to_f(vp[lane + 32 * i]), o[i]);
+    }
+    t0 += 32;
+    if (t0 >= end && end <= lo) {
+      t0 = lo;
+      end = pos + 1;
     }
   }
   float inv = l > 0.f ? 1.f / l : 0.f;
@@ -1508,16 +1514,16 @@ int tgi_attn_prep(int f32, const void* proj, long long ld, int off_k, int off_v,
 // head h is multiplied by the sigmoid of its column h.
 int tgi_attn_any(int f32, const void* q, const void* k_cache, const void* v_cache, const int* block_tables, const int* cu,
                  const int* kv_lens, void* out, int T, int B, int max_blocks, int block_size, int Hq, int Hkv, int Dk, int Dv,
-                 int ldv, float scale, float softcap, int window, int chunk, const float* sink, const void* gate,
+                 int ldv, float scale, float softcap, int window, int chunk, int keep, const float* sink, const void* gate,
                  long long ld_gate, cudaStream_t stream) {
   if (T <= 0 || B <= 0) return 0;
   if (Hq % Hkv != 0 || block_size <= 0 || (block_size & (block_size - 1)) != 0) return -10;
   int shift = 0;
   while ((1 << shift) < block_size) ++shift;
   return f32 ? attn_any<float>(q, k_cache, v_cache, block_tables, cu, kv_lens, out, T, B, max_blocks, shift, Hq, Hkv, Dk, Dv, ldv,
-                               {scale, softcap, window, chunk, sink, static_cast<const float*>(gate), ld_gate}, stream)
+                               {scale, softcap, window, chunk, keep, sink, static_cast<const float*>(gate), ld_gate}, stream)
              : attn_any<bf16>(q, k_cache, v_cache, block_tables, cu, kv_lens, out, T, B, max_blocks, shift, Hq, Hkv, Dk, Dv, ldv,
-                              {scale, softcap, window, chunk, sink, static_cast<const bf16*>(gate), ld_gate}, stream);
+                              {scale, softcap, window, chunk, keep, sink, static_cast<const bf16*>(gate), ld_gate}, stream);
 }
 
 // Rows of the [rows][channels] convolution weights tgi_delta_prep wants for `taps` taps (the first rows are zero).

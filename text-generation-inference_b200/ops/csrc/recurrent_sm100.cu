@@ -3,6 +3,7 @@
 //   gated delta rule, one decay per key channel      S <- g * S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
 //   the same with one decay per head                 (g a scalar)
 //   linear attention with a fixed decay per head     S <- d S + k v^T;                                    o = S^T q
+//                                                    (q, k, v as projected or after SiLU, k times a factor)
 //
 // The columns of S never meet: column j of a head needs k, q, g of the head and only v_j of its own.
 //
@@ -50,7 +51,7 @@ __device__ __forceinline__ float silu_t<bf16>(float x) { return __fdividef(x, 1.
 struct ScanArgs {
   // delta rule: fp32 q, k [T, G, dimP], g [T, H, dimP] (one decay per head: [T, H]), v [T, H, vdim], beta [T, H], qk = q . k [T, G]
   const float *q, *k, *g, *v, *beta, *qk;
-  // linear attention: proj [T, ld] with q, k (H x dim) and v (H x vdim) at off_q, off_k, off_v (SiLU applied here)
+  // linear attention: proj [T, ld] with q, k (H x dim) and v (H x vdim) at off_q, off_k, off_v (SiLU applied here if `silu`)
   const void* proj;
   long long ld;
   int off_q, off_k, off_v;
@@ -62,6 +63,8 @@ struct ScanArgs {
   float* out;                     // [T, H, vdim]
   int num_slots, G, H, dim, dimP, vdim;
   int vec;                        // proj: heads may be read four elements at a time
+  int silu;                       // linear attention: q, k and v go through SiLU
+  float k_scale;                  // linear attention: factor of k
 };
 
 // sum over the eight lanes of a column group
@@ -147,16 +150,19 @@ struct PairOf<bf16> {
     return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w));
   }
 };
-// columns c .. c + 3 of a head after SiLU, zero past `dim`; `vec`: the four may be read at once
+// SiLU where `on`
 template <typename T>
-__device__ __forceinline__ float4 load4_silu(const T* p, int c, int dim, bool vec) {
+__device__ __forceinline__ float act_t(float x, bool on) { return on ? silu_t<T>(x) : x; }
+// columns c .. c + 3 of a head after SiLU (where `on`) times f, zero past `dim`; `vec`: the four may be read at once
+template <typename T>
+__device__ __forceinline__ float4 load4_act(const T* p, int c, int dim, bool vec, bool on, float f) {
   if (vec && c < dim) {
     const float4 x = raw4(p + c);
-    return make_float4(silu_t<T>(x.x), silu_t<T>(x.y), silu_t<T>(x.z), silu_t<T>(x.w));
+    return make_float4(f * act_t<T>(x.x, on), f * act_t<T>(x.y, on), f * act_t<T>(x.z, on), f * act_t<T>(x.w, on));
   }
   float v[4];
 #pragma unroll
-  for (int i = 0; i < 4; ++i) v[i] = c + i < dim ? silu_t<T>(to_f(p[c + i])) : 0.f;
+  for (int i = 0; i < 4; ++i) v[i] = c + i < dim ? f * act_t<T>(to_f(p[c + i]), on) : 0.f;
   return make_float4(v[0], v[1], v[2], v[3]);
 }
 __device__ __forceinline__ float4 mul4(float4 a, float4 b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); }
@@ -304,8 +310,11 @@ scan_kernel(ScanArgs p) {
             k[e] = PairOf<T>::value(k[e]);
             q[e] = PairOf<T>::value(q[e]);
           }
-          k[e] = make_float2(silu_t<T>(k[e].x), silu_t<T>(k[e].y));   // SiLU(0) = 0: absent tokens and channels stay 0
-          q[e] = make_float2(silu_t<T>(q[e].x), silu_t<T>(q[e].y));
+          if (p.silu) {                                               // SiLU(0) = 0: absent tokens and channels stay 0
+            k[e] = make_float2(silu_t<T>(k[e].x), silu_t<T>(k[e].y));
+            q[e] = make_float2(silu_t<T>(q[e].x), silu_t<T>(q[e].y));
+          }
+          k[e] = make_float2(p.k_scale * k[e].x, p.k_scale * k[e].y);
           g[e].x = g[e].y = e < cnt ? dec : 1.f;
         }
       }
@@ -357,7 +366,7 @@ scan_kernel(ScanArgs p) {
     }
 #pragma unroll
     for (int i = 0; i < NV; ++i)
-      d[S::kOffV + tid + i * kThreads] = DELTA ? rvf[DELTA ? i : 0] : silu_t<T>(to_f(rv[DELTA ? 0 : i]));
+      d[S::kOffV + tid + i * kThreads] = DELTA ? rvf[DELTA ? i : 0] : act_t<T>(to_f(rv[DELTA ? 0 : i]), p.silu);
     if (DELTA && tid < kTile) d[S::kOffBeta + tid] = rb;
     if (HEAD && tid < kTile) d[S::kOffGate + tid] = rh;
   };
@@ -592,15 +601,16 @@ step_kernel(ScanArgs p) {
   } else {
     const T* row = static_cast<const T*>(p.proj) + static_cast<size_t>(t) * p.ld;
     const float dec = p.decay[h];
-    // SiLU of the head's k and q once per block (the state is on its way meanwhile)
+    // the head's k and q once per block (the state is on its way meanwhile)
     for (int i = threadIdx.x; i < 16 * J; i += kThreads) {
       const int c4 = (i % (8 * J)) * 4;
-      *reinterpret_cast<float4*>(kq_s + i * 4) = load4_silu(row + (i < 8 * J ? p.off_k : p.off_q) + h * p.dim, c4, p.dim, p.vec);
+      *reinterpret_cast<float4*>(kq_s + i * 4) = load4_act(row + (i < 8 * J ? p.off_k : p.off_q) + h * p.dim, c4, p.dim, p.vec,
+                                                                p.silu, i < 8 * J ? p.k_scale : 1.f);
     }
     __syncthreads();
 #pragma unroll
     for (int c = 0; c < CN; ++c) {
-      v[c] = col + c < p.vdim ? silu_t<T>(to_f(row[p.off_v + h * p.vdim + col + c])) : 0.f;
+      v[c] = col + c < p.vdim ? act_t<T>(to_f(row[p.off_v + h * p.vdim + col + c]), p.silu) : 0.f;
       o[c] = 0.f;
     }
 #pragma unroll
@@ -705,10 +715,12 @@ int tgi_delta_scan(const float* q, const float* k, const float* g, const float* 
   return head_decay ? dispatch<float, kHead>(p, B, max_q, stream) : dispatch<float, kChannel>(p, B, max_q, stream);
 }
 
+// `silu`: q, k and v go through SiLU first; k is then multiplied by k_scale
 int tgi_decay_scan(int f32, const void* proj, long long ld, int off_q, int off_k, int off_v, const float* decay, const int* cu,
                    const int* kv_lens, const int* state_slots, float* state, float* out, int B, int max_q, int num_slots,
-                   int H, int dim, int dimP, int vdim, cudaStream_t stream) {
+                   int H, int dim, int dimP, int vdim, int silu, float k_scale, cudaStream_t stream) {
   ScanArgs p{};
+  p.silu = silu; p.k_scale = k_scale;
   p.proj = proj; p.ld = ld; p.off_q = off_q; p.off_k = off_k; p.off_v = off_v; p.decay = decay;
   p.cu = cu; p.kv_lens = kv_lens; p.state_slots = state_slots;
   p.state = state; p.out = out;

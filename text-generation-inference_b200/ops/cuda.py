@@ -67,7 +67,7 @@ def load():
                  "tgi_activation", "tgi_attn_prep", "tgi_attn_any", "tgi_delta_prep", "tgi_delta_scan", "tgi_decay_scan",
                  "tgi_gated_norm", "tgi_recurrent_pitch", "tgi_delta_tap_rows", "tgi_act_mul_any", "tgi_moe_router",
                  "tgi_moe_router_splits", "tgi_moe_topk_sigmoid", "tgi_moe_topk_logits", "tgi_row_norm_store", "tgi_output_gate",
-                 "tgi_latent_store", "tgi_latent_rows", "tgi_latent_attention", "tgi_expanded_attention", "tgi_moe_grouped_f32", "tgi_moe_combine_f32"):
+                 "tgi_map_store", "tgi_map_difference", "tgi_stream_step", "tgi_input_conv", "tgi_latent_store", "tgi_latent_rows", "tgi_latent_attention", "tgi_expanded_attention", "tgi_moe_grouped_f32", "tgi_moe_combine_f32"):
         if hasattr(_LIB, name):        # a library built for one family of models lacks the other families' kernels
             getattr(_LIB, name).restype = c_int
     _LIB.tgi_gemm_workspace_floats.restype = c_ll
@@ -423,7 +423,7 @@ def attention_pitch(dim: int, vdim: int, dtype: torch.dtype) -> Tuple[int, int]:
 
 def paged_attention(q, k_cache, v_cache, block_tables, cu_seqlens_q, kv_lens, scale, window=-1, softcap=0.0,
                     k_scale=None, v_scale=None, max_q=None, max_kv=None, nsplit: Optional[int] = None, horizon=None,
-                    chunk: int = 0, sink=None):
+                    chunk: int = 0, sink=None, keep: int = 0):
     lib = load()
     if sink is False:
         sink = None
@@ -440,14 +440,14 @@ def paged_attention(q, k_cache, v_cache, block_tables, cu_seqlens_q, kv_lens, sc
     if q.dtype == torch.float32 or D != Dv or D not in ATTN_HEAD_DIMS:
         assert horizon is None and k_cache.dtype == q.dtype and v_cache.dtype == q.dtype
         return _attention_any(q.contiguous(), k_cache, v_cache, Dv, block_tables, cu_seqlens_q, kv_lens, out, scale, softcap, window,
-                              chunk, sink, None)
+                              chunk, sink, None, keep)
     if max_q is None:
         max_q = int((cu_seqlens_q[1:] - cu_seqlens_q[:-1]).max().item())
     if max_kv is None:
         max_kv = int(kv_lens.max().item())
     for span in (chunk, window or 0):
         if span > 0:
-            max_kv = min(max_kv, span)   # keys a row can see: decides how far a decode step is split
+            max_kv = min(max_kv, span + keep)   # keys a row can see: decides how far a decode step is split
     fp8 = k_cache.dtype == FP8
     st = state(q.device)
     part_o = part_ml = None
@@ -467,7 +467,7 @@ def paged_attention(q, k_cache, v_cache, block_tables, cu_seqlens_q, kv_lens, sc
         _ptr(k_scale if fp8 else None), _ptr(v_scale if fp8 else None), _ptr(out), _ptr(part_o), _ptr(part_ml),
         c_int(B), c_int(max_q), c_int(block_tables.shape[1]), c_int(bs), c_int(nblk), c_int(Hq), c_int(Hkv), c_int(D),
         c_float(scale), c_float(softcap), c_int(window if window and window > 0 else -1), c_int(chunk),
-        _ptr(sink), c_int(nsplit), c_int(1 if fp8 else 0), _ptr(horizon), _stream()), "paged_attention")
+        c_int(keep), _ptr(sink), c_int(nsplit), c_int(1 if fp8 else 0), _ptr(horizon), _stream()), "paged_attention")
     return out
 
 
@@ -482,15 +482,16 @@ def _zero_sink(device, heads: int) -> torch.Tensor:
     return _ZERO_SINKS[key]
 
 
-def _attention_any(q, k_cache, v_cache, vdim, block_tables, cu_seqlens_q, kv_lens, out, scale, softcap, window, chunk, sink, gate):
+def _attention_any(q, k_cache, v_cache, vdim, block_tables, cu_seqlens_q, kv_lens, out, scale, softcap, window, chunk, sink, gate,
+                   keep: int = 0):
     """The kernel for head sizes without an instance and for fp32; ``vdim`` columns of every value row are read."""
     T, Hq, D = q.shape
     _, bs, Hkv, ldv = v_cache.shape
     _check(load().tgi_attn_any(
         _f32(q), _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(block_tables), _ptr(cu_seqlens_q), _ptr(kv_lens), _ptr(out), c_int(T),
         c_int(kv_lens.shape[0]), c_int(block_tables.shape[1]), c_int(bs), c_int(Hq), c_int(Hkv), c_int(D), c_int(vdim), c_int(ldv),
-        c_float(scale), c_float(softcap), c_int(window if window and window > 0 else -1), c_int(chunk), _ptr(sink), _ptr(gate),
-        c_ll(0 if gate is None else gate.stride(0)), _stream()), "attn_any")
+        c_float(scale), c_float(softcap), c_int(window if window and window > 0 else -1), c_int(chunk), c_int(keep), _ptr(sink),
+        _ptr(gate), c_ll(0 if gate is None else gate.stride(0)), _stream()), "attn_any")
     return out
 
 
@@ -511,7 +512,7 @@ def expanded_dims(dim: int, vdim: int, dtype: torch.dtype):
     return (128 if dim <= 128 else 192), 128
 
 
-def expanded_attention(q, kv, plan, cu_seqlens_q, scale, window, max_q: int, gate, out):
+def expanded_attention(q, kv, plan, cu_seqlens_q, scale, window, max_q: int, gate, out, sink=None):
     T, H, dk = q.shape
     R = kv.shape[0]
     assert q.is_contiguous() and out.is_contiguous() and tuple(out.shape) == (T, H, 128) and kv.is_contiguous()
@@ -521,29 +522,35 @@ def expanded_attention(q, kv, plan, cu_seqlens_q, scale, window, max_q: int, gat
         _ptr(q), _ptr(kv), c_void_p(kv.data_ptr() + 2 * H * dk), c_ll(kv.stride(0)), _ptr(plan.tables), _ptr(cu_seqlens_q),
         _ptr(plan.kv_lens), _ptr(gate), c_ll(0 if gate is None else gate.stride(0)), _ptr(out), c_int(plan.kv_lens.shape[0]),
         c_int(max_q), c_int(plan.tables.shape[1]), c_int(R // 16), c_int(H), c_int(dk), c_float(scale),
-        c_int(window if window and window > 0 else -1), _ptr(st.status), _stream()), "expanded_attention")
+        c_int(window if window and window > 0 else -1), _ptr(sink), _ptr(st.status), _stream()), "expanded_attention")
 
 
 def latent_store(proj, off_c, weight, eps, positions, cos_sin, slots, pages, q, off_rot, rank: int, rot: int, heads: int, dim: int,
-                 q_full=None):
-    assert proj.stride(1) == 1 and pages.is_contiguous() and pages.shape[2] == 1 and pages.dtype == proj.dtype
-    assert q is None or (q.is_contiguous() and q.shape[2] == pages.shape[3] and q.dtype == proj.dtype)
+                 q_full=None, queries: bool = True, q_latent=None, width: Optional[int] = None):
+    assert proj.stride(1) == 1 and cos_sin.shape[1] == rot
+    assert pages is None or (pages.is_contiguous() and pages.shape[2] == 1 and pages.dtype == proj.dtype and weight.dtype == torch.float32)
+    width = pages.shape[3] if pages is not None else width
+    assert q is None or (q.is_contiguous() and q.shape[2] == width and q.dtype == proj.dtype)
     assert q_full is None or (q_full.is_contiguous() and q_full.dtype == proj.dtype)
-    assert weight.dtype == torch.float32 and cos_sin.shape[1] == rot
+    off_cq, cq_weight, cq = q_latent or (0, None, None)
+    assert cq is None or (cq.is_contiguous() and cq.dtype == proj.dtype and cq_weight.dtype == torch.float32)
     _check(load().tgi_latent_store(
         _f32(proj), _ptr(proj), c_ll(proj.stride(0)), c_int(off_c), _ptr(weight), c_float(eps), _ptr(positions), _ptr(cos_sin),
-        c_int(cos_sin.shape[0]), _ptr(slots), _ptr(pages), c_ll(pages.shape[0] * pages.shape[1]), _ptr(q), _ptr(q_full),
-        c_int(proj.shape[0]), c_int(heads), c_int(dim), c_int(rank), c_int(rot), c_int(off_rot), c_int(pages.shape[3]),
+        c_int(cos_sin.shape[0]), _ptr(slots), _ptr(pages), c_ll(0 if pages is None else pages.shape[0] * pages.shape[1]),
+        _ptr(proj if queries else None), c_ll(proj.stride(0)), _ptr(q), _ptr(q_full), c_int(off_cq),
+        c_int(0 if cq is None else cq_weight.shape[0]), _ptr(cq_weight), _ptr(cq), c_int(0 if cq is None else cq.shape[1]),
+        c_int(proj.shape[0]), c_int(heads), c_int(dim), c_int(rank), c_int(rot), c_int(off_rot), c_int(width),
         c_int(0 if q_full is None else q_full.shape[2]), _stream()), "latent_store")
 
 
 def latent_attention(q, pages, rank: int, block_tables, cu_seqlens_q, kv_lens, scale, window=-1, max_q=None, max_kv=None, gate=None,
-                     elsewhere=None):
+                     elsewhere=None, sink=None):
     """Tensor-core kernel for bf16 rows in 64-column pieces on pages of 16 tokens, ``tgi_attn_any`` otherwise."""
     lib = load()
     T, H, width = q.shape
     B = kv_lens.shape[0]
     assert gate is None or (gate.stride(1) == 1 and gate.dtype == q.dtype)
+    assert sink is None or (sink.dtype == torch.float32 and sink.shape == (H,) and sink.is_contiguous())
     assert q.is_contiguous() and pages.is_contiguous() and pages.shape[3] == width and pages.dtype == q.dtype
     values = (rank + 63) // 64
     if q.dtype == torch.bfloat16 and width % 64 == 0 and pages.shape[1] == 16 and max_q is not None:
@@ -554,7 +561,7 @@ def latent_attention(q, pages, rank: int, block_tables, cu_seqlens_q, kv_lens, s
             part = _latent_parts(st, N, 64 * values, B * ((H + N - 1) // N)) if max_q == 1 else (None,) * 3
             _check(lib.tgi_latent_attention(
                 _ptr(q), _ptr(pages), _ptr(block_tables), _ptr(cu_seqlens_q), _ptr(kv_lens), _ptr(gate),
-                c_ll(0 if gate is None else gate.stride(0)), _ptr(out), *map(_ptr, part), c_int(T), c_int(B), c_int(max_q),
+                c_ll(0 if gate is None else gate.stride(0)), _ptr(sink), _ptr(out), *map(_ptr, part), c_int(T), c_int(B), c_int(max_q),
                 c_int(block_tables.shape[1]), c_int(pages.shape[0]), c_int(H), c_int(width // 64), c_int(values), c_int(N),
                 c_float(scale), c_int(window if window and window > 0 else -1), _ptr(elsewhere), c_int(st.sm_count),
                 _ptr(st.status), _stream()), "latent_attention")
@@ -563,7 +570,7 @@ def latent_attention(q, pages, rank: int, block_tables, cu_seqlens_q, kv_lens, s
     out = q.new_empty(T, H, rank)
     if T == 0:
         return out
-    return _attention_any(q, pages, pages, rank, block_tables, cu_seqlens_q, kv_lens, out, scale, 0.0, window, 0, None, gate)
+    return _attention_any(q, pages, pages, rank, block_tables, cu_seqlens_q, kv_lens, out, scale, 0.0, window, 0, sink, gate)
 
 
 def _latent_parts(st, N: int, cols: int, items: int):
@@ -593,6 +600,28 @@ def row_norm_store(proj, offs, positions, slots, k_cache, v_cache, q_weight, k_w
     return q
 
 
+def map_store(proj, offs, slots, k_cache, v_cache, num_heads: int, num_kv_heads: int, dim: int, vdim: int):
+    T, Dk, Dv = proj.shape[0], k_cache.shape[3], v_cache.shape[3]
+    q = torch.empty(T, 2 * num_heads, Dk, dtype=proj.dtype, device=proj.device)
+    assert proj.stride(1) == 1 and k_cache.dtype == proj.dtype and v_cache.dtype == proj.dtype and offs[0] == 0
+    assert k_cache.is_contiguous() and v_cache.is_contiguous() and k_cache.shape[2] == v_cache.shape[2] == num_kv_heads
+    _check(load().tgi_map_store(
+        _f32(proj), _ptr(proj), c_ll(proj.stride(0)), c_int(offs[1]), c_int(offs[2]), _ptr(slots), _ptr(q), _ptr(k_cache),
+        _ptr(v_cache), c_int(T), c_int(num_heads), c_int(num_kv_heads), c_int(dim), c_int(vdim), c_int(Dk), c_int(Dv),
+        c_ll(k_cache.shape[0] * k_cache.shape[1]), _stream()), "map_store")
+    return q
+
+
+def map_difference(a, gate, lam: float, factor: float, eps: float, width: int):
+    T, H2, pitch = a.shape
+    out = torch.empty(T, H2 // 2 * width, dtype=a.dtype, device=a.device)
+    assert a.is_contiguous() and H2 % 2 == 0 and (gate is None or (gate.stride(1) == 1 and gate.dtype == a.dtype))
+    _check(load().tgi_map_difference(
+        _f32(a), _ptr(a), _ptr(gate), c_ll(0 if gate is None else gate.stride(0)), _ptr(out), c_int(T), c_int(H2 // 2), c_int(pitch),
+        c_int(width), c_float(lam), c_float(factor), c_float(eps), _stream()), "map_difference")
+    return out
+
+
 def output_gate(x, gate, width: int):
     T, H, pitch = x.shape
     out = torch.empty(T, H * width, dtype=x.dtype, device=x.device)
@@ -609,9 +638,9 @@ def _f32(t: torch.Tensor):
     return c_int(1 if t.dtype == torch.float32 else 0)
 
 
-def embed_residual(ids, table, scale: float):
+def embed_residual(ids, table, scale: float, streams: int = 1):
     T, H = ids.numel(), table.shape[1]
-    out = torch.empty(T, H, dtype=torch.float32, device=table.device)
+    out = torch.empty(*((streams, T, H) if streams > 1 else (T, H)), dtype=torch.float32, device=table.device)
     _check(load().tgi_embed_residual(_f32(table), _ptr(ids), _ptr(table), _ptr(out), c_int(T), c_int(H),
                                      c_int(table.shape[0]), c_float(scale), _stream()), "embed_residual")
     return out
@@ -637,6 +666,50 @@ def residual_norm(delta, residual, weight, eps, rows=None, keep: bool = True, sc
                                     c_float(eps), c_float(scale),
                                     c_float(1.0 if unit_offset else 0.0), _stream()), "residual_norm")
     return (out, res) if weight2 is None else (out, out2, res)
+
+
+def _conv_args(conv, H: int, dtype):
+    if conv is None:
+        return [_ptr(None)] * 5 + [c_int(0)] * 3
+    taps = conv.state.shape[1] + 1
+    assert conv.weights.is_contiguous() and conv.weights.dtype == torch.float32 and tuple(conv.weights.shape) == (taps, H)
+    assert conv.state.is_contiguous() and conv.state.shape[2] == H and conv.state.dtype == dtype
+    return [*map(_ptr, (conv.weights, conv.cu, conv.kv_lens, conv.state_slots, conv.state)), c_int(conv.kv_lens.shape[0]),
+            c_int(taps), c_int(conv.state.shape[0])]
+
+
+def stream_step(delta, post, residual, weight, eps, rows=None, keep: bool = True, gain: float = 1.0, average=None, streams=None,
+                conv=None):
+    T, H = residual.shape
+    n = T if rows is None else rows.shape[0]
+    out = torch.empty(n, H, dtype=weight.dtype, device=residual.device)
+    changed = delta is not None or average is not None or rows is not None
+    res = dst = torch.empty(n, H, dtype=torch.float32, device=residual.device) if keep and changed else None
+    if keep and not changed:
+        res = residual
+    assert residual.dtype == torch.float32 and residual.is_contiguous()
+    assert delta is None or (delta.dtype == weight.dtype and delta.is_contiguous() and delta.shape == residual.shape)
+    assert post is None or (post.dtype == weight.dtype and post.shape == (H,))
+    index = 0
+    if average is None:
+        streams = None
+    else:
+        index = average.shape[0] - 1
+        assert average.dtype == torch.float32 and streams.dtype == torch.float32 and streams.is_contiguous()
+        assert streams.shape[1:] == residual.shape and index < streams.shape[0]
+    _check(load().tgi_stream_step(
+        _f32(weight), _ptr(delta), _ptr(post), _ptr(residual), _ptr(rows), _ptr(streams), _ptr(average), c_ll(T * H), c_int(index),
+        c_int(1 if rows is None else 0), _ptr(weight), c_float(gain), _ptr(out), _ptr(dst), c_int(n), c_int(H), c_float(eps),
+        *_conv_args(conv, H, weight.dtype), _stream()), "stream_step")
+    return out, res
+
+
+def input_conv(x, conv):
+    out = torch.empty_like(x)
+    assert x.is_contiguous()
+    _check(load().tgi_input_conv(_f32(x), _ptr(x), _ptr(out), c_int(x.shape[0]), c_int(x.shape[1]), *_conv_args(conv, x.shape[1], x.dtype),
+                                 _stream()), "input_conv")
+    return out
 
 
 def activation(x, act: str):
@@ -711,13 +784,15 @@ def delta_scan(q, k, v, g, beta, qk, cu, kv_lens, state_slots, state, dim: int, 
     return out
 
 
-def decay_scan(proj, offs, decay, cu, kv_lens, state_slots, state, heads: int, dim: int, vdim: int, max_q: int):
+def decay_scan(proj, offs, decay, cu, kv_lens, state_slots, state, heads: int, dim: int, vdim: int, max_q: int,
+               act: str = "silu", k_scale: float = 1.0):
     T = proj.shape[0]
     out = torch.empty(T, heads, vdim, dtype=torch.float32, device=proj.device)
     _check(load().tgi_decay_scan(
         _f32(proj), _ptr(proj), c_ll(proj.stride(0)), c_int(offs[0]), c_int(offs[1]), c_int(offs[2]), _ptr(decay), _ptr(cu),
         _ptr(kv_lens), _ptr(state_slots), _ptr(state), _ptr(out), c_int(kv_lens.shape[0]), c_int(max_q),
-        c_int(state.shape[0]), c_int(heads), c_int(dim), c_int(state.shape[3]), c_int(vdim), _stream()), "decay_scan")
+        c_int(state.shape[0]), c_int(heads), c_int(dim), c_int(state.shape[3]), c_int(vdim), c_int({"silu": 1, "": 0}[act]),
+        c_float(k_scale), _stream()), "decay_scan")
     return out
 
 

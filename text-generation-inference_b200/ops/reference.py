@@ -130,6 +130,7 @@ def paged_attention(
     horizon: Optional[torch.Tensor] = None,
     chunk: int = 0,
     sink=None,
+    keep: int = 0,
 ) -> torch.Tensor:
     """Causal attention of ragged queries over paged KV (covers prefill, chunked prefill and decode).
     ``horizon[t]`` (optional) replaces the causal limit of query row ``t`` by a later position.  With ``chunk`` a row
@@ -180,6 +181,8 @@ def paged_attention(
             mask &= kpos > qpos - window
         if chunk > 0:
             mask &= torch.div(kpos, chunk, rounding_mode="floor") == torch.div(qpos, chunk, rounding_mode="floor")
+        if keep > 0:
+            mask |= (kpos < keep) & (kpos <= limit)
         scores = scores.masked_fill(~mask.unsqueeze(0), float("-inf"))
         if sink is not None and sink is not False:
             extra = scores.new_zeros(Hq) if sink is True else sink.float()
@@ -372,8 +375,33 @@ def moe_experts(
 
 
 # ---- token mixers of hybrid decoders -------------------------------------------------------------
-def embed_residual(ids, table, scale: float = 1.0):
-    return F.embedding(ids.long(), table).float() * scale
+def embed_residual(ids, table, scale: float = 1.0, streams: int = 1):
+    x = F.embedding(ids.long(), table).float() * scale
+    return x if streams == 1 else torch.cat([x.unsqueeze(0), x.new_zeros(streams - 1, *x.shape)])
+
+
+def stream_step(delta, post, residual, weight, eps: float, rows=None, keep: bool = True, gain: float = 1.0, average=None, streams=None,
+                conv=None):
+    r = residual
+    if delta is not None:
+        r = r + (delta.float() if post is None else _row_rms(delta, post.float(), eps))
+    if average is not None:
+        n = average.shape[0]
+        r = torch.einsum("n,nth->th", average, torch.cat([streams[:n - 1], r.unsqueeze(0)])) if rows is not None else _averaged(streams, r, average)
+    if rows is not None:
+        r = r[rows.long()]
+    out = (_row_rms(r, weight.float(), eps) * gain).to(weight.dtype)
+    return (out if conv is None else input_conv(out, conv)), r if keep else None
+
+
+def _averaged(streams, r, average):
+    n = average.shape[0]
+    streams[n - 1] = r
+    return torch.einsum("n,nth->th", average, streams[:n])
+
+
+def input_conv(x, conv):
+    return _conv_rows(x, (0,), (x.shape[1],), conv.weights, conv.cu, conv.kv_lens, conv.state_slots, conv.state).to(x.dtype)
 
 
 def residual_norm(delta, residual, weight, eps: float, rows=None, keep: bool = True, scale: float = 1.0,
@@ -478,27 +506,53 @@ def row_norm_store(proj, offs, positions, slots, k_cache, v_cache, q_weight, k_w
     return F.pad(q.view(T, num_heads, dim), (0, width - dim)).to(proj.dtype)
 
 
+def map_store(proj, offs, slots, k_cache, v_cache, num_heads: int, num_kv_heads: int, dim: int, vdim: int):
+    T = proj.shape[0]
+    part = lambda i, n: proj[:, offs[i]:offs[i] + n]
+    _store_rows(k_cache, slots, part(1, num_kv_heads * 2 * dim).reshape(T, num_kv_heads, 2 * dim))
+    _store_rows(v_cache, slots, part(2, num_kv_heads * vdim).reshape(T, num_kv_heads, vdim))
+    q = proj.new_zeros(T, num_heads, 2, k_cache.shape[3])
+    maps = part(0, num_heads * 2 * dim).reshape(T, num_heads, 2, dim)
+    for m in range(2):
+        q[:, :, m, m * dim:(m + 1) * dim] = maps[:, :, m]
+    return q.view(T, 2 * num_heads, -1)
+
+
+def map_difference(a, gate, lam: float, factor: float, eps: float, width: int):
+    T = a.shape[0]
+    x = a[..., :width].float()
+    y = _row_rms(x[:, 0::2] - lam * x[:, 1::2], factor, eps)
+    if gate is not None:
+        y = y * torch.sigmoid(gate.float()).unsqueeze(2)
+    return y.reshape(T, -1).to(a.dtype)
+
+
 def output_gate(x, gate, width: int):
     T = x.shape[0]
     return (x[:, :, :width].reshape(T, -1).float() * torch.sigmoid(gate.float())).to(x.dtype)
 
 
 def latent_store(proj, off_c, weight, eps: float, positions, cos_sin, slots, pages, q, off_rot, rank, rot, heads, dim,
-                 q_full=None):
+                 q_full=None, queries: bool = True, q_latent=None, width=None):
     assert q_full is None
     T = proj.shape[0]
-    _store_rows(pages, slots, _row_rms(proj[:, off_c:off_c + rank], weight, eps).unsqueeze(1))
-    if rot:
-        cs = cos_sin[positions.long()]
-        turn = lambda x: rotate(x.float(), cs[:, :rot // 2], cs[:, rot // 2:], rot, False)
+    cs = cos_sin[positions.long()]
+    turn = lambda x: rotate(x.float(), cs[:, :rot // 2], cs[:, rot // 2:], rot, False)
+    if pages is not None:
+        _store_rows(pages, slots, _row_rms(proj[:, off_c:off_c + rank], weight, eps).unsqueeze(1))
+    if pages is not None and rot:
         _store_rows(pages, slots, turn(proj[:, off_c + rank:off_c + rank + rot].unsqueeze(1)), off_rot)
+    if q_latent is not None:
+        off, w, out = q_latent
+        out.copy_(F.pad(_row_rms(proj[:, off:off + w.shape[0]], w, eps), (0, out.shape[1] - w.shape[0])))
+    if queries and rot:
         q[:, :, off_rot:off_rot + rot] = turn(proj[:, :heads * (dim + rot)].reshape(T, heads, dim + rot)[..., dim:]).to(q.dtype)
 
 
 def latent_attention(q, pages, rank, block_tables, cu_seqlens_q, kv_lens, scale: float, window: int = -1, max_q=None, max_kv=None,
-                     gate=None, elsewhere=None):
+                     gate=None, elsewhere=None, sink=None):
     assert elsewhere is None
-    o = paged_attention(q, pages, pages[..., :rank].contiguous(), block_tables, cu_seqlens_q, kv_lens, scale, window)
+    o = paged_attention(q, pages, pages[..., :rank].contiguous(), block_tables, cu_seqlens_q, kv_lens, scale, window, sink=sink)
     return o if gate is None else (o.float() * torch.sigmoid(gate.float()).unsqueeze(2)).to(o.dtype)
 
 
@@ -535,10 +589,13 @@ def delta_scan(q, k, v, g, beta, qk, cu, kv_lens, state_slots, state, dim: int, 
     return out
 
 
-def decay_scan(proj, offs, decay, cu, kv_lens, state_slots, state, heads: int, dim: int, vdim: int, max_q: int):
+def decay_scan(proj, offs, decay, cu, kv_lens, state_slots, state, heads: int, dim: int, vdim: int, max_q: int,
+               act: str = "silu", k_scale: float = 1.0):
     T = proj.shape[0]
-    q, k = (F.silu(proj[:, o:o + heads * dim].float()).view(T, heads, dim) for o in offs[:2])
-    v = F.silu(proj[:, offs[2]:offs[2] + heads * vdim].float()).view(T, heads, vdim)
+    fn = F.silu if act else (lambda x: x)
+    q, k = (fn(proj[:, o:o + heads * dim].float()).reshape(T, heads, dim) for o in offs[:2])
+    v = fn(proj[:, offs[2]:offs[2] + heads * vdim].float()).reshape(T, heads, vdim)
+    k = k * k_scale
     pad = (0, state.shape[3] - dim)
     q, k = F.pad(q, pad), F.pad(k, pad)
     out = torch.zeros(T, heads, vdim)
