@@ -46,8 +46,8 @@ def parse_args():
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="b200", choices=["b200", "reference"])
     ap.add_argument("--model", default="llama70b-fp8", choices=["llama70b-fp8", "llama8b-bf16", "mixtral-bf16", "tiny", "fuzuvik-bf16",
-                                                                "kipedra-bf16", "gisilix-bf16"],
-                    help="fuzuvik-bf16, kipedra-bf16, gisilix-bf16: prefill / decode rates and kernels of a decoder whose "
+                                                                "kipedra-bf16", "gisilix-bf16", "sobivik-bf16"],
+                    help="fuzuvik-bf16, kipedra-bf16, gisilix-bf16, sobivik-bf16: prefill / decode rates and kernels of a decoder whose "
                          "layers differ beside its closest relative, a Llama, Fuzuvik or DeepSeek shape (one GPU)")
     ap.add_argument("--concurrency", type=int, default=256)
     ap.add_argument("--prompt-len", type=int, default=1024)
@@ -172,7 +172,7 @@ def main():
     args = parse_args()
     if args.impl == "reference":
         return reference_main(args)
-    if args.model in ("fuzuvik-bf16", "kipedra-bf16", "gisilix-bf16"):
+    if args.model in ("fuzuvik-bf16", "kipedra-bf16", "gisilix-bf16", "sobivik-bf16"):
         from tgi_b200.ops import bench_hybrid
 
         return bench_hybrid.run(args, ClockSampler)

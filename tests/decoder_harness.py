@@ -39,14 +39,18 @@ def replay_for(ck, be, max_tokens):
     return Replay(runner_for(ck, be), max_tokens)
 
 
-def check(got, want, dtype, close_calls=False):
+def check(got, want, dtype, close_calls=False, normed_blocks=0.0):
     """Per-position error (mean over the vocabulary taken off) against the spread of the expected logits.  ``close_calls``:
-    16-bit roundings may tip an expert choice at some position, so a few of them may be further off."""
+    16-bit roundings may tip an expert choice at some position, so a few of them may be further off.  ``normed_blocks``: norms of
+    what a block (or a head) returns enlarge 16-bit roundings where it is small, at some positions up to this bound."""
     d = got.double() - want
     d = d - d.mean(-1, keepdim=True)
     err = d.pow(2).mean(-1).sqrt() / want.std()
     if close_calls and dtype != torch.float32:
         assert err.numel() < 10 or err.quantile(0.75).item() < 0.04, err
+        return
+    if normed_blocks and dtype != torch.float32:
+        assert err.max().item() < normed_blocks and (err.numel() < 30 or err.quantile(0.9).item() < 0.05), err
         return
     assert err.max().item() < (2e-5 if dtype == torch.float32 else 0.04), err
 

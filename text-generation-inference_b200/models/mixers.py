@@ -320,7 +320,7 @@ class LatentAttention(Mixer):
         if s.q_rank:
             self.q_norm = self.f32("dq.norm")
             self.uq = TensorParallelColumnLinear(FastLinear(stack_rows([self._rows("uq")])[0]))
-            self.q_cols = _up(s.q_rank)
+            self.q_cols = self.uq.linear.weight.shape[1]
         self.sink = self.f32("sink") if s.learned_sink else None
         self.off_rot, self.width = ops.latent_layout(s.kv_rank, s.rot_dims, self.dtype, self.device)
         pad = (0, self.off_rot - s.kv_rank)

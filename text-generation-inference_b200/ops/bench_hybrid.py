@@ -2,8 +2,8 @@
 active parameters per token, and the kernels of both against their rooflines.
 
 ``python bench.py --model fuzuvik-bf16`` (beside a Llama shape), ``--model kipedra-bf16`` (beside a Fuzuvik shape; expert
-kernels beside those of gated experts) and ``--model gisilix-bf16`` (beside a DeepSeek shape, ``bench_latent``) print one JSON
-line.  Weights are random; token rates are timed with CUDA
+kernels beside those of gated experts), ``--model gisilix-bf16`` (beside a DeepSeek shape, ``bench_latent``) and ``--model
+sobivik-bf16`` (beside a Fuzuvik shape, ``bench_sobivik``) print one JSON line.  Weights are random; token rates are timed with CUDA
 events around the model's forward (prefill) and around replays of its decode graph.  Kernels are timed one by one
 with the L2 flushed in front of every launch; a roofline is the larger of bytes over the measured copy bandwidth and
 FLOPs over the measured rate of the unit that does them (bf16 tensor cores, or fp32 FMA for the state recurrences).
@@ -82,6 +82,7 @@ def make_runner(cfg: dict, dev):
 
         kw = dict(dtype=torch.bfloat16, device=str(dev))
         tensors = {"Kipedra": lambda: syn.kipedra_state_dict(cfg, **kw), "Gisilix": lambda: syn.gisilix_state_dict(cfg, **kw),
+                   "Sobivik": lambda: syn.sobivik_state_dict(cfg, **kw),
                    "Fuzuvik": lambda: syn.fuzuvik_state_dict(cfg, rank=128, **kw),
                    None: lambda: deepseek_tensors(cfg, dev)}[cfg.get("architecture")]()
         w = syn.DictWeights(tensors, dev, torch.bfloat16, bare_names=bool(cfg.get("architecture")))
@@ -383,6 +384,7 @@ def kipedra_rows(dev, width: int, window: int, prefill, decode) -> list:
 def run(args, clock_sampler) -> int:
     from . import cuda as K
     from .bench_latent import deepseek_like, gisilix_like, gisilix_rows
+    from .bench_sobivik import fuzuvik_relative, sobivik_like, sobivik_rows
 
     dev = torch.device("cuda", 0)
     torch.cuda.set_device(dev)
@@ -395,6 +397,7 @@ def run(args, clock_sampler) -> int:
         # 256 x 2048 tokens of keys and values per head do not fit beside the weights
         "gisilix-bf16": ("gisilix", gisilix_like, "deepseek", lambda w, n, v, s: deepseek_like(w, n, v), gisilix_rows, 1024,
                          [(16, 2048), (64, 2048)], [(256, 2048)]),
+        "sobivik-bf16": ("sobivik", sobivik_like, "fuzuvik", fuzuvik_relative, sobivik_rows, 1024, [(16, 2048), (256, 2048)], []),
     }[args.model]
     sampler = clock_sampler(0)
     sampler.start()

@@ -9,6 +9,8 @@
 #include <cuda_runtime.h>
 #include <stdint.h>
 
+#include <type_traits>
+
 #include "launch.cuh"
 #include "mixer_util.cuh"
 
@@ -57,62 +59,116 @@ __device__ __forceinline__ T* conv_slot(const InputConv& c, int t, int H, bool& 
   return slot >= 0 && slot < c.num_slots ? static_cast<T*>(c.state) + static_cast<size_t>(slot) * (c.taps - 1) * H : nullptr;
 }
 
-template <typename T, int VPT>
-__global__ void __launch_bounds__(512)
+// four elements as they lie in memory: loaded early, converted when they are needed
+template <typename T>
+struct Quad;
+template <>
+struct Quad<float> {
+  using type = float4;
+  static __device__ __forceinline__ float4 value(float4 v) { return v; }
+};
+template <>
+struct Quad<bf16> {
+  using type = uint2;
+  static __device__ __forceinline__ float4 value(uint2 u) { return load4(reinterpret_cast<const bf16*>(&u)); }
+};
+// sum over the block with one barrier; `red` holds one float per warp and is used for one sum only
+__device__ __forceinline__ float block_sum_once(float v, float* red) {
+  v = warp_sum(v);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float t = 0.f;
+  for (int w = 0; w < static_cast<int>(blockDim.x >> 5); ++w) t += red[w];
+  return t;
+}
+__device__ __forceinline__ float4 fma4(float f, float4 a, float4 b) {
+  return make_float4(fmaf(f, a.x, b.x), fmaf(f, a.y, b.y), fmaf(f, a.z, b.z), fmaf(f, a.w, b.w));
+}
+__device__ __forceinline__ float4 fma4(float4 f, float4 a, float4 b) {
+  return make_float4(fmaf(f.x, a.x, b.x), fmaf(f.y, a.y, b.y), fmaf(f.z, a.z, b.z), fmaf(f.w, a.w, b.w));
+}
+__device__ __forceinline__ float square4(float4 a) { return a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w; }
+
+// CONV: most taps of the input convolution, 0: there is none.  AVG: with the weighted sum (VPT > 0).  A step of single tokens
+// waits for latencies, so all it reads is asked for at the start; a prompt's steps want many rows in flight: two blocks of 512
+// threads per SM, 8192 x 4096: 93 / 197 us (without / with a sum of five), 168 / 296 with one.
+template <typename T, int VPT, int CONV, bool AVG>
+__global__ void __launch_bounds__(CONV > 0 ? 1024 : 512, CONV > 0 ? 1 : 2)
 stream_step_kernel(const StreamStep<T> p) {
   tgi::pdl_wait();
   tgi::pdl_trigger();
-  __shared__ float red[33];
+  __shared__ float red[2][33];
   extern __shared__ float held[];                          // VPT == 0: [H]
   const int row = p.rows != nullptr ? p.rows[blockIdx.x] : blockIdx.x, H = p.H;
   const size_t in = static_cast<size_t>(row) * H, ob = static_cast<size_t>(blockIdx.x) * H;
   T* st = nullptr;
   bool fresh = true;
-  if (p.conv.w != nullptr) st = conv_slot<T>(p.conv, row, H, fresh);
   if constexpr (VPT > 0) {
-    float4 d[VPT], x[VPT];
-    float ss = 0.f;
+    using Raw = typename Quad<T>::type;
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
     auto col = [&](int i) { return static_cast<int>(threadIdx.x + i * blockDim.x) * 4; };
+    auto raw = [&](const T* src) { return *reinterpret_cast<const Raw*>(src); };
+    // everything a column needs is on its way before the first sum
+    float4 x[VPT];
+    Raw d[VPT], post[VPT], w[VPT], past[CONV > 1 ? VPT : 1][CONV > 1 ? CONV - 1 : 1];
+    float ss = 0.f;
 #pragma unroll
     for (int i = 0; i < VPT; ++i) {
       const int c = col(i);
-      d[i] = x[i] = make_float4(0.f, 0.f, 0.f, 0.f);
       if (c < H) {
         x[i] = *reinterpret_cast<const float4*>(p.residual + in + c);
-        if (p.delta != nullptr) {
-          d[i] = load4(p.delta + in + c);
-          ss += d[i].x * d[i].x + d[i].y * d[i].y + d[i].z * d[i].z + d[i].w * d[i].w;
+        if (p.delta != nullptr) d[i] = raw(p.delta + in + c);
+        if constexpr (CONV > 0) {
+          w[i] = raw(p.w + c);
+          if (p.post != nullptr) post[i] = raw(p.post + c);
+          for (int j = 0; j < p.conv.taps; ++j)            // wanted last
+            asm volatile("prefetch.global.L2 [%0];" ::"l"(p.conv.w + static_cast<size_t>(j) * H + c));
         }
       }
     }
-    // the earlier results are on their way while the block sums up
-    float4 sum[VPT];
-    if (p.streams != nullptr) {
+    if constexpr (CONV > 0) {
+      st = conv_slot<T>(p.conv, row, H, fresh);
+      if constexpr (CONV > 1) {
+        if (st != nullptr && !fresh) {
 #pragma unroll
-      for (int i = 0; i < VPT; ++i) {
-        const int c = col(i);
-        sum[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (c < H) {
-          const float* src = p.streams + in + c;
-#pragma unroll 4
-          for (int j = 0; j < p.index; ++j) {
-            const float4 e = *reinterpret_cast<const float4*>(src + j * p.pitch);
-            const float f = p.dw[j];
-            sum[i].x = fmaf(f, e.x, sum[i].x); sum[i].y = fmaf(f, e.y, sum[i].y);
-            sum[i].z = fmaf(f, e.z, sum[i].z); sum[i].w = fmaf(f, e.w, sum[i].w);
+          for (int i = 0; i < VPT; ++i) {
+#pragma unroll
+            for (int j = 0; j < CONV - 1; ++j)
+              if (j < p.conv.taps - 1 && col(i) < H) past[i][j] = raw(st + static_cast<size_t>(j) * H + col(i));
           }
         }
       }
     }
-    if (p.delta != nullptr) {
-      const float inv = p.post != nullptr ? 1.f / sqrtf(block_sum(ss, red) / H + p.eps) : 1.f;
+    float4 sum[AVG ? VPT : 1];
+    if constexpr (AVG) {
 #pragma unroll
       for (int i = 0; i < VPT; ++i) {
         const int c = col(i);
-        if (c >= H) continue;
-        const float4 g = p.post != nullptr ? load4(p.post + c) : make_float4(1.f, 1.f, 1.f, 1.f);
-        x[i].x = fmaf(d[i].x * inv, g.x, x[i].x); x[i].y = fmaf(d[i].y * inv, g.y, x[i].y);
-        x[i].z = fmaf(d[i].z * inv, g.z, x[i].z); x[i].w = fmaf(d[i].w * inv, g.w, x[i].w);
+        sum[i] = zero;
+        if (c < H) {
+          const float* src = p.streams + in + c;
+#pragma unroll 4
+          for (int j = 0; j < p.index; ++j) sum[i] = fma4(p.dw[j], *reinterpret_cast<const float4*>(src + j * p.pitch), sum[i]);
+        }
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = col(i);
+      if (c < H && p.delta != nullptr) ss += square4(Quad<T>::value(d[i]));
+    }
+    if (p.delta != nullptr) {
+      const float inv = p.post != nullptr ? 1.f / sqrtf(block_sum_once(ss, red[0]) / H + p.eps) : 1.f;
+#pragma unroll
+      for (int i = 0; i < VPT; ++i) {
+        if (col(i) >= H) continue;
+        float4 v = Quad<T>::value(d[i]);
+        if (p.post != nullptr) {
+          v = make_float4(v.x * inv, v.y * inv, v.z * inv, v.w * inv);
+          x[i] = fma4(v, Quad<T>::value(CONV > 0 ? post[i] : raw(p.post + col(i))), x[i]);
+        } else {
+          x[i] = make_float4(x[i].x + v.x, x[i].y + v.y, x[i].z + v.z, x[i].w + v.w);
+        }
       }
     }
     ss = 0.f;
@@ -120,56 +176,52 @@ stream_step_kernel(const StreamStep<T> p) {
     for (int i = 0; i < VPT; ++i) {
       const int c = col(i);
       if (c >= H) continue;
-      if (p.streams != nullptr) {
+      if constexpr (AVG) {
         if (p.keep) store4(p.streams + p.index * p.pitch + in + c, x[i]);
-        const float f = p.dw[p.index];
-        x[i] = make_float4(fmaf(f, x[i].x, sum[i].x), fmaf(f, x[i].y, sum[i].y), fmaf(f, x[i].z, sum[i].z), fmaf(f, x[i].w, sum[i].w));
+        x[i] = fma4(p.dw[p.index], x[i], sum[i]);
       }
       if (p.res_out != nullptr) store4(p.res_out + ob + c, x[i]);
-      ss += x[i].x * x[i].x + x[i].y * x[i].y + x[i].z * x[i].z + x[i].w * x[i].w;
+      ss += square4(x[i]);
     }
-    const float inv = p.gain / sqrtf(block_sum(ss, red) / H + p.eps);
+    const float inv = p.gain / sqrtf(block_sum_once(ss, red[1]) / H + p.eps);
 #pragma unroll
     for (int i = 0; i < VPT; ++i) {
       const int c = col(i);
       if (c >= H) continue;
-      const float4 g = load4(p.w + c);
+      const float4 g = Quad<T>::value(CONV > 0 ? w[i] : raw(p.w + c));
       float4 y = make_float4(x[i].x * inv * g.x, x[i].y * inv * g.y, x[i].z * inv * g.z, x[i].w * inv * g.w);
-      if (p.conv.w != nullptr) {
+      if constexpr (CONV > 0) {
         // the input as it is kept, so that it counts the same now and as a past one
-        T h[4];
-        put(h, y.x); put(h + 1, y.y); put(h + 2, y.z); put(h + 3, y.w);
-        const float4 own = make_float4(to_f(h[0]), to_f(h[1]), to_f(h[2]), to_f(h[3]));
+        Raw own;
+        store4(reinterpret_cast<T*>(&own), y);
         const int taps = p.conv.taps;
-        y = make_float4(0.f, 0.f, 0.f, 0.f);
-        float4 past[kMaxTaps - 1];                         // loaded together: nothing waits for the one before
+        auto tap = [&](int j) { return *reinterpret_cast<const float4*>(p.conv.w + static_cast<size_t>(j) * H + c); };
+        y = zero;
+        if constexpr (CONV > 1) {
+          const bool old = st != nullptr && !fresh;
 #pragma unroll
-        for (int j = 0; j < kMaxTaps - 1; ++j)
-          past[j] = j < taps - 1 && st != nullptr && !fresh ? load4(st + static_cast<size_t>(j) * H + c) : make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll
-        for (int j = 0; j < kMaxTaps; ++j) {
-          if (j >= taps) break;
-          const float4 f = *reinterpret_cast<const float4*>(p.conv.w + static_cast<size_t>(j) * H + c);
-          const float4 v = j < taps - 1 ? past[j < kMaxTaps - 1 ? j : 0] : own;
-          y.x = fmaf(f.x, v.x, y.x); y.y = fmaf(f.y, v.y, y.y); y.z = fmaf(f.z, v.z, y.z); y.w = fmaf(f.w, v.w, y.w);
-        }
-        if (st != nullptr) {
-#pragma unroll
-          for (int j = 1; j < kMaxTaps; ++j) {
-            if (j >= taps) break;
-            store4(st + static_cast<size_t>(j - 1) * H + c, j < taps - 1 ? past[j < kMaxTaps - 1 ? j : 0] : own);
+          for (int j = 0; j < CONV - 1; ++j) {
+            if (j >= taps - 1) break;
+            if (old) y = fma4(tap(j), Quad<T>::value(past[i][j]), y);
+            if (st != nullptr && j > 0) {
+              if (old) *reinterpret_cast<Raw*>(st + static_cast<size_t>(j - 1) * H + c) = past[i][j];
+              else store4(st + static_cast<size_t>(j - 1) * H + c, zero);
+            }
           }
+          if (st != nullptr && taps > 1) *reinterpret_cast<Raw*>(st + static_cast<size_t>(taps - 2) * H + c) = own;
         }
+        y = fma4(tap(taps - 1), Quad<T>::value(own), y);
       }
       store4(p.out + ob + c, y);
     }
   } else {
     const int first = threadIdx.x, step = blockDim.x;
+    if (p.conv.w != nullptr) st = conv_slot<T>(p.conv, row, H, fresh);
     float inv = 1.f;
     if (p.delta != nullptr && p.post != nullptr) {
       float ss = 0.f;
       for (int c = first; c < H; c += step) ss = fmaf(to_f(p.delta[in + c]), to_f(p.delta[in + c]), ss);
-      inv = 1.f / sqrtf(block_sum(ss, red) / H + p.eps);
+      inv = 1.f / sqrtf(block_sum(ss, red[0]) / H + p.eps);
     }
     float ss = 0.f;
     for (int c = first; c < H; c += step) {
@@ -185,7 +237,7 @@ stream_step_kernel(const StreamStep<T> p) {
       held[c] = x;
       ss = fmaf(x, x, ss);
     }
-    inv = p.gain / sqrtf(block_sum(ss, red) / H + p.eps);
+    inv = p.gain / sqrtf(block_sum(ss, red[0]) / H + p.eps);
     for (int c = first; c < H; c += step) {
       float y = held[c] * inv * to_f(p.w[c]);
       if (p.conv.w != nullptr) {
@@ -354,22 +406,27 @@ int done() { return cudaGetLastError() == cudaSuccess ? 0 : -3; }
 template <typename T>
 int stream_step(const StreamStep<T>& p, int n, cudaStream_t stream) {
   const int H = p.H, vecs = H / 4;
-  if (H % 4 == 0 && vecs <= 8 * 512 && (p.conv.w == nullptr || p.conv.taps <= kMaxTaps)) {
-    int threads = vecs >= 1024 ? 512 : ((vecs + 31) / 32) * 32;
-    if (threads > 256 && vecs <= 1024) threads = 256;
+  if (H % 4 == 0 && vecs <= 2048 && (p.conv.w == nullptr || p.conv.taps <= kMaxTaps)) {
+    const int most = p.conv.w != nullptr ? 1024 : 512, threads = vecs >= most ? most : ((vecs + 31) / 32) * 32;
     const int vpt = (vecs + threads - 1) / threads;
-    auto go = [&](auto kern) { tgi::launch(kern, dim3(n), dim3(threads), 0, stream, p); };
-    if (vpt <= 1) go(stream_step_kernel<T, 1>);
-    else if (vpt <= 2) go(stream_step_kernel<T, 2>);
-    else if (vpt <= 4) go(stream_step_kernel<T, 4>);
-    else go(stream_step_kernel<T, 8>);
-    return done();
+    auto go = [&](auto kern) {
+      tgi::launch(kern, dim3(n), dim3(threads), 0, stream, p);
+      return done();
+    };
+    auto pick = [&](auto avg) {
+      constexpr bool A = decltype(avg)::value;
+      if (p.conv.w == nullptr)
+        return vpt <= 1 ? go(stream_step_kernel<T, 1, 0, A>) : vpt <= 2 ? go(stream_step_kernel<T, 2, 0, A>) : go(stream_step_kernel<T, 4, 0, A>);
+      if (p.conv.taps <= 4) return vpt <= 1 ? go(stream_step_kernel<T, 1, 4, A>) : go(stream_step_kernel<T, 2, 4, A>);
+      return vpt <= 1 ? go(stream_step_kernel<T, 1, kMaxTaps, A>) : go(stream_step_kernel<T, 2, kMaxTaps, A>);
+    };
+    return p.streams != nullptr ? pick(std::true_type()) : pick(std::false_type());
   }
   const size_t smem = static_cast<size_t>(H) * 4;
   if (smem > 200 * 1024) return -12;
-  if (smem > 48 * 1024 && cudaFuncSetAttribute(stream_step_kernel<T, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)) != cudaSuccess)
+  if (smem > 48 * 1024 && cudaFuncSetAttribute(stream_step_kernel<T, 0, 1, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)) != cudaSuccess)
     return -2;
-  tgi::launch(stream_step_kernel<T, 0>, dim3(n), dim3(256), smem, stream, p);
+  tgi::launch(stream_step_kernel<T, 0, 1, true>, dim3(n), dim3(256), smem, stream, p);
   return done();
 }
 

@@ -532,3 +532,65 @@ def gisilix_state_dict(cfg: dict, seed: int = 0, dtype=torch.float32, device: st
         if mlp.get("shared"):
             feed_forward(p + "mlp.shared.", mlp["shared"]["ff"])
     return sd
+
+
+# ---- Sobivik: layers normed on both sides, input convolutions, weighted sums over all results ---------------------------
+def sobivik_retention(heads=3, dim=24, vdim=20, decay=None, mlp=None) -> dict:
+    return {"type": "retention", "mlp": mlp, "mixer": {"heads": heads, "dim": dim, "vdim": vdim,
+                                                       "decay": decay or [1 - 2.0 ** -(2 + 2 * h) for h in range(heads)]}}
+
+
+def sobivik_latent(heads=4, dim=24, vdim=20, q_rank=32, kv_rank=40, rot_dim=8, window=24, base=1000.0, scaling=(4.0, 8.0, 1.0, 128),
+                   scale=None, mlp=None) -> dict:
+    """``scaling``: (factor, fast, slow, original length)."""
+    rot = {"base": base, "dims": rot_dim}
+    if scaling is not None:
+        rot["scaling"] = dict(zip(("factor", "fast", "slow", "original"), scaling))
+    return {"type": "latent_attention", "mlp": mlp,
+            "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "q_rank": q_rank, "kv_rank": kv_rank, "rot_dim": rot_dim,
+                      "mask": {"size": window}, "rot": rot, "scale": (dim + rot_dim) ** -0.5 if scale is None else scale}}
+
+
+def sobivik_attention(heads=4, kv_heads=2, dim=12, vdim=28, window=20, keep=3, diff=0.3, scale=None, mlp=None) -> dict:
+    return {"type": "attention", "mlp": mlp,
+            "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "diff": diff,
+                      "mask": {"size": window, "keep_first": keep}, "scale": dim ** -0.5 if scale is None else scale}}
+
+
+def sobivik_config(layers, width=80, vocab=203, eps=1e-5, taps=4, embed_scale=3.0, logit_scale=1.5) -> dict:
+    return {"architecture": "Sobivik", "width": width, "vocab": vocab, "norm": {"eps": eps}, "canon": {"taps": taps},
+            "embedding": {"scale": embed_scale}, "logit_scale": logit_scale, "layers": list(layers)}
+
+
+def sobivik_state_dict(cfg: dict, seed: int = 0, dtype=torch.float32, device: str = "cpu") -> Dict[str, torch.Tensor]:
+    """Random weights of a Sobivik shape."""
+    g = torch.Generator(device=device).manual_seed(seed)
+    W, sd = cfg["width"], {}
+
+    def rnd(*shape, std=None, mean=0.0):
+        std = shape[-1] ** -0.5 if std is None else std
+        return (mean + torch.randn(shape, generator=g, device=device) * std).to(dtype)
+
+    sd.update({"embed": rnd(cfg["vocab"], W, std=0.4), "head": rnd(cfg["vocab"], W), "final.norm": rnd(std=0.2, mean=1.2)})
+    for i, layer in enumerate(cfg["layers"]):
+        p, m, mlp = f"l{i}.", layer["mixer"], layer.get("mlp")
+        H, d, dv, mix = m["heads"], m["dim"], m["vdim"], f"l{i}.mix."
+        sd.update({p + "norm1": rnd(std=0.2, mean=1.0), p + "norm1b": rnd(std=0.2, mean=0.8), mix + "o": rnd(W, H * dv),
+                   p + "canon1": rnd(W, cfg["canon"]["taps"], std=0.3), p + "dwa": rnd(i + 2, std=0.25)})
+        sd[p + "dwa"][-1] += 0.8
+        if layer["type"] == "retention":
+            sd.update({mix + n: rnd(H * w, W) for n, w in (("q", d), ("k", d), ("v", dv), ("g", dv))})
+        elif layer["type"] == "latent_attention":
+            r, qr, rot = m["kv_rank"], m["q_rank"], m["rot_dim"]
+            sd.update({mix + "dq": rnd(qr, W), mix + "dq.norm": rnd(qr, std=0.2, mean=1.0), mix + "uq": rnd(H * (d + rot), qr),
+                       mix + "dkv": rnd(r + rot, W), mix + "dkv.norm": rnd(r, std=0.2, mean=1.0), mix + "uk": rnd(H * d, r),
+                       mix + "uv": rnd(H * dv, r), mix + "sink": rnd(H, std=1.5), mix + "g": rnd(H * dv, W)})
+        else:
+            G = m["kv_heads"]
+            sd.update({mix + "q": rnd(H * 2 * d, W), mix + "k": rnd(G * 2 * d, W), mix + "v": rnd(G * dv, W), mix + "g": rnd(H, W)})
+            sd.update({mix + n: rnd(d, std=0.8 * d ** -0.25) for n in ("lq1", "lk1", "lq2", "lk2")})
+        if mlp is not None:
+            ff = mlp["ff"]
+            sd.update({p + "norm2": rnd(std=0.2, mean=1.0), p + "norm2b": rnd(std=0.2, mean=0.8), p + "mlp.gate": rnd(ff, W),
+                       p + "mlp.up": rnd(ff, W), p + "mlp.down": rnd(W, ff)})
+    return sd
