@@ -441,3 +441,18 @@ def test_sliced_product(be):
     y = ops.linear(x.to(dev), m)
     close(y[:, 24:27], x.double() @ rnd(6, 3, 200).to(dt).double().t(), dt)
     assert (y[:, 5:8] == 0).all()
+
+
+def test_split_decode_workspace_of_several_head_sizes():
+    """Layers of different head sizes share the workspace of split decode steps: both its parts grow to what each needs, and
+    what captured steps may still use is not freed."""
+    from types import SimpleNamespace
+
+    from tgi_b200.ops.cuda import _attention_parts
+
+    st = SimpleNamespace(attn_part_o=None, attn_part_ml=None, kept={}, device=torch.device("cpu"))
+    first = _attention_parts(st, 24, 256)
+    o, ml = _attention_parts(st, 90, 64)                   # fewer outputs, more rows
+    assert o is first[0] and o.numel() >= 90 * 64 and ml.numel() >= 90 * 2 and ml is not first[1]
+    assert any(t is first[1] for t in st.kept["outgrown"])
+    assert _attention_parts(st, 90, 64)[1] is ml

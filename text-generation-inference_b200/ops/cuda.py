@@ -456,10 +456,7 @@ def paged_attention(q, k_cache, v_cache, block_tables, cu_seqlens_q, kv_lens, sc
             nsplit = lib.tgi_attn_decode_splits(B, Hkv, Hq // Hkv, max_kv, st.sm_count)
         if nsplit > 1:
             need = B * Hq * nsplit
-            if st.attn_part_o is None or st.attn_part_o.numel() < need * D:
-                st.attn_part_o = torch.empty(need * D, dtype=torch.float32, device=q.device)
-                st.attn_part_ml = torch.empty(need * 2, dtype=torch.float32, device=q.device)
-            part_o, part_ml = st.attn_part_o, st.attn_part_ml
+            part_o, part_ml = _attention_parts(st, need, D)
     else:
         nsplit = 1
     _check(lib.tgi_paged_attention_ex(
@@ -469,6 +466,18 @@ def paged_attention(q, k_cache, v_cache, block_tables, cu_seqlens_q, kv_lens, sc
         c_float(scale), c_float(softcap), c_int(window if window and window > 0 else -1), c_int(chunk),
         c_int(keep), _ptr(sink), c_int(nsplit), c_int(1 if fp8 else 0), _ptr(horizon), _stream()), "paged_attention")
     return out
+
+
+def _attention_parts(st, rows: int, D: int):
+    """Workspace of a split decode step: partial outputs and their maxima and sums, each as large as it has to be (layers of
+    other head sizes share them).  What captured steps use stays alive."""
+    for name, need in (("attn_part_o", rows * D), ("attn_part_ml", rows * 2)):
+        held = getattr(st, name)
+        if held is None or held.numel() < need:
+            if held is not None:
+                st.kept.setdefault("outgrown", []).append(held)
+            setattr(st, name, torch.empty(max(need, 2 * held.numel() if held is not None else 0), dtype=torch.float32, device=st.device))
+    return st.attn_part_o, st.attn_part_ml
 
 
 _ZERO_SINKS = {}
