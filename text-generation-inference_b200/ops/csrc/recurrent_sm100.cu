@@ -37,7 +37,9 @@ namespace {
 
 using bf16 = __nv_bfloat16;
 constexpr int kTile = 8;          // tokens per staged tile
-enum { kFixed = 0, kChannel = 1, kHead = 2 };       // fixed decay, delta rule with a decay per channel, per head
+// fixed decay (of SiLU'd vectors, of vectors as projected), delta rule with a decay per channel, per head
+enum { kFixed = 0, kChannel = 1, kHead = 2, kPlain = 3 };
+__host__ __device__ constexpr bool is_delta(int mode) { return mode == kChannel || mode == kHead; }
 constexpr int kThreads = 128;
 
 __device__ __forceinline__ float to_f(float x) { return x; }
@@ -51,7 +53,7 @@ __device__ __forceinline__ float silu_t<bf16>(float x) { return __fdividef(x, 1.
 struct ScanArgs {
   // delta rule: fp32 q, k [T, G, dimP], g [T, H, dimP] (one decay per head: [T, H]), v [T, H, vdim], beta [T, H], qk = q . k [T, G]
   const float *q, *k, *g, *v, *beta, *qk;
-  // linear attention: proj [T, ld] with q, k (H x dim) and v (H x vdim) at off_q, off_k, off_v (SiLU applied here if `silu`)
+  // linear attention: proj [T, ld] with q, k (H x dim) and v (H x vdim) at off_q, off_k, off_v (SiLU, if any, applied here)
   const void* proj;
   long long ld;
   int off_q, off_k, off_v;
@@ -63,7 +65,6 @@ struct ScanArgs {
   float* out;                     // [T, H, vdim]
   int num_slots, G, H, dim, dimP, vdim;
   int vec;                        // proj: heads may be read four elements at a time
-  int silu;                       // linear attention: q, k and v go through SiLU
   float k_scale;                  // linear attention: factor of k
 };
 
@@ -150,19 +151,18 @@ struct PairOf<bf16> {
     return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w));
   }
 };
-// SiLU where `on`
-template <typename T>
-__device__ __forceinline__ float act_t(float x, bool on) { return on ? silu_t<T>(x) : x; }
-// columns c .. c + 3 of a head after SiLU (where `on`) times f, zero past `dim`; `vec`: the four may be read at once
-template <typename T>
-__device__ __forceinline__ float4 load4_act(const T* p, int c, int dim, bool vec, bool on, float f) {
+template <typename T, int MODE>
+__device__ __forceinline__ float act_t(float x) { return MODE == kFixed ? silu_t<T>(x) : x; }
+// columns c .. c + 3 of a head after SiLU (if any) times f, zero past `dim`; `vec`: the four may be read at once
+template <typename T, int MODE>
+__device__ __forceinline__ float4 load4_act(const T* p, int c, int dim, bool vec, float f) {
   if (vec && c < dim) {
     const float4 x = raw4(p + c);
-    return make_float4(f * act_t<T>(x.x, on), f * act_t<T>(x.y, on), f * act_t<T>(x.z, on), f * act_t<T>(x.w, on));
+    return make_float4(f * act_t<T, MODE>(x.x), f * act_t<T, MODE>(x.y), f * act_t<T, MODE>(x.z), f * act_t<T, MODE>(x.w));
   }
   float v[4];
 #pragma unroll
-  for (int i = 0; i < 4; ++i) v[i] = c + i < dim ? f * act_t<T>(to_f(p[c + i]), on) : 0.f;
+  for (int i = 0; i < 4; ++i) v[i] = c + i < dim ? f * act_t<T, MODE>(to_f(p[c + i])) : 0.f;
   return make_float4(v[0], v[1], v[2], v[3]);
 }
 __device__ __forceinline__ float4 mul4(float4 a, float4 b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); }
@@ -191,7 +191,7 @@ struct ScanCfg {
 template <typename T, int MODE, bool VEC, int J, int L, int CN>
 __global__ void __launch_bounds__(kThreads)
 scan_kernel(ScanArgs p) {
-  constexpr bool DELTA = MODE != kFixed, WIDE = MODE == kChannel, HEAD = MODE == kHead;
+  constexpr bool DELTA = is_delta(MODE), WIDE = MODE == kChannel, HEAD = MODE == kHead;
   tgi::pdl_wait();
   tgi::pdl_trigger();
   extern __shared__ __align__(16) float smem[];
@@ -310,11 +310,9 @@ scan_kernel(ScanArgs p) {
             k[e] = PairOf<T>::value(k[e]);
             q[e] = PairOf<T>::value(q[e]);
           }
-          if (p.silu) {                                               // SiLU(0) = 0: absent tokens and channels stay 0
-            k[e] = make_float2(silu_t<T>(k[e].x), silu_t<T>(k[e].y));
-            q[e] = make_float2(silu_t<T>(q[e].x), silu_t<T>(q[e].y));
-          }
-          k[e] = make_float2(p.k_scale * k[e].x, p.k_scale * k[e].y);
+          k[e] = make_float2(act_t<T, MODE>(k[e].x), act_t<T, MODE>(k[e].y));    // SiLU(0) = 0: absent tokens and channels stay 0
+          q[e] = make_float2(act_t<T, MODE>(q[e].x), act_t<T, MODE>(q[e].y));
+          if (MODE == kPlain) k[e] = make_float2(p.k_scale * k[e].x, p.k_scale * k[e].y);
           g[e].x = g[e].y = e < cnt ? dec : 1.f;
         }
       }
@@ -366,7 +364,7 @@ scan_kernel(ScanArgs p) {
     }
 #pragma unroll
     for (int i = 0; i < NV; ++i)
-      d[S::kOffV + tid + i * kThreads] = DELTA ? rvf[DELTA ? i : 0] : act_t<T>(to_f(rv[DELTA ? 0 : i]), p.silu);
+      d[S::kOffV + tid + i * kThreads] = DELTA ? rvf[DELTA ? i : 0] : act_t<T, MODE>(to_f(rv[DELTA ? 0 : i]));
     if (DELTA && tid < kTile) d[S::kOffBeta + tid] = rb;
     if (HEAD && tid < kTile) d[S::kOffGate + tid] = rh;
   };
@@ -537,7 +535,7 @@ scan_kernel(ScanArgs p) {
 template <typename T, int MODE, int J, int CN>
 __global__ void __launch_bounds__(kThreads)
 step_kernel(ScanArgs p) {
-  constexpr bool DELTA = MODE != kFixed, HEAD = MODE == kHead;
+  constexpr bool DELTA = is_delta(MODE), HEAD = MODE == kHead;
   tgi::pdl_wait();
   tgi::pdl_trigger();
   const int b = blockIdx.z, h = blockIdx.y;
@@ -604,13 +602,13 @@ step_kernel(ScanArgs p) {
     // the head's k and q once per block (the state is on its way meanwhile)
     for (int i = threadIdx.x; i < 16 * J; i += kThreads) {
       const int c4 = (i % (8 * J)) * 4;
-      *reinterpret_cast<float4*>(kq_s + i * 4) = load4_act(row + (i < 8 * J ? p.off_k : p.off_q) + h * p.dim, c4, p.dim, p.vec,
-                                                                p.silu, i < 8 * J ? p.k_scale : 1.f);
+      *reinterpret_cast<float4*>(kq_s + i * 4) = load4_act<T, MODE>(row + (i < 8 * J ? p.off_k : p.off_q) + h * p.dim, c4, p.dim,
+                                                                         p.vec, MODE == kPlain && i < 8 * J ? p.k_scale : 1.f);
     }
     __syncthreads();
 #pragma unroll
     for (int c = 0; c < CN; ++c) {
-      v[c] = col + c < p.vdim ? act_t<T>(to_f(row[p.off_v + h * p.vdim + col + c]), p.silu) : 0.f;
+      v[c] = col + c < p.vdim ? act_t<T, MODE>(to_f(row[p.off_v + h * p.vdim + col + c])) : 0.f;
       o[c] = 0.f;
     }
 #pragma unroll
@@ -654,7 +652,7 @@ int launch_scan(const ScanArgs& p, int B, cudaStream_t stream) {
 
 template <typename T, int MODE, int J>
 int run(const ScanArgs& p, int B, int max_q, cudaStream_t stream) {
-  constexpr bool DELTA = MODE != kFixed;
+  constexpr bool DELTA = is_delta(MODE);
   if (max_q == 1) {
     constexpr int CN = J <= 4 ? 4 : 2;
     tgi::launch(step_kernel<T, MODE, J, CN>, dim3((p.vdim + 16 * CN - 1) / (16 * CN), p.H, B), dim3(kThreads), 0, stream, p);
@@ -715,19 +713,21 @@ int tgi_delta_scan(const float* q, const float* k, const float* g, const float* 
   return head_decay ? dispatch<float, kHead>(p, B, max_q, stream) : dispatch<float, kChannel>(p, B, max_q, stream);
 }
 
-// `silu`: q, k and v go through SiLU first; k is then multiplied by k_scale
+// `silu`: q, k and v go through SiLU (and k_scale is 1); otherwise k is multiplied by k_scale
 int tgi_decay_scan(int f32, const void* proj, long long ld, int off_q, int off_k, int off_v, const float* decay, const int* cu,
                    const int* kv_lens, const int* state_slots, float* state, float* out, int B, int max_q, int num_slots,
                    int H, int dim, int dimP, int vdim, int silu, float k_scale, cudaStream_t stream) {
   ScanArgs p{};
-  p.silu = silu; p.k_scale = k_scale;
+  if (silu && k_scale != 1.f) return -13;                   // no instance
+  p.k_scale = k_scale;
   p.proj = proj; p.ld = ld; p.off_q = off_q; p.off_k = off_k; p.off_v = off_v; p.decay = decay;
   p.cu = cu; p.kv_lens = kv_lens; p.state_slots = state_slots;
   p.state = state; p.out = out;
   p.num_slots = num_slots; p.G = H; p.H = H; p.dim = dim; p.dimP = dimP; p.vdim = vdim;
   p.vec = dim % 4 == 0 && ld % 4 == 0 && off_q % 4 == 0 && off_k % 4 == 0 &&
           reinterpret_cast<uintptr_t>(proj) % (f32 ? 16 : 8) == 0;
-  return f32 ? dispatch<float, kFixed>(p, B, max_q, stream) : dispatch<bf16, kFixed>(p, B, max_q, stream);
+  if (silu) return f32 ? dispatch<float, kFixed>(p, B, max_q, stream) : dispatch<bf16, kFixed>(p, B, max_q, stream);
+  return f32 ? dispatch<float, kPlain>(p, B, max_q, stream) : dispatch<bf16, kPlain>(p, B, max_q, stream);
 }
 
 }  // extern "C"
