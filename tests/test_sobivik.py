@@ -31,10 +31,10 @@ CONFIGS = {
         Lat(heads=8, dim=128, vdim=128, q_rank=96, kv_rank=512, rot_dim=64, window=70, base=5000.0, scaling=(3.0, 16.0, 1.0, 100), mlp=dense(200)),
         Att(heads=8, kv_heads=2, dim=64, vdim=128, window=40, keep=6, diff=0.5, mlp=dense(128)),
         Ret(heads=4, dim=64, vdim=64, mlp=dense(72)),
-        Lat(heads=4, dim=64, vdim=80, q_rank=40, kv_rank=128, rot_dim=32, window=33, mlp=dense(72))], width=128, taps=2, eps=2e-2,
+        Lat(heads=4, dim=64, vdim=72, q_rank=40, kv_rank=192, rot_dim=32, window=33, mlp=dense(72))], width=128, taps=2, eps=2e-2,
         logit_scale=2.5),
     # no page is ever read
-    "recurrent": syn.sobivik_config([Ret(heads=4, dim=64, vdim=32, mlp=dense()), Ret(heads=1, dim=16, vdim=16)], width=64, taps=5,
+    "recurrent": syn.sobivik_config([Ret(heads=4, dim=64, vdim=24, mlp=dense()), Ret(heads=1, dim=16, vdim=16)], width=64, taps=5,
                                     logit_scale=1.0),
 }
 
